@@ -452,8 +452,131 @@ int b200_argmax_shard_bf16(const void* logits, int64_t ld, uint64_t* keys, int r
 int b200_argmax_merge(const uint64_t* keys, int shards, int rows, int64_t* out, b200_stream_t stream);
 int b200_topk_probs_bf16(const void* logits, int64_t ld, float* probs, int rows, int vocab, int top_k,
                          float temperature, b200_stream_t stream);
+/* b200_argmax_bf16 over fp32 logits. */
+int b200_argmax_f32(const float* logits, int64_t ld, int64_t* out, int rows, int vocab, b200_stream_t stream);
 int b200_topp_probs_bf16(const void* logits, int64_t ld, float* probs, int rows, int vocab, float top_p,
                          float temperature, b200_stream_t stream);
+
+/* ---------------------------------------------------------------------------------------
+ * Hybrid decoders (Zinurax): latent attention, the generalized delta rule, norms on the sublayers' outputs with a
+ * 32-bit residual stream.  `dtype` (B200_DTYPE_*) is the type of weights, activations and cached rows; everything the
+ * kernels do between loading and storing them is 32-bit arithmetic, except the bf16 tensor-core products (fp32 sums).
+ * --------------------------------------------------------------------------------------- */
+#define B200_DTYPE_BF16 0
+#define B200_DTYPE_F32 1
+#define B200_ACT_NONE 0
+#define B200_ACT_RELU2 1 /* max(v, 0)^2 */
+
+/* y[b][M, N] = act(x[b][M, K] * w[b][N, K]^T), `batch` independent products: batch b reads columns
+ * [b * x_batch, b * x_batch + K) of x (row stride ldx), weight rows [b * N, (b + 1) * N), writes y + b * y_batch (row
+ * stride ldy).  bf16 on tcgen05: K, ldx, x_batch multiples of 8, x and w 16-byte aligned; with batch == 1 the workspace of
+ * b200_gemm_bf16_workspace_bytes, none otherwise. */
+int b200_linear_bf16(const void* x, int64_t ldx, const void* w, void* y, int64_t ldy, int M, int N, int K, int act, int batch,
+                     int x_batch, int64_t y_batch, void* workspace, size_t workspace_bytes, b200_stream_t stream);
+/* The same product on the CUDA cores in true fp32, any sizes and strides.  y_f32 != 0: y is fp32 whatever `dtype` is. */
+int b200_linear_simt(const void* x, int64_t ldx, const void* w, void* y, int64_t ldy, int M, int N, int K, int act, int batch,
+                     int x_batch, int64_t y_batch, int dtype, int y_f32, b200_stream_t stream);
+
+/* Layer norm with a weight and no bias, (v - mean) / sqrt(variance + eps) * gamma, of a row v that is
+ *   - the sum over `num_splits` of partials[s][row] (fp32, a linear's split-K partial sums), or
+ *   - table[ids[row]] (`dtype`), or
+ *   - rows[row_index ? row_index[row] : row] (fp32).
+ * With `hidden` the normed row is ADDED to hidden[row] (fp32; `accumulate` == 0: stored) and y = `dtype` of the sum;
+ * without it y is the normed row. */
+typedef struct b200_out_norm_args {
+  const float* partials;
+  const void* table;
+  const int64_t* ids;
+  const float* rows_in;
+  const int64_t* row_index;
+  const void* gamma;
+  float* hidden;
+  void* y; /* may be NULL with hidden */
+  int64_t table_rows;
+  int32_t num_splits;
+  int32_t rows;
+  int32_t source_rows; /* rows of rows_in */
+  int32_t width;
+  int32_t accumulate;
+  int32_t dtype;
+  float eps;
+} b200_out_norm_args;
+int b200_out_norm(const b200_out_norm_args* args, b200_stream_t stream);
+
+/* Latent attention over a paged pool of [chunks][chunk][row_width] rows = (latent c, zeros, rotated key part, zeros):
+ * c at [0, kv_rank), the rotated part at [kv_pad, kv_pad + rot_dim), kv_pad = kv_rank rounded up to 16, row_width a
+ * multiple of 32.  Queries arrive "absorbed": q_full[t][head] holds W_uk^T q_unrotated in the latent's place and the
+ * rotated part in the rotated key's place, so a score is one dot product of row_width and all heads share the rows.
+ *
+ * b200_latent_append: rotates the query part of `proj` into q_full; with dkv_offset >= 0 also norms (RMS, norm_weight) and
+ *   rotates this token's row and stores it at (token_to_chunk_idx, token_to_local_pos).  The rotation turns pairs (2i, 2i+1)
+ *   of the first rot_dims dimensions by the angle whose scaled cos / sin are rope_cos / rope_sin [position][rot_dims / 2].
+ * b200_latent_attention: out[t][head][kv_rank] = sigmoid(gate) * sum_j softmax(scale * q . row_j) c_j over the keys j with
+ *   0 <= position - j < window.  units == NULL: token t is the newest of row t, kv_seq_lengths[t] tokens long (0: padding,
+ *   output undefined).  units: int32 [num_units][4] = {row, first token, tokens <= unit_tokens, 0}. */
+typedef struct b200_latent_args {
+  const void* proj;     /* [T][proj_ld]: q (heads x (dim + rot_dim)) at column 0 */
+  const void* norm_weight;
+  const float* rope_cos;
+  const float* rope_sin;
+  const int64_t* token_to_pos;
+  const int64_t* token_to_chunk_idx;
+  const int64_t* token_to_local_pos;
+  const int32_t* block_table;
+  const int32_t* kv_seq_lengths;
+  const int32_t* units;
+  void* pool;
+  void* q_full; /* [T][heads][row_width] */
+  void* out;    /* [T][heads][kv_rank] */
+  float* workspace;
+  size_t workspace_bytes;
+  int64_t proj_ld;
+  int32_t dkv_offset;  /* column of this layer's down projection, -1: the rows are another layer's */
+  int32_t gate_offset; /* column of the heads' gates, -1: no gate */
+  int32_t num_tokens;
+  int32_t heads, dim, rot_dim, rot_dims, kv_rank, kv_pad, row_width;
+  int32_t num_chunks, chunk_size, max_chunks_per_row, max_positions;
+  int32_t window; /* <= 0: unlimited */
+  int32_t num_units, unit_tokens, num_splits, dtype;
+  float scale, eps;
+} b200_latent_args;
+size_t b200_latent_attention_workspace_bytes(int num_tokens, int heads, int kv_rank, int num_splits);
+int b200_latent_append(const b200_latent_args* args, b200_stream_t stream);
+int b200_latent_attention(const b200_latent_args* args, b200_stream_t stream);
+
+/* Generalized delta rule.  Per head, with w = exp(-decay_scale * sigmoid(z + decay_bias)), a = sigmoid(x_a + removal_bias),
+ * u = k / sqrt(sum k^2 + unit_eps):   S <- diag(w) S - (a u)(u^T S) + k v^T,   o = S^T r,
+ * z = W_w2 tanh(x_w1).  S [row][heads][value channel][key channel] fp32: a step reads slot state_in[row] (-1: zeros) and
+ * writes slot state_out[row] (-1: none), two different slots, so a repeated step gives the same result.
+ * b200_delta_decode: one token per row (token t = row t), everything in one kernel including the head norm, the output gate
+ *   and the product with W_w2.
+ * b200_delta_lora: tanh of the x_w1 columns -> lora [T][rank] for the linear that makes z.
+ * b200_delta_scan: rows of any length; row's tokens are [cu_tokens[row], cu_tokens[row + 1]); writes o_f32 [T][heads * dim].
+ * b200_delta_finish: out = (o / rms(o) over the head) * norm_weight * sigmoid(x_g). */
+typedef struct b200_delta_args {
+  const void* proj; /* [T][proj_ld] */
+  const void* z;    /* [T][heads * dim] (scan) */
+  const void* w2;   /* [heads * dim][rank] (decode) */
+  const void* decay_bias;
+  const void* removal_bias;
+  const void* norm_weight;
+  float* state;
+  const int32_t* state_in;
+  const int32_t* state_out;
+  const int32_t* cu_tokens;
+  float* o_f32;
+  void* lora;
+  void* out; /* [T][heads * dim] */
+  int64_t proj_ld;
+  int64_t state_slots;
+  int32_t off_r, off_k, off_v, off_g, off_a, off_w1;
+  int32_t rank, heads, dim, num_tokens, num_rows, dtype;
+  float decay_scale, unit_eps, eps;
+} b200_delta_args;
+int b200_delta_decode(const b200_delta_args* args, b200_stream_t stream);
+int b200_delta_lora(const b200_delta_args* args, b200_stream_t stream);
+int b200_delta_scan(const b200_delta_args* args, b200_stream_t stream);
+int b200_delta_finish(const b200_delta_args* args, b200_stream_t stream);
 
 #ifdef __cplusplus
 }

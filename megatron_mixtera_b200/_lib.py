@@ -74,6 +74,17 @@ EXPORTED_SYMBOLS = (
     "b200_argmax_merge",
     "b200_topk_probs_bf16",
     "b200_topp_probs_bf16",
+    "b200_argmax_f32",
+    "b200_linear_bf16",
+    "b200_linear_simt",
+    "b200_out_norm",
+    "b200_latent_attention_workspace_bytes",
+    "b200_latent_append",
+    "b200_latent_attention",
+    "b200_delta_decode",
+    "b200_delta_lora",
+    "b200_delta_scan",
+    "b200_delta_finish",
 )
 
 
@@ -117,6 +128,38 @@ class AttentionArgs(ctypes.Structure):
         ("out_q_mode", c_int32),
         ("out_m_pad", c_int32),
     ]
+
+
+class OutNormArgs(ctypes.Structure):
+    """Mirror of ``b200_out_norm_args``."""
+
+    _fields_ = [(n, c_void_p) for n in ("partials", "table", "ids", "rows_in", "row_index", "gamma", "hidden", "y")] + [
+        ("table_rows", c_int64)] + [
+        (n, c_int32) for n in ("num_splits", "rows", "source_rows", "width", "accumulate", "dtype")] + [("eps", c_float)]
+
+
+class LatentArgs(ctypes.Structure):
+    """Mirror of ``b200_latent_args``."""
+
+    _fields_ = [(n, c_void_p) for n in (
+        "proj", "norm_weight", "rope_cos", "rope_sin", "token_to_pos", "token_to_chunk_idx", "token_to_local_pos",
+        "block_table", "kv_seq_lengths", "units", "pool", "q_full", "out", "workspace")] + [
+        ("workspace_bytes", c_size_t), ("proj_ld", c_int64)] + [
+        (n, c_int32) for n in (
+            "dkv_offset", "gate_offset", "num_tokens", "heads", "dim", "rot_dim", "rot_dims", "kv_rank", "kv_pad", "row_width",
+            "num_chunks", "chunk_size", "max_chunks_per_row", "max_positions", "window", "num_units", "unit_tokens",
+            "num_splits", "dtype")] + [("scale", c_float), ("eps", c_float)]
+
+
+class DeltaArgs(ctypes.Structure):
+    """Mirror of ``b200_delta_args``."""
+
+    _fields_ = [(n, c_void_p) for n in (
+        "proj", "z", "w2", "decay_bias", "removal_bias", "norm_weight", "state", "state_in", "state_out", "cu_tokens", "o_f32",
+        "lora", "out")] + [("proj_ld", c_int64), ("state_slots", c_int64)] + [
+        (n, c_int32) for n in (
+            "off_r", "off_k", "off_v", "off_g", "off_a", "off_w1", "rank", "heads", "dim", "num_tokens", "num_rows",
+            "dtype")] + [(n, c_float) for n in ("decay_scale", "unit_eps", "eps")]
 
 
 class TpComm(ctypes.Structure):
@@ -265,6 +308,18 @@ def load() -> ctypes.CDLL:
     lib.b200_argmax_merge.argtypes = [c_void_p, c_int, c_int, c_void_p, c_void_p]
     lib.b200_topk_probs_bf16.argtypes = [c_void_p, c_int64, c_void_p, c_int, c_int, c_int, c_float, c_void_p]
     lib.b200_topp_probs_bf16.argtypes = [c_void_p, c_int64, c_void_p, c_int, c_int, c_float, c_float, c_void_p]
+    lib.b200_argmax_f32.argtypes = [c_void_p, c_int64, c_void_p, c_int, c_int, c_void_p]
+    lib.b200_linear_bf16.argtypes = [c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_int,
+                                     c_int64, c_void_p, c_size_t, c_void_p]
+    lib.b200_linear_simt.argtypes = [c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_int,
+                                     c_int64, c_int, c_int, c_void_p]
+    lib.b200_out_norm.argtypes = [POINTER(OutNormArgs), c_void_p]
+    lib.b200_latent_attention_workspace_bytes.restype = c_size_t
+    lib.b200_latent_attention_workspace_bytes.argtypes = [c_int, c_int, c_int, c_int]
+    for name in ("b200_latent_append", "b200_latent_attention"):
+        getattr(lib, name).argtypes = [POINTER(LatentArgs), c_void_p]
+    for name in ("b200_delta_decode", "b200_delta_lora", "b200_delta_scan", "b200_delta_finish"):
+        getattr(lib, name).argtypes = [POINTER(DeltaArgs), c_void_p]
     for name in EXPORTED_SYMBOLS:
         fn = getattr(lib, name)
         if fn.restype is c_int or name.startswith("b200_") and fn.restype not in (c_char_p, c_size_t):
@@ -299,7 +354,7 @@ def load_torch_ops():
 
 TORCH_OPS = (
     "gather_rows", "add_norm", "activation", "quantize", "gemm", "gemm_splitk", "gemm_bf16_swiglu", "gemm_mxfp8_swiglu",
-    "attention", "argmax", "argmax_shard", "argmax_merge", "filtered_probs", "allreduce_add_norm",
+    "attention", "argmax", "argmax_shard", "argmax_merge", "filtered_probs", "allreduce_add_norm", "linear", "hybrid",
 )
 
 

@@ -50,14 +50,27 @@ struct Params {
   int keep_partials;    // 1: fp32 partial sums are the result (even for one split); a fused consumer reduces them
   int gated;            // 1: rows 0-63 of every 128-row weight tile are gate features, rows 64-127 the matching up
                         //    features; y[M, N/2] = bf16(bf16(silu(gate)) * up) (whole-K units only)
+  int act = B200_ACT_NONE;  // B200_ACT_*: applied to the fp32 product before its one bf16 rounding
+  // Batched form (one product per attention head): batch b multiplies columns [b * x_batch, b * x_batch + K) of x with
+  // weight rows [b * N, (b + 1) * N) into y + b * y_batch.  m_blocks: token blocks per batch (blockIdx.z holds both).
+  int m_blocks = 1, x_batch = 0;
+  int64_t y_batch = 0;
 };
+
+__device__ __forceinline__ float apply_act(float v, int act) {
+  if (act == B200_ACT_RELU2) {
+    v = fmaxf(v, 0.f);
+    v *= v;
+  }
+  return v;
+}
 
 // Sum of the split-K partial tiles: y[m, n] = bf16(sum_s partial[s][m][n]) (+ bias), splits added in order
 // (deterministic).  One thread per four consecutive features; all CTAs of the grid work in parallel, which
 // is what a single "last arriver" CTA cannot offer.
 __global__ void __launch_bounds__(256)
 splitk_reduce_kernel(const float* __restrict__ partials, int splits, int M, int N, const __nv_bfloat16* __restrict__ bias,
-                     __nv_bfloat16* __restrict__ y, int64_t ldy) {
+                     __nv_bfloat16* __restrict__ y, int64_t ldy, int act) {
   pdl_launch_dependents();
   pdl_wait();
   const int64_t split_stride = static_cast<int64_t>(M) * N;
@@ -83,6 +96,10 @@ splitk_reduce_kernel(const float* __restrict__ partials, int splits, int M, int 
       acc.z = bf16_round(acc.z) + __bfloat162float(bias[n + 2]);
       acc.w = bf16_round(acc.w) + __bfloat162float(bias[n + 3]);
     }
+    acc.x = apply_act(acc.x, act);
+    acc.y = apply_act(acc.y, act);
+    acc.z = apply_act(acc.z, act);
+    acc.w = apply_act(acc.w, act);
     __nv_bfloat16* dst = y + static_cast<int64_t>(m) * ldy + n;
     if ((ldy & 3) == 0) {
       *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16x2(acc.x, acc.y), pack_bf16x2(acc.z, acc.w));
@@ -100,7 +117,7 @@ splitk_reduce_kernel(const float* __restrict__ partials, int splits, int M, int 
     float acc = 0.f;
     for (int s = 0; s < splits; ++s) acc += __ldcg(partials + s * split_stride + idx);
     if (bias != nullptr) acc = bf16_round(acc) + __bfloat162float(bias[n]);
-    y[static_cast<int64_t>(m) * ldy + n] = __float2bfloat16_rn(acc);
+    y[static_cast<int64_t>(m) * ldy + n] = __float2bfloat16_rn(apply_act(acc, act));
   }
 }
 
@@ -108,7 +125,7 @@ static int launch_splitk_reduce(const Params& p, cudaStream_t stream) {
   const int64_t work = (p.N & 3) == 0 ? static_cast<int64_t>(p.M) * (p.N >> 2) : static_cast<int64_t>(p.M) * p.N;
   const unsigned blocks = static_cast<unsigned>((work + 255) / 256);
   return launch_pdl(splitk_reduce_kernel, dim3(blocks), dim3(256), 0, stream, static_cast<const float*>(p.partials),
-                    p.num_splits, p.M, p.N, p.bias, p.y, p.ldy);
+                    p.num_splits, p.M, p.N, p.bias, p.y, p.ldy, p.act);
 }
 
 // Barrier over the 128 threads that run the epilogue (warps 0-3 in every GEMM kernel; some kernels have more warps).
@@ -118,7 +135,7 @@ __device__ __forceinline__ void epilogue_barrier() { asm volatile("bar.sync 2, 1
 // stores (whole-K units), or stores the fp32 partial tile for splitk_reduce_kernel.
 template <int BT>
 __device__ __forceinline__ void epilogue(const Params& p, uint32_t tmem_base, uint8_t* stage_smem, int n_tile, int split,
-                                         int m_block) {
+                                         int m_block, __nv_bfloat16* __restrict__ y) {
   const int tid = threadIdx.x;
   const int warp = tid >> 5;
   const int lane = tid & 31;
@@ -160,7 +177,7 @@ __device__ __forceinline__ void epilogue(const Params& p, uint32_t tmem_base, ui
             const float g = is_gate ? mine : other;
             const float u = is_gate ? other : mine;
             const float a = bf16_round(g / (1.f + expf(-g)));
-            p.y[static_cast<int64_t>(m) * p.ldy + out_col] = __float2bfloat16_rn(a * u);
+            y[static_cast<int64_t>(m) * p.ldy + out_col] = __float2bfloat16_rn(a * u);
           }
         }
       }
@@ -168,7 +185,7 @@ __device__ __forceinline__ void epilogue(const Params& p, uint32_t tmem_base, ui
     }
   } else if (p.num_splits == 1 && !p.keep_partials) {
     const float b = (p.bias != nullptr && n_ok) ? __bfloat162float(p.bias[n]) : 0.f;
-    if (n0 + kTileN <= p.N && (p.ldy & 7) == 0 && (reinterpret_cast<uintptr_t>(p.y) & 15) == 0) {
+    if (n0 + kTileN <= p.N && (p.ldy & 7) == 0 && (reinterpret_cast<uintptr_t>(y) & 15) == 0) {
       // Whole tile, 16-byte aligned rows: transpose through shared memory (the pipeline stages are free, every UMMA
       // has completed) so that the tile leaves as 16-byte vectors along the features - one store instruction per 8
       // outputs instead of one per output.
@@ -185,7 +202,7 @@ __device__ __forceinline__ void epilogue(const Params& p, uint32_t tmem_base, ui
           for (int j = 0; j < 32; ++j) {
             float v = __uint_as_float(r[j]);
             if (p.bias != nullptr) v = bf16_round(v) + b;  // bias is added to the bf16-rounded product
-            tile[(c0 + j) * kTileN + warp * 32 + lane] = __float2bfloat16_rn(v);
+            tile[(c0 + j) * kTileN + warp * 32 + lane] = __float2bfloat16_rn(apply_act(v, p.act));
           }
         }
         epilogue_barrier();
@@ -193,7 +210,7 @@ __device__ __forceinline__ void epilogue(const Params& p, uint32_t tmem_base, ui
 #pragma unroll 1
         for (int v = tid; v < kRows * 16; v += kThreads) {
           const int m = m0 + h0 + (v >> 4);
-          if (m < p.M) *reinterpret_cast<uint4*>(p.y + static_cast<int64_t>(m) * p.ldy + n0 + (v & 15) * 8) = tile_v[v];
+          if (m < p.M) *reinterpret_cast<uint4*>(y + static_cast<int64_t>(m) * p.ldy + n0 + (v & 15) * 8) = tile_v[v];
         }
         if (h0 + kRows < BT) epilogue_barrier();
       }
@@ -211,7 +228,7 @@ __device__ __forceinline__ void epilogue(const Params& p, uint32_t tmem_base, ui
               float v = __uint_as_float(r[j]);
               // bias is added to the bf16-rounded product, as `matmul(x, w.t()) + bias` does
               if (p.bias != nullptr) v = bf16_round(v) + b;
-              p.y[static_cast<int64_t>(m) * p.ldy + n] = __float2bfloat16_rn(v);
+              y[static_cast<int64_t>(m) * p.ldy + n] = __float2bfloat16_rn(apply_act(v, p.act));
             }
           }
         }
@@ -279,9 +296,12 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
   const int lane = tid & 31;
   const int n_tile = blockIdx.x;
   const int split = blockIdx.y;
-  const int m_block = blockIdx.z;
+  const int batch = blockIdx.z / p.m_blocks;
+  const int m_block = blockIdx.z - batch * p.m_blocks;
   const int n0 = n_tile * kTileN;
   const int m0 = m_block * BT;
+  const int w_row = batch * p.N + n0;        // first weight row of this tile
+  const int x_col = batch * p.x_batch;       // first activation column of this batch
   const int kb_begin = split * p.k_blocks_per_split;
   const int kb_end = min(p.num_k_blocks, kb_begin + p.k_blocks_per_split);
   const int num_kb = kb_end - kb_begin;
@@ -315,11 +335,11 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
       const int pre = num_kb < C::kStages ? num_kb : C::kStages;
       for (int i = 0; i < pre; ++i) {
         mbar_arrive_expect_tx(&full_bar[i], C::kStageBytes);
-        tma_load_2d(smem + i * C::kStageBytes, &map_w, &full_bar[i], (kb_begin + i) * kTileK, n0);
+        tma_load_2d(smem + i * C::kStageBytes, &map_w, &full_bar[i], (kb_begin + i) * kTileK, w_row);
       }
       pdl_wait();
       for (int i = 0; i < pre; ++i)
-        tma_load_2d(smem + i * C::kStageBytes + C::kStageBytesW, &map_x, &full_bar[i], (kb_begin + i) * kTileK, m0);
+        tma_load_2d(smem + i * C::kStageBytes + C::kStageBytesW, &map_x, &full_bar[i], x_col + (kb_begin + i) * kTileK, m0);
       for (int i = pre; i < num_kb; ++i) {
         const int s = i % C::kStages;
         const uint32_t phase = (i / C::kStages) & 1;
@@ -327,8 +347,8 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
         uint8_t* stage = smem + s * C::kStageBytes;
         mbar_arrive_expect_tx(&full_bar[s], C::kStageBytes);
         const int k0 = (kb_begin + i) * kTileK;
-        tma_load_2d(stage, &map_w, &full_bar[s], k0, n0);
-        tma_load_2d(stage + C::kStageBytesW, &map_x, &full_bar[s], k0, m0);
+        tma_load_2d(stage, &map_w, &full_bar[s], k0, w_row);
+        tma_load_2d(stage + C::kStageBytesW, &map_x, &full_bar[s], x_col + k0, m0);
       }
     }
     __syncwarp();
@@ -362,7 +382,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
   mbar_wait_bounded(accum_bar, 0, abort_flag, kStatusGemmTimeout);
   tcgen05_fence_after_sync();
 
-  epilogue<BT>(p, tmem_base, smem, n_tile, split, m_block);
+  epilogue<BT>(p, tmem_base, smem, n_tile, split, m_block, p.y + batch * p.y_batch);
 
   tcgen05_fence_before_sync();
   __syncthreads();
@@ -403,12 +423,13 @@ template <int BT>
 static int launch(const void* x, int64_t ldx, const void* w, const void* bias, void* y, int64_t ldy, int M, int N,
                   int K, void* workspace, size_t workspace_bytes, cudaStream_t stream, bool cache_maps = true,
                   float* partials_out = nullptr, size_t partials_bytes = 0, int* splits_out = nullptr,
-                  bool gated = false) {
+                  bool gated = false, int act = B200_ACT_NONE, int batch = 1, int x_batch = 0, int64_t y_batch = 0) {
   using C = Config<BT>;
-  const uint64_t wd[2] = {static_cast<uint64_t>(K), static_cast<uint64_t>(N)};
+  const uint64_t wd[2] = {static_cast<uint64_t>(K), static_cast<uint64_t>(N) * batch};
   const uint64_t ws[1] = {static_cast<uint64_t>(K) * 2};
   const uint32_t wb[2] = {kTileK, kTileN};
-  const uint64_t xd[2] = {static_cast<uint64_t>(K), static_cast<uint64_t>(M)};
+  // (batched: a K block that reaches past a batch's columns meets weight columns past K, which TMA fills with zeros)
+  const uint64_t xd[2] = {static_cast<uint64_t>(batch > 1 ? (batch - 1) * x_batch + K : K), static_cast<uint64_t>(M)};
   const uint64_t xs[1] = {static_cast<uint64_t>(ldx) * 2};
   const uint32_t xb[2] = {kTileK, BT};
   CUtensorMap local_w, local_x;  // used when the descriptor cache (a host allocation) must be avoided
@@ -426,7 +447,7 @@ static int launch(const void* x, int64_t ldx, const void* w, const void* bias, v
   const int n_tiles = (N + kTileN - 1) / kTileN;
   const int m_blocks = (M + BT - 1) / BT;
   const int num_kb = (K + kTileK - 1) / kTileK;
-  const int splits = choose_splits(n_tiles * m_blocks, num_kb);
+  const int splits = batch > 1 ? 1 : choose_splits(n_tiles * m_blocks, num_kb);
   Params p;
   p.bias = static_cast<const __nv_bfloat16*>(bias);
   p.y = static_cast<__nv_bfloat16*>(y);
@@ -440,6 +461,11 @@ static int launch(const void* x, int64_t ldx, const void* w, const void* bias, v
   p.partials = nullptr;
   p.keep_partials = partials_out != nullptr;
   p.gated = gated ? 1 : 0;
+  p.act = act;
+  p.m_blocks = m_blocks;
+  p.x_batch = x_batch;
+  p.y_batch = y_batch;
+  if (static_cast<int64_t>(m_blocks) * batch > 65535) return B200_ERR_INVALID_ARGUMENT;
   if (gated && (splits != 1 || partials_out != nullptr)) return B200_ERR_INVALID_ARGUMENT;
   if (partials_out != nullptr) {
     if (partials_bytes < static_cast<size_t>(splits) * M * N * sizeof(float)) return B200_ERR_WORKSPACE;
@@ -452,7 +478,7 @@ static int launch(const void* x, int64_t ldx, const void* w, const void* bias, v
   }
   static std::atomic<uint64_t> smem_attr_done{0};
   if (ensure_dynamic_smem(gemm_bf16_kernel<BT>, C::kSmemBytes, smem_attr_done) != B200_OK) return B200_ERR_LAUNCH;
-  dim3 grid(n_tiles, splits, m_blocks);
+  dim3 grid(n_tiles, splits, m_blocks * batch);
   const int rc = launch_pdl(gemm_bf16_kernel<BT>, grid, dim3(kThreads), C::kSmemBytes, stream, *mw, *mx, p);
   if (rc != B200_OK || splits == 1 || p.keep_partials) return rc;
   return launch_splitk_reduce(p, stream);
@@ -542,6 +568,24 @@ int b200_gemm_bf16(const void* x, int64_t ldx, const void* w, const void* bias, 
     case 64: return gemm::launch<64>(x, ldx, w, bias, y, ldy, M, N, K, workspace, workspace_bytes, s);
     case 128: return gemm::launch<128>(x, ldx, w, bias, y, ldy, M, N, K, workspace, workspace_bytes, s);
     default: return gemm::launch<256>(x, ldx, w, bias, y, ldy, M, N, K, workspace, workspace_bytes, s);
+  }
+}
+
+int b200_linear_bf16(const void* x, int64_t ldx, const void* w, void* y, int64_t ldy, int M, int N, int K, int act, int batch,
+                     int x_batch, int64_t y_batch, void* workspace, size_t workspace_bytes, b200_stream_t stream) {
+  using namespace b200;
+  if (!x || !w || !y || M <= 0 || N <= 0 || K <= 0 || batch <= 0 || act < B200_ACT_NONE || act > B200_ACT_RELU2)
+    return B200_ERR_INVALID_ARGUMENT;
+  if (batch > 1 && (x_batch <= 0 || y_batch <= 0 || (batch - 1) * static_cast<int64_t>(x_batch) + K > ldx))
+    return B200_ERR_INVALID_ARGUMENT;
+  if (K % 8 != 0 || ldx % 8 != 0 || x_batch % 8 != 0 || ldx < K || ldy < N) return B200_ERR_ALIGNMENT;
+  if (!aligned16(x) || !aligned16(w)) return B200_ERR_ALIGNMENT;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  switch (gemm::pick_bt(M)) {
+    case 32: return gemm::launch<32>(x, ldx, w, nullptr, y, ldy, M, N, K, workspace, workspace_bytes, s, true, nullptr, 0, nullptr, false, act, batch, x_batch, y_batch);
+    case 64: return gemm::launch<64>(x, ldx, w, nullptr, y, ldy, M, N, K, workspace, workspace_bytes, s, true, nullptr, 0, nullptr, false, act, batch, x_batch, y_batch);
+    case 128: return gemm::launch<128>(x, ldx, w, nullptr, y, ldy, M, N, K, workspace, workspace_bytes, s, true, nullptr, 0, nullptr, false, act, batch, x_batch, y_batch);
+    default: return gemm::launch<256>(x, ldx, w, nullptr, y, ldy, M, N, K, workspace, workspace_bytes, s, true, nullptr, 0, nullptr, false, act, batch, x_batch, y_batch);
   }
 }
 

@@ -11,17 +11,22 @@ constexpr int kThreads = 1024;
 __device__ __forceinline__ uint32_t bf16_key(uint16_t b) { return (b & 0x8000u) ? (~b & 0xffffu) : (b | 0x8000u); }
 __device__ __forceinline__ float bf16_bits_to_float(uint16_t b) { return __uint_as_float(static_cast<uint32_t>(b) << 16); }
 
-// Greedy: largest value, smallest index among equal values (NaN never wins).
+__device__ __forceinline__ float logit_value(uint16_t b) { return bf16_bits_to_float(b); }
+__device__ __forceinline__ float logit_value(float f) { return f; }
+
+// Greedy: largest value, smallest index among equal values (NaN never wins).  T: bf16 bits or float (which has no
+// vocabulary-shard keys).
+template <typename T>
 __global__ void __launch_bounds__(kThreads)
-argmax_kernel(const uint16_t* __restrict__ logits, int64_t ld, int64_t* __restrict__ out, int vocab,
+argmax_kernel(const T* __restrict__ logits, int64_t ld, int64_t* __restrict__ out, int vocab,
               uint64_t* __restrict__ keys, int64_t index_offset) {
   pdl_launch_dependents();
   pdl_wait();
-  const uint16_t* row = logits + static_cast<int64_t>(blockIdx.x) * ld;
+  const T* row = logits + static_cast<int64_t>(blockIdx.x) * ld;
   float best = -INFINITY;
   int best_i = 0x7fffffff;
   for (int i = threadIdx.x; i < vocab; i += kThreads) {
-    const float v = bf16_bits_to_float(row[i]);
+    const float v = logit_value(row[i]);
     if (v > best || (best_i == 0x7fffffff && v == best)) {  // strided scan visits indices in increasing order
       best = v;
       best_i = i;
@@ -58,7 +63,9 @@ argmax_kernel(const uint16_t* __restrict__ logits, int64_t ld, int64_t* __restri
     }
     if (lane == 0) {
       const int idx = best_i == 0x7fffffff ? 0 : best_i;
-      if (keys == nullptr) {
+      if constexpr (sizeof(T) == 4) {
+        out[blockIdx.x] = idx;
+      } else if (keys == nullptr) {
         out[blockIdx.x] = idx;
       } else {
         // Vocabulary shard: a 64-bit key whose maximum over the shards is the global greedy choice - the value's
@@ -333,9 +340,17 @@ extern "C" {
 int b200_argmax_bf16(const void* logits, int64_t ld, int64_t* out, int rows, int vocab, b200_stream_t stream) {
   using namespace b200;
   if (!logits || !out || rows <= 0 || vocab <= 0 || ld < vocab) return B200_ERR_INVALID_ARGUMENT;
-  return launch_pdl(sampling::argmax_kernel, dim3(rows), dim3(sampling::kThreads), 0,
+  return launch_pdl(sampling::argmax_kernel<uint16_t>, dim3(rows), dim3(sampling::kThreads), 0,
                     reinterpret_cast<cudaStream_t>(stream), static_cast<const uint16_t*>(logits), ld, out, vocab,
                     static_cast<uint64_t*>(nullptr), static_cast<int64_t>(0));
+}
+
+int b200_argmax_f32(const float* logits, int64_t ld, int64_t* out, int rows, int vocab, b200_stream_t stream) {
+  using namespace b200;
+  if (!logits || !out || rows <= 0 || vocab <= 0 || ld < vocab) return B200_ERR_INVALID_ARGUMENT;
+  return launch_pdl(sampling::argmax_kernel<float>, dim3(rows), dim3(sampling::kThreads), 0,
+                    reinterpret_cast<cudaStream_t>(stream), logits, ld, out, vocab, static_cast<uint64_t*>(nullptr),
+                    static_cast<int64_t>(0));
 }
 
 int b200_argmax_shard_bf16(const void* logits, int64_t ld, uint64_t* keys, int rows, int vocab, int64_t index_offset,
@@ -343,7 +358,7 @@ int b200_argmax_shard_bf16(const void* logits, int64_t ld, uint64_t* keys, int r
   using namespace b200;
   if (!logits || !keys || rows <= 0 || vocab <= 0 || ld < vocab || index_offset < 0 || index_offset + vocab > 0xffffffffll)
     return B200_ERR_INVALID_ARGUMENT;
-  return launch_pdl(sampling::argmax_kernel, dim3(rows), dim3(sampling::kThreads), 0,
+  return launch_pdl(sampling::argmax_kernel<uint16_t>, dim3(rows), dim3(sampling::kThreads), 0,
                     reinterpret_cast<cudaStream_t>(stream), static_cast<const uint16_t*>(logits), ld,
                     static_cast<int64_t*>(nullptr), vocab, keys, index_offset);
 }

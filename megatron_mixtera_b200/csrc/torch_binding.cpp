@@ -288,6 +288,63 @@ void attention(const Tensor& args, const Tensor& anchor, int64_t which, const Op
 }
 
 // ---------------------------------------------------------------------------------------------------------------
+// Hybrid decoders.  linear: y = act(x w^T), optionally batched over heads.  hybrid: one of the kernels that take an argument
+// struct (a CPU uint8 tensor of exactly its size, pointing at tensors the caller keeps alive).
+// ---------------------------------------------------------------------------------------------------------------
+void linear(const Tensor& x, int64_t ldx, const Tensor& w, Tensor y, int64_t ldy, int64_t M, int64_t N, int64_t K, int64_t act,
+            int64_t batch, int64_t x_batch, int64_t y_batch, const OptTensor& workspace, bool tensor_cores) {
+  TORCH_CHECK(x.is_cuda() && w.is_cuda() && y.is_cuda(), "b200_decode.linear: CUDA tensors only (no CPU fallback exists)");
+  const bool f32 = x.scalar_type() == F32;
+  need(w, f32 ? F32 : BF16, "w");
+  TORCH_CHECK(x.scalar_type() == (f32 ? F32 : BF16), "b200_decode.linear: x must be bf16 or fp32");
+  const bool y_f32 = y.scalar_type() == F32;
+  TORCH_CHECK(y_f32 || (!f32 && y.scalar_type() == BF16), "b200_decode.linear: y must be fp32 or the type of x");
+  need_opt(workspace, U8, "workspace");
+  TORCH_CHECK(M > 0 && N > 0 && K > 0 && batch > 0 && w.numel() >= batch * N * K, "b200_decode.linear: w is too small");
+  // extents inside the storages (x may be a column range of a wider matrix)
+  auto room = [](const Tensor& t) { return static_cast<int64_t>(t.storage().nbytes() / t.element_size()) - t.storage_offset(); };
+  TORCH_CHECK((M - 1) * ldx + (batch - 1) * x_batch + K <= room(x), "b200_decode.linear: x is too small");
+  TORCH_CHECK((M - 1) * ldy + (batch - 1) * y_batch + N <= room(y), "b200_decode.linear: y is too small");
+  c10::cuda::CUDAGuard guard(x.device());
+  auto s = stream_of(x);
+  const int m = static_cast<int>(M), n = static_cast<int>(N), k = static_cast<int>(K);
+  if (tensor_cores) {
+    TORCH_CHECK(!f32 && !y_f32, "b200_decode.linear: the tensor-core path is bf16");
+    ok(b200_linear_bf16(ptr(x), ldx, ptr(w), ptr(y), ldy, m, n, k, static_cast<int>(act), static_cast<int>(batch),
+                        static_cast<int>(x_batch), y_batch, ptr(workspace),
+                        workspace.has_value() ? static_cast<size_t>(workspace->numel()) : 0, s),
+       "b200_linear_bf16");
+  } else {
+    ok(b200_linear_simt(ptr(x), ldx, ptr(w), ptr(y), ldy, m, n, k, static_cast<int>(act), static_cast<int>(batch),
+                        static_cast<int>(x_batch), y_batch, f32 ? B200_DTYPE_F32 : B200_DTYPE_BF16, y_f32 ? 1 : 0, s),
+       "b200_linear_simt");
+  }
+}
+
+template <typename A>
+const A* struct_of(const Tensor& args, const char* name) {
+  TORCH_CHECK(args.numel() == static_cast<int64_t>(sizeof(A)), "b200_decode.hybrid: args must hold one ", name, " of ", sizeof(A),
+              " bytes");
+  return static_cast<const A*>(args.data_ptr());
+}
+void hybrid(const Tensor& args, const Tensor& anchor, int64_t which) {
+  TORCH_CHECK(args.is_cpu() && args.scalar_type() == U8 && args.is_contiguous(), "b200_decode.hybrid: args must be a CPU uint8 tensor");
+  TORCH_CHECK(anchor.is_cuda(), "b200_decode.hybrid: anchor must be a CUDA tensor (no CPU fallback exists)");
+  c10::cuda::CUDAGuard guard(anchor.device());
+  auto s = stream_of(anchor);
+  switch (which) {
+    case 0: ok(b200_out_norm(struct_of<b200_out_norm_args>(args, "b200_out_norm_args"), s), "b200_out_norm"); break;
+    case 1: ok(b200_latent_append(struct_of<b200_latent_args>(args, "b200_latent_args"), s), "b200_latent_append"); break;
+    case 2: ok(b200_latent_attention(struct_of<b200_latent_args>(args, "b200_latent_args"), s), "b200_latent_attention"); break;
+    case 3: ok(b200_delta_decode(struct_of<b200_delta_args>(args, "b200_delta_args"), s), "b200_delta_decode"); break;
+    case 4: ok(b200_delta_lora(struct_of<b200_delta_args>(args, "b200_delta_args"), s), "b200_delta_lora"); break;
+    case 5: ok(b200_delta_scan(struct_of<b200_delta_args>(args, "b200_delta_args"), s), "b200_delta_scan"); break;
+    case 6: ok(b200_delta_finish(struct_of<b200_delta_args>(args, "b200_delta_args"), s), "b200_delta_finish"); break;
+    default: TORCH_CHECK(false, "b200_decode.hybrid: unknown kernel ", which);
+  }
+}
+
+// ---------------------------------------------------------------------------------------------------------------
 // Sampling
 // ---------------------------------------------------------------------------------------------------------------
 inline void need_logits(const Tensor& logits) {
@@ -295,6 +352,16 @@ inline void need_logits(const Tensor& logits) {
               "b200_decode: logits must be a 2-D bf16 CUDA tensor with unit inner stride");
 }
 void argmax(const Tensor& logits, Tensor out) {
+  if (logits.is_cuda() && logits.scalar_type() == F32) {
+    TORCH_CHECK(logits.dim() == 2 && logits.stride(1) == 1, "b200_decode: logits must be 2-D with unit inner stride");
+    need(out, I64, "out");
+    TORCH_CHECK(out.numel() >= logits.size(0), "b200_decode.argmax: out is too small");
+    c10::cuda::CUDAGuard guard(logits.device());
+    ok(b200_argmax_f32(static_cast<const float*>(ptr(logits)), logits.stride(0), static_cast<int64_t*>(ptr(out)),
+                       static_cast<int>(logits.size(0)), static_cast<int>(logits.size(1)), stream_of(logits)),
+       "b200_argmax_f32");
+    return;
+  }
   need_logits(logits);
   need(out, I64, "out");
   TORCH_CHECK(out.numel() >= logits.size(0), "b200_decode.argmax: out is too small");
@@ -410,6 +477,9 @@ TORCH_LIBRARY(b200_decode, m) {
   m.def("gemm_mxfp8_swiglu(Tensor xq, Tensor x_sf, Tensor wq, Tensor w_sf, Tensor(a!)? q_out, Tensor(b!)? sf_out, "
         "Tensor(c!)? y_out, int M, int F, int K) -> ()");
   m.def("attention(Tensor args, Tensor(a!) anchor, int which, Tensor? units, int num_units) -> ()");
+  m.def("linear(Tensor x, int ldx, Tensor w, Tensor(a!) y, int ldy, int M, int N, int K, int act, int batch, int x_batch, "
+        "int y_batch, Tensor? workspace, bool tensor_cores) -> ()");
+  m.def("hybrid(Tensor args, Tensor(a!) anchor, int which) -> ()");
   m.def("argmax(Tensor logits, Tensor(a!) out) -> ()");
   m.def("argmax_shard(Tensor logits, Tensor(a!) keys, int index_offset) -> ()");
   m.def("argmax_merge(Tensor keys, int shards, int rows, Tensor(a!) out) -> ()");
@@ -429,6 +499,8 @@ TORCH_LIBRARY_IMPL(b200_decode, CUDA, m) {
   m.impl("gemm_bf16_swiglu", &gemm_bf16_swiglu);
   m.impl("gemm_mxfp8_swiglu", &gemm_mxfp8_swiglu);
   m.impl("attention", &attention);
+  m.impl("linear", &linear);
+  m.impl("hybrid", &hybrid);
   m.impl("argmax", &argmax);
   m.impl("argmax_shard", &argmax_shard);
   m.impl("argmax_merge", &argmax_merge);

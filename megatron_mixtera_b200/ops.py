@@ -17,6 +17,7 @@ from . import _lib
 from ._lib import AttentionArgs, B200Error  # noqa: F401  (re-exported)
 
 BF16 = torch.bfloat16
+F32 = torch.float32
 
 
 def _stream() -> int:
@@ -672,8 +673,8 @@ def prefill_q_block(num_q_heads: int, num_kv_heads: int) -> int:
 
 
 def argmax(logits):
-    """Greedy token per row of bf16 logits [rows, vocab] -> int64 [rows]."""
-    _need(logits, BF16, "logits")
+    """Greedy token per row of bf16 (or fp32) logits [rows, vocab] -> int64 [rows]."""
+    _need(logits, F32 if logits.dtype == F32 else BF16, "logits")
     rows, vocab = logits.shape
     out = torch.empty((rows,), dtype=torch.int64, device=logits.device)
     _launch("argmax", logits, out)
@@ -701,7 +702,8 @@ def argmax_merge(keys):
 
 
 def topk_probs(logits, top_k: int, temperature: float = 1.0):
-    """fp32 probabilities after temperature and top-k filtering, [rows, vocab]."""
+    """fp32 probabilities after temperature and top-k filtering, [rows, vocab] (fp32 logits are rounded to bf16)."""
+    logits = logits.to(BF16) if logits.dtype == F32 else logits
     _need(logits, BF16, "logits")
     rows, vocab = logits.shape
     probs = torch.empty((rows, vocab), dtype=torch.float32, device=logits.device)
@@ -712,9 +714,135 @@ def topk_probs(logits, top_k: int, temperature: float = 1.0):
 
 
 def topp_probs(logits, top_p: float, temperature: float = 1.0):
-    """fp32 probabilities after temperature and top-p (nucleus) filtering, [rows, vocab]."""
+    """fp32 probabilities after temperature and top-p (nucleus) filtering, [rows, vocab] (fp32 logits are rounded to bf16)."""
+    logits = logits.to(BF16) if logits.dtype == F32 else logits
     _need(logits, BF16, "logits")
     rows, vocab = logits.shape
     probs = torch.empty((rows, vocab), dtype=torch.float32, device=logits.device)
     _launch("filtered_probs", logits, probs, 0, float(top_p), float(temperature))
     return probs
+
+
+# ---------------------------------------------------------------------------------------------------------------------
+# Hybrid decoders: latent attention, the generalized delta rule, norms on sublayer outputs with a 32-bit residual stream.
+# Tensors are bf16 or - the whole model in true 32-bit arithmetic - fp32.
+# ---------------------------------------------------------------------------------------------------------------------
+_DTYPE = {BF16: 0, F32: 1}
+_ACT = {None: 0, "relu2": 1}
+_OUT_NORM, _LATENT_APPEND, _LATENT_ATTENTION, _DELTA_DECODE, _DELTA_LORA, _DELTA_SCAN, _DELTA_FINISH = range(7)
+
+
+def dtype_code(dtype) -> int:
+    if dtype not in _DTYPE:
+        raise B200Error("dtype", -1, f"expected bfloat16 or float32, got {dtype}")
+    return _DTYPE[dtype]
+
+
+def linear(x, w, *, act: Optional[str] = None, out=None, batch: int = 1, x_batch: int = 0, y_batch: int = 0, K: Optional[int] = None,
+           out_dtype=None):
+    """``act(x @ w.T)`` for x [rows, ...] (unit inner stride, possibly the first columns of a wider matrix) and w [N, K].
+
+    ``batch`` > 1: one product per head: head b multiplies x columns [b * x_batch, b * x_batch + K) with w rows [b * N, ...)
+    into out columns b * y_batch (``out`` [rows, ...] given by the caller).  bf16 runs on the tensor cores where TMA can
+    address the rows (K and strides multiples of 8), everything else - fp32, odd sizes, fp32 output - on the CUDA cores."""
+    _need(w, x.dtype, "w")
+    if not x.is_cuda or x.stride(-1) != 1 or x.dim() != 2:
+        raise B200Error("linear", -1, "x must be a 2-D CUDA tensor with unit inner stride")
+    K = w.shape[1] if K is None else K
+    if w.shape[1] != K or w.shape[0] % batch or (batch == 1 and x.shape[1] != K):
+        raise B200Error("linear", -1, f"shape mismatch x{tuple(x.shape)} vs w{tuple(w.shape)}, batch {batch}, K {K}")
+    M, N, ldx = x.shape[0], w.shape[0] // batch, x.stride(0)
+    if out is None:
+        out = torch.empty((M, N), dtype=x.dtype if out_dtype is None else out_dtype, device=x.device)
+    tc = (x.dtype == BF16 and out.dtype == BF16 and K % 8 == 0 and ldx % 8 == 0 and x_batch % 8 == 0
+          and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
+    ws = None
+    if tc and batch == 1:
+        ws = _gemm_workspace(x.device, _lib.load().b200_gemm_bf16_workspace_bytes(M, N, K), True)
+    _launch("linear", x, ldx, w, out, out.stride(0), M, N, K, _ACT[act], batch, x_batch, y_batch, ws, tc)
+    return out
+
+
+def linear_partials(x, w) -> GemmPartials:
+    """``x @ w.T`` as fp32 partial sums for `out_norm`: split along K on the tensor cores, one "split" on the CUDA cores."""
+    M, (N, K) = x.shape[0], w.shape
+    if x.dtype == BF16 and x.is_contiguous() and K % 8 == 0 and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0:
+        return gemm_splitk(x, w)
+    ws = _gemm_workspace(x.device, 4 * M * N)
+    linear(x, w, out=ws[: 4 * M * N].view(F32).view(M, N))
+    return GemmPartials(ws, 1, (M, N))
+
+
+def out_norm(source, gamma, *, eps: float, hidden=None, accumulate: bool = False, want_y: bool = True, ids=None, row_index=None):
+    """Layer norm (weight only) of ``source``'s rows; see ``b200_out_norm_args``.
+
+    ``source``: `GemmPartials`, an embedding table with ``ids`` (int64), or fp32 rows, picked by ``row_index`` (int64) if
+    given.  With ``hidden`` (fp32 [rows, width]) the normed rows are stored into it or, ``accumulate``, added to it.
+    Returns the result in ``gamma``'s type (None without ``want_y``; ``hidden`` itself when that is fp32 already)."""
+    a = _lib.OutNormArgs()
+    if isinstance(source, GemmPartials):
+        if source.epoch != _gemm_epoch:
+            raise B200Error("out_norm", -1, "another GEMM has reused the workspace that held these partial sums")
+        rows, width = source.shape
+        a.partials, a.num_splits, dev = source.buf.data_ptr(), source.num_splits, source.device
+    elif ids is not None:
+        _need(source, gamma.dtype, "table")
+        _need(ids, torch.int64, "ids")
+        rows, width, dev = ids.numel(), source.shape[1], source.device
+        a.table, a.ids, a.table_rows = source.data_ptr(), ids.data_ptr(), source.shape[0]
+    else:
+        _need(source, F32, "rows")
+        rows, width, dev = source.shape[0] if row_index is None else row_index.numel(), source.shape[1], source.device
+        a.rows_in, a.source_rows = source.data_ptr(), source.shape[0]
+        if row_index is not None:
+            _need(row_index, torch.int64, "row_index")
+            a.row_index = row_index.data_ptr()
+    _need(gamma, gamma.dtype, "gamma")
+    if gamma.numel() != width:
+        raise B200Error("out_norm", -1, f"gamma has {gamma.numel()} entries, rows {width}")
+    y = None
+    if hidden is not None:
+        _need(hidden, F32, "hidden")
+        if tuple(hidden.shape) != (rows, width):
+            raise B200Error("out_norm", -1, f"hidden {tuple(hidden.shape)} vs rows {(rows, width)}")
+        a.hidden = hidden.data_ptr()
+        if gamma.dtype == F32:
+            y, want_y = hidden, False
+    if want_y:
+        y = torch.empty((rows, width), dtype=gamma.dtype, device=dev)
+        a.y = y.data_ptr()
+    a.gamma, a.rows, a.width, a.accumulate = gamma.data_ptr(), rows, width, int(accumulate)
+    a.dtype, a.eps = dtype_code(gamma.dtype), eps
+    _launch("hybrid", _blob(a), gamma, _OUT_NORM)
+    return y
+
+
+def latent_append(args, anchor) -> None:
+    _launch("hybrid", _blob(args), anchor, _LATENT_APPEND)
+
+
+def latent_attention(args, anchor) -> None:
+    """``args``: `_lib.LatentArgs` (raw pointers: the caller keeps the tensors alive); the split workspace is added here."""
+    global launch_count
+    nbytes = _lib.load().b200_latent_attention_workspace_bytes(args.num_tokens, args.heads, args.kv_rank, args.num_splits)
+    if nbytes:
+        ws = _workspace.get(anchor.device, "latent", nbytes)
+        args.workspace, args.workspace_bytes = ws.data_ptr(), ws.numel()
+        launch_count += 1  # the split-combine kernel
+    _launch("hybrid", _blob(args), anchor, _LATENT_ATTENTION)
+
+
+def delta_decode(args, anchor) -> None:
+    _launch("hybrid", _blob(args), anchor, _DELTA_DECODE)
+
+
+def delta_lora(args, anchor) -> None:
+    _launch("hybrid", _blob(args), anchor, _DELTA_LORA)
+
+
+def delta_scan(args, anchor) -> None:
+    _launch("hybrid", _blob(args), anchor, _DELTA_SCAN)
+
+
+def delta_finish(args, anchor) -> None:
+    _launch("hybrid", _blob(args), anchor, _DELTA_FINISH)

@@ -57,7 +57,30 @@ class LanguageModelEmbedding(torch.nn.Module):
         return self.word_embeddings(input_ids)
 
 
-class GPTModel(torch.nn.Module):
+class DynamicForward:
+    """The reference's ``forward`` signature over a model's ``forward_rows``."""
+
+    def forward(self, input_ids, position_ids, attention_mask=None, decoder_input=None, labels=None,
+                inference_context=None, runtime_gather_output: Optional[bool] = None, **_):
+        """``input_ids`` / ``position_ids`` ``[1, T]`` of the context's padded step.  Returns
+        ``[1, active requests, vocab]`` when the context materialises last-token logits only, else
+        ``[1, T, vocab]``."""
+        ctx = inference_context
+        if ctx is None or labels is not None:
+            raise NotImplementedError("only inference with a dynamic context is implemented")
+        if ctx.materialize_only_last_token_logits:
+            n_req = ctx.total_request_count - ctx.paused_request_count
+            if ctx.is_decode_only():
+                logits = self.forward_rows(input_ids, position_ids, ctx, None, runtime_gather_output)[:n_req]
+            else:
+                idx = torch.from_numpy(ctx.last_token_indices()).to(input_ids.device)
+                logits = self.forward_rows(input_ids, position_ids, ctx, idx, runtime_gather_output)
+        else:
+            logits = self.forward_rows(input_ids, position_ids, ctx, None, runtime_gather_output)
+        return logits.unsqueeze(0)
+
+
+class GPTModel(DynamicForward, torch.nn.Module):
     def __init__(self, config: TransformerConfig, transformer_layer_spec=None, vocab_size: int = None,
                  max_sequence_length: int = None, pre_process: bool = True, post_process: bool = True,
                  parallel_output: bool = True, share_embeddings_and_output_weights: bool = False,
@@ -98,25 +121,6 @@ class GPTModel(torch.nn.Module):
         weight = self.embedding.word_embeddings.weight if self.share_embeddings_and_output_weights else None
         logits, _ = self.output_layer(hidden, weight=weight, runtime_gather_output=runtime_gather_output)
         return logits
-
-    def forward(self, input_ids, position_ids, attention_mask=None, decoder_input=None, labels=None,
-                inference_context=None, runtime_gather_output: Optional[bool] = None, **_):
-        """``input_ids`` / ``position_ids`` ``[1, T]`` of the context's padded step.  Returns
-        ``[1, active requests, vocab]`` when the context materialises last-token logits only, else
-        ``[1, T, vocab]``."""
-        ctx = inference_context
-        if ctx is None or labels is not None:
-            raise NotImplementedError("only inference with a dynamic context is implemented")
-        if ctx.materialize_only_last_token_logits:
-            n_req = ctx.total_request_count - ctx.paused_request_count
-            if ctx.is_decode_only():
-                logits = self.forward_rows(input_ids, position_ids, ctx, None, runtime_gather_output)[:n_req]
-            else:
-                idx = torch.from_numpy(ctx.last_token_indices()).to(input_ids.device)
-                logits = self.forward_rows(input_ids, position_ids, ctx, idx, runtime_gather_output)
-        else:
-            logits = self.forward_rows(input_ids, position_ids, ctx, None, runtime_gather_output)
-        return logits.unsqueeze(0)
 
     # ------------------------------------------------------------------------------------------
     def full_parameter_shapes(self) -> Dict[str, tuple]:

@@ -12,13 +12,24 @@ with a few vectorised numpy operations, and only what the kernels consume is mir
 with asynchronous copies from pinned staging buffers: the ``token_to_*`` arrays, ``kv_seq_lengths``,
 the block table and, for prefill steps, per-token block-table rows and KV lengths.  One step costs
 one device->host read (the sampled tokens) and a handful of host->device copies.
+
+Two kinds of per-request memory exist besides the key / value pool, for decoders whose layers are not plain attention:
+
+* latent rows (``cache_mla_latent``): one row per token and caching layer, of a width that may differ between layers, in the
+  same chunks and block tables as keys and values would be;
+* recurrent state (``state_shapes``): a fixed-size fp32 block per request and recurrent layer in a slot of its own.  Every slot
+  is a pair of buffers: a step reads one and writes the other, and completing the step swaps them.  A forward that is run
+  again - under CUDA-graph capture, or because the one enqueued early was not used - therefore gives the same result.
+
+`schedule_tokens` / `complete_step` drive the context with given tokens instead of sampled ones: any portion of any live
+request per step, the others sitting out.
 """
 from __future__ import annotations
 
 import math
 import warnings
 from enum import Enum
-from typing import List, Optional, Tuple
+from typing import List, Optional, Sequence, Tuple
 
 import numpy as np
 import torch
@@ -134,6 +145,8 @@ class DynamicInferenceContext(BaseInferenceContext):
         kv_cache_dtype: Optional[torch.dtype] = None,
         kv_fp8_single_term: bool = False,
         debug_validate: bool = False,
+        latent_row_widths: Optional[Sequence[int]] = None,
+        state_shapes: Optional[Sequence[Optional[Tuple[int, ...]]]] = None,
     ):
         """``num_attention_heads`` is the number of KV heads (query groups), as in the reference.
 
@@ -143,17 +156,24 @@ class DynamicInferenceContext(BaseInferenceContext):
         extension; the reference's pool is always ``params_dtype``) stores keys and values as E4M3 bytes with
         one fp32 scale per layer and KV head (``kv_scales [L, 2, heads]``, 1.0 until the caller sets them),
         halving the bytes the attention kernel streams.
+
+        ``cache_mla_latent``: the pool holds one latent row per token instead of keys and values; ``latent_row_widths`` gives
+        the row width of every layer (0: the layer caches nothing), or ``kv_lora_rank + qk_pos_emb_head_dim`` that of all.
+        ``state_shapes``: per layer the shape of its fp32 recurrent state per request, None for layers without one.
         """
         super().__init__(materialize_only_last_token_logits=materialize_only_last_token_logits)
         # Debug mode: every `initialize_attention_state` checks on the host what the kernels are about to index with
         # (`validate_attention_state`): the stand-in for a memory checker on machines where none can be run.
         self.debug_validate = bool(debug_validate)
-        if cache_mla_latent:
-            raise NotImplementedError("multi-latent attention caches are outside this decode path")
+        if cache_mla_latent and latent_row_widths is None:
+            if kv_lora_rank is None or qk_pos_emb_head_dim is None:
+                raise ValueError("cache_mla_latent needs latent_row_widths, or kv_lora_rank and qk_pos_emb_head_dim")
+            latent_row_widths = [kv_lora_rank + qk_pos_emb_head_dim] * num_layers
         if device is None:
             device = torch.device("cuda", torch.cuda.current_device()) if torch.cuda.is_available() else "cpu"
         self.device = torch.device(device)
-        self.cache_mla_latent = False
+        self.cache_mla_latent = bool(cache_mla_latent)
+        self.latent_row_widths = list(latent_row_widths) if cache_mla_latent else None
 
         tp_size = (
             parallel_state.get_tensor_model_parallel_world_size()
@@ -178,6 +198,10 @@ class DynamicInferenceContext(BaseInferenceContext):
         self.chunk_size_bytes = (
             self.kv_cache_dtype.itemsize * 2 * num_layers * chunk_size_tokens * heads_per_partition * kv_channels
         )
+        if self.cache_mla_latent:
+            if len(self.latent_row_widths) != num_layers or self.kv_cache_fp8:
+                raise ValueError("latent_row_widths must name every layer; latent rows have no FP8 form")
+            self.chunk_size_bytes = self.latent_chunk_bytes(self.latent_row_widths, chunk_size_tokens, self.kv_cache_dtype)
         buffer_size_bytes = int(buffer_size_gb * 1024**3)
         buffer_size_bytes -= buffer_size_bytes % self.chunk_size_bytes
         chunk_count_total = buffer_size_bytes // self.chunk_size_bytes
@@ -242,7 +266,12 @@ class DynamicInferenceContext(BaseInferenceContext):
         # ---- KV pool ----
         self.memory_buffer = None
         self.kv_scales = None
-        if allocate_memory_buffer:
+        self.latent_buffers = None
+        if allocate_memory_buffer and self.cache_mla_latent:
+            self.latent_buffers = [
+                torch.zeros((chunk_count_total, chunk_size_tokens, w), dtype=self.kv_cache_dtype, device=self.device) if w else None
+                for w in self.latent_row_widths]
+        elif allocate_memory_buffer:
             shape = (2, num_layers, chunk_count_total, chunk_size_tokens, heads_per_partition, kv_channels)
             if self.kv_cache_fp8:
                 if chunk_size_tokens % 128 != 0 or kv_channels != 128:
@@ -253,6 +282,25 @@ class DynamicInferenceContext(BaseInferenceContext):
                 self.kv_scales = torch.ones((num_layers, 2, heads_per_partition), dtype=torch.float32, device=self.device)
             else:
                 self.memory_buffer = torch.full(shape, -1, dtype=params_dtype, device=self.device)
+
+        # ---- recurrent state: a pair of buffers per slot, a slot per request ----
+        self.state_shapes = list(state_shapes) if state_shapes is not None and any(sh is not None for sh in state_shapes) else None
+        self.state_buffers = None
+        if self.state_shapes is not None:
+            if len(self.state_shapes) != num_layers:
+                raise ValueError("state_shapes must name every layer")
+            self.num_state_slots = R
+            self.request_state_slots = torch.full((R,), -1, dtype=torch.int32)
+            self.request_state_side = torch.zeros((R,), dtype=torch.int32)  # which buffer of the pair holds the state
+            self._free_state_slots = list(range(R))
+            self._h_slots = torch.full((2, R + 1), -1, dtype=torch.int32, pin_memory=pin)
+            self._h_slots_np = self._h_slots.numpy()
+            self._d_slots = torch.full((2, R + 1), -1, dtype=torch.int32, device=self.device)
+            self.state_read_slots, self.state_write_slots = self._d_slots[0], self._d_slots[1]
+            if allocate_memory_buffer:
+                self.state_buffers = [
+                    torch.zeros((2 * R, *sh), dtype=torch.float32, device=self.device) if sh is not None else None
+                    for sh in self.state_shapes]
 
         # ---- CUDA-graph token counts (reference :319-356) ----
         self.cuda_graph_token_counts = None
@@ -402,7 +450,48 @@ class DynamicInferenceContext(BaseInferenceContext):
     def get_active_request_count(self) -> int:
         return int(torch.less(self.get_active_sequence_lengths(), self.get_max_sequence_lengths()).sum())
 
+    @staticmethod
+    def latent_chunk_bytes(row_widths: Sequence[int], chunk_size_tokens: int, dtype: torch.dtype) -> int:
+        """Bytes of one chunk over all caching layers (a model that caches nothing still counts tokens in chunks)."""
+        return dtype.itemsize * chunk_size_tokens * max(1, sum(row_widths))
+
+    # ------------------------------------------------------------------ recurrent state
+    def _take_state_slot(self, row: int) -> None:
+        if self.state_shapes is not None:
+            self.request_state_slots[row] = self._free_state_slots.pop()
+            self.request_state_side[row] = 0
+
+    def _release_state_slots(self, rows) -> None:
+        if self.state_shapes is not None:
+            slots = self.request_state_slots.numpy()
+            for r in np.asarray(rows).tolist():
+                self._free_state_slots.append(int(slots[r]))
+                slots[r] = -1
+
+    def _swap_state_sides(self, lo: int, hi: int) -> None:
+        if self.state_shapes is not None:
+            self.request_state_side.numpy()[lo:hi] ^= 1
+
+    def _publish_state_slots(self, p: int, t: int, n_rows: int) -> None:
+        """Buffer every row of the step reads (-1: the request starts, its state is zero) and writes (-1: padding row)."""
+        n = t - p
+        h = self._h_slots_np
+        h[:, : n_rows + 1] = -1
+        slot, side = self.request_state_slots.numpy()[p:t], self.request_state_side.numpy()[p:t]
+        ok = slot >= 0
+        h[0, :n] = np.where(ok & (self.request_kv_length_offsets.numpy()[p:t] > 0), side * self.num_state_slots + slot, -1)
+        h[1, :n] = np.where(ok, (1 - side) * self.num_state_slots + slot, -1)
+        self._push_rows(self._d_slots, self._h_slots, 2, 0, max(n_rows, 1))
+
+    def recurrent_state(self, layer_number: int) -> Tensor:
+        """fp32 state buffers ``[2 * slots, ...]`` of 1-based ``layer_number``."""
+        return self.state_buffers[layer_number - 1]
+
     # ------------------------------------------------------------------ KV pool access
+    def latent_cache(self, layer_number: int) -> Tensor:
+        """Latent rows ``[chunks, chunk, width]`` of 1-based ``layer_number``."""
+        return self.latent_buffers[layer_number - 1]
+
     def key_value_cache(self, layer_number: int) -> Tuple[Tensor, Tensor, Tensor]:
         """(K pool, V pool, block table) of 1-based ``layer_number`` (reference :547-564)."""
         return (self.memory_buffer[0, layer_number - 1], self.memory_buffer[1, layer_number - 1], self.block_table)
@@ -564,6 +653,8 @@ class DynamicInferenceContext(BaseInferenceContext):
             lens[_LEN_ORDER, : n_rows + 1] = np.arange(n_rows + 1)
             self._push_rows(self._d_len, self._h_len, 5, 0, n_rows + 1)         # ... and the cumulative lengths
         self.kv_seq_lengths = self.kv_seq_lengths_cudagraph_only[:n_rows]
+        if self.state_shapes is not None:
+            self._publish_state_slots(p, t, n_rows)
 
         state = (self._bt_version, p, t, n_rows)
         if state != self._bt_pushed or num_warmup_tokens is not None:  # unchanged since the last step: already there
@@ -621,6 +712,13 @@ class DynamicInferenceContext(BaseInferenceContext):
             raise AttentionStateError("a padding token does not point at the dummy chunk")
         if (ci[:a] == self.dummy_chunk_idx).any():
             raise AttentionStateError("an active token points at the dummy chunk")
+        if self.state_shapes is not None:
+            rd, wr = self._h_slots_np[0, :n_rows], self._h_slots_np[1, :n_rows]
+            if (rd >= 2 * self.num_state_slots).any() or (wr >= 2 * self.num_state_slots).any():
+                raise AttentionStateError("a state slot lies outside the state buffers")
+            used = wr[:n_req]
+            if np.unique(used).size != n_req or np.intersect1d(used, rd[rd >= 0]).size:
+                raise AttentionStateError("a state buffer is written twice, or read and written, in one step")
 
     def reset(self) -> None:
         """Drop every request and return all chunks (reference :827-869)."""
@@ -646,6 +744,10 @@ class DynamicInferenceContext(BaseInferenceContext):
         self._mark_copies()
         self.reset_attention_state()
         self.chunk_allocator.reset()
+        if self.state_shapes is not None:
+            self.request_state_slots.fill_(-1)
+            self.request_state_side.fill_(0)
+            self._free_state_slots = list(range(self.num_state_slots))
         self._bt_version += 1
 
     def current_input_and_position_ids(self, *, num_warmup_tokens: Optional[int] = None) -> Tuple[Tensor, Tensor]:
@@ -705,6 +807,7 @@ class DynamicInferenceContext(BaseInferenceContext):
         self.request_kv_chunk_counts[r] = num_chunks_needed
         self.request_last_kv_chunk_id[r] = new_chunk_ids[-1]
         self.request_last_kv_chunk_offset[r] = (context_length - 1) % self.chunk_size_tokens
+        self._take_state_slot(r)
 
         self._wait_copies()
         a, b = self.active_token_count, self.active_token_count + context_length
@@ -726,19 +829,120 @@ class DynamicInferenceContext(BaseInferenceContext):
         self.total_request_count += 1
         self.active_token_count += context_length
 
+    # ------------------------------------------------------------------ steps of given tokens
+    def schedule_tokens(self, entries) -> None:
+        """Make the coming step run exactly ``entries`` = [(request id, tokens)]: the next tokens of each named request, a
+        portion of a prompt or a single token alike.  An unknown id is admitted; live requests that are not named sit the
+        step out (they take the place of paused requests in the row order).  Raises an overflow error, with nothing changed,
+        if the step does not fit.  Not to be mixed with `add_request` / `update_requests` while requests are live."""
+        if self.active_token_count or self.paused_request_count != self.total_request_count:
+            raise RuntimeError("the previous step has not been completed")
+        entries = [(rid, np.asarray(toks, dtype=np.int64).reshape(-1)) for rid, toks in entries]
+        ids = [rid for rid, _ in entries]
+        if len(set(ids)) != len(ids) or any(t.size == 0 for _, t in entries):
+            raise ValueError("every entry needs tokens, and a request one entry")
+        total = self.total_request_count
+        row_of = {int(r): i for i, r in enumerate(self.request_ids[:total].tolist())}
+        offs, counts = self.request_kv_length_offsets.numpy(), self.request_kv_chunk_counts.numpy()
+        n_tokens = sum(t.size for _, t in entries)
+        if n_tokens > self.max_tokens:
+            raise TokenOverflowError(None)
+        if total + sum(rid not in row_of for rid in ids) > self.max_requests:
+            raise RequestOverflowError(None)
+        plan, chunks_needed = [], 0  # (id, tokens, row or None, tokens before, chunks to add)
+        for rid, toks in entries:
+            row = row_of.get(rid)
+            off = int(offs[row]) if row is not None else 0
+            if off + toks.size > self.max_sequence_length:
+                raise MaxSequenceLengthOverflowError(rid)
+            grow = math.ceil((off + toks.size) / self.chunk_size_tokens) - (int(counts[row]) if row is not None else 0)
+            plan.append((rid, toks, row, off, grow))
+            chunks_needed += grow
+        if not self.chunk_allocator.is_memory_available(chunks_needed):
+            raise ChunkOverflowError(None)
+        self._bt_version += 1
+        rows = []
+        for rid, toks, row, off, grow in plan:
+            if row is None:
+                row = self.total_request_count
+                self.total_request_count += 1
+                self.request_ids[row] = rid
+                self.request_output_lengths[row] = self.max_sequence_length
+                self.request_kv_length_offsets[row] = 0
+                self.request_kv_chunk_counts[row] = 0
+                self.request_to_kv_chunk_ids[row] = -1
+                self._take_state_slot(row)
+            have = int(counts[row])
+            if grow > 0:
+                self.request_to_kv_chunk_ids[row, have : have + grow] = self.chunk_allocator.allocate_memory_chunks(grow)
+                counts[row] = have + grow
+            self.request_query_lengths[row] = toks.size
+            self.request_last_kv_chunk_id[row] = self.request_to_kv_chunk_ids[row, int(counts[row]) - 1]
+            self.request_last_kv_chunk_offset[row] = (off + toks.size - 1) % self.chunk_size_tokens
+            rows.append(row)
+        # rows in the order [sitting out | this step's entries]
+        named = set(rows)
+        order = [r for r in range(self.total_request_count) if r not in named] + rows
+        self._permute_rows(order)
+        self.paused_request_count = self.total_request_count - len(rows)
+        self._wait_copies()
+        tok, table, a = self._h_tok_np, self.request_to_kv_chunk_ids.numpy(), 0
+        for k, (rid, toks, _, off, _) in enumerate(plan):
+            r, b = self.paused_request_count + k, a + toks.size
+            pos = off + np.arange(toks.size, dtype=np.int64)
+            tok[_TOK_INPUT, a:b] = toks
+            tok[_TOK_POS, a:b] = pos
+            tok[_TOK_REQ, a:b] = r
+            tok[_TOK_POS_IN_REQ, a:b] = pos
+            tok[_TOK_CHUNK, a:b] = table[r, pos // self.chunk_size_tokens]
+            tok[_TOK_LOCAL, a:b] = pos % self.chunk_size_tokens
+            a = b
+        self.active_token_count = a
+        self._push_token_rows(range(6), 0, a)
+
+    def complete_step(self, finished_ids=()) -> None:
+        """The forward of a `schedule_tokens` step has been enqueued: count its tokens as cached, drop ``finished_ids``."""
+        self.reset_attention_state()
+        p, t = self.paused_request_count, self.total_request_count
+        self.request_kv_length_offsets.numpy()[p:t] += self.request_query_lengths.numpy()[p:t]
+        self.request_query_lengths.numpy()[p:t] = 0
+        self._swap_state_sides(p, t)
+        self.active_token_count = 0
+        gone = set(finished_ids)
+        ids = self.request_ids[:t].tolist()
+        if not gone <= set(ids):
+            raise KeyError(f"not live: {sorted(gone - set(ids))}")
+        if gone:
+            drop = [r for r in range(t) if ids[r] in gone]
+            chunk_rows = self.request_to_kv_chunk_ids.numpy()[drop]
+            self.chunk_allocator.release_memory_chunks(chunk_rows[chunk_rows != -1])
+            self._release_state_slots(drop)
+            self.request_to_kv_chunk_ids.numpy()[drop] = -1
+            self.request_ids.numpy()[drop] = -1
+            self._permute_rows([r for r in range(t) if ids[r] not in gone] + drop)
+            self._bt_version += 1
+        self.total_request_count = t - len(gone)
+        self.paused_request_count = self.total_request_count
+
+    def _permute_rows(self, order: List[int]) -> None:
+        idx = np.asarray(order, dtype=np.int64)
+        if not np.array_equal(idx, np.arange(idx.size)):
+            for arr in self._request_arrays():
+                a = arr.numpy()
+                a[: idx.size] = a[idx]
+
+    def _request_arrays(self):
+        arrays = [self.request_kv_length_offsets, self.request_query_lengths, self.request_output_lengths, self.request_ids,
+                  self.request_to_kv_chunk_ids, self.request_kv_chunk_counts, self.request_last_kv_chunk_id,
+                  self.request_last_kv_chunk_offset]
+        if self.state_shapes is not None:
+            arrays += [self.request_state_slots, self.request_state_side]
+        return arrays
+
     # ------------------------------------------------------------------ per-step update
     def _move_book_keeping_tensors(self, src_idxs, dst_idxs, next_tokens) -> None:
         """rows[dst] = rows[src] for every request-level array and the pending tokens (reference :1017-1030)."""
-        for arr in (
-            self.request_kv_length_offsets,
-            self.request_query_lengths,
-            self.request_output_lengths,
-            self.request_ids,
-            self.request_to_kv_chunk_ids,
-            self.request_kv_chunk_counts,
-            self.request_last_kv_chunk_id,
-            self.request_last_kv_chunk_offset,
-        ):
+        for arr in self._request_arrays():
             a = arr.numpy()
             a[dst_idxs] = a[src_idxs]
         next_tokens[dst_idxs] = next_tokens[src_idxs]
@@ -768,6 +972,7 @@ class DynamicInferenceContext(BaseInferenceContext):
         assert active_request_count + finished_request_count + self.paused_request_count == self.total_request_count
         self.reset_attention_state()
         P = self.paused_request_count
+        self._swap_state_sides(P, self.total_request_count)  # the step has been run: its state is in the other buffers
         if self.FAST_DECODE_UPDATE and finished_request_count == 0 and P == 0 and active_request_count > 0:
             n = active_request_count
             last_off = self.request_last_kv_chunk_offset.numpy()
@@ -798,6 +1003,7 @@ class DynamicInferenceContext(BaseInferenceContext):
             if finished_request_count > 0:
                 rows = chunk_ids[np.nonzero(mask == 0)[0] + P]
                 self.chunk_allocator.release_memory_chunks(rows[rows != -1])
+                self._release_state_slots(np.nonzero(mask == 0)[0] + P)
             chunk_ids.fill(-1)
             self.total_request_count = 0
             self.active_token_count = 0
@@ -809,6 +1015,7 @@ class DynamicInferenceContext(BaseInferenceContext):
             finished_idxs = np.nonzero(mask == 0)[0] + P
             rows = chunk_ids[finished_idxs]
             self.chunk_allocator.release_memory_chunks(rows[rows != -1])
+            self._release_state_slots(finished_idxs)
             chunk_ids[finished_idxs] = -1
             if active_request_count > 0:
                 finished_on_left = np.nonzero(mask[:active_request_count] == 0)[0] + P

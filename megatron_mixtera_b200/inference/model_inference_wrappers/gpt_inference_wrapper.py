@@ -51,6 +51,9 @@ class GPTInferenceWrapper:
         if inference_context is not None and cfg is not None and hasattr(inference_context, "set_prefill_q_block"):
             from ... import ops
 
+            if hasattr(model, "prefill_unit_tokens"):  # the model's kernels cut work units of their own
+                inference_context.set_prefill_q_block(model.prefill_unit_tokens())
+                return
             groups = cfg.num_query_groups or cfg.num_attention_heads
             fp8_pool = getattr(inference_context, "kv_cache_fp8", False)  # the prefill kernel reads a bf16 pool
             inference_context.set_prefill_q_block(0 if fp8_pool else ops.prefill_q_block(cfg.num_attention_heads, groups))
@@ -108,6 +111,19 @@ class GPTInferenceWrapper:
         self.graph_replays += 1
         self.non_decode_graph_replays += 1
         return entry[1][:n_req].unsqueeze(0)
+
+    @torch.inference_mode()
+    def forward_token_rows(self, rows) -> torch.Tensor:
+        """Logits ``[len(rows), vocab]`` of the given tokens (indices into the step's flattened tokens) of the context's
+        current step; at least one row is computed."""
+        ctx = self.inference_context
+        ids, pos = ctx.current_input_and_position_ids()
+        idx = torch.as_tensor(rows if len(rows) else [0], dtype=torch.int64).to(ids.device)
+        if ctx.is_decode_only() and ctx.materialize_only_last_token_logits:  # one token per request: the decode path, graphs included
+            logits = self.run_one_forward_step({"tokens": ids, "position_ids": pos, "attention_mask": None})[0][idx]
+        else:
+            logits = self.model.forward_rows(ids, pos, ctx, idx, True)
+        return logits[: len(rows)]
 
     @torch.inference_mode()
     def run_one_forward_step(self, inference_input: Dict[str, Any], recv_buffer_seq_len: Optional[int] = None) -> torch.Tensor:

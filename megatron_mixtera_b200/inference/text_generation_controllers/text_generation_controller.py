@@ -160,6 +160,24 @@ class TextGenerationController:
         }
 
     @torch.inference_mode()
+    def run_given_tokens(self, entries, want, finished=()) -> torch.Tensor:
+        """One step over given tokens instead of sampled ones.  ``entries``: [(request id, its next tokens)], portions of
+        prompts beside single tokens (`DynamicInferenceContext.schedule_tokens`); ``want``: per entry the places among its
+        tokens whose logits are returned, in order, as ``[wanted, vocab]``; ``finished``: requests given back afterwards."""
+        context = self.inference_wrapped_model.inference_context
+        rows, base = [], 0
+        for (_, tokens), places in zip(entries, want, strict=True):
+            if any(not 0 <= p < len(tokens) for p in places):
+                raise ValueError("a wanted place lies outside its entry's tokens")
+            rows += [base + p for p in places]
+            base += len(tokens)
+        context.schedule_tokens(entries)
+        context.initialize_attention_state()
+        logits = self.inference_wrapped_model.forward_token_rows(rows)
+        context.complete_step(finished)
+        return logits
+
+    @torch.inference_mode()
     def generate_output_tokens_dynamic_batch(self, sampling_params: SamplingParams, termination_id: int):
         """Synchronous wrapper of `async_generate_output_tokens_dynamic_batch`."""
         return get_asyncio_loop().run_until_complete(

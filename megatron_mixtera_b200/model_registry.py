@@ -1,0 +1,120 @@
+"""Model classes by the ``architecture`` of a model folder (``config.json`` + ``model.safetensors``), and the serving stack
+around a loaded model."""
+from __future__ import annotations
+
+import json
+import os
+from typing import Callable, Dict, Tuple
+
+import torch
+
+from . import checkpoint
+from .transformer.hybrid_config import (DeltaRuleConfig, HybridConfig, HybridLayerConfig, LatentAttentionConfig, RotaryConfig,
+                                        YarnScaling)
+from .transformer.transformer_config import TransformerConfig
+
+
+# ---------------------------------------------------------------------------------------------------------------------
+# Zinurax
+# ---------------------------------------------------------------------------------------------------------------------
+def _latent_attention_config(m: dict) -> LatentAttentionConfig:
+    rot, scaling = m["rot"], m["rot"].get("scaling")
+    return LatentAttentionConfig(
+        heads=m["heads"], dim=m["dim"], rot_dim=m["rot_dim"], vdim=m["vdim"], kv_rank=m["kv_rank"], scale=float(m["scale"]),
+        rot=RotaryConfig(base=float(rot["base"]), dims=rot["dims"],
+                         scaling=YarnScaling(**{k: float(scaling[k]) for k in ("factor", "original", "fast", "slow")}) if scaling else None),
+        window=(m.get("mask") or {}).get("size"), kv_from=m.get("kv_from"))
+
+
+def zinurax_config(config: dict, shapes: Dict[str, tuple], dtype: torch.dtype) -> HybridConfig:
+    """``config.json`` -> `HybridConfig`; ``shapes`` (checkpoint tensor -> shape) gives what the file leaves to the tensors."""
+    layers = []
+    for i, layer in enumerate(config["layers"]):
+        m, mlp = layer["mixer"], layer.get("mlp")
+        if layer["type"] == "latent_attention":
+            mixer = _latent_attention_config(m)
+        elif layer["type"] == "general_delta":
+            mixer = DeltaRuleConfig(heads=m["heads"], dim=m["dim"], rank=shapes[f"l{i}.mix.w1"][0])
+        else:
+            raise ValueError(f"layer {i}: unknown mixer {layer['type']!r}")
+        if mlp is not None and mlp["kind"] != "dense":
+            raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+        layers.append(HybridLayerConfig(mixer=mixer, ffn_hidden_size=None if mlp is None else mlp["ff"]))
+    return HybridConfig(vocab_size=config["vocab"], hidden_size=config["width"], layers=tuple(layers),
+                        layernorm_epsilon=float(config["norm"]["eps"]), params_dtype=dtype)
+
+
+def _build_zinurax(config: dict, shapes: Dict[str, tuple], dtype: torch.dtype, max_sequence_length: int):
+    from .hybrid.hybrid_model import HybridModel
+
+    return HybridModel(zinurax_config(config, shapes, dtype), max_sequence_length)
+
+
+# ---------------------------------------------------------------------------------------------------------------------
+# GPTModel: config.json holds TransformerConfig fields under "transformer" and the model's own beside it
+# ---------------------------------------------------------------------------------------------------------------------
+def _build_gpt(config: dict, shapes: Dict[str, tuple], dtype: torch.dtype, max_sequence_length: int):
+    from .gpt.gpt_model import GPTModel
+
+    return GPTModel(TransformerConfig(params_dtype=dtype, **config["transformer"]), vocab_size=config["vocab_size"],
+                    max_sequence_length=max_sequence_length,
+                    position_embedding_type=config.get("position_embedding_type", "rope"),
+                    rotary_base=config.get("rotary_base", 10000.0),
+                    share_embeddings_and_output_weights=config.get("share_embeddings_and_output_weights", False))
+
+
+Builder = Callable[[dict, Dict[str, tuple], torch.dtype, int], torch.nn.Module]
+ARCHITECTURES: Dict[str, Builder] = {"Zinurax": _build_zinurax, "GPTModel": _build_gpt}
+
+
+def load_model(folder: str, *, dtype: torch.dtype = torch.bfloat16, max_sequence_length: int) -> torch.nn.Module:
+    """The model of a folder, weights loaded, on the current device."""
+    with open(os.path.join(folder, "config.json")) as f:
+        config = json.load(f)
+    name = config.get("architecture")
+    if name not in ARCHITECTURES:
+        raise ValueError(f"unknown architecture {name!r} (known: {', '.join(sorted(ARCHITECTURES))})")
+    path = os.path.join(folder, "model.safetensors")
+    model = ARCHITECTURES[name](config, checkpoint.tensor_shapes(path), dtype, max_sequence_length)
+    tensors = checkpoint.load_safetensors(path)
+    if hasattr(model, "load_checkpoint"):
+        model.load_checkpoint(tensors)
+    else:
+        model.load_full_state_dict(tensors)
+    return model
+
+
+def make_context(model, *, max_cached_tokens: int, max_requests: int, max_step_tokens: int, chunk_size_tokens: int = 64, **kwargs):
+    """A dynamic context whose pool holds ``max_cached_tokens`` (whole chunks), for ``max_requests`` live requests and steps of
+    up to ``max_step_tokens`` tokens."""
+    kwargs = dict(max_requests_override=max_requests, max_tokens_override=max_step_tokens, **kwargs)
+    if hasattr(model, "make_context"):
+        return model.make_context(max_cached_tokens=max_cached_tokens, chunk_size_tokens=chunk_size_tokens, **kwargs)
+    from .inference.contexts.dynamic_context import DynamicInferenceContext
+
+    c = model.config
+    chunk_bytes = c.params_dtype.itemsize * 2 * c.num_layers * chunk_size_tokens * c.num_query_groups * c.kv_channels
+    chunks = -(-max_cached_tokens // chunk_size_tokens) + 1
+    return DynamicInferenceContext(
+        params_dtype=c.params_dtype, num_layers=c.num_layers, kv_channels=c.kv_channels, num_attention_heads=c.num_query_groups,
+        max_sequence_length=model.max_sequence_length, buffer_size_gb=(chunks + 0.5) * chunk_bytes / 1024**3,
+        chunk_size_tokens=chunk_size_tokens, **{"buffer_guaranteed_fraction": 0.0, **kwargs})
+
+
+def make_controller(model, context, tokenizer=None):
+    """Wrapper and controller around a model and its context."""
+    from .inference.model_inference_wrappers.gpt_inference_wrapper import GPTInferenceWrapper, InferenceWrapperConfig
+    from .inference.text_generation_controllers.text_generation_controller import TextGenerationController
+
+    cfg = InferenceWrapperConfig(hidden_size=model.config.hidden_size, params_dtype=model.config.params_dtype,
+                                 padded_vocab_size=model.vocab_size)
+    return TextGenerationController(GPTInferenceWrapper(model, cfg, context), tokenizer)
+
+
+def serving_stack(folder: str, *, dtype: torch.dtype, max_cached_tokens: int, max_requests: int, max_sequence_length: int,
+                  max_step_tokens: int, **context_kwargs) -> Tuple[torch.nn.Module, object, object]:
+    """(model, context, controller) of a model folder."""
+    model = load_model(folder, dtype=dtype, max_sequence_length=max_sequence_length)
+    context = make_context(model, max_cached_tokens=max_cached_tokens, max_requests=max_requests, max_step_tokens=max_step_tokens,
+                           **context_kwargs)
+    return model, context, make_controller(model, context)

@@ -194,6 +194,11 @@ class ColumnParallelLinear(_ParallelLinearBase):
         return out, (self.bias if self.skip_bias_add else None)
 
 
+    def forward_activation(self, input_, act: str):
+        """Linear + elementwise activation (`ops.linear`'s) in one kernel; no bias."""
+        assert self.bias is None and not self.gather_output and self.fp8 is None
+        return ops.linear(input_.reshape(-1, input_.shape[-1]), self.weight, act=act).view(*input_.shape[:-1], -1)
+
     def forward_gated(self, input_):
         """Gated fc1 in the reference's [gate ; up] row order followed by SwiGLU: the fc2 input, quantised under an
         FP8 recipe.  One of three forms, all with the same bits: the one-kernel gate / up pair GEMM with the

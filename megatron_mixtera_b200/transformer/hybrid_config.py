@@ -1,0 +1,122 @@
+"""Configuration of hybrid decoders: a stack whose layers name their own mixer, its sizes and their feed-forward.
+
+`HybridConfig` also carries the fields that the shared modules read from a ``TransformerConfig`` (linears, MLP, wrapper,
+controller), so that those take either.
+"""
+from __future__ import annotations
+
+import dataclasses
+import math
+from dataclasses import dataclass
+from typing import Optional, Tuple, Union
+
+import torch
+
+
+@dataclass(frozen=True)
+class YarnScaling:
+    """Frequencies that turn often over the ``original`` context stay, slow ones are divided by ``factor``; a linear ramp
+    over the pair index joins them between ``fast`` and ``slow`` turns."""
+
+    factor: float
+    original: float
+    fast: float
+    slow: float
+
+
+@dataclass(frozen=True)
+class RotaryConfig:
+    base: float
+    dims: int  # leading dimensions that turn, in interleaved pairs (2i, 2i + 1)
+    scaling: Optional[YarnScaling] = None
+
+
+@dataclass(frozen=True)
+class LatentAttentionConfig:
+    heads: int
+    dim: int       # unrotated query / key dimensions per head
+    rot_dim: int   # rotated ones; the key's are shared by all heads
+    vdim: int
+    kv_rank: int
+    scale: float
+    rot: RotaryConfig
+    window: Optional[int] = None   # keys seen, the token itself included; None: all earlier ones
+    kv_from: Optional[int] = None  # 0-based layer whose cached rows this layer reads instead of making its own
+
+    def __post_init__(self):
+        if self.rot.dims % 2 or not 0 <= self.rot.dims <= self.rot_dim:
+            raise ValueError("rot.dims must be even and at most rot_dim")
+        if self.window is not None and self.window < 1:
+            raise ValueError("a window holds at least the token itself")
+
+    @property
+    def kv_pad(self) -> int:
+        """Where the rotated part starts in a cached row."""
+        return -(-self.kv_rank // 16) * 16
+
+    @property
+    def row_width(self) -> int:
+        """Elements of a cached row: latent and rotated part, padded for 16-byte copies and 16 x 32 tensor-core steps."""
+        return -(-(self.kv_pad + self.rot_dim) // 32) * 32
+
+
+@dataclass(frozen=True)
+class DeltaRuleConfig:
+    heads: int
+    dim: int   # key and value channels per head
+    rank: int  # inner width of the decay's two-step projection
+    decay_scale: float = math.exp(-0.5)  # decay = exp(-decay_scale * sigmoid(.))
+    unit_eps: float = 1e-6               # inside the unit key's root
+
+
+MixerConfig = Union[LatentAttentionConfig, DeltaRuleConfig]
+
+
+@dataclass(frozen=True)
+class HybridLayerConfig:
+    mixer: MixerConfig
+    ffn_hidden_size: Optional[int] = None  # None: no feed-forward
+
+
+@dataclass
+class HybridConfig:
+    vocab_size: int
+    hidden_size: int
+    layers: Tuple[HybridLayerConfig, ...]
+    layernorm_epsilon: float = 1e-5
+    params_dtype: torch.dtype = torch.bfloat16  # bfloat16, or float32: the whole model in true 32-bit arithmetic
+    activation: str = "relu2"
+    gated_linear_unit: bool = False
+    add_bias_linear: bool = False
+    ffn_hidden_size: Optional[int] = None       # set per layer (`for_layer`)
+    fp8: Optional[str] = None
+    tensor_model_parallel_size: int = 1
+    enable_cuda_graph: bool = False
+    inference_sampling_seed: int = 42
+    fuse_splitk_reduction_into_norm: bool = True
+    defer_logits_gather: bool = True
+
+    def __post_init__(self):
+        self.layers = tuple(self.layers)
+        if self.params_dtype not in (torch.bfloat16, torch.float32):
+            raise ValueError("hybrid decoders compute in bfloat16 or float32")
+        if self.tensor_model_parallel_size != 1:
+            raise NotImplementedError("hybrid decoders run on one GPU")
+        for i, layer in enumerate(self.layers):
+            m = layer.mixer
+            src = getattr(m, "kv_from", None)
+            if src is None:
+                continue
+            own = self.layers[src].mixer if 0 <= src < i else None
+            if not isinstance(own, LatentAttentionConfig) or own.kv_from is not None:
+                raise ValueError(f"layer {i} reads the rows of layer {src}, which is no earlier latent-attention layer with its own")
+            if (own.kv_rank, own.rot_dim, own.rot) != (m.kv_rank, m.rot_dim, m.rot):
+                raise ValueError(f"layers {src} and {i} share cached rows but differ in their shape or rotation")
+
+    @property
+    def num_layers(self) -> int:
+        return len(self.layers)
+
+    def for_layer(self, index: int) -> "HybridConfig":
+        """The view of layer ``index`` that per-layer modules (MLP) read."""
+        return dataclasses.replace(self, ffn_hidden_size=self.layers[index].ffn_hidden_size)

@@ -1,0 +1,103 @@
+"""Latent attention: keys and values of all heads come from one small row per token, the only thing cached.
+
+The key matrix is applied to the queries instead of the cached rows ("absorbed") and the value matrix to the attention
+output, both as batched per-head GEMMs, so that prompts and decoding alike read the cached rows once and never expand them.
+"""
+from __future__ import annotations
+
+import torch
+
+from .. import _lib, ops
+from ..tensor_parallel.layers import ColumnParallelLinear, RowParallelLinear, _device
+from .attention import _sm_count
+from .hybrid_config import HybridConfig, LatentAttentionConfig
+
+
+def choose_latent_splits(num_rows: int, heads: int, window, max_sequence_length: int) -> int:
+    """Key splits of a decode row: a function of capture-time constants, enough CTAs for every SM, no split below 256 keys
+    at the longest visible range."""
+    blocks = max(1, num_rows * -(-heads // 64))
+    keys = max_sequence_length if window is None else min(window, max_sequence_length)
+    return int(max(1, min(-(-_sm_count() // blocks), keys // 256, 64)))
+
+
+class LatentAttention(torch.nn.Module):
+    def __init__(self, config: HybridConfig, mixer: LatentAttentionConfig, layer_index: int):
+        super().__init__()
+        self.config, self.mixer = config, mixer
+        m, dt, dev = mixer, config.params_dtype, _device()
+        self.cache_layer_number = (layer_index if m.kv_from is None else m.kv_from) + 1
+        self.owns_rows = m.kv_from is None
+        # one linear for everything that reads the layer's input: [queries | latent, shared key | gates]
+        q_width = m.heads * (m.dim + m.rot_dim)
+        down = m.kv_rank + m.rot_dim if self.owns_rows else 0
+        self.dkv_offset = q_width if self.owns_rows else -1
+        self.gate_offset = q_width + down
+        self.in_width = q_width + down + m.heads
+        padded = -(-self.in_width // 8) * 8  # whole 16-byte vectors per row; the added rows are zero
+        self.linear_in = ColumnParallelLinear(config.hidden_size, padded, config=config, bias=False)
+        self.key_up = torch.nn.Parameter(torch.empty(m.heads * m.kv_rank, m.dim, dtype=dt, device=dev), requires_grad=False)
+        self.value_up = torch.nn.Parameter(torch.empty(m.heads * m.vdim, m.kv_rank, dtype=dt, device=dev), requires_grad=False)
+        if self.owns_rows:
+            self.latent_norm = torch.nn.Parameter(torch.ones(m.kv_rank, dtype=dt, device=dev), requires_grad=False)
+        else:
+            self.register_parameter("latent_norm", None)
+        self.linear_proj = RowParallelLinear(m.heads * m.vdim, config.hidden_size, config=config, bias=False)
+
+    def checkpoint_tensors(self) -> dict:
+        """Checkpoint name (below the layer's mixer) -> shape."""
+        m, H = self.mixer, self.config.hidden_size
+        out = {"q": (m.heads * (m.dim + m.rot_dim), H), "uk": (m.heads * m.dim, m.kv_rank), "uv": (m.heads * m.vdim, m.kv_rank),
+               "g": (m.heads, H), "o": (H, m.heads * m.vdim)}
+        if self.owns_rows:
+            out.update({"dkv": (m.kv_rank + m.rot_dim, H), "dkv.norm": (m.kv_rank,)})
+        return out
+
+    def load(self, get) -> None:
+        m = self.mixer
+        parts = [get("q")] + ([get("dkv")] if self.owns_rows else []) + [get("g")]
+        w = self.linear_in.weight.data
+        w.zero_()
+        w[: self.in_width].copy_(torch.cat([p.to(w.device) for p in parts]))
+        self.key_up.data.copy_(get("uk").view(m.heads, m.dim, m.kv_rank).transpose(1, 2).reshape(m.heads * m.kv_rank, m.dim))
+        self.value_up.data.copy_(get("uv"))
+        if self.owns_rows:
+            self.latent_norm.data.copy_(get("dkv.norm"))
+        self.linear_proj.weight.data.copy_(get("o"))
+
+    def forward(self, x, ctx, rope):
+        """``x`` [T, H] -> the output linear's partial sums."""
+        m, T, dev = self.mixer, x.shape[0], x.device
+        proj, _ = self.linear_in(x)
+        q_full = torch.empty((T, m.heads, m.row_width), dtype=x.dtype, device=dev)
+        latent_out = torch.empty((T, m.heads * m.kv_rank), dtype=x.dtype, device=dev)
+        pool = ctx.latent_cache(self.cache_layer_number)
+        decode = ctx.is_decode_only()
+        a = _lib.LatentArgs()
+        a.proj, a.proj_ld, a.dkv_offset, a.gate_offset = proj.data_ptr(), proj.stride(0), self.dkv_offset, self.gate_offset
+        a.norm_weight = None if self.latent_norm is None else self.latent_norm.data_ptr()
+        a.rope_cos, a.rope_sin, a.max_positions = rope[0].data_ptr(), rope[1].data_ptr(), rope[0].shape[0]
+        a.token_to_pos = ctx.token_to_position_in_request.data_ptr()
+        a.token_to_chunk_idx = ctx.token_to_chunk_idx.data_ptr()
+        a.token_to_local_pos = ctx.token_to_local_position_within_kv_chunk.data_ptr()
+        a.block_table = ctx.request_to_kv_chunk_ids_cudagraph_only.data_ptr()
+        a.max_chunks_per_row = ctx.request_to_kv_chunk_ids_cudagraph_only.shape[1]
+        a.pool, a.num_chunks, a.chunk_size = pool.data_ptr(), pool.shape[0], pool.shape[1]
+        a.q_full, a.out = q_full.data_ptr(), latent_out.data_ptr()
+        a.num_tokens, a.heads, a.dim, a.rot_dim, a.rot_dims = T, m.heads, m.dim, m.rot_dim, m.rot.dims
+        a.kv_rank, a.kv_pad, a.row_width = m.kv_rank, m.kv_pad, m.row_width
+        a.window, a.scale, a.eps = m.window or 0, m.scale, self.config.layernorm_epsilon
+        a.dtype, a.num_splits = ops.dtype_code(x.dtype), 1
+        if decode:
+            a.kv_seq_lengths = ctx.kv_seq_lengths_cudagraph_only.data_ptr()
+            if x.dtype == torch.bfloat16:
+                a.num_splits = choose_latent_splits(T, m.heads, m.window, ctx.max_sequence_length)
+        else:
+            a.units, a.num_units, a.unit_tokens = ctx.prefill_units.data_ptr(), ctx.prefill_unit_count, ctx.prefill_q_block
+        # absorbed queries: per head W_uk^T q
+        ops.linear(proj, self.key_up, out=q_full.view(T, -1), batch=m.heads, x_batch=m.dim + m.rot_dim, y_batch=m.row_width, K=m.dim)
+        ops.latent_append(a, pool)
+        ops.latent_attention(a, pool)
+        values = torch.empty((T, m.heads * m.vdim), dtype=x.dtype, device=dev)
+        ops.linear(latent_out, self.value_up, out=values, batch=m.heads, x_batch=m.kv_rank, y_batch=m.vdim, K=m.kv_rank)
+        return self.linear_proj(values, defer_reduction=True)[0]

@@ -1,4 +1,4 @@
-"""Feed-forward block: fc1 -> SwiGLU or bias+GELU -> fc2 (reference ``megatron/core/transformer/mlp.py:140-234``).
+"""Feed-forward block: fc1 -> SwiGLU, bias+GELU or squared ReLU -> fc2 (reference ``megatron/core/transformer/mlp.py:140-234``).
 fc1's weight holds ``[gate ; up]`` halves per rank for the gated case (``fused_bias_swiglu.py:25``)."""
 from __future__ import annotations
 
@@ -55,6 +55,8 @@ class MLP(torch.nn.Module):
             return self.linear_fc1.forward_swiglu(hidden_states)
         if self.config.gated_linear_unit and self.linear_fc1.bias is None and hasattr(self.linear_fc1, "forward_gated"):
             return self.linear_fc1.forward_gated(hidden_states)
+        if self.config.activation == "relu2":  # squared ReLU: in the GEMM's epilogue
+            return self.linear_fc1.forward_activation(hidden_states, "relu2")
         inter, bias = self.linear_fc1(hidden_states)
         act = {None: ops.activation, "mxfp8": ops.activation_mxfp8, "blockwise": ops.activation_fp8_rowblock}[self.config.fp8]
         if self.config.gated_linear_unit:

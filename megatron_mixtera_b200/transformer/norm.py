@@ -45,3 +45,30 @@ class B200Norm(torch.nn.Module):
             return ops.add_norm_splitk(x, self.weight, bias=bias, residual=residual, beta=self.bias, eps=self.eps,
                                        want_hidden=True, quantize=quantize or None)
         return self._op(quantize)(x, self.weight, bias=bias, residual=residual, beta=self.bias, eps=self.eps, want_hidden=True)
+
+
+class OutputNorm(torch.nn.Module):
+    """Layer norm (a weight, no bias) of a sublayer's OUTPUT, added to a 32-bit residual stream by the same kernel:
+    ``hidden += norm(f(x))``, where the sublayer read the stream itself.  The stream is fp32 ``[T, H]``; what the next
+    sublayer reads is its copy in the activation type (the stream itself when that is fp32)."""
+
+    accepts_gemm_partials = True
+
+    def __init__(self, config, hidden_size: int, eps: float = 1e-5, **_):
+        super().__init__()
+        dev = torch.device("cuda", torch.cuda.current_device()) if torch.cuda.is_available() else torch.device("cpu")
+        self.eps = eps
+        self.weight = torch.nn.Parameter(torch.ones(hidden_size, dtype=config.params_dtype, device=dev), requires_grad=False)
+
+    def start_stream(self, table, ids):
+        """(fp32 stream, activations) of ``norm(table[ids])``."""
+        hidden = torch.empty((ids.numel(), table.shape[1]), dtype=torch.float32, device=table.device)
+        return hidden, ops.out_norm(table, self.weight, eps=self.eps, hidden=hidden, ids=ids)
+
+    def add_to_stream(self, hidden, source):
+        """hidden += norm(source) in place; ``source``: `ops.GemmPartials` of the sublayer's last linear."""
+        return ops.out_norm(source, self.weight, eps=self.eps, hidden=hidden, accumulate=True)
+
+    def of_rows(self, hidden, row_index=None):
+        """norm of the stream's rows (all, or those picked by ``row_index``) in the activation type."""
+        return ops.out_norm(hidden, self.weight, eps=self.eps, row_index=row_index)

@@ -753,8 +753,9 @@ def linear(x, w, *, act: Optional[str] = None, out=None, batch: int = 1, x_batch
     _need(w, x.dtype, "w")
     if not x.is_cuda or x.stride(-1) != 1 or x.dim() != 2:
         raise B200Error("linear", -1, "x must be a 2-D CUDA tensor with unit inner stride")
-    K = w.shape[1] if K is None else K
-    if w.shape[1] != K or w.shape[0] % batch or (batch == 1 and x.shape[1] != K):
+    if K is None:
+        K = x.shape[1]
+    if w.shape[1] != K or w.shape[0] % batch or (batch - 1) * x_batch + K > x.shape[1]:
         raise B200Error("linear", -1, f"shape mismatch x{tuple(x.shape)} vs w{tuple(w.shape)}, batch {batch}, K {K}")
     M, N, ldx = x.shape[0], w.shape[0] // batch, x.stride(0)
     if out is None:

@@ -7,7 +7,12 @@
 //
 //   latent_append_kernel   one CTA per token: norms the latent, rotates the shared key part and stores the row; rotates
 //                          the query part of every head into the absorbed query.
-//   latent_mma_kernel      bf16.  One CTA per (block of MT query rows, key split); a query row is a (token, head) pair, and
+//   latent_decode_kernel   bf16 decode steps of up to 32 heads.  One CTA per (token, key split); a producer warp fetches 32 pool
+//                          rows per stage (one bulk copy per row, addresses through the block table, completion on an
+//                          mbarrier).  Eight consumer warps split S = Q R^T by key half and by quarter of row_width - a warp's
+//                          part of Q stays in registers - add the quarters through shared memory, do the softmax two rows per
+//                          warp, and split O += P C by columns.  Bound by reading the rows once.
+//   latent_mma_kernel      bf16, everything else (prompts, more heads).  One CTA per (block of MT query rows, key split); a query row is a (token, head) pair, and
 //                          consecutive pairs of one request share the key tiles.  A producer warp fetches KT pool rows per
 //                          stage (one bulk copy per row, addresses through the block table, completion on an mbarrier); eight
 //                          consumer warps compute S = Q R^T (each its 16 query rows x KW keys), exchange row maxima, write the
@@ -445,6 +450,292 @@ latent_mma_kernel(b200_latent_args a, int stages) {
   }
 }
 
+// ---------------------------------------------------------------------------------------------------------------
+// Decode: one token's heads (up to 16 * RG) against a range of keys
+// ---------------------------------------------------------------------------------------------------------------
+constexpr int kDecKeys = 32;
+constexpr int kSxStride = 40;  // floats per row of the score exchange: 64-bit stores of a half warp hit all banks once
+constexpr int kDecPStride = kDecKeys + 8;
+
+template <int RG, int KVT>
+struct DecodeShape {
+  static constexpr int kRows = 16 * RG;
+  static constexpr int kQSteps = KVT == 512 ? 10 : 6;  // 16-wide steps of a row_width quarter
+  static constexpr int kMaxWidth = 4 * 16 * kQSteps;
+  static constexpr int kCols = KVT / kWarps / 16;
+  static __host__ __device__ int fixed_bytes() {
+    return 4 * kRows * kSxStride * 4 + 2 * kRows * kDecPStride * 2 + 3 * kRows * 4 + 128;
+  }
+  static __host__ __device__ int stage_bytes(int row_stride) { return kDecKeys * row_stride * 2; }
+};
+
+template <int RG, int KVT>
+__global__ void __launch_bounds__(kThreads, RG == 1 ? 2 : 1)
+latent_decode_kernel(b200_latent_args a, int stages) {
+  using D = DecodeShape<RG, KVT>;
+  constexpr int KT = kDecKeys, ROWS = D::kRows, SR = ROWS / kWarps;  // SR: softmax rows per warp
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  pdl_launch_dependents();
+  const int t = blockIdx.x, split = blockIdx.z;
+  const int kv_len = a.kv_seq_lengths[t];
+  int start = window_start(kv_len - 1, a.window), end = kv_len;
+  if (a.num_splits > 1) {
+    const int len = split_length(end - start, a.num_splits);
+    start += split * len;
+    end = min(end, start + len);
+  }
+  if (kv_len <= 0 || start >= end) {
+    pdl_wait();  // (a kernel never ends before its predecessor)
+    return;
+  }
+  const int n_tiles = (end - start + KT - 1) / KT;
+
+  extern __shared__ __align__(128) uint8_t smem[];
+  const int rs = a.row_width + 8;
+  __nv_bfloat16* k_s = reinterpret_cast<__nv_bfloat16*>(smem);
+  float* sx = reinterpret_cast<float*>(k_s + stages * KT * rs);  // [quarter][row][key]
+  __nv_bfloat16* p_hi = reinterpret_cast<__nv_bfloat16*>(sx + 4 * ROWS * kSxStride);
+  __nv_bfloat16* p_lo = p_hi + ROWS * kDecPStride;
+  float* al = reinterpret_cast<float*>(p_lo + ROWS * kDecPStride);  // per row: rescale factor, later 1 / sum
+  float* lse = al + ROWS;
+  uint64_t* full_bar = reinterpret_cast<uint64_t*>(lse + 2 * ROWS);
+  uint64_t* empty_bar = full_bar + kMaxStages;
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(empty_bar + kMaxStages);
+  if (tid == 0) {
+    for (int s = 0; s < stages; ++s) {
+      mbar_init(&full_bar[s], 1);
+      mbar_init(&empty_bar[s], kWarps);
+    }
+    *abort_flag = 0;
+    fence_barrier_init();
+  }
+  const int tail = end - start - (n_tiles - 1) * KT;
+  if (n_tiles <= stages && tail < KT) {  // missing keys get weight 0, but 0 times a stray NaN is a NaN
+    uint32_t* z = reinterpret_cast<uint32_t*>(k_s + ((n_tiles - 1) * KT + tail) * rs);
+    for (int i = tid; i < (KT - tail) * rs / 2; i += kThreads) z[i] = 0u;
+  }
+  __syncthreads();
+
+  if (warp == kWarps) {
+    // ------------------------------- producer warp -------------------------------
+    const int32_t* bt = a.block_table + static_cast<int64_t>(t) * a.max_chunks_per_row;
+    const uint32_t row_bytes = a.row_width * 2;
+    bool waited = false;
+    for (int i = 0; i < n_tiles; ++i) {
+      const int s = i % stages;
+      const int key = start + i * KT + lane;
+      const int n = min(KT, end - start - i * KT);
+      // Only the newest token's row is written by this step (by the append kernel before this one); older rows are there.
+      if (!waited && start + i * KT + n >= kv_len) {
+        pdl_wait();
+        waited = true;
+      }
+      if (lane == 0) {
+        mbar_wait_bounded(&empty_bar[s], ((i / stages) & 1) ^ 1, abort_flag, kStatusAttnTimeout);
+        mbar_arrive_expect_tx(&full_bar[s], n * row_bytes);
+      }
+      __syncwarp();
+      if (lane < n)
+        bulk_load_1d(k_s + (s * KT + lane) * rs, static_cast<const __nv_bfloat16*>(a.pool) + pool_row(a, bt, key) * a.row_width,
+                     row_bytes, &full_bar[s]);
+    }
+    if (!waited) pdl_wait();
+    return;
+  }
+
+  // --------------------------------- consumer warps ---------------------------------
+  const int kg = warp & 1, kq = warp >> 1;
+  const int gid = lane >> 2, tig = lane & 3;
+  const int k_steps = a.row_width / 16;
+  const int per_q = (k_steps + 3) / 4;
+  const int ks0 = kq * per_q, ks_n = min(per_q, k_steps - ks0);  // this warp's steps (none: ks_n <= 0)
+  pdl_wait();
+  uint32_t qf[RG][D::kQSteps][4];
+  {
+    const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(a.q_full) + static_cast<int64_t>(t) * a.heads * a.row_width;
+#pragma unroll
+    for (int g = 0; g < RG; ++g)
+#pragma unroll
+      for (int s = 0; s < D::kQSteps; ++s)
+#pragma unroll
+        for (int f = 0; f < 4; ++f) {
+          const int r = g * 16 + gid + (f & 1) * 8, c = (ks0 + s) * 16 + tig * 2 + (f >> 1) * 8;
+          qf[g][s][f] = (s < ks_n && r < a.heads) ? *reinterpret_cast<const uint32_t*>(q + r * a.row_width + c) : 0u;
+        }
+  }
+  const float scale_log2 = a.scale * kLog2e;
+  float o_acc[RG][D::kCols][2][4];
+#pragma unroll
+  for (int g = 0; g < RG; ++g)
+#pragma unroll
+    for (int j = 0; j < D::kCols; ++j)
+#pragma unroll
+      for (int c = 0; c < 4; ++c) o_acc[g][j][0][c] = o_acc[g][j][1][c] = 0.f;
+  float m_run[SR], l_run[SR];  // softmax rows warp * SR + r: the maximum is the warp's, the sum a lane's share
+#pragma unroll
+  for (int r = 0; r < SR; ++r) {
+    m_run[r] = -INFINITY;
+    l_run[r] = 0.f;
+  }
+  const int col_blocks = a.kv_pad / 16;
+
+  for (int i = 0; i < n_tiles; ++i) {
+    const int s = i % stages;
+    mbar_wait_bounded(&full_bar[s], (i / stages) & 1, abort_flag, kStatusAttnTimeout);
+    const __nv_bfloat16* tile = k_s + s * KT * rs;
+    // ---- S: 16 keys, one quarter of row_width ----
+    float sc[RG][2][4];
+#pragma unroll
+    for (int g = 0; g < RG; ++g)
+#pragma unroll
+      for (int c = 0; c < 4; ++c) sc[g][0][c] = sc[g][1][c] = 0.f;
+    const uint32_t k_addr = smem_u32(tile + (kg * 16 + ((lane >> 4) << 3) + (lane & 7)) * rs + ks0 * 16 + ((lane >> 3) & 1) * 8);
+#pragma unroll
+    for (int q = 0; q < D::kQSteps; ++q) {
+      if (q < ks_n) {
+        uint32_t b0, b1, b2, b3;
+        ldmatrix_x4(k_addr + q * 32, b0, b1, b2, b3);
+#pragma unroll
+        for (int g = 0; g < RG; ++g) {
+          mma_bf16_16816(sc[g][0], qf[g][q], b0, b1);
+          mma_bf16_16816(sc[g][1], qf[g][q], b2, b3);
+        }
+      }
+    }
+#pragma unroll
+    for (int g = 0; g < RG; ++g)
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int r = 0; r < 2; ++r)
+          *reinterpret_cast<float2*>(sx + (kq * ROWS + g * 16 + gid + r * 8) * kSxStride + kg * 16 + n * 8 + tig * 2) =
+              make_float2(sc[g][n][2 * r], sc[g][n][2 * r + 1]);
+    consumer_barrier();
+    // ---- softmax (log2 domain): lane = key ----
+    const bool seen = start + i * KT + lane < end;
+#pragma unroll
+    for (int r = 0; r < SR; ++r) {
+      const int row = warp * SR + r;
+      const float* x = sx + row * kSxStride + lane;
+      float v = (x[0] + x[ROWS * kSxStride]) + (x[2 * ROWS * kSxStride] + x[3 * ROWS * kSxStride]);
+      v = seen ? v * scale_log2 : -INFINITY;
+      const float m_new = fmaxf(m_run[r], warp_max(v));  // finite: a tile has a key
+      const float alpha = exp2f(m_run[r] - m_new);
+      const float p = exp2f(v - m_new);
+      m_run[r] = m_new;
+      l_run[r] = l_run[r] * alpha + p;
+      const __nv_bfloat16 hi = __float2bfloat16_rn(p);
+      p_hi[row * kDecPStride + lane] = hi;
+      p_lo[row * kDecPStride + lane] = __float2bfloat16_rn(p - __bfloat162float(hi));
+      if (lane == 0) al[row] = alpha;
+    }
+    consumer_barrier();
+    // ---- O += P C: every kWarps-th 16-column block, weights as hi + lo terms ----
+    const uint32_t v_addr = smem_u32(tile + ((((lane >> 3) & 1) << 3) + (lane & 7)) * rs + (lane >> 4) * 8);
+    float f[RG][2];
+    bool scaled = false;
+#pragma unroll
+    for (int g = 0; g < RG; ++g)
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        f[g][r] = al[g * 16 + gid + r * 8];
+        scaled |= f[g][r] != 1.f;
+      }
+    if (__any_sync(0xffffffffu, scaled)) {
+#pragma unroll
+      for (int g = 0; g < RG; ++g)
+#pragma unroll
+        for (int j = 0; j < D::kCols; ++j)
+#pragma unroll
+          for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int c = 0; c < 4; ++c) o_acc[g][j][n][c] *= f[g][c >> 1];
+    }
+#pragma unroll
+    for (int kk = 0; kk < KT / 16; ++kk) {
+      uint32_t ph[RG][4], pl[RG][4];
+#pragma unroll
+      for (int g = 0; g < RG; ++g) {
+        const int off = (g * 16 + (lane & 15)) * kDecPStride + kk * 16 + (lane >> 4) * 8;
+        ldmatrix_x4(smem_u32(p_hi + off), ph[g][0], ph[g][1], ph[g][2], ph[g][3]);
+        ldmatrix_x4(smem_u32(p_lo + off), pl[g][0], pl[g][1], pl[g][2], pl[g][3]);
+      }
+#pragma unroll
+      for (int j = 0; j < D::kCols; ++j) {
+        const int cb = j * kWarps + warp;
+        if (cb < col_blocks) {
+          uint32_t b0, b1, b2, b3;
+          ldmatrix_x4_trans(v_addr + (kk * 16 * rs + cb * 16) * 2, b0, b1, b2, b3);
+#pragma unroll
+          for (int g = 0; g < RG; ++g) {
+            mma_bf16_16816(o_acc[g][j][0], ph[g], b0, b1);
+            mma_bf16_16816(o_acc[g][j][1], ph[g], b2, b3);
+            mma_bf16_16816(o_acc[g][j][0], pl[g], b0, b1);
+            mma_bf16_16816(o_acc[g][j][1], pl[g], b2, b3);
+          }
+        }
+      }
+    }
+    __syncwarp();
+    if (lane == 0) mbar_arrive(&empty_bar[s]);
+  }
+
+  consumer_barrier();  // `al` is read by the last tile until here
+#pragma unroll
+  for (int r = 0; r < SR; ++r) {
+    const float l = warp_sum(l_run[r]);
+    if (lane == 0) {
+      al[warp * SR + r] = 1.f / l;
+      lse[warp * SR + r] = m_run[r] + log2f(l);
+    }
+  }
+  consumer_barrier();
+  const bool even = (a.kv_rank & 1) == 0;
+#pragma unroll
+  for (int g = 0; g < RG; ++g)
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      const int head = g * 16 + gid + r * 8;
+      if (head >= a.heads) continue;
+      const int64_t pair = static_cast<int64_t>(t) * a.heads + head;
+      if (a.num_splits > 1) {
+        float* dst = a.workspace + (pair * a.num_splits + split) * a.kv_rank;
+        if (warp == 0 && tig == 0)
+          a.workspace[static_cast<int64_t>(a.num_tokens) * a.heads * a.num_splits * a.kv_rank + pair * a.num_splits + split] = lse[head];
+        const float inv = al[head];
+#pragma unroll
+        for (int j = 0; j < D::kCols; ++j)
+#pragma unroll
+          for (int n = 0; n < 2; ++n) {
+            const int col = (j * kWarps + warp) * 16 + n * 8 + tig * 2;
+            const float v0 = o_acc[g][j][n][2 * r] * inv, v1 = o_acc[g][j][n][2 * r + 1] * inv;
+            if (even && col + 1 < a.kv_rank) {
+              *reinterpret_cast<float2*>(dst + col) = make_float2(v0, v1);
+            } else {
+              if (col < a.kv_rank) dst[col] = v0;
+              if (col + 1 < a.kv_rank) dst[col + 1] = v1;
+            }
+          }
+      } else {
+        const float gate = gate_of<__nv_bfloat16>(a, t, head) * al[head];
+        __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(a.out) + pair * a.kv_rank;
+#pragma unroll
+        for (int j = 0; j < D::kCols; ++j)
+#pragma unroll
+          for (int n = 0; n < 2; ++n) {
+            const int col = (j * kWarps + warp) * 16 + n * 8 + tig * 2;
+            const float v0 = o_acc[g][j][n][2 * r] * gate, v1 = o_acc[g][j][n][2 * r + 1] * gate;
+            if (even && col + 1 < a.kv_rank) {
+              *reinterpret_cast<uint32_t*>(dst + col) = pack_bf16x2(v0, v1);
+            } else {
+              if (col < a.kv_rank) dst[col] = __float2bfloat16_rn(v0);
+              if (col + 1 < a.kv_rank) dst[col + 1] = __float2bfloat16_rn(v1);
+            }
+          }
+      }
+    }
+}
+
 // One CTA per (token, head): merge the splits' normalised partial outputs by their log-sum-exp.
 __global__ void __launch_bounds__(128)
 latent_combine_kernel(b200_latent_args a) {
@@ -582,6 +873,27 @@ static int launch_mma(const b200_latent_args& a, cudaStream_t s) {
   return launch_pdl(latent_combine_kernel, dim3(a.num_tokens * a.heads), dim3(128), 0, s, a);
 }
 
+// Whether the decode kernel takes this call, and its launch.
+template <int RG, int KVT>
+static bool decode_fits(const b200_latent_args& a) {
+  return !a.units && a.heads <= 16 * RG && a.kv_pad <= KVT && a.row_width <= DecodeShape<RG, KVT>::kMaxWidth;
+}
+template <int RG, int KVT>
+static int launch_decode(const b200_latent_args& a, cudaStream_t s) {
+  using D = DecodeShape<RG, KVT>;
+  const int rs = a.row_width + 8;
+  auto fit = [&](int budget) { return (budget - D::fixed_bytes()) / D::stage_bytes(rs); };
+  int stages = fit(kMaxSmem / 2 - 1024);  // two CTAs per SM
+  if (stages < 2) stages = fit(kMaxSmem);
+  stages = stages > kMaxStages ? kMaxStages : stages;
+  static std::atomic<uint64_t> done{0};
+  if (ensure_dynamic_smem(latent_decode_kernel<RG, KVT>, kMaxSmem, done) != B200_OK) return B200_ERR_LAUNCH;
+  const int rc = launch_pdl(latent_decode_kernel<RG, KVT>, dim3(a.num_tokens, 1, a.num_splits), dim3(kThreads),
+                            D::fixed_bytes() + stages * D::stage_bytes(rs), s, a, stages);
+  if (rc != B200_OK || a.num_splits == 1) return rc;
+  return launch_pdl(latent_combine_kernel, dim3(a.num_tokens * a.heads), dim3(128), 0, s, a);
+}
+
 }  // namespace latent
 }  // namespace b200
 
@@ -622,6 +934,10 @@ int b200_latent_attention(const b200_latent_args* a, b200_stream_t stream) {
     if (a->num_splits > 1 &&
         (!a->workspace || a->workspace_bytes < b200_latent_attention_workspace_bytes(a->num_tokens, a->heads, a->kv_rank, a->num_splits)))
       return B200_ERR_WORKSPACE;
+    if (decode_fits<1, 256>(*a)) return launch_decode<1, 256>(*a, s);
+    if (decode_fits<1, 512>(*a)) return launch_decode<1, 512>(*a, s);
+    if (decode_fits<2, 256>(*a)) return launch_decode<2, 256>(*a, s);
+    if (decode_fits<2, 512>(*a)) return launch_decode<2, 512>(*a, s);
     const bool wide = a->kv_pad > 256;
     if (mt == 16) return wide ? launch_mma<16, 512>(*a, s) : launch_mma<16, 256>(*a, s);
     if (mt == 32) return wide ? launch_mma<32, 512>(*a, s) : launch_mma<32, 256>(*a, s);

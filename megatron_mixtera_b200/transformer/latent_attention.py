@@ -14,11 +14,21 @@ from .hybrid_config import HybridConfig, LatentAttentionConfig
 
 
 def choose_latent_splits(num_rows: int, heads: int, window, max_sequence_length: int) -> int:
-    """Key splits of a decode row: a function of capture-time constants, enough CTAs for every SM, no split below 256 keys
-    at the longest visible range."""
+    """Key splits of a decode row: a function of capture-time constants.  The fewest splits that fill the CTAs the GPU holds
+    at once to 85 % (else the best there is), none below 256 keys at the longest visible range."""
+    slots = _sm_count() * (2 if heads <= 16 else 1)
     blocks = max(1, num_rows * -(-heads // 64))
     keys = max_sequence_length if window is None else min(window, max_sequence_length)
-    return int(max(1, min(-(-_sm_count() // blocks), keys // 256, 64)))
+    best, best_fill = 1, 0.0
+    for splits in range(1, max(1, min(keys // 256, 64)) + 1):
+        length = -(-(-(-keys // splits)) // 64) * 64  # whole tiles, as the kernels cut
+        units = blocks * -(-keys // length)
+        fill = units / (-(-units // slots) * slots)
+        if fill > best_fill:
+            best, best_fill = splits, fill
+        if fill >= 0.85:
+            return splits
+    return best
 
 
 class LatentAttention(torch.nn.Module):

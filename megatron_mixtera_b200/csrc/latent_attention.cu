@@ -7,17 +7,14 @@
 //
 //   latent_append_kernel   one CTA per token: norms the latent, rotates the shared key part and stores the row; rotates
 //                          the query part of every head into the absorbed query.
-//   latent_decode_kernel   bf16 decode steps of up to 32 heads.  One CTA per (token, key split); a producer warp fetches 32 pool
+//   latent_umma_kernel     bf16: prompts, and decode steps of more than 16 heads.  tcgen05.mma with tensor-memory accumulators, up
+//                          to 64 query rows - (token, head) pairs of one request - against 64-key tiles by TMA.
+//   latent_decode_kernel   bf16 decode steps of up to 16 heads.  One CTA per (token, key split); a producer warp fetches 32 pool
 //                          rows per stage (one bulk copy per row, addresses through the block table, completion on an
 //                          mbarrier).  Eight consumer warps split S = Q R^T by key half and by quarter of row_width - a warp's
 //                          part of Q stays in registers - add the quarters through shared memory, do the softmax two rows per
 //                          warp, and split O += P C by columns.  Bound by reading the rows once.
-//   latent_mma_kernel      bf16, everything else (prompts, more heads).  One CTA per (block of MT query rows, key split); a query row is a (token, head) pair, and
-//                          consecutive pairs of one request share the key tiles.  A producer warp fetches KT pool rows per
-//                          stage (one bulk copy per row, addresses through the block table, completion on an mbarrier); eight
-//                          consumer warps compute S = Q R^T (each its 16 query rows x KW keys), exchange row maxima, write the
-//                          weights as hi + lo bf16 terms and accumulate O += P C (each its 16 query rows x its columns).
-//   latent_simt_kernel     any type and size, fp32 arithmetic throughout: the 32-bit mode and latents wider than 512.
+//   latent_simt_kernel     any type and size, fp32 arithmetic throughout: the 32-bit mode and shapes the others do not take.
 //   latent_combine_kernel  merges the key splits of decode rows.
 //
 // Only keys inside the window are visited: [first query's oldest visible key, last query's position].
@@ -141,325 +138,16 @@ __device__ __forceinline__ int64_t pool_row(const b200_latent_args& a, const int
 
 __device__ __forceinline__ void consumer_barrier() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
 
-template <int MT>
-struct Shape {
-  static constexpr int kKeys = MT == 64 ? 32 : 64;   // keys per tile
-  static constexpr int kRowGroups = MT / 16;
-  static constexpr int kKeyGroups = kWarps / kRowGroups;  // also the column groups of the second product
-  static constexpr int kKeysPerWarp = kKeys / kKeyGroups; // 8 or 16
-  static constexpr int kPStride = kKeys + 8;
-  static __host__ __device__ int fixed_bytes(int row_stride) {  // everything but the key stages
-    return MT * row_stride * 2 + 2 * MT * kPStride * 2 + kKeyGroups * MT * 4 + 128;
-  }
-  static __host__ __device__ int stage_bytes(int row_stride) { return kKeys * row_stride * 2; }
-};
-
-template <int MT, int KVT>
-__global__ void __launch_bounds__(kThreads, 1)
-latent_mma_kernel(b200_latent_args a, int stages) {
-  using S = Shape<MT>;
-  constexpr int KT = S::kKeys;
-  constexpr int kCols = KVT / S::kKeyGroups / 16;  // 16-column blocks of the output per warp
-  constexpr int NT = S::kKeysPerWarp / 8;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  pdl_launch_dependents();
-
-  // ---- which rows, which keys ----
-  const int sub = blockIdx.y, split = blockIdx.z;
-  int row, tok0, count;
-  if (a.units != nullptr) {
-    const int4 u = reinterpret_cast<const int4*>(a.units)[blockIdx.x];
-    row = u.x;
-    tok0 = u.y;
-    count = u.z;
-  } else {
-    row = tok0 = blockIdx.x;
-    count = a.kv_seq_lengths[row] > 0 ? 1 : 0;
-  }
-  const int q_rows = min(MT, count * a.heads - sub * MT);
-  pdl_wait();  // (a kernel never ends before its predecessor; everything below reads what predecessors wrote)
-  if (q_rows <= 0) return;
-  const int first_tok = tok0 + (sub * MT) / a.heads, last_tok = tok0 + (sub * MT + q_rows - 1) / a.heads;
-  int first_pos, last_pos;
-  if (a.units != nullptr) {
-    first_pos = static_cast<int>(a.token_to_pos[first_tok]);
-    last_pos = first_pos + (last_tok - first_tok);
-  } else {
-    first_pos = last_pos = a.kv_seq_lengths[row] - 1;
-  }
-  int start = window_start(first_pos, a.window), end = last_pos + 1;
-  if (a.num_splits > 1) {
-    const int len = split_length(end - start, a.num_splits);
-    start += split * len;
-    end = min(end, start + len);
-    if (start >= end) return;
-  }
-  const int n_tiles = (end - start + KT - 1) / KT;
-
-  // ---- shared memory ----
-  extern __shared__ __align__(128) uint8_t smem[];
-  const int rs = a.row_width + 8;  // elements; an odd number of 16-byte units, so that ldmatrix rows miss each other's banks
-  __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(smem);
-  __nv_bfloat16* k_s = q_s + MT * rs;
-  __nv_bfloat16* p_hi = k_s + stages * KT * rs;
-  __nv_bfloat16* p_lo = p_hi + MT * S::kPStride;
-  float* stat = reinterpret_cast<float*>(p_lo + MT * S::kPStride);  // [key group][MT]
-  uint64_t* full_bar = reinterpret_cast<uint64_t*>(stat + S::kKeyGroups * MT);
-  uint64_t* empty_bar = full_bar + kMaxStages;
-  volatile int* abort_flag = reinterpret_cast<volatile int*>(empty_bar + kMaxStages);
-  if (tid == 0) {
-    for (int s = 0; s < stages; ++s) {
-      mbar_init(&full_bar[s], 1);
-      mbar_init(&empty_bar[s], kWarps);
-    }
-    *abort_flag = 0;
-    fence_barrier_init();
-  }
-  const int tail = end - start - (n_tiles - 1) * KT;  // keys of the last tile
-  if (n_tiles <= stages && tail < KT) {
-    // The last tile's missing keys get weight 0, but 0 times a stray NaN is a NaN: clear rows nothing has written.
-    uint32_t* z = reinterpret_cast<uint32_t*>(k_s + ((n_tiles - 1) * KT + tail) * rs);
-    for (int i = tid; i < (KT - tail) * rs / 2; i += kThreads) z[i] = 0u;
-  }
-  __syncthreads();
-
-  if (warp == kWarps) {
-    // ------------------------------- producer warp -------------------------------
-    const int32_t* bt = a.block_table + static_cast<int64_t>(row) * a.max_chunks_per_row;
-    const uint32_t row_bytes = a.row_width * 2;
-    for (int i = 0; i < n_tiles; ++i) {
-      const int s = i % stages;
-      const uint32_t phase = (i / stages) & 1;
-      const int key0 = start + i * KT;
-      const int n = min(KT, end - key0);
-      if (lane == 0) {
-        mbar_wait_bounded(&empty_bar[s], phase ^ 1, abort_flag, kStatusAttnTimeout);
-        mbar_arrive_expect_tx(&full_bar[s], n * row_bytes);
-      }
-      __syncwarp();
-      for (int r = lane; r < n; r += 32)
-        bulk_load_1d(k_s + (s * KT + r) * rs, static_cast<const __nv_bfloat16*>(a.pool) + pool_row(a, bt, key0 + r) * a.row_width,
-                     row_bytes, &full_bar[s]);
-    }
-    return;
-  }
-
-  // --------------------------------- consumer warps ---------------------------------
-  const int rg = warp % S::kRowGroups, kg = warp / S::kRowGroups;
-  const int gid = lane >> 2, tig = lane & 3;
-  {
-    const uint4* src = reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(a.q_full) +
-                                                      (static_cast<int64_t>(tok0) * a.heads + sub * MT) * a.row_width);
-    const int per_row = a.row_width / 8;
-    for (int i = tid; i < MT * per_row; i += kConsumerThreads) {
-      const int r = i / per_row, c = i - r * per_row;
-      *reinterpret_cast<uint4*>(q_s + r * rs + c * 8) = r < q_rows ? src[i] : make_uint4(0, 0, 0, 0);
-    }
-  }
-  // visible keys [lo, hi] of this thread's two query rows
-  int lo[2], hi[2], q_row[2];
-#pragma unroll
-  for (int r = 0; r < 2; ++r) {
-    q_row[r] = rg * 16 + gid + r * 8;
-    const bool ok = q_row[r] < q_rows;
-    const int pos = first_pos + (sub * MT + q_row[r]) / a.heads - (sub * MT) / a.heads;
-    hi[r] = ok ? pos : -1;
-    lo[r] = window_start(pos, a.window);
-  }
-  const float scale_log2 = a.scale * kLog2e;
-  float o_acc[kCols][2][4];
-#pragma unroll
-  for (int j = 0; j < kCols; ++j)
-#pragma unroll
-    for (int c = 0; c < 4; ++c) o_acc[j][0][c] = o_acc[j][1][c] = 0.f;
-  float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
-  const int k_steps = a.row_width / 16;
-  const int col_blocks = a.kv_pad / 16;
-  const uint32_t q_addr = smem_u32(q_s + (rg * 16 + (lane & 15)) * rs + (lane >> 4) * 8);
-  consumer_barrier();
-
-  for (int i = 0; i < n_tiles; ++i) {
-    const int s = i % stages;
-    const int key0 = start + i * KT;
-    mbar_wait_bounded(&full_bar[s], (i / stages) & 1, abort_flag, kStatusAttnTimeout);
-    const __nv_bfloat16* tile = k_s + s * KT * rs;
-
-    // ---- S = Q R^T: 16 query rows x kKeysPerWarp keys ----
-    float sc[NT][4];
-#pragma unroll
-    for (int n = 0; n < NT; ++n) sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.f;
-    if constexpr (NT == 2) {
-      const uint32_t k_addr = smem_u32(tile + (kg * 16 + ((lane >> 4) << 3) + (lane & 7)) * rs + ((lane >> 3) & 1) * 8);
-#pragma unroll 4
-      for (int ks = 0; ks < k_steps; ++ks) {
-        uint32_t q[4], b0, b1, b2, b3;
-        ldmatrix_x4(q_addr + ks * 32, q[0], q[1], q[2], q[3]);
-        ldmatrix_x4(k_addr + ks * 32, b0, b1, b2, b3);
-        mma_bf16_16816(sc[0], q, b0, b1);
-        mma_bf16_16816(sc[1], q, b2, b3);
-      }
-    } else {
-      // 8 keys: one ldmatrix brings two k-steps (row_width is a multiple of 32); two accumulators break the chain
-      float s2[4] = {0.f, 0.f, 0.f, 0.f};
-      const uint32_t k_addr = smem_u32(tile + (kg * 8 + (lane & 7)) * rs + (lane >> 3) * 8);
-#pragma unroll 4
-      for (int ks = 0; ks < k_steps; ks += 2) {
-        uint32_t q[4], q2[4], b0, b1, b2, b3;
-        ldmatrix_x4(q_addr + ks * 32, q[0], q[1], q[2], q[3]);
-        ldmatrix_x4(q_addr + ks * 32 + 32, q2[0], q2[1], q2[2], q2[3]);
-        ldmatrix_x4(k_addr + ks * 32, b0, b1, b2, b3);
-        mma_bf16_16816(sc[0], q, b0, b1);
-        mma_bf16_16816(s2, q2, b2, b3);
-      }
-#pragma unroll
-      for (int c = 0; c < 4; ++c) sc[0][c] += s2[c];
-    }
-
-    // ---- online softmax (log2 domain); the row maximum spans the key groups ----
-    float mx[2] = {-INFINITY, -INFINITY};
-#pragma unroll
-    for (int n = 0; n < NT; ++n)
-#pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        const int key = key0 + kg * S::kKeysPerWarp + n * 8 + tig * 2 + (c & 1);
-        const int r = c >> 1;
-        const float v = (key >= lo[r] && key <= hi[r] && key < end) ? sc[n][c] * scale_log2 : -INFINITY;
-        sc[n][c] = v;
-        mx[r] = fmaxf(mx[r], v);
-      }
-#pragma unroll
-    for (int r = 0; r < 2; ++r) {
-      mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
-      mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
-      if (tig == 0) stat[kg * MT + q_row[r]] = mx[r];
-    }
-    consumer_barrier();
-    float alpha[2], m_use[2];
-#pragma unroll
-    for (int r = 0; r < 2; ++r) {
-      float m_new = m_run[r];
-#pragma unroll
-      for (int g = 0; g < S::kKeyGroups; ++g) m_new = fmaxf(m_new, stat[g * MT + q_row[r]]);
-      m_use[r] = m_new == -INFINITY ? 0.f : m_new;
-      alpha[r] = exp2f(m_run[r] - m_use[r]);
-      m_run[r] = m_new;
-      l_run[r] *= alpha[r];
-    }
-#pragma unroll
-    for (int n = 0; n < NT; ++n) {
-      float p[4];
-#pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        p[c] = exp2f(sc[n][c] - m_use[c >> 1]);
-        l_run[c >> 1] += p[c];
-      }
-#pragma unroll
-      for (int r = 0; r < 2; ++r) {
-        const float h0 = bf16_round(p[2 * r]), h1 = bf16_round(p[2 * r + 1]);
-        const int off = q_row[r] * S::kPStride + kg * S::kKeysPerWarp + n * 8 + tig * 2;
-        *reinterpret_cast<uint32_t*>(p_hi + off) = pack_bf16x2(h0, h1);
-        *reinterpret_cast<uint32_t*>(p_lo + off) = pack_bf16x2(p[2 * r] - h0, p[2 * r + 1] - h1);
-      }
-    }
-    consumer_barrier();
-
-    // ---- O += P C: 16 query rows x every kKeyGroups-th 16-column block, weights as hi + lo terms ----
-    if (__any_sync(0xffffffffu, alpha[0] != 1.f || alpha[1] != 1.f)) {
-#pragma unroll
-      for (int j = 0; j < kCols; ++j)
-#pragma unroll
-        for (int n = 0; n < 2; ++n) {
-          o_acc[j][n][0] *= alpha[0];
-          o_acc[j][n][1] *= alpha[0];
-          o_acc[j][n][2] *= alpha[1];
-          o_acc[j][n][3] *= alpha[1];
-        }
-    }
-    const int p_off = (rg * 16 + (lane & 15)) * S::kPStride + (lane >> 4) * 8;
-    const uint32_t ph_addr = smem_u32(p_hi + p_off), pl_addr = smem_u32(p_lo + p_off);
-    const uint32_t v_addr = smem_u32(tile + ((((lane >> 3) & 1) << 3) + (lane & 7)) * rs + (lane >> 4) * 8);
-#pragma unroll
-    for (int kk = 0; kk < KT / 16; ++kk) {
-      uint32_t ph[4], pl[4];
-      ldmatrix_x4(ph_addr + kk * 32, ph[0], ph[1], ph[2], ph[3]);
-      ldmatrix_x4(pl_addr + kk * 32, pl[0], pl[1], pl[2], pl[3]);
-#pragma unroll
-      for (int j = 0; j < kCols; ++j) {
-        const int cb = j * S::kKeyGroups + kg;
-        if (cb < col_blocks) {
-          uint32_t b0, b1, b2, b3;
-          ldmatrix_x4_trans(v_addr + (kk * 16 * rs + cb * 16) * 2, b0, b1, b2, b3);
-          mma_bf16_16816(o_acc[j][0], ph, b0, b1);
-          mma_bf16_16816(o_acc[j][1], ph, b2, b3);
-          mma_bf16_16816(o_acc[j][0], pl, b0, b1);
-          mma_bf16_16816(o_acc[j][1], pl, b2, b3);
-        }
-      }
-    }
-    __syncwarp();
-    if (lane == 0) mbar_arrive(&empty_bar[s]);
-  }
-
-  // ---- row sums over the quad and the key groups, then the output ----
-#pragma unroll
-  for (int r = 0; r < 2; ++r) {
-    l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 1);
-    l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 2);
-    if (tig == 0) stat[kg * MT + q_row[r]] = l_run[r];
-  }
-  consumer_barrier();
-#pragma unroll
-  for (int r = 0; r < 2; ++r) {
-    if (q_row[r] >= q_rows) continue;
-    float l = 0.f;
-#pragma unroll
-    for (int g = 0; g < S::kKeyGroups; ++g) l += stat[g * MT + q_row[r]];
-    const float inv = l > 0.f ? 1.f / l : 0.f;
-    const int64_t pair = static_cast<int64_t>(tok0) * a.heads + sub * MT + q_row[r];  // token * heads + head
-    if (a.num_splits > 1) {
-      float* dst = a.workspace + (pair * a.num_splits + split) * a.kv_rank;
-      if (kg == 0 && tig == 0)
-        a.workspace[static_cast<int64_t>(a.num_tokens) * a.heads * a.num_splits * a.kv_rank + pair * a.num_splits + split] =
-            l > 0.f ? m_run[r] + log2f(l) : -INFINITY;
-#pragma unroll
-      for (int j = 0; j < kCols; ++j)
-#pragma unroll
-        for (int n = 0; n < 2; ++n) {
-          const int col = (j * S::kKeyGroups + kg) * 16 + n * 8 + tig * 2;
-          if (col < a.kv_rank) dst[col] = o_acc[j][n][2 * r] * inv;
-          if (col + 1 < a.kv_rank) dst[col + 1] = o_acc[j][n][2 * r + 1] * inv;
-        }
-    } else {
-      const float g = gate_of<__nv_bfloat16>(a, pair / a.heads, static_cast<int>(pair % a.heads)) * inv;
-      __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(a.out) + pair * a.kv_rank;
-      const bool even = (a.kv_rank & 1) == 0;
-#pragma unroll
-      for (int j = 0; j < kCols; ++j)
-#pragma unroll
-        for (int n = 0; n < 2; ++n) {
-          const int col = (j * S::kKeyGroups + kg) * 16 + n * 8 + tig * 2;
-          const float v0 = o_acc[j][n][2 * r] * g, v1 = o_acc[j][n][2 * r + 1] * g;
-          if (even && col + 1 < a.kv_rank) {
-            *reinterpret_cast<uint32_t*>(dst + col) = pack_bf16x2(v0, v1);
-          } else {
-            if (col < a.kv_rank) dst[col] = __float2bfloat16_rn(v0);
-            if (col + 1 < a.kv_rank) dst[col + 1] = __float2bfloat16_rn(v1);
-          }
-        }
-    }
-  }
-}
-
 // ---------------------------------------------------------------------------------------------------------------
-// Decode: one token's heads (up to 16 * RG) against a range of keys
+// Decode: one token's heads (up to 16) against a range of keys
 // ---------------------------------------------------------------------------------------------------------------
 constexpr int kDecKeys = 32;
 constexpr int kSxStride = 40;  // floats per row of the score exchange: 64-bit stores of a half warp hit all banks once
 constexpr int kDecPStride = kDecKeys + 8;
 
-template <int RG, int KVT>
+template <int KVT>
 struct DecodeShape {
-  static constexpr int kRows = 16 * RG;
+  static constexpr int kRows = 16;
   static constexpr int kQSteps = KVT == 512 ? 10 : 6;  // 16-wide steps of a row_width quarter
   static constexpr int kMaxWidth = 4 * 16 * kQSteps;
   static constexpr int kCols = KVT / kWarps / 16;
@@ -469,10 +157,11 @@ struct DecodeShape {
   static __host__ __device__ int stage_bytes(int row_stride) { return kDecKeys * row_stride * 2; }
 };
 
-template <int RG, int KVT>
-__global__ void __launch_bounds__(kThreads, RG == 1 ? 2 : 1)
+template <int KVT>
+__global__ void __launch_bounds__(kThreads, 2)
 latent_decode_kernel(b200_latent_args a, int stages) {
-  using D = DecodeShape<RG, KVT>;
+  using D = DecodeShape<KVT>;
+  constexpr int RG = 1;  // groups of 16 query rows
   constexpr int KT = kDecKeys, ROWS = D::kRows, SR = ROWS / kWarps;  // SR: softmax rows per warp
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   pdl_launch_dependents();
@@ -736,6 +425,410 @@ latent_decode_kernel(b200_latent_args a, int stages) {
     }
 }
 
+// K-major operands in shared memory: per 64 columns a [KEYS][64] sub-tile of 128-byte rows, 16-byte pieces swizzled.  Byte
+// offset of piece `c8` (8 columns each) of row `r`.
+template <int KEYS>
+__device__ __forceinline__ int piece_offset(int r, int c8) {
+  return (c8 >> 3) * (KEYS * 128) + r * 128 + (((c8 & 7) ^ (r & 7)) << 4);
+}
+// ---------------------------------------------------------------------------------------------------------------
+// Tensor-memory kernel: up to N query rows ((token, head) pairs of one request) against a range of keys, 64 keys a tile.
+//
+// Both products are tcgen05.mma with the cached rows on the M side, so that few query rows waste nothing:
+//   S^T [64 keys x N]           = tile (K-major, rows = keys)      x Q (K-major, rows = query rows)
+//   O^T [128 channels x 2N] (+)= tile (MN-major, the same bytes)  x P (K-major, rows = query rows: N of the weights' bf16 values,
+//                                                                      N of what that rounding left over; added at the end)
+// Warps 0-3: softmax - a thread owns a key (a 64-row accumulator sits in lanes 0-15 of each warp's part of tensor memory): it
+// reads its N scores and writes its 2N weight terms to shared memory as the B operand.  Weights are taken relative to a
+// reference per query row that trails the running maximum by at most kGrow (in log2): only when a score exceeds that are
+// maxima exchanged and O rescaled, which after the first tiles hardly ever happens.  Warp 4: TMA, warp 5: MMA issue.
+// The scores of the next tile are computed before the values of the current one, so that its softmax runs beside them.
+// ---------------------------------------------------------------------------------------------------------------
+constexpr int kUmKeys = 64;
+constexpr int kUmThreads = 192;
+constexpr int kUmMaxStages = 4;
+constexpr int kSubBytes = kUmKeys * 128;
+constexpr float kGrow = 8.f;
+
+__device__ __forceinline__ float exp2_approx(float x) {  // 2^x to fp32 accuracy (2 ulp), 0 below the normal range
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+template <int N>
+struct UmmaShape {
+  static __host__ __device__ int subs(int row_width, int kv_pad) {
+    const int s = (row_width + 63) / 64, o = (kv_pad + 127) / 128 * 2;
+    return s > o ? s : o;
+  }
+  static __host__ __device__ int q_bytes(int row_width) { return (row_width + 63) / 64 * N * 128; }
+  static constexpr int kPBytes = 2 * N * 128;
+  static constexpr int kMiscBytes = (4 + 3 + 2) * N * 4 + 1024;
+  static __host__ __device__ int bytes(int row_width, int kv_pad, int stages) {
+    return 1024 + stages * subs(row_width, kv_pad) * kSubBytes + q_bytes(row_width) + 2 * kPBytes + kMiscBytes;
+  }
+};
+
+template <int N>
+__global__ void __launch_bounds__(kUmThreads, 1)
+latent_umma_kernel(const __grid_constant__ CUtensorMap map, b200_latent_args a, int stages, int tmem_cols) {
+  using U = UmmaShape<N>;
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int subs_loaded = (a.row_width + 63) / 64, subs = U::subs(a.row_width, a.kv_pad);
+  const int m_tiles = (a.kv_pad + 127) / 128;
+  uint8_t* q_s = smem + stages * subs * kSubBytes;
+  uint8_t* p_s = q_s + U::q_bytes(a.row_width);  // two buffers of [2N rows][128 bytes]
+  float* red = reinterpret_cast<float*>(p_s + 2 * U::kPBytes);  // [4 warps][N]
+  float* m_s = red + 4 * N;                                      // references
+  float* al_s = m_s + N;                                         // rescale factors; at the end output factors
+  int* lo_s = reinterpret_cast<int*>(al_s + 2 * N);              // visible keys of every query row
+  int* hi_s = lo_s + N;
+  uint64_t* full_bar = reinterpret_cast<uint64_t*>(hi_s + N);
+  uint64_t* empty_bar = full_bar + kUmMaxStages;
+  uint64_t* s_full = empty_bar + kUmMaxStages;  // [2]
+  uint64_t* p_ready = s_full + 2;             // [2]
+  uint64_t* pv_done = p_ready + 2;            // [2]
+  uint64_t* patched = pv_done + 2;            // [2]: the first and the last tile
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(patched + 2);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+
+  if (tid == 0) {
+    for (int s = 0; s < stages; ++s) {
+      mbar_init(&full_bar[s], 1);
+      mbar_init(&empty_bar[s], 1);
+    }
+    for (int s = 0; s < 2; ++s) {
+      mbar_init(&s_full[s], 1);
+      mbar_init(&p_ready[s], 128);
+      mbar_init(&pv_done[s], 1);
+      mbar_init(&patched[s], 128);
+    }
+    *abort_flag = 0;
+    fence_barrier_init();
+    prefetch_tensormap(&map);
+  }
+  if (warp == 0) {
+    tmem_alloc(tmem_slot, tmem_cols);
+    tmem_relinquish_alloc_permit();
+  }
+  tcgen05_fence_before_sync();
+  __syncthreads();
+  tcgen05_fence_after_sync();
+  const uint32_t tmem = *tmem_slot;   // S^T buffers at columns 0 and N, O^T tiles behind them
+  const uint32_t tmem_o = tmem + 2 * N;
+  pdl_launch_dependents();            // (behind the allocation: a successor's CTA must not hold tensor memory we wait for)
+
+  // ---- which rows, which keys ----
+  const int sub = blockIdx.y, split = blockIdx.z;
+  int row, tok0, count;
+  if (a.units != nullptr) {
+    const int4 u = reinterpret_cast<const int4*>(a.units)[blockIdx.x];
+    row = u.x;
+    tok0 = u.y;
+    count = u.z;
+  } else {
+    row = tok0 = blockIdx.x;
+    count = a.kv_seq_lengths[row] > 0 ? 1 : 0;
+  }
+  const int q_rows = min(N, count * a.heads - sub * N);
+  int first_pos = 0, last_pos = 0, start = 0, end = 0;
+  if (q_rows > 0) {
+    const int first_tok = tok0 + (sub * N) / a.heads, last_tok = tok0 + (sub * N + q_rows - 1) / a.heads;
+    first_pos = a.units != nullptr ? static_cast<int>(a.token_to_pos[first_tok]) : a.kv_seq_lengths[row] - 1;
+    last_pos = first_pos + (last_tok - first_tok);
+    start = window_start(first_pos, a.window);
+    end = last_pos + 1;
+    if (a.num_splits > 1) {
+      const int len = split_length(end - start, a.num_splits);
+      start += split * len;
+      end = min(end, start + len);
+    }
+  }
+  const int base = start / kUmKeys * kUmKeys;
+  const int n_tiles = end > start ? (end - base + kUmKeys - 1) / kUmKeys : 0;
+  const int32_t* bt = a.block_table + static_cast<int64_t>(row) * a.max_chunks_per_row;
+  const int stage_bytes = subs * kSubBytes;
+  int load_stage = 0, load_phase = 1;
+  auto load = [&](int i) {  // one thread, tiles in order
+    const int y = static_cast<int>(pool_row(a, bt, base + i * kUmKeys));
+    uint64_t* bar = &full_bar[load_stage];
+    mbar_wait_bounded(&empty_bar[load_stage], load_phase, abort_flag, kStatusAttnTimeout);
+    mbar_arrive_expect_tx(bar, subs_loaded * kSubBytes);
+    uint8_t* dst = smem + load_stage * stage_bytes;
+    for (int c = 0; c < subs_loaded; ++c) tma_load_2d(dst + c * kSubBytes, &map, bar, c * 64, y);
+    if (++load_stage == stages) {
+      load_stage = 0;
+      load_phase ^= 1;
+    }
+  };
+  // Decode: only the newest token's row is written by this step (by the append kernel before this one); the others are there.
+  int loaded = 0;
+  if (warp == 4 && lane == 0 && a.units == nullptr)
+    for (; loaded < min(stages, n_tiles) && base + (loaded + 1) * kUmKeys <= last_pos; ++loaded) load(loaded);
+  pdl_wait();
+  // Q as a K-major operand, rows past q_rows and columns past row_width zero
+  if (n_tiles > 0) {
+    const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(a.q_full) + (static_cast<int64_t>(tok0) * a.heads + sub * N) * a.row_width;
+    for (int i = tid; i < subs_loaded * 8 * N; i += kUmThreads) {
+      const int r = i / (subs_loaded * 8), c8 = i - r * (subs_loaded * 8);
+      uint4 v = make_uint4(0, 0, 0, 0);
+      if (r < q_rows && c8 * 8 < a.row_width) v = *reinterpret_cast<const uint4*>(q + static_cast<int64_t>(r) * a.row_width + c8 * 8);
+      *reinterpret_cast<uint4*>(q_s + piece_offset<N>(r, c8)) = v;
+    }
+    for (int n = tid; n < N; n += kUmThreads) {
+      const int pos = first_pos + (sub * N + n) / a.heads - (sub * N) / a.heads;
+      hi_s[n] = n < q_rows ? min(pos, end - 1) : -1;
+      lo_s[n] = max(window_start(pos, a.window), start);
+      m_s[n] = -INFINITY;
+    }
+  }
+  fence_proxy_async_smem();
+  __syncthreads();
+
+  if (n_tiles > 0 && warp == 4) {
+    // ------------------------------- TMA -------------------------------
+    if (lane == 0)
+      for (; loaded < n_tiles; ++loaded) load(loaded);
+    __syncwarp();
+  } else if (n_tiles > 0 && warp == 5) {
+    if (lane == 0) {
+      // ------------------------------- MMA -------------------------------
+      constexpr uint32_t idesc_s = umma_idesc_bf16(kUmKeys, N);
+      constexpr uint32_t idesc_o = umma_idesc_bf16(128, 2 * N) | kUmmaTransposeA;
+      const uint64_t tile_k = umma_desc_k_major_sw128(smem_u32(smem));
+      const uint64_t tile_mn = umma_desc_mn_major_sw128(smem_u32(smem), kSubBytes);
+      const uint64_t q_desc = umma_desc_k_major_sw128(smem_u32(q_s)), p_desc = umma_desc_k_major_sw128(smem_u32(p_s));
+      int patches = 0, s_stage = 0, s_phase = 0, v_stage = 0;
+      auto scores = [&](int i) {
+        const int k0 = base + i * kUmKeys;
+        if (k0 < start || k0 + kUmKeys > end) mbar_wait_bounded(&patched[patches++], 0, abort_flag, kStatusAttnTimeout);
+        mbar_wait_bounded(&full_bar[s_stage], s_phase, abort_flag, kStatusAttnTimeout);
+        tcgen05_fence_after_sync();
+        uint64_t ad = tile_k + static_cast<uint64_t>(s_stage * stage_bytes >> 4), bd = q_desc;
+        const uint32_t d = tmem + (i & 1) * N;
+        for (int c = 0; c < subs_loaded; ++c) {
+#pragma unroll
+          for (int k = 0; k < 4; ++k) umma_f16(d, ad + 2 * k, bd + 2 * k, idesc_s, (c > 0 || k > 0) ? 1u : 0u);
+          ad += kSubBytes >> 4;
+          bd += N * 128 >> 4;
+        }
+        umma_commit(&s_full[i & 1]);
+        if (++s_stage == stages) {
+          s_stage = 0;
+          s_phase ^= 1;
+        }
+      };
+      scores(0);
+      for (int i = 0; i < n_tiles; ++i) {
+        // The next tile's scores go first where the tile is there: their softmax then runs beside this tile's values.
+        const bool ahead = stages > 1 && i + 1 < n_tiles && mbar_try_wait(&full_bar[s_stage], s_phase);
+        if (ahead) scores(i + 1);
+        mbar_wait_bounded(&p_ready[i & 1], (i >> 1) & 1, abort_flag, kStatusAttnTimeout);
+        tcgen05_fence_after_sync();
+        uint64_t ad = tile_mn + static_cast<uint64_t>(v_stage * stage_bytes >> 4);
+        const uint64_t bd = p_desc + static_cast<uint64_t>((i & 1) * U::kPBytes >> 4);
+        uint32_t d = tmem_o;
+        for (int j = 0; j < m_tiles; ++j) {
+#pragma unroll
+          for (int ks = 0; ks < kUmKeys / 16; ++ks) umma_f16(d, ad + 128 * ks, bd + 2 * ks, idesc_o, (i > 0 || ks > 0) ? 1u : 0u);
+          ad += 2 * kSubBytes >> 4;
+          d += 2 * N;
+        }
+        umma_commit(&empty_bar[v_stage]);
+        umma_commit(&pv_done[i & 1]);
+        if (++v_stage == stages) v_stage = 0;
+        if (!ahead && i + 1 < n_tiles) scores(i + 1);
+      }
+    }
+    __syncwarp();
+  } else if (n_tiles > 0) {
+    // ------------------------------- softmax -------------------------------
+    const uint32_t lanes = static_cast<uint32_t>(warp * 32) << 16;
+    const float scale_log2 = a.scale * kLog2e;
+    const bool owner = lane < 16;                  // this thread owns key `mine` of every tile
+    const int mine = warp * 16 + (lane & 15);
+    // tiles whose keys every query row sees need no masks
+    const int all_lo = max(window_start(last_pos, a.window), start), all_hi = min(first_pos, end - 1);
+    float l_part[N], m[N];  // sums of this thread's weights, references
+#pragma unroll
+    for (int n = 0; n < N; ++n) {
+      l_part[n] = 0.f;
+      m[n] = -INFINITY;
+    }
+    auto group_sync = [] { asm volatile("bar.sync 1, 128;" ::: "memory"); };
+    auto group_any = [](bool p) {
+      int r;
+      asm volatile(
+          "{\n.reg .pred p, q;\nsetp.ne.s32 p, %1, 0;\nbarrier.red.or.pred q, 2, 128, p;\nselp.s32 %0, 1, 0, q;\n}\n"
+          : "=r"(r)
+          : "r"(static_cast<int>(p))
+          : "memory");
+      return r != 0;
+    };
+    int patches = 0, f_stage = 0, f_phase = 0;
+    auto patch = [&](int i) {  // tiles in order: clear the rows of a boundary tile that are not keys of the range
+      const int k0 = base + i * kUmKeys;
+      if (k0 < start || k0 + kUmKeys > end) {
+        const int lo = max(start - k0, 0), hi = min(end - k0, kUmKeys), r = tid >> 1;
+        mbar_wait_bounded(&full_bar[f_stage], f_phase, abort_flag, kStatusAttnTimeout);
+        if (r < lo || r >= hi)
+          for (int c = 0; c < subs_loaded; ++c) {
+            uint8_t* t = smem + f_stage * stage_bytes + c * kSubBytes + r * 128 + (tid & 1) * 64;
+#pragma unroll
+            for (int q = 0; q < 4; ++q) *reinterpret_cast<uint4*>(t + q * 16) = make_uint4(0, 0, 0, 0);
+          }
+        fence_proxy_async_smem();
+        mbar_arrive(&patched[patches++]);
+      }
+      if (++f_stage == stages) {
+        f_stage = 0;
+        f_phase ^= 1;
+      }
+    };
+    // where this key's weights go: 2 bytes in row n of a buffer, its 16-byte pieces swizzled
+    const uint32_t p_addr = smem_u32(p_s) + (mine & 7) * 2;
+    const int piece = mine >> 3;
+    patch(0);
+    for (int i = 0; i < n_tiles; ++i) {
+      if (stages > 1 && i + 1 < n_tiles) patch(i + 1);
+      mbar_wait_bounded(&s_full[i & 1], (i >> 1) & 1, abort_flag, kStatusAttnTimeout);
+      tcgen05_fence_after_sync();
+      const int key0 = base + i * kUmKeys, key = key0 + mine;
+      uint32_t raw[N];
+#pragma unroll
+      for (int n0 = 0; n0 < N; n0 += 16)
+        tmem_ld_32x32b_x16(tmem + (i & 1) * N + n0 + lanes, *reinterpret_cast<uint32_t(*)[16]>(raw + n0));
+      tmem_ld_wait();
+      float x[N];
+#pragma unroll
+      for (int n = 0; n < N; ++n) x[n] = owner ? __uint_as_float(raw[n]) * scale_log2 : -INFINITY;
+      if (key0 < all_lo || key0 + kUmKeys - 1 > all_hi) {
+#pragma unroll
+        for (int n = 0; n < N; ++n) x[n] = key >= lo_s[n] && key <= hi_s[n] ? x[n] : -INFINITY;
+      }
+      float over[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};  // how far a score exceeds its row's reference
+#pragma unroll
+      for (int n = 0; n < N; ++n) over[n & 3] = fmaxf(over[n & 3], x[n] - m[n]);  // (-inf less -inf: NaN, which fmaxf drops)
+      if (group_any(fmaxf(fmaxf(over[0], over[1]), fmaxf(over[2], over[3])) > kGrow)) {
+        // New references: the column maxima cross the warp by redux and the warps through shared memory.
+#pragma unroll
+        for (int n0 = 0; n0 < N; n0 += 32) {
+          float best = -INFINITY;
+#pragma unroll
+          for (int n = 0; n < (N < 32 ? N : 32); ++n) {
+            const float c = warp_redux_max(x[n0 + n]);
+            if (lane == n) best = c;
+          }
+          if (N >= 32 || lane < N) red[warp * N + n0 + lane] = best;
+        }
+        group_sync();
+        if (tid < N) {
+          const float m_old = m_s[tid];
+          const float m_new = fmaxf(m_old, fmaxf(fmaxf(red[tid], red[N + tid]), fmaxf(red[2 * N + tid], red[3 * N + tid])));
+          al_s[tid] = m_new == -INFINITY ? 1.f : exp2f(m_old - m_new);
+          m_s[tid] = m_new;
+        }
+        group_sync();
+        if (i > 0) {
+          mbar_wait_bounded(&pv_done[(i - 1) & 1], ((i - 1) >> 1) & 1, abort_flag, kStatusAttnTimeout);  // O is at rest
+          tcgen05_fence_after_sync();
+#pragma unroll 1
+          for (int c = 0; c < m_tiles * 2 * N; c += 16) {
+            uint32_t r[16];
+            tmem_ld_32x32b_x16(tmem_o + c + lanes, r);
+            tmem_ld_wait();
+#pragma unroll
+            for (int n = 0; n < 16; ++n) r[n] = __float_as_uint(__uint_as_float(r[n]) * al_s[(c & (N - 1)) + n]);
+            tmem_st_32x32b_x16(tmem_o + c + lanes, r);
+          }
+          tmem_st_wait();
+        }
+#pragma unroll
+        for (int n = 0; n < N; ++n) {
+          l_part[n] *= al_s[n];
+          m[n] = m_s[n];
+        }
+      }
+      // this key's weights: two bf16 terms each, into rows n and N + n
+      if (i > 1) mbar_wait_bounded(&pv_done[i & 1], ((i - 2) >> 1) & 1, abort_flag, kStatusAttnTimeout);  // the buffer is free
+      if (owner) {
+        const uint32_t dst = p_addr + (i & 1) * U::kPBytes;
+#pragma unroll
+        for (int n = 0; n < N; ++n) {
+          const float p = exp2_approx(fmaxf(x[n] - m[n], -1000.f));  // (a row without a key so far: NaN -> 0)
+          l_part[n] += p;
+          const __nv_bfloat16 hi = __float2bfloat16_rn(p), lo = __float2bfloat16_rn(p - __bfloat162float(hi));
+          const uint32_t at = dst + n * 128 + ((piece ^ (n & 7)) << 4);
+          asm volatile("st.shared.u16 [%0], %1;" ::"r"(at), "h"(__bfloat16_as_ushort(hi)));
+          asm volatile("st.shared.u16 [%0], %1;" ::"r"(at + N * 128), "h"(__bfloat16_as_ushort(lo)));
+        }
+      }
+      fence_proxy_async_smem();
+      tcgen05_fence_before_sync();
+      mbar_arrive(&p_ready[i & 1]);
+      if (stages == 1 && i + 1 < n_tiles) patch(i + 1);
+    }
+    // ---- row sums, output factors, output ----
+#pragma unroll
+    for (int n0 = 0; n0 < N; n0 += 32) {
+      float best = 0.f;
+#pragma unroll
+      for (int n = 0; n < (N < 32 ? N : 32); ++n) {
+        const float l = warp_sum(l_part[n0 + n]);
+        if (lane == n) best = l;
+      }
+      if (N >= 32 || lane < N) red[warp * N + n0 + lane] = best;
+    }
+    group_sync();
+    const int64_t pair0 = static_cast<int64_t>(tok0) * a.heads + sub * N;  // token * heads + head of row 0
+    if (tid < q_rows) {
+      const float l = (red[tid] + red[N + tid]) + (red[2 * N + tid] + red[3 * N + tid]);
+      const float inv = l > 0.f ? 1.f / l : 0.f;
+      const int64_t pair = pair0 + tid;
+      if (a.num_splits > 1) {
+        al_s[tid] = inv;
+        a.workspace[static_cast<int64_t>(a.num_tokens) * a.heads * a.num_splits * a.kv_rank + pair * a.num_splits + split] =
+            l > 0.f ? m_s[tid] + log2f(l) : -INFINITY;
+      } else {
+        al_s[tid] = inv * gate_of<__nv_bfloat16>(a, pair / a.heads, static_cast<int>(pair % a.heads));
+      }
+    }
+    group_sync();
+    mbar_wait_bounded(&pv_done[(n_tiles - 1) & 1], ((n_tiles - 1) >> 1) & 1, abort_flag, kStatusAttnTimeout);
+    tcgen05_fence_after_sync();
+#pragma unroll 1
+    for (int j = 0; j < m_tiles; ++j) {
+      const int ch = j * 128 + tid;
+#pragma unroll 1
+      for (int n0 = 0; n0 < N; n0 += 16) {
+        if (n0 >= q_rows) break;
+        uint32_t r[16], q[16];
+        tmem_ld_32x32b_x16(tmem_o + j * 2 * N + n0 + lanes, r);
+        tmem_ld_32x32b_x16(tmem_o + j * 2 * N + N + n0 + lanes, q);
+        tmem_ld_wait();
+        if (ch < a.kv_rank) {
+#pragma unroll
+          for (int n = 0; n < 16; ++n) {
+            if (n0 + n >= q_rows) break;
+            const float o = (__uint_as_float(r[n]) + __uint_as_float(q[n])) * al_s[n0 + n];
+            const int64_t pair = pair0 + n0 + n;
+            if (a.num_splits > 1)
+              a.workspace[(pair * a.num_splits + split) * a.kv_rank + ch] = o;
+            else
+              static_cast<__nv_bfloat16*>(a.out)[pair * a.kv_rank + ch] = __float2bfloat16_rn(o);
+          }
+        }
+      }
+    }
+    tcgen05_fence_before_sync();
+  }
+  __syncthreads();
+  if (warp == 0) tmem_dealloc(tmem, tmem_cols);
+}
+
 // One CTA per (token, head): merge the splits' normalised partial outputs by their log-sum-exp.
 __global__ void __launch_bounds__(128)
 latent_combine_kernel(b200_latent_args a) {
@@ -847,48 +940,56 @@ static bool valid_common(const b200_latent_args* a) {
 
 constexpr int kMaxSmem = 227 * 1024;
 
-// Key stages that fit one CTA (0: the block of query rows itself does not fit).
-template <int MT>
-static int stages_for(int row_width) {
-  const int rs = row_width + 8;
-  const int left = kMaxSmem - Shape<MT>::fixed_bytes(rs);
-  const int n = left / Shape<MT>::stage_bytes(rs);
-  return n < 2 ? 0 : (n > kMaxStages ? kMaxStages : n);
+// The pool as rows x row_width, fetched 64 columns x `keys` rows at a time (columns past the row read as zeros).
+static const CUtensorMap* pool_map(const b200_latent_args& a, int keys) {
+  const uint64_t dims[2] = {static_cast<uint64_t>(a.row_width), static_cast<uint64_t>(a.num_chunks) * a.chunk_size};
+  const uint64_t strides[1] = {static_cast<uint64_t>(a.row_width) * 2};
+  const uint32_t box[2] = {64, static_cast<uint32_t>(keys)};
+  return get_tensor_map(a.pool, 2, dims, strides, box, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B);
 }
 
-template <int MT, int KVT>
-static int launch_mma(const b200_latent_args& a, cudaStream_t s) {
-  const int rs = a.row_width + 8;
-  // enough stages to hide the fetch, but no more than lets a second CTA onto the SM where two would fit
-  int stages = stages_for<MT>(a.row_width);
-  const int two = (kMaxSmem / 2 - 1024 - Shape<MT>::fixed_bytes(rs)) / Shape<MT>::stage_bytes(rs);
-  if (two >= 2) stages = two > kMaxStages ? kMaxStages : two;
-  const int bytes = Shape<MT>::fixed_bytes(rs) + stages * Shape<MT>::stage_bytes(rs);
+template <int N>
+static int umma_stages(const b200_latent_args& a) {  // 0: does not fit
+  const int m_tiles = (a.kv_pad + 127) / 128;
+  if (2 * N + m_tiles * 2 * N > 512 || a.chunk_size % kUmKeys != 0) return 0;
+  for (int stages = kUmMaxStages; stages >= 1; --stages)
+    if (UmmaShape<N>::bytes(a.row_width, a.kv_pad, stages) <= kMaxSmem) return stages;
+  return 0;
+}
+template <int N>
+static int launch_umma(const b200_latent_args& a, cudaStream_t s) {
+  const int stages = umma_stages<N>(a);
+  const CUtensorMap* map = pool_map(a, kUmKeys);
+  if (!map) return B200_ERR_DRIVER;
+  const int need = 2 * N + (a.kv_pad + 127) / 128 * 2 * N;
+  int cols = 32;
+  while (cols < need) cols *= 2;
   static std::atomic<uint64_t> done{0};
-  if (ensure_dynamic_smem(latent_mma_kernel<MT, KVT>, kMaxSmem, done) != B200_OK) return B200_ERR_LAUNCH;
+  if (ensure_dynamic_smem(latent_umma_kernel<N>, kMaxSmem, done) != B200_OK) return B200_ERR_LAUNCH;
   const int q_tokens = a.units ? a.unit_tokens : 1;
-  const dim3 grid(a.units ? a.num_units : a.num_tokens, (q_tokens * a.heads + MT - 1) / MT, a.num_splits);
-  const int rc = launch_pdl(latent_mma_kernel<MT, KVT>, grid, dim3(kThreads), bytes, s, a, stages);
+  const dim3 grid(a.units ? a.num_units : a.num_tokens, (q_tokens * a.heads + N - 1) / N, a.num_splits);
+  const int rc = launch_pdl(latent_umma_kernel<N>, grid, dim3(kUmThreads), UmmaShape<N>::bytes(a.row_width, a.kv_pad, stages), s, *map,
+                            a, stages, cols);
   if (rc != B200_OK || a.num_splits == 1) return rc;
   return launch_pdl(latent_combine_kernel, dim3(a.num_tokens * a.heads), dim3(128), 0, s, a);
 }
 
 // Whether the decode kernel takes this call, and its launch.
-template <int RG, int KVT>
+template <int KVT>
 static bool decode_fits(const b200_latent_args& a) {
-  return !a.units && a.heads <= 16 * RG && a.kv_pad <= KVT && a.row_width <= DecodeShape<RG, KVT>::kMaxWidth;
+  return !a.units && a.heads <= 16 && a.kv_pad <= KVT && a.row_width <= DecodeShape<KVT>::kMaxWidth;
 }
-template <int RG, int KVT>
+template <int KVT>
 static int launch_decode(const b200_latent_args& a, cudaStream_t s) {
-  using D = DecodeShape<RG, KVT>;
+  using D = DecodeShape<KVT>;
   const int rs = a.row_width + 8;
   auto fit = [&](int budget) { return (budget - D::fixed_bytes()) / D::stage_bytes(rs); };
   int stages = fit(kMaxSmem / 2 - 1024);  // two CTAs per SM
   if (stages < 2) stages = fit(kMaxSmem);
   stages = stages > kMaxStages ? kMaxStages : stages;
   static std::atomic<uint64_t> done{0};
-  if (ensure_dynamic_smem(latent_decode_kernel<RG, KVT>, kMaxSmem, done) != B200_OK) return B200_ERR_LAUNCH;
-  const int rc = launch_pdl(latent_decode_kernel<RG, KVT>, dim3(a.num_tokens, 1, a.num_splits), dim3(kThreads),
+  if (ensure_dynamic_smem(latent_decode_kernel<KVT>, kMaxSmem, done) != B200_OK) return B200_ERR_LAUNCH;
+  const int rc = launch_pdl(latent_decode_kernel<KVT>, dim3(a.num_tokens, 1, a.num_splits), dim3(kThreads),
                             D::fixed_bytes() + stages * D::stage_bytes(rs), s, a, stages);
   if (rc != B200_OK || a.num_splits == 1) return rc;
   return launch_pdl(latent_combine_kernel, dim3(a.num_tokens * a.heads), dim3(128), 0, s, a);
@@ -928,20 +1029,15 @@ int b200_latent_attention(const b200_latent_args* a, b200_stream_t stream) {
   }
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const int pairs = (a->units ? a->unit_tokens : 1) * a->heads;
-  const int mt = pairs <= 16 ? 16 : (pairs <= 32 ? 32 : 64);
-  const int fit = mt == 16 ? stages_for<16>(a->row_width) : (mt == 32 ? stages_for<32>(a->row_width) : stages_for<64>(a->row_width));
-  if (a->dtype == B200_DTYPE_BF16 && a->kv_pad <= 512 && fit > 0) {
+  if (a->dtype == B200_DTYPE_BF16) {
     if (a->num_splits > 1 &&
         (!a->workspace || a->workspace_bytes < b200_latent_attention_workspace_bytes(a->num_tokens, a->heads, a->kv_rank, a->num_splits)))
       return B200_ERR_WORKSPACE;
-    if (decode_fits<1, 256>(*a)) return launch_decode<1, 256>(*a, s);
-    if (decode_fits<1, 512>(*a)) return launch_decode<1, 512>(*a, s);
-    if (decode_fits<2, 256>(*a)) return launch_decode<2, 256>(*a, s);
-    if (decode_fits<2, 512>(*a)) return launch_decode<2, 512>(*a, s);
-    const bool wide = a->kv_pad > 256;
-    if (mt == 16) return wide ? launch_mma<16, 512>(*a, s) : launch_mma<16, 256>(*a, s);
-    if (mt == 32) return wide ? launch_mma<32, 512>(*a, s) : launch_mma<32, 256>(*a, s);
-    return wide ? launch_mma<64, 512>(*a, s) : launch_mma<64, 256>(*a, s);
+    if (decode_fits<256>(*a)) return launch_decode<256>(*a, s);
+    if (decode_fits<512>(*a)) return launch_decode<512>(*a, s);
+    if (pairs > 32 && umma_stages<64>(*a) > 1) return launch_umma<64>(*a, s);
+    if (pairs > 16 && umma_stages<32>(*a) > 1) return launch_umma<32>(*a, s);
+    if (umma_stages<16>(*a) > 0) return launch_umma<16>(*a, s);
   }
   if (a->kv_rank > kSimtThreads * kSimtMaxCols || a->row_width > 8192) return B200_ERR_INVALID_ARGUMENT;
   const dim3 grid(a->units ? a->num_units * a->unit_tokens : a->num_tokens, a->heads);

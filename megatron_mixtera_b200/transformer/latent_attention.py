@@ -17,7 +17,7 @@ def choose_latent_splits(num_rows: int, heads: int, window, max_sequence_length:
     """Key splits of a decode row: a function of capture-time constants.  The fewest splits that fill the CTAs the GPU holds
     at once to 85 % (else the best there is), none below 256 keys at the longest visible range."""
     slots = _sm_count() * (2 if heads <= 16 else 1)
-    blocks = max(1, num_rows * -(-heads // 64))
+    blocks = max(1, num_rows * (1 if heads <= 32 else -(-heads // 32)))
     keys = max_sequence_length if window is None else min(window, max_sequence_length)
     best, best_fill = 1, 0.0
     for splits in range(1, max(1, min(keys // 256, 64)) + 1):

@@ -539,10 +539,28 @@ typedef struct b200_latent_args {
   int32_t window; /* <= 0: unlimited */
   int32_t num_units, unit_tokens, num_splits, dtype;
   float scale, eps;
+  /* q_full rows as b200_latent_append writes them: elements per head and where the rotated part starts (row_width and
+   * kv_pad for the absorbed form; a rotated part alone for the expanded one). */
+  int32_t q_stride, q_rot_at;
+  /* Expanded form (prompts): keys and values spelled out per head for the keys a step's queries see, E of them in all. */
+  const int32_t* cu_tokens; /* [rows + 1]: a row's query tokens */
+  const int32_t* cu_keys;   /* [rows + 1]: a row's expanded keys */
+  const int32_t* key_start; /* [rows]: position of a row's first expanded key */
+  void* key_rows;           /* [E][row_width]: the cached rows, in key order */
+  const void* key_values;   /* [E][heads * (dim + vdim)]: W_uk c of all heads, then W_uv c of all heads */
+  int32_t num_rows, num_keys, max_row_tokens, vdim;
 } b200_latent_args;
+/* b200_latent_gather: key_rows[e] = the pool row of expanded key e.
+ * b200_latent_prompt_attention: out[t][head][vdim] = sigmoid(gate) * sum_j softmax(scale * (q . k_j + q_rot . k_rot_j)) v_j, the same
+ *   attention on the expanded keys and values: several times fewer products per (query, key) than the absorbed form, worth
+ *   it where the expansion serves many queries.  bf16; dim, vdim, rot_dim multiples of 8, dim and rot_dim rounded up to 16 at
+ *   most 192 together, vdim at most 128 (b200_latent_prompt_supported). */
 size_t b200_latent_attention_workspace_bytes(int num_tokens, int heads, int kv_rank, int num_splits);
 int b200_latent_append(const b200_latent_args* args, b200_stream_t stream);
 int b200_latent_attention(const b200_latent_args* args, b200_stream_t stream);
+int b200_latent_prompt_supported(int dim, int rot_dim, int vdim, int heads);
+int b200_latent_gather(const b200_latent_args* args, b200_stream_t stream);
+int b200_latent_prompt_attention(const b200_latent_args* args, b200_stream_t stream);
 
 /* Generalized delta rule.  Per head, with w = exp(-decay_scale * sigmoid(z + decay_bias)), a = sigmoid(x_a + removal_bias),
  * u = k / sqrt(sum k^2 + unit_eps):   S <- diag(w) S - (a u)(u^T S) + k v^T,   o = S^T r,

@@ -81,6 +81,9 @@ EXPORTED_SYMBOLS = (
     "b200_latent_attention_workspace_bytes",
     "b200_latent_append",
     "b200_latent_attention",
+    "b200_latent_prompt_supported",
+    "b200_latent_gather",
+    "b200_latent_prompt_attention",
     "b200_delta_decode",
     "b200_delta_lora",
     "b200_delta_scan",
@@ -148,7 +151,9 @@ class LatentArgs(ctypes.Structure):
         (n, c_int32) for n in (
             "dkv_offset", "gate_offset", "num_tokens", "heads", "dim", "rot_dim", "rot_dims", "kv_rank", "kv_pad", "row_width",
             "num_chunks", "chunk_size", "max_chunks_per_row", "max_positions", "window", "num_units", "unit_tokens",
-            "num_splits", "dtype")] + [("scale", c_float), ("eps", c_float)]
+            "num_splits", "dtype")] + [("scale", c_float), ("eps", c_float), ("q_stride", c_int32), ("q_rot_at", c_int32)] + [
+        (n, c_void_p) for n in ("cu_tokens", "cu_keys", "key_start", "key_rows", "key_values")] + [
+        (n, c_int32) for n in ("num_rows", "num_keys", "max_row_tokens", "vdim")]
 
 
 class DeltaArgs(ctypes.Structure):
@@ -316,7 +321,8 @@ def load() -> ctypes.CDLL:
     lib.b200_out_norm.argtypes = [POINTER(OutNormArgs), c_void_p]
     lib.b200_latent_attention_workspace_bytes.restype = c_size_t
     lib.b200_latent_attention_workspace_bytes.argtypes = [c_int, c_int, c_int, c_int]
-    for name in ("b200_latent_append", "b200_latent_attention"):
+    lib.b200_latent_prompt_supported.argtypes = [c_int, c_int, c_int, c_int]
+    for name in ("b200_latent_append", "b200_latent_attention", "b200_latent_gather", "b200_latent_prompt_attention"):
         getattr(lib, name).argtypes = [POINTER(LatentArgs), c_void_p]
     for name in ("b200_delta_decode", "b200_delta_lora", "b200_delta_scan", "b200_delta_finish"):
         getattr(lib, name).argtypes = [POINTER(DeltaArgs), c_void_p]

@@ -14,6 +14,9 @@
 //                          mbarrier).  Eight consumer warps split S = Q R^T by key half and by quarter of row_width - a warp's
 //                          part of Q stays in registers - add the quarters through shared memory, do the softmax two rows per
 //                          warp, and split O += P C by columns.  Bound by reading the rows once.
+//   latent_prompt_kernel   bf16 prompts on expanded keys and values (latent_gather_kernel, then one GEMM with W_uk and W_uv): one CTA
+//                          per (64 queries, head), FlashAttention-style with mma.sync and everything of a query row in
+//                          registers.  For steps whose keys are mostly their own tokens.
 //   latent_simt_kernel     any type and size, fp32 arithmetic throughout: the 32-bit mode and shapes the others do not take.
 //   latent_combine_kernel  merges the key splits of decode rows.
 //
@@ -75,19 +78,19 @@ latent_append_kernel(b200_latent_args a) {
   const int rot_pairs = (a.row_width - a.kv_pad) / 2;
 
   // queries
-  T* qf = static_cast<T*>(a.q_full) + t * a.heads * a.row_width;
+  T* qf = static_cast<T*>(a.q_full) + t * a.heads * a.q_stride;
   const int qd = a.dim + a.rot_dim;
   for (int idx = tid; idx < a.heads * rot_pairs; idx += kAppendThreads) {
     const int h = idx / rot_pairs, i = idx - h * rot_pairs;
     float u, v;
     rotated_pair(a, row + h * qd + a.dim, cs, sn, i, u, v);
-    T* dst = qf + h * a.row_width + a.kv_pad + 2 * i;
+    T* dst = qf + h * a.q_stride + a.q_rot_at + 2 * i;
     simt::store_as(dst, u);
     simt::store_as(dst + 1, v);
   }
-  const int lat_pad = a.kv_pad - a.kv_rank;
+  const int lat_pad = a.q_rot_at > 0 ? a.kv_pad - a.kv_rank : 0;
   for (int idx = tid; idx < a.heads * lat_pad; idx += kAppendThreads)
-    simt::store_as(qf + (idx / lat_pad) * a.row_width + a.kv_rank + idx % lat_pad, 0.f);
+    simt::store_as(qf + (idx / lat_pad) * a.q_stride + a.kv_rank + idx % lat_pad, 0.f);
   if (a.dkv_offset < 0) return;
 
   // this token's pool row
@@ -856,6 +859,228 @@ latent_combine_kernel(b200_latent_args a) {
 }
 
 // ---------------------------------------------------------------------------------------------------------------
+// Prompts on expanded keys and values
+// ---------------------------------------------------------------------------------------------------------------
+// One warp per expanded key: its pool row, 16 bytes a lane at a time.
+__global__ void __launch_bounds__(256)
+latent_gather_kernel(b200_latent_args a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int e = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (e >= a.num_keys) return;
+  int lo = 0, hi = a.num_rows - 1;  // the row with cu_keys[row] <= e < cu_keys[row + 1]
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) >> 1;
+    if (a.cu_keys[mid] <= e) lo = mid; else hi = mid - 1;
+  }
+  const int key = a.key_start[lo] + e - a.cu_keys[lo];
+  const int32_t* bt = a.block_table + static_cast<int64_t>(lo) * a.max_chunks_per_row;
+  const uint4* src = reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(a.pool) + pool_row(a, bt, key) * a.row_width);
+  uint4* dst = reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(a.key_rows) + static_cast<int64_t>(e) * a.row_width);
+  for (int c = lane; c < a.row_width / 8; c += 32) dst[c] = src[c];
+}
+
+constexpr int kPrQueries = 64;
+constexpr int kPrKeys = 64;
+constexpr int kPrThreads = 128;
+constexpr int kPrSteps = 12;    // 16-wide steps of (dim, rot_dim), each rounded up to 16
+constexpr int kPrMaxV = 128;
+
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool valid) {  // invalid: 16 bytes of zeros
+  const int n = valid ? 16 : 0;
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(n) : "memory");
+}
+
+__global__ void __launch_bounds__(kPrThreads, 2)
+latent_prompt_kernel(b200_latent_args a) {
+  extern __shared__ __align__(128) uint8_t smem[];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gid = lane >> 2, tig = lane & 3;
+  const int row = blockIdx.y, head = blockIdx.z;
+  pdl_launch_dependents();
+  const int t_begin = a.cu_tokens[row], n_tok = a.cu_tokens[row + 1] - t_begin;
+  const int q0 = (gridDim.x - 1 - blockIdx.x) * kPrQueries;  // the blocks with the most keys start first
+  const int e_begin = a.cu_keys[row], key_begin = a.key_start[row];
+  pdl_wait();
+  if (q0 >= n_tok) return;
+  const int n_q = min(kPrQueries, n_tok - q0);
+  const int pos0 = key_begin + (a.cu_keys[row + 1] - e_begin) - n_tok + q0;  // position of query q0: the newest keys are the row's tokens
+  const int start = max(window_start(pos0, a.window), key_begin), end = pos0 + n_q;
+  const int n_tiles = (end - start + kPrKeys - 1) / kPrKeys;
+
+  const int dp = (a.dim + 15) / 16 * 16, rp = (a.rot_dim + 15) / 16 * 16, steps = (dp + rp) / 16;
+  const int vp = (a.vdim + 15) / 16 * 16;
+  const int ks = dp + rp + 8, vs = vp + 8;  // row strides: odd numbers of 16-byte pieces
+  __nv_bfloat16* k_s = reinterpret_cast<__nv_bfloat16*>(smem);  // [2][keys][ks]
+  __nv_bfloat16* v_s = k_s + 2 * kPrKeys * ks;                  // [2][keys][vs]
+  __nv_bfloat16* q_s = v_s + 2 * kPrKeys * vs;                  // [queries][ks]
+
+  const int kv_ld = a.heads * (a.dim + a.vdim), rot_w = a.row_width - a.kv_pad;
+  const __nv_bfloat16* kv = static_cast<const __nv_bfloat16*>(a.key_values);
+  const __nv_bfloat16* rows = static_cast<const __nv_bfloat16*>(a.key_rows);
+  const int d8 = dp / 8, r8 = rp / 8, v8 = vp / 8, pieces = d8 + r8 + v8;
+  auto load = [&](int i) {
+    __nv_bfloat16* kd = k_s + (i & 1) * kPrKeys * ks;
+    __nv_bfloat16* vd = v_s + (i & 1) * kPrKeys * vs;
+    for (int x = tid; x < kPrKeys * pieces; x += kPrThreads) {
+      const int r = x / pieces, c = x - r * pieces;
+      const int key = start + i * kPrKeys + r;
+      const bool in = key < end;
+      const int64_t e = e_begin + (in ? key - key_begin : 0);
+      if (c < d8) {
+        cp_async16(smem_u32(kd + r * ks + c * 8), kv + e * kv_ld + head * a.dim + c * 8, in && c * 8 < a.dim);
+      } else if (c < d8 + r8) {
+        const int p = c - d8;
+        cp_async16(smem_u32(kd + r * ks + dp + p * 8), rows + e * a.row_width + a.kv_pad + p * 8, in && p * 8 < rot_w);
+      } else {
+        const int p = c - d8 - r8;
+        cp_async16(smem_u32(vd + r * vs + p * 8), kv + e * kv_ld + a.heads * a.dim + head * a.vdim + p * 8, in && p * 8 < a.vdim);
+      }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  {
+    const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(a.proj);
+    const __nv_bfloat16* qr = static_cast<const __nv_bfloat16*>(a.q_full);
+    for (int x = tid; x < kPrQueries * (d8 + r8); x += kPrThreads) {
+      const int r = x / (d8 + r8), c = x - r * (d8 + r8);
+      const int64_t t = t_begin + q0 + min(r, n_q - 1);
+      if (c < d8)
+        cp_async16(smem_u32(q_s + r * ks + c * 8), q + t * a.proj_ld + head * (a.dim + a.rot_dim) + c * 8, r < n_q && c * 8 < a.dim);
+      else
+        cp_async16(smem_u32(q_s + r * ks + dp + (c - d8) * 8), qr + (t * a.heads + head) * a.q_stride + a.q_rot_at + (c - d8) * 8,
+                   r < n_q && (c - d8) * 8 < rot_w);
+    }
+  }
+  load(0);
+  asm volatile("cp.async.wait_all;" ::: "memory");
+  __syncthreads();
+  uint32_t qf[kPrSteps][4];
+#pragma unroll
+  for (int s = 0; s < kPrSteps; ++s)
+    if (s < steps)
+      ldmatrix_x4(smem_u32(q_s + (warp * 16 + (lane & 15)) * ks + s * 16 + (lane >> 4) * 8), qf[s][0], qf[s][1], qf[s][2], qf[s][3]);
+  int lo[2], hi[2];  // visible keys of this thread's two queries
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    const int i = warp * 16 + gid + r * 8, pos = pos0 + i;
+    hi[r] = i < n_q ? pos : -1;
+    lo[r] = window_start(pos, a.window);
+  }
+  const int w_first = pos0 + warp * 16, w_last = min(w_first + 15, pos0 + n_q - 1);  // this warp's queries
+  const float scale_log2 = a.scale * kLog2e;
+  float o[kPrMaxV / 8][4];
+#pragma unroll
+  for (int j = 0; j < kPrMaxV / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+  float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
+
+  for (int i = 0; i < n_tiles; ++i) {
+    if (i + 1 < n_tiles) load(i + 1);
+    const int key0 = start + i * kPrKeys;
+    // tiles this warp's queries cannot see (the others' may): nothing to do
+    const bool any = warp * 16 < n_q && key0 <= w_last && key0 + kPrKeys > window_start(w_first, a.window);
+    if (any) {
+      const uint32_t kb = smem_u32(k_s + (i & 1) * kPrKeys * ks), vb = smem_u32(v_s + (i & 1) * kPrKeys * vs);
+      float sc[8][4];
+#pragma unroll
+      for (int n = 0; n < 8; ++n) sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.f;
+#pragma unroll
+      for (int s = 0; s < kPrSteps; ++s) {
+        if (s < steps) {
+#pragma unroll
+          for (int n = 0; n < 4; ++n) {
+            uint32_t b0, b1, b2, b3;
+            ldmatrix_x4(kb + ((n * 16 + ((lane >> 4) << 3) + (lane & 7)) * ks + s * 16 + ((lane >> 3) & 1) * 8) * 2, b0, b1, b2, b3);
+            mma_bf16_16816(sc[2 * n], qf[s], b0, b1);
+            mma_bf16_16816(sc[2 * n + 1], qf[s], b2, b3);
+          }
+        }
+      }
+      const bool whole = key0 + kPrKeys - 1 <= w_first && key0 >= window_start(w_last, a.window) && warp * 16 + 16 <= n_q;
+      float mx[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+      for (int n = 0; n < 8; ++n)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          const int key = key0 + n * 8 + tig * 2 + (c & 1), r = c >> 1;
+          const float v = whole || (key >= lo[r] && key <= hi[r]) ? sc[n][c] * scale_log2 : -INFINITY;
+          sc[n][c] = v;
+          mx[r] = fmaxf(mx[r], v);
+        }
+      float m_use[2], alpha[2];
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
+        mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
+        const float m_new = fmaxf(m_run[r], mx[r]);
+        m_use[r] = m_new == -INFINITY ? 0.f : m_new;
+        alpha[r] = exp2_approx(m_run[r] - m_use[r]);
+        m_run[r] = m_new;
+        l_run[r] *= alpha[r];
+      }
+      if (__any_sync(0xffffffffu, alpha[0] != 1.f || alpha[1] != 1.f)) {
+#pragma unroll
+        for (int j = 0; j < kPrMaxV / 8; ++j) {
+          o[j][0] *= alpha[0];
+          o[j][1] *= alpha[0];
+          o[j][2] *= alpha[1];
+          o[j][3] *= alpha[1];
+        }
+      }
+#pragma unroll
+      for (int kk = 0; kk < kPrKeys / 16; ++kk) {
+        // the accumulator layout of two 8-key columns is the A operand of one 16-key step; weights as hi + lo terms
+        uint32_t ph[4], pl[4];
+#pragma unroll
+        for (int h = 0; h < 2; ++h)
+#pragma unroll
+          for (int r = 0; r < 2; ++r) {
+            const float p0 = exp2_approx(sc[2 * kk + h][2 * r] - m_use[r]), p1 = exp2_approx(sc[2 * kk + h][2 * r + 1] - m_use[r]);
+            l_run[r] += p0 + p1;
+            const float h0 = bf16_round(p0), h1 = bf16_round(p1);
+            ph[h * 2 + r] = pack_bf16x2(h0, h1);
+            pl[h * 2 + r] = pack_bf16x2(p0 - h0, p1 - h1);
+          }
+#pragma unroll
+        for (int j = 0; j < kPrMaxV / 16; ++j) {
+          if (j * 16 < vp) {
+            uint32_t b0, b1, b2, b3;
+            ldmatrix_x4_trans(vb + ((kk * 16 + (((lane >> 3) & 1) << 3) + (lane & 7)) * vs + j * 16 + (lane >> 4) * 8) * 2, b0, b1, b2, b3);
+            mma_bf16_16816(o[2 * j], ph, b0, b1);
+            mma_bf16_16816(o[2 * j + 1], ph, b2, b3);
+            mma_bf16_16816(o[2 * j], pl, b0, b1);
+            mma_bf16_16816(o[2 * j + 1], pl, b2, b3);
+          }
+        }
+      }
+    }
+    asm volatile("cp.async.wait_all;" ::: "memory");
+    __syncthreads();  // the next tile is there, this one has been read
+  }
+
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    float l = l_run[r];
+    l += __shfl_xor_sync(0xffffffffu, l, 1);
+    l += __shfl_xor_sync(0xffffffffu, l, 2);
+    const int q = warp * 16 + gid + r * 8;
+    if (q >= n_q) continue;
+    const int64_t t = t_begin + q0 + q;
+    const float g = gate_of<__nv_bfloat16>(a, t, head) / l;
+    __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(a.out) + (t * a.heads + head) * a.vdim;
+#pragma unroll
+    for (int j = 0; j < kPrMaxV / 8; ++j) {
+      const int col = j * 8 + tig * 2;
+      if (col < a.vdim) *reinterpret_cast<uint32_t*>(dst + col) = pack_bf16x2(o[j][2 * r] * g, o[j][2 * r + 1] * g);
+    }
+  }
+}
+
+static int prompt_smem(int dim, int rot_dim, int vdim) {
+  const int ks = (dim + 15) / 16 * 16 + (rot_dim + 15) / 16 * 16 + 8, vs = (vdim + 15) / 16 * 16 + 8;
+  return (2 * kPrKeys * (ks + vs) + kPrQueries * ks) * 2;
+}
+
+// ---------------------------------------------------------------------------------------------------------------
 // Any type, any size: one CTA per (token, head), 64 keys at a time.
 // ---------------------------------------------------------------------------------------------------------------
 template <typename T>
@@ -1009,6 +1234,8 @@ int b200_latent_append(const b200_latent_args* a, b200_stream_t stream) {
   using namespace b200;
   if (!latent::valid_common(a) || !a->token_to_pos || a->max_positions <= 0 || (a->rot_dims > 0 && (!a->rope_cos || !a->rope_sin)))
     return B200_ERR_INVALID_ARGUMENT;
+  if (a->q_rot_at < 0 || a->q_stride < a->q_rot_at + a->row_width - a->kv_pad || (a->q_rot_at > 0 && a->q_rot_at < a->kv_pad))
+    return B200_ERR_INVALID_ARGUMENT;
   if (a->dkv_offset >= 0 && (!a->norm_weight || !a->token_to_chunk_idx || !a->token_to_local_pos)) return B200_ERR_INVALID_ARGUMENT;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (a->dtype == B200_DTYPE_F32)
@@ -1044,6 +1271,37 @@ int b200_latent_attention(const b200_latent_args* a, b200_stream_t stream) {
   const size_t bytes = static_cast<size_t>(a->row_width) * sizeof(float);
   if (a->dtype == B200_DTYPE_F32) return launch_pdl(latent_simt_kernel<float>, grid, dim3(kSimtThreads), bytes, s, *a);
   return launch_pdl(latent_simt_kernel<__nv_bfloat16>, grid, dim3(kSimtThreads), bytes, s, *a);
+}
+
+int b200_latent_prompt_supported(int dim, int rot_dim, int vdim, int heads) {
+  using namespace b200::latent;
+  return dim > 0 && rot_dim > 0 && vdim > 0 && heads > 0 && heads <= 65535 && dim % 8 == 0 && rot_dim % 8 == 0 && vdim % 8 == 0 &&
+         vdim <= kPrMaxV && (dim + 15) / 16 + (rot_dim + 15) / 16 <= kPrSteps;
+}
+
+int b200_latent_gather(const b200_latent_args* a, b200_stream_t stream) {
+  using namespace b200;
+  if (!latent::valid_common(a) || a->dtype != B200_DTYPE_BF16 || !a->block_table || !a->cu_keys || !a->key_start || !a->key_rows ||
+      a->num_rows <= 0 || a->num_keys <= 0 || a->max_chunks_per_row <= 0 || !aligned16(a->key_rows))
+    return B200_ERR_INVALID_ARGUMENT;
+  return launch_pdl(latent::latent_gather_kernel, dim3((a->num_keys + 7) / 8), dim3(256), 0, reinterpret_cast<cudaStream_t>(stream), *a);
+}
+
+int b200_latent_prompt_attention(const b200_latent_args* a, b200_stream_t stream) {
+  using namespace b200;
+  using namespace b200::latent;
+  if (!valid_common(a) || a->dtype != B200_DTYPE_BF16 || !a->cu_tokens || !a->cu_keys || !a->key_start || !a->key_rows || !a->key_values ||
+      !a->out || a->num_rows <= 0 || a->num_rows > 65535 || a->max_row_tokens <= 0 ||
+      !b200_latent_prompt_supported(a->dim, a->rot_dim, a->vdim, a->heads))
+    return B200_ERR_INVALID_ARGUMENT;
+  if (a->proj_ld % 8 != 0 || a->q_stride % 8 != 0 || a->q_rot_at % 8 != 0 || !aligned16(a->proj) || !aligned16(a->key_rows) ||
+      !aligned16(a->key_values) || a->q_stride < a->q_rot_at + a->row_width - a->kv_pad)
+    return B200_ERR_ALIGNMENT;
+  static std::atomic<uint64_t> done{0};
+  if (ensure_dynamic_smem(latent_prompt_kernel, kMaxSmem, done) != B200_OK) return B200_ERR_LAUNCH;
+  const dim3 grid((a->max_row_tokens + kPrQueries - 1) / kPrQueries, a->num_rows, a->heads);
+  return launch_pdl(latent_prompt_kernel, grid, dim3(kPrThreads), prompt_smem(a->dim, a->rot_dim, a->vdim),
+                    reinterpret_cast<cudaStream_t>(stream), *a);
 }
 
 }  // extern "C"

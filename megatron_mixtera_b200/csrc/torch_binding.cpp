@@ -340,6 +340,10 @@ void hybrid(const Tensor& args, const Tensor& anchor, int64_t which) {
     case 4: ok(b200_delta_lora(struct_of<b200_delta_args>(args, "b200_delta_args"), s), "b200_delta_lora"); break;
     case 5: ok(b200_delta_scan(struct_of<b200_delta_args>(args, "b200_delta_args"), s), "b200_delta_scan"); break;
     case 6: ok(b200_delta_finish(struct_of<b200_delta_args>(args, "b200_delta_args"), s), "b200_delta_finish"); break;
+    case 7: ok(b200_latent_gather(struct_of<b200_latent_args>(args, "b200_latent_args"), s), "b200_latent_gather"); break;
+    case 8:
+      ok(b200_latent_prompt_attention(struct_of<b200_latent_args>(args, "b200_latent_args"), s), "b200_latent_prompt_attention");
+      break;
     default: TORCH_CHECK(false, "b200_decode.hybrid: unknown kernel ", which);
   }
 }

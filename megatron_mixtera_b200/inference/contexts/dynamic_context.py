@@ -492,6 +492,30 @@ class DynamicInferenceContext(BaseInferenceContext):
         """Latent rows ``[chunks, chunk, width]`` of 1-based ``layer_number``."""
         return self.latent_buffers[layer_number - 1]
 
+    def expanded_keys(self, window: Optional[int]):
+        """For attention that spells out the keys of a prompt step: which keys the step's queries see under ``window``.
+        Returns (device int32 ``[2, rows + 1]`` = cumulative key counts, position of a row's first key; total) or None where
+        that does not pay - decode steps, CUDA-graph steps, or more than twice as many keys as query tokens."""
+        if self.is_decode_only() or self.using_cuda_graph_this_step():
+            return None
+        if window not in self._expanded:
+            p, t = self.paused_request_count, self.total_request_count
+            ql = self.request_query_lengths.numpy()[p:t].astype(np.int64)
+            off = self.request_kv_length_offsets.numpy()[p:t].astype(np.int64)
+            first = np.zeros_like(off) if window is None else np.maximum(off - window + 1, 0)
+            counts = off + ql - first
+            total = int(counts.sum())
+            if total > 2 * int(ql.sum()):
+                self._expanded[window] = None
+            else:
+                table = torch.zeros((2, ql.size + 1), dtype=torch.int32, pin_memory=self.device.type == "cuda")
+                table[0, 1:] = torch.from_numpy(np.cumsum(counts))
+                table[1, :-1] = torch.from_numpy(first)
+                self.h2d_bytes += table.numel() * 4
+                self._expanded[window] = (table.to(self.device, non_blocking=True), total, table)  # (the staging copy lives as long)
+        entry = self._expanded[window]
+        return None if entry is None else entry[:2]
+
     def key_value_cache(self, layer_number: int) -> Tuple[Tensor, Tensor, Tensor]:
         """(K pool, V pool, block table) of 1-based ``layer_number`` (reference :547-564)."""
         return (self.memory_buffer[0, layer_number - 1], self.memory_buffer[1, layer_number - 1], self.block_table)
@@ -556,6 +580,7 @@ class DynamicInferenceContext(BaseInferenceContext):
         self.cu_kv_seq_lengths = None
         self.kv_seq_lengths = None
         self.block_table = None
+        self._expanded = {}
 
     def using_cuda_graph_this_step(self) -> bool:
         has = self.cuda_graph_token_counts is not None
@@ -585,6 +610,7 @@ class DynamicInferenceContext(BaseInferenceContext):
 
         graphs = self.using_cuda_graph_this_step()
         decode = self.is_decode_only()
+        self._expanded = {}
         if graphs:
             padded = math.ceil(active_token_count / self.cuda_graph_step_size) * self.cuda_graph_step_size
             padded = min(padded, self.max_requests)

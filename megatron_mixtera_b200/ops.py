@@ -734,7 +734,7 @@ def topp_probs(logits, top_p: float, temperature: float = 1.0):
 # ---------------------------------------------------------------------------------------------------------------------
 _DTYPE = {BF16: 0, F32: 1}
 _ACT = {None: 0, "relu2": 1}
-_OUT_NORM, _LATENT_APPEND, _LATENT_ATTENTION, _DELTA_DECODE, _DELTA_LORA, _DELTA_SCAN, _DELTA_FINISH = range(7)
+_OUT_NORM, _LATENT_APPEND, _LATENT_ATTENTION, _DELTA_DECODE, _DELTA_LORA, _DELTA_SCAN, _DELTA_FINISH, _LATENT_GATHER, _LATENT_PROMPT = range(9)
 
 
 def dtype_code(dtype) -> int:
@@ -834,6 +834,18 @@ def latent_attention(args, anchor) -> None:
         args.workspace, args.workspace_bytes = ws.data_ptr(), ws.numel()
         launch_count += 1  # the split-combine kernel
     _launch("hybrid", _blob(args), anchor, _LATENT_ATTENTION)
+
+
+def latent_prompt_supported(dim: int, rot_dim: int, vdim: int, heads: int) -> bool:
+    return bool(_lib.load().b200_latent_prompt_supported(dim, rot_dim, vdim, heads))
+
+
+def latent_gather(args, anchor) -> None:
+    _launch("hybrid", _blob(args), anchor, _LATENT_GATHER)
+
+
+def latent_prompt_attention(args, anchor) -> None:
+    _launch("hybrid", _blob(args), anchor, _LATENT_PROMPT)
 
 
 def delta_decode(args, anchor) -> None:

@@ -1,7 +1,9 @@
 """Latent attention: keys and values of all heads come from one small row per token, the only thing cached.
 
-The key matrix is applied to the queries instead of the cached rows ("absorbed") and the value matrix to the attention
-output, both as batched per-head GEMMs, so that prompts and decoding alike read the cached rows once and never expand them.
+Two forms of the same attention.  Absorbed: the key matrix is applied to the queries instead of the cached rows and the value
+matrix to the attention output, both as batched per-head GEMMs; the cached rows are read once and never expanded.  This is
+how decoding runs, and portions of prompts with a long past.  Expanded: one GEMM spells out the keys and values of all heads,
+which costs several times fewer products per (query, key) pair; it pays where most of the keys belong to the step itself.
 """
 from __future__ import annotations
 
@@ -46,8 +48,10 @@ class LatentAttention(torch.nn.Module):
         self.in_width = q_width + down + m.heads
         padded = -(-self.in_width // 8) * 8  # whole 16-byte vectors per row; the added rows are zero
         self.linear_in = ColumnParallelLinear(config.hidden_size, padded, config=config, bias=False)
+        # absorbed: per head [latent][dim]; expanded: [keys of all heads | values of all heads] x latent
         self.key_up = torch.nn.Parameter(torch.empty(m.heads * m.kv_rank, m.dim, dtype=dt, device=dev), requires_grad=False)
-        self.value_up = torch.nn.Parameter(torch.empty(m.heads * m.vdim, m.kv_rank, dtype=dt, device=dev), requires_grad=False)
+        self.key_value_up = torch.nn.Parameter(torch.empty(m.heads * (m.dim + m.vdim), m.kv_rank, dtype=dt, device=dev),
+                                               requires_grad=False)
         if self.owns_rows:
             self.latent_norm = torch.nn.Parameter(torch.ones(m.kv_rank, dtype=dt, device=dev), requires_grad=False)
         else:
@@ -70,17 +74,31 @@ class LatentAttention(torch.nn.Module):
         w.zero_()
         w[: self.in_width].copy_(torch.cat([p.to(w.device) for p in parts]))
         self.key_up.data.copy_(get("uk").view(m.heads, m.dim, m.kv_rank).transpose(1, 2).reshape(m.heads * m.kv_rank, m.dim))
-        self.value_up.data.copy_(get("uv"))
+        self.key_value_up.data.copy_(torch.cat([get("uk"), get("uv")]))
         if self.owns_rows:
             self.latent_norm.data.copy_(get("dkv.norm"))
         self.linear_proj.weight.data.copy_(get("o"))
+
+    @property
+    def value_up(self):
+        return self.key_value_up[self.mixer.heads * self.mixer.dim:]
+
+    expand_prompts = True  # False: the absorbed form everywhere
+
+    def _expansion(self, x, ctx):
+        m = self.mixer
+        if not (self.expand_prompts and x.dtype == torch.bfloat16 and ops.latent_prompt_supported(m.dim, m.rot_dim, m.vdim, m.heads)):
+            return None
+        return ctx.expanded_keys(m.window)
 
     def forward(self, x, ctx, rope):
         """``x`` [T, H] -> the output linear's partial sums."""
         m, T, dev = self.mixer, x.shape[0], x.device
         proj, _ = self.linear_in(x)
-        q_full = torch.empty((T, m.heads, m.row_width), dtype=x.dtype, device=dev)
-        latent_out = torch.empty((T, m.heads * m.kv_rank), dtype=x.dtype, device=dev)
+        expanded = self._expansion(x, ctx)
+        # queries: the absorbed form fills whole rows, the expanded one needs the rotated part alone
+        q_stride, q_rot_at = (m.row_width, m.kv_pad) if expanded is None else (m.row_width - m.kv_pad, 0)
+        q_full = torch.empty((T, m.heads, q_stride), dtype=x.dtype, device=dev)
         pool = ctx.latent_cache(self.cache_layer_number)
         decode = ctx.is_decode_only()
         a = _lib.LatentArgs()
@@ -93,11 +111,26 @@ class LatentAttention(torch.nn.Module):
         a.block_table = ctx.request_to_kv_chunk_ids_cudagraph_only.data_ptr()
         a.max_chunks_per_row = ctx.request_to_kv_chunk_ids_cudagraph_only.shape[1]
         a.pool, a.num_chunks, a.chunk_size = pool.data_ptr(), pool.shape[0], pool.shape[1]
-        a.q_full, a.out = q_full.data_ptr(), latent_out.data_ptr()
+        a.q_full, a.q_stride, a.q_rot_at = q_full.data_ptr(), q_stride, q_rot_at
         a.num_tokens, a.heads, a.dim, a.rot_dim, a.rot_dims = T, m.heads, m.dim, m.rot_dim, m.rot.dims
         a.kv_rank, a.kv_pad, a.row_width = m.kv_rank, m.kv_pad, m.row_width
         a.window, a.scale, a.eps = m.window or 0, m.scale, self.config.layernorm_epsilon
         a.dtype, a.num_splits = ops.dtype_code(x.dtype), 1
+        values = torch.empty((T, m.heads * m.vdim), dtype=x.dtype, device=dev)
+        if expanded is not None:
+            table, num_keys = expanded
+            key_rows = torch.empty((num_keys, m.row_width), dtype=x.dtype, device=dev)
+            ops.latent_append(a, pool)
+            a.num_rows, a.num_keys, a.max_row_tokens, a.vdim = table.shape[1] - 1, num_keys, ctx.max_seqlen_q, m.vdim
+            a.cu_tokens = ctx.cu_query_seq_lengths_cudagraph_only.data_ptr()
+            a.cu_keys, a.key_start, a.key_rows = table[0].data_ptr(), table[1].data_ptr(), key_rows.data_ptr()
+            ops.latent_gather(a, pool)
+            key_values = ops.linear(key_rows, self.key_value_up, K=m.kv_rank)
+            a.key_values, a.out = key_values.data_ptr(), values.data_ptr()
+            ops.latent_prompt_attention(a, pool)
+            return self.linear_proj(values, defer_reduction=True)[0]
+        latent_out = torch.empty((T, m.heads * m.kv_rank), dtype=x.dtype, device=dev)
+        a.out = latent_out.data_ptr()
         if decode:
             a.kv_seq_lengths = ctx.kv_seq_lengths_cudagraph_only.data_ptr()
             if x.dtype == torch.bfloat16:
@@ -108,6 +141,5 @@ class LatentAttention(torch.nn.Module):
         ops.linear(proj, self.key_up, out=q_full.view(T, -1), batch=m.heads, x_batch=m.dim + m.rot_dim, y_batch=m.row_width, K=m.dim)
         ops.latent_append(a, pool)
         ops.latent_attention(a, pool)
-        values = torch.empty((T, m.heads * m.vdim), dtype=x.dtype, device=dev)
         ops.linear(latent_out, self.value_up, out=values, batch=m.heads, x_batch=m.kv_rank, y_batch=m.vdim, K=m.kv_rank)
         return self.linear_proj(values, defer_reduction=True)[0]

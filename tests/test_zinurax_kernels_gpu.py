@@ -239,6 +239,64 @@ def test_latent_prompt_attention(dtype, shape):
     compare(out, want, dtype)
 
 
+@pytest.mark.parametrize("heads,dim,rot,vdim,window", [(5, 24, 16, 40, 33), (3, 128, 64, 128, None), (20, 8, 24, 16, 7), (2, 64, 32, 64, 1),
+                                                       (1, 112, 8, 8, 150), (4, 16, 64, 72, 64)])
+def test_latent_prompt_attention_on_expanded_keys(heads, dim, rot, vdim, window):
+    """Gathered rows and the attention on spelled-out keys and values: rows that start and that continue, a row without
+    tokens, heads that look at the key just inside the window, the one just outside, the token itself and the first."""
+    from megatron_mixtera_b200 import ops
+
+    dtype, kv_rank, chunk = torch.bfloat16, 48, 64
+    lengths, begin = [40, 130, 64, 200], [0, 63, 64, 137]
+    pg = Paged(lengths, kv_rank, rot, heads, window, dtype, chunk=chunk, seed=2, dim=dim)
+    m = pg.m
+    first = [0 if window is None else max(0, b - window + 1) for b in begin]
+    first[2] = 64  # no tokens, no keys
+    cu_t, cu_k = [0], [0]
+    for r in range(4):
+        cu_t.append(cu_t[-1] + lengths[r] - begin[r])
+        cu_k.append(cu_k[-1] + lengths[r] - first[r])
+    T, E = cu_t[-1], cu_k[-1]
+    keys, vals = rand(E, heads, dim, seed=50, dtype=dtype) * 0.3, rand(E, heads, vdim, seed=51, dtype=dtype)
+    q = rand(T, heads, dim + rot, seed=52, dtype=dtype) * 0.1
+    gates = rand(T, heads, seed=53, dtype=dtype)
+    want = torch.empty(T, heads, vdim, dtype=torch.float64)
+    for r in range(4):
+        for t in range(cu_t[r], cu_t[r + 1]):
+            pos = begin[r] + t - cu_t[r]
+            lo = 0 if window is None else max(0, pos - window + 1)
+            rows = torch.arange(cu_k[r] + lo - first[r], cu_k[r] + pos - first[r] + 1)
+            full = torch.cat([keys[rows], pg.rows[r][lo: pos + 1, None, kv_rank:].expand(-1, heads, -1)], -1)
+            for h, key in enumerate([max(lo, pos + 1 - (window or pos + 1)), lo - 1, pos, 0]):
+                if h < heads and lo <= key <= pos:
+                    k = full[key - lo, h].float()
+                    q[t, h] = (k * (12.0 / m.scale / float(k @ k))).to(dtype)
+            p = torch.softmax(torch.einsum("hd,khd->hk", q[t].double(), full.double()) * m.scale, -1)
+            want[t] = torch.einsum("hk,khv->hv", p, vals[rows].double()) * torch.sigmoid(gates[t].double())[:, None]
+    proj = torch.zeros(T, heads * (dim + rot) + -(-heads // 8) * 8, dtype=dtype)
+    proj[:, : heads * (dim + rot)] = q.reshape(T, -1)
+    proj[:, heads * (dim + rot): heads * (dim + rot) + heads] = gates
+    q_rot = torch.zeros(T, heads, m.row_width - m.kv_pad, dtype=dtype)
+    q_rot[..., :rot] = q[..., dim:]
+    kv = torch.cat([keys.reshape(E, -1), vals.reshape(E, -1)], 1).contiguous()
+    pool = pg.pool()
+    d = [t.to(DEV) for t in (proj, q_rot, kv, torch.tensor(cu_t, dtype=torch.int32), torch.tensor(cu_k, dtype=torch.int32),
+                             torch.tensor(first, dtype=torch.int32))]
+    key_rows = torch.empty(E, m.row_width, dtype=dtype, device=DEV)
+    out = torch.empty(T, heads, vdim, dtype=dtype, device=DEV)
+    a = pg.args(T, d[1], pool, d[0], out)
+    a.gate_offset, a.q_stride, a.q_rot_at, a.vdim = heads * (dim + rot), m.row_width - m.kv_pad, 0, vdim
+    a.cu_tokens, a.cu_keys, a.key_start, a.key_rows, a.key_values = (d[3].data_ptr(), d[4].data_ptr(), d[5].data_ptr(),
+                                                                     key_rows.data_ptr(), d[2].data_ptr())
+    a.num_rows, a.num_keys, a.max_row_tokens = 4, E, max(lengths[r] - begin[r] for r in range(4))
+    assert ops.latent_prompt_supported(dim, rot, vdim, heads)
+    ops.latent_gather(a, pool)
+    plain = torch.cat([pg.padded(pg.rows[r][first[r]: lengths[r]]) for r in range(4)])
+    assert torch.equal(key_rows.cpu(), plain)
+    ops.latent_prompt_attention(a, pool)
+    compare(out, want, dtype)
+
+
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("kv_rank,rot,dims,heads,dim", [(96, 16, 16, 5, 24), (36, 6, 6, 3, 12), (72, 24, 10, 2, 8), (512, 64, 64, 16, 128)])
 def test_latent_append(dtype, kv_rank, rot, dims, heads, dim):
@@ -266,7 +324,7 @@ def test_latent_append(dtype, kv_rank, rot, dims, heads, dim):
     a.token_to_pos, a.token_to_chunk_idx, a.token_to_local_pos = (t.data_ptr() for t in d[2:])
     a.pool, a.num_chunks, a.chunk_size, a.q_full, a.num_tokens = pool.data_ptr(), 3, 64, qf.data_ptr(), T
     a.heads, a.dim, a.rot_dim, a.rot_dims, a.kv_rank, a.kv_pad, a.row_width = heads, dim, rot, dims, kv_rank, m.kv_pad, m.row_width
-    a.eps, a.dtype = eps, ops.dtype_code(dtype)
+    a.eps, a.dtype, a.q_stride, a.q_rot_at = eps, ops.dtype_code(dtype), m.row_width, m.kv_pad
     ops.latent_append(a, pool)
     tol = 2e-5 if dtype == torch.float32 else 2e-2
     lat = proj[:, q_w: q_w + kv_rank + rot].double()

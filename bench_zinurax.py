@@ -118,7 +118,8 @@ class Recorder:
         self.ops._launch, torch.empty = self.launch, self.empty
 
 
-HYBRID = ("out_norm", "latent_append", "latent_attention", "delta_decode", "delta_lora", "delta_scan", "delta_finish")
+HYBRID = ("out_norm", "latent_append", "latent_attention", "delta_decode", "delta_lora", "delta_scan", "delta_finish",
+          "latent_gather", "latent_prompt_attention")
 
 
 def label(name, args):
@@ -146,6 +147,11 @@ def costs(s, T, visible_pairs, keys, zinurax, decode, requests):
         R, H, r = s["kv_rank"] + s["rot_dim"], s["heads"], s["kv_rank"]
         out["latent_append"] = (2.0 * T * (H * s["rot_dim"] * 2 + 2 * R), 0, 0)
         out["latent_attention"] = (2.0 * (keys * R + T * H * (R + r)), 2.0 * visible_pairs * H * (R + r), 0)
+        # expanded keys and values: (dim + rot_dim) and vdim products per pair; every key's vectors once
+        e = s["dim"] + s["vdim"]
+        out["latent_prompt_attention"] = (2.0 * (keys * (H * e + s["rot_dim"]) + T * H * (e + s["rot_dim"])),
+                                          2.0 * visible_pairs * H * (e + s["rot_dim"]), 0)
+        out["latent_gather"] = (4.0 * keys * R, 0, 0)
         n, d = s["d_heads"] * s["d_dim"], s["d_dim"]
         state = 8.0 * requests * s["d_heads"] * d * d
         vec = 2.0 * T * n * 6

@@ -24,10 +24,13 @@ constexpr int kScanTokens = 16;  // tokens prepared at a time
 
 __device__ __forceinline__ float sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
 
-template <int NI>
-__device__ __forceinline__ float lane_sum(float v) {  // over the NI lanes of a column (neighbouring lanes)
+// For output gates: fp32 arithmetic with the fast exponential and division (about 1e-6 relative).
+__device__ __forceinline__ float gate_sigmoid(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
+
+template <int NI, int STRIDE = 1>
+__device__ __forceinline__ float lane_sum(float v) {  // over the NI lanes of a column, STRIDE lanes apart
 #pragma unroll
-  for (int o = NI / 2; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  for (int o = NI / 2; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o * STRIDE);
   return v;
 }
 
@@ -99,7 +102,7 @@ __device__ __forceinline__ ulonglong2 piece(const float* p) { return *reinterpre
 
 // One token on N columns: `o` gets this lane's part of each column's output (the caller sums it over the NI lanes).  The
 // vectors are read once for all columns.
-template <int NI, int I, int N>
+template <int NI, int I, int N, int STRIDE = 1>
 __device__ __forceinline__ void step(f32x2 (&s)[N][I / 2], const TokenVectors& tv, const float (&v)[N], int ni, float (&o)[N]) {
   f32x2 nd[N], acc[N][2];
 #pragma unroll
@@ -115,7 +118,7 @@ __device__ __forceinline__ void step(f32x2 (&s)[N][I / 2], const TokenVectors& t
   }
 #pragma unroll
   for (int n = 0; n < N; ++n) {
-    const float d = -lane_sum<NI>(sum2(acc[n][0]) + sum2(acc[n][1]));
+    const float d = -lane_sum<NI, STRIDE>(sum2(acc[n][0]) + sum2(acc[n][1]));
     nd[n] = pack2(d, d);
     acc[n][0] = acc[n][1] = 0ull;
   }
@@ -174,7 +177,7 @@ __device__ __forceinline__ float dot16(const float* w, const float* l, float z) 
 
 // Shared memory: per warp six vectors [DIM] and tanh(x_w1) [rank, rounded up]; then W_w2's rows of the head.
 template <typename T, int DIM>
-__global__ void __launch_bounds__(DecodeShape<DIM>::kWarps * 32, DIM <= 64 ? 2 : 4)
+__global__ void __launch_bounds__(DecodeShape<DIM>::kWarps * 32, DIM <= 64 ? 1 : 2)
 delta_decode_kernel(b200_delta_args a, int w2_stride) {
   using D = DecodeShape<DIM>;
   constexpr int NI = D::NI, I = D::kI, N = D::kCols, EL = D::kElems, VEC = 16 / sizeof(T);
@@ -323,7 +326,7 @@ delta_decode_kernel(b200_delta_args a, int w2_stride) {
 #pragma unroll
   for (int e = 0; e < EL; ++e) {
     const int i = lane + e * 32;
-    if (i < dim) simt::store_as(dst + i, live ? vec[5 * DIM + i] * inv * norm[e] * sigmoid(simt::to_f32(xg[e])) : 0.f);
+    if (i < dim) simt::store_as(dst + i, live ? vec[5 * DIM + i] * inv * norm[e] * gate_sigmoid(simt::to_f32(xg[e])) : 0.f);
   }
 }
 
@@ -332,8 +335,9 @@ delta_decode_kernel(b200_delta_args a, int w2_stride) {
 // ---------------------------------------------------------------------------------------------------------------
 template <int DIM, int COLS, int N>
 struct ScanShape {  // COLS columns per CTA, N of them per thread
-  static constexpr int I = DIM <= 128 ? DIM : 128;
-  static constexpr int NI = DIM / I;
+  static constexpr int I = DIM <= 128 ? DIM / 2 : 128;
+  static constexpr int NI = DIM / I;  // lanes of a column: half a warp apart, so that a quarter warp reads one address
+  static constexpr int kStride = 32 / NI;
   static constexpr int kComputeThreads = COLS / N * NI;
   static constexpr int kComputeWarps = kComputeThreads / 32;
   static constexpr int kPrepWarps = kComputeWarps < 2 ? 2 : kComputeWarps;
@@ -435,7 +439,8 @@ delta_scan_kernel(b200_delta_args a) {
   const bool full = dim == DIM;
   const int in = a.state_in[row], out = a.state_out[row];
   const int64_t head_elems = static_cast<int64_t>(dim) * dim;
-  const int ni = tid % NI, group = tid / NI;  // this thread's columns: cb * COLS + n * kGroups + group
+  constexpr int ST = Sh::kStride;
+  const int ni = lane / ST, group = (tid >> 5) * ST + lane % ST;  // this thread's columns: cb * COLS + n * kGroups + group
   f32x2 s[N][I / 2];
 #pragma unroll
   for (int n = 0; n < N; ++n) {
@@ -460,10 +465,10 @@ delta_scan_kernel(b200_delta_args a) {
       float v[N], o[N];
 #pragma unroll
       for (int n = 0; n < N; ++n) v[n] = values[tt * COLS + n * Sh::kGroups];
-      step<NI, I, N>(s, tv, v, ni, o);
+      step<NI, I, N, ST>(s, tv, v, ni, o);
 #pragma unroll
       for (int n = 0; n < N; ++n) {
-        const float sum = lane_sum<NI>(o[n]);
+        const float sum = lane_sum<NI, ST>(o[n]);
         if (ni == 0 && cb * COLS + n * Sh::kGroups + group < dim) o_dst[n * Sh::kGroups] = sum;
       }
       o_dst += hd;
@@ -486,8 +491,8 @@ delta_finish_kernel(b200_delta_args a) {
   pdl_launch_dependents();
   pdl_wait();
   const int lane = threadIdx.x & 31, dim = a.dim;
-  const int64_t total = static_cast<int64_t>(a.num_tokens) * a.heads;
-  const int64_t first = (static_cast<int64_t>(blockIdx.x) * 8 + (threadIdx.x >> 5)) * kFinishUnits;
+  const uint32_t total = static_cast<uint32_t>(a.num_tokens) * a.heads, heads = a.heads;  // (the launch checks that it fits)
+  const uint32_t first = (blockIdx.x * 8 + (threadIdx.x >> 5)) * kFinishUnits;
   const T* proj = static_cast<const T*>(a.proj);
   const T* weight = static_cast<const T*>(a.norm_weight);
   T* out = static_cast<T*>(a.out);
@@ -496,13 +501,13 @@ delta_finish_kernel(b200_delta_args a) {
     T g[kFinishUnits][4];
 #pragma unroll
     for (int k = 0; k < kFinishUnits; ++k) {
-      const int64_t unit = min(first + k, total - 1), t = unit / a.heads;
-      const int at = static_cast<int>(unit - t * a.heads) * dim;
+      const uint32_t unit = min(first + k, total - 1), t = unit / heads;
+      const int at = static_cast<int>(unit - t * heads) * dim;
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         if (e * 32 >= dim) break;
         const int i = min(lane + e * 32, dim - 1);
-        v[k][e] = a.o_f32[unit * dim + i];
+        v[k][e] = a.o_f32[static_cast<int64_t>(unit) * dim + i];
         g[k][e] = proj[t * a.proj_ld + a.off_g + at + i];
         w[k][e] = simt::to_f32(weight[at + i]);
       }
@@ -516,15 +521,16 @@ delta_finish_kernel(b200_delta_args a) {
 #pragma unroll
       for (int e = 0; e < 4; ++e)
         if (lane + e * 32 < dim && first + k < total)
-          simt::store_as(out + (first + k) * dim + lane + e * 32, v[k][e] * inv * w[k][e] * sigmoid(simt::to_f32(g[k][e])));
+          simt::store_as(out + static_cast<int64_t>(first + k) * dim + lane + e * 32,
+                         v[k][e] * inv * w[k][e] * gate_sigmoid(simt::to_f32(g[k][e])));
     }
     return;
   }
   for (int k = 0; k < kFinishUnits; ++k) {
     const int64_t unit = first + k;
     if (unit >= total) return;
-    const int64_t t = unit / a.heads;
-    const int at = static_cast<int>(unit - t * a.heads) * dim;
+    const int64_t t = unit / heads;
+    const int at = static_cast<int>(unit - t * heads) * dim;
     const float* o = a.o_f32 + unit * dim;
     float sq = 0.f;
     for (int i = lane; i < dim; i += 32) sq += o[i] * o[i];
@@ -636,7 +642,8 @@ int b200_delta_scan(const b200_delta_args* a, b200_stream_t stream) {
 
 int b200_delta_finish(const b200_delta_args* a, b200_stream_t stream) {
   using namespace b200;
-  if (!delta::valid_common(a) || !a->o_f32 || !a->norm_weight || !a->out) return B200_ERR_INVALID_ARGUMENT;
+  if (!delta::valid_common(a) || !a->o_f32 || !a->norm_weight || !a->out || static_cast<int64_t>(a->num_tokens) * a->heads > (1u << 30))
+    return B200_ERR_INVALID_ARGUMENT;
   const unsigned blocks = static_cast<unsigned>((static_cast<int64_t>(a->num_tokens) * a->heads + 8 * delta::kFinishUnits - 1) / (8 * delta::kFinishUnits));
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (a->dtype == B200_DTYPE_F32) return launch_pdl(delta::delta_finish_kernel<float>, dim3(blocks), dim3(256), 0, s, *a);

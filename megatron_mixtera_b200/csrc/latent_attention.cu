@@ -917,24 +917,24 @@ latent_prompt_kernel(b200_latent_args a) {
   const int kv_ld = a.heads * (a.dim + a.vdim), rot_w = a.row_width - a.kv_pad;
   const __nv_bfloat16* kv = static_cast<const __nv_bfloat16*>(a.key_values);
   const __nv_bfloat16* rows = static_cast<const __nv_bfloat16*>(a.key_rows);
-  const int d8 = dp / 8, r8 = rp / 8, v8 = vp / 8, pieces = d8 + r8 + v8;
+  const int d8 = dp / 8, r8 = rp / 8, v8 = vp / 8;
+  const int l_row = tid >> 3, l_piece = tid & 7;  // eight threads fetch a row, 128 bytes at a time
   auto load = [&](int i) {
     __nv_bfloat16* kd = k_s + (i & 1) * kPrKeys * ks;
     __nv_bfloat16* vd = v_s + (i & 1) * kPrKeys * vs;
-    for (int x = tid; x < kPrKeys * pieces; x += kPrThreads) {
-      const int r = x / pieces, c = x - r * pieces;
+#pragma unroll
+    for (int pass = 0; pass < kPrKeys * 8 / kPrThreads; ++pass) {
+      const int r = l_row + pass * (kPrThreads / 8);
       const int key = start + i * kPrKeys + r;
       const bool in = key < end;
       const int64_t e = e_begin + (in ? key - key_begin : 0);
-      if (c < d8) {
-        cp_async16(smem_u32(kd + r * ks + c * 8), kv + e * kv_ld + head * a.dim + c * 8, in && c * 8 < a.dim);
-      } else if (c < d8 + r8) {
-        const int p = c - d8;
-        cp_async16(smem_u32(kd + r * ks + dp + p * 8), rows + e * a.row_width + a.kv_pad + p * 8, in && p * 8 < rot_w);
-      } else {
-        const int p = c - d8 - r8;
-        cp_async16(smem_u32(vd + r * vs + p * 8), kv + e * kv_ld + a.heads * a.dim + head * a.vdim + p * 8, in && p * 8 < a.vdim);
-      }
+      const __nv_bfloat16* ksrc = kv + e * kv_ld + head * a.dim;
+      const __nv_bfloat16* vsrc = kv + e * kv_ld + a.heads * a.dim + head * a.vdim;
+      const __nv_bfloat16* rsrc = rows + e * a.row_width + a.kv_pad;
+      const uint32_t kdst = smem_u32(kd + r * ks), vdst = smem_u32(vd + r * vs);
+      for (int c = l_piece; c < d8; c += 8) cp_async16(kdst + c * 16, ksrc + c * 8, in && c * 8 < a.dim);
+      for (int c = l_piece; c < r8; c += 8) cp_async16(kdst + dp * 2 + c * 16, rsrc + c * 8, in && c * 8 < rot_w);
+      for (int c = l_piece; c < v8; c += 8) cp_async16(vdst + c * 16, vsrc + c * 8, in && c * 8 < a.vdim);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };

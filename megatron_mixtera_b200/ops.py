@@ -224,10 +224,7 @@ def gemm_swiglu(x, w_interleaved, out=None):
 
 
 def gemm(x, w, bias=None, out=None):
-    """y[M, N] = x[M, K] @ w[N, K].T (+ bias), bf16 with fp32 accumulation on tcgen05 (fp32 operands and rows TMA cannot
-    address: `linear` on the CUDA cores)."""
-    if bias is None and out is None and (x.dtype == F32 or x.shape[-1] % 8):
-        return linear(x.reshape(-1, x.shape[-1]), w).view(*x.shape[:-1], w.shape[0])
+    """y[M, N] = x[M, K] @ w[N, K].T (+ bias), bf16 with fp32 accumulation on tcgen05."""
     _need(x, BF16, "x")
     _need(w, BF16, "w")
     K = x.shape[-1]
@@ -478,8 +475,6 @@ def gemm_splitk(x, w) -> GemmPartials:
         ws = _gemm_workspace(dev, lib.b200_gemm_fp8_block_splitk_bytes(M, N, K))
         n = _launch("gemm_splitk", 2, x.q, x.scale, x.m_pad, w.q, w.scale, ws, M, N, K)
     else:
-        if x.dtype == F32 or x.shape[-1] % 8:
-            return linear_partials(x.reshape(-1, x.shape[-1]), w)
         _need(x, BF16, "x")
         _need(w, BF16, "w")
         K = x.shape[-1]
@@ -770,7 +765,10 @@ def linear(x, w, *, act: Optional[str] = None, out=None, batch: int = 1, x_batch
 
 
 def linear_partials(x, w) -> GemmPartials:
-    """``x @ w.T`` on the CUDA cores as one fp32 "partial sum" for a consumer that reduces (`gemm_splitk`'s other shapes)."""
+    """``x @ w.T`` as fp32 partial sums for a consumer that reduces them: split along K on the tensor cores (`gemm_splitk`), one
+    "split" on the CUDA cores for fp32 and for rows TMA cannot address."""
+    if x.dtype == BF16 and x.shape[-1] % 8 == 0:
+        return gemm_splitk(x, w)
     M, N = x.shape[0], w.shape[0]
     ws = _gemm_workspace(x.device, 4 * M * N)
     linear(x, w, out=ws[: 4 * M * N].view(F32).view(M, N))

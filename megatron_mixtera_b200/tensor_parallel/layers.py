@@ -143,6 +143,10 @@ class _ParallelLinearBase(torch.nn.Module):
             return ops.gemm_splitk(x, self._wq) if defer_reduction else ops.gemm_fp8_block(x, self._wq, bias, out=out)
         if quantised_input:
             raise ops.B200Error("linear", -1, "got an FP8 input but this layer runs in bf16")
+        if bias is None and out is None and (input_.dtype == torch.float32 or input_.shape[-1] % 8):
+            # 32-bit models, and row lengths the bf16 GEMM's TMA cannot address
+            x = input_.reshape(-1, input_.shape[-1])
+            return ops.linear_partials(x, weight) if defer_reduction else ops.linear(x, weight).view(*input_.shape[:-1], -1)
         return ops.gemm_splitk(input_, weight) if defer_reduction else ops.gemm(input_, weight, bias, out=out)
 
 

@@ -205,3 +205,48 @@ def test_trace_replay_of_a_model_folder(case, tmp_path):
     assert not (out / "0.f32").exists()
     got = torch.from_numpy(np.fromfile(out / "1.f32", dtype="<f4")).view(3, cfg["vocab"])
     assert H.error(got, torch.stack([want[1][2], want[1][0], want[0][70]])) < LIMIT[torch.float32]
+
+
+def test_generate_command_line(case, tmp_path, capsys):
+    """Token ids in, greedy token ids out, in the prompts' order and independent of how they are batched."""
+    import json
+
+    from megatron_mixtera_b200 import checkpoint, generate
+
+    cfg, rank = H.CONFIGS["mixed"]
+    w = H.weights(cfg, rank, seed=3)
+    (tmp_path / "config.json").write_text(json.dumps(cfg))
+    checkpoint.save_safetensors(str(tmp_path / "model.safetensors"), w)
+    prompts = [H.tokens(k, cfg["vocab"], 30 + k) for k in (50, 1, 64)]
+    want = [greedy_oracle(cfg, w, p, 8)[0] for p in prompts]
+    base = ["--model", str(tmp_path), "--dtype", "float32", "--num-tokens", "8"] + [x for p in prompts for x in ("--prompt", ",".join(map(str, p)))]
+    for extra in ([], ["--cuda-graphs", "0", "--max-requests", "1"]):
+        assert generate.main(base + extra) == 0
+        lines = [[int(t) for t in x.split(",")] for x in capsys.readouterr().out.strip().splitlines()]
+        assert lines == want
+
+
+def test_registry_serves_the_dense_model_too(tmp_path):
+    """A GPT model folder through the same registry, context and steps of given tokens: a prompt whole, in portions and token
+    by token gives the same logits."""
+    import json
+
+    from megatron_mixtera_b200 import build, checkpoint
+    from megatron_mixtera_b200 import model_registry as R
+
+    build.build_torch_ops()
+    cfg = {"architecture": "GPTModel", "vocab_size": 320, "rotary_base": 10000.0,
+           "transformer": dict(num_layers=2, hidden_size=256, num_attention_heads=4, num_query_groups=2, kv_channels=64,
+                               ffn_hidden_size=512, normalization="RMSNorm", gated_linear_unit=True, activation="silu",
+                               add_bias_linear=False)}
+    shapes = {k: v for k, v in R.ARCHITECTURES["GPTModel"](cfg, {}, torch.bfloat16, 128).full_parameter_shapes().items()}
+    from megatron_mixtera_b200.synthetic import canonical_state_dict
+
+    checkpoint.save_safetensors(str(tmp_path / "model.safetensors"), canonical_state_dict(shapes, std=0.05, dtype=torch.bfloat16))
+    (tmp_path / "config.json").write_text(json.dumps(cfg))
+    _, _, ctl = R.serving_stack(str(tmp_path), dtype=torch.bfloat16, max_cached_tokens=256, max_requests=4, max_sequence_length=128,
+                                max_step_tokens=128)
+    toks = [H.tokens(90, 320, 5)]
+    whole = H.replay(ctl, [[(0, 90)]], toks)[0].float()
+    for parts in ([3, 60, 27], [64] + [1] * 26):
+        assert H.error(H.replay(ctl, [[(0, n)] for n in parts], toks)[0], whole) < 0.03

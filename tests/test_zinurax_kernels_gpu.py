@@ -39,7 +39,7 @@ def test_linear(dtype, M, N, K, act):
     tol = 1e-5 if dtype == torch.float32 else 8e-3
     assert (got - want).abs().max() <= tol * want.abs().max()
     if dtype == torch.bfloat16 and act is None:  # fp32 partial sums for a consumer that reduces
-        p = ops.gemm_splitk(x.to(DEV), w.to(DEV))
+        p = ops.linear_partials(x.to(DEV), w.to(DEV))
         parts = p.buf[: 4 * p.num_splits * M * N].view(torch.float32).view(p.num_splits, M, N).sum(0).cpu().double()
         assert (parts - want).abs().max() <= 1e-5 * want.abs().max()
 

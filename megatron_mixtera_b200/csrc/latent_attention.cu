@@ -883,7 +883,7 @@ latent_gather_kernel(b200_latent_args a) {
 constexpr int kPrQueries = 64;
 constexpr int kPrKeys = 64;
 constexpr int kPrThreads = 128;
-constexpr int kPrSteps = 12;    // 16-wide steps of (dim, rot_dim), each rounded up to 16
+constexpr int kPrSteps = 12;    // most 16-wide steps of (dim, rot_dim), each rounded up to 16
 constexpr int kPrMaxV = 128;
 
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool valid) {  // invalid: 16 bytes of zeros
@@ -891,7 +891,9 @@ __device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool v
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(n) : "memory");
 }
 
-__global__ void __launch_bounds__(kPrThreads, 2)
+// STEPS, MAXV: what the registers of a query row hold; smaller heads leave room for a third CTA per SM.
+template <int STEPS, int MAXV>
+__global__ void __launch_bounds__(kPrThreads, STEPS <= 8 ? 3 : 2)
 latent_prompt_kernel(b200_latent_args a) {
   extern __shared__ __align__(128) uint8_t smem[];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gid = lane >> 2, tig = lane & 3;
@@ -954,9 +956,9 @@ latent_prompt_kernel(b200_latent_args a) {
   load(0);
   asm volatile("cp.async.wait_all;" ::: "memory");
   __syncthreads();
-  uint32_t qf[kPrSteps][4];
+  uint32_t qf[STEPS][4];
 #pragma unroll
-  for (int s = 0; s < kPrSteps; ++s)
+  for (int s = 0; s < STEPS; ++s)
     if (s < steps)
       ldmatrix_x4(smem_u32(q_s + (warp * 16 + (lane & 15)) * ks + s * 16 + (lane >> 4) * 8), qf[s][0], qf[s][1], qf[s][2], qf[s][3]);
   int lo[2], hi[2];  // visible keys of this thread's two queries
@@ -968,9 +970,9 @@ latent_prompt_kernel(b200_latent_args a) {
   }
   const int w_first = pos0 + warp * 16, w_last = min(w_first + 15, pos0 + n_q - 1);  // this warp's queries
   const float scale_log2 = a.scale * kLog2e;
-  float o[kPrMaxV / 8][4];
+  float o[MAXV / 8][4];
 #pragma unroll
-  for (int j = 0; j < kPrMaxV / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+  for (int j = 0; j < MAXV / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
 
   for (int i = 0; i < n_tiles; ++i) {
@@ -984,7 +986,7 @@ latent_prompt_kernel(b200_latent_args a) {
 #pragma unroll
       for (int n = 0; n < 8; ++n) sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.f;
 #pragma unroll
-      for (int s = 0; s < kPrSteps; ++s) {
+      for (int s = 0; s < STEPS; ++s) {
         if (s < steps) {
 #pragma unroll
           for (int n = 0; n < 4; ++n) {
@@ -1019,7 +1021,7 @@ latent_prompt_kernel(b200_latent_args a) {
       }
       if (__any_sync(0xffffffffu, alpha[0] != 1.f || alpha[1] != 1.f)) {
 #pragma unroll
-        for (int j = 0; j < kPrMaxV / 8; ++j) {
+        for (int j = 0; j < MAXV / 8; ++j) {
           o[j][0] *= alpha[0];
           o[j][1] *= alpha[0];
           o[j][2] *= alpha[1];
@@ -1041,7 +1043,7 @@ latent_prompt_kernel(b200_latent_args a) {
             pl[h * 2 + r] = pack_bf16x2(p0 - h0, p1 - h1);
           }
 #pragma unroll
-        for (int j = 0; j < kPrMaxV / 16; ++j) {
+        for (int j = 0; j < MAXV / 16; ++j) {
           if (j * 16 < vp) {
             uint32_t b0, b1, b2, b3;
             ldmatrix_x4_trans(vb + ((kk * 16 + (((lane >> 3) & 1) << 3) + (lane & 7)) * vs + j * 16 + (lane >> 4) * 8) * 2, b0, b1, b2, b3);
@@ -1068,7 +1070,7 @@ latent_prompt_kernel(b200_latent_args a) {
     const float g = gate_of<__nv_bfloat16>(a, t, head) / l;
     __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(a.out) + (t * a.heads + head) * a.vdim;
 #pragma unroll
-    for (int j = 0; j < kPrMaxV / 8; ++j) {
+    for (int j = 0; j < MAXV / 8; ++j) {
       const int col = j * 8 + tig * 2;
       if (col < a.vdim) *reinterpret_cast<uint32_t*>(dst + col) = pack_bf16x2(o[j][2 * r] * g, o[j][2 * r + 1] * g);
     }
@@ -1199,6 +1201,14 @@ static int launch_umma(const b200_latent_args& a, cudaStream_t s) {
   return launch_pdl(latent_combine_kernel, dim3(a.num_tokens * a.heads), dim3(128), 0, s, a);
 }
 
+template <int STEPS, int MAXV>
+static int launch_prompt(const b200_latent_args& a, cudaStream_t s) {
+  static std::atomic<uint64_t> done{0};
+  if (ensure_dynamic_smem(latent_prompt_kernel<STEPS, MAXV>, kMaxSmem, done) != B200_OK) return B200_ERR_LAUNCH;
+  const dim3 grid((a.max_row_tokens + kPrQueries - 1) / kPrQueries, a.num_rows, a.heads);
+  return launch_pdl(latent_prompt_kernel<STEPS, MAXV>, grid, dim3(kPrThreads), prompt_smem(a.dim, a.rot_dim, a.vdim), s, a);
+}
+
 // Whether the decode kernel takes this call, and its launch.
 template <int KVT>
 static bool decode_fits(const b200_latent_args& a) {
@@ -1297,11 +1307,9 @@ int b200_latent_prompt_attention(const b200_latent_args* a, b200_stream_t stream
   if (a->proj_ld % 8 != 0 || a->q_stride % 8 != 0 || a->q_rot_at % 8 != 0 || !aligned16(a->proj) || !aligned16(a->key_rows) ||
       !aligned16(a->key_values) || a->q_stride < a->q_rot_at + a->row_width - a->kv_pad)
     return B200_ERR_ALIGNMENT;
-  static std::atomic<uint64_t> done{0};
-  if (ensure_dynamic_smem(latent_prompt_kernel, kMaxSmem, done) != B200_OK) return B200_ERR_LAUNCH;
-  const dim3 grid((a->max_row_tokens + kPrQueries - 1) / kPrQueries, a->num_rows, a->heads);
-  return launch_pdl(latent_prompt_kernel, grid, dim3(kPrThreads), prompt_smem(a->dim, a->rot_dim, a->vdim),
-                    reinterpret_cast<cudaStream_t>(stream), *a);
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  const int steps = (a->dim + 15) / 16 + (a->rot_dim + 15) / 16;
+  return steps <= 8 && a->vdim <= 64 ? launch_prompt<8, 64>(*a, s) : launch_prompt<kPrSteps, kPrMaxV>(*a, s);
 }
 
 }  // extern "C"

@@ -1,6 +1,6 @@
 """Generate from a model folder (`config.json` + `model.safetensors`) with token ids in and token ids out.
 
-    python -m megatron_mixtera_b200.generate --model DIR --prompt 5,17,3 --prompt 9,9 --num-tokens 16
+    python -m megatron_mixtera_b200.generate --model DIR --prompt 11,250,4 --prompt 9,9 --num-tokens 16
 
 One line per prompt, in order: the generated ids, comma-separated.  Prompts may also come from standard input, one per line.
 """

@@ -4,11 +4,12 @@
 
 Reads one JSON object per line from standard input,
 
-    {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": []}
+    {"step": 7, "entries": [{"id": "chat-1", "tokens": [90, 4], "want": [1]}, {"id": "chat-2", "tokens": [33], "want": []}], "end": ["chat-2"]}
 
 runs all entries of a step as one batch from the cache and state that earlier steps left, writes the logits at the wanted
 places to ``<out>/<step>.f32`` ([wanted, vocab] little-endian floats, in the order of entries and places), gives back the
-requests in ``end``, and prints ``done <step>``.  ``--max-tokens``: the most tokens live requests hold at any time.
+requests in ``end``, and prints ``done <step>``.  ``--max-tokens`` sizes the
+cache pool: requests that are live together never hold more tokens than that, each counted in whole chunks of 64.
 """
 from __future__ import annotations
 
@@ -25,7 +26,7 @@ def main(argv=None) -> int:
     ap.add_argument("--model", required=True, help="folder with config.json and model.safetensors")
     ap.add_argument("--dtype", choices=("bfloat16", "float32"), default="bfloat16")
     ap.add_argument("--out", required=True, help="folder for the <step>.f32 files")
-    ap.add_argument("--max-tokens", type=int, required=True, help="most tokens that live requests hold at any time")
+    ap.add_argument("--max-tokens", type=int, required=True, help="size of the cache pool in tokens (whole chunks of 64 per live request)")
     args = ap.parse_args(argv)
 
     import torch

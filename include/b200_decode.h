@@ -412,6 +412,15 @@ typedef struct {
                                out_q_mode 2: fp32 [nq][out_m_pad], one scale per token per head (head_dim 128 only) */
   int32_t out_q_mode;       /* 1: MXFP8, 2: 128-block recipe */
   int32_t out_m_pad;        /* out_q_mode 2: row stride of out_scales (>= T, multiple of 4) */
+  /* separate != 0: `qkv` holds finished queries [T][nq][head_dim] (no RoPE, no fused append); k_cache and v_cache point at the
+   * first token's keys and values, tokens pool_row_elems elements apart, heads next to one another; head_dim and value_dim
+   * multiples of 8 up to 128; out [T][nq][value_dim]; any group size up to 16 (prefill units of at most 64 / (nq / nkv) tokens,
+   * rounded down).  In decode steps (row_of_token == NULL) the kernel before this one may write the newest token's key and
+   * value, nothing older.  window > 0 (separate only): a token sees itself and the window - 1 tokens before it. */
+  int32_t separate;
+  int32_t value_dim;
+  int32_t window;
+  int64_t pool_row_elems;
 } b200_attention_args;
 
 size_t b200_paged_attention_workspace_bytes(int num_tokens, int num_q_heads, int head_dim, int num_splits);
@@ -595,6 +604,170 @@ int b200_delta_decode(const b200_delta_args* args, b200_stream_t stream);
 int b200_delta_lora(const b200_delta_args* args, b200_stream_t stream);
 int b200_delta_scan(const b200_delta_args* args, b200_stream_t stream);
 int b200_delta_finish(const b200_delta_args* args, b200_stream_t stream);
+
+/* Attention with separate queries (see b200_attention_args) on the CUDA cores: fp32 models and head dims the tensor-core kernels
+ * do not take (up to 256).  One warp per (token, query head); decode and prefill steps alike. */
+int b200_attention_simt(const b200_attention_args* args, int dtype, b200_stream_t stream);
+
+/* ---------------------------------------------------------------------------------------
+ * Parallel blocks (Fabivik): x += mixer(norm1(x)) + ff(norm2(x)) on a 32-bit residual stream.
+ * b200_residual_norm: h = hidden[row] (or table[ids[row]] * table_scale), plus
+ *     sum over num_splits of partials[s][row]            (fp32, a linear's split-K partial sums)
+ *   + branch[row]                                        (`dtype`)
+ *   + sum over j < top of expert_rows[offsets[pairs[row][j].expert] + pairs[row][j].rank]   (`dtype`)
+ *   + shared_gate[row] * shared_rows[row]                (`dtype`; shared_gate NULL: 1)
+ * each part optional; then y_i[out row] = h / sqrt(mean(h^2) + eps) * (gain + gamma_i) * out_scale for up to two gammas.
+ * row_index == NULL: out row = row, h is stored back to hidden.  row_index: out row r shows row row_index[r] of `source_rows`
+ * rows; nothing is stored back. */
+typedef struct b200_residual_norm_args {
+  const void* table;
+  const int64_t* ids;
+  const float* partials;
+  const void* branch;
+  const void* expert_rows;
+  const int32_t* pairs; /* [rows][top][2] = {expert, rank inside the expert} */
+  const int32_t* offsets;
+  const void* shared_rows;
+  const float* shared_gate;
+  const int64_t* row_index;
+  float* hidden;
+  const void* gamma[2];
+  void* y[2];
+  int64_t table_rows;
+  int64_t expert_row_count;
+  int32_t num_splits, rows, source_rows, width, top, experts, dtype;
+  float table_scale, eps, gain, out_scale;
+} b200_residual_norm_args;
+int b200_residual_norm(const b200_residual_norm_args* args, b200_stream_t stream);
+
+/* Short causal convolutions over time, one filter per channel, with the last taps - 1 inputs of every request as state:
+ *   y_t = sum_j filter[j][c] * u_(t - taps + 1 + j),  u = proj[:, 0:channels), zeros before a sequence's start.
+ * State [slot][taps - 1][channels] (`dtype`): read from slot state_in[row] (-1: zeros), written to state_out[row] (-1: nowhere), never
+ * the same slot.  cu_tokens == NULL: one token per row (token t = row t); else row_of_token and cu_tokens [rows + 1].
+ * At most 8 taps.
+ * b200_conv_silu: out[t][c] = silu(y).
+ * b200_conv_qkv: channels = queries (heads x dim) | keys (kv_heads x dim) | values (kv_heads x vdim); queries and keys are RMS-normed
+ *   per head (q_norm, k_norm [dim]); values become (1 - mix) y + mix * v_first_in when v_first_in is given, and are copied to
+ *   v_first_out ([T][kv_heads * vdim]) when that is; queries go to out [T][heads * dim], keys and values to the pool. */
+typedef struct b200_conv_args {
+  const void* proj;
+  const void* filter; /* [taps][channels] */
+  void* state;
+  const int32_t* state_in;
+  const int32_t* state_out;
+  const int32_t* cu_tokens;
+  const int32_t* row_of_token;
+  void* out;
+  const void* q_norm;
+  const void* k_norm;
+  void* k_pool;
+  void* v_pool;
+  const int64_t* chunk_idx;
+  const int64_t* local_pos;
+  const void* v_first_in;
+  void* v_first_out;
+  const void* mix; /* one value */
+  int64_t proj_ld, state_slots, pool_row_elems;
+  int32_t channels, taps, num_tokens, num_rows, heads, kv_heads, dim, vdim, chunk_size, num_chunks, dtype;
+  float eps;
+} b200_conv_args;
+int b200_conv_silu(const b200_conv_args* args, b200_stream_t stream);
+int b200_conv_qkv(const b200_conv_args* args, b200_stream_t stream);
+
+/* Token shift: out[t][s][c] = x_t + (x_(t-1) - x_t) * mu[s][c] for `mixes` rows of mu; the previous token's row of a portion's first
+ * token comes from state [slot][width] (`dtype`), which receives the portion's last row.  Slots and rows as above. */
+typedef struct b200_shift_args {
+  const void* x;
+  const void* mu;
+  void* state;
+  const int32_t* state_in;
+  const int32_t* state_out;
+  const int32_t* cu_tokens;
+  const int32_t* row_of_token;
+  void* out;      /* [T][mixes (- 1 with out_last)][width] */
+  void* out_last; /* NULL, or [T][width]: the last mix goes there */
+  int64_t state_slots;
+  int32_t num_tokens, num_rows, width, mixes, dtype;
+} b200_shift_args;
+int b200_token_shift(const b200_shift_args* args, b200_stream_t stream);
+
+/* Linear recurrences per head over a [key channel] x [value channel] fp32 state, stored [slot][head][vdim][dim]:
+ *   B200_RECURRENCE_WKV    o = (S + diag(bonus) k v^T)^T r, S <- diag(w) S + k v^T, w = exp(-exp(z + decay_bias)), z = W_w2 lora
+ *   B200_RECURRENCE_DELTA  S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q; q, k unit vectors (q also * dim^-1/2), beta =
+ *                          sigmoid(x_b), g = exp(-exp(decay_rate) * softplus(x_a + decay_bias)), one each per head
+ * then out = o / rms(o) over the head * norm_weight * silu(gate).
+ * b200_recurrence_decode: one token per row, everything in one kernel (WKV: the product with W_w2; DELTA: the short
+ *   convolutions of q | k | v at columns [0, 2 kv_heads dim + heads vdim) of proj, with silu, and their state).
+ * b200_recurrence_scan: rows of any length; WKV reads z as fp32 partial sums, DELTA reads the convolved q | k | v from `conv`.
+ * b200_recurrence_finish: head norm, weight and gate behind the scan.
+ * b200_recurrence_lora: lora = tanh(sum of partial sums) in `dtype` (WKV). */
+#define B200_RECURRENCE_WKV 0
+#define B200_RECURRENCE_DELTA 1
+typedef struct b200_recurrence_args {
+  const void* proj;
+  const void* conv;       /* DELTA scan: [T][conv channels] */
+  const float* z;         /* WKV scan: [z_splits][T][heads * dim]; lora: [z_splits][T][rank] */
+  void* lora;             /* [T][rank] */
+  const void* w2;         /* [heads * dim][rank] */
+  const void* decay_bias; /* WKV [heads * dim], DELTA [heads] */
+  const void* decay_rate; /* DELTA [heads] */
+  const void* bonus;      /* WKV [heads * dim] */
+  const void* norm_weight;
+  const void* conv_filter; /* DELTA decode, as in b200_conv_args */
+  void* conv_state;
+  float* state;
+  const int32_t* state_in;
+  const int32_t* state_out;
+  const int32_t* cu_tokens;
+  float* o_f32; /* [T][heads * vdim] */
+  void* out;    /* [T][heads * vdim] */
+  int64_t proj_ld, state_slots;
+  int32_t kind, off_r, off_k, off_v, off_g, off_a, off_b; /* columns of proj (r: also q) */
+  int32_t rank, heads, kv_heads, dim, vdim, taps, num_tokens, num_rows, z_splits, norm_per_head, dtype;
+  float unit_eps, eps;
+} b200_recurrence_args;
+int b200_recurrence_decode(const b200_recurrence_args* args, b200_stream_t stream);
+int b200_recurrence_scan(const b200_recurrence_args* args, b200_stream_t stream);
+int b200_recurrence_finish(const b200_recurrence_args* args, b200_stream_t stream);
+int b200_recurrence_lora(const b200_recurrence_args* args, b200_stream_t stream);
+
+/* Mixture of experts.  Expert: y = W_down act(W_gate x', W_up x') with x' = weight * x (the weight is applied to the products, in
+ * fp32), act(g, u) = g' sigmoid(alpha g') (u' + 1), g' = min(g, limit), u' = clamp(u, -limit, limit).
+ * up weights [experts][2 * ff][width]: every 128 rows are 64 gate rows and the 64 matching up rows; ff a multiple of 64 (padded with
+ * zero rows).  down weights [experts][width][ff].  A shared expert of its own size may run on every token in the same launches.
+ * b200_moe_route: scores = sigmoid(router logits [router_splits][T][router_ld], fp32 partial sums), the `top` largest per token; their
+ *   places when tokens are sorted by expert; shared_gate = sigmoid(logit column `experts`); the list of (expert, first row, rows)
+ *   tiles of at most tile_tokens rows.
+ * b200_moe_gather: x_sorted, row_scale.
+ * b200_moe_up / b200_moe_down: the grouped products.  simt != 0: CUDA cores (fp32, or widths TMA cannot address), tile_tokens 64;
+ *   else tcgen05, tile_tokens in {32, 64, 128, 256}. */
+typedef struct b200_moe_args {
+  const void* x;
+  const float* router;
+  const void* up;
+  const void* down;
+  const void* shared_up;
+  const void* shared_down;
+  int32_t* counts; /* [experts + 1]: zero before the first call, left zero by every call */
+  int32_t* pairs;  /* [T][top][2] */
+  float* pair_weight;
+  int32_t* offsets; /* [experts + 1] */
+  int32_t* tiles;   /* [max_tiles][4] */
+  int32_t* num_tiles;
+  float* shared_gate;
+  void* x_sorted;
+  float* row_scale;
+  void* inter;
+  void* y;
+  void* shared_inter;
+  void* shared_y;
+  int32_t num_tokens, width, experts, top, ff, shared_ff, router_splits, router_ld, tile_tokens, max_tiles, simt, dtype;
+  float limit, shared_limit, alpha;
+} b200_moe_args;
+int b200_moe_route(const b200_moe_args* args, b200_stream_t stream);
+int b200_moe_gather(const b200_moe_args* args, b200_stream_t stream);
+int b200_moe_up(const b200_moe_args* args, b200_stream_t stream);
+int b200_moe_down(const b200_moe_args* args, b200_stream_t stream);
 
 #ifdef __cplusplus
 }

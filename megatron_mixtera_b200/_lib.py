@@ -88,6 +88,19 @@ EXPORTED_SYMBOLS = (
     "b200_delta_lora",
     "b200_delta_scan",
     "b200_delta_finish",
+    "b200_attention_simt",
+    "b200_residual_norm",
+    "b200_conv_silu",
+    "b200_conv_qkv",
+    "b200_token_shift",
+    "b200_recurrence_decode",
+    "b200_recurrence_scan",
+    "b200_recurrence_finish",
+    "b200_recurrence_lora",
+    "b200_moe_route",
+    "b200_moe_gather",
+    "b200_moe_up",
+    "b200_moe_down",
 )
 
 
@@ -130,6 +143,10 @@ class AttentionArgs(ctypes.Structure):
         ("out_scales", c_void_p),
         ("out_q_mode", c_int32),
         ("out_m_pad", c_int32),
+        ("separate", c_int32),
+        ("value_dim", c_int32),
+        ("window", c_int32),
+        ("pool_row_elems", c_int64),
     ]
 
 
@@ -165,6 +182,57 @@ class DeltaArgs(ctypes.Structure):
         (n, c_int32) for n in (
             "off_r", "off_k", "off_v", "off_g", "off_a", "off_w1", "rank", "heads", "dim", "num_tokens", "num_rows",
             "dtype")] + [(n, c_float) for n in ("decay_scale", "unit_eps", "eps")]
+
+
+def _fields(*groups):
+    return [(name, ctype) for ctype, names in groups for name in names.split()]
+
+
+class ResidualNormArgs(ctypes.Structure):
+    """Mirror of ``b200_residual_norm_args``."""
+
+    _fields_ = _fields((c_void_p, "table ids partials branch expert_rows pairs offsets shared_rows shared_gate row_index hidden")) + [
+        ("gamma", c_void_p * 2), ("y", c_void_p * 2)] + _fields(
+        (c_int64, "table_rows expert_row_count"), (c_int32, "num_splits rows source_rows width top experts dtype"),
+        (c_float, "table_scale eps gain out_scale"))
+
+
+class ConvArgs(ctypes.Structure):
+    """Mirror of ``b200_conv_args``."""
+
+    _fields_ = _fields(
+        (c_void_p, "proj filter state state_in state_out cu_tokens row_of_token out q_norm k_norm k_pool v_pool chunk_idx local_pos "
+                   "v_first_in v_first_out mix"),
+        (c_int64, "proj_ld state_slots pool_row_elems"),
+        (c_int32, "channels taps num_tokens num_rows heads kv_heads dim vdim chunk_size num_chunks dtype"), (c_float, "eps"))
+
+
+class ShiftArgs(ctypes.Structure):
+    """Mirror of ``b200_shift_args``."""
+
+    _fields_ = _fields((c_void_p, "x mu state state_in state_out cu_tokens row_of_token out out_last"), (c_int64, "state_slots"),
+                       (c_int32, "num_tokens num_rows width mixes dtype"))
+
+
+class RecurrenceArgs(ctypes.Structure):
+    """Mirror of ``b200_recurrence_args``."""
+
+    _fields_ = _fields(
+        (c_void_p, "proj conv z lora w2 decay_bias decay_rate bonus norm_weight conv_filter conv_state state state_in state_out cu_tokens "
+                   "o_f32 out"),
+        (c_int64, "proj_ld state_slots"),
+        (c_int32, "kind off_r off_k off_v off_g off_a off_b rank heads kv_heads dim vdim taps num_tokens num_rows z_splits norm_per_head "
+                  "dtype"), (c_float, "unit_eps eps"))
+
+
+class MoeArgs(ctypes.Structure):
+    """Mirror of ``b200_moe_args``."""
+
+    _fields_ = _fields(
+        (c_void_p, "x router up down shared_up shared_down counts pairs pair_weight offsets tiles num_tiles shared_gate x_sorted row_scale "
+                   "inter y shared_inter shared_y"),
+        (c_int32, "num_tokens width experts top ff shared_ff router_splits router_ld tile_tokens max_tiles simt dtype"),
+        (c_float, "limit shared_limit alpha"))
 
 
 class TpComm(ctypes.Structure):
@@ -326,6 +394,15 @@ def load() -> ctypes.CDLL:
         getattr(lib, name).argtypes = [POINTER(LatentArgs), c_void_p]
     for name in ("b200_delta_decode", "b200_delta_lora", "b200_delta_scan", "b200_delta_finish"):
         getattr(lib, name).argtypes = [POINTER(DeltaArgs), c_void_p]
+    lib.b200_attention_simt.argtypes = [POINTER(AttentionArgs), c_int, c_void_p]
+    lib.b200_residual_norm.argtypes = [POINTER(ResidualNormArgs), c_void_p]
+    for name in ("b200_conv_silu", "b200_conv_qkv"):
+        getattr(lib, name).argtypes = [POINTER(ConvArgs), c_void_p]
+    lib.b200_token_shift.argtypes = [POINTER(ShiftArgs), c_void_p]
+    for name in ("b200_recurrence_decode", "b200_recurrence_scan", "b200_recurrence_finish", "b200_recurrence_lora"):
+        getattr(lib, name).argtypes = [POINTER(RecurrenceArgs), c_void_p]
+    for name in ("b200_moe_route", "b200_moe_gather", "b200_moe_up", "b200_moe_down"):
+        getattr(lib, name).argtypes = [POINTER(MoeArgs), c_void_p]
     for name in EXPORTED_SYMBOLS:
         fn = getattr(lib, name)
         if fn.restype is c_int or name.startswith("b200_") and fn.restype not in (c_char_p, c_size_t):

@@ -1,5 +1,7 @@
-// Paged-KV attention for the dynamic inference context (GQA, bf16 KV pool, head dim 64 / 128; the E4M3 pool has
-// kernels of its own in attention_fp8.cu).
+// Paged-KV attention for the dynamic inference context (GQA, bf16 KV pool; the E4M3 pool has kernels of its own in
+// attention_fp8.cu).  Two layouts: fused qkv rows with RoPE and equal head dims of 64 / 128, or (`separate`) finished queries
+// and a pool of [keys | values] rows with key and value dims of their own up to 128 (the tile's missing columns are the zeros
+// TMA fills in), optionally under a sliding window.  DK / DV are the tile widths of keys and values.
 //
 // One CTA works on one (token row, KV head, context split) unit:
 //   * a producer warp walks the row's block table and streams 64-token K and V tiles of that KV
@@ -30,17 +32,17 @@ constexpr int kThreads = kConsumerThreads + 32;
 constexpr int kStages = 3;
 constexpr int kMaxSplits = 64;
 
-template <int D>
+template <int DK, int DV = DK>
 struct Cfg {
-  static constexpr int kSub = D / 64;                 // 128-byte swizzle rows hold 64 bf16 values
-  static constexpr int kSubBytes = kTile * 128;       // one [64 tokens x 64 dims] sub-tile
-  static constexpr int kTileBytes = kSub * kSubBytes; // K or V tile in the ring
-  static constexpr int kStageBytes = 2 * kTileBytes;
-  static constexpr int kQStride = D + 8;              // bf16 elements, padded against bank conflicts
+  static constexpr int kSubK = DK / 64, kSubV = DV / 64;  // 128-byte swizzle rows hold 64 bf16 values
+  static constexpr int kSubBytes = kTile * 128;           // one [64 tokens x 64 dims] sub-tile
+  static constexpr int kTileBytesK = kSubK * kSubBytes;   // key tile in the ring, followed by the value tile
+  static constexpr int kStageBytes = kTileBytesK + kSubV * kSubBytes;
+  static constexpr int kQStride = DK + 8;                 // bf16 elements, padded against bank conflicts
   static constexpr int kQBytes = 16 * kQStride * 2;
-  static constexpr int kQkvBytes = 18 * D * 2;        // (G + 2) <= 18 head vectors of this unit, when they are summed
-                                                      // here from the QKV GEMM's split-K partial sums
-  static constexpr int kMergeBytes = kConsumerWarps * 16 * (D + 2) * 4;
+  static constexpr int kQkvBytes = DK == DV ? 18 * DK * 2 : 0;  // (G + 2) <= 18 head vectors of this unit, when they are
+                                                                // summed here from the QKV GEMM's split-K partial sums
+  static constexpr int kMergeBytes = kConsumerWarps * 16 * (DV + 2) * 4;
   static_assert(kMergeBytes <= kStages * kStageBytes, "merge buffers reuse the tile ring");
   static constexpr int kSmemBytes = kStages * kStageBytes + kQBytes + 256 + kQkvBytes + 1024;
 };
@@ -72,9 +74,19 @@ struct Params {
   const float* v_scale;
   float* ws_o;    // [T][nq][splits][D]
   float* ws_lse;  // [T][nq][splits]   (log2 domain)
+  int separate;      // 1: finished queries and a [keys | values] pool; 0: fused qkv rows
   int T, nq, nkv, G, chunk, num_chunks, max_chunks, num_splits, fused, min_split;
   float scale_log2;  // softmax scale * log2(e)
+  // Query head g of KV head h of token t starts at qkv + t * q_token + h * q_group + g * q_head; dk / dv: real head dims.
+  int64_t q_token;
+  int q_group, q_head, dk, dv;
+  int64_t pool_row;  // elements from one token's keys (or values) to the next token's
+  int window;        // keys a token sees, itself included; 0: all of its request's
 };
+
+// First key that a token whose newest visible key is kv_len - 1 sees, and the tile that holds it.
+__device__ __forceinline__ int first_key(const Params& p, int kv_len) { return p.window > 0 ? max(kv_len - p.window, 0) : 0; }
+__device__ __forceinline__ int first_tile_key(const Params& p, int kv_len) { return first_key(p, kv_len) / kTile * kTile; }
 
 // Tokens per split for a row of kv_len tokens: equal shares rounded up to whole tiles, never
 // smaller than min_split.  The combine kernel uses the same formula.
@@ -101,7 +113,7 @@ __device__ __forceinline__ void consumer_barrier() { asm volatile("bar.sync 1, 1
 template <int D, typename Sync>
 __device__ __forceinline__ void store_output(const Params& p, int t, int head, int d, float o, float* red, Sync block_sync) {
   if (p.out_q == nullptr) {
-    p.out[(static_cast<int64_t>(t) * p.nq + head) * D + d] = __float2bfloat16_rn(o);
+    if (d < p.dv) p.out[(static_cast<int64_t>(t) * p.nq + head) * p.dv + d] = __float2bfloat16_rn(o);
     return;
   }
   const float ob = bf16_round(o);
@@ -126,10 +138,11 @@ __device__ __forceinline__ void store_output(const Params& p, int t, int head, i
   }
 }
 
-template <int D>
+template <int DK, int DV, bool SEPARATE>
 __global__ void __launch_bounds__(kThreads, 2)
 paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, Params p) {
-  using C = Cfg<D>;
+  using C = Cfg<DK, DV>;
+  constexpr int D = DK;  // fused layout: one width for queries, keys and values
   const int tid = threadIdx.x;
   const int warp = tid >> 5;
   const int lane = tid & 31;
@@ -155,12 +168,13 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     if (p.num_splits == 1) {
       __shared__ float red0[4];
       if (tid < kConsumerThreads)
-        for (int i = tid; i < G * D; i += kConsumerThreads) store_output<D>(p, t, h * G + i / D, i % D, 0.f, red0, consumer_barrier);
+        for (int i = tid; i < G * DV; i += kConsumerThreads) store_output<DV>(p, t, h * G + i / DV, i % DV, 0.f, red0, consumer_barrier);
     }
     return;
   }
-  const int L = split_length(kv_len, p.num_splits, p.min_split);
-  const int start = split * L;
+  const int base = SEPARATE ? first_tile_key(p, kv_len) : 0, key_begin = SEPARATE ? first_key(p, kv_len) : 0;
+  const int L = split_length(kv_len - base, p.num_splits, p.min_split);
+  const int start = base + split * L;
   if (start >= kv_len) {
     pdl_wait();
     return;
@@ -194,8 +208,12 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     if (lane == 0) {
       // Decode steps: the pool holds only what earlier steps wrote (this step's key/value is patched
       // in by the consumers), so K/V streaming starts without waiting for the QKV GEMM before us.
-      // Prefill steps: the append kernel right before us writes the pool, so wait for it.
-      if (!p.fused) pdl_wait();
+      // Separate append (decode): only the tile with the new token waits for the append kernel right before us.
+      // Prefill steps: that kernel writes any part of the pool, so wait for it.
+      const int wait_tile = p.fused ? n_tiles : (SEPARATE && p.row_of_token == nullptr && end == kv_len) ? n_tiles - 1
+                            : (SEPARATE && p.row_of_token == nullptr)                                     ? n_tiles
+                                                                                                            : 0;
+      if (wait_tile == 0) pdl_wait();
       const int32_t* bt_row = p.block_table + static_cast<int64_t>(row) * p.max_chunks;
       int cur_c = -1;
       int cur_id = 0;
@@ -211,13 +229,16 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
         const int tok_row = cur_id * p.chunk + (tok0 - c * p.chunk);
         mbar_wait_bounded(&empty_bar[s], phase ^ 1, abort_flag, kStatusAttnTimeout);
         uint8_t* kdst = smem + s * C::kStageBytes;
-        uint8_t* vdst = kdst + C::kTileBytes;
+        uint8_t* vdst = kdst + C::kTileBytesK;
+        if (i > 0 && i == wait_tile) {
+          pdl_wait();
+          fence_proxy_async_global();  // the append kernel wrote with ordinary stores, TMA reads
+        }
         mbar_arrive_expect_tx(&full_bar[s], C::kStageBytes);
 #pragma unroll
-        for (int sub = 0; sub < C::kSub; ++sub) {
-          tma_load_3d(kdst + sub * C::kSubBytes, &map_k, &full_bar[s], sub * 64, h, tok_row);
-          tma_load_3d(vdst + sub * C::kSubBytes, &map_v, &full_bar[s], sub * 64, h, tok_row);
-        }
+        for (int sub = 0; sub < C::kSubK; ++sub) tma_load_3d(kdst + sub * C::kSubBytes, &map_k, &full_bar[s], sub * 64, h, tok_row);
+#pragma unroll
+        for (int sub = 0; sub < C::kSubV; ++sub) tma_load_3d(vdst + sub * C::kSubBytes, &map_v, &full_bar[s], sub * 64, h, tok_row);
       }
     }
     return;
@@ -226,7 +247,7 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
   // --------------------------------- consumer warps ---------------------------------
   const int gid = lane >> 2;
   const int tig = lane & 3;
-  const __nv_bfloat16* qkv_t = p.qkv + (static_cast<int64_t>(t) * p.nkv + h) * (G + 2) * D;
+  const __nv_bfloat16* qkv_t = p.qkv + t * p.q_token + static_cast<int64_t>(h) * p.q_group;
 
   pdl_wait();  // qkv is the previous kernel's output
   if (p.qkv_partials != nullptr) {
@@ -254,7 +275,13 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
   for (int i = tid; i < 16 * C::kQStride / 2; i += kConsumerThreads)
     reinterpret_cast<uint32_t*>(q_smem)[i] = 0u;
   consumer_barrier();
-  {
+  if (SEPARATE) {
+    for (int i = tid; i < G * (DK / 2); i += kConsumerThreads) {
+      const int g = i / (DK / 2), j = (i - g * (DK / 2)) * 2;
+      if (j < p.dk)
+        *reinterpret_cast<uint32_t*>(&q_smem[g * C::kQStride + j]) = *reinterpret_cast<const uint32_t*>(qkv_t + g * p.q_head + j);
+    }
+  } else {
     const bool rope = p.cos != nullptr;
     const int64_t pq = rope ? p.pos_q[t] : 0;
     const __nv_bfloat16* cs = p.cos + pq * (D / 2);
@@ -271,9 +298,9 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
   }
   consumer_barrier();
 
-  uint32_t qf[D / 16][4];
+  uint32_t qf[DK / 16][4];
 #pragma unroll
-  for (int ks = 0; ks < D / 16; ++ks) {
+  for (int ks = 0; ks < DK / 16; ++ks) {
     const int col = ks * 16 + tig * 2;
     qf[ks][0] = *reinterpret_cast<const uint32_t*>(&q_smem[gid * C::kQStride + col]);
     qf[ks][1] = *reinterpret_cast<const uint32_t*>(&q_smem[(gid + 8) * C::kQStride + col]);
@@ -281,16 +308,16 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     qf[ks][3] = *reinterpret_cast<const uint32_t*>(&q_smem[(gid + 8) * C::kQStride + col + 8]);
   }
 
-  float oacc[D / 8][4];
+  float oacc[DV / 8][4];
 #pragma unroll
-  for (int i = 0; i < D / 8; ++i) oacc[i][0] = oacc[i][1] = oacc[i][2] = oacc[i][3] = 0.f;
+  for (int i = 0; i < DV / 8; ++i) oacc[i][0] = oacc[i][1] = oacc[i][2] = oacc[i][3] = 0.f;
   float m_run[2] = {-INFINITY, -INFINITY};
   float l_run[2] = {0.f, 0.f};  // per-thread partial row sums (reduced over the quad at the end)
 
   // FP8 pool: K and V are bytes * per-head scale; the scales factor out of both products
   const float scale_log2 = p.scale_log2;
   const int new_pos = kv_len - 1;  // position of this step's token (decode)
-  const bool owns_new = p.fused && new_pos >= start && new_pos < end;
+  const bool owns_new = !SEPARATE && p.fused && new_pos >= start && new_pos < end;
   const int r0 = warp * 16;        // this warp's token slice inside a tile
 
   for (int i = 0; i < n_tiles; ++i) {
@@ -299,9 +326,9 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     const int tok0 = start + i * kTile;
     mbar_wait_bounded(&full_bar[s], phase, abort_flag, kStatusAttnTimeout);
     uint8_t* ktile = smem + s * C::kStageBytes;
-    uint8_t* vtile = ktile + C::kTileBytes;
+    uint8_t* vtile = ktile + C::kTileBytesK;
 
-    if (owns_new && new_pos >= tok0 + r0 && new_pos < tok0 + r0 + 16) {
+    if (!SEPARATE && owns_new && new_pos >= tok0 + r0 && new_pos < tok0 + r0 + 16) {
       // This warp's slice contains the new token: rotate k, store k and v to the pool and patch the tile.
       const int rr = new_pos - tok0;
       const __nv_bfloat16* kn = qkv_t + G * D;
@@ -344,14 +371,14 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
       __syncwarp();
     }
 
-    if (tok0 + r0 < end) {
+    if (tok0 + r0 < end && (!SEPARATE || tok0 + r0 + 16 > key_begin)) {
       // ---- S = Q K^T for this warp's 16 tokens ----
       float sacc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
       const int ld_row = r0 + ((lane >> 4) << 3) + (lane & 7);  // token row this lane addresses
       const int ld_kh = (lane >> 3) & 1;
       const uint32_t kbase = smem_u32(ktile) + ld_row * 128;
 #pragma unroll
-      for (int ks = 0; ks < D / 16; ++ks) {
+      for (int ks = 0; ks < DK / 16; ++ks) {
         const int chunk16 = (ks * 2 + ld_kh) & 7;
         const int sub = (ks * 2) >> 3;
         uint32_t b0, b1, b2, b3;
@@ -367,7 +394,7 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
         for (int c = 0; c < 4; ++c) {
           const int tok = tok0 + r0 + nt * 8 + tig * 2 + (c & 1);
           float v = sacc[nt][c] * scale_log2;
-          if (tok >= end) v = -INFINITY;
+          if (tok >= end || (SEPARATE && tok < key_begin)) v = -INFINITY;
           sacc[nt][c] = v;
           mx[c >> 1] = fmaxf(mx[c >> 1], v);
         }
@@ -408,7 +435,7 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
         pl[3] = pack_bf16x2(pr[1][2], pr[1][3]);
       }
 #pragma unroll
-      for (int i2 = 0; i2 < D / 8; ++i2) {
+      for (int i2 = 0; i2 < DV / 8; ++i2) {
         oacc[i2][0] *= alpha[0];
         oacc[i2][1] *= alpha[0];
         oacc[i2][2] *= alpha[1];
@@ -419,7 +446,7 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
       const int v_dh = lane >> 4;
       const uint32_t vbase = smem_u32(vtile) + v_row * 128;
 #pragma unroll
-      for (int dn = 0; dn < D / 16; ++dn) {
+      for (int dn = 0; dn < DV / 16; ++dn) {
         const int chunk16 = (dn * 2 + v_dh) & 7;
         const int sub = (dn * 2) >> 3;
         uint32_t b0, b1, b2, b3;
@@ -441,14 +468,14 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 2);
   }
   consumer_barrier();  // every warp is done with the tile ring; reuse it
-  float* mo = reinterpret_cast<float*>(smem);                 // [warp][16][D]
-  float* mm = mo + kConsumerWarps * 16 * D;                   // [warp][16]
+  float* mo = reinterpret_cast<float*>(smem);                 // [warp][16][DV]
+  float* mm = mo + kConsumerWarps * 16 * DV;                   // [warp][16]
   float* ml = mm + kConsumerWarps * 16;                       // [warp][16]
 #pragma unroll
-  for (int i2 = 0; i2 < D / 8; ++i2) {
+  for (int i2 = 0; i2 < DV / 8; ++i2) {
     const int col = i2 * 8 + tig * 2;
-    float* o0 = mo + (warp * 16 + gid) * D + col;
-    float* o1 = mo + (warp * 16 + gid + 8) * D + col;
+    float* o0 = mo + (warp * 16 + gid) * DV + col;
+    float* o1 = mo + (warp * 16 + gid + 8) * DV + col;
     o0[0] = oacc[i2][0];
     o0[1] = oacc[i2][1];
     o1[0] = oacc[i2][2];
@@ -461,9 +488,9 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     ml[warp * 16 + gid + 8] = l_run[1];
   }
   consumer_barrier();
-  for (int i = tid; i < G * D; i += kConsumerThreads) {
-    const int g = i / D;
-    const int d = i - g * D;
+  for (int i = tid; i < G * DV; i += kConsumerThreads) {
+    const int g = i / DV;
+    const int d = i - g * DV;
     float m = -INFINITY;
 #pragma unroll
     for (int w = 0; w < kConsumerWarps; ++w) m = fmaxf(m, mm[w * 16 + g]);
@@ -472,16 +499,16 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
 #pragma unroll
       for (int w = 0; w < kConsumerWarps; ++w) {
         const float sc = exp2f(mm[w * 16 + g] - m);
-        acc += mo[(w * 16 + g) * D + d] * sc;
+        acc += mo[(w * 16 + g) * DV + d] * sc;
         lsum += ml[w * 16 + g] * sc;
       }
     }
     const float o = lsum > 0.f ? acc / lsum : 0.f;
     const int64_t qh = static_cast<int64_t>(t) * p.nq + h * G + g;
     if (p.num_splits == 1) {
-      store_output<D>(p, t, h * G + g, d, o, ml + kConsumerWarps * 16, consumer_barrier);
+      store_output<DV>(p, t, h * G + g, d, o, ml + kConsumerWarps * 16, consumer_barrier);
     } else {
-      p.ws_o[(qh * p.num_splits + split) * D + d] = o;
+      p.ws_o[(qh * p.num_splits + split) * DV + d] = o;
       if (d == 0) p.ws_lse[qh * p.num_splits + split] = lsum > 0.f ? m + log2f(lsum) : -INFINITY;
     }
   }
@@ -498,11 +525,12 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
 // once per token.  Keys and values are already in the pool (b200_rope_append ran before); the queries are
 // rotated here, in registers.  bf16 pool only.
 // ---------------------------------------------------------------------------------------------
-template <int D>
+template <int DK, int DV, bool SEPARATE>
 __global__ void __launch_bounds__(kThreads, 2)
 paged_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, Params p,
                      const int32_t* __restrict__ units) {
-  using C = Cfg<D>;
+  using C = Cfg<DK, DV>;
+  constexpr int D = DK;  // fused layout: one width for queries, keys and values
   const int tid = threadIdx.x;
   const int warp = tid >> 5;
   const int lane = tid & 31;
@@ -519,9 +547,13 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
     pdl_wait();
     return;
   }
-  int max_kv = 0;
-  for (int j = 0; j < n_tok; ++j) max_kv = max(max_kv, p.kv_len[t0 + j]);
-  const int n_tiles = (max_kv + kTile - 1) / kTile;
+  int max_kv = 0, min_kv = 0x7fffffff;
+  for (int j = 0; j < n_tok; ++j) {
+    max_kv = max(max_kv, p.kv_len[t0 + j]);
+    min_kv = min(min_kv, p.kv_len[t0 + j]);
+  }
+  const int base = SEPARATE ? first_tile_key(p, min_kv) : 0;
+  const int n_tiles = (max_kv - base + kTile - 1) / kTile;
 
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -549,7 +581,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
       for (int i = 0; i < n_tiles; ++i) {
         const int s = i % kStages;
         const uint32_t phase = (i / kStages) & 1;
-        const int tok0 = i * kTile;
+        const int tok0 = base + i * kTile;
         const int c = tok0 / p.chunk;
         if (c != cur_c) {
           cur_c = c;
@@ -558,13 +590,12 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
         const int tok_row = cur_id * p.chunk + (tok0 - c * p.chunk);
         mbar_wait_bounded(&empty_bar[s], phase ^ 1, abort_flag, kStatusAttnTimeout);
         uint8_t* kdst = smem + s * C::kStageBytes;
-        uint8_t* vdst = kdst + C::kTileBytes;
+        uint8_t* vdst = kdst + C::kTileBytesK;
         mbar_arrive_expect_tx(&full_bar[s], C::kStageBytes);
 #pragma unroll
-        for (int sub = 0; sub < C::kSub; ++sub) {
-          tma_load_3d(kdst + sub * C::kSubBytes, &map_k, &full_bar[s], sub * 64, h, tok_row);
-          tma_load_3d(vdst + sub * C::kSubBytes, &map_v, &full_bar[s], sub * 64, h, tok_row);
-        }
+        for (int sub = 0; sub < C::kSubK; ++sub) tma_load_3d(kdst + sub * C::kSubBytes, &map_k, &full_bar[s], sub * 64, h, tok_row);
+#pragma unroll
+        for (int sub = 0; sub < C::kSubV; ++sub) tma_load_3d(vdst + sub * C::kSubBytes, &map_v, &full_bar[s], sub * 64, h, tok_row);
       }
     }
     return;
@@ -576,7 +607,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
   pdl_wait();  // qkv is an earlier kernel's output
 
   // This thread's two MMA rows: (token, head) and the keys the token may see.
-  int tok_r[2], head_r[2], kv_r[2];
+  int tok_r[2], head_r[2], kv_r[2], first_r[2];
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
     const int rho = warp * 16 + gid + r * 8;
@@ -584,18 +615,32 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
     head_r[r] = rho - j * G;
     tok_r[r] = j < n_tok ? t0 + j : -1;
     kv_r[r] = j < n_tok ? p.kv_len[t0 + j] : 0;
+    first_r[r] = SEPARATE ? first_key(p, kv_r[r]) : 0;
   }
   // Q fragments straight from global memory, rotated in registers: the thread that holds columns
   // (c, c+1) of a row also holds (c + D/2, c + 1 + D/2), the RoPE partners.
-  uint32_t qf[D / 16][4];
+  uint32_t qf[DK / 16][4];
 #pragma unroll
-  for (int ks = 0; ks < D / 16; ++ks) qf[ks][0] = qf[ks][1] = qf[ks][2] = qf[ks][3] = 0u;
-  {
+  for (int ks = 0; ks < DK / 16; ++ks) qf[ks][0] = qf[ks][1] = qf[ks][2] = qf[ks][3] = 0u;
+  if (SEPARATE) {
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      if (tok_r[r] < 0) continue;
+      const __nv_bfloat16* q = p.qkv + tok_r[r] * p.q_token + static_cast<int64_t>(h) * p.q_group + head_r[r] * p.q_head;
+#pragma unroll
+      for (int ks = 0; ks < DK / 16; ++ks)
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          const int j = ks * 16 + tig * 2 + half * 8;
+          if (j < p.dk) qf[ks][r + 2 * half] = *reinterpret_cast<const uint32_t*>(q + j);
+        }
+    }
+  } else {
     const bool rope = p.cos != nullptr;
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
       if (tok_r[r] < 0) continue;
-      const __nv_bfloat16* q = p.qkv + (static_cast<int64_t>(tok_r[r]) * p.nkv + h) * (G + 2) * D + head_r[r] * D;
+      const __nv_bfloat16* q = p.qkv + tok_r[r] * p.q_token + static_cast<int64_t>(h) * p.q_group + head_r[r] * p.q_head;
       const int64_t pq = rope ? p.pos_q[tok_r[r]] : 0;
       const __nv_bfloat16* cs = p.cos + pq * (D / 2);
       const __nv_bfloat16* sn = p.sin + pq * (D / 2);
@@ -620,9 +665,9 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
     }
   }
 
-  float oacc[D / 8][4];
+  float oacc[DV / 8][4];
 #pragma unroll
-  for (int i = 0; i < D / 8; ++i) oacc[i][0] = oacc[i][1] = oacc[i][2] = oacc[i][3] = 0.f;
+  for (int i = 0; i < DV / 8; ++i) oacc[i][0] = oacc[i][1] = oacc[i][2] = oacc[i][3] = 0.f;
   float m_run[2] = {-INFINITY, -INFINITY};
   float l_run[2] = {0.f, 0.f};
   const float scale_log2 = p.scale_log2;
@@ -630,15 +675,19 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
   int warp_kv = max(kv_r[0], kv_r[1]);
 #pragma unroll
   for (int o = 4; o < 32; o <<= 1) warp_kv = max(warp_kv, __shfl_xor_sync(0xffffffffu, warp_kv, o));
+  // ... and, under a window, the first key any of them sees (rows without a token see none)
+  int warp_first = min(kv_r[0] > 0 ? first_r[0] : 0x7fffffff, kv_r[1] > 0 ? first_r[1] : 0x7fffffff);
+#pragma unroll
+  for (int o = 4; o < 32; o <<= 1) warp_first = min(warp_first, __shfl_xor_sync(0xffffffffu, warp_first, o));
 
   for (int i = 0; i < n_tiles; ++i) {
     const int s = i % kStages;
     const uint32_t phase = (i / kStages) & 1;
-    const int tok0 = i * kTile;
+    const int tok0 = base + i * kTile;
     mbar_wait_bounded(&full_bar[s], phase, abort_flag, kStatusAttnTimeout);
     uint8_t* ktile = smem + s * C::kStageBytes;
-    uint8_t* vtile = ktile + C::kTileBytes;
-    if (tok0 < warp_kv) {
+    uint8_t* vtile = ktile + C::kTileBytesK;
+    if (tok0 < warp_kv && (!SEPARATE || tok0 + kTile > warp_first)) {
       // ---- S = Q K^T: 16 rows x 64 tokens ----
       float sacc[8][4];
 #pragma unroll
@@ -646,7 +695,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
       const int ld_sub = ((lane >> 4) << 3) + (lane & 7);  // token row inside a 16-token slab
       const int ld_kh = (lane >> 3) & 1;
 #pragma unroll
-      for (int ks = 0; ks < D / 16; ++ks) {
+      for (int ks = 0; ks < DK / 16; ++ks) {
         const int chunk16 = (ks * 2 + ld_kh) & 7;
         const int sub = (ks * 2) >> 3;
 #pragma unroll
@@ -666,7 +715,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
         for (int c = 0; c < 4; ++c) {
           const int tok = tok0 + nt * 8 + tig * 2 + (c & 1);
           float v = sacc[nt][c] * scale_log2;
-          if (tok >= kv_r[c >> 1]) v = -INFINITY;
+          if (tok >= kv_r[c >> 1] || (SEPARATE && tok < first_r[c >> 1])) v = -INFINITY;
           sacc[nt][c] = v;
           mx[c >> 1] = fmaxf(mx[c >> 1], v);
         }
@@ -683,7 +732,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
         l_run[r] *= alpha[r];
       }
 #pragma unroll
-      for (int i2 = 0; i2 < D / 8; ++i2) {
+      for (int i2 = 0; i2 < DV / 8; ++i2) {
         oacc[i2][0] *= alpha[0];
         oacc[i2][1] *= alpha[0];
         oacc[i2][2] *= alpha[1];
@@ -712,7 +761,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
         const int v_row = slab * 16 + v_sub;
         const uint32_t vbase = smem_u32(vtile) + v_row * 128;
 #pragma unroll
-        for (int dn = 0; dn < D / 16; ++dn) {
+        for (int dn = 0; dn < DV / 16; ++dn) {
           const int chunk16 = (dn * 2 + v_dh) & 7;
           const int sub = (dn * 2) >> 3;
           uint32_t b0, b1, b2, b3;
@@ -735,11 +784,11 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
     l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 2);
     if (tok_r[r] < 0) continue;
     const float inv = l_run[r] > 0.f ? 1.f / l_run[r] : 0.f;  // a token that sees no key gets zeros, as flash-attn does
-    __nv_bfloat16* o = p.out + (static_cast<int64_t>(tok_r[r]) * p.nq + h * G + head_r[r]) * D;
+    __nv_bfloat16* o = p.out + (static_cast<int64_t>(tok_r[r]) * p.nq + h * G + head_r[r]) * p.dv;
 #pragma unroll
-    for (int i2 = 0; i2 < D / 8; ++i2) {
+    for (int i2 = 0; i2 < DV / 8; ++i2) {
       const int col = i2 * 8 + tig * 2;
-      *reinterpret_cast<uint32_t*>(o + col) = pack_bf16x2(oacc[i2][2 * r] * inv, oacc[i2][2 * r + 1] * inv);
+      if (col < p.dv) *reinterpret_cast<uint32_t*>(o + col) = pack_bf16x2(oacc[i2][2 * r] * inv, oacc[i2][2 * r + 1] * inv);
     }
   }
 }
@@ -755,8 +804,9 @@ __global__ void __launch_bounds__(D) combine_kernel(Params p) {
   const int kv_len = p.kv_len[t];
   float o = 0.f;
   if (kv_len > 0) {
-    const int L = split_length(kv_len, p.num_splits, p.min_split);
-    const int n_act = (kv_len + L - 1) / L;
+    const int keys = kv_len - first_tile_key(p, kv_len);
+    const int L = split_length(keys, p.num_splits, p.min_split);
+    const int n_act = (keys + L - 1) / L;
     const float* lse = p.ws_lse + static_cast<int64_t>(qh) * p.num_splits;
     float mx = -INFINITY;
     for (int s = 0; s < n_act; ++s) mx = fmaxf(mx, lse[s]);
@@ -805,7 +855,13 @@ static int fill_params(const b200_attention_args* a, Params& p) {
   if (!a || (!a->qkv && !a->qkv_partials) || !a->k_cache || !a->v_cache || !a->kv_seq_lengths || !a->block_table)
     return B200_ERR_INVALID_ARGUMENT;
   if (a->qkv_partials && (a->qkv_num_splits < 1 || !aligned16(a->qkv_partials))) return B200_ERR_INVALID_ARGUMENT;
-  if (a->head_dim != 64 && a->head_dim != 128) return B200_ERR_INVALID_ARGUMENT;
+  if (a->separate) {  // finished queries, [keys | values] pool rows
+    if (a->head_dim <= 0 || a->head_dim > 128 || a->value_dim <= 0 || a->value_dim > 128 || a->head_dim % 8 != 0 ||
+        a->value_dim % 8 != 0 || a->pool_row_elems % 8 != 0 || a->kv_cache_fp8 || a->fuse_rope_append || a->out_q || !a->qkv)
+      return B200_ERR_INVALID_ARGUMENT;
+  } else if ((a->head_dim != 64 && a->head_dim != 128) || a->window > 0) {
+    return B200_ERR_INVALID_ARGUMENT;
+  }
   if (a->num_tokens <= 0 || a->num_kv_heads <= 0 || a->num_q_heads % a->num_kv_heads != 0)
     return B200_ERR_INVALID_ARGUMENT;
   const int G = a->num_q_heads / a->num_kv_heads;
@@ -857,6 +913,14 @@ static int fill_params(const b200_attention_args* a, Params& p) {
   p.min_split = a->chunk_size < 256 ? a->chunk_size : 256;
   const float scale = a->softmax_scale > 0.f ? a->softmax_scale : 1.0f / sqrtf(static_cast<float>(a->head_dim));
   p.scale_log2 = scale * 1.4426950408889634f;
+  p.separate = a->separate;
+  p.dk = a->head_dim;
+  p.dv = a->separate ? a->value_dim : a->head_dim;
+  p.q_head = p.dk;
+  p.q_group = (a->separate ? G : G + 2) * p.dk;
+  p.q_token = static_cast<int64_t>(p.nkv) * p.q_group;
+  p.pool_row = a->separate ? a->pool_row_elems : static_cast<int64_t>(p.nkv) * p.dk;
+  p.window = a->window > 0 ? a->window : 0;
   p.ws_o = nullptr;
   p.ws_lse = nullptr;
   p.k_scale = a->k_scale;
@@ -867,49 +931,57 @@ static int fill_params(const b200_attention_args* a, Params& p) {
   return B200_OK;
 }
 
-template <int D>
-static int launch_attention(const b200_attention_args* a, Params& p, cudaStream_t stream) {
-  using C = Cfg<D>;
-  constexpr int kElem = 2;
-  const uint64_t dims[3] = {static_cast<uint64_t>(D), static_cast<uint64_t>(p.nkv),
-                            static_cast<uint64_t>(p.num_chunks) * p.chunk};
-  const uint64_t strides[2] = {static_cast<uint64_t>(D) * kElem, static_cast<uint64_t>(p.nkv) * D * kElem};
+static bool pool_maps(const Params& p, const CUtensorMap*& mk, const CUtensorMap*& mv) {
+  const uint64_t tokens = static_cast<uint64_t>(p.num_chunks) * p.chunk;
+  const uint64_t kd[3] = {static_cast<uint64_t>(p.dk), static_cast<uint64_t>(p.nkv), tokens};
+  const uint64_t vd[3] = {static_cast<uint64_t>(p.dv), static_cast<uint64_t>(p.nkv), tokens};
+  const uint64_t ks[2] = {static_cast<uint64_t>(p.dk) * 2, static_cast<uint64_t>(p.pool_row) * 2};
+  const uint64_t vs[2] = {static_cast<uint64_t>(p.dv) * 2, static_cast<uint64_t>(p.pool_row) * 2};
   const uint32_t box[3] = {64u, 1, kTile};
-  const CUtensorMapDataType dt = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
-  const CUtensorMap* mk = get_tensor_map(p.k_cache, 3, dims, strides, box, CU_TENSOR_MAP_SWIZZLE_128B,
-                                         CU_TENSOR_MAP_L2_PROMOTION_L2_256B, dt);
-  const CUtensorMap* mv = get_tensor_map(p.v_cache, 3, dims, strides, box, CU_TENSOR_MAP_SWIZZLE_128B,
-                                         CU_TENSOR_MAP_L2_PROMOTION_L2_256B, dt);
-  if (!mk || !mv) return B200_ERR_DRIVER;
+  mk = get_tensor_map(p.k_cache, 3, kd, ks, box, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B);
+  mv = get_tensor_map(p.v_cache, 3, vd, vs, box, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B);
+  return mk && mv;
+}
+
+template <int DK, int DV, bool SEPARATE>
+static int launch_attention(Params& p, cudaStream_t stream) {
+  using C = Cfg<DK, DV>;
+  const CUtensorMap *mk, *mv;
+  if (!pool_maps(p, mk, mv)) return B200_ERR_DRIVER;
   static std::atomic<uint64_t> smem_attr_done{0};
-  if (ensure_dynamic_smem(paged_attention_kernel<D>, C::kSmemBytes, smem_attr_done) != B200_OK) return B200_ERR_LAUNCH;
+  if (ensure_dynamic_smem(paged_attention_kernel<DK, DV, SEPARATE>, C::kSmemBytes, smem_attr_done) != B200_OK) return B200_ERR_LAUNCH;
   const int64_t units = static_cast<int64_t>(p.T) * p.nkv * p.num_splits;
   if (units > 0x7fffffff) return B200_ERR_INVALID_ARGUMENT;
-  int rc = launch_pdl(paged_attention_kernel<D>, dim3(static_cast<unsigned>(units)), dim3(kThreads), C::kSmemBytes,
+  int rc = launch_pdl(paged_attention_kernel<DK, DV, SEPARATE>, dim3(static_cast<unsigned>(units)), dim3(kThreads), C::kSmemBytes,
                       stream, *mk, *mv, p);
   if (rc != B200_OK) return rc;
-  if (p.num_splits > 1) rc = launch_pdl(combine_kernel<D>, dim3(p.T * p.nq), dim3(D), 0, stream, p);
+  if (p.num_splits > 1) rc = launch_pdl(combine_kernel<DV>, dim3(p.T * p.nq), dim3(DV), 0, stream, p);
   return rc;
 }
 
-template <int D>
+template <int DK, int DV, bool SEPARATE>
 static int launch_prefill(Params& p, const int32_t* units, int num_units, cudaStream_t stream) {
-  using C = Cfg<D>;
-  const uint64_t dims[3] = {static_cast<uint64_t>(D), static_cast<uint64_t>(p.nkv),
-                            static_cast<uint64_t>(p.num_chunks) * p.chunk};
-  const uint64_t strides[2] = {static_cast<uint64_t>(D) * 2, static_cast<uint64_t>(p.nkv) * D * 2};
-  const uint32_t box[3] = {64u, 1, kTile};
-  const CUtensorMap* mk = get_tensor_map(p.k_cache, 3, dims, strides, box, CU_TENSOR_MAP_SWIZZLE_128B,
-                                         CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16);
-  const CUtensorMap* mv = get_tensor_map(p.v_cache, 3, dims, strides, box, CU_TENSOR_MAP_SWIZZLE_128B,
-                                         CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16);
-  if (!mk || !mv) return B200_ERR_DRIVER;
+  using C = Cfg<DK, DV>;
+  const CUtensorMap *mk, *mv;
+  if (!pool_maps(p, mk, mv)) return B200_ERR_DRIVER;
   static std::atomic<uint64_t> smem_attr_done{0};
-  if (ensure_dynamic_smem(paged_prefill_kernel<D>, C::kSmemBytes, smem_attr_done) != B200_OK) return B200_ERR_LAUNCH;
+  if (ensure_dynamic_smem(paged_prefill_kernel<DK, DV, SEPARATE>, C::kSmemBytes, smem_attr_done) != B200_OK) return B200_ERR_LAUNCH;
   const int64_t ctas = static_cast<int64_t>(num_units) * p.nkv;
   if (ctas > 0x7fffffff) return B200_ERR_INVALID_ARGUMENT;
-  return launch_pdl(paged_prefill_kernel<D>, dim3(static_cast<unsigned>(ctas)), dim3(kThreads), C::kSmemBytes, stream, *mk,
+  return launch_pdl(paged_prefill_kernel<DK, DV, SEPARATE>, dim3(static_cast<unsigned>(ctas)), dim3(kThreads), C::kSmemBytes, stream, *mk,
                     *mv, p, units);
+}
+
+// The layout and the tile widths that hold the head dims.
+template <typename F>
+static int by_layout(const Params& p, F&& f) {
+  const std::integral_constant<int, 64> w64;
+  const std::integral_constant<int, 128> w128;
+  const std::false_type fused;
+  const std::true_type separate;
+  if (!p.separate) return p.dk == 128 ? f(w128, w128, fused) : f(w64, w64, fused);
+  if (p.dk <= 64) return p.dv <= 64 ? f(w64, w64, separate) : f(w64, w128, separate);
+  return p.dv <= 64 ? f(w128, w64, separate) : f(w128, w128, separate);
 }
 
 }  // namespace attn
@@ -930,10 +1002,9 @@ int b200_paged_prefill_attention(const b200_attention_args* a, const int32_t* un
   int rc = attn::fill_params(a, p);
   if (rc != B200_OK) return rc;
   if (!a->out || a->out_q || !a->qkv || !units || num_units <= 0 || a->kv_cache_fp8) return B200_ERR_INVALID_ARGUMENT;
-  if (64 % p.G != 0) return B200_ERR_INVALID_ARGUMENT;  // group sizes 1, 2, 4, 8, 16
+  if (64 % p.G != 0 && !p.separate) return B200_ERR_INVALID_ARGUMENT;  // group sizes 1, 2, 4, 8, 16
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  return a->head_dim == 128 ? attn::launch_prefill<128>(p, units, num_units, s)
-                            : attn::launch_prefill<64>(p, units, num_units, s);
+  return attn::by_layout(p, [&](auto dk, auto dv, auto sep) { return attn::launch_prefill<dk, dv, sep>(p, units, num_units, s); });
 }
 
 size_t b200_paged_attention_workspace_bytes(int num_tokens, int num_q_heads, int head_dim, int num_splits) {
@@ -964,14 +1035,14 @@ int b200_paged_attention(const b200_attention_args* a, b200_stream_t stream) {
   if (a->qkv_partials && (a->num_q_heads / a->num_kv_heads + 2) * a->head_dim % 4 != 0) return B200_ERR_ALIGNMENT;
   if (a->num_splits > 1) {
     const size_t need =
-        b200_paged_attention_workspace_bytes(a->num_tokens, a->num_q_heads, a->head_dim, a->num_splits);
+        b200_paged_attention_workspace_bytes(a->num_tokens, a->num_q_heads, a->separate ? (a->value_dim <= 64 ? 64 : 128) : a->head_dim, a->num_splits);
     if (!a->workspace || a->workspace_bytes < need) return B200_ERR_WORKSPACE;
     p.ws_o = static_cast<float*>(a->workspace);
-    p.ws_lse = p.ws_o + static_cast<size_t>(a->num_tokens) * a->num_q_heads * a->num_splits * a->head_dim;
+    p.ws_lse = p.ws_o + static_cast<size_t>(a->num_tokens) * a->num_q_heads * a->num_splits * (a->separate ? (a->value_dim <= 64 ? 64 : 128) : a->head_dim);
   }
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (a->kv_cache_fp8) return attn8::launch_attention_fp8(p, a->kv_cache_fp8 != 2, s);
-  return a->head_dim == 128 ? attn::launch_attention<128>(a, p, s) : attn::launch_attention<64>(a, p, s);
+  return attn::by_layout(p, [&](auto dk, auto dv, auto sep) { return attn::launch_attention<dk, dv, sep>(p, s); });
 }
 
 }  // extern "C"

@@ -1,0 +1,83 @@
+// Attention over the [keys | values] pool on the CUDA cores, for 32-bit models and head dims the tensor-core kernels do not
+// take: one warp per (token, query head), 32 keys at a time, online softmax in fp32.
+#include "common.cuh"
+
+namespace b200 {
+namespace attn_simt {
+
+constexpr int kWarps = 4;
+constexpr int kMaxDim = 256;
+
+template <typename T>
+__global__ void __launch_bounds__(kWarps * 32)
+attention_kernel(b200_attention_args a) {
+  __shared__ float q_s[kWarps][kMaxDim];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int64_t unit = static_cast<int64_t>(blockIdx.x) * kWarps + warp;
+  if (unit >= static_cast<int64_t>(a.num_tokens) * a.num_q_heads) return;
+  const int t = static_cast<int>(unit / a.num_q_heads), head = static_cast<int>(unit - static_cast<int64_t>(t) * a.num_q_heads);
+  const int g = head / (a.num_q_heads / a.num_kv_heads), dk = a.head_dim, dv = a.value_dim;
+  const int kv_len = a.kv_seq_lengths[t], row = a.row_of_token ? a.row_of_token[t] : t;
+  const int first = a.window > 0 ? max(kv_len - a.window, 0) : 0;
+  const T* q = static_cast<const T*>(a.qkv) + unit * dk;
+  for (int i = lane; i < dk; i += 32) q_s[warp][i] = simt::to_f32(q[i]);
+  __syncwarp();
+  const int32_t* table = a.block_table + static_cast<int64_t>(row) * a.max_chunks_per_row;
+  const T* keys = static_cast<const T*>(a.k_cache) + g * dk;
+  const T* values = static_cast<const T*>(a.v_cache) + g * dv;
+  float m = -INFINITY, l = 0.f, acc[kMaxDim / 32];
+#pragma unroll
+  for (int e = 0; e < kMaxDim / 32; ++e) acc[e] = 0.f;
+  for (int k0 = first; k0 < kv_len; k0 += 32) {
+    const int key = k0 + lane;
+    int64_t at = 0;
+    float s = -INFINITY;
+    if (key < kv_len) {
+      const int c = key / a.chunk_size;
+      at = (static_cast<int64_t>(table[c]) * a.chunk_size + (key - c * a.chunk_size)) * a.pool_row_elems;
+      const T* k = keys + at;
+      float d = 0.f;
+      for (int i = 0; i < dk; ++i) d = fmaf(q_s[warp][i], simt::to_f32(k[i]), d);
+      s = d * a.softmax_scale;
+    }
+    const float m_new = fmaxf(m, warp_max(s));
+    const float alpha = expf(m - m_new), p = expf(s - m_new);  // (some key is visible: m_new is finite)
+    m = m_new;
+    l = l * alpha + warp_sum(p);
+#pragma unroll
+    for (int e = 0; e < kMaxDim / 32; ++e) acc[e] *= alpha;
+    const int n = min(32, kv_len - k0);
+    for (int j = 0; j < n; ++j) {
+      const float pj = __shfl_sync(0xffffffffu, p, j);
+      const T* v = values + __shfl_sync(0xffffffffu, at, j);
+#pragma unroll
+      for (int e = 0; e < kMaxDim / 32; ++e)
+        if (lane + e * 32 < dv) acc[e] = fmaf(pj, simt::to_f32(v[lane + e * 32]), acc[e]);
+    }
+  }
+  T* out = static_cast<T*>(a.out) + unit * dv;
+#pragma unroll
+  for (int e = 0; e < kMaxDim / 32; ++e)
+    if (lane + e * 32 < dv) simt::store_as(out + lane + e * 32, l > 0.f ? acc[e] / l : 0.f);
+}
+
+}  // namespace attn_simt
+}  // namespace b200
+
+extern "C" int b200_attention_simt(const b200_attention_args* a, int dtype, b200_stream_t stream) {
+  using namespace b200;
+  if (!a || !a->separate || !a->qkv || !a->k_cache || !a->v_cache || !a->kv_seq_lengths || !a->block_table || !a->out ||
+      a->num_tokens <= 0 || a->num_kv_heads <= 0 || a->num_q_heads <= 0 || a->num_q_heads % a->num_kv_heads != 0 || a->head_dim <= 0 ||
+      a->head_dim > attn_simt::kMaxDim || a->value_dim <= 0 || a->value_dim > attn_simt::kMaxDim || a->chunk_size <= 0 ||
+      a->pool_row_elems < a->num_kv_heads * (a->head_dim + a->value_dim))
+    return B200_ERR_INVALID_ARGUMENT;
+  const int64_t units = static_cast<int64_t>(a->num_tokens) * a->num_q_heads;
+  const dim3 grid(static_cast<unsigned>((units + attn_simt::kWarps - 1) / attn_simt::kWarps));
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (dtype == B200_DTYPE_F32) return launch_pdl(attn_simt::attention_kernel<float>, grid, dim3(attn_simt::kWarps * 32), 0, s, *a);
+  if (dtype == B200_DTYPE_BF16)
+    return launch_pdl(attn_simt::attention_kernel<__nv_bfloat16>, grid, dim3(attn_simt::kWarps * 32), 0, s, *a);
+  return B200_ERR_INVALID_ARGUMENT;
+}

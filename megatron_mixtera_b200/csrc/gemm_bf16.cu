@@ -55,7 +55,18 @@ struct Params {
   // weight rows [b * N, (b + 1) * N) into y + b * y_batch.  m_blocks: token blocks per batch (blockIdx.z holds both).
   int m_blocks = 1, x_batch = 0;
   int64_t y_batch = 0;
+  // gated == kGatedClamped: y = g' sigmoid(glu_alpha g') (u' + 1) with g' = min(g, glu_limit), u' clamped to [-glu_limit, glu_limit], all
+  // in fp32; row_scale (NULL: 1) multiplies both products of a token first.
+  float glu_limit = 0.f, glu_alpha = 0.f;
+  const float* row_scale = nullptr;
 };
+constexpr int kGatedSilu = 1, kGatedClamped = 2;  // Params::gated
+
+__device__ __forceinline__ float clamped_glu(float g, float u, float limit, float alpha) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g / (1.f + expf(-alpha * g)) * (u + 1.f);
+}
 
 __device__ __forceinline__ float apply_act(float v, int act) {
   if (act == B200_ACT_RELU2) {
@@ -135,12 +146,11 @@ __device__ __forceinline__ void epilogue_barrier() { asm volatile("bar.sync 2, 1
 // stores (whole-K units), or stores the fp32 partial tile for splitk_reduce_kernel.
 template <int BT>
 __device__ __forceinline__ void epilogue(const Params& p, uint32_t tmem_base, uint8_t* stage_smem, int n_tile, int split,
-                                         int m_block, __nv_bfloat16* __restrict__ y) {
+                                         int m0, int m_end, __nv_bfloat16* __restrict__ y) {
   const int tid = threadIdx.x;
   const int warp = tid >> 5;
   const int lane = tid & 31;
   const int n0 = n_tile * kTileN;
-  const int m0 = m_block * BT;
   const int n = n0 + warp * 32 + lane;          // output feature held by this thread (TMEM lane)
   const bool n_ok = n < p.N;
   const uint32_t lane_addr = tmem_base + (static_cast<uint32_t>(warp * 32) << 16);
@@ -164,16 +174,24 @@ __device__ __forceinline__ void epilogue(const Params& p, uint32_t tmem_base, ui
 #pragma unroll
       for (int j = 0; j < 16; ++j) {
         const int jj = is_gate ? j + 16 : j;            // the other side's tokens
-        xch[(c0 + jj) * 64 + f] = bf16_round(__uint_as_float(is_gate ? r[j + 16] : r[j]));
+        const float parked = __uint_as_float(is_gate ? r[j + 16] : r[j]);
+        xch[(c0 + jj) * 64 + f] = p.gated == kGatedClamped ? parked : bf16_round(parked);
       }
       __syncthreads();
       if (col_ok) {
 #pragma unroll
         for (int j = 0; j < 16; ++j) {
           const int m = m0 + c0 + own0 + j;
-          if (m < p.M) {
-            const float mine = bf16_round(__uint_as_float(is_gate ? r[j] : r[j + 16]));
+          if (m < m_end) {
+            const float raw = __uint_as_float(is_gate ? r[j] : r[j + 16]);
             const float other = xch[(c0 + own0 + j) * 64 + f];
+            if (p.gated == kGatedClamped) {
+              const float sc = p.row_scale != nullptr ? p.row_scale[m] : 1.f;
+              const float v = clamped_glu((is_gate ? raw : other) * sc, (is_gate ? other : raw) * sc, p.glu_limit, p.glu_alpha);
+              y[static_cast<int64_t>(m) * p.ldy + out_col] = __float2bfloat16_rn(v);
+              continue;
+            }
+            const float mine = bf16_round(raw);
             const float g = is_gate ? mine : other;
             const float u = is_gate ? other : mine;
             const float a = bf16_round(g / (1.f + expf(-g)));
@@ -210,7 +228,7 @@ __device__ __forceinline__ void epilogue(const Params& p, uint32_t tmem_base, ui
 #pragma unroll 1
         for (int v = tid; v < kRows * 16; v += kThreads) {
           const int m = m0 + h0 + (v >> 4);
-          if (m < p.M) *reinterpret_cast<uint4*>(y + static_cast<int64_t>(m) * p.ldy + n0 + (v & 15) * 8) = tile_v[v];
+          if (m < m_end) *reinterpret_cast<uint4*>(y + static_cast<int64_t>(m) * p.ldy + n0 + (v & 15) * 8) = tile_v[v];
         }
         if (h0 + kRows < BT) epilogue_barrier();
       }
@@ -224,7 +242,7 @@ __device__ __forceinline__ void epilogue(const Params& p, uint32_t tmem_base, ui
 #pragma unroll
           for (int j = 0; j < 32; ++j) {
             const int m = m0 + c0 + j;
-            if (m < p.M) {
+            if (m < m_end) {
               float v = __uint_as_float(r[j]);
               // bias is added to the bf16-rounded product, as `matmul(x, w.t()) + bias` does
               if (p.bias != nullptr) v = bf16_round(v) + b;
@@ -255,7 +273,7 @@ __device__ __forceinline__ void epilogue(const Params& p, uint32_t tmem_base, ui
 #pragma unroll 1
         for (int v = tid; v < kRows * 32; v += kThreads) {
           const int m = m0 + h0 + (v >> 5);
-          if (m < p.M) __stcg(reinterpret_cast<float4*>(part + static_cast<int64_t>(m) * p.N + n0) + (v & 31), tile_v[v]);
+          if (m < m_end) __stcg(reinterpret_cast<float4*>(part + static_cast<int64_t>(m) * p.N + n0) + (v & 31), tile_v[v]);
         }
         if (h0 + kRows < BT) epilogue_barrier();
       }
@@ -269,7 +287,7 @@ __device__ __forceinline__ void epilogue(const Params& p, uint32_t tmem_base, ui
 #pragma unroll
           for (int j = 0; j < 32; ++j) {
             const int m = m0 + c0 + j;
-            if (m < p.M) __stcg(&part[static_cast<int64_t>(m) * p.N + n], __uint_as_float(r[j]));
+            if (m < m_end) __stcg(&part[static_cast<int64_t>(m) * p.N + n], __uint_as_float(r[j]));
           }
         }
       }
@@ -382,11 +400,180 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
   mbar_wait_bounded(accum_bar, 0, abort_flag, kStatusGemmTimeout);
   tcgen05_fence_after_sync();
 
-  epilogue<BT>(p, tmem_base, smem, n_tile, split, m_block, p.y + batch * p.y_batch);
+  epilogue<BT>(p, tmem_base, smem, n_tile, split, m0, p.M, p.y + batch * p.y_batch);
 
   tcgen05_fence_before_sync();
   __syncthreads();
   if (warp == 0) tmem_dealloc(tmem_base, C::kTmemCols);
+}
+
+// ---------------------------------------------------------------------------------------------
+// Grouped form (experts): tokens sorted by expert, a device-built list of (expert, first row, rows) tiles, each multiplied with
+// its expert's rows of the stacked weights.  A second problem (a shared expert: all tokens, weights and sizes of its own) may ride
+// in the same launch: its units come first.  Rows that a tile's box fetches past its expert's last one are computed and dropped.
+// ---------------------------------------------------------------------------------------------
+struct GroupedParams {
+  Params routed, shared;  // M, N, K, y, ldy, num_k_blocks, gated ...; N: weight rows per expert
+  const int4* tiles;
+  const int32_t* num_tiles;
+  int max_tiles, experts, routed_n_tiles, shared_n_tiles, shared_units;
+};
+
+template <int BT>
+__global__ void __launch_bounds__(kThreads, 1)
+gemm_grouped_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
+                    const __grid_constant__ CUtensorMap map_ws, const __grid_constant__ CUtensorMap map_xs,
+                    const __grid_constant__ GroupedParams gp) {
+  using C = Config<BT>;
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  uint64_t* full_bar = reinterpret_cast<uint64_t*>(smem + C::kStages * C::kStageBytes);
+  uint64_t* empty_bar = full_bar + C::kStages;
+  uint64_t* accum_bar = empty_bar + C::kStages;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(accum_bar + 1);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+
+  pdl_launch_dependents();
+  int unit = blockIdx.x;
+  const bool is_shared = unit < gp.shared_units;
+  const Params& p = is_shared ? gp.shared : gp.routed;
+  int n_tile, m0, m_end, w_row;
+  if (is_shared) {
+    n_tile = unit % gp.shared_n_tiles;
+    m0 = unit / gp.shared_n_tiles * BT;
+    m_end = p.M;
+    w_row = n_tile * kTileN;
+  } else {
+    unit -= gp.shared_units;
+    n_tile = unit % gp.routed_n_tiles;
+    const int tile = unit / gp.routed_n_tiles;
+    pdl_wait();  // the tile list is a kernel's output
+    if (tile >= min(*gp.num_tiles, gp.max_tiles)) return;
+    const int4 e = gp.tiles[tile];
+    if (static_cast<unsigned>(e.x) >= static_cast<unsigned>(gp.experts) || e.y < 0 || e.z <= 0) return;
+    m0 = e.y;
+    m_end = min(e.y + min(e.z, BT), p.M);
+    w_row = e.x * p.N + n_tile * kTileN;
+  }
+  const CUtensorMap* mw = is_shared ? &map_ws : &map_w;
+  const CUtensorMap* mx = is_shared ? &map_xs : &map_x;
+  const int num_kb = p.num_k_blocks;
+
+  if (tid == 0) {
+    for (int s = 0; s < C::kStages; ++s) {
+      mbar_init(&full_bar[s], 1);
+      mbar_init(&empty_bar[s], 1);
+    }
+    mbar_init(accum_bar, 1);
+    *abort_flag = 0;
+    fence_barrier_init();
+    prefetch_tensormap(mw);
+    prefetch_tensormap(mx);
+  }
+  if (warp == 0) {
+    tmem_alloc(tmem_slot, C::kTmemCols);
+    tmem_relinquish_alloc_permit();
+  }
+  tcgen05_fence_before_sync();
+  __syncthreads();
+  tcgen05_fence_after_sync();
+  const uint32_t tmem_base = *tmem_slot;
+
+  if (warp == 0) {
+    if (lane == 0) {
+      const int pre = num_kb < C::kStages ? num_kb : C::kStages;
+      for (int i = 0; i < pre; ++i) {
+        mbar_arrive_expect_tx(&full_bar[i], C::kStageBytes);
+        tma_load_2d(smem + i * C::kStageBytes, mw, &full_bar[i], i * kTileK, w_row);
+      }
+      pdl_wait();
+      for (int i = 0; i < pre; ++i)
+        tma_load_2d(smem + i * C::kStageBytes + C::kStageBytesW, mx, &full_bar[i], i * kTileK, m0);
+      for (int i = pre; i < num_kb; ++i) {
+        const int s = i % C::kStages;
+        mbar_wait_bounded(&empty_bar[s], ((i / C::kStages) & 1) ^ 1, abort_flag, kStatusGemmTimeout);
+        uint8_t* stage = smem + s * C::kStageBytes;
+        mbar_arrive_expect_tx(&full_bar[s], C::kStageBytes);
+        tma_load_2d(stage, mw, &full_bar[s], i * kTileK, w_row);
+        tma_load_2d(stage + C::kStageBytesW, mx, &full_bar[s], i * kTileK, m0);
+      }
+    }
+    __syncwarp();
+  } else if (warp == 1) {
+    if (lane == 0) {
+      constexpr uint32_t idesc = umma_idesc_bf16(kTileN, BT);
+      for (int i = 0; i < num_kb; ++i) {
+        const int s = i % C::kStages;
+        mbar_wait_bounded(&full_bar[s], (i / C::kStages) & 1, abort_flag, kStatusGemmTimeout);
+        tcgen05_fence_after_sync();
+        const uint32_t a_addr = smem_u32(smem + s * C::kStageBytes);
+        const uint64_t a_desc = umma_desc_k_major_sw128(a_addr);
+        const uint64_t b_desc = umma_desc_k_major_sw128(a_addr + C::kStageBytesW);
+#pragma unroll
+        for (int k = 0; k < kTileK / kUmmaK; ++k) umma_f16(tmem_base, a_desc + 2 * k, b_desc + 2 * k, idesc, (i > 0 || k > 0) ? 1u : 0u);
+        umma_commit(&empty_bar[s]);
+      }
+      umma_commit(accum_bar);
+    }
+    __syncwarp();
+  }
+  pdl_wait();
+  mbar_wait_bounded(accum_bar, 0, abort_flag, kStatusGemmTimeout);
+  tcgen05_fence_after_sync();
+  epilogue<BT>(p, tmem_base, smem, n_tile, 0, m0, m_end, p.y);
+  tcgen05_fence_before_sync();
+  __syncthreads();
+  if (warp == 0) tmem_dealloc(tmem_base, C::kTmemCols);
+}
+
+// One problem of a grouped launch: x [M][K] (row stride ldx), weights [experts * N][K].
+struct GroupedProblem {
+  const void* x;
+  const void* w;
+  int64_t ldx;
+  int experts;
+};
+
+template <int BT>
+static int launch_grouped(const GroupedProblem& routed, const GroupedProblem& shared, GroupedParams& gp, cudaStream_t stream) {
+  using C = Config<BT>;
+  auto maps = [&](const GroupedProblem& g, const Params& p, const CUtensorMap*& mw, const CUtensorMap*& mx) {
+    const uint64_t wd[2] = {static_cast<uint64_t>(p.K), static_cast<uint64_t>(p.N) * g.experts};
+    const uint64_t ws[1] = {static_cast<uint64_t>(p.K) * 2};
+    const uint32_t wb[2] = {kTileK, kTileN};
+    const uint64_t xd[2] = {static_cast<uint64_t>(p.K), static_cast<uint64_t>(p.M)};
+    const uint64_t xs[1] = {static_cast<uint64_t>(g.ldx) * 2};
+    const uint32_t xb[2] = {kTileK, BT};
+    mw = get_tensor_map(g.w, 2, wd, ws, wb, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B);
+    mx = get_tensor_map(g.x, 2, xd, xs, xb, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B);
+    return mw && mx;
+  };
+  const CUtensorMap *mw, *mx, *mws, *mxs;
+  if (!maps(routed, gp.routed, mw, mx)) return B200_ERR_DRIVER;
+  mws = mw;
+  mxs = mx;
+  gp.shared_units = 0;
+  gp.shared_n_tiles = 1;
+  if (shared.x != nullptr) {
+    if (!maps(shared, gp.shared, mws, mxs)) return B200_ERR_DRIVER;
+    gp.shared_n_tiles = (gp.shared.N + kTileN - 1) / kTileN;
+    gp.shared_units = gp.shared_n_tiles * ((gp.shared.M + BT - 1) / BT);
+  }
+  gp.routed_n_tiles = (gp.routed.N + kTileN - 1) / kTileN;
+  for (Params* p : {&gp.routed, &gp.shared}) {
+    p->num_k_blocks = (p->K + kTileK - 1) / kTileK;
+    p->num_splits = 1;
+    p->keep_partials = 0;
+    p->partials = nullptr;
+    p->bias = nullptr;
+  }
+  const int64_t units = gp.shared_units + static_cast<int64_t>(gp.routed_n_tiles) * gp.max_tiles;
+  if (units > 0x7fffffff) return B200_ERR_INVALID_ARGUMENT;
+  static std::atomic<uint64_t> smem_attr_done{0};
+  if (ensure_dynamic_smem(gemm_grouped_kernel<BT>, C::kSmemBytes, smem_attr_done) != B200_OK) return B200_ERR_LAUNCH;
+  return launch_pdl(gemm_grouped_kernel<BT>, dim3(static_cast<unsigned>(units)), dim3(kThreads), C::kSmemBytes, stream, *mw, *mx, *mws,
+                    *mxs, gp);
 }
 
 // Number of K splits: fill `ctas_per_sm` CTAs per SM when there are too few output tiles, keep at least

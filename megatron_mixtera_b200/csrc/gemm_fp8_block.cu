@@ -215,7 +215,7 @@ gemm_fp8_block_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_co
     tmem_st_32x32b_x32(lane_addr + c0, r);
   }
   tmem_st_wait();
-  epilogue<BT>(p, tmem_base, smem, n_tile, split, m_block, p.y);
+  epilogue<BT>(p, tmem_base, smem, n_tile, split, m_block * BT, p.M, p.y);
   }
 
   tcgen05_fence_before_sync();

@@ -167,7 +167,7 @@ gemm_mxfp8_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_consta
   pdl_wait();
   mbar_wait_bounded(accum_bar, 0, abort_flag, kStatusGemmTimeout);
   tcgen05_fence_after_sync();
-  epilogue<BT>(p, tmem_base, smem, n_tile, split, m_block, p.y);
+  epilogue<BT>(p, tmem_base, smem, n_tile, split, m_block * BT, p.M, p.y);
 
   tcgen05_fence_before_sync();
   __syncthreads();

@@ -1,0 +1,307 @@
+// Mixture of experts with sigmoid scores: routing, the sort of the tokens by expert, and the experts' grouped products (tcgen05:
+// gemm_grouped_kernel in gemm_bf16.cu; CUDA cores here).
+//
+//   route_kernel   a warp per token: scores from the router's fp32 partial sums, the `top` best, a place behind the tokens that
+//                  already chose the same expert; the CTA that finishes last turns the counts into offsets and the tile list
+//   gather_kernel  x_sorted[offset[expert] + rank] = x[token]
+//   simt_kernel    64 x 64 outputs per CTA in true fp32
+#include "common.cuh"
+
+namespace b200 {
+namespace moe {
+
+constexpr int kWarps = 8;
+constexpr int kMaxExperts = 1024;
+
+// Shared memory: [kWarps][experts] scores; the last CTA reuses none of it.
+__global__ void __launch_bounds__(kWarps * 32)
+route_kernel(b200_moe_args a) {
+  extern __shared__ float score_s[];
+  __shared__ int is_last;
+  __shared__ int warp_rows[kWarps], warp_tiles[kWarps];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, E = a.experts;
+  const int t = blockIdx.x * kWarps + warp;
+  if (t < a.num_tokens) {
+    float* score = score_s + warp * E;
+    const int64_t stride = static_cast<int64_t>(a.num_tokens) * a.router_ld;
+    const float* z = a.router + static_cast<int64_t>(t) * a.router_ld;
+    for (int e = lane; e < E + (a.shared_gate != nullptr ? 1 : 0); e += 32) {
+      float x = 0.f;
+      for (int s = 0; s < a.router_splits; ++s) x += z[s * stride + e];
+      x = 1.f / (1.f + expf(-x));
+      if (e < E)
+        score[e] = x;
+      else
+        a.shared_gate[t] = x;
+    }
+    __syncwarp();
+    for (int k = 0; k < a.top; ++k) {
+      float best = -1.f;  // (scores are positive; a chosen one is marked -2)
+      int at = E;
+      for (int e = lane; e < E; e += 32)
+        if (score[e] > best) {
+          best = score[e];
+          at = e;
+        }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float b = __shfl_xor_sync(0xffffffffu, best, o);
+        const int i = __shfl_xor_sync(0xffffffffu, at, o);
+        if (b > best || (b == best && i < at)) {
+          best = b;
+          at = i;
+        }
+      }
+      if (at >= E) at = k;  // no number left (NaN scores): any expert, its output is NaN too
+      if (lane == 0) {
+        const int rank = atomicAdd(&a.counts[at], 1);
+        const int64_t pair = static_cast<int64_t>(t) * a.top + k;
+        reinterpret_cast<int2*>(a.pairs)[pair] = make_int2(at, rank);
+        a.pair_weight[pair] = score[at];
+        score[at] = -2.f;
+      }
+      __syncwarp();
+    }
+  }
+  __syncthreads();
+  if (threadIdx.x == 0) {
+    __threadfence();  // this CTA's counts are visible before its ticket
+    is_last = atomicAdd(&a.counts[E], 1) == static_cast<int>(gridDim.x) - 1;
+  }
+  __syncthreads();
+  if (!is_last) return;
+  __threadfence();
+  // offsets and tiles: every thread takes a run of experts; sums over lanes, then over warps
+  const int per = (E + kWarps * 32 - 1) / (kWarps * 32), e0 = threadIdx.x * per;
+  int rows = 0, tiles = 0;
+  for (int e = e0; e < min(e0 + per, E); ++e) {
+    const int c = __ldcg(&a.counts[e]);
+    rows += c;
+    tiles += (c + a.tile_tokens - 1) / a.tile_tokens;
+  }
+  int rows_incl = rows, tiles_incl = tiles;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const int r = __shfl_up_sync(0xffffffffu, rows_incl, o), i = __shfl_up_sync(0xffffffffu, tiles_incl, o);
+    if (lane >= o) {
+      rows_incl += r;
+      tiles_incl += i;
+    }
+  }
+  if (lane == 31) {
+    warp_rows[warp] = rows_incl;
+    warp_tiles[warp] = tiles_incl;
+  }
+  __syncthreads();
+  int row_at = rows_incl - rows, tile_at = tiles_incl - tiles;
+  for (int w = 0; w < warp; ++w) {
+    row_at += warp_rows[w];
+    tile_at += warp_tiles[w];
+  }
+  for (int e = e0; e < min(e0 + per, E); ++e) {
+    const int c = __ldcg(&a.counts[e]);
+    a.offsets[e] = row_at;
+    for (int r = 0; r < c; r += a.tile_tokens, ++tile_at)
+      if (tile_at < a.max_tiles) reinterpret_cast<int4*>(a.tiles)[tile_at] = make_int4(e, row_at + r, min(a.tile_tokens, c - r), 0);
+    row_at += c;
+    a.counts[e] = 0;
+  }
+  if (threadIdx.x == kWarps * 32 - 1) {
+    a.offsets[E] = row_at;
+    *a.num_tiles = min(tile_at, a.max_tiles);
+    a.counts[E] = 0;
+  }
+}
+
+// One warp per (token, choice) pair.
+template <typename V>
+__global__ void __launch_bounds__(256)
+gather_kernel(b200_moe_args a, int vectors) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int lane = threadIdx.x & 31;
+  const int64_t pairs = static_cast<int64_t>(a.num_tokens) * a.top;
+  const int64_t pair = static_cast<int64_t>(blockIdx.x) * 8 + (threadIdx.x >> 5);
+  if (pair >= pairs) return;
+  const int2 p = reinterpret_cast<const int2*>(a.pairs)[pair];
+  if (static_cast<unsigned>(p.x) >= static_cast<unsigned>(a.experts)) return;
+  const int64_t at = static_cast<int64_t>(a.offsets[p.x]) + p.y;
+  if (at < 0 || at >= pairs) return;
+  const V* src = static_cast<const V*>(a.x) + pair / a.top * vectors;
+  V* dst = static_cast<V*>(a.x_sorted) + at * vectors;
+  if (lane == 0) a.row_scale[at] = a.pair_weight[pair];
+  int i = lane;
+  for (; i + 96 < vectors; i += 128) {  // four loads in flight
+    const V v0 = src[i], v1 = src[i + 32], v2 = src[i + 64], v3 = src[i + 96];
+    dst[i] = v0;
+    dst[i + 32] = v1;
+    dst[i + 64] = v2;
+    dst[i + 96] = v3;
+  }
+  for (; i < vectors; i += 32) dst[i] = src[i];
+}
+
+// CUDA-core grouped product.  GATED: 64 features of an up product (gate and up rows of one 128-row block), else 64 features of a down product.
+// blockIdx.y < shared_blocks: the shared expert's token blocks, then the tile list.
+template <typename T, bool GATED>
+__global__ void __launch_bounds__(256)
+simt_kernel(b200_moe_args a, int shared_blocks) {
+  constexpr int kK = 16, kTile = 64;
+  __shared__ float xs[kK][kTile + 4], ws[GATED ? 2 : 1][kK][kTile + 4];
+  pdl_launch_dependents();
+  pdl_wait();
+  const bool shared = static_cast<int>(blockIdx.y) < shared_blocks;
+  const int ff = shared ? a.shared_ff : a.ff, K = GATED ? a.width : ff, N = GATED ? ff : a.width;
+  const int n0 = blockIdx.x * kTile;
+  if (n0 >= N) return;
+  int m0 = blockIdx.y * kTile, rows = min(kTile, a.num_tokens - m0), expert = 0;
+  if (!shared) {
+    const int tile = blockIdx.y - shared_blocks;
+    if (tile >= *a.num_tiles) return;
+    const int4 e = reinterpret_cast<const int4*>(a.tiles)[tile];
+    if (static_cast<unsigned>(e.x) >= static_cast<unsigned>(a.experts) || e.y < 0 || e.z > kTile ||
+        e.y + e.z > static_cast<int64_t>(a.num_tokens) * a.top)
+      return;
+    expert = e.x;
+    m0 = e.y;
+    rows = e.z;
+  }
+  const T* x = static_cast<const T*>(GATED ? (shared ? a.x : a.x_sorted) : (shared ? a.shared_inter : a.inter));
+  const T* w = static_cast<const T*>(GATED ? (shared ? a.shared_up : a.up) : (shared ? a.shared_down : a.down)) +
+               static_cast<int64_t>(expert) * (GATED ? 2 * ff : a.width) * K + (GATED ? static_cast<int64_t>(blockIdx.x) * 128 * K : static_cast<int64_t>(n0) * K);
+  T* y = static_cast<T*>(GATED ? (shared ? a.shared_inter : a.inter) : (shared ? a.shared_y : a.y));
+  const int tid = threadIdx.x, tr = (tid >> 4) * 4, tc = (tid & 15) * 4;
+  float acc[4][4] = {}, up[4][4] = {};
+  for (int k0 = 0; k0 < K; k0 += kK) {
+    for (int i = tid; i < kTile * kK; i += 256) {
+      const int r = i / kK, k = i - r * kK;
+      const bool kin = k0 + k < K;
+      xs[k][r] = kin && r < rows ? simt::to_f32(x[static_cast<int64_t>(m0 + r) * K + k0 + k]) : 0.f;
+      ws[0][k][r] = kin && n0 + r < N ? simt::to_f32(w[static_cast<int64_t>(r) * K + k0 + k]) : 0.f;
+      if (GATED) ws[GATED ? 1 : 0][k][r] = kin ? simt::to_f32(w[static_cast<int64_t>(64 + r) * K + k0 + k]) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < kK; ++k)
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          acc[i][j] = fmaf(xs[k][tr + i], ws[0][k][tc + j], acc[i][j]);
+          if (GATED) up[i][j] = fmaf(xs[k][tr + i], ws[GATED ? 1 : 0][k][tc + j], up[i][j]);
+        }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    if (tr + i >= rows) continue;
+    const int m = m0 + tr + i;
+    const float scale = GATED && !shared ? a.row_scale[m] : 1.f;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      if (n0 + tc + j >= N) continue;
+      float v = acc[i][j];
+      if (GATED) v = gemm::clamped_glu(v * scale, up[i][j] * scale, shared ? a.shared_limit : a.limit, a.alpha);
+      simt::store_as(y + static_cast<int64_t>(m) * N + n0 + tc + j, v);
+    }
+  }
+}
+
+static bool valid(const b200_moe_args* a) {
+  return a && a->num_tokens > 0 && a->width > 0 && a->experts > 0 && a->experts <= kMaxExperts && a->top > 0 && a->top <= a->experts &&
+         a->top <= 64 && a->ff > 0 && a->ff % 64 == 0 && a->tile_tokens > 0 && a->max_tiles > 0 && a->pairs && a->offsets && a->tiles && a->num_tiles &&
+         static_cast<int64_t>(a->num_tokens) * a->top < (1 << 30) && (!a->shared_up || (a->shared_ff > 0 && a->shared_ff % 64 == 0)) &&
+         (a->dtype == B200_DTYPE_BF16 || a->dtype == B200_DTYPE_F32);
+}
+
+static int grouped(const b200_moe_args& a, bool up, cudaStream_t s) {
+  const bool with_shared = a.shared_up != nullptr;
+  if (a.simt || a.dtype == B200_DTYPE_F32) {
+    if (a.tile_tokens != 64) return B200_ERR_INVALID_ARGUMENT;
+    const int shared_blocks = with_shared ? (a.num_tokens + 63) / 64 : 0;
+    const int widest = up ? (with_shared && a.shared_ff > a.ff ? a.shared_ff : a.ff) : a.width;
+    if (shared_blocks + a.max_tiles > 65535) return B200_ERR_INVALID_ARGUMENT;
+    const dim3 grid((widest + 63) / 64, shared_blocks + a.max_tiles);
+    if (a.dtype == B200_DTYPE_F32)
+      return up ? launch_pdl(simt_kernel<float, true>, grid, dim3(256), 0, s, a, shared_blocks)
+                : launch_pdl(simt_kernel<float, false>, grid, dim3(256), 0, s, a, shared_blocks);
+    return up ? launch_pdl(simt_kernel<__nv_bfloat16, true>, grid, dim3(256), 0, s, a, shared_blocks)
+              : launch_pdl(simt_kernel<__nv_bfloat16, false>, grid, dim3(256), 0, s, a, shared_blocks);
+  }
+  const int64_t pairs = static_cast<int64_t>(a.num_tokens) * a.top;
+  gemm::GroupedProblem routed{up ? a.x_sorted : a.inter, up ? a.up : a.down, up ? a.width : a.ff, a.experts}, shared{};
+  gemm::GroupedParams gp{};
+  auto fill = [&](gemm::Params& p, int64_t M, int ff, void* y, float limit, const float* scale) {
+    p.M = static_cast<int>(M);
+    p.N = up ? 2 * ff : a.width;
+    p.K = up ? a.width : ff;
+    p.y = static_cast<__nv_bfloat16*>(y);
+    p.ldy = up ? ff : a.width;
+    p.gated = up ? gemm::kGatedClamped : 0;
+    p.glu_limit = limit;
+    p.glu_alpha = a.alpha;
+    p.row_scale = up ? scale : nullptr;
+  };
+  fill(gp.routed, pairs, a.ff, up ? a.inter : a.y, a.limit, a.row_scale);
+  if (with_shared) {
+    shared = gemm::GroupedProblem{up ? a.x : a.shared_inter, up ? a.shared_up : a.shared_down, up ? a.width : a.shared_ff, 1};
+    fill(gp.shared, a.num_tokens, a.shared_ff, up ? a.shared_inter : a.shared_y, a.shared_limit, nullptr);
+  }
+  for (const void* p : {routed.x, routed.w, shared.x, shared.w})
+    if (!aligned16(p)) return B200_ERR_ALIGNMENT;
+  if (a.width % 8 != 0) return B200_ERR_ALIGNMENT;
+  gp.tiles = reinterpret_cast<const int4*>(a.tiles);
+  gp.num_tiles = a.num_tiles;
+  gp.max_tiles = a.max_tiles;
+  gp.experts = a.experts;
+  switch (a.tile_tokens) {
+    case 32: return gemm::launch_grouped<32>(routed, shared, gp, s);
+    case 64: return gemm::launch_grouped<64>(routed, shared, gp, s);
+    case 128: return gemm::launch_grouped<128>(routed, shared, gp, s);
+    case 256: return gemm::launch_grouped<256>(routed, shared, gp, s);
+    default: return B200_ERR_INVALID_ARGUMENT;
+  }
+}
+
+}  // namespace moe
+}  // namespace b200
+
+extern "C" {
+
+int b200_moe_route(const b200_moe_args* a, b200_stream_t stream) {
+  using namespace b200;
+  if (!moe::valid(a) || !a->router || a->router_splits < 1 || a->router_ld < a->experts + (a->shared_gate ? 1 : 0) || !a->counts || !a->pair_weight)
+    return B200_ERR_INVALID_ARGUMENT;
+  const unsigned blocks = static_cast<unsigned>((a->num_tokens + moe::kWarps - 1) / moe::kWarps);
+  return launch_pdl(moe::route_kernel, dim3(blocks), dim3(moe::kWarps * 32), static_cast<size_t>(moe::kWarps) * a->experts * 4,
+                    reinterpret_cast<cudaStream_t>(stream), *a);
+}
+
+int b200_moe_gather(const b200_moe_args* a, b200_stream_t stream) {
+  using namespace b200;
+  if (!moe::valid(a) || !a->x || !a->x_sorted || !a->row_scale || !a->pair_weight) return B200_ERR_INVALID_ARGUMENT;
+  const int64_t pairs = static_cast<int64_t>(a->num_tokens) * a->top, bytes = static_cast<int64_t>(a->width) * (a->dtype == B200_DTYPE_F32 ? 4 : 2);
+  const dim3 grid(static_cast<unsigned>((pairs + 7) / 8));
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (bytes % 16 == 0 && aligned16(a->x) && aligned16(a->x_sorted))
+    return launch_pdl(moe::gather_kernel<uint4>, grid, dim3(256), 0, s, *a, static_cast<int>(bytes / 16));
+  return launch_pdl(moe::gather_kernel<uint16_t>, grid, dim3(256), 0, s, *a, static_cast<int>(bytes / 2));
+}
+
+int b200_moe_up(const b200_moe_args* a, b200_stream_t stream) {
+  using namespace b200;
+  if (!moe::valid(a) || !a->x || !a->x_sorted || !a->row_scale || !a->up || !a->inter || (a->shared_up && !a->shared_inter))
+    return B200_ERR_INVALID_ARGUMENT;
+  return moe::grouped(*a, true, reinterpret_cast<cudaStream_t>(stream));
+}
+
+int b200_moe_down(const b200_moe_args* a, b200_stream_t stream) {
+  using namespace b200;
+  if (!moe::valid(a) || !a->down || !a->inter || !a->y || (a->shared_up && (!a->shared_down || !a->shared_inter || !a->shared_y)))
+    return B200_ERR_INVALID_ARGUMENT;
+  return moe::grouped(*a, false, reinterpret_cast<cudaStream_t>(stream));
+}
+
+}  // extern "C"

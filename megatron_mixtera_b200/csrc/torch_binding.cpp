@@ -278,6 +278,8 @@ void attention(const Tensor& args, const Tensor& anchor, int64_t which, const Op
     ok(b200_rope_append(a, s), "b200_rope_append");
   } else if (which == 1) {
     ok(b200_paged_attention(a, s), "b200_paged_attention");
+  } else if (which == 3) {  // num_units: B200_DTYPE_*
+    ok(b200_attention_simt(a, static_cast<int>(num_units), s), "b200_attention_simt");
   } else {
     TORCH_CHECK(units.has_value(), "b200_decode.attention: the prefill kernel needs `units`");
     need(*units, I32, "units");
@@ -344,6 +346,18 @@ void hybrid(const Tensor& args, const Tensor& anchor, int64_t which) {
     case 8:
       ok(b200_latent_prompt_attention(struct_of<b200_latent_args>(args, "b200_latent_args"), s), "b200_latent_prompt_attention");
       break;
+    case 9: ok(b200_residual_norm(struct_of<b200_residual_norm_args>(args, "b200_residual_norm_args"), s), "b200_residual_norm"); break;
+    case 10: ok(b200_conv_silu(struct_of<b200_conv_args>(args, "b200_conv_args"), s), "b200_conv_silu"); break;
+    case 11: ok(b200_conv_qkv(struct_of<b200_conv_args>(args, "b200_conv_args"), s), "b200_conv_qkv"); break;
+    case 12: ok(b200_token_shift(struct_of<b200_shift_args>(args, "b200_shift_args"), s), "b200_token_shift"); break;
+    case 13: ok(b200_recurrence_decode(struct_of<b200_recurrence_args>(args, "b200_recurrence_args"), s), "b200_recurrence_decode"); break;
+    case 14: ok(b200_recurrence_scan(struct_of<b200_recurrence_args>(args, "b200_recurrence_args"), s), "b200_recurrence_scan"); break;
+    case 15: ok(b200_recurrence_finish(struct_of<b200_recurrence_args>(args, "b200_recurrence_args"), s), "b200_recurrence_finish"); break;
+    case 16: ok(b200_recurrence_lora(struct_of<b200_recurrence_args>(args, "b200_recurrence_args"), s), "b200_recurrence_lora"); break;
+    case 17: ok(b200_moe_route(struct_of<b200_moe_args>(args, "b200_moe_args"), s), "b200_moe_route"); break;
+    case 18: ok(b200_moe_gather(struct_of<b200_moe_args>(args, "b200_moe_args"), s), "b200_moe_gather"); break;
+    case 19: ok(b200_moe_up(struct_of<b200_moe_args>(args, "b200_moe_args"), s), "b200_moe_up"); break;
+    case 20: ok(b200_moe_down(struct_of<b200_moe_args>(args, "b200_moe_args"), s), "b200_moe_down"); break;
     default: TORCH_CHECK(false, "b200_decode.hybrid: unknown kernel ", which);
   }
 }

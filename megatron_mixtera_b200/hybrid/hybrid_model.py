@@ -1,5 +1,8 @@
-"""Hybrid decoder for the dynamic inference path: layers of latent attention or the generalized delta rule with norms on the
-sublayers' outputs, a 32-bit residual stream and tied embeddings.  Same calls as `GPTModel` (`forward`, `forward_rows`)."""
+"""Hybrid decoders for the dynamic inference path, with the same calls as `GPTModel` (`forward`, `forward_rows`).
+
+`HybridDecoder`: what they share - the context made for their layers, strict checkpoint loading, synthetic weights.
+`HybridModel`: layers of latent attention or the generalized delta rule with norms on the sublayers' outputs, a 32-bit residual
+stream and tied embeddings.  (`ParallelHybridModel` is in parallel_model.py.)"""
 from __future__ import annotations
 
 from typing import Dict, Optional
@@ -42,10 +45,66 @@ class HybridLayer(torch.nn.Module):
         return x
 
 
-class HybridModel(DynamicForward, torch.nn.Module):
+class HybridDecoder(DynamicForward, torch.nn.Module):
     def __init__(self, config: HybridConfig, max_sequence_length: int):
         super().__init__()
         self.config, self.vocab_size, self.max_sequence_length = config, config.vocab_size, max_sequence_length
+
+    def make_context(self, *, buffer_size_gb: Optional[float] = None, max_cached_tokens: Optional[int] = None,
+                     chunk_size_tokens: int = 64, **kwargs) -> DynamicInferenceContext:
+        """A context with the token rows and the state this model's layers keep.  The pool is given in GB, or as the number of
+        tokens it must hold (in whole chunks; one more chunk takes the padding tokens' writes)."""
+        c = self.config
+        widths = [layer.mixer.cached_row_width() for layer in c.layers]
+        states = [layer.mixer.request_state(c.hidden_size, c.params_dtype) for layer in c.layers]
+        if max_cached_tokens is not None:
+            chunks = -(-max_cached_tokens // chunk_size_tokens) + 1
+            nbytes = DynamicInferenceContext.latent_chunk_bytes(widths, chunk_size_tokens, c.params_dtype)
+            buffer_size_gb = (chunks + 0.5) * nbytes / 1024**3
+        return DynamicInferenceContext(
+            params_dtype=c.params_dtype, num_layers=c.num_layers, kv_channels=0, num_attention_heads=0,
+            max_sequence_length=self.max_sequence_length, buffer_size_gb=buffer_size_gb, cache_mla_latent=True,
+            latent_row_widths=widths, state_shapes=states, chunk_size_tokens=chunk_size_tokens,
+            tensor_model_parallel_size=1, **{"buffer_guaranteed_fraction": 0.0, **kwargs})
+
+    # ------------------------------------------------------------------------------------------
+    def checkpoint_tensors(self) -> Dict[str, tuple]:
+        """Checkpoint tensor name -> shape of everything this model loads."""
+        raise NotImplementedError
+
+    def ignored_tensors(self) -> set:
+        """Names that a checkpoint may hold although nothing reads them."""
+        return set()
+
+    def _load(self, tensors: Dict[str, torch.Tensor]) -> None:
+        raise NotImplementedError
+
+    def load_checkpoint(self, tensors: Dict[str, torch.Tensor]) -> None:
+        """Load checkpoint tensors (any float type; converted to the model's)."""
+        want = self.checkpoint_tensors()
+        for name, shape in want.items():
+            if name not in tensors:
+                raise KeyError(f"checkpoint tensor {name!r} is missing")
+            if tuple(tensors[name].shape) != tuple(shape):
+                raise ValueError(f"checkpoint tensor {name!r} has shape {tuple(tensors[name].shape)}, expected {tuple(shape)}")
+        unknown = sorted(set(tensors) - set(want) - self.ignored_tensors())
+        if unknown:
+            raise KeyError(f"checkpoint tensors this model does not use: {unknown[:4]}")
+        self._load(tensors)
+
+    def synthetic_tensor(self, name: str, shape: tuple, seed: int, std: float, device) -> torch.Tensor:
+        """Seeded N(0, std) values (norm scales 1 + N(0, std))."""
+        t = canonical_tensor(name, shape, seed=seed, std=std, dtype=torch.float32, device=device)
+        return t + 1.0 if name.rsplit(".", 1)[-1] in ("norm", "norm1", "norm2") else t
+
+    def init_synthetic_weights(self, seed: int = 0, std: float = 0.02, device=None) -> None:
+        dev = self.word_embeddings.weight.device if device is None else device
+        self.load_checkpoint({n: self.synthetic_tensor(n, s, seed, std, dev) for n, s in self.checkpoint_tensors().items()})
+
+
+class HybridModel(HybridDecoder):
+    def __init__(self, config: HybridConfig, max_sequence_length: int):
+        super().__init__(config, max_sequence_length)
         kw = dict(config=config, hidden_size=config.hidden_size, eps=config.layernorm_epsilon)
         self.word_embeddings = VocabParallelEmbedding(config.vocab_size, config.hidden_size, config=config)
         self.embedding_norm = OutputNorm(**kw)
@@ -66,25 +125,6 @@ class HybridModel(DynamicForward, torch.nn.Module):
         """Tokens per work unit of the prompt attention kernel (it cuts a unit into blocks of query rows itself)."""
         return 16
 
-    def make_context(self, *, buffer_size_gb: Optional[float] = None, max_cached_tokens: Optional[int] = None,
-                     chunk_size_tokens: int = 64, **kwargs) -> DynamicInferenceContext:
-        """A context with the latent rows and recurrent state this model needs.  The pool is given in GB, or as the number of
-        tokens it must hold (in whole chunks; one more chunk takes the padding tokens' writes)."""
-        c = self.config
-        widths = [layer.mixer.row_width if isinstance(layer.mixer, LatentAttentionConfig) and layer.mixer.kv_from is None else 0
-                  for layer in c.layers]
-        states = [(layer.mixer.heads, layer.mixer.dim, layer.mixer.dim) if isinstance(layer.mixer, DeltaRuleConfig) else None
-                  for layer in c.layers]
-        if max_cached_tokens is not None:
-            chunks = -(-max_cached_tokens // chunk_size_tokens) + 1
-            nbytes = DynamicInferenceContext.latent_chunk_bytes(widths, chunk_size_tokens, c.params_dtype)
-            buffer_size_gb = (chunks + 0.5) * nbytes / 1024**3
-        return DynamicInferenceContext(
-            params_dtype=c.params_dtype, num_layers=c.num_layers, kv_channels=0, num_attention_heads=0,
-            max_sequence_length=self.max_sequence_length, buffer_size_gb=buffer_size_gb, cache_mla_latent=True,
-            latent_row_widths=widths, state_shapes=states, chunk_size_tokens=chunk_size_tokens,
-            tensor_model_parallel_size=1, **{"buffer_guaranteed_fraction": 0.0, **kwargs})
-
     # ------------------------------------------------------------------------------------------
     def forward_rows(self, input_ids, position_ids, inference_context, row_indices=None,
                      runtime_gather_output: Optional[bool] = None, streams: Optional[list] = None):
@@ -100,7 +140,6 @@ class HybridModel(DynamicForward, torch.nn.Module):
 
     # ------------------------------------------------------------------------------------------
     def checkpoint_tensors(self) -> Dict[str, tuple]:
-        """Checkpoint tensor name -> shape of everything this model loads."""
         c = self.config
         out = {"embed": (c.vocab_size, c.hidden_size), "embed.norm": (c.hidden_size,), "final.norm": (c.hidden_size,)}
         for i, layer in enumerate(self.layers):
@@ -111,18 +150,7 @@ class HybridModel(DynamicForward, torch.nn.Module):
                 out.update({f"l{i}.norm2": (c.hidden_size,), f"l{i}.mlp.up": (ffn, c.hidden_size), f"l{i}.mlp.down": (c.hidden_size, ffn)})
         return out
 
-    def load_checkpoint(self, tensors: Dict[str, torch.Tensor]) -> None:
-        """Load checkpoint tensors (any float type; converted to the model's)."""
-        want = self.checkpoint_tensors()
-        for name, shape in want.items():
-            if name not in tensors:
-                raise KeyError(f"checkpoint tensor {name!r} is missing")
-            if tuple(tensors[name].shape) != tuple(shape):
-                raise ValueError(f"checkpoint tensor {name!r} has shape {tuple(tensors[name].shape)}, expected {tuple(shape)}")
-        unknown = sorted(set(tensors) - set(want))
-        if unknown:
-            raise KeyError(f"checkpoint tensors this model does not use: {unknown[:4]}")
-
+    def _load(self, tensors: Dict[str, torch.Tensor]) -> None:
         def put(param, name):
             param.data.copy_(tensors[name])
 
@@ -136,12 +164,3 @@ class HybridModel(DynamicForward, torch.nn.Module):
                 put(layer.mlp_norm.weight, f"l{i}.norm2")
                 put(layer.mlp.linear_fc1.weight, f"l{i}.mlp.up")
                 put(layer.mlp.linear_fc2.weight, f"l{i}.mlp.down")
-
-    def init_synthetic_weights(self, seed: int = 0, std: float = 0.02, device=None) -> None:
-        """Seeded N(0, std) weights (norm scales 1 + N(0, std))."""
-        dev = self.word_embeddings.weight.device if device is None else device
-        out = {}
-        for name, shape in self.checkpoint_tensors().items():
-            t = canonical_tensor(name, shape, seed=seed, std=std, dtype=torch.float32, device=dev)
-            out[name] = t + 1.0 if name.rsplit(".", 1)[-1] in ("norm", "norm1", "norm2") else t
-        self.load_checkpoint(out)

@@ -15,9 +15,10 @@ one device->host read (the sampled tokens) and a handful of host->device copies.
 
 Two kinds of per-request memory exist besides the key / value pool, for decoders whose layers are not plain attention:
 
-* latent rows (``cache_mla_latent``): one row per token and caching layer, of a width that may differ between layers, in the
-  same chunks and block tables as keys and values would be;
-* recurrent state (``state_shapes``): a fixed-size fp32 block per request and recurrent layer in a slot of its own.  Every slot
+* token rows (``cache_mla_latent``): one row per token and caching layer, of a width that may differ between layers - a latent
+  row, or the keys of a layer's heads followed by their values - in the same chunks and block tables as keys and values of one
+  shape would be;
+* recurrent state (``state_shapes``): fixed-size blocks per request and layer in a slot of their own.  Every slot
   is a pair of buffers: a step reads one and writes the other, and completing the step swaps them.  A forward that is run
   again - under CUDA-graph capture, or because the one enqueued early was not used - therefore gives the same result.
 
@@ -146,7 +147,7 @@ class DynamicInferenceContext(BaseInferenceContext):
         kv_fp8_single_term: bool = False,
         debug_validate: bool = False,
         latent_row_widths: Optional[Sequence[int]] = None,
-        state_shapes: Optional[Sequence[Optional[Tuple[int, ...]]]] = None,
+        state_shapes: Optional[Sequence] = None,
     ):
         """``num_attention_heads`` is the number of KV heads (query groups), as in the reference.
 
@@ -159,7 +160,8 @@ class DynamicInferenceContext(BaseInferenceContext):
 
         ``cache_mla_latent``: the pool holds one latent row per token instead of keys and values; ``latent_row_widths`` gives
         the row width of every layer (0: the layer caches nothing), or ``kv_lora_rank + qk_pos_emb_head_dim`` that of all.
-        ``state_shapes``: per layer the shape of its fp32 recurrent state per request, None for layers without one.
+        ``state_shapes``: per layer the shape of its fp32 recurrent state per request, or a dict name -> (shape, dtype) where it
+        keeps several parts; None for layers without any.
         """
         super().__init__(materialize_only_last_token_logits=materialize_only_last_token_logits)
         # Debug mode: every `initialize_attention_state` checks on the host what the kernels are about to index with
@@ -298,9 +300,12 @@ class DynamicInferenceContext(BaseInferenceContext):
             self._d_slots = torch.full((2, R + 1), -1, dtype=torch.int32, device=self.device)
             self.state_read_slots, self.state_write_slots = self._d_slots[0], self._d_slots[1]
             if allocate_memory_buffer:
-                self.state_buffers = [
-                    torch.zeros((2 * R, *sh), dtype=torch.float32, device=self.device) if sh is not None else None
-                    for sh in self.state_shapes]
+                def buffers(sh):
+                    if isinstance(sh, dict):
+                        return {k: torch.zeros((2 * R, *s), dtype=dt, device=self.device) for k, (s, dt) in sh.items()}
+                    return torch.zeros((2 * R, *sh), dtype=torch.float32, device=self.device) if sh is not None else None
+
+                self.state_buffers = [buffers(sh) for sh in self.state_shapes]
 
         # ---- CUDA-graph token counts (reference :319-356) ----
         self.cuda_graph_token_counts = None
@@ -347,6 +352,7 @@ class DynamicInferenceContext(BaseInferenceContext):
         self.prefill_q_block = 0
         self.prefill_units = None
         self.prefill_unit_count = 0
+        self._more_units = {}  # further block sizes (head groupings that differ between layers) -> [host, numpy, device, count]
         self._copy_event = torch.cuda.Event() if pin else None
         self._copies_pending = False
         self.h2d_bytes = 0  # bytes mirrored host -> device so far (benchmark accounting)
@@ -363,24 +369,37 @@ class DynamicInferenceContext(BaseInferenceContext):
 
         self.reset_attention_state()
 
-    def set_prefill_q_block(self, q_block: int) -> None:
-        """Tokens per prefill work unit (64 / query heads per KV head); 0 disables the work list."""
+    def _unit_buffers(self, q_block: int) -> list:
+        n = -(-self.max_tokens // q_block) + self.max_requests + 1
+        host = torch.zeros((n, 4), dtype=torch.int32, pin_memory=self.device.type == "cuda")
+        return [host, host.numpy(), torch.zeros((n, 4), dtype=torch.int32, device=self.device), 0]
+
+    def set_prefill_q_block(self, q_block: int, *more: int) -> None:
+        """Tokens per prefill work unit (64 / query heads per KV head); 0 disables the work list.  ``more``: further sizes, for
+        models whose layers group their heads differently (`prefill_units_of`)."""
         self.prefill_q_block = int(q_block)
         if self.prefill_q_block > 0:
-            n = -(-self.max_tokens // self.prefill_q_block) + self.max_requests + 1
-            pin = self.device.type == "cuda"
-            self._h_units = torch.zeros((n, 4), dtype=torch.int32, pin_memory=pin)
-            self._h_units_np = self._h_units.numpy()
-            self.prefill_units = torch.zeros((n, 4), dtype=torch.int32, device=self.device)
-            self.prefill_unit_count = 0
+            self._h_units, self._h_units_np, self.prefill_units, self.prefill_unit_count = self._unit_buffers(self.prefill_q_block)
+        self._more_units = {int(q): self._unit_buffers(int(q)) for q in more if int(q) != self.prefill_q_block}
+
+    def prefill_units_of(self, q_block: int) -> Tuple[Tensor, int]:
+        """(work list, number of units) of this step for blocks of ``q_block`` tokens."""
+        if q_block == self.prefill_q_block:
+            return self.prefill_units, self.prefill_unit_count
+        _, _, device, count = self._more_units[q_block]
+        return device, count
 
     def _build_prefill_units(self, ql: np.ndarray, n_rows: int, padded: int, graphs: bool) -> None:
-        """Split every request's query tokens into blocks of `prefill_q_block` (host side, vectorised)."""
-        qb = self.prefill_q_block
+        self.prefill_unit_count = self._fill_units(self.prefill_q_block, self._h_units, self._h_units_np, self.prefill_units, ql, n_rows,
+                                                   padded, graphs)
+        for qb, entry in self._more_units.items():
+            entry[3] = self._fill_units(qb, *entry[:3], ql, n_rows, padded, graphs)
+
+    def _fill_units(self, qb: int, host: Tensor, u: np.ndarray, device: Tensor, ql: np.ndarray, n_rows: int, padded: int, graphs: bool) -> int:
+        """Split every request's query tokens into blocks of ``qb`` (host side, vectorised); returns how many."""
         ql = ql.astype(np.int64)
         nb = -(-ql // qb)
         total = int(nb.sum())
-        u = self._h_units_np
         # under a CUDA graph the launch size is fixed by the padded sizes; unused entries have 0 tokens
         bound = (-(-padded // qb) + n_rows) if graphs else max(total, 1)
         bound = min(max(bound, total), u.shape[0])
@@ -393,9 +412,9 @@ class DynamicInferenceContext(BaseInferenceContext):
             u[:total, 2] = np.minimum(qb, np.repeat(ql, nb) - within * qb)
             u[:total, 3] = 0
         u[total:bound] = 0
-        self.prefill_units[:bound].copy_(self._h_units[:bound], non_blocking=True)
-        self.prefill_unit_count = bound
+        device[:bound].copy_(host[:bound], non_blocking=True)
         self.h2d_bytes += 16 * bound
+        return bound
 
     # ------------------------------------------------------------------ rounding helpers
     @classmethod
@@ -483,14 +502,18 @@ class DynamicInferenceContext(BaseInferenceContext):
         h[1, :n] = np.where(ok, (1 - side) * self.num_state_slots + slot, -1)
         self._push_rows(self._d_slots, self._h_slots, 2, 0, max(n_rows, 1))
 
-    def recurrent_state(self, layer_number: int) -> Tensor:
-        """fp32 state buffers ``[2 * slots, ...]`` of 1-based ``layer_number``."""
-        return self.state_buffers[layer_number - 1]
+    def recurrent_state(self, layer_number: int, part: Optional[str] = None) -> Optional[Tensor]:
+        """State buffers ``[2 * slots, ...]`` of 1-based ``layer_number``; ``part``: of a layer that keeps several (None where it
+        does not keep this one)."""
+        buffers = self.state_buffers[layer_number - 1]
+        return buffers.get(part) if part is not None else buffers
 
     # ------------------------------------------------------------------ KV pool access
     def latent_cache(self, layer_number: int) -> Tensor:
-        """Latent rows ``[chunks, chunk, width]`` of 1-based ``layer_number``."""
+        """Token rows ``[chunks, chunk, width]`` of 1-based ``layer_number``."""
         return self.latent_buffers[layer_number - 1]
+
+    token_rows = latent_cache
 
     def expanded_keys(self, window: Optional[int]):
         """For attention that spells out the keys of a prompt step: which keys the step's queries see under ``window``.

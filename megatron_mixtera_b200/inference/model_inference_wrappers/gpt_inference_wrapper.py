@@ -52,7 +52,8 @@ class GPTInferenceWrapper:
             from ... import ops
 
             if hasattr(model, "prefill_unit_tokens"):  # the model's kernels cut work units of their own
-                inference_context.set_prefill_q_block(model.prefill_unit_tokens())
+                sizes = model.prefill_unit_tokens()  # one size, or one per head grouping
+                inference_context.set_prefill_q_block(*(sizes if isinstance(sizes, (list, tuple)) else (sizes,)))
                 return
             groups = cfg.num_query_groups or cfg.num_attention_heads
             fp8_pool = getattr(inference_context, "kv_cache_fp8", False)  # the prefill kernel reads a bf16 pool

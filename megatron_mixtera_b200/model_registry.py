@@ -9,7 +9,8 @@ from typing import Callable, Dict, Tuple
 import torch
 
 from . import checkpoint
-from .transformer.hybrid_config import (DeltaRuleConfig, HybridConfig, HybridLayerConfig, LatentAttentionConfig, RotaryConfig,
+from .transformer.hybrid_config import (DeltaRuleConfig, ExpertConfig, GatedDeltaConfig, HybridConfig, HybridLayerConfig,
+                                        LatentAttentionConfig, MoeConfig, RotaryConfig, ShortConvAttentionConfig, WkvConfig,
                                         YarnScaling)
 from .transformer.transformer_config import TransformerConfig
 
@@ -51,6 +52,46 @@ def _build_zinurax(config: dict, shapes: Dict[str, tuple], dtype: torch.dtype, m
 
 
 # ---------------------------------------------------------------------------------------------------------------------
+# Fabivik
+# ---------------------------------------------------------------------------------------------------------------------
+def _expert(e: dict) -> ExpertConfig:
+    return ExpertConfig(ff=e["ff"], limit=float(e["limit"]))
+
+
+def fabivik_config(config: dict, shapes: Dict[str, tuple], dtype: torch.dtype) -> HybridConfig:
+    """``config.json`` -> `HybridConfig`; ``shapes`` (checkpoint tensor -> shape) gives what the file leaves to the tensors."""
+    layers = []
+    for i, layer in enumerate(config["layers"]):
+        m, mlp = layer["mixer"], layer.get("mlp")
+        if layer["type"] == "attention":
+            mixer = ShortConvAttentionConfig(
+                heads=m["heads"], kv_heads=m["kv_heads"], dim=m["dim"], vdim=m["vdim"], scale=float(m["scale"]), conv=m["conv"],
+                window=(m.get("mask") or {}).get("size"), value_mix=bool(m.get("v_mix", False)))
+        elif layer["type"] == "wkv":
+            mixer = WkvConfig(heads=m["heads"], dim=m["dim"], rank=shapes[f"l{i}.mix.w1"][0])
+        elif layer["type"] == "delta":
+            mixer = GatedDeltaConfig(heads=m["heads"], kv_heads=m["kv_heads"], dim=m["dim"], vdim=m["vdim"], conv=m["conv"])
+        else:
+            raise ValueError(f"layer {i}: unknown mixer {layer['type']!r}")
+        moe = None
+        if mlp is not None:
+            if mlp["kind"] != "moe":
+                raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+            moe = MoeConfig(experts=mlp["router"]["experts"], top=mlp["router"]["top"], expert=_expert(mlp["expert"]),
+                            shared=_expert(mlp["shared"]) if mlp.get("shared") else None)
+        layers.append(HybridLayerConfig(mixer=mixer, moe=moe))
+    return HybridConfig(vocab_size=config["vocab"], hidden_size=config["width"], layers=tuple(layers), block="parallel",
+                        layernorm_epsilon=float(config["norm"]["eps"]), params_dtype=dtype,
+                        embedding_scale=float(config["embedding"]["scale"]), logit_scale=float(config["logit_scale"]))
+
+
+def _build_fabivik(config: dict, shapes: Dict[str, tuple], dtype: torch.dtype, max_sequence_length: int):
+    from .hybrid.parallel_model import ParallelHybridModel
+
+    return ParallelHybridModel(fabivik_config(config, shapes, dtype), max_sequence_length)
+
+
+# ---------------------------------------------------------------------------------------------------------------------
 # GPTModel: config.json holds TransformerConfig fields under "transformer" and the model's own beside it
 # ---------------------------------------------------------------------------------------------------------------------
 def _build_gpt(config: dict, shapes: Dict[str, tuple], dtype: torch.dtype, max_sequence_length: int):
@@ -64,7 +105,7 @@ def _build_gpt(config: dict, shapes: Dict[str, tuple], dtype: torch.dtype, max_s
 
 
 Builder = Callable[[dict, Dict[str, tuple], torch.dtype, int], torch.nn.Module]
-ARCHITECTURES: Dict[str, Builder] = {"Zinurax": _build_zinurax, "GPTModel": _build_gpt}
+ARCHITECTURES: Dict[str, Builder] = {"Fabivik": _build_fabivik, "Zinurax": _build_zinurax, "GPTModel": _build_gpt}
 
 
 def load_model(folder: str, *, dtype: torch.dtype = torch.bfloat16, max_sequence_length: int) -> torch.nn.Module:

@@ -730,6 +730,10 @@ def topp_probs(logits, top_p: float, temperature: float = 1.0):
 _DTYPE = {BF16: 0, F32: 1}
 _ACT = {None: 0, "relu2": 1}
 _OUT_NORM, _LATENT_APPEND, _LATENT_ATTENTION, _DELTA_DECODE, _DELTA_LORA, _DELTA_SCAN, _DELTA_FINISH, _LATENT_GATHER, _LATENT_PROMPT = range(9)
+# kernels that take an argument struct and nothing else (`struct_kernel`)
+_STRUCT_KERNELS = {name: 9 + i for i, name in enumerate((
+    "residual_norm", "conv_silu", "conv_qkv", "token_shift", "recurrence_decode", "recurrence_scan", "recurrence_finish",
+    "recurrence_lora", "moe_route", "moe_gather", "moe_up", "moe_down"))}
 
 
 def dtype_code(dtype) -> int:
@@ -860,3 +864,81 @@ def delta_scan(args, anchor) -> None:
 
 def delta_finish(args, anchor) -> None:
     _launch("hybrid", _blob(args), anchor, _DELTA_FINISH)
+
+
+# ---------------------------------------------------------------------------------------------------------------------
+# Parallel blocks: residual stream with two norms, short convolutions, linear recurrences, experts
+# ---------------------------------------------------------------------------------------------------------------------
+def struct_kernel(name: str, args, anchor) -> None:
+    """Launch ``b200_<name>`` with its argument struct (raw pointers: the caller keeps the tensors alive)."""
+    _launch("hybrid", _blob(args), anchor, _STRUCT_KERNELS[name])
+
+
+def partials_of(p: GemmPartials):
+    """(address, number of splits) of partial sums that no later GEMM has overwritten."""
+    if p.epoch != _gemm_epoch:
+        raise B200Error("partials", -1, "another GEMM has reused the workspace that held these partial sums")
+    return p.buf.data_ptr(), p.num_splits
+
+
+def separate_attention(args: AttentionArgs, dtype, *, units=None, num_units: int = 0, tensor_cores: bool) -> None:
+    """Attention of finished queries over a [keys | values] pool (``AttentionArgs.separate``); ``units``: a prefill step's work list."""
+    global launch_count
+    if not tensor_cores:
+        _launch("attention", _blob(args), args._anchor, 3, None, dtype_code(dtype))
+        return
+    if units is not None:
+        paged_prefill_attention(args, units, num_units)
+        return
+    nbytes = _lib.load().b200_paged_attention_workspace_bytes(args.num_tokens, args.num_q_heads, 64 if args.value_dim <= 64 else 128,
+                                                              args.num_splits)
+    if nbytes:
+        ws = _workspace.get(args._anchor.device, "attn", nbytes)
+        args.workspace, args.workspace_bytes = ws.data_ptr(), ws.numel()
+    paged_attention(args)
+
+
+def moe_counters(device, experts: int) -> torch.Tensor:
+    """The routing kernel's counters: zero, and left zero by every launch."""
+    return _workspace.get(device, "moe_counts", 4 * (experts + 1))
+
+
+class PendingRows:
+    """What still has to be added to the residual stream: scaled embeddings, or the outputs of a block's branches."""
+
+    __slots__ = ("table", "ids", "table_scale", "partials", "experts")
+
+    def __init__(self, *, table=None, ids=None, table_scale: float = 1.0, partials: Optional[GemmPartials] = None, experts=None):
+        self.table, self.ids, self.table_scale, self.partials, self.experts = table, ids, table_scale, partials, experts
+
+
+def residual_norm(hidden, pending: Optional[PendingRows], gammas, outs, *, eps: float, gain: float = 1.0, out_scale: float = 1.0,
+                  row_index=None) -> None:
+    """hidden += pending (the first rows of a stream: hidden = embeddings); outs[i] = rms norm of hidden times (gain + gammas[i])."""
+    _need(hidden, F32, "hidden")
+    a = _lib.ResidualNormArgs()
+    a.hidden, a.source_rows, a.width = hidden.data_ptr(), hidden.shape[0], hidden.shape[1]
+    a.rows, a.eps, a.gain, a.out_scale = hidden.shape[0], eps, gain, out_scale
+    dtype = gammas[0].dtype if gammas else (pending.table if pending.table is not None else pending.experts.rows if pending.experts is not None
+                                            else hidden).dtype
+    a.dtype = dtype_code(dtype)
+    if row_index is not None:
+        _need(row_index, torch.int64, "row_index")
+        a.row_index, a.rows = row_index.data_ptr(), row_index.numel()
+    if pending is not None:
+        if pending.table is not None:
+            _need(pending.table, dtype, "table")
+            _need(pending.ids, torch.int64, "ids")
+            a.table, a.ids, a.table_rows, a.table_scale = pending.table.data_ptr(), pending.ids.data_ptr(), pending.table.shape[0], pending.table_scale
+        if pending.partials is not None:
+            a.partials, a.num_splits = partials_of(pending.partials)
+        e = pending.experts
+        if e is not None:
+            a.expert_rows, a.expert_row_count, a.pairs, a.offsets = e.rows.data_ptr(), e.rows.shape[0], e.pairs.data_ptr(), e.offsets.data_ptr()
+            a.top, a.experts = e.top, e.experts
+            if e.shared_rows is not None:
+                a.shared_rows, a.shared_gate = e.shared_rows.data_ptr(), _p(e.shared_gate)
+    for i, (g, y) in enumerate(zip(gammas, outs)):
+        _need(y, dtype, "out")
+        a.gamma[i], a.y[i] = g.data_ptr(), y.data_ptr()
+    struct_kernel("residual_norm", a, hidden)

@@ -44,7 +44,7 @@ class GeneralDeltaRule(torch.nn.Module):
         decay with a GEMM and scan every request's tokens."""
         m, T, n, dev = self.mixer, x.shape[0], self.width, x.device
         proj, _ = self.linear_in(x)
-        state = ctx.recurrent_state(self.layer_number)
+        state = ctx.recurrent_state(self.layer_number, "state")
         out = torch.empty((T, n), dtype=x.dtype, device=dev)
         a = _lib.DeltaArgs()
         a.proj, a.proj_ld, a.out = proj.data_ptr(), proj.stride(0), out.data_ptr()

@@ -49,6 +49,12 @@ class LatentAttentionConfig:
         if self.window is not None and self.window < 1:
             raise ValueError("a window holds at least the token itself")
 
+    def cached_row_width(self) -> int:
+        return self.row_width if self.kv_from is None else 0
+
+    def request_state(self, hidden_size: int, dtype: torch.dtype) -> Optional[dict]:
+        return None
+
     @property
     def kv_pad(self) -> int:
         """Where the rotated part starts in a cached row."""
@@ -68,14 +74,136 @@ class DeltaRuleConfig:
     decay_scale: float = math.exp(-0.5)  # decay = exp(-decay_scale * sigmoid(.))
     unit_eps: float = 1e-6               # inside the unit key's root
 
+    def cached_row_width(self) -> int:
+        return 0
 
-MixerConfig = Union[LatentAttentionConfig, DeltaRuleConfig]
+    def request_state(self, hidden_size: int, dtype: torch.dtype) -> Optional[dict]:
+        return {"state": ((self.heads, self.dim, self.dim), torch.float32)}
+
+
+def _conv_state(channels: int, taps: int, dtype: torch.dtype) -> dict:
+    """The inputs a short convolution looks back at."""
+    return {"conv": ((taps - 1, channels), dtype)} if taps > 1 else {}
+
+
+def _check_taps(taps: int) -> None:
+    if not 1 <= taps <= 8:
+        raise ValueError("short convolutions have 1 to 8 taps")
+
+
+@dataclass(frozen=True)
+class ShortConvAttentionConfig:
+    """Grouped-query attention whose queries, keys and values pass a short causal convolution, with per-head norms of queries and
+    keys, no rotation, and optionally a window and values mixed with those of the first mixing layer."""
+
+    heads: int
+    kv_heads: int
+    dim: int                      # query / key dimensions per head
+    vdim: int                     # value dimensions per head
+    scale: float
+    conv: int                     # taps of the convolutions
+    window: Optional[int] = None  # keys seen, the token itself included; None: all earlier ones
+    value_mix: bool = False
+
+    def __post_init__(self):
+        if self.heads % self.kv_heads:
+            raise ValueError("heads must be a multiple of kv_heads")
+        if self.window is not None and self.window < 1:
+            raise ValueError("a window holds at least the token itself")
+        if max(self.dim, self.vdim) > 256:
+            raise ValueError("head dimensions go up to 256")
+        _check_taps(self.conv)
+
+    @property
+    def conv_channels(self) -> int:
+        return (self.heads + self.kv_heads) * self.dim + self.kv_heads * self.vdim
+
+    @property
+    def tensor_cores(self) -> bool:
+        """Head sizes that the tensor-core kernels take."""
+        return (self.dim % 8 == 0 and self.vdim % 8 == 0 and max(self.dim, self.vdim) <= 128 and self.heads // self.kv_heads <= 16)
+
+    def cached_row_width(self) -> int:
+        """Elements of a cached row: the keys of all heads, then the values."""
+        return self.kv_heads * (self.dim + self.vdim)
+
+    def request_state(self, hidden_size: int, dtype: torch.dtype) -> Optional[dict]:
+        return _conv_state(self.conv_channels, self.conv, dtype)
+
+
+@dataclass(frozen=True)
+class WkvConfig:
+    heads: int
+    dim: int   # key and value channels per head
+    rank: int  # inner width of the decay's two-step projection
+
+    def __post_init__(self):
+        if self.dim > 256:
+            raise ValueError("recurrent heads have up to 256 channels")
+
+    def cached_row_width(self) -> int:
+        return 0
+
+    def request_state(self, hidden_size: int, dtype: torch.dtype) -> Optional[dict]:
+        return {"state": ((self.heads, self.dim, self.dim), torch.float32), "shift": ((hidden_size,), dtype)}
+
+
+@dataclass(frozen=True)
+class GatedDeltaConfig:
+    heads: int
+    kv_heads: int
+    dim: int   # query / key channels per head
+    vdim: int  # value channels per head
+    conv: int  # taps of the convolutions
+    unit_eps: float = 1e-6  # inside the unit vectors' root
+
+    def __post_init__(self):
+        if self.heads % self.kv_heads:
+            raise ValueError("heads must be a multiple of kv_heads")
+        if self.dim > 256:
+            raise ValueError("recurrent heads have up to 256 key channels")
+        _check_taps(self.conv)
+
+    @property
+    def conv_channels(self) -> int:
+        return 2 * self.kv_heads * self.dim + self.heads * self.vdim
+
+    def cached_row_width(self) -> int:
+        return 0
+
+    def request_state(self, hidden_size: int, dtype: torch.dtype) -> Optional[dict]:
+        return {"state": ((self.heads, self.vdim, self.dim), torch.float32), **_conv_state(self.conv_channels, self.conv, dtype)}
+
+
+MixerConfig = Union[LatentAttentionConfig, DeltaRuleConfig, ShortConvAttentionConfig, WkvConfig, GatedDeltaConfig]
+
+
+@dataclass(frozen=True)
+class ExpertConfig:
+    """One gated feed-forward: g' sigmoid(alpha g') (u' + 1), g' = min(g, limit), u' clamped to [-limit, limit]."""
+
+    ff: int
+    limit: float
+    alpha: float = 1.702
+
+
+@dataclass(frozen=True)
+class MoeConfig:
+    experts: int
+    top: int  # experts per token; their weights are their sigmoid scores
+    expert: ExpertConfig
+    shared: Optional[ExpertConfig] = None  # runs for every token, times a gate of its own
+
+    def __post_init__(self):
+        if not 1 <= self.top <= min(self.experts, 64) or self.experts > 1024:
+            raise ValueError("1 <= top <= experts, at most 64 of 1024")
 
 
 @dataclass(frozen=True)
 class HybridLayerConfig:
     mixer: MixerConfig
-    ffn_hidden_size: Optional[int] = None  # None: no feed-forward
+    ffn_hidden_size: Optional[int] = None  # width of a dense feed-forward
+    moe: Optional[MoeConfig] = None        # or a mixture of experts; both None: no feed-forward
 
 
 @dataclass
@@ -95,6 +223,12 @@ class HybridConfig:
     inference_sampling_seed: int = 42
     fuse_splitk_reduction_into_norm: bool = True
     defer_logits_gather: bool = True
+    # "output_norm": sublayers one after the other with norms on their outputs, embedding norm, tied head (`HybridModel`);
+    # "parallel": mixer and feed-forward side by side on two norms of the same stream, scaled embedding, a head of its own
+    # (`ParallelHybridModel`)
+    block: str = "output_norm"
+    embedding_scale: float = 1.0
+    logit_scale: float = 1.0
 
     def __post_init__(self):
         self.layers = tuple(self.layers)
@@ -102,6 +236,10 @@ class HybridConfig:
             raise ValueError("hybrid decoders compute in bfloat16 or float32")
         if self.tensor_model_parallel_size != 1:
             raise NotImplementedError("hybrid decoders run on one GPU")
+        if self.block == "parallel":
+            mixing = [x.mixer for x in self.layers if isinstance(x.mixer, ShortConvAttentionConfig) and x.mixer.value_mix]
+            if len({(m.kv_heads, m.vdim) for m in mixing}) > 1:
+                raise ValueError("layers whose values are mixed must agree in their number and size")
         for i, layer in enumerate(self.layers):
             m = layer.mixer
             src = getattr(m, "kv_from", None)

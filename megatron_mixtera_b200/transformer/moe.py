@@ -1,0 +1,120 @@
+"""Mixture of experts with sigmoid scores: every token runs its `top` best experts on its input times their scores, and a gated
+shared expert.  Tokens are sorted by expert on the device; the products of all experts are one grouped GEMM."""
+from __future__ import annotations
+
+import torch
+
+from .. import _lib, ops
+from ..tensor_parallel.layers import _device
+from .hybrid_config import HybridConfig, MoeConfig
+
+
+def _padded(ff: int) -> int:
+    """Whole blocks of 64 features: a 128-row tile of the up weights holds 64 gate rows and the matching up rows."""
+    return -(-ff // 64) * 64
+
+
+def interleave_up(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
+    """[ff, H] each -> [2 * padded ff, H], blocks of 64 gate rows and 64 up rows, missing rows zero."""
+    ff, H = gate.shape
+    pad = _padded(ff)
+    out = torch.zeros((pad // 64, 2, 64, H), dtype=gate.dtype, device=gate.device)
+    for i, w in enumerate((gate, up)):
+        full = torch.zeros((pad, H), dtype=gate.dtype, device=gate.device)
+        full[:ff] = w
+        out[:, i] = full.view(pad // 64, 64, H)
+    return out.view(2 * pad, H)
+
+
+class ExpertOutputs:
+    """What `MixtureOfExperts` hands to the kernel that adds it to the stream: expert outputs sorted by expert, where a token's rows
+    lie among them, and the shared expert's rows with their gates."""
+
+    __slots__ = ("rows", "pairs", "offsets", "top", "experts", "shared_rows", "shared_gate")
+
+    def __init__(self, rows, pairs, offsets, top, experts, shared_rows, shared_gate):
+        self.rows, self.pairs, self.offsets, self.top, self.experts = rows, pairs, offsets, top, experts
+        self.shared_rows, self.shared_gate = shared_rows, shared_gate
+
+
+class MixtureOfExperts(torch.nn.Module):
+    def __init__(self, config: HybridConfig, moe: MoeConfig):
+        super().__init__()
+        self.config, self.moe = config, moe
+        H = config.hidden_size
+
+        def param(*shape):
+            return torch.nn.Parameter(torch.zeros(shape, dtype=config.params_dtype, device=_device()), requires_grad=False)
+
+        self.ff = _padded(moe.expert.ff)
+        # router rows, then the shared expert's gate
+        self.router = param(-(-(moe.experts + (moe.shared is not None)) // 8) * 8, H)
+        self.up, self.down = param(moe.experts, 2 * self.ff, H), param(moe.experts, H, self.ff)
+        self.shared_ff, self.shared_up, self.shared_down = 0, None, None
+        if moe.shared is not None:
+            self.shared_ff = _padded(moe.shared.ff)
+            self.shared_up, self.shared_down = param(2 * self.shared_ff, H), param(H, self.shared_ff)
+
+    def checkpoint_tensors(self) -> dict:
+        H, c = self.config.hidden_size, self.moe
+        out = {"router": (c.experts, H)}
+        parts = [(f"e{e}", c.expert.ff) for e in range(c.experts)]
+        if c.shared is not None:
+            parts.append(("shared", c.shared.ff))
+            out["shared.sg"] = (1, H)
+        for name, ff in parts:
+            out.update({f"{name}.gate": (ff, H), f"{name}.up": (ff, H), f"{name}.down": (H, ff)})
+        return out
+
+    def load(self, get) -> None:
+        c, dev = self.moe, self.router.device
+        self.router.data[: c.experts].copy_(get("router"))
+        for e in range(c.experts):
+            self.up.data[e].copy_(interleave_up(get(f"e{e}.gate").to(dev), get(f"e{e}.up").to(dev)))
+            self.down.data[e, :, : c.expert.ff].copy_(get(f"e{e}.down"))
+        if c.shared is not None:
+            self.router.data[c.experts].copy_(get("shared.sg")[0])
+            self.shared_up.data.copy_(interleave_up(get("shared.gate").to(dev), get("shared.up").to(dev)))
+            self.shared_down.data[:, : c.shared.ff].copy_(get("shared.down"))
+
+    @staticmethod
+    def tile_tokens(pairs: int, experts: int, simt: bool) -> int:
+        """Tokens of a tile of the grouped products, by how many an expert gets on average."""
+        if simt:
+            return 64
+        average = pairs / experts
+        return 256 if average >= 768 else 128 if average >= 128 else 64 if average >= 40 else 32
+
+    def forward(self, x) -> ExpertOutputs:
+        c, (T, H), dev, dt = self.moe, x.shape, x.device, x.dtype
+        pairs, simt = T * c.top, dt == torch.float32 or H % 8 != 0
+        a = _lib.MoeArgs()
+        a.num_tokens, a.width, a.experts, a.top, a.ff, a.shared_ff = T, H, c.experts, c.top, self.ff, self.shared_ff
+        a.limit, a.alpha, a.simt, a.dtype = c.expert.limit, c.expert.alpha, int(simt), ops.dtype_code(dt)
+        a.tile_tokens = self.tile_tokens(pairs, c.experts, simt)
+        a.max_tiles = pairs // a.tile_tokens + min(c.experts, pairs)
+        # bookkeeping in one block of 32-bit words: pairs | weights | row scales | shared gates | offsets | tiles | number of tiles
+        sizes = (2 * pairs, pairs, pairs, T, c.experts + 1, 4 * a.max_tiles, 1)
+        starts = [0]
+        for n in sizes:
+            starts.append(starts[-1] + -(-n // 4) * 4)  # 16-byte aligned
+        words = torch.empty(starts[-1], dtype=torch.int32, device=dev)
+        at = [words.data_ptr() + 4 * s for s in starts]
+        a.pairs, a.pair_weight, a.row_scale, shared_gate, a.offsets, a.tiles, a.num_tiles = at[:7]
+        a.counts = ops.moe_counters(dev, c.experts).data_ptr()
+        a.x, a.up, a.down = x.data_ptr(), self.up.data_ptr(), self.down.data_ptr()
+        x_sorted = torch.empty((pairs, H), dtype=dt, device=dev)
+        inter, rows = torch.empty((pairs, self.ff), dtype=dt, device=dev), torch.empty((pairs, H), dtype=dt, device=dev)
+        a.x_sorted, a.inter, a.y = x_sorted.data_ptr(), inter.data_ptr(), rows.data_ptr()
+        shared_rows = shared_inter = None
+        if c.shared is not None:
+            shared_inter, shared_rows = torch.empty((T, self.shared_ff), dtype=dt, device=dev), torch.empty((T, H), dtype=dt, device=dev)
+            a.shared_gate, a.shared_up, a.shared_down = shared_gate, self.shared_up.data_ptr(), self.shared_down.data_ptr()
+            a.shared_inter, a.shared_y, a.shared_limit = shared_inter.data_ptr(), shared_rows.data_ptr(), c.shared.limit
+        logits = ops.linear_partials(x, self.router)  # fp32 sums of exact products: the router's 32-bit logits
+        a.router, a.router_splits = ops.partials_of(logits)
+        a.router_ld = self.router.shape[0]
+        for kernel in ("moe_route", "moe_gather", "moe_up", "moe_down"):
+            ops.struct_kernel(kernel, a, x)
+        gates = words[starts[3]: starts[3] + T].view(torch.float32) if c.shared is not None else None
+        return ExpertOutputs(rows, words, words[starts[4]:], c.top, c.experts, shared_rows, gates)

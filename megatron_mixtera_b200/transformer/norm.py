@@ -72,3 +72,22 @@ class OutputNorm(torch.nn.Module):
     def of_rows(self, hidden, row_index=None):
         """norm of the stream's rows (all, or those picked by ``row_index``) in the activation type."""
         return ops.out_norm(hidden, self.weight, eps=self.eps, row_index=row_index)
+
+
+class ParallelNorm(torch.nn.Module):
+    """Everything a parallel block adds to the 32-bit residual stream and the RMS norms of the result, in one kernel.  ``outputs``
+    norms of the same row (weights stored as the distance from one) feed the branches that run side by side."""
+
+    def __init__(self, config, hidden_size: int, eps: float, outputs: int = 2, out_scale: float = 1.0):
+        super().__init__()
+        dev = torch.device("cuda", torch.cuda.current_device()) if torch.cuda.is_available() else torch.device("cpu")
+        self.eps, self.out_scale = eps, out_scale
+        self.weight = torch.nn.Parameter(torch.zeros((outputs, hidden_size), dtype=config.params_dtype, device=dev), requires_grad=False)
+
+    def forward(self, hidden, pending, row_index=None):
+        """Adds ``pending`` (a `PendingRows`, or None) to ``hidden`` [T, H] in place and returns the norms; with ``row_index`` (int64)
+        only those rows are computed and ``hidden`` stays as it is."""
+        rows = hidden.shape[0] if row_index is None else row_index.numel()
+        out = [torch.empty((rows, hidden.shape[1]), dtype=self.weight.dtype, device=hidden.device) for _ in range(self.weight.shape[0])]
+        ops.residual_norm(hidden, pending, list(self.weight), out, eps=self.eps, gain=1.0, out_scale=self.out_scale, row_index=row_index)
+        return out

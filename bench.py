@@ -821,21 +821,21 @@ def main():
                          "pool with seeded noise (decode timing does not depend on the pool's contents)")
     ap.add_argument("--deadline", type=int, default=1500,
                     help="seconds after which a stuck run dumps every thread's stack and exits instead of waiting to be killed")
-    ap.add_argument("--design", default=None, choices=["zinurax"],
+    ap.add_argument("--design", default=None, choices=["zinurax", "fabivik"],
                     help="time this design's prefill, decode and kernels beside the closest GPT model instead of the workload (one GPU)")
-    ap.add_argument("--zinurax-sizes", default=None, help="with --design zinurax: sizes, comma-separated (default: all)")
-    ap.add_argument("--zinurax-window", type=int, default=4096, help="with --design zinurax: attention window in tokens")
+    ap.add_argument("--design-sizes", "--zinurax-sizes", default=None, help="with --design: sizes, comma-separated (default: all)")
+    ap.add_argument("--design-window", "--zinurax-window", type=int, default=4096, help="with --design: attention window in tokens")
     args = ap.parse_args()
     import faulthandler
 
     faulthandler.dump_traceback_later(args.deadline, exit=True)
     protect_stdout()
-    if args.design == "zinurax":
-        import bench_zinurax
+    if args.design:
+        import importlib
 
         with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
             peaks = json.load(f)
-        bench_zinurax.run(args, emit, (float(peaks["hbm_gbs"]), float(peaks["bf16_tflops"])))
+        importlib.import_module("bench_" + args.design).run(args, emit, (float(peaks["hbm_gbs"]), float(peaks["bf16_tflops"])))
         return
     w = configs.WORKLOADS[args.workload]
     if args.synthesize_kv and not w.synthesize_kv:

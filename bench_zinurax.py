@@ -123,6 +123,8 @@ HYBRID = ("out_norm", "latent_append", "latent_attention", "delta_decode", "delt
 
 
 def label(name, args):
+    from megatron_mixtera_b200 import _lib, ops
+
     if name == "linear":
         batch = args[9]
         return "gemm %dx%dx%d%s" % (args[5], args[6], args[7], " x%d heads" % batch if batch > 1 else ""), (args[5], args[6] * batch, args[7], batch)
@@ -133,7 +135,10 @@ def label(name, args):
         M, (N, K) = args[0].numel() // args[0].shape[-1], args[1].shape
         return "gemm %dx%dx%d +swiglu" % (M, N, K), (M, N, K, 1)
     if name == "hybrid":
-        return HYBRID[args[2]], None
+        kernel = (HYBRID + tuple(ops._STRUCT_KERNELS))[args[2]]
+        if kernel in ("recurrence_decode", "recurrence_scan", "recurrence_finish"):  # one kernel, two rules
+            kernel = ("wkv", "delta")[_lib.RecurrenceArgs.from_buffer_copy(args[0].numpy().tobytes()).kind] + kernel[len("recurrence"):]
+        return kernel, None
     if name == "attention":
         return ("rope_append", "paged_attention", "paged_prefill_attention")[args[2]], None
     return name, None
@@ -190,10 +195,12 @@ def kernel_table(rec, cost, hbm, tflops):
     return table
 
 
-def measure(kind, s, hbm, tflops, window):
+def measure(kind, s, hbm, tflops, window, build=None, costs=costs):
+    """``kind`` "gpt": the GPT model; anything else: the design that ``build`` makes, with ``costs`` for its kernels."""
     requests, max_len = REQUESTS, CONTEXT + 64
     tokens = requests * (-(-max_len // 256) * 256) + PROMPTS * (PROMPT_LEN + 256)
-    model, ctx, wrapper = (build_zinurax if kind == "zinurax" else build_gpt)(s, max_len, tokens, requests, window)
+    gpt = kind == "gpt"
+    model, ctx, wrapper = (build_gpt if gpt else build or build_zinurax)(s, max_len, tokens, requests, window)
     out = {"parameters": sum(p.numel() for p in model.parameters())}
     with torch.inference_mode():
         # ---- prefill ----
@@ -206,10 +213,10 @@ def measure(kind, s, hbm, tflops, window):
         fwd = lambda: model.forward_rows(ids, pos, ctx, last, True)
         fwd()
         us = elapsed_us(fwd, 5)
-        per_prompt = sum(min(p + 1, window) if kind == "zinurax" else p + 1 for p in range(PROMPT_LEN))
+        per_prompt = sum(p + 1 if gpt else min(p + 1, window) for p in range(PROMPT_LEN))
         with Recorder() as rec:
             fwd()
-        cost = costs(s, T, PROMPTS * per_prompt, T, kind == "zinurax", False, PROMPTS)
+        cost = costs(s, T, PROMPTS * per_prompt, T, not gpt, False, PROMPTS)
         out["prefill"] = {"tokens": T, "ms": round(us / 1e3, 3), "tokens_per_s": round(T / us * 1e6),
                           "kernels": kernel_table(rec, cost, hbm, tflops)}
         del rec
@@ -227,8 +234,8 @@ def measure(kind, s, hbm, tflops, window):
         us = elapsed_us(graph.replay, 20)
         with Recorder() as rec:
             fwd()
-        keys = requests * (min(CONTEXT, window) if kind == "zinurax" else CONTEXT)
-        cost = costs(s, requests, keys, keys, kind == "zinurax", True, requests)
+        keys = requests * (CONTEXT if gpt else min(CONTEXT, window))
+        cost = costs(s, requests, keys, keys, not gpt, True, requests)
         out["decode"] = {"requests": requests, "context": CONTEXT, "us": round(us, 1), "tokens_per_s": round(requests / us * 1e6),
                          "kernels": kernel_table(rec, cost, hbm, tflops)}
         del rec, graph
@@ -240,14 +247,14 @@ def run(args, emit, peaks):
 
     build.build_torch_ops()
     hbm, tflops = peaks
-    line = {"bench": "zinurax", "data": "synthetic", "dtype": "bf16", "n_gpus": 1, "window": args.zinurax_window,
+    line = {"bench": "zinurax", "data": "synthetic", "dtype": "bf16", "n_gpus": 1, "window": args.design_window,
             "peaks": {"hbm_gbs": hbm, "bf16_tflops": tflops, "fp32_tflops_nominal": round(FP32_FLOPS / 1e12, 1)},
             "l2": "every sweep runs over all layers' own weights, cache and state", "sizes": {}}
-    for name in (args.zinurax_sizes.split(",") if args.zinurax_sizes else SIZES):
+    for name in (args.design_sizes.split(",") if args.design_sizes else SIZES):
         s = SIZES[name]
         line["sizes"][name] = {"shape": s}
         for kind in ("zinurax", "gpt"):
-            line["sizes"][name][kind] = measure(kind, s, hbm, tflops, args.zinurax_window)
+            line["sizes"][name][kind] = measure(kind, s, hbm, tflops, args.design_window)
             torch.cuda.empty_cache()
     line["device_status"] = ops.device_status()
     line["gpu_launches"] = ops.launch_count

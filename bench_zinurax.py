@@ -226,7 +226,7 @@ def measure(kind, s, hbm, tflops, window, build=None, costs=costs):
         for i in range(requests):
             ctx.schedule_tokens([(i, torch.zeros(CONTEXT - 1, dtype=torch.int64))])
             ctx.complete_step()
-        ctx.schedule_tokens([(i, [1]) for i in range(requests)])
+        ctx.schedule_tokens([(i, torch.randint(0, VOCAB, (1,), generator=g)) for i in range(requests)])
         ctx.initialize_attention_state()
         ids, pos = ctx.current_input_and_position_ids()
         fwd = lambda: model.forward_rows(ids, pos, ctx, None, True)

@@ -733,7 +733,7 @@ int b200_recurrence_lora(const b200_recurrence_args* args, b200_stream_t stream)
 
 /* Mixture of experts.  Expert: y = W_down act(W_gate x', W_up x') with x' = weight * x (the weight is applied to the products, in
  * fp32), act(g, u) = g' sigmoid(alpha g') (u' + 1), g' = min(g, limit), u' = clamp(u, -limit, limit).
- * up weights [experts][2 * ff][width]: every 128 rows are 64 gate rows and the 64 matching up rows; ff a multiple of 64 (padded with
+ * up weights [experts][2 * ff][width]: every 32 rows are 16 gate rows and the 16 matching up rows; ff a multiple of 64 (padded with
  * zero rows).  down weights [experts][width][ff].  A shared expert of its own size may run on every token in the same launches.
  * b200_moe_route: scores = sigmoid(router logits [router_splits][T][router_ld], fp32 partial sums), the `top` largest per token; their
  *   places when tokens are sorted by expert; shared_gate = sigmoid(logit column `experts`); the list of (expert, first row, rows)

@@ -55,7 +55,7 @@ struct Params {
   // weight rows [b * N, (b + 1) * N) into y + b * y_batch.  m_blocks: token blocks per batch (blockIdx.z holds both).
   int m_blocks = 1, x_batch = 0;
   int64_t y_batch = 0;
-  // gated == kGatedClamped: y = g' sigmoid(glu_alpha g') (u' + 1) with g' = min(g, glu_limit), u' clamped to [-glu_limit, glu_limit], all
+  // gated == kGatedClamped: every 32 rows of a weight tile are 16 gate features and the matching 16 up features; y = g' sigmoid(glu_alpha g') (u' + 1) with g' = min(g, glu_limit), u' clamped to [-glu_limit, glu_limit], all
   // in fp32; row_scale (NULL: 1) multiplies both products of a token first.
   float glu_limit = 0.f, glu_alpha = 0.f;
   const float* row_scale = nullptr;
@@ -66,6 +66,12 @@ __device__ __forceinline__ float clamped_glu(float g, float u, float limit, floa
   g = fminf(g, limit);
   u = fminf(fmaxf(u, -limit), limit);
   return g / (1.f + expf(-alpha * g)) * (u + 1.f);
+}
+// The same with the fast exponential and division (about 1e-6 relative), for outputs that are rounded to bf16.
+__device__ __forceinline__ float clamped_glu_fast(float g, float u, float limit, float alpha) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return __fdividef(g, 1.f + __expf(-alpha * g)) * (u + 1.f);
 }
 
 __device__ __forceinline__ float apply_act(float v, int act) {
@@ -155,7 +161,30 @@ __device__ __forceinline__ void epilogue(const Params& p, uint32_t tmem_base, ui
   const bool n_ok = n < p.N;
   const uint32_t lane_addr = tmem_base + (static_cast<uint32_t>(warp * 32) << 16);
 
-  if (p.gated) {
+  if (p.gated == kGatedClamped) {
+    // A warp's lanes 0-15 hold gate features, lanes 16-31 the matching up features.  Of every 32 tokens the gate lanes finish the
+    // first 16 and the up lanes the others: one shuffle per finished output, no barrier.
+    const bool is_gate = lane < 16;
+    const int out_col = n_tile * 64 + warp * 16 + (lane & 15);
+    const bool col_ok = out_col < (p.N >> 1);
+#pragma unroll 1
+    for (int c0 = 0; c0 < BT && m0 + c0 < m_end; c0 += 32) {
+      uint32_t r[32];
+      tmem_ld_32x32b_x32(lane_addr + c0, r);
+      tmem_ld_wait();
+      const int own0 = m0 + c0 + (is_gate ? 0 : 16);
+      float sc[16];
+#pragma unroll
+      for (int j = 0; j < 16; ++j) sc[j] = p.row_scale != nullptr ? p.row_scale[min(own0 + j, m_end - 1)] : 1.f;
+#pragma unroll
+      for (int j = 0; j < 16; ++j) {
+        const float mine = __uint_as_float(is_gate ? r[j] : r[j + 16]);
+        const float other = __shfl_xor_sync(0xffffffffu, __uint_as_float(is_gate ? r[j + 16] : r[j]), 16);
+        const float v = clamped_glu_fast((is_gate ? mine : other) * sc[j], (is_gate ? other : mine) * sc[j], p.glu_limit, p.glu_alpha);
+        if (col_ok && own0 + j < m_end) y[static_cast<int64_t>(own0 + j) * p.ldy + out_col] = __float2bfloat16_rn(v);
+      }
+    }
+  } else if (p.gated) {
     // SwiGLU in the epilogue.  Warps 0-1 hold gate features, warps 2-3 the matching up features (same lane).  Of
     // every 32 tokens the gate warps finish the first 16 and the up warps the last 16: each side parks the half it
     // does not finish in shared memory (the pipeline stages are free, every UMMA has completed).  Rounding points as
@@ -174,8 +203,7 @@ __device__ __forceinline__ void epilogue(const Params& p, uint32_t tmem_base, ui
 #pragma unroll
       for (int j = 0; j < 16; ++j) {
         const int jj = is_gate ? j + 16 : j;            // the other side's tokens
-        const float parked = __uint_as_float(is_gate ? r[j + 16] : r[j]);
-        xch[(c0 + jj) * 64 + f] = p.gated == kGatedClamped ? parked : bf16_round(parked);
+        xch[(c0 + jj) * 64 + f] = bf16_round(__uint_as_float(is_gate ? r[j + 16] : r[j]));
       }
       __syncthreads();
       if (col_ok) {
@@ -183,15 +211,8 @@ __device__ __forceinline__ void epilogue(const Params& p, uint32_t tmem_base, ui
         for (int j = 0; j < 16; ++j) {
           const int m = m0 + c0 + own0 + j;
           if (m < m_end) {
-            const float raw = __uint_as_float(is_gate ? r[j] : r[j + 16]);
+            const float mine = bf16_round(__uint_as_float(is_gate ? r[j] : r[j + 16]));
             const float other = xch[(c0 + own0 + j) * 64 + f];
-            if (p.gated == kGatedClamped) {
-              const float sc = p.row_scale != nullptr ? p.row_scale[m] : 1.f;
-              const float v = clamped_glu((is_gate ? raw : other) * sc, (is_gate ? other : raw) * sc, p.glu_limit, p.glu_alpha);
-              y[static_cast<int64_t>(m) * p.ldy + out_col] = __float2bfloat16_rn(v);
-              continue;
-            }
-            const float mine = bf16_round(raw);
             const float g = is_gate ? mine : other;
             const float u = is_gate ? other : mine;
             const float a = bf16_round(g / (1.f + expf(-g)));

@@ -37,6 +37,9 @@ route_kernel(b200_moe_args a) {
         a.shared_gate[t] = x;
     }
     __syncwarp();
+    int chosen = 0;       // lane k: the k-th choice and its score
+    float weight = 0.f;
+    int taken = 0;
     for (int k = 0; k < a.top; ++k) {
       float best = -1.f;  // (scores are positive; a chosen one is marked -2)
       int at = E;
@@ -55,14 +58,21 @@ route_kernel(b200_moe_args a) {
         }
       }
       if (at >= E) at = k;  // no number left (NaN scores): any expert, its output is NaN too
-      if (lane == 0) {
-        const int rank = atomicAdd(&a.counts[at], 1);
-        const int64_t pair = static_cast<int64_t>(t) * a.top + k;
-        reinterpret_cast<int2*>(a.pairs)[pair] = make_int2(at, rank);
-        a.pair_weight[pair] = score[at];
-        score[at] = -2.f;
+      if (lane == (k & 31)) {
+        chosen = at;
+        weight = score[at];
       }
       __syncwarp();
+      if (lane == (at & 31)) score[at] = -2.f;  // (only this lane looks at it again)
+      __syncwarp();
+      if ((k & 31) == 31 || k == a.top - 1) {  // up to 32 choices count themselves at once
+        if (lane <= (k & 31)) {
+          const int64_t pair = static_cast<int64_t>(t) * a.top + taken + lane;
+          reinterpret_cast<int2*>(a.pairs)[pair] = make_int2(chosen, atomicAdd(&a.counts[chosen], 1));
+          a.pair_weight[pair] = weight;
+        }
+        taken = k + 1;
+      }
     }
   }
   __syncthreads();
@@ -179,8 +189,9 @@ simt_kernel(b200_moe_args a, int shared_blocks) {
       const int r = i / kK, k = i - r * kK;
       const bool kin = k0 + k < K;
       xs[k][r] = kin && r < rows ? simt::to_f32(x[static_cast<int64_t>(m0 + r) * K + k0 + k]) : 0.f;
-      ws[0][k][r] = kin && n0 + r < N ? simt::to_f32(w[static_cast<int64_t>(r) * K + k0 + k]) : 0.f;
-      if (GATED) ws[GATED ? 1 : 0][k][r] = kin ? simt::to_f32(w[static_cast<int64_t>(64 + r) * K + k0 + k]) : 0.f;
+      const int wr = GATED ? r / 16 * 32 + r % 16 : r;  // (gated: every 32 rows are 16 gate rows and the matching 16 up rows)
+      ws[0][k][r] = kin && n0 + r < N ? simt::to_f32(w[static_cast<int64_t>(wr) * K + k0 + k]) : 0.f;
+      if (GATED) ws[GATED ? 1 : 0][k][r] = kin ? simt::to_f32(w[static_cast<int64_t>(wr + 16) * K + k0 + k]) : 0.f;
     }
     __syncthreads();
 #pragma unroll

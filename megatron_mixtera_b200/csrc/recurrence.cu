@@ -106,28 +106,69 @@ struct Delta {
   }
 };
 
-// Queries and keys of one token, EL channels per lane (zeros past dim) -> unit vectors in shared memory and the scalars.
-template <int DIM, int EL>
-__device__ __forceinline__ void put_delta(float* vec, float* scalar, const float (&q)[EL], const float (&k)[EL], int lane, int dim,
-                                          float unit_eps, float decay_rate, float x_a, float x_b) {
-  float qq = 0.f, kk = 0.f, qk = 0.f;
+// A lane owns channels [lane * EL, lane * EL + EL) while a token is prepared: one vector load each where the layout allows (VEC).
+// Addresses are clamped instead of branched over, so that the loads of several tokens are in flight together; channels past dim
+// are zeroed by `clear_tail`.
+template <bool VEC, typename T, int EL>
+__device__ __forceinline__ void load_channels(const T* p, int lane, int dim, float (&v)[EL]) {
+  if constexpr (VEC) {
+    conv::load<T, EL>(p + min(lane * EL, dim - EL), v);
+  } else {
 #pragma unroll
-  for (int e = 0; e < EL; ++e) {
-    qq = fmaf(q[e], q[e], qq);
-    kk = fmaf(k[e], k[e], kk);
-    qk = fmaf(q[e], k[e], qk);
+    for (int e = 0; e < EL; ++e) v[e] = simt::to_f32(p[min(lane * EL + e, dim - 1)]);
   }
-  const float uq = 1.f / (sqrtf(warp_sum(qq) + unit_eps) * sqrtf(static_cast<float>(dim))), uk = 1.f / sqrtf(warp_sum(kk) + unit_eps);
-  qk = warp_sum(qk);
+}
+template <int EL>
+__device__ __forceinline__ void clear_tail(float (&v)[EL], int lane, int dim) {
 #pragma unroll
-  for (int e = 0; e < EL; ++e) {
-    vec[lane + e * 32] = q[e] * uq;
-    vec[DIM + lane + e * 32] = k[e] * uk;
+  for (int e = 0; e < EL; ++e) v[e] = lane * EL + e < dim ? v[e] : 0.f;
+}
+
+// Queries and keys of Q tokens (zeros past dim) -> unit vectors in shared memory, `pitch` floats from one token's to the next's, and
+// the scalars behind them (`scalar_at`).  The sums of all tokens run side by side, the scalars on a lane per token.
+template <int DIM, int EL, int Q>
+__device__ __forceinline__ void put_delta(float* vec, int pitch, int scalar_at, const float (&q)[Q][EL], const float (&k)[Q][EL], int lane,
+                                          int dim, float unit_eps, float decay_rate, const float (&x_a)[Q], const float (&x_b)[Q]) {
+  float qq[Q], kk[Q], qk[Q];
+#pragma unroll
+  for (int t = 0; t < Q; ++t) {
+    qq[t] = kk[t] = qk[t] = 0.f;
+#pragma unroll
+    for (int e = 0; e < EL; ++e) {
+      qq[t] = fmaf(q[t][e], q[t][e], qq[t]);
+      kk[t] = fmaf(k[t][e], k[t][e], kk[t]);
+      qk[t] = fmaf(q[t][e], k[t][e], qk[t]);
+    }
   }
-  if (lane == 0) {
-    scalar[0] = expf(-expf(decay_rate) * softplus(x_a));
-    scalar[1] = sigmoid(x_b);
-    scalar[2] = qk * uq * uk;
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+    for (int t = 0; t < Q; ++t) {
+      qq[t] += __shfl_xor_sync(0xffffffffu, qq[t], o);
+      kk[t] += __shfl_xor_sync(0xffffffffu, kk[t], o);
+      qk[t] += __shfl_xor_sync(0xffffffffu, qk[t], o);
+    }
+  const float root = sqrtf(static_cast<float>(dim));
+  float mine_a = x_a[0], mine_b = x_b[0], mine_qk = 0.f;
+#pragma unroll
+  for (int t = 0; t < Q; ++t) {
+    const float uq = 1.f / (sqrtf(qq[t] + unit_eps) * root), uk = 1.f / sqrtf(kk[t] + unit_eps);
+#pragma unroll
+    for (int e = 0; e < EL; ++e) {
+      vec[t * pitch + lane * EL + e] = q[t][e] * uq;
+      vec[t * pitch + DIM + lane * EL + e] = k[t][e] * uk;
+    }
+    if (lane == t) {
+      mine_a = x_a[t];
+      mine_b = x_b[t];
+      mine_qk = qk[t] * uq * uk;
+    }
+  }
+  if (lane < Q) {
+    float* scalar = vec + lane * pitch + scalar_at;
+    scalar[0] = expf(-expf(decay_rate) * softplus(mine_a));
+    scalar[1] = sigmoid(mine_b);
+    scalar[2] = mine_qk;
   }
 }
 template <int DIM, int EL>
@@ -137,9 +178,9 @@ __device__ __forceinline__ void put_wkv(float* vec, float* scalar, const float (
 #pragma unroll
   for (int e = 0; e < EL; ++e) {
     b = fmaf(r[e] * bonus[e], k[e], b);
-    vec[lane + e * 32] = r[e];
-    vec[DIM + lane + e * 32] = lane + e * 32 < dim ? expf(-expf(z[e])) : 0.f;
-    vec[2 * DIM + lane + e * 32] = k[e];
+    vec[lane * EL + e] = r[e];
+    vec[DIM + lane * EL + e] = lane * EL + e < dim ? expf(-expf(z[e])) : 0.f;
+    vec[2 * DIM + lane * EL + e] = k[e];
   }
   b = warp_sum(b);
   if (lane == 0) scalar[0] = b;
@@ -158,28 +199,29 @@ struct DecodeShape {
   static constexpr int kElems = DIM / 32;
 };
 
-// One channel of the short convolution of row `row`'s token, its state moved on by one token where `keep` says so.
-template <typename T>
-__device__ __forceinline__ float conv_channel(const b200_recurrence_args& a, int channels, float now, int c, int in, int out, bool keep) {
-  const T* filter = static_cast<const T*>(a.conv_filter) + c;
-  const int64_t n = a.taps - 1;
-  const T* src = static_cast<const T*>(a.conv_state) + in * n * channels + c;
-  T* dst = static_cast<T*>(a.conv_state) + out * n * channels + c;
-  float y = simt::to_f32(filter[n * channels]) * now;
-  for (int j = 0; j < n; ++j) {
-    const float u = in >= 0 ? simt::to_f32(src[j * static_cast<int64_t>(channels)]) : 0.f;
-    y = fmaf(simt::to_f32(filter[j * static_cast<int64_t>(channels)]), u, y);
-    if (keep && out >= 0 && j > 0) simt::store_as(dst + (j - 1) * static_cast<int64_t>(channels), u);
+// Short convolution and silu of N neighbouring channels of one token, in two halves so that all loads go out first.
+template <typename T, int N, int TAPS>
+struct ConvChannels {
+  conv::Window<T, N, TAPS> win;
+  float now[N];
+  __device__ __forceinline__ void load(const b200_conv_args& c, const conv::Row& r, int channel) {
+    conv::load<T, N>(static_cast<const T*>(c.proj) + r.first * c.proj_ld + channel, now);
+    win.load_filter(c, channel);
+    win.load_history(c, r, r.first, channel);
   }
-  if (keep && out >= 0 && n > 0) simt::store_as(dst + (n - 1) * channels, now);
-  return silu(y);
-}
+  __device__ __forceinline__ void finish(const b200_conv_args& c, const conv::Row& r, int channel, bool keep, float (&y)[N]) {
+    win.step(now, y);
+    if (keep) win.store_history(c, r, channel);
+#pragma unroll
+    for (int e = 0; e < N; ++e) y[e] = silu(y[e]);
+  }
+};
 
 // Shared memory: per warp kVecs vectors [DIM], the values (later the outputs) [vpad], kScalars (8 floats); Wkv: lora [rank_pad] too,
 // then W_w2's rows of the head.
-template <typename T, typename Rule, int DIM>
-__global__ void __launch_bounds__(DecodeShape<DIM>::kWarps * 32, DIM <= 64 ? 1 : 2)
-decode_kernel(b200_recurrence_args a, int vpad, int rank_pad, int w2_stride) {
+template <typename T, typename Rule, int DIM, int TAPS>
+__global__ void __launch_bounds__(DecodeShape<DIM>::kWarps * 32, DIM <= 64 ? 2 : DIM <= 128 ? 4 : 2)
+decode_kernel(b200_recurrence_args a, int vpad, int rank_pad, int w2_stride, bool vec_k, bool vec_v) {
   using D = DecodeShape<DIM>;
   constexpr int NI = D::NI, I = D::kI, N = D::kCols, EL = D::kElems, VEC = 16 / sizeof(T);
   extern __shared__ __align__(16) float dyn[];
@@ -232,61 +274,104 @@ decode_kernel(b200_recurrence_args a, int vpad, int rank_pad, int w2_stride) {
   fetch(cur, 0);
   pdl_wait();
   const T* p = static_cast<const T*>(a.proj) + static_cast<int64_t>(min(row, a.num_rows - 1)) * a.proj_ld;
-  fetch(ahead, 1);
   if constexpr (Rule::kKind == B200_RECURRENCE_WKV) {
     const T* lora_in = static_cast<const T*>(a.lora) + static_cast<int64_t>(min(row, a.num_rows - 1)) * a.rank;
-    for (int i = lane; i < a.rank; i += 32) lora[i] = simt::to_f32(lora_in[i]);
     float r[EL], k[EL], z[EL], bonus[EL];
-#pragma unroll
-    for (int e = 0; e < EL; ++e) {
-      const bool ok = lane + e * 32 < dim;
-      const int i = head * dim + min(lane + e * 32, dim - 1);  // clamped: no branches, all loads in flight together
-      const float xr = simt::to_f32(p[a.off_r + i]), xk = simt::to_f32(p[a.off_k + i]);
-      z[e] = simt::to_f32(static_cast<const T*>(a.decay_bias)[i]);
-      bonus[e] = simt::to_f32(static_cast<const T*>(a.bonus)[i]);
-      r[e] = ok ? xr : 0.f;
-      k[e] = ok ? xk : 0.f;
-    }
+    auto fetch_token = [&](auto vec_c) {
+      constexpr bool V = decltype(vec_c)::value;
+      load_channels<V, T, EL>(p + a.off_r + head * dim, lane, dim, r);
+      load_channels<V, T, EL>(p + a.off_k + head * dim, lane, dim, k);
+      load_channels<V, T, EL>(static_cast<const T*>(a.decay_bias) + head * dim, lane, dim, z);
+      load_channels<V, T, EL>(static_cast<const T*>(a.bonus) + head * dim, lane, dim, bonus);
+    };
+    if (vec_k)
+      fetch_token(std::true_type{});
+    else
+      fetch_token(std::false_type{});
+    clear_tail(r, lane, dim);
+    clear_tail(k, lane, dim);
+    for (int i = lane; i < a.rank; i += 32) lora[i] = simt::to_f32(lora_in[i]);
     for (int i = lane; i < vdim; i += 32) values[i] = simt::to_f32(p[a.off_v + head * vdim + i]);
+    fetch(ahead, 1);
     if (w2_stride > 0) asm volatile("cp.async.wait_all;" ::: "memory");
     __syncthreads();  // W_w2's rows (and, within the warp, lora)
     if (w2_stride > 0) {
 #pragma unroll 2
       for (int q = 0; q < a.rank; q += VEC)
 #pragma unroll
-        for (int e = 0; e < EL; ++e) z[e] = delta::dot16(w2_s + min(lane + e * 32, dim - 1) * w2_stride + q, lora + q, z[e]);
+        for (int e = 0; e < EL; ++e) z[e] = delta::dot16(w2_s + min(lane * EL + e, dim - 1) * w2_stride + q, lora + q, z[e]);
     } else {
       const T* w2 = static_cast<const T*>(a.w2) + static_cast<int64_t>(head) * dim * a.rank;
       for (int q = 0; q < a.rank; ++q)
 #pragma unroll
         for (int e = 0; e < EL; ++e)
-          z[e] = fmaf(simt::to_f32(w2[static_cast<int64_t>(min(lane + e * 32, dim - 1)) * a.rank + q]), lora[q], z[e]);
+          z[e] = fmaf(simt::to_f32(w2[static_cast<int64_t>(min(lane * EL + e, dim - 1)) * a.rank + q]), lora[q], z[e]);
     }
     put_wkv<DIM, EL>(vec, scalar, r, k, z, bonus, lane, dim);
   } else {
     if (row < a.num_rows) {
       const int ratio = a.heads / a.kv_heads, kvh = head / ratio;
-      const int channels = 2 * a.kv_heads * dim + a.heads * vdim;
       const bool keep = head == kvh * ratio;  // one head of a group moves the group's query and key state on
-      float q[EL], k[EL];
+      b200_conv_args c{};
+      c.proj = static_cast<const T*>(a.proj) + a.off_r;
+      c.proj_ld = a.proj_ld;
+      c.filter = a.conv_filter;
+      c.state = a.conv_state;
+      c.channels = 2 * a.kv_heads * dim + a.heads * vdim;
+      c.taps = a.taps;
+      const conv::Row cr{row, row + 1, in, out};
+      const int cq = kvh * dim, ck = (a.kv_heads + kvh) * dim, cv = 2 * a.kv_heads * dim + head * vdim;
+      float q1[1][EL], k1[1][EL];
+      float (&q)[EL] = q1[0], (&k)[EL] = k1[0];
 #pragma unroll
-      for (int e = 0; e < EL; ++e) {
-        const int i = lane + e * 32;
-        q[e] = k[e] = 0.f;
+      for (int e = 0; e < EL; ++e) q[e] = k[e] = 0.f;
+      if (vec_k) {
+        const int i = lane * EL;
+        ConvChannels<T, EL, TAPS> wq, wk;
         if (i < dim) {
-          const int cq = kvh * dim + i, ck = (a.kv_heads + kvh) * dim + i;
-          q[e] = conv_channel<T>(a, channels, simt::to_f32(p[a.off_r + cq]), cq, in, out, keep);
-          k[e] = conv_channel<T>(a, channels, simt::to_f32(p[a.off_r + ck]), ck, in, out, keep);
+          wq.load(c, cr, cq + i);
+          wk.load(c, cr, ck + i);
+          wq.finish(c, cr, cq + i, keep, q);
+          wk.finish(c, cr, ck + i, keep, k);
+        }
+      } else {
+#pragma unroll
+        for (int e = 0; e < EL; ++e) {
+          const int i = lane * EL + e;
+          ConvChannels<T, 1, TAPS> wq, wk;
+          float y[1];
+          if (i >= dim) continue;
+          wq.load(c, cr, cq + i);
+          wk.load(c, cr, ck + i);
+          wq.finish(c, cr, cq + i, keep, y);
+          q[e] = y[0];
+          wk.finish(c, cr, ck + i, keep, y);
+          k[e] = y[0];
         }
       }
-      for (int i = lane; i < vdim; i += 32) {
-        const int c = 2 * a.kv_heads * dim + head * vdim + i;
-        values[i] = conv_channel<T>(a, channels, simt::to_f32(p[a.off_r + c]), c, in, out, true);
+      if (vec_v) {
+        for (int i = lane * 4; i < vdim; i += 128) {
+          ConvChannels<T, 4, TAPS> wv;
+          float y[4];
+          wv.load(c, cr, cv + i);
+          wv.finish(c, cr, cv + i, true, y);
+          *reinterpret_cast<float4*>(values + i) = make_float4(y[0], y[1], y[2], y[3]);
+        }
+      } else {
+        for (int i = lane; i < vdim; i += 32) {
+          ConvChannels<T, 1, TAPS> wv;
+          float y[1];
+          wv.load(c, cr, cv + i);
+          wv.finish(c, cr, cv + i, true, y);
+          values[i] = y[0];
+        }
       }
-      put_delta<DIM, EL>(vec, scalar, q, k, lane, dim, a.unit_eps, simt::to_f32(static_cast<const T*>(a.decay_rate)[head]),
-                         simt::to_f32(p[a.off_a + head]) + simt::to_f32(static_cast<const T*>(a.decay_bias)[head]),
-                         simt::to_f32(p[a.off_b + head]));
+      const float x_a[1] = {simt::to_f32(p[a.off_a + head]) + simt::to_f32(static_cast<const T*>(a.decay_bias)[head])};
+      const float x_b[1] = {simt::to_f32(p[a.off_b + head])};
+      put_delta<DIM, EL, 1>(vec, 0, static_cast<int>(scalar - vec), q1, k1, lane, dim, a.unit_eps,
+                            simt::to_f32(static_cast<const T*>(a.decay_rate)[head]), x_a, x_b);
     }
+    fetch(ahead, 1);
   }
   __syncwarp();
   if (row >= a.num_rows) return;
@@ -330,10 +415,10 @@ decode_kernel(b200_recurrence_args a, int vpad, int rank_pad, int w2_stride) {
 // ---------------------------------------------------------------------------------------------------------------
 // Scan
 // ---------------------------------------------------------------------------------------------------------------
-template <typename Rule, int DIM, int COLS, int N>
-struct ScanShape {  // COLS columns per CTA, N of them per thread
-  static constexpr int I = DIM <= 128 ? DIM / 2 : 128;
-  static constexpr int NI = DIM / I;  // lanes of a column: half a warp apart, so that a quarter warp reads one address
+template <typename Rule, int DIM, int COLS, int N, int LANES>
+struct ScanShape {  // COLS columns per CTA, N of them per thread, LANES lanes per column
+  static constexpr int I = DIM / LANES;
+  static constexpr int NI = LANES;  // 32 / NI apart, so that neighbouring lanes read one address
   static constexpr int kStride = 32 / NI;
   static constexpr int kComputeThreads = COLS / N * NI;
   static constexpr int kComputeWarps = kComputeThreads / 32;
@@ -349,10 +434,10 @@ struct ScanShape {  // COLS columns per CTA, N of them per thread
   static_assert(kComputeThreads % 32 == 0 && kScanTokens % kPrepWarps == 0 && kTokPerWarp % kBatch == 0 && COLS % 4 == 0, "");
 };
 
-template <typename T, typename Rule, int DIM, int COLS, int N>
-__global__ void __launch_bounds__(ScanShape<Rule, DIM, COLS, N>::kThreads)
-scan_kernel(b200_recurrence_args a) {
-  using Sh = ScanShape<Rule, DIM, COLS, N>;
+template <typename T, typename Rule, int DIM, int COLS, int N, int LANES, int CTAS>
+__global__ void __launch_bounds__(ScanShape<Rule, DIM, COLS, N, LANES>::kThreads, CTAS)
+scan_kernel(b200_recurrence_args a, bool vec_k) {
+  using Sh = ScanShape<Rule, DIM, COLS, N, LANES>;
   constexpr int NI = Sh::NI, I = Sh::I, EL = Sh::kElems, VL = (COLS + 31) / 32, ST = Sh::kStride;
   extern __shared__ __align__(16) float smem[];
   const int tid = threadIdx.x, lane = tid & 31, dim = a.dim, vdim = a.vdim;
@@ -376,7 +461,7 @@ scan_kernel(b200_recurrence_args a) {
     if constexpr (Rule::kKind == B200_RECURRENCE_WKV) {
 #pragma unroll
       for (int e = 0; e < EL; ++e) {
-        const int i = head * dim + min(lane + e * 32, dim - 1);
+        const int i = head * dim + min(lane * EL + e, dim - 1);
         bias[e] = simt::to_f32(static_cast<const T*>(a.decay_bias)[i]);
         bonus[e] = simt::to_f32(static_cast<const T*>(a.bonus)[i]);
       }
@@ -388,62 +473,75 @@ scan_kernel(b200_recurrence_args a) {
       float* buf = smem + (c & 1) * Sh::kBufFloats;
 #pragma unroll 1
       for (int q0 = 0; q0 < Sh::kTokPerWarp; q0 += Sh::kBatch) {
-        // addresses are clamped, so that the loads need no branches and are all in flight together
-        T xr[Sh::kBatch][EL], xk[Sh::kBatch][EL], xv[Sh::kBatch][VL], xa[Sh::kBatch], xb[Sh::kBatch];
-        float xz[Sh::kBatch][EL];
+        T xv[Sh::kBatch][VL], xa[Sh::kBatch], xb[Sh::kBatch];
+        float xr[Sh::kBatch][EL], xk[Sh::kBatch][EL], xz[Sh::kBatch][EL];
+        auto fetch = [&](auto vec_c) {  // no branches between the loads: all in flight together
+          constexpr bool V = decltype(vec_c)::value;
 #pragma unroll
-        for (int q = 0; q < Sh::kBatch; ++q) {
-          const int64_t t = t_begin + min(c * kScanTokens + warp * Sh::kTokPerWarp + q0 + q, n_tok - 1);
-          const T *r, *k, *v;
-          if constexpr (Rule::kKind == B200_RECURRENCE_WKV) {
-            const T* p = proj + t * a.proj_ld;
-            r = p + a.off_r + head * dim;
-            k = p + a.off_k + head * dim;
-            v = p + a.off_v + head * vdim;
-          } else {
-            const T* p = static_cast<const T*>(a.conv) + t * channels;
-            r = p + kvh * dim;
-            k = p + (a.kv_heads + kvh) * dim;
-            v = p + 2 * a.kv_heads * dim + head * vdim;
-            xa[q] = proj[t * a.proj_ld + a.off_a + head];
-            xb[q] = proj[t * a.proj_ld + a.off_b + head];
+          for (int q = 0; q < Sh::kBatch; ++q) {
+            const int64_t t = t_begin + min(c * kScanTokens + warp * Sh::kTokPerWarp + q0 + q, n_tok - 1);
+            const T *r, *k, *v;
+            if constexpr (Rule::kKind == B200_RECURRENCE_WKV) {
+              const T* p = proj + t * a.proj_ld;
+              r = p + a.off_r + head * dim;
+              k = p + a.off_k + head * dim;
+              v = p + a.off_v + head * vdim;
+              load_channels<V, float, EL>(a.z + t * hd + head * dim, lane, dim, xz[q]);
+            } else {
+              const T* p = static_cast<const T*>(a.conv) + t * channels;
+              r = p + kvh * dim;
+              k = p + (a.kv_heads + kvh) * dim;
+              v = p + 2 * a.kv_heads * dim + head * vdim;
+              xa[q] = proj[t * a.proj_ld + a.off_a + head];
+              xb[q] = proj[t * a.proj_ld + a.off_b + head];
+            }
+            load_channels<V, T, EL>(r, lane, dim, xr[q]);
+            load_channels<V, T, EL>(k, lane, dim, xk[q]);
+#pragma unroll
+            for (int e = 0; e < VL; ++e) xv[q][e] = v[min(cb * COLS + lane + e * 32, vdim - 1)];
           }
-#pragma unroll
-          for (int e = 0; e < EL; ++e) {
-            const int i = min(lane + e * 32, dim - 1);
-            xr[q][e] = r[i];
-            xk[q][e] = k[i];
-            if constexpr (Rule::kKind == B200_RECURRENCE_WKV) xz[q][e] = a.z[t * hd + head * dim + i];
-          }
-#pragma unroll
-          for (int e = 0; e < VL; ++e) xv[q][e] = v[min(cb * COLS + lane + e * 32, vdim - 1)];
           if constexpr (Rule::kKind == B200_RECURRENCE_WKV) {
             for (int s = 1; s < a.z_splits; ++s)
 #pragma unroll
-              for (int e = 0; e < EL; ++e) xz[q][e] += a.z[(static_cast<int64_t>(s) * a.num_tokens + t) * hd + head * dim + min(lane + e * 32, dim - 1)];
+              for (int q = 0; q < Sh::kBatch; ++q) {
+                const int64_t t = t_begin + min(c * kScanTokens + warp * Sh::kTokPerWarp + q0 + q, n_tok - 1);
+                float more[EL];
+                load_channels<V, float, EL>(a.z + (static_cast<int64_t>(s) * a.num_tokens + t) * hd + head * dim, lane, dim, more);
+#pragma unroll
+                for (int e = 0; e < EL; ++e) xz[q][e] += more[e];
+              }
           }
-        }
+        };
+        if (vec_k)
+          fetch(std::true_type{});
+        else
+          fetch(std::false_type{});
+        float* vec = buf + (warp * Sh::kTokPerWarp + q0) * Sh::kTokenFloats;
 #pragma unroll
         for (int q = 0; q < Sh::kBatch; ++q) {
-          float* vec = buf + (warp * Sh::kTokPerWarp + q0 + q) * Sh::kTokenFloats;
-          float* values = vec + Rule::kVecs * DIM;
-          float r[EL], k[EL];
+          clear_tail(xr[q], lane, dim);
+          clear_tail(xk[q], lane, dim);
 #pragma unroll
-          for (int e = 0; e < EL; ++e) {
-            r[e] = lane + e * 32 < dim ? simt::to_f32(xr[q][e]) : 0.f;
-            k[e] = lane + e * 32 < dim ? simt::to_f32(xk[q][e]) : 0.f;
-          }
-          if constexpr (Rule::kKind == B200_RECURRENCE_WKV) {
+          for (int e = 0; e < VL; ++e)
+            if (lane + e * 32 < COLS) vec[q * Sh::kTokenFloats + Rule::kVecs * DIM + lane + e * 32] = simt::to_f32(xv[q][e]);
+        }
+        if constexpr (Rule::kKind == B200_RECURRENCE_WKV) {
+#pragma unroll
+          for (int q = 0; q < Sh::kBatch; ++q) {
             float z[EL];
 #pragma unroll
             for (int e = 0; e < EL; ++e) z[e] = xz[q][e] + bias[e];
-            put_wkv<DIM, EL>(vec, values + COLS, r, k, z, bonus, lane, dim);
-          } else {
-            put_delta<DIM, EL>(vec, values + COLS, r, k, lane, dim, a.unit_eps, decay_rate, simt::to_f32(xa[q]) + decay_bias, simt::to_f32(xb[q]));
+            float* at = vec + q * Sh::kTokenFloats;
+            put_wkv<DIM, EL>(at, at + Rule::kVecs * DIM + COLS, xr[q], xk[q], z, bonus, lane, dim);
           }
+        } else {
+          float fa[Sh::kBatch], fb[Sh::kBatch];
 #pragma unroll
-          for (int e = 0; e < VL; ++e)
-            if (lane + e * 32 < COLS) values[lane + e * 32] = simt::to_f32(xv[q][e]);
+          for (int q = 0; q < Sh::kBatch; ++q) {
+            fa[q] = simt::to_f32(xa[q]) + decay_bias;
+            fb[q] = simt::to_f32(xb[q]);
+          }
+          put_delta<DIM, EL, Sh::kBatch>(vec, Sh::kTokenFloats, Rule::kVecs * DIM + COLS, xr, xk, lane, dim, a.unit_eps, decay_rate, fa, fb);
         }
       }
       __syncthreads();  // chunk c is ready, chunk c - 1 has been read: its buffer is free
@@ -497,49 +595,47 @@ scan_kernel(b200_recurrence_args a) {
   }
 }
 
-// A warp per (token, head), four of them in turn with all their loads in flight.
+// LPH lanes of 4 channels per (token, head), kFinishUnits units in turn with all their loads in flight (LPH == 0: a warp, any size).
 constexpr int kFinishUnits = 4;
-template <typename T>
+template <typename T, int LPH>
 __global__ void __launch_bounds__(256)
 finish_kernel(b200_recurrence_args a) {
   pdl_launch_dependents();
   pdl_wait();
-  const int lane = threadIdx.x & 31, dim = a.vdim;
+  const int dim = a.vdim;
   const uint32_t total = static_cast<uint32_t>(a.num_tokens) * a.heads, heads = a.heads;  // (the launch checks that it fits)
-  const uint32_t first = (blockIdx.x * 8 + (threadIdx.x >> 5)) * kFinishUnits;
   const T* proj = static_cast<const T*>(a.proj);
   const T* weight = static_cast<const T*>(a.norm_weight);
   T* out = static_cast<T*>(a.out);
-  constexpr int E = 4;
-  if (dim <= 32 * E) {  // heads in registers
-    float v[kFinishUnits][E], w[kFinishUnits][E];
-    T g[kFinishUnits][E];
+  if constexpr (LPH > 0) {
+    constexpr int kGroups = 256 / LPH;
+    const int lane = threadIdx.x % LPH, i = min(lane * 4, dim - 4);
+    const uint32_t first = blockIdx.x * kGroups * kFinishUnits + threadIdx.x / LPH;  // then kGroups apart
+    float v[kFinishUnits][4], g[kFinishUnits][4], w[kFinishUnits][4];
 #pragma unroll
     for (int k = 0; k < kFinishUnits; ++k) {
-      const uint32_t unit = min(first + k, total - 1), t = unit / heads;
+      const uint32_t unit = min(first + k * kGroups, total - 1), t = unit / heads;
       const int at = static_cast<int>(unit - t * heads) * dim;
-#pragma unroll
-      for (int e = 0; e < E; ++e) {
-        if (e * 32 >= dim) break;
-        const int i = min(lane + e * 32, dim - 1);
-        v[k][e] = a.o_f32[static_cast<int64_t>(unit) * dim + i];
-        g[k][e] = proj[t * a.proj_ld + a.off_g + at + i];
-        w[k][e] = simt::to_f32(weight[(a.norm_per_head ? at : 0) + i]);
-      }
+      conv::load<float, 4>(a.o_f32 + static_cast<int64_t>(unit) * dim + i, v[k]);
+      conv::load<T, 4>(proj + t * a.proj_ld + a.off_g + at + i, g[k]);
+      conv::load<T, 4>(weight + (a.norm_per_head ? at : 0) + i, w[k]);
     }
 #pragma unroll
     for (int k = 0; k < kFinishUnits; ++k) {
-      float sq = 0.f;
+      float sq = lane * 4 < dim ? v[k][0] * v[k][0] + v[k][1] * v[k][1] + v[k][2] * v[k][2] + v[k][3] * v[k][3] : 0.f;
 #pragma unroll
-      for (int e = 0; e < E; ++e) sq += lane + e * 32 < dim ? v[k][e] * v[k][e] : 0.f;
-      const float inv = 1.f / sqrtf(warp_sum(sq) / dim + a.eps);
+      for (int o = LPH / 2; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
+      const float inv = 1.f / sqrtf(sq / dim + a.eps);
+      float y[4];
 #pragma unroll
-      for (int e = 0; e < E; ++e)
-        if (lane + e * 32 < dim && first + k < total)
-          simt::store_as(out + static_cast<int64_t>(first + k) * dim + lane + e * 32, v[k][e] * inv * w[k][e] * silu(simt::to_f32(g[k][e])));
+      for (int e = 0; e < 4; ++e) y[e] = v[k][e] * inv * w[k][e] * silu(g[k][e]);
+      const uint32_t unit = first + k * kGroups;
+      if (lane * 4 < dim && unit < total) conv::store<T, 4>(out + static_cast<int64_t>(unit) * dim + i, y);
     }
     return;
   }
+  const int lane = threadIdx.x & 31;
+  const uint32_t first = (blockIdx.x * 8 + (threadIdx.x >> 5)) * kFinishUnits;
   for (int k = 0; k < kFinishUnits; ++k) {
     const int64_t unit = first + k;
     if (unit >= total) return;
@@ -595,10 +691,26 @@ static int launch_decode(const b200_recurrence_args& a, cudaStream_t s) {
   }
   const size_t bytes = static_cast<size_t>(D::kWarps) * (Rule::kVecs * DIM + vpad + 8 + rank_pad) * 4 + w2_bytes;
   if (bytes > 200 * 1024) return B200_ERR_INVALID_ARGUMENT;
-  static std::atomic<uint64_t> done{0};
-  if (ensure_dynamic_smem(decode_kernel<T, Rule, DIM>, 200 * 1024, done) != B200_OK) return B200_ERR_LAUNCH;
-  return launch_pdl(decode_kernel<T, Rule, DIM>, dim3(a.heads, (a.num_rows + D::kWarps - 1) / D::kWarps), dim3(D::kWarps * 32), bytes, s,
-                    a, vpad, rank_pad, w2_stride);
+  // Whole vectors of EL query / key channels and of 4 value channels: rows of proj, of the filter and of the convolution's state.
+  constexpr int EL = D::kElems;
+  const int channels = 2 * a.kv_heads * a.dim + a.heads * a.vdim;
+  bool vec_k = a.dim % EL == 0 && a.proj_ld % 8 == 0 && aligned16(a.proj) && a.off_r % 8 == 0 && a.off_k % 8 == 0;
+  if (Rule::kKind == B200_RECURRENCE_WKV)
+    vec_k = vec_k && aligned16(a.decay_bias) && aligned16(a.bonus);
+  else
+    vec_k = vec_k && aligned16(a.conv_filter) && aligned16(a.conv_state);
+  const bool vec_v = vec_k && a.vdim % 4 == 0 && a.dim % 4 == 0;  // (then channels % 4 == 0)
+  if (Rule::kKind == B200_RECURRENCE_DELTA) vec_k = vec_k && channels % EL == 0;
+  auto go = [&](auto taps) {
+    constexpr int TAPS = decltype(taps)::value;
+    static std::atomic<uint64_t> done{0};
+    if (ensure_dynamic_smem(decode_kernel<T, Rule, DIM, TAPS>, 200 * 1024, done) != B200_OK) return static_cast<int>(B200_ERR_LAUNCH);
+    return launch_pdl(decode_kernel<T, Rule, DIM, TAPS>, dim3(a.heads, (a.num_rows + D::kWarps - 1) / D::kWarps), dim3(D::kWarps * 32), bytes,
+                      s, a, vpad, rank_pad, w2_stride, vec_k, vec_v);
+  };
+  if constexpr (Rule::kKind == B200_RECURRENCE_DELTA)
+    if (a.taps > 4) return go(std::integral_constant<int, 8>{});
+  return go(std::integral_constant<int, 4>{});
 }
 template <typename T, typename Rule>
 static int decode_by_dim(const b200_recurrence_args& a, cudaStream_t s) {
@@ -607,23 +719,32 @@ static int decode_by_dim(const b200_recurrence_args& a, cudaStream_t s) {
   if (a.dim <= 128) return launch_decode<T, Rule, 128>(a, s);
   return launch_decode<T, Rule, 256>(a, s);
 }
-template <typename T, typename Rule, int DIM, int COLS, int N>
+template <typename T, typename Rule, int DIM, int COLS, int N, int LANES, int CTAS>
 static int launch_scan(const b200_recurrence_args& a, cudaStream_t s) {
-  using Sh = ScanShape<Rule, DIM, COLS, N>;
+  using Sh = ScanShape<Rule, DIM, COLS, N, LANES>;
   static std::atomic<uint64_t> done{0};
-  if (ensure_dynamic_smem(scan_kernel<T, Rule, DIM, COLS, N>, Sh::kSmemBytes, done) != B200_OK) return B200_ERR_LAUNCH;
+  if (ensure_dynamic_smem(scan_kernel<T, Rule, DIM, COLS, N, LANES, CTAS>, Sh::kSmemBytes, done) != B200_OK) return B200_ERR_LAUNCH;
   const int col_blocks = (a.vdim + COLS - 1) / COLS;
+  constexpr int EL = Sh::kElems;
+  bool vec_k = a.dim % EL == 0 && a.proj_ld % 8 == 0 && aligned16(a.proj) && a.off_r % 8 == 0 && a.off_k % 8 == 0 && aligned16(a.conv) && aligned16(a.z);
+  if (Rule::kKind == B200_RECURRENCE_DELTA) vec_k = vec_k && (2 * a.kv_heads * a.dim + a.heads * a.vdim) % EL == 0;
   // Not a programmatic launch: CTAs that arrive while the previous kernel still holds most SMs would pile up on the others,
   // and a CTA stays where it is for the length of a prompt.
-  scan_kernel<T, Rule, DIM, COLS, N><<<dim3(a.heads * col_blocks, a.num_rows), Sh::kThreads, Sh::kSmemBytes, s>>>(a);
+  scan_kernel<T, Rule, DIM, COLS, N, LANES, CTAS><<<dim3(a.heads * col_blocks, a.num_rows), Sh::kThreads, Sh::kSmemBytes, s>>>(a, vec_k);
   return launch_status();
 }
 template <typename T, typename Rule>
 static int scan_by_dim(const b200_recurrence_args& a, cudaStream_t s) {
-  if (a.dim <= 32) return launch_scan<T, Rule, 32, 32, 1>(a, s);
-  if (a.dim <= 64) return launch_scan<T, Rule, 64, 64, 1>(a, s);
-  if (a.dim <= 128) return launch_scan<T, Rule, 128, 64, 1>(a, s);
-  return launch_scan<T, Rule, 256, 32, 1>(a, s);
+  if (a.dim <= 32) return launch_scan<T, Rule, 32, 32, 1, 2, 1>(a, s);
+  if constexpr (Rule::kKind == B200_RECURRENCE_WKV) {
+    if (a.dim <= 64) return launch_scan<T, Rule, 64, 64, 1, 2, 2>(a, s);
+    // Two columns per thread on twice the lanes: half the shared-memory reads per product, the same state per thread.
+    if (a.dim <= 128) return launch_scan<T, Rule, 128, 64, 2, 4, 2>(a, s);
+  } else {
+    if (a.dim <= 64) return launch_scan<T, Rule, 64, 64, 1, 4, 1>(a, s);
+    if (a.dim <= 128) return launch_scan<T, Rule, 128, 64, 1, 2, 1>(a, s);
+  }
+  return launch_scan<T, Rule, 256, 32, 1, 2, 1>(a, s);
 }
 template <typename T>
 static int decode_by_kind(const b200_recurrence_args& a, cudaStream_t s) {
@@ -663,10 +784,20 @@ int b200_recurrence_finish(const b200_recurrence_args* a, b200_stream_t stream) 
   using namespace b200;
   if (!rec::valid(a) || !a->proj || !a->o_f32 || !a->norm_weight || !a->out || static_cast<int64_t>(a->num_tokens) * a->heads > (1u << 30))
     return B200_ERR_INVALID_ARGUMENT;
-  const unsigned blocks = static_cast<unsigned>((static_cast<int64_t>(a->num_tokens) * a->heads + 8 * rec::kFinishUnits - 1) / (8 * rec::kFinishUnits));
+  const int64_t units = static_cast<int64_t>(a->num_tokens) * a->heads;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  if (a->dtype == B200_DTYPE_F32) return launch_pdl(rec::finish_kernel<float>, dim3(blocks), dim3(256), 0, s, *a);
-  return launch_pdl(rec::finish_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, s, *a);
+  const bool vec = a->vdim % 4 == 0 && a->vdim <= 128 && a->proj_ld % 4 == 0 && a->off_g % 4 == 0 && aligned16(a->proj) && aligned16(a->o_f32) &&
+                   aligned16(a->norm_weight) && aligned16(a->out);
+  const int lanes = !vec ? 0 : a->vdim <= 64 ? 16 : 32;
+  const int per_block = (lanes ? 256 / lanes : 8) * rec::kFinishUnits;
+  const dim3 grid(static_cast<unsigned>((units + per_block - 1) / per_block));
+  auto go = [&](auto zero) {
+    using T = decltype(zero);
+    if (lanes == 16) return launch_pdl(rec::finish_kernel<T, 16>, grid, dim3(256), 0, s, *a);
+    if (lanes == 32) return launch_pdl(rec::finish_kernel<T, 32>, grid, dim3(256), 0, s, *a);
+    return launch_pdl(rec::finish_kernel<T, 0>, grid, dim3(256), 0, s, *a);
+  };
+  return a->dtype == B200_DTYPE_F32 ? go(0.f) : go(__nv_bfloat16{});
 }
 
 int b200_recurrence_lora(const b200_recurrence_args* a, b200_stream_t stream) {

@@ -66,6 +66,7 @@ residual_norm_kernel(b200_residual_norm_args a) {
     for (int e = 0; e < VEC; ++e) add[e] = 0.f;
     if (a.partials != nullptr) {
       const int64_t stride = static_cast<int64_t>(a.source_rows) * W;
+#pragma unroll 4
       for (int s = 0; s < a.num_splits; ++s) {
         load<float, VEC>(a.partials + s * stride + row * W + c, x);
 #pragma unroll
@@ -78,12 +79,19 @@ residual_norm_kernel(b200_residual_norm_args a) {
       for (int e = 0; e < VEC; ++e) add[e] += x[e];
     }
     if (a.expert_rows != nullptr) {
-      for (int k = 0; k < a.top; ++k) {
-        const int64_t at = expert_row[k];
-        if (at < 0) continue;
-        load<T, VEC>(static_cast<const T*>(a.expert_rows) + at * W + c, x);
+      for (int k = 0; k < a.top; k += 4) {  // four rows in flight (a row that is missing counts nothing)
+        float rows[4][VEC];
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) add[e] += x[e];
+        for (int j = 0; j < 4; ++j) {
+          const int64_t at = expert_row[min(k + j, a.top - 1)];
+          load<T, VEC>(static_cast<const T*>(a.expert_rows) + (at < 0 ? 0 : at) * W + c, rows[j]);
+        }
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+          if (k + j < a.top && expert_row[min(k + j, a.top - 1)] >= 0) {
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) add[e] += rows[j][e];
+          }
       }
     }
     if (a.shared_rows != nullptr) {

@@ -4,7 +4,7 @@
 // last taps - 1 inputs, or the last row), read from one buffer of its slot and written to the other.
 //
 //   conv_silu_kernel    16 bytes of channels per thread, a run of tokens, the filter and the last inputs in registers
-//   conv_qkv_kernel     a warp per (head, run of tokens): convolution, then the per-head RMS norm of queries and keys or the
+//   conv_qkv_kernel     some lanes per (head, run of tokens): convolution, then the per-head RMS norm of queries and keys or the
 //                       value mixing, then the stores (queries, pool rows, first values)
 //   token_shift_kernel  16 bytes of a row per thread, a run of tokens, every mix from the two rows in registers
 #include "common.cuh"
@@ -78,6 +78,16 @@ __device__ __forceinline__ void store(T* p, const float (&v)[VEC]) {
   }
 }
 
+// VEC elements as they lie in memory (half the registers of their fp32 values).
+template <typename T, int VEC>
+struct alignas(sizeof(T) * VEC) Raw {
+  T e[VEC];
+  __device__ __forceinline__ void to(float (&v)[VEC]) const {
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] = simt::to_f32(e[i]);
+  }
+};
+
 // The filter and the last TAPS - 1 inputs of VEC neighbouring channels.  Filters shorter than TAPS have leading zeros.
 template <typename T, int VEC, int TAPS>
 struct Window {
@@ -145,102 +155,131 @@ conv_silu_kernel(b200_conv_args a, int run) {
   if (c < a.channels) win.load_filter(a, c);
   pdl_wait();
   if (c >= a.channels) return;
+  constexpr int B = 4;  // tokens whose loads are in flight together
   Row r{0, -1, -1, -1};
-  for (int t = t0; t < t1; ++t) {
-    if (t >= r.end) {
-      r = row_of(a, t);
-      win.load_history(a, r, t, c);
-    }
-    float now[VEC], y[VEC];
-    load<T, VEC>(static_cast<const T*>(a.proj) + t * a.proj_ld + c, now);
-    win.step(now, y);
-    if (t == r.end - 1) win.store_history(a, r, c);
+  for (int tb = t0; tb < t1; tb += B) {
+    Raw<T, VEC> now[B];
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) y[e] = y[e] / (1.f + expf(-y[e]));
-    store<T, VEC>(static_cast<T*>(a.out) + static_cast<int64_t>(t) * a.channels + c, y);
+    for (int q = 0; q < B; ++q) now[q] = *reinterpret_cast<const Raw<T, VEC>*>(static_cast<const T*>(a.proj) + min(tb + q, t1 - 1) * a.proj_ld + c);
+#pragma unroll
+    for (int q = 0; q < B; ++q) {
+      const int t = tb + q;
+      if (t >= t1) break;
+      if (t >= r.end) {
+        r = row_of(a, t);
+        win.load_history(a, r, t, c);
+      }
+      float x[VEC], y[VEC];
+      now[q].to(x);
+      win.step(x, y);
+      if (t == r.end - 1) win.store_history(a, r, c);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) y[e] = y[e] / (1.f + expf(-y[e]));
+      store<T, VEC>(static_cast<T*>(a.out) + static_cast<int64_t>(t) * a.channels + c, y);
+    }
   }
 }
 
-template <typename T, int VEC, int EL, int TAPS>
+// LPH lanes per head, VEC * EL channels each; a warp holds 32 / LPH (head, run) units.
+template <typename T, int VEC, int EL, int LPH, int TAPS>
 __global__ void __launch_bounds__(kThreads)
 conv_qkv_kernel(b200_conv_args a, int run) {
+  constexpr int B = EL == 1 && TAPS == 4 ? 4 : 1;  // tokens whose loads are in flight together
+  using V = Raw<T, VEC>;
   pdl_launch_dependents();
-  const int lane = threadIdx.x & 31;
-  const int heads = a.heads + 2 * a.kv_heads;
-  const int unit = blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5);
-  const int runs = (a.num_tokens + run - 1) / run;
-  if (unit >= heads * runs) {
-    pdl_wait();
-    return;
-  }
-  const int hh = unit % heads, t0 = unit / heads * run, t1 = min(t0 + run, a.num_tokens);
+  const int lane = threadIdx.x % LPH;
+  const int heads = a.heads + 2 * a.kv_heads, runs = (a.num_tokens + run - 1) / run;
+  const int unit_raw = (blockIdx.x * kThreads + threadIdx.x) / LPH;
+  const bool active = unit_raw < heads * runs;
+  const int unit = active ? unit_raw : 0;  // (lanes without a unit take part in the sums only)
+  const int hh = unit % heads, t0 = unit / heads * run;
   const int kind = hh < a.heads ? 0 : hh < a.heads + a.kv_heads ? 1 : 2;  // query, key, value
   const int g = kind == 0 ? hh : kind == 1 ? hh - a.heads : hh - a.heads - a.kv_heads;
   const int d = kind == 2 ? a.vdim : a.dim;
   const int c0 = kind == 2 ? (a.heads + a.kv_heads) * a.dim + g * a.vdim : hh * a.dim;
   Window<T, VEC, TAPS> win[EL];
-  float weight[EL][VEC];
+  V weight[EL];
 #pragma unroll
   for (int e = 0; e < EL; ++e) {
-    const int i = (e * 32 + lane) * VEC;
+    const int i = (e * LPH + lane) * VEC;
     if (i >= d) continue;
     win[e].load_filter(a, c0 + i);
-    if (kind != 2) load<T, VEC>(static_cast<const T*>(kind == 0 ? a.q_norm : a.k_norm) + i, weight[e]);
+    if (kind != 2) weight[e] = *reinterpret_cast<const V*>(static_cast<const T*>(kind == 0 ? a.q_norm : a.k_norm) + i);
   }
   const float mix = kind == 2 && a.v_first_in != nullptr ? simt::to_f32(*static_cast<const T*>(a.mix)) : 0.f;
+  const int64_t pool_tokens = static_cast<int64_t>(a.num_chunks) * a.chunk_size;
   pdl_wait();
   Row r{0, -1, -1, -1};
-  for (int t = t0; t < t1; ++t) {
-    if (t >= r.end) {
-      r = row_of(a, t);
+  for (int tb = 0; tb < run; tb += B) {
+    V now[B][EL], first[B][EL];
+    int64_t token[B];
+#pragma unroll
+    for (int q = 0; q < B; ++q) {
+      const int t = min(t0 + tb + q, a.num_tokens - 1);
+      token[q] = kind == 0 ? 0 : a.chunk_idx[t] * a.chunk_size + a.local_pos[t];
+#pragma unroll
+      for (int e = 0; e < EL; ++e) {
+        const int i = (e * LPH + lane) * VEC;
+        if (i >= d) continue;
+        now[q][e] = *reinterpret_cast<const V*>(static_cast<const T*>(a.proj) + t * a.proj_ld + c0 + i);
+        if (kind == 2 && a.v_first_in != nullptr)
+          first[q][e] = *reinterpret_cast<const V*>(static_cast<const T*>(a.v_first_in) + (static_cast<int64_t>(t) * a.kv_heads + g) * d + i);
+      }
+    }
+#pragma unroll
+    for (int q = 0; q < B; ++q) {
+      const int t = t0 + tb + q;
+      const bool on = active && tb + q < run && t < a.num_tokens;
+      if (on && t >= r.end) {
+        r = row_of(a, t);
+#pragma unroll
+        for (int e = 0; e < EL; ++e)
+          if ((e * LPH + lane) * VEC < d) win[e].load_history(a, r, t, c0 + (e * LPH + lane) * VEC);
+      }
+      float y[EL][VEC], sq = 0.f;
+#pragma unroll
+      for (int e = 0; e < EL; ++e) {
+        const int i = (e * LPH + lane) * VEC;
+        if (!on || i >= d) continue;
+        float x[VEC];
+        now[q][e].to(x);
+        win[e].step(x, y[e]);
+        if (t == r.end - 1) win[e].store_history(a, r, c0 + i);
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) sq = fmaf(y[e][k], y[e][k], sq);
+      }
+#pragma unroll
+      for (int o = LPH / 2; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
+      if (!on) continue;
+      T* dst;
+      if (kind != 2) {
+        const float inv = 1.f / sqrtf(sq / d + a.eps);
+#pragma unroll
+        for (int e = 0; e < EL; ++e) {
+          if ((e * LPH + lane) * VEC >= d) continue;
+#pragma unroll
+          for (int k = 0; k < VEC; ++k) y[e][k] *= inv * simt::to_f32(weight[e].e[k]);
+        }
+        dst = kind == 0 ? static_cast<T*>(a.out) + (static_cast<int64_t>(t) * a.heads + g) * d
+                        : static_cast<T*>(a.k_pool) + token[q] * a.pool_row_elems + g * d;
+      } else {
+#pragma unroll
+        for (int e = 0; e < EL; ++e) {
+          const int i = (e * LPH + lane) * VEC;
+          if (i >= d) continue;
+          if (a.v_first_out != nullptr) store<T, VEC>(static_cast<T*>(a.v_first_out) + (static_cast<int64_t>(t) * a.kv_heads + g) * d + i, y[e]);
+          if (a.v_first_in != nullptr) {
+#pragma unroll
+            for (int k = 0; k < VEC; ++k) y[e][k] = fmaf(mix, simt::to_f32(first[q][e].e[k]), (1.f - mix) * y[e][k]);
+          }
+        }
+        dst = static_cast<T*>(a.v_pool) + token[q] * a.pool_row_elems + g * d;
+      }
+      if (token[q] < 0 || token[q] >= pool_tokens) continue;
 #pragma unroll
       for (int e = 0; e < EL; ++e)
-        if ((e * 32 + lane) * VEC < d) win[e].load_history(a, r, t, c0 + (e * 32 + lane) * VEC);
+        if ((e * LPH + lane) * VEC < d) store<T, VEC>(dst + (e * LPH + lane) * VEC, y[e]);
     }
-    float y[EL][VEC], sq = 0.f;
-#pragma unroll
-    for (int e = 0; e < EL; ++e) {
-      const int i = (e * 32 + lane) * VEC;
-      if (i >= d) continue;
-      float now[VEC];
-      load<T, VEC>(static_cast<const T*>(a.proj) + t * a.proj_ld + c0 + i, now);
-      win[e].step(now, y[e]);
-      if (t == r.end - 1) win[e].store_history(a, r, c0 + i);
-#pragma unroll
-      for (int k = 0; k < VEC; ++k) sq = fmaf(y[e][k], y[e][k], sq);
-    }
-    const int64_t token = a.chunk_idx[t] * a.chunk_size + a.local_pos[t];
-    T* dst;
-    if (kind != 2) {
-      const float inv = 1.f / sqrtf(warp_sum(sq) / d + a.eps);
-#pragma unroll
-      for (int e = 0; e < EL; ++e) {
-        if ((e * 32 + lane) * VEC >= d) continue;
-#pragma unroll
-        for (int k = 0; k < VEC; ++k) y[e][k] *= inv * weight[e][k];
-      }
-      dst = kind == 0 ? static_cast<T*>(a.out) + (static_cast<int64_t>(t) * a.heads + g) * d
-                      : static_cast<T*>(a.k_pool) + token * a.pool_row_elems + g * d;
-    } else {
-      const int64_t at = (static_cast<int64_t>(t) * a.kv_heads + g) * d;
-#pragma unroll
-      for (int e = 0; e < EL; ++e) {
-        const int i = (e * 32 + lane) * VEC;
-        if (i >= d) continue;
-        if (a.v_first_out != nullptr) store<T, VEC>(static_cast<T*>(a.v_first_out) + at + i, y[e]);
-        if (a.v_first_in != nullptr) {
-          float first[VEC];
-          load<T, VEC>(static_cast<const T*>(a.v_first_in) + at + i, first);
-#pragma unroll
-          for (int k = 0; k < VEC; ++k) y[e][k] = fmaf(mix, first[k], (1.f - mix) * y[e][k]);
-        }
-      }
-      dst = static_cast<T*>(a.v_pool) + token * a.pool_row_elems + g * d;
-    }
-    if (kind != 0 && static_cast<uint64_t>(token) >= static_cast<uint64_t>(a.num_chunks) * a.chunk_size) continue;
-#pragma unroll
-    for (int e = 0; e < EL; ++e)
-      if ((e * 32 + lane) * VEC < d) store<T, VEC>(dst + (e * 32 + lane) * VEC, y[e]);
   }
 }
 
@@ -313,29 +352,29 @@ static int silu(const b200_conv_args& a, cudaStream_t s) {
   return vec ? launch_silu<T, VEC, 8>(a, s) : launch_silu<T, 1, 8>(a, s);
 }
 
-template <typename T, int VEC, int EL, int TAPS>
+template <typename T, int VEC, int EL, int LPH, int TAPS>
 static int launch_qkv(const b200_conv_args& a, cudaStream_t s) {
   const int heads = a.heads + 2 * a.kv_heads;
-  const int run = run_length(a, heads);
-  const int64_t units = static_cast<int64_t>(heads) * ((a.num_tokens + run - 1) / run);
-  if (units > 0x3fffffff) return B200_ERR_INVALID_ARGUMENT;
-  return launch_pdl(conv_qkv_kernel<T, VEC, EL, TAPS>, dim3(static_cast<unsigned>((units + 3) / 4)), dim3(kThreads), 0, s, a, run);
+  const int run = run_length(a, static_cast<int64_t>(heads) * LPH / 32 + 1);
+  const int64_t threads = static_cast<int64_t>(heads) * ((a.num_tokens + run - 1) / run) * LPH;
+  if (threads > 0x3fffffff) return B200_ERR_INVALID_ARGUMENT;
+  return launch_pdl(conv_qkv_kernel<T, VEC, EL, LPH, TAPS>, dim3(static_cast<unsigned>((threads + kThreads - 1) / kThreads)), dim3(kThreads), 0,
+                    s, a, run);
 }
 template <typename T, int TAPS>
 static int qkv(const b200_conv_args& a, cudaStream_t s) {
   const int widest = a.dim > a.vdim ? a.dim : a.vdim;
-  auto fits = [&](int vec) {
-    bool ok = a.dim % vec == 0 && a.vdim % vec == 0 && a.proj_ld % vec == 0 && a.pool_row_elems % vec == 0;
-    for (const void* p : {a.proj, a.filter, static_cast<const void*>(a.state), static_cast<const void*>(a.out), a.q_norm, a.k_norm,
-                          static_cast<const void*>(a.k_pool), static_cast<const void*>(a.v_pool), a.v_first_in,
-                          static_cast<const void*>(a.v_first_out)})
-      ok = ok && reinterpret_cast<uintptr_t>(p) % (vec * sizeof(T)) == 0;
-    return ok;
-  };
-  if (widest <= 64 && fits(2)) return launch_qkv<T, 2, 1, TAPS>(a, s);
-  if (widest <= 128 && fits(4)) return launch_qkv<T, 4, 1, TAPS>(a, s);
-  if (fits(4)) return launch_qkv<T, 4, 2, TAPS>(a, s);
-  return launch_qkv<T, 1, 8, TAPS>(a, s);
+  constexpr int VEC = 4;
+  bool vec = a.dim % VEC == 0 && a.vdim % VEC == 0 && a.proj_ld % VEC == 0 && a.pool_row_elems % VEC == 0;
+  for (const void* p : {a.proj, a.filter, static_cast<const void*>(a.state), static_cast<const void*>(a.out), a.q_norm, a.k_norm,
+                        static_cast<const void*>(a.k_pool), static_cast<const void*>(a.v_pool), a.v_first_in,
+                        static_cast<const void*>(a.v_first_out)})
+    vec = vec && reinterpret_cast<uintptr_t>(p) % (VEC * sizeof(T)) == 0;
+  if (!vec) return launch_qkv<T, 1, 8, 32, TAPS>(a, s);
+  if (widest <= 8 * VEC) return launch_qkv<T, VEC, 1, 8, TAPS>(a, s);
+  if (widest <= 16 * VEC) return launch_qkv<T, VEC, 1, 16, TAPS>(a, s);
+  if (widest <= 32 * VEC) return launch_qkv<T, VEC, 1, 32, TAPS>(a, s);
+  return launch_qkv<T, VEC, 2, 32, TAPS>(a, s);
 }
 
 template <typename T>

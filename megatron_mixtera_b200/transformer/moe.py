@@ -10,19 +10,19 @@ from .hybrid_config import HybridConfig, MoeConfig
 
 
 def _padded(ff: int) -> int:
-    """Whole blocks of 64 features: a 128-row tile of the up weights holds 64 gate rows and the matching up rows."""
+    """Whole blocks of 64 features: a 128-row tile of the up weights holds 64 gate rows and the matching up rows (16 in turn)."""
     return -(-ff // 64) * 64
 
 
 def interleave_up(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
-    """[ff, H] each -> [2 * padded ff, H], blocks of 64 gate rows and 64 up rows, missing rows zero."""
+    """[ff, H] each -> [2 * padded ff, H], blocks of 16 gate rows and 16 up rows, missing rows zero."""
     ff, H = gate.shape
     pad = _padded(ff)
-    out = torch.zeros((pad // 64, 2, 64, H), dtype=gate.dtype, device=gate.device)
+    out = torch.zeros((pad // 16, 2, 16, H), dtype=gate.dtype, device=gate.device)
     for i, w in enumerate((gate, up)):
         full = torch.zeros((pad, H), dtype=gate.dtype, device=gate.device)
         full[:ff] = w
-        out[:, i] = full.view(pad // 64, 64, H)
+        out[:, i] = full.view(pad // 16, 16, H)
     return out.view(2 * pad, H)
 
 

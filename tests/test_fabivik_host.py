@@ -65,15 +65,15 @@ def test_unknown_parts_are_refused():
 
 
 def test_expert_weight_layout():
-    """Blocks of 64 gate rows and the 64 matching up rows, padded with zero rows; down columns of the padding are zero."""
+    """Blocks of 16 gate rows and the 16 matching up rows, padded with zero rows; down columns of the padding are zero."""
     from megatron_mixtera_b200.transformer.moe import interleave_up
 
     gate, up = torch.randn(100, 8), torch.randn(100, 8)
     x = interleave_up(gate, up)
     assert x.shape == (256, 8)
-    assert torch.equal(x[:64], gate[:64]) and torch.equal(x[64:128], up[:64])
-    assert torch.equal(x[128:164], gate[64:]) and torch.equal(x[192:228], up[64:])
-    assert float(x[164:192].abs().max()) == 0.0 and float(x[228:].abs().max()) == 0.0
+    x = x.view(8, 2, 16, 8)
+    for i, w in enumerate((gate, up)):
+        assert torch.equal(x[:, i].reshape(128, 8)[:100], w) and float(x[:, i].reshape(128, 8)[100:].abs().max()) == 0.0
     _, w, model = build("wide")
     model.load_checkpoint(w)
     moe = model.layers[0].moe

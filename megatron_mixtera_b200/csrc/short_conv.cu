@@ -180,19 +180,21 @@ conv_silu_kernel(b200_conv_args a, int run) {
   }
 }
 
-// LPH lanes per head, VEC * EL channels each; a warp holds 32 / LPH (head, run) units.
+// LPH lanes per head, VEC * EL channels each; a warp holds 32 / LPH (head, run) units.  Heads [head0, head0 + heads_here) of
+// queries | keys | values.
 template <typename T, int VEC, int EL, int LPH, int TAPS>
-__global__ void __launch_bounds__(kThreads)
-conv_qkv_kernel(b200_conv_args a, int run) {
-  constexpr int B = EL == 1 && TAPS == 4 ? 4 : 1;  // tokens whose loads are in flight together
+__global__ void __launch_bounds__(kThreads, EL == 1 && TAPS == 4 ? 4 : 1)
+conv_qkv_kernel(b200_conv_args a, int run, int head0, int heads_here) {
   using V = Raw<T, VEC>;
   pdl_launch_dependents();
   const int lane = threadIdx.x % LPH;
-  const int heads = a.heads + 2 * a.kv_heads, runs = (a.num_tokens + run - 1) / run;
-  const int unit_raw = (blockIdx.x * kThreads + threadIdx.x) / LPH;
-  const bool active = unit_raw < heads * runs;
-  const int unit = active ? unit_raw : 0;  // (lanes without a unit take part in the sums only)
-  const int hh = unit % heads, t0 = unit / heads * run;
+  const unsigned group = LPH == 32 ? 0xffffffffu : ((1u << LPH) - 1) << (threadIdx.x % 32 / LPH * LPH);  // lanes that work together
+  const int unit = (blockIdx.x * kThreads + threadIdx.x) / LPH;
+  const int t0 = unit / heads_here * run, hh = head0 + unit % heads_here, t1 = min(t0 + run, a.num_tokens);
+  if (t0 >= t1) {
+    pdl_wait();
+    return;
+  }
   const int kind = hh < a.heads ? 0 : hh < a.heads + a.kv_heads ? 1 : 2;  // query, key, value
   const int g = kind == 0 ? hh : kind == 1 ? hh - a.heads : hh - a.heads - a.kv_heads;
   const int d = kind == 2 ? a.vdim : a.dim;
@@ -208,78 +210,105 @@ conv_qkv_kernel(b200_conv_args a, int run) {
   }
   const float mix = kind == 2 && a.v_first_in != nullptr ? simt::to_f32(*static_cast<const T*>(a.mix)) : 0.f;
   const int64_t pool_tokens = static_cast<int64_t>(a.num_chunks) * a.chunk_size;
-  pdl_wait();
-  Row r{0, -1, -1, -1};
-  for (int tb = 0; tb < run; tb += B) {
-    V now[B][EL], first[B][EL];
-    int64_t token[B];
+  const T* src = static_cast<const T*>(a.proj) + c0;
+  // Norm or mixing of a token's convolved channels, and their store.
+  auto finish = [&](int t, float (&y)[EL][VEC]) {
+    T* dst;
+    if (kind != 2) {
+      float sq = 0.f;
 #pragma unroll
-    for (int q = 0; q < B; ++q) {
-      const int t = min(t0 + tb + q, a.num_tokens - 1);
-      token[q] = kind == 0 ? 0 : a.chunk_idx[t] * a.chunk_size + a.local_pos[t];
+      for (int e = 0; e < EL; ++e)
+        if ((e * LPH + lane) * VEC < d) {
+#pragma unroll
+          for (int k = 0; k < VEC; ++k) sq = fmaf(y[e][k], y[e][k], sq);
+        }
+#pragma unroll
+      for (int o = LPH / 2; o > 0; o >>= 1) sq += __shfl_xor_sync(group, sq, o);
+      const float inv = 1.f / sqrtf(sq / d + a.eps);
+#pragma unroll
+      for (int e = 0; e < EL; ++e)
+        if ((e * LPH + lane) * VEC < d) {
+#pragma unroll
+          for (int k = 0; k < VEC; ++k) y[e][k] *= inv * simt::to_f32(weight[e].e[k]);
+        }
+    } else {
 #pragma unroll
       for (int e = 0; e < EL; ++e) {
         const int i = (e * LPH + lane) * VEC;
         if (i >= d) continue;
-        now[q][e] = *reinterpret_cast<const V*>(static_cast<const T*>(a.proj) + t * a.proj_ld + c0 + i);
-        if (kind == 2 && a.v_first_in != nullptr)
-          first[q][e] = *reinterpret_cast<const V*>(static_cast<const T*>(a.v_first_in) + (static_cast<int64_t>(t) * a.kv_heads + g) * d + i);
+        const int64_t at = (static_cast<int64_t>(t) * a.kv_heads + g) * d + i;
+        if (a.v_first_out != nullptr) store<T, VEC>(static_cast<T*>(a.v_first_out) + at, y[e]);
+        if (a.v_first_in != nullptr) {
+          const V first = *reinterpret_cast<const V*>(static_cast<const T*>(a.v_first_in) + at);
+#pragma unroll
+          for (int k = 0; k < VEC; ++k) y[e][k] = fmaf(mix, simt::to_f32(first.e[k]), (1.f - mix) * y[e][k]);
+        }
       }
     }
+    if (kind == 0) {
+      dst = static_cast<T*>(a.out) + (static_cast<int64_t>(t) * a.heads + g) * d;
+    } else {
+      const int64_t token = a.chunk_idx[t] * a.chunk_size + a.local_pos[t];
+      if (token < 0 || token >= pool_tokens) return;
+      dst = static_cast<T*>(kind == 1 ? a.k_pool : a.v_pool) + token * a.pool_row_elems + g * d;
+    }
 #pragma unroll
-    for (int q = 0; q < B; ++q) {
-      const int t = t0 + tb + q;
-      const bool on = active && tb + q < run && t < a.num_tokens;
-      if (on && t >= r.end) {
-        r = row_of(a, t);
-#pragma unroll
-        for (int e = 0; e < EL; ++e)
-          if ((e * LPH + lane) * VEC < d) win[e].load_history(a, r, t, c0 + (e * LPH + lane) * VEC);
-      }
-      float y[EL][VEC], sq = 0.f;
-#pragma unroll
-      for (int e = 0; e < EL; ++e) {
-        const int i = (e * LPH + lane) * VEC;
-        if (!on || i >= d) continue;
-        float x[VEC];
-        now[q][e].to(x);
-        win[e].step(x, y[e]);
-        if (t == r.end - 1) win[e].store_history(a, r, c0 + i);
-#pragma unroll
-        for (int k = 0; k < VEC; ++k) sq = fmaf(y[e][k], y[e][k], sq);
-      }
-#pragma unroll
-      for (int o = LPH / 2; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
-      if (!on) continue;
-      T* dst;
-      if (kind != 2) {
-        const float inv = 1.f / sqrtf(sq / d + a.eps);
-#pragma unroll
-        for (int e = 0; e < EL; ++e) {
-          if ((e * LPH + lane) * VEC >= d) continue;
-#pragma unroll
-          for (int k = 0; k < VEC; ++k) y[e][k] *= inv * simt::to_f32(weight[e].e[k]);
-        }
-        dst = kind == 0 ? static_cast<T*>(a.out) + (static_cast<int64_t>(t) * a.heads + g) * d
-                        : static_cast<T*>(a.k_pool) + token[q] * a.pool_row_elems + g * d;
-      } else {
-#pragma unroll
-        for (int e = 0; e < EL; ++e) {
-          const int i = (e * LPH + lane) * VEC;
-          if (i >= d) continue;
-          if (a.v_first_out != nullptr) store<T, VEC>(static_cast<T*>(a.v_first_out) + (static_cast<int64_t>(t) * a.kv_heads + g) * d + i, y[e]);
-          if (a.v_first_in != nullptr) {
-#pragma unroll
-            for (int k = 0; k < VEC; ++k) y[e][k] = fmaf(mix, simt::to_f32(first[q][e].e[k]), (1.f - mix) * y[e][k]);
-          }
-        }
-        dst = static_cast<T*>(a.v_pool) + token[q] * a.pool_row_elems + g * d;
-      }
-      if (token[q] < 0 || token[q] >= pool_tokens) continue;
+    for (int e = 0; e < EL; ++e)
+      if ((e * LPH + lane) * VEC < d) store<T, VEC>(dst + (e * LPH + lane) * VEC, y[e]);
+  };
+  pdl_wait();
+  Row r{0, -1, -1, -1};
+  for (int t = t0; t < t1;) {
+    if (t >= r.end) {
+      r = row_of(a, t);
 #pragma unroll
       for (int e = 0; e < EL; ++e)
-        if ((e * LPH + lane) * VEC < d) store<T, VEC>(dst + (e * LPH + lane) * VEC, y[e]);
+        if ((e * LPH + lane) * VEC < d) win[e].load_history(a, r, t, c0 + (e * LPH + lane) * VEC);
     }
+    if constexpr (EL == 1 && TAPS == 4) {
+      if (t + 4 <= min(r.end, t1)) {  // four tokens of one request at once
+        const int i = lane * VEC;
+        const bool mine = i < d;
+        V now[4];
+#pragma unroll
+        for (int q = 0; q < 4; ++q)
+          if (mine) now[q] = *reinterpret_cast<const V*>(src + (t + q) * a.proj_ld + i);
+        float u[7][VEC];
+#pragma unroll
+        for (int q = 0; q < 3; ++q)
+#pragma unroll
+          for (int k = 0; k < VEC; ++k) u[q][k] = win[0].u[q][k];
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+          now[q].to(u[q + 3]);
+          float y[1][VEC];
+#pragma unroll
+          for (int k = 0; k < VEC; ++k)
+            y[0][k] = fmaf(win[0].w[3][k], u[q + 3][k],
+                           fmaf(win[0].w[2][k], u[q + 2][k], fmaf(win[0].w[1][k], u[q + 1][k], win[0].w[0][k] * u[q][k])));
+          finish(t + q, y);
+        }
+#pragma unroll
+        for (int q = 0; q < 3; ++q)
+#pragma unroll
+          for (int k = 0; k < VEC; ++k) win[0].u[q][k] = u[q + 4][k];
+        t += 4;
+        if (t == r.end && mine) win[0].store_history(a, r, c0 + i);
+        continue;
+      }
+    }
+    float y[EL][VEC];
+#pragma unroll
+    for (int e = 0; e < EL; ++e) {
+      const int i = (e * LPH + lane) * VEC;
+      if (i >= d) continue;
+      float now[VEC];
+      load<T, VEC>(src + t * a.proj_ld + i, now);
+      win[e].step(now, y[e]);
+      if (t == r.end - 1) win[e].store_history(a, r, c0 + i);
+    }
+    finish(t, y);
+    ++t;
   }
 }
 
@@ -353,28 +382,34 @@ static int silu(const b200_conv_args& a, cudaStream_t s) {
 }
 
 template <typename T, int VEC, int EL, int LPH, int TAPS>
-static int launch_qkv(const b200_conv_args& a, cudaStream_t s) {
-  const int heads = a.heads + 2 * a.kv_heads;
+static int launch_qkv(const b200_conv_args& a, int head0, int heads, cudaStream_t s) {
   const int run = run_length(a, static_cast<int64_t>(heads) * LPH / 32 + 1);
   const int64_t threads = static_cast<int64_t>(heads) * ((a.num_tokens + run - 1) / run) * LPH;
   if (threads > 0x3fffffff) return B200_ERR_INVALID_ARGUMENT;
   return launch_pdl(conv_qkv_kernel<T, VEC, EL, LPH, TAPS>, dim3(static_cast<unsigned>((threads + kThreads - 1) / kThreads)), dim3(kThreads), 0,
-                    s, a, run);
+                    s, a, run, head0, heads);
+}
+// Heads [head0, head0 + heads), all of `d` channels.
+template <typename T, int TAPS>
+static int qkv_heads(const b200_conv_args& a, int head0, int heads, int d, bool vec, cudaStream_t s) {
+  constexpr int VEC = 16 / sizeof(T);
+  if (!vec) return launch_qkv<T, 1, 8, 32, TAPS>(a, head0, heads, s);
+  if (d <= 8 * VEC) return launch_qkv<T, VEC, 1, 8, TAPS>(a, head0, heads, s);
+  if (d <= 16 * VEC) return launch_qkv<T, VEC, 1, 16, TAPS>(a, head0, heads, s);
+  if (d <= 32 * VEC) return launch_qkv<T, VEC, 1, 32, TAPS>(a, head0, heads, s);
+  return launch_qkv<T, VEC, 256 / (32 * VEC), 32, TAPS>(a, head0, heads, s);
 }
 template <typename T, int TAPS>
 static int qkv(const b200_conv_args& a, cudaStream_t s) {
-  const int widest = a.dim > a.vdim ? a.dim : a.vdim;
-  constexpr int VEC = 4;
+  constexpr int VEC = 16 / sizeof(T);
   bool vec = a.dim % VEC == 0 && a.vdim % VEC == 0 && a.proj_ld % VEC == 0 && a.pool_row_elems % VEC == 0;
   for (const void* p : {a.proj, a.filter, static_cast<const void*>(a.state), static_cast<const void*>(a.out), a.q_norm, a.k_norm,
                         static_cast<const void*>(a.k_pool), static_cast<const void*>(a.v_pool), a.v_first_in,
                         static_cast<const void*>(a.v_first_out)})
-    vec = vec && reinterpret_cast<uintptr_t>(p) % (VEC * sizeof(T)) == 0;
-  if (!vec) return launch_qkv<T, 1, 8, 32, TAPS>(a, s);
-  if (widest <= 8 * VEC) return launch_qkv<T, VEC, 1, 8, TAPS>(a, s);
-  if (widest <= 16 * VEC) return launch_qkv<T, VEC, 1, 16, TAPS>(a, s);
-  if (widest <= 32 * VEC) return launch_qkv<T, VEC, 1, 32, TAPS>(a, s);
-  return launch_qkv<T, VEC, 2, 32, TAPS>(a, s);
+    vec = vec && aligned16(p);
+  if (a.dim == a.vdim) return qkv_heads<T, TAPS>(a, 0, a.heads + 2 * a.kv_heads, a.dim, vec, s);
+  const int rc = qkv_heads<T, TAPS>(a, 0, a.heads + a.kv_heads, a.dim, vec, s);
+  return rc != B200_OK ? rc : qkv_heads<T, TAPS>(a, a.heads + a.kv_heads, a.kv_heads, a.vdim, vec, s);
 }
 
 template <typename T>

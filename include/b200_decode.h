@@ -421,6 +421,21 @@ typedef struct {
   int32_t value_dim;
   int32_t window;
   int64_t pool_row_elems;
+  /* separate == 2: the same layout with extras (zero / NULL: without).
+   *   score = scale * q . k; with softcap > 0: softcap * tanh(score / softcap); plus distance_bias[head][min(distance, bias_len - 1)];
+   *   under a window positions [0, keep_first) stay visible; the softmax denominator also holds exp(sinks[head]); out * out_scale.
+   * maps == 2: every head has two query / key vectors (head by head [map 1 | map 2], head_dim each) over one value vector; out =
+   *   (a1 - lambda a2) / sqrt(mean(.^2) + eps) * diff_scale * sigmoid(gate) * out_scale of their attention outputs a1, a2 (gate NULL: 1; no
+   *   sinks, no bias).  Needs a workspace of num_tokens * 2 * num_q_heads * num_splits * (d + 1) floats, d = 64 or 128 >= value_dim (on the
+   *   CUDA cores: num_splits 1, d = value_dim). */
+  int64_t q_ld;   /* elements between tokens' queries (0: packed) */
+  int64_t out_ld; /* elements between tokens' outputs (0: packed) */
+  const float* distance_bias;
+  const float* sinks;
+  const void* gate; /* [T][gate_ld]: num_q_heads * value_dim columns */
+  int64_t gate_ld;
+  float out_scale, softcap, lambda, diff_scale, eps;
+  int32_t bias_len, keep_first, maps;
 } b200_attention_args;
 
 size_t b200_paged_attention_workspace_bytes(int num_tokens, int num_q_heads, int head_dim, int num_splits);
@@ -700,9 +715,17 @@ int b200_token_shift(const b200_shift_args* args, b200_stream_t stream);
  *   convolutions of q | k | v at columns [0, 2 kv_heads dim + heads vdim) of proj, with silu, and their state).
  * b200_recurrence_scan: rows of any length; WKV reads z as fp32 partial sums, DELTA reads the convolved q | k | v from `conv`.
  * b200_recurrence_finish: head norm, weight and gate behind the scan.
- * b200_recurrence_lora: lora = tanh(sum of partial sums) in `dtype` (WKV). */
+ * b200_recurrence_lora: lora = tanh(sum of partial sums) in `dtype` (WKV).
+ *   B200_RECURRENCE_MEMORY q = proj[off_r] * dim^-1/2, k = proj[off_k], v = proj[off_v]; log gates from the fp32 partial sums z
+ *                          [z_splits][T][z_ld] (columns: heads input gates, heads forget gates) and decay_bias [2 * heads] in that
+ *                          order: i = cap tanh((z_i + b_i) / cap), f = logsigmoid(cap tanh((z_f + b_f) / cap)).  With the running
+ *                          maximum m (starting at 0), m' = max(f + m, i): S <- e^(f + m - m') S + e^(i - m') k v^T, n likewise with k alone,
+ *                          o = S^T q / (max(|n . q|, e^-m') + 1e-6).  State [slot][head][vdim + 1][dim]: n is the last "value channel".
+ *                          out = o / rms(o) * norm_weight * sigmoid(gate).
+ * b200_recurrence_gates: the maximum and the factors of every token of a step, before b200_recurrence_scan (MEMORY). */
 #define B200_RECURRENCE_WKV 0
 #define B200_RECURRENCE_DELTA 1
+#define B200_RECURRENCE_MEMORY 2
 typedef struct b200_recurrence_args {
   const void* proj;
   const void* conv;       /* DELTA scan: [T][conv channels] */
@@ -725,11 +748,20 @@ typedef struct b200_recurrence_args {
   int32_t kind, off_r, off_k, off_v, off_g, off_a, off_b; /* columns of proj (r: also q) */
   int32_t rank, heads, kv_heads, dim, vdim, taps, num_tokens, num_rows, z_splits, norm_per_head, dtype;
   float unit_eps, eps;
+  /* MEMORY */
+  float* top;   /* [slot][heads]: the running maximum */
+  float* gates; /* [T][heads][4]: written by b200_recurrence_gates, read by the scan */
+  float* below; /* [T][heads]: what the scan's outputs are to be divided by */
+  float gate_cap, out_scale; /* out_scale: factor on the output */
+  int32_t z_ld;
+  /* every kind: elements between tokens' outputs (0: heads * vdim) */
+  int64_t out_ld;
 } b200_recurrence_args;
 int b200_recurrence_decode(const b200_recurrence_args* args, b200_stream_t stream);
 int b200_recurrence_scan(const b200_recurrence_args* args, b200_stream_t stream);
 int b200_recurrence_finish(const b200_recurrence_args* args, b200_stream_t stream);
 int b200_recurrence_lora(const b200_recurrence_args* args, b200_stream_t stream);
+int b200_recurrence_gates(const b200_recurrence_args* args, b200_stream_t stream);
 
 /* Mixture of experts.  Expert: y = W_down act(W_gate x', W_up x') with x' = weight * x (the weight is applied to the products, in
  * fp32), act(g, u) = g' sigmoid(alpha g') (u' + 1), g' = min(g, limit), u' = clamp(u, -limit, limit).
@@ -763,11 +795,84 @@ typedef struct b200_moe_args {
   void* shared_y;
   int32_t num_tokens, width, experts, top, ff, shared_ff, router_splits, router_ld, tile_tokens, max_tiles, simt, dtype;
   float limit, shared_limit, alpha;
+  /* plain != 0: scores = softmax over experts + identity router columns; chosen by score + correction among the keep_groups of
+   * `groups` equal groups of neighbours with the largest best choice score; pair_weight = chosen score / (their sum + 1e-20) *
+   * weight_scale.  Columns [experts, experts + identity) are experts whose output is their input: their pairs count no rows.  Experts
+   * then are W_down (silu(W_gate x) * W_up x), unweighted: whoever adds the rows up applies pair_weight. */
+  int32_t plain, identity, groups, keep_groups;
+  const void* correction; /* [experts + identity] (`dtype`) */
+  float weight_scale;
 } b200_moe_args;
 int b200_moe_route(const b200_moe_args* args, b200_stream_t stream);
 int b200_moe_gather(const b200_moe_args* args, b200_stream_t stream);
 int b200_moe_up(const b200_moe_args* args, b200_stream_t stream);
 int b200_moe_down(const b200_moe_args* args, b200_stream_t stream);
+
+/* ---------------------------------------------------------------------------------------
+ * Attention with finished queries: what lies between the projections and the attention kernel.  Per token: query vectors (q_vecs x dim at
+ * column off_q of proj), key vectors (k_vecs x dim at off_k) and value vectors (v_vecs x vdim at off_v), each plus its bias (NULL: none; value
+ * columns may be the key columns).  Queries and keys turn in pairs (2i, 2i + 1), or (i, i + rot_dims / 2) with `halves`, on their
+ * first rot_dims dimensions by the angle whose scaled cos / sin are rope_cos / rope_sin [position][rot_dims / 2]; with rms != 0 they are
+ * then divided by their root mean square.  Queries go to q_out, keys and values to the pool.  Any of the counts may be 0. */
+typedef struct b200_rotate_append_args {
+  const void* proj; /* [T][proj_ld] */
+  const void* q_bias;
+  const void* k_bias;
+  const void* v_bias;
+  const float* rope_cos;
+  const float* rope_sin;
+  const int64_t* token_to_pos;
+  const int64_t* chunk_idx;
+  const int64_t* local_pos;
+  void* q_out; /* [T][q_vecs * dim] */
+  void* k_pool;
+  void* v_pool;
+  int64_t proj_ld, pool_row_elems;
+  int32_t off_q, off_k, off_v, q_vecs, k_vecs, v_vecs, dim, vdim, rot_dims, halves, rms, num_tokens, chunk_size, num_chunks, max_positions,
+      dtype;
+  float eps;
+} b200_rotate_append_args;
+int b200_rotate_append(const b200_rotate_append_args* args, b200_stream_t stream);
+
+/* Several residual streams x_1 .. x_s in place of one, fp32 [row][streams][width].  One sublayer's end and the next one's start:
+ *   x_t <- sum_s mix[s][t] x_s + out[t] * y                    (mix NULL: x stays as it is)
+ *   y_out = layer norm(sum_s in[s] x_s) * gamma + beta         (in NULL: all ones; y_out NULL: no norm)
+ * y = sum over num_splits of partials[s][row] (fp32) + branch_bias + sum over j < top of pair_weight[row][j] * (expert_rows[offsets[expert] +
+ * rank], or expert_input[row] for the pairs of identity experts), each part optional.  With `table` the streams start instead:
+ * x_s = table[ids[row]] * table_scale.  row_index == NULL: all rows, the streams are stored back; else out row r shows row row_index[r] of
+ * source_rows rows and nothing is stored back.  At most 16 streams. */
+typedef struct b200_stream_norm_args {
+  const void* table;
+  const int64_t* ids;
+  const float* partials;
+  const void* branch_bias;
+  const void* expert_rows;
+  const int32_t* pairs;
+  const float* pair_weight;
+  const int32_t* offsets;
+  const void* expert_input;
+  const int64_t* row_index;
+  float* hidden;
+  const float* mix;
+  const float* out;
+  const float* in;
+  const void* gamma;
+  const void* beta;
+  void* y;
+  int64_t table_rows, expert_row_count;
+  int32_t num_splits, rows, source_rows, width, streams, top, experts, identity, dtype;
+  float table_scale, eps;
+} b200_stream_norm_args;
+int b200_stream_norm(const b200_stream_norm_args* args, b200_stream_t stream);
+
+/* out[r][i] = silu(in[r][i]) * in[r][F + i] in fp32 arithmetic, any width. */
+typedef struct b200_swiglu_args {
+  const void* in;
+  void* out;
+  int64_t rows;
+  int32_t width, dtype;
+} b200_swiglu_args;
+int b200_swiglu(const b200_swiglu_args* args, b200_stream_t stream);
 
 #ifdef __cplusplus
 }

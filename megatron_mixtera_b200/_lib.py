@@ -101,6 +101,10 @@ EXPORTED_SYMBOLS = (
     "b200_moe_gather",
     "b200_moe_up",
     "b200_moe_down",
+    "b200_recurrence_gates",
+    "b200_rotate_append",
+    "b200_stream_norm",
+    "b200_swiglu",
 )
 
 
@@ -147,6 +151,20 @@ class AttentionArgs(ctypes.Structure):
         ("value_dim", c_int32),
         ("window", c_int32),
         ("pool_row_elems", c_int64),
+        ("q_ld", c_int64),
+        ("out_ld", c_int64),
+        ("distance_bias", c_void_p),
+        ("sinks", c_void_p),
+        ("gate", c_void_p),
+        ("gate_ld", c_int64),
+        ("out_scale", c_float),
+        ("softcap", c_float),
+        ("lambda_", c_float),
+        ("diff_scale", c_float),
+        ("eps", c_float),
+        ("bias_len", c_int32),
+        ("keep_first", c_int32),
+        ("maps", c_int32),
     ]
 
 
@@ -222,7 +240,8 @@ class RecurrenceArgs(ctypes.Structure):
                    "o_f32 out"),
         (c_int64, "proj_ld state_slots"),
         (c_int32, "kind off_r off_k off_v off_g off_a off_b rank heads kv_heads dim vdim taps num_tokens num_rows z_splits norm_per_head "
-                  "dtype"), (c_float, "unit_eps eps"))
+                  "dtype"), (c_float, "unit_eps eps"), (c_void_p, "top gates below"), (c_float, "gate_cap out_scale"),
+        (c_int32, "z_ld"), (c_int64, "out_ld"))
 
 
 class MoeArgs(ctypes.Structure):
@@ -232,7 +251,33 @@ class MoeArgs(ctypes.Structure):
         (c_void_p, "x router up down shared_up shared_down counts pairs pair_weight offsets tiles num_tiles shared_gate x_sorted row_scale "
                    "inter y shared_inter shared_y"),
         (c_int32, "num_tokens width experts top ff shared_ff router_splits router_ld tile_tokens max_tiles simt dtype"),
-        (c_float, "limit shared_limit alpha"))
+        (c_float, "limit shared_limit alpha"), (c_int32, "plain identity groups keep_groups"), (c_void_p, "correction"),
+        (c_float, "weight_scale"))
+
+
+class RotateAppendArgs(ctypes.Structure):
+    """Mirror of ``b200_rotate_append_args``."""
+
+    _fields_ = _fields(
+        (c_void_p, "proj q_bias k_bias v_bias rope_cos rope_sin token_to_pos chunk_idx local_pos q_out k_pool v_pool"),
+        (c_int64, "proj_ld pool_row_elems"),
+        (c_int32, "off_q off_k off_v q_vecs k_vecs v_vecs dim vdim rot_dims halves rms num_tokens chunk_size num_chunks max_positions dtype"),
+        (c_float, "eps"))
+
+
+class StreamNormArgs(ctypes.Structure):
+    """Mirror of ``b200_stream_norm_args``."""
+
+    _fields_ = _fields(
+        (c_void_p, "table ids partials branch_bias expert_rows pairs pair_weight offsets expert_input row_index hidden mix out in_ gamma beta y"),
+        (c_int64, "table_rows expert_row_count"),
+        (c_int32, "num_splits rows source_rows width streams top experts identity dtype"), (c_float, "table_scale eps"))
+
+
+class SwigluArgs(ctypes.Structure):
+    """Mirror of ``b200_swiglu_args``."""
+
+    _fields_ = _fields((c_void_p, "in_ out"), (c_int64, "rows"), (c_int32, "width dtype"))
 
 
 class TpComm(ctypes.Structure):
@@ -399,10 +444,14 @@ def load() -> ctypes.CDLL:
     for name in ("b200_conv_silu", "b200_conv_qkv"):
         getattr(lib, name).argtypes = [POINTER(ConvArgs), c_void_p]
     lib.b200_token_shift.argtypes = [POINTER(ShiftArgs), c_void_p]
-    for name in ("b200_recurrence_decode", "b200_recurrence_scan", "b200_recurrence_finish", "b200_recurrence_lora"):
+    for name in ("b200_recurrence_decode", "b200_recurrence_scan", "b200_recurrence_finish", "b200_recurrence_lora",
+                 "b200_recurrence_gates"):
         getattr(lib, name).argtypes = [POINTER(RecurrenceArgs), c_void_p]
     for name in ("b200_moe_route", "b200_moe_gather", "b200_moe_up", "b200_moe_down"):
         getattr(lib, name).argtypes = [POINTER(MoeArgs), c_void_p]
+    lib.b200_rotate_append.argtypes = [POINTER(RotateAppendArgs), c_void_p]
+    lib.b200_stream_norm.argtypes = [POINTER(StreamNormArgs), c_void_p]
+    lib.b200_swiglu.argtypes = [POINTER(SwigluArgs), c_void_p]
     for name in EXPORTED_SYMBOLS:
         fn = getattr(lib, name)
         if fn.restype is c_int or name.startswith("b200_") and fn.restype not in (c_char_p, c_size_t):

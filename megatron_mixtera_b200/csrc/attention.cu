@@ -1,7 +1,9 @@
 // Paged-KV attention for the dynamic inference context (GQA, bf16 KV pool; the E4M3 pool has kernels of its own in
 // attention_fp8.cu).  Two layouts: fused qkv rows with RoPE and equal head dims of 64 / 128, or (`separate`) finished queries
 // and a pool of [keys | values] rows with key and value dims of their own up to 128 (the tile's missing columns are the zeros
-// TMA fills in), optionally under a sliding window.  DK / DV are the tile widths of keys and values.
+// TMA fills in), optionally under a sliding window.  DK / DV are the tile widths of keys and values.  The `separate` layout has a
+// second form with extras (kExtra): first tokens that stay visible under the window, a bias by distance, capped scores, a sink in the
+// denominator, and two attention maps over the same values whose difference leaves through diff_combine_kernel.
 //
 // One CTA works on one (token row, KV head, context split) unit:
 //   * a producer warp walks the row's block table and streams 64-token K and V tiles of that KV
@@ -31,6 +33,8 @@ constexpr int kConsumerThreads = kConsumerWarps * 32;
 constexpr int kThreads = kConsumerThreads + 32;
 constexpr int kStages = 3;
 constexpr int kMaxSplits = 64;
+constexpr int kFused = 0, kSeparate = 1, kExtra = 2;  // FORM
+constexpr float kLog2e = 1.4426950408889634f;
 
 template <int DK, int DV = DK>
 struct Cfg {
@@ -82,11 +86,46 @@ struct Params {
   int q_group, q_head, dk, dv;
   int64_t pool_row;  // elements from one token's keys (or values) to the next token's
   int window;        // keys a token sees, itself included; 0: all of its request's
+  int64_t out_ld;    // elements from one token's output to the next's
+  // kExtra
+  int keep_first;       // keys that a window never hides: positions [0, keep_first)
+  const float* bias;    // [nq][bias_len]: added to the scores at distance min(d, bias_len - 1); nullptr: none
+  int bias_len;
+  const float* sinks;   // [nq]: one more term exp(sink) in the denominator; nullptr: none
+  float cap_in, cap_out;  // score = cap_out * tanh(cap_in * q . k) (log2 domain); cap_out 0: no cap
+  float out_scale;
+  int diff;             // 1: outputs are two maps' (head = 2 * query head + map), fp32, for diff_combine_kernel
+  int kshift;           // 1: KV "heads" are (head, map) pairs that share a value head
+  int pad_dim;          // > 0: keys of both maps side by side; query row r fills columns [(r & 1) * pad_dim, + pad_dim) of dk
+  float lambda, diff_scale, eps;
+  const __nv_bfloat16* gate;  // [T][gate_ld]: the difference is multiplied with sigmoid(gate)
+  int64_t gate_ld;
 };
 
 // First key that a token whose newest visible key is kv_len - 1 sees, and the tile that holds it.
 __device__ __forceinline__ int first_key(const Params& p, int kv_len) { return p.window > 0 ? max(kv_len - p.window, 0) : 0; }
 __device__ __forceinline__ int first_tile_key(const Params& p, int kv_len) { return first_key(p, kv_len) / kTile * kTile; }
+// Tiles in front of the window's first one that hold keys which stay visible.  Tiles are counted through both ranges.
+__device__ __forceinline__ int kept_tiles(const Params& p, int base) { return (min(p.keep_first, base) + kTile - 1) / kTile; }
+// Query head of row g under KV head h.
+template <int FORM>
+__device__ __forceinline__ int query_head(const Params& p, int h, int g) {
+  if (FORM != kExtra) return h * p.G + g;
+  return ((((h >> p.kshift) * p.G) + g) << p.kshift) + (h & p.kshift);
+}
+// Where query row (h, g)'s vector starts inside a token's queries.
+template <int FORM>
+__device__ __forceinline__ int64_t query_offset(const Params& p, int h, int g) {
+  if (FORM != kExtra) return static_cast<int64_t>(h) * p.q_group + g * p.q_head;
+  return static_cast<int64_t>(h >> p.kshift) * p.q_group + (h & p.kshift) * p.dk + g * p.q_head;
+}
+// Score in the log2 domain (without the mask).
+__device__ __forceinline__ float extra_score(const Params& p, float qk, const float* bias, int distance) {
+  float v = qk * p.scale_log2;
+  if (p.cap_out > 0.f) v = p.cap_out * (1.f - __fdividef(2.f, 1.f + exp2f(qk * p.cap_in * (2.f * kLog2e))));
+  if (bias != nullptr) v = fmaf(__ldg(bias + min(max(distance, 0), p.bias_len - 1)), kLog2e, v);
+  return v;
+}
 
 // Tokens per split for a row of kv_len tokens: equal shares rounded up to whole tiles, never
 // smaller than min_split.  The combine kernel uses the same formula.
@@ -95,6 +134,11 @@ __device__ __forceinline__ int split_length(int kv_len, int num_splits, int min_
   per = ((per + kTile - 1) / kTile) * kTile;
   return per < min_split ? min_split : per;
 }
+
+__device__ __forceinline__ float to_float(float v) { return v; }
+__device__ __forceinline__ float to_float(__nv_bfloat16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ void store_float(float* p, float v) { *p = v; }
+__device__ __forceinline__ void store_float(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
 
 // out = bf16(bf16(x1 * c) - bf16(x2 * s)), bf16(bf16(x2 * c) + bf16(x1 * s)): the rounding points of
 // `t * cos + rotate_half(t) * sin` evaluated in bf16.
@@ -113,7 +157,7 @@ __device__ __forceinline__ void consumer_barrier() { asm volatile("bar.sync 1, 1
 template <int D, typename Sync>
 __device__ __forceinline__ void store_output(const Params& p, int t, int head, int d, float o, float* red, Sync block_sync) {
   if (p.out_q == nullptr) {
-    if (d < p.dv) p.out[(static_cast<int64_t>(t) * p.nq + head) * p.dv + d] = __float2bfloat16_rn(o);
+    if (d < p.dv) p.out[t * p.out_ld + head * p.dv + d] = __float2bfloat16_rn(o);
     return;
   }
   const float ob = bf16_round(o);
@@ -138,10 +182,11 @@ __device__ __forceinline__ void store_output(const Params& p, int t, int head, i
   }
 }
 
-template <int DK, int DV, bool SEPARATE>
+template <int DK, int DV, int FORM>
 __global__ void __launch_bounds__(kThreads, 2)
 paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, Params p) {
   using C = Cfg<DK, DV>;
+  constexpr bool SEPARATE = FORM != kFused, EXTRA = FORM == kExtra;
   constexpr int D = DK;  // fused layout: one width for queries, keys and values
   const int tid = threadIdx.x;
   const int warp = tid >> 5;
@@ -165,7 +210,7 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
 
   if (kv_len <= 0) {  // padding row: flash-attn returns zeros for it
     pdl_wait();
-    if (p.num_splits == 1) {
+    if (p.num_splits == 1 && !(EXTRA && p.diff)) {
       __shared__ float red0[4];
       if (tid < kConsumerThreads)
         for (int i = tid; i < G * DV; i += kConsumerThreads) store_output<DV>(p, t, h * G + i / DV, i % DV, 0.f, red0, consumer_barrier);
@@ -173,14 +218,22 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     return;
   }
   const int base = SEPARATE ? first_tile_key(p, kv_len) : 0, key_begin = SEPARATE ? first_key(p, kv_len) : 0;
-  const int L = split_length(kv_len - base, p.num_splits, p.min_split);
-  const int start = base + split * L;
-  if (start >= kv_len) {
+  // Positions in what follows are those of the visible tiles in a row: `kept` tiles of first keys, then the window's from `base` on.
+  const int kept = EXTRA ? kept_tiles(p, base) * kTile : 0;
+  const int keys = kv_len - base + kept;
+  const int L = split_length(keys, p.num_splits, p.min_split);
+  const int first = split * L;
+  if (first >= keys) {
     pdl_wait();
     return;
   }
-  const int end = min(kv_len, start + L);
-  const int n_tiles = (end - start + kTile - 1) / kTile;
+  const int last = min(keys, first + L);
+  const int n_tiles = (last - first + kTile - 1) / kTile;
+  const int start = first + base, end = EXTRA ? kv_len : last + base;  // (without kept tiles: keys of this split)
+  auto tile_key = [&](int i) {
+    const int at = first + i * kTile;
+    return EXTRA && at < kept ? at : at - kept + base;
+  };
   const int row = p.row_of_token ? p.row_of_token[t] : t;
 
   extern __shared__ uint8_t smem_raw[];
@@ -210,7 +263,7 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
       // in by the consumers), so K/V streaming starts without waiting for the QKV GEMM before us.
       // Separate append (decode): only the tile with the new token waits for the append kernel right before us.
       // Prefill steps: that kernel writes any part of the pool, so wait for it.
-      const int wait_tile = p.fused ? n_tiles : (SEPARATE && p.row_of_token == nullptr && end == kv_len) ? n_tiles - 1
+      const int wait_tile = p.fused ? n_tiles : (SEPARATE && p.row_of_token == nullptr && last == keys) ? n_tiles - 1
                             : (SEPARATE && p.row_of_token == nullptr)                                     ? n_tiles
                                                                                                             : 0;
       if (wait_tile == 0) pdl_wait();
@@ -220,7 +273,7 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
       for (int i = 0; i < n_tiles; ++i) {
         const int s = i % kStages;
         const uint32_t phase = (i / kStages) & 1;
-        const int tok0 = start + i * kTile;
+        const int tok0 = tile_key(i);
         const int c = tok0 / p.chunk;
         if (c != cur_c) {
           cur_c = c;
@@ -238,7 +291,7 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
 #pragma unroll
         for (int sub = 0; sub < C::kSubK; ++sub) tma_load_3d(kdst + sub * C::kSubBytes, &map_k, &full_bar[s], sub * 64, h, tok_row);
 #pragma unroll
-        for (int sub = 0; sub < C::kSubV; ++sub) tma_load_3d(vdst + sub * C::kSubBytes, &map_v, &full_bar[s], sub * 64, h, tok_row);
+        for (int sub = 0; sub < C::kSubV; ++sub) tma_load_3d(vdst + sub * C::kSubBytes, &map_v, &full_bar[s], sub * 64, EXTRA ? h >> p.kshift : h, tok_row);
       }
     }
     return;
@@ -247,7 +300,7 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
   // --------------------------------- consumer warps ---------------------------------
   const int gid = lane >> 2;
   const int tig = lane & 3;
-  const __nv_bfloat16* qkv_t = p.qkv + t * p.q_token + static_cast<int64_t>(h) * p.q_group;
+  const __nv_bfloat16* qkv_t = p.qkv + t * p.q_token + query_offset<FORM>(p, h, 0);
 
   pdl_wait();  // qkv is the previous kernel's output
   if (p.qkv_partials != nullptr) {
@@ -278,7 +331,11 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
   if (SEPARATE) {
     for (int i = tid; i < G * (DK / 2); i += kConsumerThreads) {
       const int g = i / (DK / 2), j = (i - g * (DK / 2)) * 2;
-      if (j < p.dk)
+      if (EXTRA && p.pad_dim > 0) {  // this row's map only: the other map's columns stay zero
+        const int at = (g & 1) * p.pad_dim;
+        if (j >= at && j < at + p.pad_dim)
+          *reinterpret_cast<uint32_t*>(&q_smem[g * C::kQStride + j]) = *reinterpret_cast<const uint32_t*>(qkv_t + g * p.q_head + j - at);
+      } else if (j < p.dk)
         *reinterpret_cast<uint32_t*>(&q_smem[g * C::kQStride + j]) = *reinterpret_cast<const uint32_t*>(qkv_t + g * p.q_head + j);
     }
   } else {
@@ -319,11 +376,15 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
   const int new_pos = kv_len - 1;  // position of this step's token (decode)
   const bool owns_new = !SEPARATE && p.fused && new_pos >= start && new_pos < end;
   const int r0 = warp * 16;        // this warp's token slice inside a tile
+  const float* bias_r[2] = {nullptr, nullptr};
+  if (EXTRA && p.bias != nullptr)
+#pragma unroll
+    for (int r = 0; r < 2; ++r) bias_r[r] = p.bias + static_cast<int64_t>(query_head<FORM>(p, h, min(gid + r * 8, G - 1))) * p.bias_len;
 
   for (int i = 0; i < n_tiles; ++i) {
     const int s = i % kStages;
     const uint32_t phase = (i / kStages) & 1;
-    const int tok0 = start + i * kTile;
+    const int tok0 = tile_key(i);
     mbar_wait_bounded(&full_bar[s], phase, abort_flag, kStatusAttnTimeout);
     uint8_t* ktile = smem + s * C::kStageBytes;
     uint8_t* vtile = ktile + C::kTileBytesK;
@@ -371,7 +432,7 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
       __syncwarp();
     }
 
-    if (tok0 + r0 < end && (!SEPARATE || tok0 + r0 + 16 > key_begin)) {
+    if (tok0 + r0 < end && (!SEPARATE || tok0 + r0 + 16 > key_begin || (EXTRA && tok0 + r0 < p.keep_first))) {
       // ---- S = Q K^T for this warp's 16 tokens ----
       float sacc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
       const int ld_row = r0 + ((lane >> 4) << 3) + (lane & 7);  // token row this lane addresses
@@ -393,8 +454,8 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
           const int tok = tok0 + r0 + nt * 8 + tig * 2 + (c & 1);
-          float v = sacc[nt][c] * scale_log2;
-          if (tok >= end || (SEPARATE && tok < key_begin)) v = -INFINITY;
+          float v = EXTRA ? extra_score(p, sacc[nt][c], bias_r[c >> 1], new_pos - tok) : sacc[nt][c] * scale_log2;
+          if (tok >= end || (SEPARATE && tok < key_begin && !(EXTRA && tok < p.keep_first))) v = -INFINITY;
           sacc[nt][c] = v;
           mx[c >> 1] = fmaxf(mx[c >> 1], v);
         }
@@ -503,10 +564,17 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
         lsum += ml[w * 16 + g] * sc;
       }
     }
-    const float o = lsum > 0.f ? acc / lsum : 0.f;
-    const int64_t qh = static_cast<int64_t>(t) * p.nq + h * G + g;
-    if (p.num_splits == 1) {
-      store_output<DV>(p, t, h * G + g, d, o, ml + kConsumerWarps * 16, consumer_barrier);
+    const int head = query_head<FORM>(p, h, g);
+    const int64_t qh = static_cast<int64_t>(t) * p.nq + head;
+    if (EXTRA && p.sinks != nullptr && p.num_splits == 1) {
+      const float sink = p.sinks[head] * kLog2e, top = fmaxf(m, sink), sc = exp2f(m - top);
+      acc *= sc;
+      lsum = lsum * sc + exp2f(sink - top);
+    }
+    float o = lsum > 0.f ? acc / lsum : 0.f;
+    if (p.num_splits == 1 && !(EXTRA && p.diff)) {
+      if (EXTRA) o *= p.out_scale;
+      store_output<DV>(p, t, head, d, o, ml + kConsumerWarps * 16, consumer_barrier);
     } else {
       p.ws_o[(qh * p.num_splits + split) * DV + d] = o;
       if (d == 0) p.ws_lse[qh * p.num_splits + split] = lsum > 0.f ? m + log2f(lsum) : -INFINITY;
@@ -525,11 +593,12 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
 // once per token.  Keys and values are already in the pool (b200_rope_append ran before); the queries are
 // rotated here, in registers.  bf16 pool only.
 // ---------------------------------------------------------------------------------------------
-template <int DK, int DV, bool SEPARATE>
+template <int DK, int DV, int FORM>
 __global__ void __launch_bounds__(kThreads, 2)
 paged_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, Params p,
                      const int32_t* __restrict__ units) {
   using C = Cfg<DK, DV>;
+  constexpr bool SEPARATE = FORM != kFused, EXTRA = FORM == kExtra;
   constexpr int D = DK;  // fused layout: one width for queries, keys and values
   const int tid = threadIdx.x;
   const int warp = tid >> 5;
@@ -553,7 +622,9 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
     min_kv = min(min_kv, p.kv_len[t0 + j]);
   }
   const int base = SEPARATE ? first_tile_key(p, min_kv) : 0;
-  const int n_tiles = (max_kv - base + kTile - 1) / kTile;
+  const int kept = EXTRA ? kept_tiles(p, base) : 0;  // tiles of first keys in front of the window's
+  const int n_tiles = kept + (max_kv - base + kTile - 1) / kTile;
+  auto tile_key = [&](int i) { return EXTRA && i < kept ? i * kTile : base + (i - kept) * kTile; };
 
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -581,7 +652,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
       for (int i = 0; i < n_tiles; ++i) {
         const int s = i % kStages;
         const uint32_t phase = (i / kStages) & 1;
-        const int tok0 = base + i * kTile;
+        const int tok0 = tile_key(i);
         const int c = tok0 / p.chunk;
         if (c != cur_c) {
           cur_c = c;
@@ -595,7 +666,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
 #pragma unroll
         for (int sub = 0; sub < C::kSubK; ++sub) tma_load_3d(kdst + sub * C::kSubBytes, &map_k, &full_bar[s], sub * 64, h, tok_row);
 #pragma unroll
-        for (int sub = 0; sub < C::kSubV; ++sub) tma_load_3d(vdst + sub * C::kSubBytes, &map_v, &full_bar[s], sub * 64, h, tok_row);
+        for (int sub = 0; sub < C::kSubV; ++sub) tma_load_3d(vdst + sub * C::kSubBytes, &map_v, &full_bar[s], sub * 64, EXTRA ? h >> p.kshift : h, tok_row);
       }
     }
     return;
@@ -626,7 +697,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
       if (tok_r[r] < 0) continue;
-      const __nv_bfloat16* q = p.qkv + tok_r[r] * p.q_token + static_cast<int64_t>(h) * p.q_group + head_r[r] * p.q_head;
+      const __nv_bfloat16* q = p.qkv + tok_r[r] * p.q_token + query_offset<FORM>(p, h, head_r[r]);
 #pragma unroll
       for (int ks = 0; ks < DK / 16; ++ks)
 #pragma unroll
@@ -640,7 +711,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
       if (tok_r[r] < 0) continue;
-      const __nv_bfloat16* q = p.qkv + tok_r[r] * p.q_token + static_cast<int64_t>(h) * p.q_group + head_r[r] * p.q_head;
+      const __nv_bfloat16* q = p.qkv + tok_r[r] * p.q_token + query_offset<FORM>(p, h, head_r[r]);
       const int64_t pq = rope ? p.pos_q[tok_r[r]] : 0;
       const __nv_bfloat16* cs = p.cos + pq * (D / 2);
       const __nv_bfloat16* sn = p.sin + pq * (D / 2);
@@ -671,6 +742,10 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
   float m_run[2] = {-INFINITY, -INFINITY};
   float l_run[2] = {0.f, 0.f};
   const float scale_log2 = p.scale_log2;
+  const float* bias_r[2] = {nullptr, nullptr};
+  if (EXTRA && p.bias != nullptr)
+#pragma unroll
+    for (int r = 0; r < 2; ++r) bias_r[r] = p.bias + static_cast<int64_t>(query_head<FORM>(p, h, head_r[r])) * p.bias_len;
   // keys this warp's rows can see at most (warp-uniform): later tiles are skipped
   int warp_kv = max(kv_r[0], kv_r[1]);
 #pragma unroll
@@ -683,11 +758,11 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
   for (int i = 0; i < n_tiles; ++i) {
     const int s = i % kStages;
     const uint32_t phase = (i / kStages) & 1;
-    const int tok0 = base + i * kTile;
+    const int tok0 = tile_key(i);
     mbar_wait_bounded(&full_bar[s], phase, abort_flag, kStatusAttnTimeout);
     uint8_t* ktile = smem + s * C::kStageBytes;
     uint8_t* vtile = ktile + C::kTileBytesK;
-    if (tok0 < warp_kv && (!SEPARATE || tok0 + kTile > warp_first)) {
+    if (tok0 < warp_kv && (!SEPARATE || tok0 + kTile > warp_first || (EXTRA && tok0 < p.keep_first))) {
       // ---- S = Q K^T: 16 rows x 64 tokens ----
       float sacc[8][4];
 #pragma unroll
@@ -714,8 +789,8 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
           const int tok = tok0 + nt * 8 + tig * 2 + (c & 1);
-          float v = sacc[nt][c] * scale_log2;
-          if (tok >= kv_r[c >> 1] || (SEPARATE && tok < first_r[c >> 1])) v = -INFINITY;
+          float v = EXTRA ? extra_score(p, sacc[nt][c], bias_r[c >> 1], kv_r[c >> 1] - 1 - tok) : sacc[nt][c] * scale_log2;
+          if (tok >= kv_r[c >> 1] || (SEPARATE && tok < first_r[c >> 1] && !(EXTRA && tok < p.keep_first))) v = -INFINITY;
           sacc[nt][c] = v;
           mx[c >> 1] = fmaxf(mx[c >> 1], v);
         }
@@ -783,8 +858,23 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
     l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 1);
     l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 2);
     if (tok_r[r] < 0) continue;
-    const float inv = l_run[r] > 0.f ? 1.f / l_run[r] : 0.f;  // a token that sees no key gets zeros, as flash-attn does
-    __nv_bfloat16* o = p.out + (static_cast<int64_t>(tok_r[r]) * p.nq + h * G + head_r[r]) * p.dv;
+    const int head = query_head<FORM>(p, h, head_r[r]);
+    float top_scale = 1.f;
+    if (EXTRA && p.sinks != nullptr) {
+      const float sink = p.sinks[head] * kLog2e, top = fmaxf(m_run[r], sink);
+      top_scale = exp2f(m_run[r] - top);
+      l_run[r] = l_run[r] * top_scale + exp2f(sink - top);
+    }
+    float inv = l_run[r] > 0.f ? 1.f / l_run[r] : 0.f;  // a token that sees no key gets zeros, as flash-attn does
+    if (EXTRA) inv *= top_scale * p.out_scale;
+    if (EXTRA && p.diff) {
+      float* o32 = p.ws_o + (static_cast<int64_t>(tok_r[r]) * p.nq + head) * DV;
+#pragma unroll
+      for (int i2 = 0; i2 < DV / 8; ++i2)
+        *reinterpret_cast<float2*>(o32 + i2 * 8 + tig * 2) = make_float2(oacc[i2][2 * r] * inv, oacc[i2][2 * r + 1] * inv);
+      continue;
+    }
+    __nv_bfloat16* o = p.out + tok_r[r] * p.out_ld + head * p.dv;
 #pragma unroll
     for (int i2 = 0; i2 < DV / 8; ++i2) {
       const int col = i2 * 8 + tig * 2;
@@ -804,24 +894,90 @@ __global__ void __launch_bounds__(D) combine_kernel(Params p) {
   const int kv_len = p.kv_len[t];
   float o = 0.f;
   if (kv_len > 0) {
-    const int keys = kv_len - first_tile_key(p, kv_len);
+    const int base = first_tile_key(p, kv_len), keys = kv_len - base + kept_tiles(p, base) * kTile;
     const int L = split_length(keys, p.num_splits, p.min_split);
     const int n_act = (keys + L - 1) / L;
     const float* lse = p.ws_lse + static_cast<int64_t>(qh) * p.num_splits;
-    float mx = -INFINITY;
+    const float sink = p.sinks != nullptr ? p.sinks[qh - t * p.nq] * kLog2e : -INFINITY;  // a split of its own, without values
+    float mx = sink;
     for (int s = 0; s < n_act; ++s) mx = fmaxf(mx, lse[s]);
     if (mx != -INFINITY) {
-      float acc = 0.f, wsum = 0.f;
+      float acc = 0.f, wsum = exp2f(sink - mx);
       for (int s = 0; s < n_act; ++s) {
         const float w = exp2f(lse[s] - mx);
         acc += w * p.ws_o[(static_cast<int64_t>(qh) * p.num_splits + s) * D + d];
         wsum += w;
       }
-      o = acc / wsum;
+      o = acc / wsum * p.out_scale;
     }
   }
   __shared__ float red[4];
   store_output<D>(p, t, qh - t * p.nq, d, o, red, [] { __syncthreads(); });
+}
+
+// Two maps over the same values: out = (a1 - lambda a2) / rms * diff_scale * sigmoid(gate) per head, a1 and a2 merged over the context
+// splits first (splits == 1: whole outputs, no log-sum-exps).  A warp per (token, head); ws_o rows are `stride` floats.
+template <typename T>
+__global__ void __launch_bounds__(256) diff_combine_kernel(Params p, const void* gate, void* out, int stride, int splits) {
+  constexpr int kElems = 8;  // up to 256 value channels
+  pdl_launch_dependents();
+  pdl_wait();
+  const int lane = threadIdx.x & 31, heads = p.nq / 2;
+  const int64_t unit = static_cast<int64_t>(blockIdx.x) * 8 + (threadIdx.x >> 5);
+  if (unit >= static_cast<int64_t>(p.T) * heads) return;
+  const int64_t t = unit / heads;
+  const int head = static_cast<int>(unit - t * heads);
+  const int kv_len = p.kv_len[t];
+  float a[2][kElems];
+#pragma unroll
+  for (int m = 0; m < 2; ++m)
+#pragma unroll
+    for (int e = 0; e < kElems; ++e) a[m][e] = 0.f;
+  if (kv_len > 0) {
+    int n_act = 1;
+    if (splits > 1) {
+      const int base = first_tile_key(p, kv_len), keys = kv_len - base + kept_tiles(p, base) * kTile;
+      const int L = split_length(keys, splits, p.min_split);
+      n_act = (keys + L - 1) / L;
+    }
+#pragma unroll
+    for (int m = 0; m < 2; ++m) {
+      const int64_t qh = t * p.nq + head * 2 + m;
+      float mx = 0.f, wsum = 0.f;
+      if (splits > 1) {
+        mx = -INFINITY;
+        for (int s = 0; s < n_act; ++s) mx = fmaxf(mx, p.ws_lse[qh * splits + s]);
+      }
+      for (int s = 0; s < n_act; ++s) {
+        const float w = splits > 1 ? exp2f(p.ws_lse[qh * splits + s] - mx) : 1.f;
+        const float* row = p.ws_o + (qh * splits + s) * stride;
+#pragma unroll
+        for (int e = 0; e < kElems; ++e)
+          if (e * 32 + lane < p.dv) a[m][e] = fmaf(w, row[e * 32 + lane], a[m][e]);
+        wsum += w;
+      }
+      if (splits > 1)
+#pragma unroll
+        for (int e = 0; e < kElems; ++e) a[m][e] /= wsum;
+    }
+  }
+  float sq = 0.f;
+#pragma unroll
+  for (int e = 0; e < kElems; ++e) {
+    a[0][e] = fmaf(-p.lambda, a[1][e], a[0][e]);
+    sq = fmaf(a[0][e], a[0][e], sq);
+  }
+  const float inv = p.diff_scale / sqrtf(warp_sum(sq) / p.dv + p.eps);
+  const T* g = gate == nullptr ? nullptr : static_cast<const T*>(gate) + t * p.gate_ld + head * p.dv;
+  T* dst = static_cast<T*>(out) + t * p.out_ld + head * p.dv;
+#pragma unroll
+  for (int e = 0; e < kElems; ++e) {
+    const int d = e * 32 + lane;
+    if (d >= p.dv) continue;
+    float v = a[0][e] * inv;
+    if (g != nullptr) v /= 1.f + expf(-to_float(g[d]));
+    store_float(dst + d, v);
+  }
 }
 
 // Prefill / mixed steps: rotate k, then scatter k and v of every token into the pool.
@@ -921,6 +1077,27 @@ static int fill_params(const b200_attention_args* a, Params& p) {
   p.q_token = static_cast<int64_t>(p.nkv) * p.q_group;
   p.pool_row = a->separate ? a->pool_row_elems : static_cast<int64_t>(p.nkv) * p.dk;
   p.window = a->window > 0 ? a->window : 0;
+  p.out_ld = static_cast<int64_t>(p.nq) * p.dv;
+  p.keep_first = 0;
+  p.bias = p.sinks = nullptr;
+  p.bias_len = p.diff = p.kshift = p.pad_dim = 0;
+  p.cap_in = p.cap_out = 0.f;
+  p.out_scale = 1.f;
+  p.gate = nullptr;
+  if (a->separate == kExtra) {
+    if (a->q_ld > 0) p.q_token = a->q_ld;
+    if (a->out_ld > 0) p.out_ld = a->out_ld;
+    p.keep_first = p.window > 0 && a->keep_first > 0 ? a->keep_first : 0;
+    p.bias = a->distance_bias;
+    p.bias_len = a->bias_len;
+    p.sinks = a->sinks;
+    p.out_scale = a->out_scale;
+    if (a->softcap > 0.f) {
+      p.cap_in = scale / a->softcap;
+      p.cap_out = a->softcap * kLog2e;
+    }
+    if ((p.bias && p.bias_len < 1) || p.q_token % 2 != 0 || (!a->maps && p.out_ld % 2 != 0)) return B200_ERR_INVALID_ARGUMENT;
+  }
   p.ws_o = nullptr;
   p.ws_lse = nullptr;
   p.k_scale = a->k_scale;
@@ -931,10 +1108,50 @@ static int fill_params(const b200_attention_args* a, Params& p) {
   return B200_OK;
 }
 
+// Two maps: each a "head" of its own with its own keys (`side_by_side` false), or both maps' keys in one tile and two query rows per head,
+// each zero in the other map's columns: keys and values are read once, the products of the zeros cost what decode steps have to spare.
+static int set_maps(const b200_attention_args* a, Params& p, bool side_by_side) {
+  if (a->maps != 2) return a->maps == 0 || a->maps == 1 ? B200_OK : B200_ERR_INVALID_ARGUMENT;
+  if (a->separate != kExtra || !a->workspace || p.bias || p.sinks) return B200_ERR_INVALID_ARGUMENT;
+  p.diff = 1;
+  p.lambda = a->lambda;
+  p.diff_scale = a->diff_scale * a->out_scale;
+  p.out_scale = 1.f;
+  p.eps = a->eps;
+  p.gate = static_cast<const __nv_bfloat16*>(a->gate);
+  p.gate_ld = a->gate_ld;
+  p.nq = 2 * a->num_q_heads;
+  p.q_token = a->q_ld > 0 ? a->q_ld : static_cast<int64_t>(p.nq) * a->head_dim;
+  p.q_group = 2 * p.G * a->head_dim;
+  p.out_ld = a->out_ld > 0 ? a->out_ld : static_cast<int64_t>(a->num_q_heads) * p.dv;
+  if (side_by_side && 2 * a->head_dim <= 128 && 2 * p.G <= 16) {
+    p.pad_dim = a->head_dim;
+    p.q_head = a->head_dim;
+    p.dk = 2 * a->head_dim;
+    p.G *= 2;
+  } else {
+    p.kshift = 1;
+    p.nkv *= 2;
+    p.q_head = 2 * a->head_dim;
+  }
+  return B200_OK;
+}
+
+static size_t maps_workspace(const b200_attention_args* a, int tile) {
+  return static_cast<size_t>(a->num_tokens) * 2 * a->num_q_heads * a->num_splits * (tile + 1) * sizeof(float);
+}
+
+template <typename T>
+static int launch_diff_combine(const Params& p, const void* gate, void* out, int stride, int splits, cudaStream_t stream) {
+  if (p.dv > 256) return B200_ERR_INVALID_ARGUMENT;
+  const int64_t units = static_cast<int64_t>(p.T) * (p.nq / 2);
+  return launch_pdl(diff_combine_kernel<T>, dim3(static_cast<unsigned>((units + 7) / 8)), dim3(256), 0, stream, p, gate, out, stride, splits);
+}
+
 static bool pool_maps(const Params& p, const CUtensorMap*& mk, const CUtensorMap*& mv) {
   const uint64_t tokens = static_cast<uint64_t>(p.num_chunks) * p.chunk;
   const uint64_t kd[3] = {static_cast<uint64_t>(p.dk), static_cast<uint64_t>(p.nkv), tokens};
-  const uint64_t vd[3] = {static_cast<uint64_t>(p.dv), static_cast<uint64_t>(p.nkv), tokens};
+  const uint64_t vd[3] = {static_cast<uint64_t>(p.dv), static_cast<uint64_t>(p.nkv >> p.kshift), tokens};
   const uint64_t ks[2] = {static_cast<uint64_t>(p.dk) * 2, static_cast<uint64_t>(p.pool_row) * 2};
   const uint64_t vs[2] = {static_cast<uint64_t>(p.dv) * 2, static_cast<uint64_t>(p.pool_row) * 2};
   const uint32_t box[3] = {64u, 1, kTile};
@@ -943,33 +1160,36 @@ static bool pool_maps(const Params& p, const CUtensorMap*& mk, const CUtensorMap
   return mk && mv;
 }
 
-template <int DK, int DV, bool SEPARATE>
+template <int DK, int DV, int FORM>
 static int launch_attention(Params& p, cudaStream_t stream) {
   using C = Cfg<DK, DV>;
   const CUtensorMap *mk, *mv;
   if (!pool_maps(p, mk, mv)) return B200_ERR_DRIVER;
   static std::atomic<uint64_t> smem_attr_done{0};
-  if (ensure_dynamic_smem(paged_attention_kernel<DK, DV, SEPARATE>, C::kSmemBytes, smem_attr_done) != B200_OK) return B200_ERR_LAUNCH;
+  if (ensure_dynamic_smem(paged_attention_kernel<DK, DV, FORM>, C::kSmemBytes, smem_attr_done) != B200_OK) return B200_ERR_LAUNCH;
   const int64_t units = static_cast<int64_t>(p.T) * p.nkv * p.num_splits;
   if (units > 0x7fffffff) return B200_ERR_INVALID_ARGUMENT;
-  int rc = launch_pdl(paged_attention_kernel<DK, DV, SEPARATE>, dim3(static_cast<unsigned>(units)), dim3(kThreads), C::kSmemBytes,
+  int rc = launch_pdl(paged_attention_kernel<DK, DV, FORM>, dim3(static_cast<unsigned>(units)), dim3(kThreads), C::kSmemBytes,
                       stream, *mk, *mv, p);
   if (rc != B200_OK) return rc;
+  if (p.diff) return launch_diff_combine<__nv_bfloat16>(p, p.gate, p.out, DV, p.num_splits, stream);
   if (p.num_splits > 1) rc = launch_pdl(combine_kernel<DV>, dim3(p.T * p.nq), dim3(DV), 0, stream, p);
   return rc;
 }
 
-template <int DK, int DV, bool SEPARATE>
+template <int DK, int DV, int FORM>
 static int launch_prefill(Params& p, const int32_t* units, int num_units, cudaStream_t stream) {
   using C = Cfg<DK, DV>;
   const CUtensorMap *mk, *mv;
   if (!pool_maps(p, mk, mv)) return B200_ERR_DRIVER;
   static std::atomic<uint64_t> smem_attr_done{0};
-  if (ensure_dynamic_smem(paged_prefill_kernel<DK, DV, SEPARATE>, C::kSmemBytes, smem_attr_done) != B200_OK) return B200_ERR_LAUNCH;
+  if (ensure_dynamic_smem(paged_prefill_kernel<DK, DV, FORM>, C::kSmemBytes, smem_attr_done) != B200_OK) return B200_ERR_LAUNCH;
   const int64_t ctas = static_cast<int64_t>(num_units) * p.nkv;
   if (ctas > 0x7fffffff) return B200_ERR_INVALID_ARGUMENT;
-  return launch_pdl(paged_prefill_kernel<DK, DV, SEPARATE>, dim3(static_cast<unsigned>(ctas)), dim3(kThreads), C::kSmemBytes, stream, *mk,
-                    *mv, p, units);
+  const int rc = launch_pdl(paged_prefill_kernel<DK, DV, FORM>, dim3(static_cast<unsigned>(ctas)), dim3(kThreads), C::kSmemBytes, stream,
+                            *mk, *mv, p, units);
+  if (rc != B200_OK || !p.diff) return rc;
+  return launch_diff_combine<__nv_bfloat16>(p, p.gate, p.out, DV, 1, stream);
 }
 
 // The layout and the tile widths that hold the head dims.
@@ -977,11 +1197,14 @@ template <typename F>
 static int by_layout(const Params& p, F&& f) {
   const std::integral_constant<int, 64> w64;
   const std::integral_constant<int, 128> w128;
-  const std::false_type fused;
-  const std::true_type separate;
+  const std::integral_constant<int, kFused> fused;
   if (!p.separate) return p.dk == 128 ? f(w128, w128, fused) : f(w64, w64, fused);
-  if (p.dk <= 64) return p.dv <= 64 ? f(w64, w64, separate) : f(w64, w128, separate);
-  return p.dv <= 64 ? f(w128, w64, separate) : f(w128, w128, separate);
+  auto by_dims = [&](auto form) {
+    if (p.dk <= 64) return p.dv <= 64 ? f(w64, w64, form) : f(w64, w128, form);
+    return p.dv <= 64 ? f(w128, w64, form) : f(w128, w128, form);
+  };
+  if (p.separate == kExtra) return by_dims(std::integral_constant<int, kExtra>{});
+  return by_dims(std::integral_constant<int, kSeparate>{});
 }
 
 }  // namespace attn
@@ -1002,6 +1225,12 @@ int b200_paged_prefill_attention(const b200_attention_args* a, const int32_t* un
   int rc = attn::fill_params(a, p);
   if (rc != B200_OK) return rc;
   if (!a->out || a->out_q || !a->qkv || !units || num_units <= 0 || a->kv_cache_fp8) return B200_ERR_INVALID_ARGUMENT;
+  rc = attn::set_maps(a, p, false);
+  if (rc != B200_OK) return rc;
+  if (p.diff) {
+    if (a->num_splits != 1 || a->workspace_bytes < attn::maps_workspace(a, p.dv <= 64 ? 64 : 128)) return B200_ERR_WORKSPACE;
+    p.ws_o = static_cast<float*>(a->workspace);
+  }
   if (64 % p.G != 0 && !p.separate) return B200_ERR_INVALID_ARGUMENT;  // group sizes 1, 2, 4, 8, 16
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   return attn::by_layout(p, [&](auto dk, auto dv, auto sep) { return attn::launch_prefill<dk, dv, sep>(p, units, num_units, s); });
@@ -1033,7 +1262,14 @@ int b200_paged_attention(const b200_attention_args* a, b200_stream_t stream) {
   if (!a->out && !a->out_q) return B200_ERR_INVALID_ARGUMENT;
   if (a->fuse_rope_append && (!a->token_to_chunk_idx || !a->token_to_local_pos)) return B200_ERR_INVALID_ARGUMENT;
   if (a->qkv_partials && (a->num_q_heads / a->num_kv_heads + 2) * a->head_dim % 4 != 0) return B200_ERR_ALIGNMENT;
-  if (a->num_splits > 1) {
+  rc = attn::set_maps(a, p, true);
+  if (rc != B200_OK) return rc;
+  if (p.diff) {
+    const int tile = p.dv <= 64 ? 64 : 128;
+    if (a->workspace_bytes < attn::maps_workspace(a, tile)) return B200_ERR_WORKSPACE;
+    p.ws_o = static_cast<float*>(a->workspace);
+    p.ws_lse = p.ws_o + static_cast<size_t>(p.T) * p.nq * p.num_splits * tile;
+  } else if (a->num_splits > 1) {
     const size_t need =
         b200_paged_attention_workspace_bytes(a->num_tokens, a->num_q_heads, a->separate ? (a->value_dim <= 64 ? 64 : 128) : a->head_dim, a->num_splits);
     if (!a->workspace || a->workspace_bytes < need) return B200_ERR_WORKSPACE;

@@ -369,10 +369,33 @@ __global__ void activation_kernel(const __nv_bfloat16* __restrict__ in, const __
   }
 }
 
+// SwiGLU of [gate | up] rows in fp32 arithmetic, any width and type.
+template <typename T>
+__global__ void __launch_bounds__(256) swiglu_kernel(b200_swiglu_args a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int64_t at = static_cast<int64_t>(blockIdx.x) * 256 + threadIdx.x, row = at / a.width;
+  if (row >= a.rows) return;
+  const int c = static_cast<int>(at - row * a.width);
+  const T* in = static_cast<const T*>(a.in) + row * 2 * a.width + c;
+  const float g = attn::to_float(in[0]), u = attn::to_float(in[a.width]);
+  attn::store_float(static_cast<T*>(a.out) + at, g / (1.f + expf(-g)) * u);
+}
+
 }  // namespace ew
 }  // namespace b200
 
 extern "C" {
+
+int b200_swiglu(const b200_swiglu_args* a, b200_stream_t stream) {
+  using namespace b200;
+  if (!a || !a->in || !a->out || a->rows <= 0 || a->width <= 0 || a->rows * a->width > (int64_t{1} << 38)) return B200_ERR_INVALID_ARGUMENT;
+  const dim3 grid(static_cast<unsigned>((a->rows * a->width + 255) / 256));
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (a->dtype == B200_DTYPE_F32) return launch_pdl(ew::swiglu_kernel<float>, grid, dim3(256), 0, s, *a);
+  if (a->dtype == B200_DTYPE_BF16) return launch_pdl(ew::swiglu_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, *a);
+  return B200_ERR_INVALID_ARGUMENT;
+}
 
 int b200_gather_rows_bf16(const void* table, const int64_t* ids, void* out, int n_rows, int row_elems,
                           int64_t vocab_start, int64_t vocab_end, const void* add_table, const int64_t* add_ids,

@@ -56,11 +56,11 @@ struct Params {
   int m_blocks = 1, x_batch = 0;
   int64_t y_batch = 0;
   // gated == kGatedClamped: every 32 rows of a weight tile are 16 gate features and the matching 16 up features; y = g' sigmoid(glu_alpha g') (u' + 1) with g' = min(g, glu_limit), u' clamped to [-glu_limit, glu_limit], all
-  // in fp32; row_scale (NULL: 1) multiplies both products of a token first.
+  // in fp32; row_scale (NULL: 1) multiplies both products of a token first.  kGatedPlain: the same layout, y = g sigmoid(g) u.
   float glu_limit = 0.f, glu_alpha = 0.f;
   const float* row_scale = nullptr;
 };
-constexpr int kGatedSilu = 1, kGatedClamped = 2;  // Params::gated
+constexpr int kGatedSilu = 1, kGatedClamped = 2, kGatedPlain = 3;  // Params::gated
 
 __device__ __forceinline__ float clamped_glu(float g, float u, float limit, float alpha) {
   g = fminf(g, limit);
@@ -161,7 +161,7 @@ __device__ __forceinline__ void epilogue(const Params& p, uint32_t tmem_base, ui
   const bool n_ok = n < p.N;
   const uint32_t lane_addr = tmem_base + (static_cast<uint32_t>(warp * 32) << 16);
 
-  if (p.gated == kGatedClamped) {
+  if (p.gated == kGatedClamped || p.gated == kGatedPlain) {
     // A warp's lanes 0-15 hold gate features, lanes 16-31 the matching up features.  Of every 32 tokens the gate lanes finish the
     // first 16 and the up lanes the others: one shuffle per finished output, no barrier.
     const bool is_gate = lane < 16;
@@ -180,7 +180,8 @@ __device__ __forceinline__ void epilogue(const Params& p, uint32_t tmem_base, ui
       for (int j = 0; j < 16; ++j) {
         const float mine = __uint_as_float(is_gate ? r[j] : r[j + 16]);
         const float other = __shfl_xor_sync(0xffffffffu, __uint_as_float(is_gate ? r[j + 16] : r[j]), 16);
-        const float v = clamped_glu_fast((is_gate ? mine : other) * sc[j], (is_gate ? other : mine) * sc[j], p.glu_limit, p.glu_alpha);
+        const float g = (is_gate ? mine : other) * sc[j], u = (is_gate ? other : mine) * sc[j];
+        const float v = p.gated == kGatedPlain ? __fdividef(g, 1.f + __expf(-g)) * u : clamped_glu_fast(g, u, p.glu_limit, p.glu_alpha);
         if (col_ok && own0 + j < m_end) y[static_cast<int64_t>(own0 + j) * p.ldy + out_col] = __float2bfloat16_rn(v);
       }
     }

@@ -1,8 +1,10 @@
-// Mixture of experts with sigmoid scores: routing, the sort of the tokens by expert, and the experts' grouped products (tcgen05:
+// Mixture of experts with sigmoid or softmax scores: routing, the sort of the tokens by expert, and the experts' grouped products (tcgen05:
 // gemm_grouped_kernel in gemm_bf16.cu; CUDA cores here).
 //
 //   route_kernel   a warp per token: scores from the router's fp32 partial sums, the `top` best, a place behind the tokens that
 //                  already chose the same expert; the CTA that finishes last turns the counts into offsets and the tile list
+//   route_softmax_kernel  the same with softmax scores, a correction of the choice, groups of experts, identity experts and weights that
+//                  add up to one
 //   gather_kernel  x_sorted[offset[expert] + rank] = x[token]
 //   simt_kernel    64 x 64 outputs per CTA in true fp32
 #include "common.cuh"
@@ -13,12 +15,65 @@ namespace moe {
 constexpr int kWarps = 8;
 constexpr int kMaxExperts = 1024;
 
+// Every CTA of a routing kernel ends here: the one that finishes last turns the counts into offsets and the tile list.
+__device__ __forceinline__ void finish_routing(const b200_moe_args& a) {
+  __shared__ int is_last;
+  __shared__ int warp_rows[kWarps], warp_tiles[kWarps];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, E = a.experts;
+  __syncthreads();
+  if (threadIdx.x == 0) {
+    __threadfence();  // this CTA's counts are visible before its ticket
+    is_last = atomicAdd(&a.counts[E], 1) == static_cast<int>(gridDim.x) - 1;
+  }
+  __syncthreads();
+  if (!is_last) return;
+  __threadfence();
+  // offsets and tiles: every thread takes a run of experts; sums over lanes, then over warps
+  const int per = (E + kWarps * 32 - 1) / (kWarps * 32), e0 = threadIdx.x * per;
+  int rows = 0, tiles = 0;
+  for (int e = e0; e < min(e0 + per, E); ++e) {
+    const int c = __ldcg(&a.counts[e]);
+    rows += c;
+    tiles += (c + a.tile_tokens - 1) / a.tile_tokens;
+  }
+  int rows_incl = rows, tiles_incl = tiles;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const int r = __shfl_up_sync(0xffffffffu, rows_incl, o), i = __shfl_up_sync(0xffffffffu, tiles_incl, o);
+    if (lane >= o) {
+      rows_incl += r;
+      tiles_incl += i;
+    }
+  }
+  if (lane == 31) {
+    warp_rows[warp] = rows_incl;
+    warp_tiles[warp] = tiles_incl;
+  }
+  __syncthreads();
+  int row_at = rows_incl - rows, tile_at = tiles_incl - tiles;
+  for (int w = 0; w < warp; ++w) {
+    row_at += warp_rows[w];
+    tile_at += warp_tiles[w];
+  }
+  for (int e = e0; e < min(e0 + per, E); ++e) {
+    const int c = __ldcg(&a.counts[e]);
+    a.offsets[e] = row_at;
+    for (int r = 0; r < c; r += a.tile_tokens, ++tile_at)
+      if (tile_at < a.max_tiles) reinterpret_cast<int4*>(a.tiles)[tile_at] = make_int4(e, row_at + r, min(a.tile_tokens, c - r), 0);
+    row_at += c;
+    a.counts[e] = 0;
+  }
+  if (threadIdx.x == kWarps * 32 - 1) {
+    a.offsets[E] = row_at;
+    *a.num_tiles = min(tile_at, a.max_tiles);
+    a.counts[E] = 0;
+  }
+}
+
 // Shared memory: [kWarps][experts] scores; the last CTA reuses none of it.
 __global__ void __launch_bounds__(kWarps * 32)
 route_kernel(b200_moe_args a) {
   extern __shared__ float score_s[];
-  __shared__ int is_last;
-  __shared__ int warp_rows[kWarps], warp_tiles[kWarps];
   pdl_launch_dependents();
   pdl_wait();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, E = a.experts;
@@ -75,54 +130,105 @@ route_kernel(b200_moe_args a) {
       }
     }
   }
-  __syncthreads();
-  if (threadIdx.x == 0) {
-    __threadfence();  // this CTA's counts are visible before its ticket
-    is_last = atomicAdd(&a.counts[E], 1) == static_cast<int>(gridDim.x) - 1;
-  }
-  __syncthreads();
-  if (!is_last) return;
-  __threadfence();
-  // offsets and tiles: every thread takes a run of experts; sums over lanes, then over warps
-  const int per = (E + kWarps * 32 - 1) / (kWarps * 32), e0 = threadIdx.x * per;
-  int rows = 0, tiles = 0;
-  for (int e = e0; e < min(e0 + per, E); ++e) {
-    const int c = __ldcg(&a.counts[e]);
-    rows += c;
-    tiles += (c + a.tile_tokens - 1) / a.tile_tokens;
-  }
-  int rows_incl = rows, tiles_incl = tiles;
+  finish_routing(a);
+}
+
+// Softmax over experts and identity experts, choice by score + correction inside the best groups.
+// Shared memory: [kWarps][columns + groups] scores and the groups' best choice scores.
+template <typename T>
+__global__ void __launch_bounds__(kWarps * 32)
+route_softmax_kernel(b200_moe_args a) {
+  extern __shared__ float score_s[];
+  __shared__ int chosen_s[kWarps][64];
+  __shared__ float weight_s[kWarps][64];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, E = a.experts, C = a.experts + a.identity;
+  const int t = blockIdx.x * kWarps + warp;
+  const T* correction = static_cast<const T*>(a.correction);
+  if (t < a.num_tokens) {
+    float* score = score_s + warp * (C + a.groups);
+    float* group_best = score + C;
+    const int64_t stride = static_cast<int64_t>(a.num_tokens) * a.router_ld;
+    const float* z = a.router + static_cast<int64_t>(t) * a.router_ld;
+    float top = -INFINITY, sum = 0.f;
+    for (int e = lane; e < C; e += 32) {
+      float x = 0.f;
+      for (int s = 0; s < a.router_splits; ++s) x += z[s * stride + e];
+      score[e] = x;
+      top = fmaxf(top, x);
+    }
+    top = warp_max(top);
+    for (int e = lane; e < C; e += 32) {
+      score[e] = expf(score[e] - top);
+      sum += score[e];
+    }
+    sum = warp_sum(sum);
+    for (int e = lane; e < C; e += 32) score[e] /= sum;
+    auto choice = [&](int e) { return score[e] < 0.f ? -INFINITY : score[e] + simt::to_f32(correction[e]); };  // (negative: marked)
+    // The largest of f over [0, n), the smallest index among equals (n: nothing above minus infinity).
+    auto best_of = [&](int n, auto f) {
+      float best = -INFINITY;
+      int at = n;
+      for (int e = lane; e < n; e += 32) {
+        const float v = f(e);
+        if (v > best) {
+          best = v;
+          at = e;
+        }
+      }
 #pragma unroll
-  for (int o = 1; o < 32; o <<= 1) {
-    const int r = __shfl_up_sync(0xffffffffu, rows_incl, o), i = __shfl_up_sync(0xffffffffu, tiles_incl, o);
-    if (lane >= o) {
-      rows_incl += r;
-      tiles_incl += i;
+      for (int o = 16; o > 0; o >>= 1) {
+        const float b = __shfl_xor_sync(0xffffffffu, best, o);
+        const int i = __shfl_xor_sync(0xffffffffu, at, o);
+        if (b > best || (b == best && i < at)) {
+          best = b;
+          at = i;
+        }
+      }
+      return at;
+    };
+    __syncwarp();
+    if (a.groups > 1) {
+      const int size = C / a.groups;
+      for (int g = lane; g < a.groups; g += 32) {
+        float m = -INFINITY;
+        for (int e = g * size; e < (g + 1) * size; ++e) m = fmaxf(m, choice(e));
+        group_best[g] = m;
+      }
+      __syncwarp();
+      for (int k = 0; k < a.keep_groups; ++k) {
+        const int g = best_of(a.groups, [&](int i) { return group_best[i] == INFINITY ? -INFINITY : group_best[i]; });
+        __syncwarp();
+        if (g < a.groups && lane == 0) group_best[g] = INFINITY;  // kept
+        __syncwarp();
+      }
+      for (int e = lane; e < C; e += 32)
+        if (group_best[e / size] != INFINITY) score[e] = -1.f;
+      __syncwarp();
+    }
+    float total = 0.f;
+    for (int k = 0; k < a.top; ++k) {
+      int at = best_of(C, choice);
+      if (at >= C) at = k;  // no number left (NaN scores): any expert, its output is NaN too
+      const float s = score[at];
+      __syncwarp();
+      if (lane == 0) {
+        chosen_s[warp][k] = at;
+        weight_s[warp][k] = s;
+        score[at] = -1.f;
+      }
+      total += s;
+      __syncwarp();
+    }
+    for (int k = lane; k < a.top; k += 32) {
+      const int64_t pair = static_cast<int64_t>(t) * a.top + k;
+      const int e = chosen_s[warp][k];
+      reinterpret_cast<int2*>(a.pairs)[pair] = make_int2(e, e < E ? atomicAdd(&a.counts[e], 1) : 0);
+      a.pair_weight[pair] = weight_s[warp][k] / (total + 1e-20f) * a.weight_scale;
     }
   }
-  if (lane == 31) {
-    warp_rows[warp] = rows_incl;
-    warp_tiles[warp] = tiles_incl;
-  }
-  __syncthreads();
-  int row_at = rows_incl - rows, tile_at = tiles_incl - tiles;
-  for (int w = 0; w < warp; ++w) {
-    row_at += warp_rows[w];
-    tile_at += warp_tiles[w];
-  }
-  for (int e = e0; e < min(e0 + per, E); ++e) {
-    const int c = __ldcg(&a.counts[e]);
-    a.offsets[e] = row_at;
-    for (int r = 0; r < c; r += a.tile_tokens, ++tile_at)
-      if (tile_at < a.max_tiles) reinterpret_cast<int4*>(a.tiles)[tile_at] = make_int4(e, row_at + r, min(a.tile_tokens, c - r), 0);
-    row_at += c;
-    a.counts[e] = 0;
-  }
-  if (threadIdx.x == kWarps * 32 - 1) {
-    a.offsets[E] = row_at;
-    *a.num_tiles = min(tile_at, a.max_tiles);
-    a.counts[E] = 0;
-  }
+  finish_routing(a);
 }
 
 // One warp per (token, choice) pair.
@@ -209,19 +315,22 @@ simt_kernel(b200_moe_args a, int shared_blocks) {
   for (int i = 0; i < 4; ++i) {
     if (tr + i >= rows) continue;
     const int m = m0 + tr + i;
-    const float scale = GATED && !shared ? a.row_scale[m] : 1.f;
+    const float scale = GATED && !shared && !a.plain ? a.row_scale[m] : 1.f;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       if (n0 + tc + j >= N) continue;
       float v = acc[i][j];
-      if (GATED) v = gemm::clamped_glu(v * scale, up[i][j] * scale, shared ? a.shared_limit : a.limit, a.alpha);
+      if (GATED && a.plain)
+        v = v / (1.f + expf(-v)) * up[i][j];
+      else if (GATED)
+        v = gemm::clamped_glu(v * scale, up[i][j] * scale, shared ? a.shared_limit : a.limit, a.alpha);
       simt::store_as(y + static_cast<int64_t>(m) * N + n0 + tc + j, v);
     }
   }
 }
 
 static bool valid(const b200_moe_args* a) {
-  return a && a->num_tokens > 0 && a->width > 0 && a->experts > 0 && a->experts <= kMaxExperts && a->top > 0 && a->top <= a->experts &&
+  return a && a->num_tokens > 0 && a->width > 0 && a->experts > 0 && a->experts <= kMaxExperts && a->top > 0 && a->top <= a->experts + (a->plain ? a->identity : 0) &&
          a->top <= 64 && a->ff > 0 && a->ff % 64 == 0 && a->tile_tokens > 0 && a->max_tiles > 0 && a->pairs && a->offsets && a->tiles && a->num_tiles &&
          static_cast<int64_t>(a->num_tokens) * a->top < (1 << 30) && (!a->shared_up || (a->shared_ff > 0 && a->shared_ff % 64 == 0)) &&
          (a->dtype == B200_DTYPE_BF16 || a->dtype == B200_DTYPE_F32);
@@ -250,10 +359,10 @@ static int grouped(const b200_moe_args& a, bool up, cudaStream_t s) {
     p.K = up ? a.width : ff;
     p.y = static_cast<__nv_bfloat16*>(y);
     p.ldy = up ? ff : a.width;
-    p.gated = up ? gemm::kGatedClamped : 0;
+    p.gated = !up ? 0 : a.plain ? gemm::kGatedPlain : gemm::kGatedClamped;
     p.glu_limit = limit;
     p.glu_alpha = a.alpha;
-    p.row_scale = up ? scale : nullptr;
+    p.row_scale = up && !a.plain ? scale : nullptr;
   };
   fill(gp.routed, pairs, a.ff, up ? a.inter : a.y, a.limit, a.row_scale);
   if (with_shared) {
@@ -286,6 +395,21 @@ int b200_moe_route(const b200_moe_args* a, b200_stream_t stream) {
   if (!moe::valid(a) || !a->router || a->router_splits < 1 || a->router_ld < a->experts + (a->shared_gate ? 1 : 0) || !a->counts || !a->pair_weight)
     return B200_ERR_INVALID_ARGUMENT;
   const unsigned blocks = static_cast<unsigned>((a->num_tokens + moe::kWarps - 1) / moe::kWarps);
+  if (a->plain) {
+    const int columns = a->experts + a->identity, groups = a->groups;
+    if (a->identity < 0 || columns > moe::kMaxExperts || a->router_ld < columns || !a->correction || a->shared_gate || groups < 1 ||
+        columns % groups != 0 || a->keep_groups < 1 || a->keep_groups > groups || a->top > columns / groups * a->keep_groups)
+      return B200_ERR_INVALID_ARGUMENT;
+    const size_t bytes = static_cast<size_t>(moe::kWarps) * (columns + groups) * 4;
+    auto go = [&](auto zero) {
+      using T = decltype(zero);
+      static std::atomic<uint64_t> done{0};
+      if (ensure_dynamic_smem(moe::route_softmax_kernel<T>, moe::kWarps * 2 * moe::kMaxExperts * 4, done) != B200_OK)
+        return static_cast<int>(B200_ERR_LAUNCH);
+      return launch_pdl(moe::route_softmax_kernel<T>, dim3(blocks), dim3(moe::kWarps * 32), bytes, reinterpret_cast<cudaStream_t>(stream), *a);
+    };
+    return a->dtype == B200_DTYPE_F32 ? go(0.f) : go(__nv_bfloat16{});
+  }
   return launch_pdl(moe::route_kernel, dim3(blocks), dim3(moe::kWarps * 32), static_cast<size_t>(moe::kWarps) * a->experts * 4,
                     reinterpret_cast<cudaStream_t>(stream), *a);
 }

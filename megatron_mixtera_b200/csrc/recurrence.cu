@@ -2,6 +2,7 @@
 //
 //   Wkv    o = (S + diag(b) k v^T)^T r,   S <- diag(w) S + k v^T                     (w per key channel)
 //   Delta  S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q                 (g, beta per head)
+//   Memory S <- f S + i k v^T, n <- f n + i k, o = S^T q / max(|n . q|, floor)         (f, i, floor per head, from a running maximum)
 //
 // As in delta_rule.cu, the value channels (columns of S) do not talk to each other: a column's state lives in the registers of NI
 // lanes, everything is fp32 from the loads on with two key channels per instruction, and the state is stored
@@ -11,6 +12,10 @@
 //   decode_kernel  one token per row, a warp per (row, head), everything from the projections to the gated output
 //   scan_kernel    rows of any length, one CTA per (row, head, block of columns); other warps prepare the next 16 tokens
 //   finish_kernel  head norm, weight and gate behind the scan
+//   gates_kernel   Memory: the running maximum and the factors of every token of a step, a warp per (row, head)
+//
+// Memory's normaliser n is one more column of S whose value is always 1: the decode kernel treats it so; in the scan a warp of its own
+// carries it beside the columns of the first column block.
 #include "common.cuh"
 
 namespace b200 {
@@ -30,9 +35,14 @@ __device__ __forceinline__ float sigmoid(float x) { return 1.f / (1.f + expf(-x)
 __device__ __forceinline__ float silu(float x) { return x / (1.f + expf(-x)); }
 __device__ __forceinline__ float softplus(float x) { return log1pf(expf(-fabsf(x))) + fmaxf(x, 0.f); }
 
+template <typename Rule>
+__device__ __forceinline__ float output_gate(float x) {
+  return Rule::kKind == B200_RECURRENCE_MEMORY ? sigmoid(x) : silu(x);
+}
+
 // What one token brings: shared-memory vectors of DIM entries and a few scalars.
 struct Wkv {
-  static constexpr int kKind = B200_RECURRENCE_WKV;
+  static constexpr int kKind = B200_RECURRENCE_WKV, kMoreCols = 0;
   static constexpr int kVecs = 3, kScalars = 1;  // r, w, k | r . (b k)
   template <int NI, int I, int N, int STRIDE, int DIM>
   static __device__ __forceinline__ void step(f32x2 (&s)[N][I / 2], const float* vec, const float* scalar, const float (&v)[N], int ni,
@@ -64,7 +74,7 @@ struct Wkv {
 };
 
 struct Delta {
-  static constexpr int kKind = B200_RECURRENCE_DELTA;
+  static constexpr int kKind = B200_RECURRENCE_DELTA, kMoreCols = 0;
   static constexpr int kVecs = 2, kScalars = 3;  // q, k | g, beta, q . k
   template <int NI, int I, int N, int STRIDE, int DIM>
   static __device__ __forceinline__ void step(f32x2 (&s)[N][I / 2], const float* vec, const float* scalar, const float (&v)[N], int ni,
@@ -105,6 +115,60 @@ struct Delta {
     }
   }
 };
+
+struct Memory {
+  static constexpr int kKind = B200_RECURRENCE_MEMORY, kMoreCols = 1;
+  static constexpr int kVecs = 2, kScalars = 2;  // q, i k | f, e^-maximum
+  template <int NI, int I, int N, int STRIDE, int DIM>
+  static __device__ __forceinline__ void step(f32x2 (&s)[N][I / 2], const float* vec, const float* scalar, const float (&v)[N], int ni,
+                                              float (&o)[N]) {
+    f32x2 acc[N][2], vv[N];
+    const f32x2 keep = pack2(scalar[0], scalar[0]);
+#pragma unroll
+    for (int n = 0; n < N; ++n) {
+      acc[n][0] = acc[n][1] = 0ull;
+      vv[n] = pack2(v[n], v[n]);
+    }
+#pragma unroll
+    for (int q = 0; q < I / 4; ++q) {
+      const int i = (q * NI + ni) * 4;
+      const ulonglong2 a = piece(vec + i), k = piece(vec + DIM + i);
+#pragma unroll
+      for (int n = 0; n < N; ++n) {
+        f32x2& x = s[n][q * 2];
+        f32x2& y = s[n][q * 2 + 1];
+        x = fma2(keep, x, mul2(k.x, vv[n]));
+        y = fma2(keep, y, mul2(k.y, vv[n]));
+        acc[n][0] = fma2(a.x, x, acc[n][0]);
+        acc[n][1] = fma2(a.y, y, acc[n][1]);
+      }
+    }
+#pragma unroll
+    for (int n = 0; n < N; ++n) o[n] = lane_sum<NI, STRIDE>(sum2(acc[n][0]) + sum2(acc[n][1]));
+  }
+};
+
+// Log input and forget gates of (token, head) from the projection's partial sums.
+struct LogGates {
+  float i, f;
+};
+template <typename T>
+__device__ __forceinline__ LogGates log_gates(const b200_recurrence_args& a, int64_t t, int head) {
+  const T* bias = static_cast<const T*>(a.decay_bias);
+  const int64_t stride = static_cast<int64_t>(a.num_tokens) * a.z_ld;
+  const float* z = a.z + t * a.z_ld + head;
+  float zi = 0.f, zf = 0.f;
+#pragma unroll 4
+  for (int s = 0; s < a.z_splits; ++s) {
+    zi += z[s * stride];
+    zf += z[s * stride + a.heads];
+  }
+  zi += simt::to_f32(bias[head]);
+  zf += simt::to_f32(bias[a.heads + head]);
+  const float cap = a.gate_cap;
+  return {cap * tanhf(zi / cap), -softplus(-cap * tanhf(zf / cap))};
+}
+__device__ __forceinline__ float memory_below(float nq, float floor_) { return fmaxf(fabsf(nq), floor_) + 1e-6f; }
 
 // A lane owns channels [lane * EL, lane * EL + EL) while a token is prepared: one vector load each where the layout allows (VEC).
 // Addresses are clamped instead of branched over, so that the loads of several tokens are in flight together; channels past dim
@@ -253,7 +317,8 @@ decode_kernel(b200_recurrence_args a, int vpad, int rank_pad, int w2_stride, boo
       asm volatile("cp.async.commit_group;" ::: "memory");
     }
   }
-  const int64_t head_elems = static_cast<int64_t>(dim) * vdim;
+  const int cols = vdim + Rule::kMoreCols;
+  const int64_t head_elems = static_cast<int64_t>(dim) * cols;
   const int ni = lane % NI, group = lane / NI;
   const float* src = a.state + (static_cast<int64_t>(in >= 0 ? in : 0) * a.heads + head) * head_elems;
   float* dst_state = a.state + (static_cast<int64_t>(live ? out : 0) * a.heads + head) * head_elems;
@@ -261,7 +326,7 @@ decode_kernel(b200_recurrence_args a, int vpad, int rank_pad, int w2_stride, boo
 #pragma unroll
     for (int n = 0; n < N; ++n) {
       const int j = (pass * N + n) * D::kGroups + group;
-      if (in >= 0 && j < vdim) {
+      if (in >= 0 && j < cols) {
         delta::load_column<NI, I>(src + static_cast<int64_t>(j) * dim, dim, ni, full, s[n]);
       } else {
 #pragma unroll
@@ -308,6 +373,34 @@ decode_kernel(b200_recurrence_args a, int vpad, int rank_pad, int w2_stride, boo
           z[e] = fmaf(simt::to_f32(w2[static_cast<int64_t>(min(lane * EL + e, dim - 1)) * a.rank + q]), lora[q], z[e]);
     }
     put_wkv<DIM, EL>(vec, scalar, r, k, z, bonus, lane, dim);
+  } else if constexpr (Rule::kKind == B200_RECURRENCE_MEMORY) {
+    const int64_t t = min(row, a.num_rows - 1);
+    float q[EL], k[EL];
+    if (vec_k) {
+      load_channels<true, T, EL>(p + a.off_r + head * dim, lane, dim, q);
+      load_channels<true, T, EL>(p + a.off_k + head * dim, lane, dim, k);
+    } else {
+      load_channels<false, T, EL>(p + a.off_r + head * dim, lane, dim, q);
+      load_channels<false, T, EL>(p + a.off_k + head * dim, lane, dim, k);
+    }
+    clear_tail(q, lane, dim);
+    clear_tail(k, lane, dim);
+    for (int i = lane; i < vdim; i += 32) values[i] = simt::to_f32(p[a.off_v + head * vdim + i]);
+    const LogGates g = log_gates<T>(a, t, head);
+    const float before = in >= 0 ? a.top[static_cast<int64_t>(in) * a.heads + head] : 0.f, top = fmaxf(g.f + before, g.i);
+    const float write = expf(g.i - top), unit = 1.f / sqrtf(static_cast<float>(dim));
+#pragma unroll
+    for (int e = 0; e < EL; ++e) {
+      vec[lane * EL + e] = q[e] * unit;
+      vec[DIM + lane * EL + e] = k[e] * write;
+    }
+    if (lane == 0) {
+      values[vdim] = 1.f;
+      scalar[0] = expf(g.f + before - top);
+      scalar[1] = expf(-top);
+      if (live) a.top[static_cast<int64_t>(out) * a.heads + head] = top;
+    }
+    fetch(ahead, 1);
   } else {
     if (row < a.num_rows) {
       const int ratio = a.heads / a.kv_heads, kvh = head / ratio;
@@ -379,24 +472,24 @@ decode_kernel(b200_recurrence_args a, int vpad, int rank_pad, int w2_stride, boo
   auto run = [&](f32x2 (&s)[N][I / 2], int pass) {
     float v[N], o[N];
 #pragma unroll
-    for (int n = 0; n < N; ++n) v[n] = values[min((pass * N + n) * D::kGroups + group, vdim - 1)];
+    for (int n = 0; n < N; ++n) v[n] = values[min((pass * N + n) * D::kGroups + group, cols - 1)];
     Rule::template step<NI, I, N, 1, DIM>(s, vec, scalar, v, ni, o);
 #pragma unroll
     for (int n = 0; n < N; ++n) {
       const int j = (pass * N + n) * D::kGroups + group;
-      if (j < vdim) {
+      if (j < cols) {
         if (live) delta::store_column<NI, I>(dst_state + static_cast<int64_t>(j) * dim, dim, ni, full, s[n]);
-        if (ni == 0) osq = fmaf(o[n], o[n], osq);
+        if (ni == 0 && j < vdim) osq = fmaf(o[n], o[n], osq);
       }
     }
     __syncwarp();  // every lane of a column has its value
 #pragma unroll
     for (int n = 0; n < N; ++n) {
       const int j = (pass * N + n) * D::kGroups + group;
-      if (j < vdim && ni == 0) values[j] = o[n];
+      if (j < cols && ni == 0) values[j] = o[n];
     }
   };
-  const int passes = (vdim + D::kGroups * N - 1) / (D::kGroups * N);
+  const int passes = (cols + D::kGroups * N - 1) / (D::kGroups * N);
 #pragma unroll 1
   for (int pass = 0; pass < passes; pass += 2) {
     run(cur, pass);
@@ -404,12 +497,17 @@ decode_kernel(b200_recurrence_args a, int vpad, int rank_pad, int w2_stride, boo
     if (pass + 1 < passes) run(ahead, pass + 1);
     if (pass + 3 < passes) fetch(ahead, pass + 3);
   }
-  const float inv = 1.f / sqrtf(warp_sum(osq) / vdim + a.eps);
   __syncwarp();
-  T* dst = static_cast<T*>(a.out) + (static_cast<int64_t>(row) * a.heads + head) * vdim;
+  osq = warp_sum(osq) / vdim;
+  float inv = 1.f / sqrtf(osq + a.eps);
+  if constexpr (Rule::kKind == B200_RECURRENCE_MEMORY) {
+    const float unit = 1.f / memory_below(values[vdim], scalar[1]);
+    inv = unit / sqrtf(osq * unit * unit + a.eps) * a.out_scale;
+  }
+  T* dst = static_cast<T*>(a.out) + (a.out_ld > 0 ? row * a.out_ld + head * vdim : (static_cast<int64_t>(row) * a.heads + head) * vdim);
   const T* weight = static_cast<const T*>(a.norm_weight) + (a.norm_per_head ? head * vdim : 0);
   for (int i = lane; i < vdim; i += 32)
-    simt::store_as(dst + i, live ? values[i] * inv * simt::to_f32(weight[i]) * silu(simt::to_f32(p[a.off_g + head * vdim + i])) : 0.f);
+    simt::store_as(dst + i, live ? values[i] * inv * simt::to_f32(weight[i]) * output_gate<Rule>(simt::to_f32(p[a.off_g + head * vdim + i])) : 0.f);
 }
 
 // ---------------------------------------------------------------------------------------------------------------
@@ -423,7 +521,8 @@ struct ScanShape {  // COLS columns per CTA, N of them per thread, LANES lanes p
   static constexpr int kComputeThreads = COLS / N * NI;
   static constexpr int kComputeWarps = kComputeThreads / 32;
   static constexpr int kPrepWarps = kComputeWarps < 2 ? 2 : kComputeWarps;
-  static constexpr int kThreads = kComputeThreads + kPrepWarps * 32;
+  static constexpr int kNormAt = kComputeThreads + kPrepWarps * 32;            // Memory: the warp that carries n
+  static constexpr int kThreads = kNormAt + Rule::kMoreCols * 32;
   static constexpr int kGroups = COLS / N;
   static constexpr int kTokPerWarp = kScanTokens / kPrepWarps;
   static constexpr int kBatch = kTokPerWarp < 4 ? kTokPerWarp : 4;
@@ -449,6 +548,40 @@ scan_kernel(b200_recurrence_args a, bool vec_k) {
   if (n_tok <= 0) return;
   const int chunks = (n_tok + kScanTokens - 1) / kScanTokens;
 
+  if (Rule::kMoreCols > 0 && tid >= Sh::kNormAt) {
+    // ------------------------------- n: EL key channels per lane -------------------------------
+    const int in = a.state_in[row], out = a.state_out[row];
+    const bool carries = cb == 0;
+    const int64_t column = (static_cast<int64_t>(head) * (vdim + 1) + vdim) * dim, slot = static_cast<int64_t>(a.heads) * (vdim + 1) * dim;
+    float n[EL];
+#pragma unroll
+    for (int e = 0; e < EL; ++e)
+      n[e] = carries && static_cast<unsigned>(in) < static_cast<unsigned>(a.state_slots) && lane * EL + e < dim ? a.state[in * slot + column + lane * EL + e] : 0.f;
+    __syncthreads();  // chunk 0 is ready
+    for (int c = 0; c < chunks; ++c) {
+      const float* buf = smem + (c & 1) * Sh::kBufFloats;
+      const int cnt = carries ? min(kScanTokens, n_tok - c * kScanTokens) : 0;
+#pragma unroll 1
+      for (int tt = 0; tt < cnt; ++tt) {
+        const float* vec = buf + tt * Sh::kTokenFloats;
+        const float* scalar = vec + Rule::kVecs * DIM + COLS;
+        float nq = 0.f;
+#pragma unroll
+        for (int e = 0; e < EL; ++e) {
+          n[e] = fmaf(scalar[0], n[e], vec[DIM + lane * EL + e]);
+          nq = fmaf(vec[lane * EL + e], n[e], nq);
+        }
+        nq = warp_sum(nq);
+        if (lane == 0) a.below[static_cast<int64_t>(t_begin + c * kScanTokens + tt) * a.heads + head] = memory_below(nq, scalar[1]);
+      }
+      __syncthreads();  // chunk c has been read, chunk c + 1 is ready
+    }
+    if (carries && static_cast<unsigned>(out) < static_cast<unsigned>(a.state_slots))
+#pragma unroll
+      for (int e = 0; e < EL; ++e)
+        if (lane * EL + e < dim) a.state[out * slot + column + lane * EL + e] = n[e];
+    return;
+  }
   if (tid >= Sh::kComputeThreads) {
     // ------------------------------- preparing warps -------------------------------
     const int warp = (tid - Sh::kComputeThreads) >> 5;
@@ -465,16 +598,18 @@ scan_kernel(b200_recurrence_args a, bool vec_k) {
         bias[e] = simt::to_f32(static_cast<const T*>(a.decay_bias)[i]);
         bonus[e] = simt::to_f32(static_cast<const T*>(a.bonus)[i]);
       }
-    } else {
+    } else if constexpr (Rule::kKind == B200_RECURRENCE_DELTA) {
       decay_rate = simt::to_f32(static_cast<const T*>(a.decay_rate)[head]);
       decay_bias = simt::to_f32(static_cast<const T*>(a.decay_bias)[head]);
     }
+    const float unit = 1.f / sqrtf(static_cast<float>(dim));  // (Memory)
     for (int c = 0; c < chunks; ++c) {
       float* buf = smem + (c & 1) * Sh::kBufFloats;
 #pragma unroll 1
       for (int q0 = 0; q0 < Sh::kTokPerWarp; q0 += Sh::kBatch) {
         T xv[Sh::kBatch][VL], xa[Sh::kBatch], xb[Sh::kBatch];
         float xr[Sh::kBatch][EL], xk[Sh::kBatch][EL], xz[Sh::kBatch][EL];
+        float4 factors[Sh::kBatch];
         auto fetch = [&](auto vec_c) {  // no branches between the loads: all in flight together
           constexpr bool V = decltype(vec_c)::value;
 #pragma unroll
@@ -487,6 +622,12 @@ scan_kernel(b200_recurrence_args a, bool vec_k) {
               k = p + a.off_k + head * dim;
               v = p + a.off_v + head * vdim;
               load_channels<V, float, EL>(a.z + t * hd + head * dim, lane, dim, xz[q]);
+            } else if constexpr (Rule::kKind == B200_RECURRENCE_MEMORY) {
+              const T* p = proj + t * a.proj_ld;
+              r = p + a.off_r + head * dim;
+              k = p + a.off_k + head * dim;
+              v = p + a.off_v + head * vdim;
+              factors[q] = reinterpret_cast<const float4*>(a.gates)[t * a.heads + head];
             } else {
               const T* p = static_cast<const T*>(a.conv) + t * channels;
               r = p + kvh * dim;
@@ -534,6 +675,20 @@ scan_kernel(b200_recurrence_args a, bool vec_k) {
             float* at = vec + q * Sh::kTokenFloats;
             put_wkv<DIM, EL>(at, at + Rule::kVecs * DIM + COLS, xr[q], xk[q], z, bonus, lane, dim);
           }
+        } else if constexpr (Rule::kKind == B200_RECURRENCE_MEMORY) {
+#pragma unroll
+          for (int q = 0; q < Sh::kBatch; ++q) {
+            float* at = vec + q * Sh::kTokenFloats;
+#pragma unroll
+            for (int e = 0; e < EL; ++e) {
+              at[lane * EL + e] = xr[q][e] * unit;
+              at[DIM + lane * EL + e] = xk[q][e] * factors[q].y;
+            }
+            if (lane == 0) {
+              at[Rule::kVecs * DIM + COLS] = factors[q].x;
+              at[Rule::kVecs * DIM + COLS + 1] = factors[q].z;
+            }
+          }
         } else {
           float fa[Sh::kBatch], fb[Sh::kBatch];
 #pragma unroll
@@ -553,7 +708,7 @@ scan_kernel(b200_recurrence_args a, bool vec_k) {
   // --------------------------------- compute warps ---------------------------------
   const bool full = dim == DIM;
   const int in = a.state_in[row], out = a.state_out[row];
-  const int64_t head_elems = static_cast<int64_t>(dim) * vdim;
+  const int64_t head_elems = static_cast<int64_t>(dim) * (vdim + Rule::kMoreCols);
   const int ni = lane / ST, group = (tid >> 5) * ST + lane % ST;  // this thread's columns: cb * COLS + n * kGroups + group
   f32x2 s[N][I / 2];
 #pragma unroll
@@ -600,6 +755,14 @@ constexpr int kFinishUnits = 4;
 template <typename T, int LPH>
 __global__ void __launch_bounds__(256)
 finish_kernel(b200_recurrence_args a) {
+  // Memory: outputs are still to be divided, the gate is a plain sigmoid.
+  const bool memory = a.kind == B200_RECURRENCE_MEMORY;
+  auto scale_of = [&](float mean_sq, int64_t unit) {
+    if (!memory) return 1.f / sqrtf(mean_sq + a.eps);
+    const float b = 1.f / a.below[unit];
+    return b / sqrtf(mean_sq * b * b + a.eps) * a.out_scale;
+  };
+  auto gate_of = [&](float x) { return memory ? sigmoid(x) : silu(x); };
   pdl_launch_dependents();
   pdl_wait();
   const int dim = a.vdim;
@@ -607,6 +770,7 @@ finish_kernel(b200_recurrence_args a) {
   const T* proj = static_cast<const T*>(a.proj);
   const T* weight = static_cast<const T*>(a.norm_weight);
   T* out = static_cast<T*>(a.out);
+  const int64_t out_ld = a.out_ld > 0 ? a.out_ld : static_cast<int64_t>(heads) * dim;
   if constexpr (LPH > 0) {
     constexpr int kGroups = 256 / LPH;
     const int lane = threadIdx.x % LPH, i = min(lane * 4, dim - 4);
@@ -625,12 +789,13 @@ finish_kernel(b200_recurrence_args a) {
       float sq = lane * 4 < dim ? v[k][0] * v[k][0] + v[k][1] * v[k][1] + v[k][2] * v[k][2] + v[k][3] * v[k][3] : 0.f;
 #pragma unroll
       for (int o = LPH / 2; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
-      const float inv = 1.f / sqrtf(sq / dim + a.eps);
+      const uint32_t unit = first + k * kGroups;
+      const float inv = scale_of(sq / dim, min(unit, total - 1));
       float y[4];
 #pragma unroll
-      for (int e = 0; e < 4; ++e) y[e] = v[k][e] * inv * w[k][e] * silu(g[k][e]);
-      const uint32_t unit = first + k * kGroups;
-      if (lane * 4 < dim && unit < total) conv::store<T, 4>(out + static_cast<int64_t>(unit) * dim + i, y);
+      for (int e = 0; e < 4; ++e) y[e] = v[k][e] * inv * w[k][e] * gate_of(g[k][e]);
+      const uint32_t t = unit / heads;
+      if (lane * 4 < dim && unit < total) conv::store<T, 4>(out + t * out_ld + (unit - t * heads) * dim + i, y);
     }
     return;
   }
@@ -644,11 +809,45 @@ finish_kernel(b200_recurrence_args a) {
     const float* o = a.o_f32 + unit * dim;
     float sq = 0.f;
     for (int i = lane; i < dim; i += 32) sq += o[i] * o[i];
-    const float inv = 1.f / sqrtf(warp_sum(sq) / dim + a.eps);
+    const float inv = scale_of(warp_sum(sq) / dim, unit);
     for (int i = lane; i < dim; i += 32)
-      simt::store_as(out + unit * dim + i, o[i] * inv * simt::to_f32(weight[(a.norm_per_head ? at : 0) + i]) *
-                                               silu(simt::to_f32(proj[t * a.proj_ld + a.off_g + at + i])));
+      simt::store_as(out + t * out_ld + at + i, o[i] * inv * simt::to_f32(weight[(a.norm_per_head ? at : 0) + i]) *
+                                                    gate_of(simt::to_f32(proj[t * a.proj_ld + a.off_g + at + i])));
   }
+}
+
+// m_t = max(f_t + m_(t-1), i_t) is associative over (f, i) pairs: 32 tokens at a time by shuffles.
+template <typename T>
+__global__ void __launch_bounds__(256)
+gates_kernel(b200_recurrence_args a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int lane = threadIdx.x & 31, head = blockIdx.x * 8 + (threadIdx.x >> 5), row = blockIdx.y;
+  if (head >= a.heads) return;
+  const int t_begin = a.cu_tokens[row], n_tok = min(a.cu_tokens[row + 1], a.num_tokens) - t_begin;
+  const int in = a.state_in[row], out = a.state_out[row];
+  float carry = static_cast<unsigned>(in) < static_cast<unsigned>(a.state_slots) ? a.top[static_cast<int64_t>(in) * a.heads + head] : 0.f;
+  for (int t0 = 0; t0 < n_tok; t0 += 32) {
+    const int64_t t = t_begin + min(t0 + lane, n_tok - 1);
+    const LogGates g = log_gates<T>(a, t, head);
+    float f = g.f, i = g.i;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float fp = __shfl_up_sync(0xffffffffu, f, o), ip = __shfl_up_sync(0xffffffffu, i, o);
+      if (lane >= o) {
+        i = fmaxf(ip + f, i);
+        f += fp;
+      }
+    }
+    const float top = fmaxf(carry + f, i);
+    float before = __shfl_up_sync(0xffffffffu, top, 1);
+    if (lane == 0) before = carry;
+    if (t0 + lane < n_tok)
+      reinterpret_cast<float4*>(a.gates)[t * a.heads + head] = make_float4(expf(g.f + before - top), expf(g.i - top), expf(-top), 0.f);
+    carry = __shfl_sync(0xffffffffu, top, min(31, n_tok - 1 - t0));
+  }
+  if (n_tok > 0 && lane == 0 && static_cast<unsigned>(out) < static_cast<unsigned>(a.state_slots))
+    a.top[static_cast<int64_t>(out) * a.heads + head] = carry;
 }
 
 template <typename T>
@@ -668,19 +867,23 @@ lora_kernel(b200_recurrence_args a) {
 // ---------------------------------------------------------------------------------------------------------------
 static bool valid(const b200_recurrence_args* a) {
   return a && a->num_tokens > 0 && a->heads > 0 && a->heads <= 65535 && a->dim > 0 && a->dim <= 256 && a->vdim > 0 && a->vdim <= 1024 &&
-         (a->kind == B200_RECURRENCE_WKV || (a->kind == B200_RECURRENCE_DELTA && a->kv_heads > 0 && a->heads % a->kv_heads == 0)) &&
+         (a->kind == B200_RECURRENCE_WKV || a->kind == B200_RECURRENCE_MEMORY || (a->kind == B200_RECURRENCE_DELTA && a->kv_heads > 0 && a->heads % a->kv_heads == 0)) &&
          (a->dtype == B200_DTYPE_BF16 || a->dtype == B200_DTYPE_F32);
 }
 static bool valid_state(const b200_recurrence_args* a) {
   return a->proj && a->state && a->state_in && a->state_out && a->state_slots > 0 && aligned16(a->state) && a->decay_bias &&
-         (a->kind == B200_RECURRENCE_WKV ? a->bonus != nullptr : a->decay_rate != nullptr);
+         (a->kind == B200_RECURRENCE_WKV ? a->bonus != nullptr : a->kind == B200_RECURRENCE_DELTA ? a->decay_rate != nullptr : a->top != nullptr);
+}
+
+static bool valid_gates(const b200_recurrence_args* a) {
+  return a->z && a->z_splits >= 1 && a->z_ld >= 2 * a->heads && a->decay_bias && a->top && a->gate_cap > 0.f && a->state_slots > 0;
 }
 
 template <typename T, typename Rule, int DIM>
 static int launch_decode(const b200_recurrence_args& a, cudaStream_t s) {
   using D = DecodeShape<DIM>;
   const int vec = 16 / static_cast<int>(sizeof(T));
-  const int vpad = (a.vdim + 3) / 4 * 4;
+  const int vpad = (a.vdim + Rule::kMoreCols + 3) / 4 * 4;
   int rank_pad = 0, w2_stride = 0;
   size_t w2_bytes = 0;
   if (Rule::kKind == B200_RECURRENCE_WKV) {
@@ -697,7 +900,7 @@ static int launch_decode(const b200_recurrence_args& a, cudaStream_t s) {
   bool vec_k = a.dim % EL == 0 && a.proj_ld % 8 == 0 && aligned16(a.proj) && a.off_r % 8 == 0 && a.off_k % 8 == 0;
   if (Rule::kKind == B200_RECURRENCE_WKV)
     vec_k = vec_k && aligned16(a.decay_bias) && aligned16(a.bonus);
-  else
+  else if (Rule::kKind == B200_RECURRENCE_DELTA)
     vec_k = vec_k && aligned16(a.conv_filter) && aligned16(a.conv_state);
   const bool vec_v = vec_k && a.vdim % 4 == 0 && a.dim % 4 == 0;  // (then channels % 4 == 0)
   if (Rule::kKind == B200_RECURRENCE_DELTA) vec_k = vec_k && channels % EL == 0;
@@ -736,7 +939,7 @@ static int launch_scan(const b200_recurrence_args& a, cudaStream_t s) {
 template <typename T, typename Rule>
 static int scan_by_dim(const b200_recurrence_args& a, cudaStream_t s) {
   if (a.dim <= 32) return launch_scan<T, Rule, 32, 32, 1, 2, 1>(a, s);
-  if constexpr (Rule::kKind == B200_RECURRENCE_WKV) {
+  if constexpr (Rule::kKind != B200_RECURRENCE_DELTA) {
     if (a.dim <= 64) return launch_scan<T, Rule, 64, 64, 1, 2, 2>(a, s);
     // Two columns per thread on twice the lanes: half the shared-memory reads per product, the same state per thread.
     if (a.dim <= 128) return launch_scan<T, Rule, 128, 64, 2, 4, 2>(a, s);
@@ -748,10 +951,12 @@ static int scan_by_dim(const b200_recurrence_args& a, cudaStream_t s) {
 }
 template <typename T>
 static int decode_by_kind(const b200_recurrence_args& a, cudaStream_t s) {
+  if (a.kind == B200_RECURRENCE_MEMORY) return decode_by_dim<T, Memory>(a, s);
   return a.kind == B200_RECURRENCE_WKV ? decode_by_dim<T, Wkv>(a, s) : decode_by_dim<T, Delta>(a, s);
 }
 template <typename T>
 static int scan_by_kind(const b200_recurrence_args& a, cudaStream_t s) {
+  if (a.kind == B200_RECURRENCE_MEMORY) return scan_by_dim<T, Memory>(a, s);
   return a.kind == B200_RECURRENCE_WKV ? scan_by_dim<T, Wkv>(a, s) : scan_by_dim<T, Delta>(a, s);
 }
 
@@ -765,6 +970,7 @@ int b200_recurrence_decode(const b200_recurrence_args* a, b200_stream_t stream) 
   if (!rec::valid(a) || !rec::valid_state(a) || !a->norm_weight || !a->out || a->num_rows != a->num_tokens || a->num_rows > 65535)
     return B200_ERR_INVALID_ARGUMENT;
   if (a->kind == B200_RECURRENCE_WKV && (!a->lora || !a->w2 || a->rank <= 0 || a->rank > 4096)) return B200_ERR_INVALID_ARGUMENT;
+  if (a->kind == B200_RECURRENCE_MEMORY && !rec::valid_gates(a)) return B200_ERR_INVALID_ARGUMENT;
   if (a->kind == B200_RECURRENCE_DELTA && (!a->conv_filter || a->taps < 1 || (a->taps > 1 && !a->conv_state))) return B200_ERR_INVALID_ARGUMENT;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   return a->dtype == B200_DTYPE_F32 ? rec::decode_by_kind<float>(*a, s) : rec::decode_by_kind<__nv_bfloat16>(*a, s);
@@ -774,7 +980,9 @@ int b200_recurrence_scan(const b200_recurrence_args* a, b200_stream_t stream) {
   using namespace b200;
   if (!rec::valid(a) || !rec::valid_state(a) || !a->o_f32 || !a->cu_tokens || a->num_rows < 0 || a->num_rows > 65535)
     return B200_ERR_INVALID_ARGUMENT;
-  if (a->kind == B200_RECURRENCE_WKV ? (!a->z || a->z_splits < 1) : !a->conv) return B200_ERR_INVALID_ARGUMENT;
+  if (a->kind == B200_RECURRENCE_MEMORY && (!a->gates || !aligned16(a->gates) || !a->below)) return B200_ERR_INVALID_ARGUMENT;
+  if ((a->kind == B200_RECURRENCE_WKV && (!a->z || a->z_splits < 1)) || (a->kind == B200_RECURRENCE_DELTA && !a->conv))
+    return B200_ERR_INVALID_ARGUMENT;
   if (a->num_rows == 0) return B200_OK;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   return a->dtype == B200_DTYPE_F32 ? rec::scan_by_kind<float>(*a, s) : rec::scan_by_kind<__nv_bfloat16>(*a, s);
@@ -786,7 +994,8 @@ int b200_recurrence_finish(const b200_recurrence_args* a, b200_stream_t stream) 
     return B200_ERR_INVALID_ARGUMENT;
   const int64_t units = static_cast<int64_t>(a->num_tokens) * a->heads;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  const bool vec = a->vdim % 4 == 0 && a->vdim <= 128 && a->proj_ld % 4 == 0 && a->off_g % 4 == 0 && aligned16(a->proj) && aligned16(a->o_f32) &&
+  if (a->kind == B200_RECURRENCE_MEMORY && !a->below) return B200_ERR_INVALID_ARGUMENT;
+  const bool vec = a->vdim % 4 == 0 && a->vdim <= 128 && a->out_ld % 4 == 0 && a->proj_ld % 4 == 0 && a->off_g % 4 == 0 && aligned16(a->proj) && aligned16(a->o_f32) &&
                    aligned16(a->norm_weight) && aligned16(a->out);
   const int lanes = !vec ? 0 : a->vdim <= 64 ? 16 : 32;
   const int per_block = (lanes ? 256 / lanes : 8) * rec::kFinishUnits;
@@ -798,6 +1007,18 @@ int b200_recurrence_finish(const b200_recurrence_args* a, b200_stream_t stream) 
     return launch_pdl(rec::finish_kernel<T, 0>, grid, dim3(256), 0, s, *a);
   };
   return a->dtype == B200_DTYPE_F32 ? go(0.f) : go(__nv_bfloat16{});
+}
+
+int b200_recurrence_gates(const b200_recurrence_args* a, b200_stream_t stream) {
+  using namespace b200;
+  if (!rec::valid(a) || a->kind != B200_RECURRENCE_MEMORY || !rec::valid_gates(a) || !a->gates || !aligned16(a->gates) || !a->state_in ||
+      !a->state_out || !a->cu_tokens || a->num_rows < 0 || a->num_rows > 65535)
+    return B200_ERR_INVALID_ARGUMENT;
+  if (a->num_rows == 0) return B200_OK;
+  const dim3 grid((a->heads + 7) / 8, a->num_rows);
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (a->dtype == B200_DTYPE_F32) return launch_pdl(rec::gates_kernel<float>, grid, dim3(256), 0, s, *a);
+  return launch_pdl(rec::gates_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, *a);
 }
 
 int b200_recurrence_lora(const b200_recurrence_args* a, b200_stream_t stream) {

@@ -358,6 +358,10 @@ void hybrid(const Tensor& args, const Tensor& anchor, int64_t which) {
     case 18: ok(b200_moe_gather(struct_of<b200_moe_args>(args, "b200_moe_args"), s), "b200_moe_gather"); break;
     case 19: ok(b200_moe_up(struct_of<b200_moe_args>(args, "b200_moe_args"), s), "b200_moe_up"); break;
     case 20: ok(b200_moe_down(struct_of<b200_moe_args>(args, "b200_moe_args"), s), "b200_moe_down"); break;
+    case 21: ok(b200_recurrence_gates(struct_of<b200_recurrence_args>(args, "b200_recurrence_args"), s), "b200_recurrence_gates"); break;
+    case 22: ok(b200_rotate_append(struct_of<b200_rotate_append_args>(args, "b200_rotate_append_args"), s), "b200_rotate_append"); break;
+    case 23: ok(b200_stream_norm(struct_of<b200_stream_norm_args>(args, "b200_stream_norm_args"), s), "b200_stream_norm"); break;
+    case 24: ok(b200_swiglu(struct_of<b200_swiglu_args>(args, "b200_swiglu_args"), s), "b200_swiglu"); break;
     default: TORCH_CHECK(false, "b200_decode.hybrid: unknown kernel ", which);
   }
 }

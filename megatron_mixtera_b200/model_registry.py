@@ -9,22 +9,25 @@ from typing import Callable, Dict, Tuple
 import torch
 
 from . import checkpoint
-from .transformer.hybrid_config import (DeltaRuleConfig, ExpertConfig, GatedDeltaConfig, HybridConfig, HybridLayerConfig,
-                                        LatentAttentionConfig, MoeConfig, RotaryConfig, ShortConvAttentionConfig, WkvConfig,
-                                        YarnScaling)
+from .transformer.hybrid_config import (DeltaRuleConfig, DistanceBias, ExpertConfig, GatedDeltaConfig, GroupedAttentionConfig, HybridConfig,
+                                        HybridLayerConfig, LatentAttentionConfig, MatrixMemoryConfig, MoeConfig, RotaryConfig,
+                                        ShortConvAttentionConfig, SideBySideConfig, SoftmaxRouting, WkvConfig, YarnScaling)
 from .transformer.transformer_config import TransformerConfig
 
 
 # ---------------------------------------------------------------------------------------------------------------------
 # Zinurax
 # ---------------------------------------------------------------------------------------------------------------------
+def _rotary(rot: dict, halves: bool = False) -> RotaryConfig:
+    scaling = rot.get("scaling")
+    return RotaryConfig(base=float(rot["base"]), dims=rot["dims"], halves=halves,
+                        scaling=YarnScaling(**{k: float(scaling[k]) for k in ("factor", "original", "fast", "slow")}) if scaling else None)
+
+
 def _latent_attention_config(m: dict) -> LatentAttentionConfig:
-    rot, scaling = m["rot"], m["rot"].get("scaling")
     return LatentAttentionConfig(
         heads=m["heads"], dim=m["dim"], rot_dim=m["rot_dim"], vdim=m["vdim"], kv_rank=m["kv_rank"], scale=float(m["scale"]),
-        rot=RotaryConfig(base=float(rot["base"]), dims=rot["dims"],
-                         scaling=YarnScaling(**{k: float(scaling[k]) for k in ("factor", "original", "fast", "slow")}) if scaling else None),
-        window=(m.get("mask") or {}).get("size"), kv_from=m.get("kv_from"))
+        rot=_rotary(m["rot"]), window=(m.get("mask") or {}).get("size"), kv_from=m.get("kv_from"))
 
 
 def zinurax_config(config: dict, shapes: Dict[str, tuple], dtype: torch.dtype) -> HybridConfig:
@@ -92,6 +95,57 @@ def _build_fabivik(config: dict, shapes: Dict[str, tuple], dtype: torch.dtype, m
 
 
 # ---------------------------------------------------------------------------------------------------------------------
+# Lukarax
+# ---------------------------------------------------------------------------------------------------------------------
+def _grouped(m: dict, **kwargs) -> GroupedAttentionConfig:
+    mask = m.get("mask") or {}
+    return GroupedAttentionConfig(heads=m["heads"], kv_heads=m["kv_heads"], dim=m["dim"], vdim=m["vdim"], scale=float(m["scale"]),
+                                  window=mask.get("size"), keep_first=mask.get("keep_first") or 0, **kwargs)
+
+
+def lukarax_config(config: dict, shapes: Dict[str, tuple], dtype: torch.dtype) -> HybridConfig:
+    """``config.json`` -> `HybridConfig`; ``shapes`` (checkpoint tensor -> shape) gives what the file leaves to the tensors."""
+    layers = []
+    for i, layer in enumerate(config["layers"]):
+        m, mlp = layer["mixer"], layer.get("mlp")
+        if layer["type"] == "attention":
+            mixer = _grouped(m, rot=_rotary(m["rot"]), diff=float(m["diff"]), gate=True, kv_from=m.get("kv_from"))
+        elif layer["type"] == "attention_2":
+            mixer = _grouped(m, rot=_rotary(m["rot"], halves=True), unit_queries_keys=True, values_from_keys=True, biases=True, sink=True,
+                             softcap=float(m["softcap"]))
+        elif layer["type"] == "parallel":
+            left, right = m["left"], m["right"]
+            bias = DistanceBias(rows=shapes[f"l{i}.mix.left.rel"][0], longest=float(left["bias_max"]))
+            memory = MatrixMemoryConfig(heads=right["heads"], dim=right["dim"], vdim=right["vdim"], gate_cap=float(right["gate_cap"]))
+            mixer = SideBySideConfig((("left", _grouped(left, distance_bias=bias), float(m["left_scale"])),
+                                      ("right", memory, float(m["right_scale"]))))
+        else:
+            raise ValueError(f"layer {i}: unknown mixer {layer['type']!r}")
+        ff = moe = None
+        if mlp is not None and mlp["kind"] == "dense":
+            ff = mlp["ff"]
+        elif mlp is not None and mlp["kind"] == "moe":
+            r = mlp["router"]
+            groups = r.get("groups") or {"count": 1, "keep": 1}
+            moe = MoeConfig(experts=r["experts"], top=r["top"], expert=ExpertConfig(ff=mlp["expert"]["ff"]),
+                            routing=SoftmaxRouting(identity=r.get("identity") or 0, groups=groups["count"], keep_groups=groups["keep"],
+                                                   scale=float(r["scale"])))
+        elif mlp is not None:
+            raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+        layers.append(HybridLayerConfig(mixer=mixer, ffn_hidden_size=ff, moe=moe))
+    return HybridConfig(vocab_size=config["vocab"], hidden_size=config["width"], layers=tuple(layers), block="streams",
+                        streams=config.get("streams") or 0, gated_linear_unit=True, activation="silu",
+                        layernorm_epsilon=float(config["norm"]["eps"]), params_dtype=dtype,
+                        embedding_scale=float(config["embedding"]["scale"]))
+
+
+def _build_lukarax(config: dict, shapes: Dict[str, tuple], dtype: torch.dtype, max_sequence_length: int):
+    from .hybrid.stream_model import StreamHybridModel
+
+    return StreamHybridModel(lukarax_config(config, shapes, dtype), max_sequence_length)
+
+
+# ---------------------------------------------------------------------------------------------------------------------
 # GPTModel: config.json holds TransformerConfig fields under "transformer" and the model's own beside it
 # ---------------------------------------------------------------------------------------------------------------------
 def _build_gpt(config: dict, shapes: Dict[str, tuple], dtype: torch.dtype, max_sequence_length: int):
@@ -105,7 +159,7 @@ def _build_gpt(config: dict, shapes: Dict[str, tuple], dtype: torch.dtype, max_s
 
 
 Builder = Callable[[dict, Dict[str, tuple], torch.dtype, int], torch.nn.Module]
-ARCHITECTURES: Dict[str, Builder] = {"Fabivik": _build_fabivik, "Zinurax": _build_zinurax, "GPTModel": _build_gpt}
+ARCHITECTURES: Dict[str, Builder] = {"Fabivik": _build_fabivik, "Lukarax": _build_lukarax, "Zinurax": _build_zinurax, "GPTModel": _build_gpt}
 
 
 def load_model(folder: str, *, dtype: torch.dtype = torch.bfloat16, max_sequence_length: int) -> torch.nn.Module:

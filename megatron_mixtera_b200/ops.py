@@ -733,7 +733,7 @@ _OUT_NORM, _LATENT_APPEND, _LATENT_ATTENTION, _DELTA_DECODE, _DELTA_LORA, _DELTA
 # kernels that take an argument struct and nothing else (`struct_kernel`)
 _STRUCT_KERNELS = {name: 9 + i for i, name in enumerate((
     "residual_norm", "conv_silu", "conv_qkv", "token_shift", "recurrence_decode", "recurrence_scan", "recurrence_finish",
-    "recurrence_lora", "moe_route", "moe_gather", "moe_up", "moe_down"))}
+    "recurrence_lora", "moe_route", "moe_gather", "moe_up", "moe_down", "recurrence_gates", "rotate_append", "stream_norm", "swiglu"))}
 
 
 def dtype_code(dtype) -> int:
@@ -892,7 +892,7 @@ def separate_attention(args: AttentionArgs, dtype, *, units=None, num_units: int
         return
     nbytes = _lib.load().b200_paged_attention_workspace_bytes(args.num_tokens, args.num_q_heads, 64 if args.value_dim <= 64 else 128,
                                                               args.num_splits)
-    if nbytes:
+    if nbytes and args.maps != 2:  # (two maps: the caller's workspace)
         ws = _workspace.get(args._anchor.device, "attn", nbytes)
         args.workspace, args.workspace_bytes = ws.data_ptr(), ws.numel()
     paged_attention(args)
@@ -942,3 +942,67 @@ def residual_norm(hidden, pending: Optional[PendingRows], gammas, outs, *, eps: 
         _need(y, dtype, "out")
         a.gamma[i], a.y[i] = g.data_ptr(), y.data_ptr()
     struct_kernel("residual_norm", a, hidden)
+
+
+class PendingStreams:
+    """What still has to be written into the residual streams: scaled embeddings, or a sublayer's output with the weights that spread it."""
+
+    __slots__ = ("table", "ids", "table_scale", "partials", "bias", "experts", "mix", "gain")
+
+    def __init__(self, *, table=None, ids=None, table_scale: float = 1.0, partials: Optional[GemmPartials] = None, bias=None, experts=None,
+                 mix=None, gain=None):
+        self.table, self.ids, self.table_scale = table, ids, table_scale
+        self.partials, self.bias, self.experts, self.mix, self.gain = partials, bias, experts, mix, gain
+
+
+def stream_norm(hidden, pending: Optional[PendingStreams], *, blend=None, gamma=None, beta=None, out=None, eps: float = 1.0, row_index=None) -> None:
+    """Writes ``pending`` into the streams ``hidden`` [rows, streams, width]; out = layer norm of sum_s blend[s] hidden[:, s]."""
+    _need(hidden, F32, "hidden")
+    a = _lib.StreamNormArgs()
+    a.hidden, (a.source_rows, a.streams, a.width) = hidden.data_ptr(), hidden.shape
+    a.rows, a.eps = hidden.shape[0], eps
+    p = pending
+    dtype = gamma.dtype if gamma is not None else F32
+    if p is not None:
+        dtype = next((t.dtype for t in (gamma, p.table, p.bias, p.experts.rows if p.experts is not None else None) if t is not None), F32)
+    a.dtype = dtype_code(dtype)
+    if row_index is not None:
+        _need(row_index, torch.int64, "row_index")
+        a.row_index, a.rows = row_index.data_ptr(), row_index.numel()
+    if p is not None:
+        if p.table is not None:
+            _need(p.table, dtype, "table")
+            _need(p.ids, torch.int64, "ids")
+            a.table, a.ids, a.table_rows, a.table_scale = p.table.data_ptr(), p.ids.data_ptr(), p.table.shape[0], p.table_scale
+        else:
+            _need(p.mix, F32, "mix")
+            _need(p.gain, F32, "gain")
+            a.mix, a.out = p.mix.data_ptr(), p.gain.data_ptr()
+        if p.partials is not None:
+            a.partials, a.num_splits = partials_of(p.partials)
+        if p.bias is not None:
+            _need(p.bias, dtype, "bias")
+            a.branch_bias = p.bias.data_ptr()
+        e = p.experts
+        if e is not None:
+            a.expert_rows, a.expert_row_count, a.pairs, a.offsets = e.rows.data_ptr(), e.rows.shape[0], e.pairs.data_ptr(), e.offsets.data_ptr()
+            a.pair_weight, a.top, a.experts, a.identity = e.weights.data_ptr(), e.top, e.experts, e.identity
+            a.expert_input = e.input.data_ptr()
+    if blend is not None:
+        _need(blend, F32, "blend")
+        a.in_ = blend.data_ptr()
+    if out is not None:
+        _need(out, dtype, "out")
+        a.gamma, a.beta, a.y = gamma.data_ptr(), beta.data_ptr(), out.data_ptr()
+    struct_kernel("stream_norm", a, hidden)
+
+
+def swiglu(x):
+    """silu(gate) * up of x [rows, 2F] = [gate | up], in fp32 arithmetic; any width, bf16 or fp32."""
+    a = _lib.SwigluArgs()
+    _need(x, x.dtype, "x")
+    F = x.shape[-1] // 2
+    out = torch.empty((*x.shape[:-1], F), dtype=x.dtype, device=x.device)
+    a.in_, a.out, a.rows, a.width, a.dtype = x.data_ptr(), out.data_ptr(), x.numel() // (2 * F), F, dtype_code(x.dtype)
+    struct_kernel("swiglu", a, x)
+    return out

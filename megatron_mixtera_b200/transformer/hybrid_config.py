@@ -29,6 +29,7 @@ class RotaryConfig:
     base: float
     dims: int  # leading dimensions that turn, in interleaved pairs (2i, 2i + 1)
     scaling: Optional[YarnScaling] = None
+    halves: bool = False  # pairs are (i, i + dims / 2) instead
 
 
 @dataclass(frozen=True)
@@ -175,28 +176,175 @@ class GatedDeltaConfig:
         return {"state": ((self.heads, self.vdim, self.dim), torch.float32), **_conv_state(self.conv_channels, self.conv, dtype)}
 
 
-MixerConfig = Union[LatentAttentionConfig, DeltaRuleConfig, ShortConvAttentionConfig, WkvConfig, GatedDeltaConfig]
+@dataclass(frozen=True)
+class DistanceBias:
+    """A learned bias per head and distance class: one class per distance up to half the rows, logarithmic ones up to ``longest``."""
+
+    rows: int
+    longest: float
+
+    def row(self, distance: int) -> int:
+        half = self.rows // 2
+        if distance < half:
+            return distance
+        if self.longest <= half:
+            return self.rows - 1
+        return min(self.rows - 1, half + math.floor(math.log(distance / half) / math.log(self.longest / half) * (self.rows - half)))
+
+    def rows_by_distance(self) -> list:
+        """The row of every distance, up to the first one from which on it stays the last."""
+        out = [self.row(0)]
+        while out[-1] < self.rows - 1:
+            out.append(self.row(len(out)))
+        return out
+
+
+@dataclass(frozen=True)
+class GroupedAttentionConfig:
+    """Grouped-query attention with its parts as parameters.  ``diff`` makes it differential: two maps per head over the same values, out =
+    rms-normed (a1 - lambda a2) (1 - diff)."""
+
+    heads: int
+    kv_heads: int
+    dim: int                             # query / key dimensions per head (and map)
+    vdim: int                            # value dimensions per head
+    scale: float
+    window: Optional[int] = None         # keys seen, the token itself included; None: all earlier ones
+    keep_first: int = 0                  # keys at the sequence's start that a window never hides
+    rot: Optional[RotaryConfig] = None
+    unit_queries_keys: bool = False      # queries and keys divided by their root mean square after the rotation
+    values_from_keys: bool = False       # the values are the projected keys
+    biases: bool = False                 # on queries, keys and the output
+    softcap: Optional[float] = None
+    sink: bool = False                   # one more term per head in the softmax denominator
+    distance_bias: Optional[DistanceBias] = None
+    diff: Optional[float] = None
+    gate: bool = False                   # heads times sigmoid of a projection (differential attention)
+    kv_from: Optional[int] = None        # 0-based layer whose cached rows this layer reads instead of making its own
+
+    def __post_init__(self):
+        if self.heads % self.kv_heads:
+            raise ValueError("heads must be a multiple of kv_heads")
+        if self.window is not None and self.window < 1:
+            raise ValueError("a window holds at least the token itself")
+        if max(self.dim, self.vdim) > 256:
+            raise ValueError("head dimensions go up to 256")
+        if self.rot is not None and (self.rot.dims % 2 or not 0 <= self.rot.dims <= self.dim):
+            raise ValueError("rot.dims must be even and at most dim")
+        if self.diff is None and self.gate or self.diff is not None and (self.sink or self.distance_bias is not None):
+            raise ValueError("differential attention comes with a gate and without sinks or a distance bias")
+        if self.values_from_keys and (self.dim != self.vdim or self.diff is not None):
+            raise ValueError("values that are keys have their size, and one map")
+
+    @property
+    def maps(self) -> int:
+        return 1 if self.diff is None else 2
+
+    @property
+    def tensor_cores(self) -> bool:
+        """Head sizes that the tensor-core kernels take."""
+        return self.dim % 8 == 0 and self.vdim % 8 == 0 and max(self.dim, self.vdim) <= 128 and self.heads // self.kv_heads <= 16
+
+    @property
+    def row_width(self) -> int:
+        return self.kv_heads * (self.maps * self.dim + self.vdim)
+
+    def cached_row_width(self) -> int:
+        """Elements of a cached row: the keys of all heads, then the values."""
+        return self.row_width if self.kv_from is None else 0
+
+    def request_state(self, hidden_size: int, dtype: torch.dtype) -> Optional[dict]:
+        return None
+
+
+@dataclass(frozen=True)
+class MatrixMemoryConfig:
+    """Linear recurrence with scalar input and forget gates in the log domain, scaled by a running maximum, and a normaliser."""
+
+    heads: int
+    dim: int   # query / key channels per head
+    vdim: int  # value channels per head
+    gate_cap: float
+
+    def __post_init__(self):
+        if self.dim > 256 or self.vdim > 1023:
+            raise ValueError("recurrent heads have up to 256 key and 1023 value channels")
+
+    def cached_row_width(self) -> int:
+        return 0
+
+    def request_state(self, hidden_size: int, dtype: torch.dtype) -> Optional[dict]:
+        """The matrix, its normaliser as one more value channel, and the maximum."""
+        return {"state": ((self.heads, self.vdim + 1, self.dim), torch.float32), "top": ((self.heads,), torch.float32)}
+
+
+@dataclass(frozen=True)
+class SideBySideConfig:
+    """Mixers that read the same input and whose outputs are added up with constant factors."""
+
+    parts: Tuple[Tuple[str, Union[GroupedAttentionConfig, MatrixMemoryConfig], float], ...]  # (checkpoint prefix, mixer, factor)
+
+    def __post_init__(self):
+        if sum(m.cached_row_width() > 0 for _, m, _ in self.parts) > 1 or sum(m.request_state(1, torch.float32) is not None for _, m, _ in self.parts) > 1:
+            raise ValueError("one of the mixers caches rows, one keeps state")
+        if any(getattr(m, "biases", False) or getattr(m, "kv_from", None) is not None for _, m, _ in self.parts):
+            raise ValueError("mixers side by side have no biases and read no other layer's rows")
+
+    def cached_row_width(self) -> int:
+        return max(m.cached_row_width() for _, m, _ in self.parts)
+
+    def request_state(self, hidden_size: int, dtype: torch.dtype) -> Optional[dict]:
+        out = {}
+        for _, m, _ in self.parts:
+            out.update(m.request_state(hidden_size, dtype) or {})
+        return out or None
+
+
+MixerConfig = Union[LatentAttentionConfig, DeltaRuleConfig, ShortConvAttentionConfig, WkvConfig, GatedDeltaConfig, GroupedAttentionConfig,
+                    MatrixMemoryConfig, SideBySideConfig]
 
 
 @dataclass(frozen=True)
 class ExpertConfig:
-    """One gated feed-forward: g' sigmoid(alpha g') (u' + 1), g' = min(g, limit), u' clamped to [-limit, limit]."""
+    """One gated feed-forward: g' sigmoid(alpha g') (u' + 1), g' = min(g, limit), u' clamped to [-limit, limit]; without a limit silu(g) u."""
 
     ff: int
-    limit: float
+    limit: Optional[float] = None
     alpha: float = 1.702
+
+
+@dataclass(frozen=True)
+class SoftmaxRouting:
+    """Scores are a softmax; a learned correction takes part in the choice only; only the experts of the best groups can be chosen; the
+    chosen scores, divided by their sum and times ``scale``, weigh the experts' outputs.  The last ``identity`` router outputs are
+    experts whose output is their input."""
+
+    identity: int = 0
+    groups: int = 1
+    keep_groups: int = 1
+    scale: float = 1.0
 
 
 @dataclass(frozen=True)
 class MoeConfig:
     experts: int
-    top: int  # experts per token; their weights are their sigmoid scores
+    top: int  # experts per token; without ``routing`` their sigmoid scores weigh their inputs
     expert: ExpertConfig
     shared: Optional[ExpertConfig] = None  # runs for every token, times a gate of its own
+    routing: Optional[SoftmaxRouting] = None
 
     def __post_init__(self):
-        if not 1 <= self.top <= min(self.experts, 64) or self.experts > 1024:
-            raise ValueError("1 <= top <= experts, at most 64 of 1024")
+        r = self.routing
+        columns, reachable = self.experts, self.experts
+        if (r is None) != (self.expert.limit is not None) or (r is not None and self.shared is not None):
+            raise ValueError("softmax routing goes with plain gated experts and no shared one")
+        if r is not None:
+            columns = self.experts + r.identity
+            if r.identity < 0 or not 1 <= r.keep_groups <= r.groups or columns % r.groups:
+                raise ValueError("experts and identity experts form equal groups, at least one of which is kept")
+            reachable = columns // r.groups * r.keep_groups
+        if not 1 <= self.top <= min(reachable, 64) or not 1 <= columns <= 1024 or self.experts < 1:
+            raise ValueError("1 <= top <= experts that can be chosen, at most 64 of 1024")
 
 
 @dataclass(frozen=True)
@@ -226,7 +374,10 @@ class HybridConfig:
     # "output_norm": sublayers one after the other with norms on their outputs, embedding norm, tied head (`HybridModel`);
     # "parallel": mixer and feed-forward side by side on two norms of the same stream, scaled embedding, a head of its own
     # (`ParallelHybridModel`)
+    # "streams": sublayers one after the other with layer norms on their inputs, ``streams`` residual streams that every sublayer blends
+    # and mixes (0: one plain residual stream), scaled embedding, tied head (`StreamHybridModel`)
     block: str = "output_norm"
+    streams: int = 0
     embedding_scale: float = 1.0
     logit_scale: float = 1.0
 
@@ -240,12 +391,20 @@ class HybridConfig:
             mixing = [x.mixer for x in self.layers if isinstance(x.mixer, ShortConvAttentionConfig) and x.mixer.value_mix]
             if len({(m.kv_heads, m.vdim) for m in mixing}) > 1:
                 raise ValueError("layers whose values are mixed must agree in their number and size")
+        if self.streams > 16:
+            raise ValueError("at most 16 residual streams")
         for i, layer in enumerate(self.layers):
             m = layer.mixer
             src = getattr(m, "kv_from", None)
             if src is None:
                 continue
             own = self.layers[src].mixer if 0 <= src < i else None
+            if isinstance(m, GroupedAttentionConfig):
+                if not isinstance(own, GroupedAttentionConfig) or own.kv_from is not None:
+                    raise ValueError(f"layer {i} reads the rows of layer {src}, which is no earlier attention layer with its own")
+                if (own.kv_heads, own.maps, own.dim, own.vdim, own.rot) != (m.kv_heads, m.maps, m.dim, m.vdim, m.rot):
+                    raise ValueError(f"layers {src} and {i} share cached rows but differ in their shape or rotation")
+                continue
             if not isinstance(own, LatentAttentionConfig) or own.kv_from is not None:
                 raise ValueError(f"layer {i} reads the rows of layer {src}, which is no earlier latent-attention layer with its own")
             if (own.kv_rank, own.rot_dim, own.rot) != (m.kv_rank, m.rot_dim, m.rot):

@@ -32,7 +32,9 @@ class MLP(torch.nn.Module):
 
         # bf16 SwiGLU: fc1 and the activation run as one kernel on a weight whose gate / up rows are interleaved
         # per 64 (arranged in place when the weights are loaded)
-        if (config.gated_linear_unit and config.fp8 is None and getattr(config, "fuse_swiglu_into_fc1", True)
+        # 32-bit models and widths that the tensor-core kernels cannot address: a plain linear and an fp32 activation kernel
+        self.simt = config.gated_linear_unit and (config.params_dtype == torch.float32 or config.hidden_size % 8 != 0 or config.ffn_hidden_size % 8 != 0)
+        if (config.gated_linear_unit and not self.simt and config.fp8 is None and getattr(config, "fuse_swiglu_into_fc1", True)
                 and hasattr(self.linear_fc1, "forward_swiglu") and self.linear_fc1.bias is None
                 and (self.linear_fc1.weight.shape[0] // 2) % 64 == 0):
             self.linear_fc1.gate_up_interleaved = True
@@ -50,7 +52,16 @@ class MLP(torch.nn.Module):
         nvtx_range_pop(REF_MLP, "linear_fc2")
         return out
 
+    def load_gated(self, gate: torch.Tensor, up: torch.Tensor, down: torch.Tensor) -> None:
+        """Weights of a gated feed-forward as a checkpoint holds them."""
+        self.linear_fc1._layout_interleaved = False
+        self.linear_fc1.weight.data.copy_(torch.cat([gate, up]))
+        self.linear_fc2.weight.data.copy_(down)
+        self.linear_fc1.quantize_weights()
+
     def _fc1_and_activation(self, hidden_states):
+        if self.simt:
+            return ops.swiglu(self.linear_fc1(hidden_states)[0])
         if getattr(self.linear_fc1, "_layout_interleaved", False):
             return self.linear_fc1.forward_swiglu(hidden_states)
         if self.config.gated_linear_unit and self.linear_fc1.bias is None and hasattr(self.linear_fc1, "forward_gated"):

@@ -1,5 +1,6 @@
-"""Mixture of experts with sigmoid scores: every token runs its `top` best experts on its input times their scores, and a gated
-shared expert.  Tokens are sorted by expert on the device; the products of all experts are one grouped GEMM."""
+"""Mixture of experts: every token runs its `top` best experts - on its input times their sigmoid scores, beside a gated shared expert, or
+(`SoftmaxRouting`) with their softmax scores as weights of the outputs.  Tokens are sorted by expert on the device; the products of all experts are
+one grouped GEMM."""
 from __future__ import annotations
 
 import torch
@@ -28,13 +29,14 @@ def interleave_up(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
 
 class ExpertOutputs:
     """What `MixtureOfExperts` hands to the kernel that adds it to the stream: expert outputs sorted by expert, where a token's rows
-    lie among them, and the shared expert's rows with their gates."""
+    lie among them, and the shared expert's rows with their gates; under softmax routing the rows' weights, and the input for the pairs of
+    identity experts."""
 
-    __slots__ = ("rows", "pairs", "offsets", "top", "experts", "shared_rows", "shared_gate")
+    __slots__ = ("rows", "pairs", "offsets", "top", "experts", "shared_rows", "shared_gate", "weights", "identity", "input")
 
-    def __init__(self, rows, pairs, offsets, top, experts, shared_rows, shared_gate):
+    def __init__(self, rows, pairs, offsets, top, experts, shared_rows=None, shared_gate=None, weights=None, identity=0, input=None):
         self.rows, self.pairs, self.offsets, self.top, self.experts = rows, pairs, offsets, top, experts
-        self.shared_rows, self.shared_gate = shared_rows, shared_gate
+        self.shared_rows, self.shared_gate, self.weights, self.identity, self.input = shared_rows, shared_gate, weights, identity, input
 
 
 class MixtureOfExperts(torch.nn.Module):
@@ -47,8 +49,10 @@ class MixtureOfExperts(torch.nn.Module):
             return torch.nn.Parameter(torch.zeros(shape, dtype=config.params_dtype, device=_device()), requires_grad=False)
 
         self.ff = _padded(moe.expert.ff)
-        # router rows, then the shared expert's gate
-        self.router = param(-(-(moe.experts + (moe.shared is not None)) // 8) * 8, H)
+        # router rows (identity experts' included), then the shared expert's gate
+        self.columns = moe.experts + (moe.routing.identity if moe.routing is not None else 0)
+        self.router = param(-(-(self.columns + (moe.shared is not None)) // 8) * 8, H)
+        self.correction = param(self.columns) if moe.routing is not None else None
         self.up, self.down = param(moe.experts, 2 * self.ff, H), param(moe.experts, H, self.ff)
         self.shared_ff, self.shared_up, self.shared_down = 0, None, None
         if moe.shared is not None:
@@ -57,7 +61,9 @@ class MixtureOfExperts(torch.nn.Module):
 
     def checkpoint_tensors(self) -> dict:
         H, c = self.config.hidden_size, self.moe
-        out = {"router": (c.experts, H)}
+        out = {"router": (self.columns, H)}
+        if c.routing is not None:
+            out["correction"] = (self.columns,)
         parts = [(f"e{e}", c.expert.ff) for e in range(c.experts)]
         if c.shared is not None:
             parts.append(("shared", c.shared.ff))
@@ -68,7 +74,9 @@ class MixtureOfExperts(torch.nn.Module):
 
     def load(self, get) -> None:
         c, dev = self.moe, self.router.device
-        self.router.data[: c.experts].copy_(get("router"))
+        self.router.data[: self.columns].copy_(get("router"))
+        if self.correction is not None:
+            self.correction.data.copy_(get("correction"))
         for e in range(c.experts):
             self.up.data[e].copy_(interleave_up(get(f"e{e}.gate").to(dev), get(f"e{e}.up").to(dev)))
             self.down.data[e, :, : c.expert.ff].copy_(get(f"e{e}.down"))
@@ -90,7 +98,11 @@ class MixtureOfExperts(torch.nn.Module):
         pairs, simt = T * c.top, dt == torch.float32 or H % 8 != 0
         a = _lib.MoeArgs()
         a.num_tokens, a.width, a.experts, a.top, a.ff, a.shared_ff = T, H, c.experts, c.top, self.ff, self.shared_ff
-        a.limit, a.alpha, a.simt, a.dtype = c.expert.limit, c.expert.alpha, int(simt), ops.dtype_code(dt)
+        a.limit, a.alpha, a.simt, a.dtype = c.expert.limit or 0.0, c.expert.alpha, int(simt), ops.dtype_code(dt)
+        if c.routing is not None:
+            r = c.routing
+            a.plain, a.identity, a.groups, a.keep_groups, a.weight_scale = 1, r.identity, r.groups, r.keep_groups, r.scale
+            a.correction = self.correction.data_ptr()
         a.tile_tokens = self.tile_tokens(pairs, c.experts, simt)
         a.max_tiles = pairs // a.tile_tokens + min(c.experts, pairs)
         # bookkeeping in one block of 32-bit words: pairs | weights | row scales | shared gates | offsets | tiles | number of tiles
@@ -116,5 +128,7 @@ class MixtureOfExperts(torch.nn.Module):
         a.router_ld = self.router.shape[0]
         for kernel in ("moe_route", "moe_gather", "moe_up", "moe_down"):
             ops.struct_kernel(kernel, a, x)
+        if c.routing is not None:
+            return ExpertOutputs(rows, words, words[starts[4]:], c.top, c.experts, weights=words[starts[1]:], identity=c.routing.identity, input=x)
         gates = words[starts[3]: starts[3] + T].view(torch.float32) if c.shared is not None else None
         return ExpertOutputs(rows, words, words[starts[4]:], c.top, c.experts, shared_rows, gates)

@@ -74,6 +74,50 @@ class OutputNorm(torch.nn.Module):
         return ops.out_norm(hidden, self.weight, eps=self.eps, row_index=row_index)
 
 
+class StreamNorm(torch.nn.Module):
+    """Several 32-bit residual streams ``[T, streams, H]`` in place of one: what one sublayer left is written into all of them, and their blend
+    (``blend``) is layer-normed for the next, in one kernel.  ``mix`` [from, to] and ``gain`` say what the sublayer behind this norm does to
+    the streams (`left_by`).  ``plain`` without these weights: the streams' sum, and an ordinary residual sum."""
+
+    def __init__(self, config, hidden_size: int, eps: float, streams: int, plain: bool = False):
+        super().__init__()
+        dev = torch.device("cuda", torch.cuda.current_device()) if torch.cuda.is_available() else torch.device("cpu")
+        self.eps, self.streams, self.plain = eps, streams, plain
+
+        def param(value, dtype):
+            return torch.nn.Parameter(value.to(device=dev, dtype=dtype), requires_grad=False)
+
+        self.weight, self.bias = param(torch.ones(hidden_size), config.params_dtype), param(torch.zeros(hidden_size), config.params_dtype)
+        self.blend, self.gain = param(torch.ones(streams), torch.float32), param(torch.ones(streams), torch.float32)
+        self.mix = param(torch.eye(streams), torch.float32)
+
+    def checkpoint_tensors(self, norm: str, blends: str) -> dict:
+        """Checkpoint tensor name -> shape, with the norm under ``norm`` and the streams' weights under ``blends``."""
+        out = {norm: tuple(self.weight.shape), norm + ".b": tuple(self.weight.shape)}
+        if not self.plain:
+            out.update({blends + ".in": (self.streams,), blends + ".out": (self.streams,), blends + ".mix": (self.streams, self.streams)})
+        return out
+
+    def load(self, get, norm: str, blends: str) -> None:
+        self.weight.data.copy_(get(norm))
+        self.bias.data.copy_(get(norm + ".b"))
+        if not self.plain:
+            for dst, name in ((self.blend, ".in"), (self.gain, ".out"), (self.mix, ".mix")):
+                dst.data.copy_(get(blends + name))
+
+    def left_by(self, partials=None, bias=None, experts=None) -> "ops.PendingStreams":
+        """What the sublayer behind this norm computed, for the next norm to write into the streams."""
+        return ops.PendingStreams(partials=partials, bias=bias, experts=experts, mix=self.mix, gain=self.gain)
+
+    def forward(self, hidden, pending, row_index=None):
+        """Writes ``pending`` (a `PendingStreams`, or None) into ``hidden`` and returns the normed blend; with ``row_index`` (int64) only those
+        rows are computed and ``hidden`` stays as it is."""
+        rows = hidden.shape[0] if row_index is None else row_index.numel()
+        out = torch.empty((rows, hidden.shape[2]), dtype=self.weight.dtype, device=hidden.device)
+        ops.stream_norm(hidden, pending, blend=self.blend, gamma=self.weight, beta=self.bias, out=out, eps=self.eps, row_index=row_index)
+        return out
+
+
 class ParallelNorm(torch.nn.Module):
     """Everything a parallel block adds to the 32-bit residual stream and the RMS norms of the result, in one kernel.  ``outputs``
     norms of the same row (weights stored as the distance from one) feed the branches that run side by side."""

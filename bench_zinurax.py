@@ -173,7 +173,7 @@ def costs(s, T, visible_pairs, keys, zinurax, decode, requests):
     return out
 
 
-def kernel_table(rec, cost, hbm, tflops):
+def kernel_table(rec, cost, hbm, tflops, label=label):
     groups = {}
     for name, args in rec.calls:
         key, shape = label(name, args)
@@ -195,8 +195,9 @@ def kernel_table(rec, cost, hbm, tflops):
     return table
 
 
-def measure(kind, s, hbm, tflops, window, build=None, costs=costs):
-    """``kind`` "gpt": the GPT model; anything else: the design that ``build`` makes, with ``costs`` for its kernels."""
+def measure(kind, s, hbm, tflops, window, build=None, costs=costs, label=label):
+    """``kind`` "gpt": the GPT model; anything else: the design that ``build`` makes, with ``costs`` for its kernels, told apart by
+    ``label``."""
     requests, max_len = REQUESTS, CONTEXT + 64
     tokens = requests * (-(-max_len // 256) * 256) + PROMPTS * (PROMPT_LEN + 256)
     gpt = kind == "gpt"
@@ -218,7 +219,7 @@ def measure(kind, s, hbm, tflops, window, build=None, costs=costs):
             fwd()
         cost = costs(s, T, PROMPTS * per_prompt, T, not gpt, False, PROMPTS)
         out["prefill"] = {"tokens": T, "ms": round(us / 1e3, 3), "tokens_per_s": round(T / us * 1e6),
-                          "kernels": kernel_table(rec, cost, hbm, tflops)}
+                          "kernels": kernel_table(rec, cost, hbm, tflops, label)}
         del rec
         ctx.reset_attention_state()
         ctx.reset()
@@ -237,7 +238,7 @@ def measure(kind, s, hbm, tflops, window, build=None, costs=costs):
         keys = requests * (CONTEXT if gpt else min(CONTEXT, window))
         cost = costs(s, requests, keys, keys, not gpt, True, requests)
         out["decode"] = {"requests": requests, "context": CONTEXT, "us": round(us, 1), "tokens_per_s": round(requests / us * 1e6),
-                         "kernels": kernel_table(rec, cost, hbm, tflops)}
+                         "kernels": kernel_table(rec, cost, hbm, tflops, label)}
         del rec, graph
     return out
 

@@ -119,10 +119,13 @@ __device__ __forceinline__ int64_t query_offset(const Params& p, int h, int g) {
   if (FORM != kExtra) return static_cast<int64_t>(h) * p.q_group + g * p.q_head;
   return static_cast<int64_t>(h >> p.kshift) * p.q_group + (h & p.kshift) * p.dk + g * p.q_head;
 }
+__device__ __forceinline__ float capped(const Params& p, float qk) {
+  return p.cap_out * (1.f - __fdividef(2.f, 1.f + exp2f(qk * p.cap_in * (2.f * kLog2e))));
+}
 // Score in the log2 domain (without the mask).
 __device__ __forceinline__ float extra_score(const Params& p, float qk, const float* bias, int distance) {
   float v = qk * p.scale_log2;
-  if (p.cap_out > 0.f) v = p.cap_out * (1.f - __fdividef(2.f, 1.f + exp2f(qk * p.cap_in * (2.f * kLog2e))));
+  if (p.cap_out > 0.f) v = capped(p, qk);
   if (bias != nullptr) v = fmaf(__ldg(bias + min(max(distance, 0), p.bias_len - 1)), kLog2e, v);
   return v;
 }
@@ -754,6 +757,19 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
   int warp_first = min(kv_r[0] > 0 ? first_r[0] : 0x7fffffff, kv_r[1] > 0 ? first_r[1] : 0x7fffffff);
 #pragma unroll
   for (int o = 4; o < 32; o <<= 1) warp_first = min(warp_first, __shfl_xor_sync(0xffffffffu, warp_first, o));
+  // Keys that all of the warp's rows see: [all_first, all_kv); and where the distance bias is the same for all of them: in front of same_bias.
+  int all_kv = min(kv_r[0] > 0 ? kv_r[0] : 0x7fffffff, kv_r[1] > 0 ? kv_r[1] : 0x7fffffff), all_first = max(first_r[0], first_r[1]);
+  if (EXTRA)
+#pragma unroll
+    for (int o = 4; o < 32; o <<= 1) {
+      all_kv = min(all_kv, __shfl_xor_sync(0xffffffffu, all_kv, o));
+      all_first = max(all_first, __shfl_xor_sync(0xffffffffu, all_first, o));
+    }
+  const int same_bias = all_kv - p.bias_len;
+  float far_bias[2] = {0.f, 0.f};
+  if (EXTRA && p.bias != nullptr)
+#pragma unroll
+    for (int r = 0; r < 2; ++r) far_bias[r] = __ldg(bias_r[r] + p.bias_len - 1) * kLog2e;
 
   for (int i = 0; i < n_tiles; ++i) {
     const int s = i % kStages;
@@ -784,6 +800,28 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
       }
       // ---- causal mask + online softmax (log2 domain) ----
       float mx[2] = {-INFINITY, -INFINITY};
+      // (kExtra: the plain tile first - everything in sight, no bias or one bias per row)
+      const bool plain = EXTRA && tok0 >= all_first && tok0 + kTile <= all_kv && (p.bias == nullptr || tok0 + kTile <= same_bias + 1);
+      if (plain) {
+        if (p.cap_out > 0.f) {
+#pragma unroll
+          for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+            for (int c = 0; c < 4; ++c) sacc[nt][c] = capped(p, sacc[nt][c]);
+        } else {
+#pragma unroll
+          for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+            for (int c = 0; c < 4; ++c) sacc[nt][c] *= scale_log2;
+        }
+#pragma unroll
+        for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            sacc[nt][c] += far_bias[c >> 1];
+            mx[c >> 1] = fmaxf(mx[c >> 1], sacc[nt][c]);
+          }
+      } else
 #pragma unroll
       for (int nt = 0; nt < 8; ++nt) {
 #pragma unroll

@@ -12,7 +12,7 @@
 //   decode_kernel  one token per row, a warp per (row, head), everything from the projections to the gated output
 //   scan_kernel    rows of any length, one CTA per (row, head, block of columns); other warps prepare the next 16 tokens
 //   finish_kernel  head norm, weight and gate behind the scan
-//   gates_kernel   Memory: the running maximum and the factors of every token of a step, a warp per (row, head)
+//   gates_kernel   Memory: the running maximum and the factors of every token of a step, a CTA per (row, head)
 //
 // Memory's normaliser n is one more column of S whose value is always 1: the decode kernel treats it so; in the scan a warp of its own
 // carries it beside the columns of the first column block.
@@ -757,9 +757,9 @@ __global__ void __launch_bounds__(256)
 finish_kernel(b200_recurrence_args a) {
   // Memory: outputs are still to be divided, the gate is a plain sigmoid.
   const bool memory = a.kind == B200_RECURRENCE_MEMORY;
-  auto scale_of = [&](float mean_sq, int64_t unit) {
+  auto scale_of = [&](float mean_sq, float below) {
     if (!memory) return 1.f / sqrtf(mean_sq + a.eps);
-    const float b = 1.f / a.below[unit];
+    const float b = 1.f / below;
     return b / sqrtf(mean_sq * b * b + a.eps) * a.out_scale;
   };
   auto gate_of = [&](float x) { return memory ? sigmoid(x) : silu(x); };
@@ -775,7 +775,7 @@ finish_kernel(b200_recurrence_args a) {
     constexpr int kGroups = 256 / LPH;
     const int lane = threadIdx.x % LPH, i = min(lane * 4, dim - 4);
     const uint32_t first = blockIdx.x * kGroups * kFinishUnits + threadIdx.x / LPH;  // then kGroups apart
-    float v[kFinishUnits][4], g[kFinishUnits][4], w[kFinishUnits][4];
+    float v[kFinishUnits][4], g[kFinishUnits][4], w[kFinishUnits][4], below[kFinishUnits];
 #pragma unroll
     for (int k = 0; k < kFinishUnits; ++k) {
       const uint32_t unit = min(first + k * kGroups, total - 1), t = unit / heads;
@@ -783,6 +783,7 @@ finish_kernel(b200_recurrence_args a) {
       conv::load<float, 4>(a.o_f32 + static_cast<int64_t>(unit) * dim + i, v[k]);
       conv::load<T, 4>(proj + t * a.proj_ld + a.off_g + at + i, g[k]);
       conv::load<T, 4>(weight + (a.norm_per_head ? at : 0) + i, w[k]);
+      below[k] = memory ? a.below[unit] : 1.f;
     }
 #pragma unroll
     for (int k = 0; k < kFinishUnits; ++k) {
@@ -790,7 +791,7 @@ finish_kernel(b200_recurrence_args a) {
 #pragma unroll
       for (int o = LPH / 2; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
       const uint32_t unit = first + k * kGroups;
-      const float inv = scale_of(sq / dim, min(unit, total - 1));
+      const float inv = scale_of(sq / dim, below[k]);
       float y[4];
 #pragma unroll
       for (int e = 0; e < 4; ++e) y[e] = v[k][e] * inv * w[k][e] * gate_of(g[k][e]);
@@ -809,28 +810,41 @@ finish_kernel(b200_recurrence_args a) {
     const float* o = a.o_f32 + unit * dim;
     float sq = 0.f;
     for (int i = lane; i < dim; i += 32) sq += o[i] * o[i];
-    const float inv = scale_of(warp_sum(sq) / dim, unit);
+    const float inv = scale_of(warp_sum(sq) / dim, memory ? a.below[unit] : 1.f);
     for (int i = lane; i < dim; i += 32)
       simt::store_as(out + t * out_ld + at + i, o[i] * inv * simt::to_f32(weight[(a.norm_per_head ? at : 0) + i]) *
                                                     gate_of(simt::to_f32(proj[t * a.proj_ld + a.off_g + at + i])));
   }
 }
 
-// m_t = max(f_t + m_(t-1), i_t) is associative over (f, i) pairs: 32 tokens at a time by shuffles.
+// m_t = max(f_t + m_(t-1), i_t) is associative over (f, i) pairs: a CTA per (row, head) takes kGateTokens consecutive tokens per thread,
+// composes them, and scans the threads' pairs by shuffles and over the warps.
+constexpr int kGateThreads = 256, kGateTokens = 4;
 template <typename T>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(kGateThreads)
 gates_kernel(b200_recurrence_args a) {
+  __shared__ float2 warp_pair[kGateThreads / 32];
   pdl_launch_dependents();
   pdl_wait();
-  const int lane = threadIdx.x & 31, head = blockIdx.x * 8 + (threadIdx.x >> 5), row = blockIdx.y;
-  if (head >= a.heads) return;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, head = blockIdx.x, row = blockIdx.y;
   const int t_begin = a.cu_tokens[row], n_tok = min(a.cu_tokens[row + 1], a.num_tokens) - t_begin;
   const int in = a.state_in[row], out = a.state_out[row];
   float carry = static_cast<unsigned>(in) < static_cast<unsigned>(a.state_slots) ? a.top[static_cast<int64_t>(in) * a.heads + head] : 0.f;
-  for (int t0 = 0; t0 < n_tok; t0 += 32) {
-    const int64_t t = t_begin + min(t0 + lane, n_tok - 1);
-    const LogGates g = log_gates<T>(a, t, head);
-    float f = g.f, i = g.i;
+  for (int t0 = 0; t0 < n_tok; t0 += kGateThreads * kGateTokens) {
+    const int first = t0 + tid * kGateTokens;
+    LogGates g[kGateTokens];
+    float f = 0.f, i = -INFINITY;  // this thread's tokens as one pair
+#pragma unroll
+    for (int k = 0; k < kGateTokens; ++k) {
+      g[k].f = 0.f;  // past the end: nothing happens
+      g[k].i = -INFINITY;
+      if (first + k < n_tok) g[k] = log_gates<T>(a, t_begin + first + k, head);
+    }
+#pragma unroll
+    for (int k = 0; k < kGateTokens; ++k) {
+      i = fmaxf(i + g[k].f, g[k].i);
+      f += g[k].f;
+    }
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
       const float fp = __shfl_up_sync(0xffffffffu, f, o), ip = __shfl_up_sync(0xffffffffu, i, o);
@@ -839,14 +853,29 @@ gates_kernel(b200_recurrence_args a) {
         f += fp;
       }
     }
-    const float top = fmaxf(carry + f, i);
-    float before = __shfl_up_sync(0xffffffffu, top, 1);
-    if (lane == 0) before = carry;
-    if (t0 + lane < n_tok)
-      reinterpret_cast<float4*>(a.gates)[t * a.heads + head] = make_float4(expf(g.f + before - top), expf(g.i - top), expf(-top), 0.f);
-    carry = __shfl_sync(0xffffffffu, top, min(31, n_tok - 1 - t0));
+    if (lane == 31) warp_pair[warp] = make_float2(f, i);
+    float fp = __shfl_up_sync(0xffffffffu, f, 1), ip = __shfl_up_sync(0xffffffffu, i, 1);
+    if (lane == 0) fp = 0.f, ip = -INFINITY;
+    __syncthreads();
+    float top = carry;  // the maximum before this thread's first token
+#pragma unroll
+    for (int w = 0; w < kGateThreads / 32; ++w) {
+      const float2 p = warp_pair[w];
+      if (w < warp) top = fmaxf(top + p.x, p.y);
+      carry = fmaxf(carry + p.x, p.y);
+    }
+    top = fmaxf(top + fp, ip);
+#pragma unroll
+    for (int k = 0; k < kGateTokens; ++k) {
+      if (first + k >= n_tok) break;
+      const float before = top;
+      top = fmaxf(g[k].f + before, g[k].i);
+      reinterpret_cast<float4*>(a.gates)[static_cast<int64_t>(t_begin + first + k) * a.heads + head] =
+          make_float4(expf(g[k].f + before - top), expf(g[k].i - top), expf(-top), 0.f);
+    }
+    __syncthreads();
   }
-  if (n_tok > 0 && lane == 0 && static_cast<unsigned>(out) < static_cast<unsigned>(a.state_slots))
+  if (n_tok > 0 && tid == 0 && static_cast<unsigned>(out) < static_cast<unsigned>(a.state_slots))
     a.top[static_cast<int64_t>(out) * a.heads + head] = carry;
 }
 
@@ -939,7 +968,10 @@ static int launch_scan(const b200_recurrence_args& a, cudaStream_t s) {
 template <typename T, typename Rule>
 static int scan_by_dim(const b200_recurrence_args& a, cudaStream_t s) {
   if (a.dim <= 32) return launch_scan<T, Rule, 32, 32, 1, 2, 1>(a, s);
-  if constexpr (Rule::kKind != B200_RECURRENCE_DELTA) {
+  if constexpr (Rule::kKind == B200_RECURRENCE_MEMORY) {
+    if (a.dim <= 64) return launch_scan<T, Rule, 64, 64, 2, 4, 2>(a, s);
+    if (a.dim <= 128) return launch_scan<T, Rule, 128, 64, 1, 4, 1>(a, s);
+  } else if constexpr (Rule::kKind == B200_RECURRENCE_WKV) {
     if (a.dim <= 64) return launch_scan<T, Rule, 64, 64, 1, 2, 2>(a, s);
     // Two columns per thread on twice the lanes: half the shared-memory reads per product, the same state per thread.
     if (a.dim <= 128) return launch_scan<T, Rule, 128, 64, 2, 4, 2>(a, s);
@@ -1015,10 +1047,10 @@ int b200_recurrence_gates(const b200_recurrence_args* a, b200_stream_t stream) {
       !a->state_out || !a->cu_tokens || a->num_rows < 0 || a->num_rows > 65535)
     return B200_ERR_INVALID_ARGUMENT;
   if (a->num_rows == 0) return B200_OK;
-  const dim3 grid((a->heads + 7) / 8, a->num_rows);
+  const dim3 grid(a->heads, a->num_rows);
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  if (a->dtype == B200_DTYPE_F32) return launch_pdl(rec::gates_kernel<float>, grid, dim3(256), 0, s, *a);
-  return launch_pdl(rec::gates_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, *a);
+  if (a->dtype == B200_DTYPE_F32) return launch_pdl(rec::gates_kernel<float>, grid, dim3(rec::kGateThreads), 0, s, *a);
+  return launch_pdl(rec::gates_kernel<__nv_bfloat16>, grid, dim3(rec::kGateThreads), 0, s, *a);
 }
 
 int b200_recurrence_lora(const b200_recurrence_args* a, b200_stream_t stream) {

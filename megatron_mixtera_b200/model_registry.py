@@ -112,7 +112,7 @@ def lukarax_config(config: dict, shapes: Dict[str, tuple], dtype: torch.dtype) -
             mixer = _grouped(m, rot=_rotary(m["rot"]), diff=float(m["diff"]), gate=True, kv_from=m.get("kv_from"))
         elif layer["type"] == "attention_2":
             mixer = _grouped(m, rot=_rotary(m["rot"], halves=True), unit_queries_keys=True, values_from_keys=True, biases=True, sink=True,
-                             softcap=float(m["softcap"]))
+                             softcap=float(m["softcap"]) if m.get("softcap") else None)
         elif layer["type"] == "parallel":
             left, right = m["left"], m["right"]
             bias = DistanceBias(rows=shapes[f"l{i}.mix.left.rel"][0], longest=float(left["bias_max"]))

@@ -1,7 +1,7 @@
 """Plain CPU oracle of the Lukarax design.  TEST INFRASTRUCTURE ONLY.
 
-One slow function per mechanism, whole sequences only: no cache, no state between calls, no batching, experts one token at a
-time.  It shares no code with the shipped package.  Weights come as a dict of float tensors named as in a checkpoint, the
+One slow function per mechanism, whole sequences only: no cache, no state between calls, no batching.
+It shares no code with the shipped package.  Weights come as a dict of float tensors named as in a checkpoint, the
 configuration as the dict of its ``config.json``.
 """
 from __future__ import annotations
@@ -217,11 +217,13 @@ def route(z: Tensor, correction: Tensor, r: dict) -> tuple:
 
 
 def mixture(h: Tensor, w: Weights, p: str, m: dict) -> Tensor:
-    z, out = h @ w[p + ".router"].T, torch.zeros_like(h)
-    for t in range(h.shape[0]):
-        chosen, weight = route(z[t], w[p + ".correction"], m["router"])
-        for e, a in zip(chosen, weight):
-            out[t] += a * (gated(h[t], w, f"{p}.e{e}") if e < m["router"]["experts"] else h[t])
+    out, tokens_of = torch.zeros_like(h), {}
+    for t, z in enumerate(h @ w[p + ".router"].T):
+        for e, a in zip(*route(z, w[p + ".correction"], m["router"])):
+            tokens_of.setdefault(e, []).append((t, a))
+    for e, pairs in tokens_of.items():
+        t, a = [t for t, _ in pairs], torch.stack([a for _, a in pairs])
+        out[t] += a[:, None] * (gated(h[t], w, f"{p}.e{e}") if e < m["router"]["experts"] else h[t])
     return out
 
 

@@ -11,7 +11,7 @@ def dense(ff=72):
     return {"kind": "dense", "ff": ff}
 
 
-def experts(n=6, top=2, ff=40, identity=2, groups=(4, 2), scale=1.7):
+def experts(n=6, top=3, ff=40, identity=2, groups=(4, 2), scale=1.7):
     return {"kind": "moe", "expert": {"ff": ff},
             "router": {"experts": n, "identity": identity, "top": top, "scale": scale, "groups": {"count": groups[0], "keep": groups[1]}}}
 
@@ -71,9 +71,10 @@ CONFIGS = {
 }
 
 
-def weights(cfg, seed=0, gain=1.0):
+def weights(cfg, seed=0, gain=1.0, settled=False):
     """Random weights as a checkpoint holds them (bf16 values).  Linears keep the scale of their input; ``gain`` sharpens attention (through the
-    queries); forget gates spread the heads between short and long memory; the streams differ from one another."""
+    queries); forget gates spread the heads between short and long memory; the streams differ from one another.  ``settled``: which
+    experts are chosen is beyond the doubt of 16-bit rounding (the weights still differ from token to token)."""
     g = torch.Generator().manual_seed(seed)
 
     def mat(n, k, s=1.0):
@@ -129,6 +130,11 @@ def weights(cfg, seed=0, gain=1.0):
             r = mlp["router"]
             columns = r["experts"] + r["identity"]
             out[p + "router"], out[p + "correction"] = mat(columns, W, 1.5), vec(columns, -0.1, 0.1)
+            if settled:
+                out[p + "router"] *= 0.3
+                out[p + "correction"] = 0.5 * torch.randperm(columns, generator=g) - 1.0
+                if r["identity"] and r["top"] > 1:
+                    out[p + "correction"][-1] = 0.5 * columns
             parts = [(f"e{e}.", mlp["expert"]["ff"]) for e in range(r["experts"])]
         for name, ff in parts:
             out[p + name + "gate"], out[p + name + "up"], out[p + name + "down"] = mat(ff, W, 2.0), mat(ff, W), mat(W, ff)

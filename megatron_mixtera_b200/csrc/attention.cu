@@ -1018,6 +1018,71 @@ __global__ void __launch_bounds__(256) diff_combine_kernel(Params p, const void*
   }
 }
 
+// The same for bf16 and up to 4 * LANES value channels, a multiple of 4: LANES lanes per (token, head), kCombineUnits of them in turn with
+// all their loads in flight where there is one split.
+constexpr int kCombineUnits = 2;
+template <int LANES>
+__global__ void __launch_bounds__(256) diff_combine_vec_kernel(Params p, int stride, int splits) {
+  pdl_launch_dependents();
+  pdl_wait();
+  constexpr int kGroups = 256 / LANES;
+  const int lane = threadIdx.x % LANES, d = lane * 4, heads = p.nq / 2;
+  const bool mine = d < p.dv;
+  const uint32_t total = static_cast<uint32_t>(p.T) * heads;
+  const uint32_t first = blockIdx.x * kGroups * kCombineUnits + threadIdx.x / LANES;  // then kGroups apart
+  float4 a[kCombineUnits][2];
+  uint2 gate[kCombineUnits];
+#pragma unroll
+  for (int k = 0; k < kCombineUnits; ++k) {
+    const uint32_t unit = min(first + k * kGroups, total - 1), t = unit / heads, head = unit - t * heads;
+    const int kv_len = p.kv_len[t];
+    gate[k] = make_uint2(0u, 0u);
+    if (p.gate != nullptr && mine) gate[k] = *reinterpret_cast<const uint2*>(p.gate + t * p.gate_ld + head * p.dv + d);
+#pragma unroll
+    for (int m = 0; m < 2; ++m) {
+      a[k][m] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (kv_len <= 0 || !mine) continue;
+      const int64_t qh = static_cast<int64_t>(unit) * 2 + m;
+      const float* rows = p.ws_o + qh * splits * stride + d;
+      if (splits == 1) {
+        a[k][m] = *reinterpret_cast<const float4*>(rows);
+        continue;
+      }
+      const int base = first_tile_key(p, kv_len), keys = kv_len - base + kept_tiles(p, base) * kTile;
+      const int L = split_length(keys, splits, p.min_split), n_act = (keys + L - 1) / L;
+      const float* lse = p.ws_lse + qh * splits;
+      float mx = -INFINITY, wsum = 0.f;
+      for (int s = 0; s < n_act; ++s) mx = fmaxf(mx, lse[s]);
+      for (int s = 0; s < n_act; ++s) {
+        const float w = exp2f(lse[s] - mx);
+        const float4 v = *reinterpret_cast<const float4*>(rows + s * stride);
+        a[k][m].x = fmaf(w, v.x, a[k][m].x);
+        a[k][m].y = fmaf(w, v.y, a[k][m].y);
+        a[k][m].z = fmaf(w, v.z, a[k][m].z);
+        a[k][m].w = fmaf(w, v.w, a[k][m].w);
+        wsum += w;
+      }
+      const float inv = 1.f / wsum;
+      a[k][m] = make_float4(a[k][m].x * inv, a[k][m].y * inv, a[k][m].z * inv, a[k][m].w * inv);
+    }
+  }
+#pragma unroll
+  for (int k = 0; k < kCombineUnits; ++k) {
+    const uint32_t unit = first + k * kGroups, t = unit / heads, head = unit - t * heads;
+    float v[4] = {fmaf(-p.lambda, a[k][1].x, a[k][0].x), fmaf(-p.lambda, a[k][1].y, a[k][0].y), fmaf(-p.lambda, a[k][1].z, a[k][0].z),
+                  fmaf(-p.lambda, a[k][1].w, a[k][0].w)};
+    float sq = v[0] * v[0] + v[1] * v[1] + v[2] * v[2] + v[3] * v[3];
+#pragma unroll
+    for (int o = LANES / 2; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
+    const float inv = p.diff_scale / sqrtf(sq / p.dv + p.eps);
+    const float g[4] = {bf16_lo(gate[k].x), bf16_hi(gate[k].x), bf16_lo(gate[k].y), bf16_hi(gate[k].y)};
+#pragma unroll
+    for (int e = 0; e < 4; ++e) v[e] *= p.gate != nullptr ? inv / (1.f + expf(-g[e])) : inv;
+    if (mine && unit < total)
+      *reinterpret_cast<uint2*>(p.out + t * p.out_ld + head * p.dv + d) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
+  }
+}
+
 // Prefill / mixed steps: rotate k, then scatter k and v of every token into the pool.
 template <int D>
 __global__ void __launch_bounds__(128) rope_append_kernel(Params p) {
@@ -1183,6 +1248,14 @@ template <typename T>
 static int launch_diff_combine(const Params& p, const void* gate, void* out, int stride, int splits, cudaStream_t stream) {
   if (p.dv > 256) return B200_ERR_INVALID_ARGUMENT;
   const int64_t units = static_cast<int64_t>(p.T) * (p.nq / 2);
+  auto aligned8 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 7u) == 0; };
+  if (std::is_same<T, __nv_bfloat16>::value && p.dv % 4 == 0 && p.dv <= 128 && p.out_ld % 4 == 0 && p.gate_ld % 4 == 0 && aligned8(out) &&
+      aligned8(gate) && aligned16(p.ws_o) && units < (1 << 30)) {
+    const int lanes = p.dv <= 64 ? 16 : 32, per_block = 256 / lanes * kCombineUnits;
+    const dim3 grid(static_cast<unsigned>((units + per_block - 1) / per_block));
+    return lanes == 16 ? launch_pdl(diff_combine_vec_kernel<16>, grid, dim3(256), 0, stream, p, stride, splits)
+                       : launch_pdl(diff_combine_vec_kernel<32>, grid, dim3(256), 0, stream, p, stride, splits);
+  }
   return launch_pdl(diff_combine_kernel<T>, dim3(static_cast<unsigned>((units + 7) / 8)), dim3(256), 0, stream, p, gate, out, stride, splits);
 }
 

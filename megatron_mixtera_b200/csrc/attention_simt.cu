@@ -117,6 +117,8 @@ extern "C" int b200_attention_simt(const b200_attention_args* a, int dtype, b200
     p.lambda = a->lambda;
     p.diff_scale = a->diff_scale * a->out_scale;
     p.eps = a->eps;
+    p.gate = static_cast<const __nv_bfloat16*>(a->gate);
+    p.out = static_cast<__nv_bfloat16*>(a->out);
     p.gate_ld = a->gate_ld;
     p.out_ld = a->out_ld > 0 ? a->out_ld : static_cast<int64_t>(a->num_q_heads) * a->value_dim;
     return attn::launch_diff_combine<T>(p, a->gate, a->out, a->value_dim, 1, s);

@@ -752,11 +752,11 @@ scan_kernel(b200_recurrence_args a, bool vec_k) {
 
 // LPH lanes of 4 channels per (token, head), kFinishUnits units in turn with all their loads in flight (LPH == 0: a warp, any size).
 constexpr int kFinishUnits = 4;
-template <typename T, int LPH>
-__global__ void __launch_bounds__(256)
+// MEMORY: outputs are still to be divided, the gate is a plain sigmoid.
+template <typename T, int LPH, bool MEMORY>
+__global__ void __launch_bounds__(256, 4)
 finish_kernel(b200_recurrence_args a) {
-  // Memory: outputs are still to be divided, the gate is a plain sigmoid.
-  const bool memory = a.kind == B200_RECURRENCE_MEMORY;
+  constexpr bool memory = MEMORY;
   auto scale_of = [&](float mean_sq, float below) {
     if (!memory) return 1.f / sqrtf(mean_sq + a.eps);
     const float b = 1.f / below;
@@ -1032,13 +1032,17 @@ int b200_recurrence_finish(const b200_recurrence_args* a, b200_stream_t stream) 
   const int lanes = !vec ? 0 : a->vdim <= 64 ? 16 : 32;
   const int per_block = (lanes ? 256 / lanes : 8) * rec::kFinishUnits;
   const dim3 grid(static_cast<unsigned>((units + per_block - 1) / per_block));
-  auto go = [&](auto zero) {
+  auto go = [&](auto zero, auto memory) {
     using T = decltype(zero);
-    if (lanes == 16) return launch_pdl(rec::finish_kernel<T, 16>, grid, dim3(256), 0, s, *a);
-    if (lanes == 32) return launch_pdl(rec::finish_kernel<T, 32>, grid, dim3(256), 0, s, *a);
-    return launch_pdl(rec::finish_kernel<T, 0>, grid, dim3(256), 0, s, *a);
+    constexpr bool M = decltype(memory)::value;
+    if (lanes == 16) return launch_pdl(rec::finish_kernel<T, 16, M>, grid, dim3(256), 0, s, *a);
+    if (lanes == 32) return launch_pdl(rec::finish_kernel<T, 32, M>, grid, dim3(256), 0, s, *a);
+    return launch_pdl(rec::finish_kernel<T, 0, M>, grid, dim3(256), 0, s, *a);
   };
-  return a->dtype == B200_DTYPE_F32 ? go(0.f) : go(__nv_bfloat16{});
+  const std::true_type yes;
+  const std::false_type no;
+  if (a->kind == B200_RECURRENCE_MEMORY) return a->dtype == B200_DTYPE_F32 ? go(0.f, yes) : go(__nv_bfloat16{}, yes);
+  return a->dtype == B200_DTYPE_F32 ? go(0.f, no) : go(__nv_bfloat16{}, no);
 }
 
 int b200_recurrence_gates(const b200_recurrence_args* a, b200_stream_t stream) {

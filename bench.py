@@ -821,7 +821,7 @@ def main():
                          "pool with seeded noise (decode timing does not depend on the pool's contents)")
     ap.add_argument("--deadline", type=int, default=1500,
                     help="seconds after which a stuck run dumps every thread's stack and exits instead of waiting to be killed")
-    ap.add_argument("--design", default=None, choices=["zinurax", "fabivik", "lukarax"],
+    ap.add_argument("--design", default=None, choices=["zinurax", "fabivik", "lukarax", "maginex"],
                     help="time this design's prefill, decode and kernels beside the closest GPT model instead of the workload (one GPU)")
     ap.add_argument("--design-sizes", "--zinurax-sizes", default=None, help="with --design: sizes, comma-separated (default: all)")
     ap.add_argument("--design-window", "--zinurax-window", type=int, default=4096, help="with --design: attention window in tokens")

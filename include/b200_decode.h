@@ -423,7 +423,8 @@ typedef struct {
   int64_t pool_row_elems;
   /* separate == 2: the same layout with extras (zero / NULL: without).
    *   score = scale * q . k; with softcap > 0: softcap * tanh(score / softcap); plus distance_bias[head][min(distance, bias_len - 1)];
-   *   under a window positions [0, keep_first) stay visible; the softmax denominator also holds exp(sinks[head]); out * out_scale.
+   *   under a window positions [0, keep_first) stay visible; the softmax denominator also holds exp(sinks[head]); out * out_scale
+   *   * sigmoid(gate[t][head]) (maps < 2: a gate is one column per query head).
    * maps == 2: every head has two query / key vectors (head by head [map 1 | map 2], head_dim each) over one value vector; out =
    *   (a1 - lambda a2) / sqrt(mean(.^2) + eps) * diff_scale * sigmoid(gate) * out_scale of their attention outputs a1, a2 (gate NULL: 1; no
    *   sinks, no bias).  Needs a workspace of num_tokens * 2 * num_q_heads * num_splits * (d + 1) floats, d = 64 or 128 >= value_dim (on the
@@ -432,7 +433,7 @@ typedef struct {
   int64_t out_ld; /* elements between tokens' outputs (0: packed) */
   const float* distance_bias;
   const float* sinks;
-  const void* gate; /* [T][gate_ld]: num_q_heads * value_dim columns */
+  const void* gate; /* [T][gate_ld]: num_q_heads columns; maps == 2: num_q_heads * value_dim columns */
   int64_t gate_ld;
   float out_scale, softcap, lambda, diff_scale, eps;
   int32_t bias_len, keep_first, maps;
@@ -494,12 +495,14 @@ int b200_topp_probs_bf16(const void* logits, int64_t ld, float* probs, int rows,
 /* y[b][M, N] = act(x[b][M, K] * w[b][N, K]^T), `batch` independent products: batch b reads columns
  * [b * x_batch, b * x_batch + K) of x (row stride ldx), weight rows [b * N, (b + 1) * N), writes y + b * y_batch (row
  * stride ldy).  bf16 on tcgen05: K, ldx, x_batch multiples of 8, x and w 16-byte aligned; with batch == 1 the workspace of
- * b200_gemm_bf16_workspace_bytes, none otherwise. */
+ * b200_gemm_bf16_workspace_bytes, none otherwise.
+ * gate != NULL ([M][gate_ld], the type of x): outputs are multiplied with sigmoid of the gate in the column where they go, b * y_batch + n. */
 int b200_linear_bf16(const void* x, int64_t ldx, const void* w, void* y, int64_t ldy, int M, int N, int K, int act, int batch,
-                     int x_batch, int64_t y_batch, void* workspace, size_t workspace_bytes, b200_stream_t stream);
+                     int x_batch, int64_t y_batch, void* workspace, size_t workspace_bytes, const void* gate, int64_t gate_ld,
+                     b200_stream_t stream);
 /* The same product on the CUDA cores in true fp32, any sizes and strides.  y_f32 != 0: y is fp32 whatever `dtype` is. */
 int b200_linear_simt(const void* x, int64_t ldx, const void* w, void* y, int64_t ldy, int M, int N, int K, int act, int batch,
-                     int x_batch, int64_t y_batch, int dtype, int y_f32, b200_stream_t stream);
+                     int x_batch, int64_t y_batch, int dtype, int y_f32, const void* gate, int64_t gate_ld, b200_stream_t stream);
 
 /* Layer norm with a weight and no bias, (v - mean) / sqrt(variance + eps) * gamma, of a row v that is
  *   - the sum over `num_splits` of partials[s][row] (fp32, a linear's split-K partial sums), or
@@ -537,7 +540,10 @@ int b200_out_norm(const b200_out_norm_args* args, b200_stream_t stream);
  *   of the first rot_dims dimensions by the angle whose scaled cos / sin are rope_cos / rope_sin [position][rot_dims / 2].
  * b200_latent_attention: out[t][head][kv_rank] = sigmoid(gate) * sum_j softmax(scale * q . row_j) c_j over the keys j with
  *   0 <= position - j < window.  units == NULL: token t is the newest of row t, kv_seq_lengths[t] tokens long (0: padding,
- *   output undefined).  units: int32 [num_units][4] = {row, first token, tokens <= unit_tokens, 0}. */
+ *   output undefined).  units: int32 [num_units][4] = {row, first token, tokens <= unit_tokens, 0}.
+ * With `sinks` a head's softmax denominator also holds exp(sinks[head]) (unscaled, without key or value).
+ * Queries made in two steps: with q_latent_out b200_latent_append also writes the RMS-normed (q_norm_weight) query latent, columns
+ *   [q_latent_offset, + q_rank) of proj, and the queries themselves are `q` rows of another linear. */
 typedef struct b200_latent_args {
   const void* proj;     /* [T][proj_ld]: q (heads x (dim + rot_dim)) at column 0 */
   const void* norm_weight;
@@ -573,6 +579,13 @@ typedef struct b200_latent_args {
   void* key_rows;           /* [E][row_width]: the cached rows, in key order */
   const void* key_values;   /* [E][heads * (dim + vdim)]: W_uk c of all heads, then W_uv c of all heads */
   int32_t num_rows, num_keys, max_row_tokens, vdim;
+  const float* sinks;        /* [heads] or NULL */
+  const void* q;             /* [T][q_ld]: heads x (dim + rot_dim) unrotated queries; NULL: columns [0, ..) of proj */
+  const void* q_norm_weight; /* [q_rank] */
+  void* q_latent_out;        /* [T][q_rank] or NULL */
+  int64_t q_ld;
+  int32_t q_rank, q_latent_offset;
+  int32_t value_gates; /* b200_latent_prompt_attention: the gates are heads * vdim columns, one per value channel */
 } b200_latent_args;
 /* b200_latent_gather: key_rows[e] = the pool row of expanded key e.
  * b200_latent_prompt_attention: out[t][head][vdim] = sigmoid(gate) * sum_j softmax(scale * (q . k_j + q_rot . k_rot_j)) v_j, the same
@@ -629,11 +642,15 @@ int b200_attention_simt(const b200_attention_args* args, int dtype, b200_stream_
  * b200_residual_norm: h = hidden[row] (or table[ids[row]] * table_scale), plus
  *     sum over num_splits of partials[s][row]            (fp32, a linear's split-K partial sums)
  *   + branch[row]                                        (`dtype`)
- *   + sum over j < top of expert_rows[offsets[pairs[row][j].expert] + pairs[row][j].rank]   (`dtype`)
+ *   + sum over j < top of pair_weight[row][j] * expert_rows[offsets[pairs[row][j].expert] + pairs[row][j].rank]   (`dtype`; pair_weight
+ *     NULL: 1)
  *   + shared_gate[row] * shared_rows[row]                (`dtype`; shared_gate NULL: 1)
  * each part optional; then y_i[out row] = h / sqrt(mean(h^2) + eps) * (gain + gamma_i) * out_scale for up to two gammas.
  * row_index == NULL: out row = row, h is stored back to hidden.  row_index: out row r shows row row_index[r] of `source_rows`
- * rows; nothing is stored back. */
+ * rows; nothing is stored back.
+ * taps > 0 (no row_index; steps of one token per row): both outputs come from the norm with gamma_0, rounded to `dtype`, call it u, through a
+ * short causal filter over time each: y_i = u + sum_j filter_i[j] * u_(t - taps + 1 + j); earlier u from state slot state_in[row] (-1: zeros),
+ * the last taps - 1 go to state_out[row] (-1: nowhere), as in b200_conv_args. */
 typedef struct b200_residual_norm_args {
   const void* table;
   const int64_t* ids;
@@ -652,6 +669,13 @@ typedef struct b200_residual_norm_args {
   int64_t expert_row_count;
   int32_t num_splits, rows, source_rows, width, top, experts, dtype;
   float table_scale, eps, gain, out_scale;
+  const float* pair_weight;
+  const void* filter[2]; /* [taps][width] */
+  void* state;           /* [slot][taps - 1][width] (`dtype`) */
+  const int32_t* state_in;
+  const int32_t* state_out;
+  int64_t state_slots;
+  int32_t taps;
 } b200_residual_norm_args;
 int b200_residual_norm(const b200_residual_norm_args* args, b200_stream_t stream);
 
@@ -661,6 +685,7 @@ int b200_residual_norm(const b200_residual_norm_args* args, b200_stream_t stream
  * the same slot.  cu_tokens == NULL: one token per row (token t = row t); else row_of_token and cu_tokens [rows + 1].
  * At most 8 taps.
  * b200_conv_silu: out[t][c] = silu(y).
+ * b200_conv_add: out[t][c] = u_t + y, and with filter_2 a second output of the same inputs, out_2[t][c] = u_t + y_2.
  * b200_conv_qkv: channels = queries (heads x dim) | keys (kv_heads x dim) | values (kv_heads x vdim); queries and keys are RMS-normed
  *   per head (q_norm, k_norm [dim]); values become (1 - mix) y + mix * v_first_in when v_first_in is given, and are copied to
  *   v_first_out ([T][kv_heads * vdim]) when that is; queries go to out [T][heads * dim], keys and values to the pool. */
@@ -685,8 +710,11 @@ typedef struct b200_conv_args {
   int64_t proj_ld, state_slots, pool_row_elems;
   int32_t channels, taps, num_tokens, num_rows, heads, kv_heads, dim, vdim, chunk_size, num_chunks, dtype;
   float eps;
+  const void* filter_2; /* [taps][channels] */
+  void* out_2;
 } b200_conv_args;
 int b200_conv_silu(const b200_conv_args* args, b200_stream_t stream);
+int b200_conv_add(const b200_conv_args* args, b200_stream_t stream);
 int b200_conv_qkv(const b200_conv_args* args, b200_stream_t stream);
 
 /* Token shift: out[t][s][c] = x_t + (x_(t-1) - x_t) * mu[s][c] for `mixes` rows of mu; the previous token's row of a portion's first
@@ -798,10 +826,14 @@ typedef struct b200_moe_args {
   /* plain != 0: scores = softmax over experts + identity router columns; chosen by score + correction among the keep_groups of
    * `groups` equal groups of neighbours with the largest best choice score; pair_weight = chosen score / (their sum + 1e-20) *
    * weight_scale.  Columns [experts, experts + identity) are experts whose output is their input: their pairs count no rows.  Experts
-   * then are W_down (silu(W_gate x) * W_up x), unweighted: whoever adds the rows up applies pair_weight. */
+   * then are W_down (silu(W_gate x) * W_up x), unweighted: whoever adds the rows up applies pair_weight.
+   * plain == 2: the `correction` is a bias on the logits and part of the score, and the weights are the softmax over the chosen scores
+   * alone, times weight_scale.
+   * relu2 != 0: experts (the shared one too) are W_down (max(W_up x, 0))^2 without a gate; up weights [experts][ff][width]. */
   int32_t plain, identity, groups, keep_groups;
   const void* correction; /* [experts + identity] (`dtype`) */
   float weight_scale;
+  int32_t relu2;
 } b200_moe_args;
 int b200_moe_route(const b200_moe_args* args, b200_stream_t stream);
 int b200_moe_gather(const b200_moe_args* args, b200_stream_t stream);
@@ -813,7 +845,8 @@ int b200_moe_down(const b200_moe_args* args, b200_stream_t stream);
  * column off_q of proj), key vectors (k_vecs x dim at off_k) and value vectors (v_vecs x vdim at off_v), each plus its bias (NULL: none; value
  * columns may be the key columns).  Queries and keys turn in pairs (2i, 2i + 1), or (i, i + rot_dims / 2) with `halves`, on their
  * first rot_dims dimensions by the angle whose scaled cos / sin are rope_cos / rope_sin [position][rot_dims / 2]; with rms != 0 they are
- * then divided by their root mean square.  Queries go to q_out, keys and values to the pool.  Any of the counts may be 0. */
+ * then divided by their root mean square.  Queries go to q_out, keys and values to the pool.  Any of the counts may be 0.
+ * Values become (1 - mix) v + mix * v_first_in when v_first_in is given, and are copied to v_first_out (both [T][v_vecs * vdim]) when that is. */
 typedef struct b200_rotate_append_args {
   const void* proj; /* [T][proj_ld] */
   const void* q_bias;
@@ -831,6 +864,9 @@ typedef struct b200_rotate_append_args {
   int32_t off_q, off_k, off_v, q_vecs, k_vecs, v_vecs, dim, vdim, rot_dims, halves, rms, num_tokens, chunk_size, num_chunks, max_positions,
       dtype;
   float eps;
+  const void* v_first_in;
+  void* v_first_out;
+  const void* mix; /* one value */
 } b200_rotate_append_args;
 int b200_rotate_append(const b200_rotate_append_args* args, b200_stream_t stream);
 
@@ -873,6 +909,26 @@ typedef struct b200_swiglu_args {
   int32_t width, dtype;
 } b200_swiglu_args;
 int b200_swiglu(const b200_swiglu_args* args, b200_stream_t stream);
+
+/* Gated scan (minGRU), element by element: with z = sigmoid(x_z + z_bias), u = x_u + u_bias and the candidate u + 1/2 where u >= 0, else sigmoid(u):
+ *   S <- (1 - z) S + z * candidate,   out = S * silu(x_g).
+ * x_z, x_u, x_g are `width` columns each, at off_z, off_u, off_g of proj or of the fp32 partial sums [num_splits][T][proj_ld] in its
+ * place.  State [slot][width] fp32: read from state_in[row] (-1: zeros), written to state_out[row] (-1: nowhere), never the same slot.
+ * cu_tokens == NULL: one token per row (token t = row t); else row's tokens are [cu_tokens[row], cu_tokens[row + 1]). */
+typedef struct b200_gated_scan_args {
+  const void* proj; /* [T][proj_ld] */
+  const float* partials;
+  const void* z_bias;
+  const void* u_bias;
+  float* state;
+  const int32_t* state_in;
+  const int32_t* state_out;
+  const int32_t* cu_tokens;
+  void* out; /* [T][out_ld] */
+  int64_t proj_ld, out_ld, state_slots;
+  int32_t off_z, off_u, off_g, width, num_tokens, num_rows, num_splits, dtype;
+} b200_gated_scan_args;
+int b200_gated_scan(const b200_gated_scan_args* args, b200_stream_t stream);
 
 #ifdef __cplusplus
 }

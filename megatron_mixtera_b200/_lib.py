@@ -105,6 +105,8 @@ EXPORTED_SYMBOLS = (
     "b200_rotate_append",
     "b200_stream_norm",
     "b200_swiglu",
+    "b200_conv_add",
+    "b200_gated_scan",
 )
 
 
@@ -188,7 +190,9 @@ class LatentArgs(ctypes.Structure):
             "num_chunks", "chunk_size", "max_chunks_per_row", "max_positions", "window", "num_units", "unit_tokens",
             "num_splits", "dtype")] + [("scale", c_float), ("eps", c_float), ("q_stride", c_int32), ("q_rot_at", c_int32)] + [
         (n, c_void_p) for n in ("cu_tokens", "cu_keys", "key_start", "key_rows", "key_values")] + [
-        (n, c_int32) for n in ("num_rows", "num_keys", "max_row_tokens", "vdim")]
+        (n, c_int32) for n in ("num_rows", "num_keys", "max_row_tokens", "vdim")] + [
+        (n, c_void_p) for n in ("sinks", "q", "q_norm_weight", "q_latent_out")] + [
+        ("q_ld", c_int64)] + [(n, c_int32) for n in ("q_rank", "q_latent_offset", "value_gates")]
 
 
 class DeltaArgs(ctypes.Structure):
@@ -212,7 +216,8 @@ class ResidualNormArgs(ctypes.Structure):
     _fields_ = _fields((c_void_p, "table ids partials branch expert_rows pairs offsets shared_rows shared_gate row_index hidden")) + [
         ("gamma", c_void_p * 2), ("y", c_void_p * 2)] + _fields(
         (c_int64, "table_rows expert_row_count"), (c_int32, "num_splits rows source_rows width top experts dtype"),
-        (c_float, "table_scale eps gain out_scale"))
+        (c_float, "table_scale eps gain out_scale"), (c_void_p, "pair_weight")) + [("filter", c_void_p * 2)] + _fields(
+        (c_void_p, "state state_in state_out"), (c_int64, "state_slots"), (c_int32, "taps"))
 
 
 class ConvArgs(ctypes.Structure):
@@ -222,7 +227,8 @@ class ConvArgs(ctypes.Structure):
         (c_void_p, "proj filter state state_in state_out cu_tokens row_of_token out q_norm k_norm k_pool v_pool chunk_idx local_pos "
                    "v_first_in v_first_out mix"),
         (c_int64, "proj_ld state_slots pool_row_elems"),
-        (c_int32, "channels taps num_tokens num_rows heads kv_heads dim vdim chunk_size num_chunks dtype"), (c_float, "eps"))
+        (c_int32, "channels taps num_tokens num_rows heads kv_heads dim vdim chunk_size num_chunks dtype"), (c_float, "eps"),
+        (c_void_p, "filter_2 out_2"))
 
 
 class ShiftArgs(ctypes.Structure):
@@ -252,7 +258,7 @@ class MoeArgs(ctypes.Structure):
                    "inter y shared_inter shared_y"),
         (c_int32, "num_tokens width experts top ff shared_ff router_splits router_ld tile_tokens max_tiles simt dtype"),
         (c_float, "limit shared_limit alpha"), (c_int32, "plain identity groups keep_groups"), (c_void_p, "correction"),
-        (c_float, "weight_scale"))
+        (c_float, "weight_scale"), (c_int32, "relu2"))
 
 
 class RotateAppendArgs(ctypes.Structure):
@@ -262,7 +268,7 @@ class RotateAppendArgs(ctypes.Structure):
         (c_void_p, "proj q_bias k_bias v_bias rope_cos rope_sin token_to_pos chunk_idx local_pos q_out k_pool v_pool"),
         (c_int64, "proj_ld pool_row_elems"),
         (c_int32, "off_q off_k off_v q_vecs k_vecs v_vecs dim vdim rot_dims halves rms num_tokens chunk_size num_chunks max_positions dtype"),
-        (c_float, "eps"))
+        (c_float, "eps"), (c_void_p, "v_first_in v_first_out mix"))
 
 
 class StreamNormArgs(ctypes.Structure):
@@ -278,6 +284,13 @@ class SwigluArgs(ctypes.Structure):
     """Mirror of ``b200_swiglu_args``."""
 
     _fields_ = _fields((c_void_p, "in_ out"), (c_int64, "rows"), (c_int32, "width dtype"))
+
+
+class GatedScanArgs(ctypes.Structure):
+    """Mirror of ``b200_gated_scan_args``."""
+
+    _fields_ = _fields((c_void_p, "proj partials z_bias u_bias state state_in state_out cu_tokens out"), (c_int64, "proj_ld out_ld state_slots"),
+                       (c_int32, "off_z off_u off_g width num_tokens num_rows num_splits dtype"))
 
 
 class TpComm(ctypes.Structure):
@@ -428,9 +441,9 @@ def load() -> ctypes.CDLL:
     lib.b200_topp_probs_bf16.argtypes = [c_void_p, c_int64, c_void_p, c_int, c_int, c_float, c_float, c_void_p]
     lib.b200_argmax_f32.argtypes = [c_void_p, c_int64, c_void_p, c_int, c_int, c_void_p]
     lib.b200_linear_bf16.argtypes = [c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_int,
-                                     c_int64, c_void_p, c_size_t, c_void_p]
+                                     c_int64, c_void_p, c_size_t, c_void_p, c_int64, c_void_p]
     lib.b200_linear_simt.argtypes = [c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_int,
-                                     c_int64, c_int, c_int, c_void_p]
+                                     c_int64, c_int, c_int, c_void_p, c_int64, c_void_p]
     lib.b200_out_norm.argtypes = [POINTER(OutNormArgs), c_void_p]
     lib.b200_latent_attention_workspace_bytes.restype = c_size_t
     lib.b200_latent_attention_workspace_bytes.argtypes = [c_int, c_int, c_int, c_int]
@@ -441,7 +454,7 @@ def load() -> ctypes.CDLL:
         getattr(lib, name).argtypes = [POINTER(DeltaArgs), c_void_p]
     lib.b200_attention_simt.argtypes = [POINTER(AttentionArgs), c_int, c_void_p]
     lib.b200_residual_norm.argtypes = [POINTER(ResidualNormArgs), c_void_p]
-    for name in ("b200_conv_silu", "b200_conv_qkv"):
+    for name in ("b200_conv_silu", "b200_conv_add", "b200_conv_qkv"):
         getattr(lib, name).argtypes = [POINTER(ConvArgs), c_void_p]
     lib.b200_token_shift.argtypes = [POINTER(ShiftArgs), c_void_p]
     for name in ("b200_recurrence_decode", "b200_recurrence_scan", "b200_recurrence_finish", "b200_recurrence_lora",
@@ -452,6 +465,7 @@ def load() -> ctypes.CDLL:
     lib.b200_rotate_append.argtypes = [POINTER(RotateAppendArgs), c_void_p]
     lib.b200_stream_norm.argtypes = [POINTER(StreamNormArgs), c_void_p]
     lib.b200_swiglu.argtypes = [POINTER(SwigluArgs), c_void_p]
+    lib.b200_gated_scan.argtypes = [POINTER(GatedScanArgs), c_void_p]
     for name in EXPORTED_SYMBOLS:
         fn = getattr(lib, name)
         if fn.restype is c_int or name.startswith("b200_") and fn.restype not in (c_char_p, c_size_t):

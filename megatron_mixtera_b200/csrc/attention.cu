@@ -98,7 +98,7 @@ struct Params {
   int kshift;           // 1: KV "heads" are (head, map) pairs that share a value head
   int pad_dim;          // > 0: keys of both maps side by side; query row r fills columns [(r & 1) * pad_dim, + pad_dim) of dk
   float lambda, diff_scale, eps;
-  const __nv_bfloat16* gate;  // [T][gate_ld]: the difference is multiplied with sigmoid(gate)
+  const __nv_bfloat16* gate;  // [T][gate_ld]: the difference is multiplied with sigmoid(gate), or (diff 0) a head's output with its column's
   int64_t gate_ld;
 };
 
@@ -118,6 +118,10 @@ template <int FORM>
 __device__ __forceinline__ int64_t query_offset(const Params& p, int h, int g) {
   if (FORM != kExtra) return static_cast<int64_t>(h) * p.q_group + g * p.q_head;
   return static_cast<int64_t>(h >> p.kshift) * p.q_group + (h & p.kshift) * p.dk + g * p.q_head;
+}
+// Factor on a finished output (kExtra, one map).
+__device__ __forceinline__ float output_factor(const Params& p, int64_t t, int head) {
+  return p.gate == nullptr ? p.out_scale : p.out_scale / (1.f + expf(-__bfloat162float(p.gate[t * p.gate_ld + head])));
 }
 __device__ __forceinline__ float capped(const Params& p, float qk) {
   return p.cap_out * (1.f - __fdividef(2.f, 1.f + exp2f(qk * p.cap_in * (2.f * kLog2e))));
@@ -576,7 +580,7 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     }
     float o = lsum > 0.f ? acc / lsum : 0.f;
     if (p.num_splits == 1 && !(EXTRA && p.diff)) {
-      if (EXTRA) o *= p.out_scale;
+      if (EXTRA) o *= output_factor(p, t, head);
       store_output<DV>(p, t, head, d, o, ml + kConsumerWarps * 16, consumer_barrier);
     } else {
       p.ws_o[(qh * p.num_splits + split) * DV + d] = o;
@@ -904,7 +908,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
       l_run[r] = l_run[r] * top_scale + exp2f(sink - top);
     }
     float inv = l_run[r] > 0.f ? 1.f / l_run[r] : 0.f;  // a token that sees no key gets zeros, as flash-attn does
-    if (EXTRA) inv *= top_scale * p.out_scale;
+    if (EXTRA) inv *= top_scale * (p.diff ? p.out_scale : output_factor(p, tok_r[r], head));
     if (EXTRA && p.diff) {
       float* o32 = p.ws_o + (static_cast<int64_t>(tok_r[r]) * p.nq + head) * DV;
 #pragma unroll
@@ -946,7 +950,7 @@ __global__ void __launch_bounds__(D) combine_kernel(Params p) {
         acc += w * p.ws_o[(static_cast<int64_t>(qh) * p.num_splits + s) * D + d];
         wsum += w;
       }
-      o = acc / wsum * p.out_scale;
+      o = acc / wsum * output_factor(p, t, qh - t * p.nq);
     }
   }
   __shared__ float red[4];
@@ -1195,6 +1199,11 @@ static int fill_params(const b200_attention_args* a, Params& p) {
     p.bias_len = a->bias_len;
     p.sinks = a->sinks;
     p.out_scale = a->out_scale;
+    if (a->maps != 2) {
+      p.gate = static_cast<const __nv_bfloat16*>(a->gate);
+      p.gate_ld = a->gate_ld;
+      if (p.gate && p.gate_ld < p.nq) return B200_ERR_INVALID_ARGUMENT;
+    }
     if (a->softcap > 0.f) {
       p.cap_in = scale / a->softcap;
       p.cap_out = a->softcap * kLog2e;

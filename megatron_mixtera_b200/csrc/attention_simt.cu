@@ -80,6 +80,7 @@ attention_kernel(b200_attention_args a) {
     return;
   }
   if (extra) scale *= a.out_scale;
+  if (extra && a.gate != nullptr) scale /= 1.f + expf(-simt::to_f32(static_cast<const T*>(a.gate)[t * a.gate_ld + head]));
   T* out = static_cast<T*>(a.out) + (extra && a.out_ld > 0 ? t * a.out_ld + head * dv : unit * dv);
 #pragma unroll
   for (int e = 0; e < kMaxDim / 32; ++e)
@@ -99,6 +100,7 @@ extern "C" int b200_attention_simt(const b200_attention_args* a, int dtype, b200
   const bool extra = a->separate == attn::kExtra, diff = extra && a->maps == 2;
   if (a->maps == 2 && !extra) return B200_ERR_INVALID_ARGUMENT;
   if (extra && a->distance_bias && a->bias_len < 1) return B200_ERR_INVALID_ARGUMENT;
+  if (extra && !diff && a->gate && a->gate_ld < a->num_q_heads) return B200_ERR_INVALID_ARGUMENT;
   if (diff && (!a->workspace || a->workspace_bytes < static_cast<size_t>(a->num_tokens) * 2 * a->num_q_heads * a->value_dim * sizeof(float)))
     return B200_ERR_WORKSPACE;
   const int64_t units = static_cast<int64_t>(a->num_tokens) * a->num_q_heads * (diff ? 2 : 1);

@@ -59,6 +59,8 @@ struct Params {
   // in fp32; row_scale (NULL: 1) multiplies both products of a token first.  kGatedPlain: the same layout, y = g sigmoid(g) u.
   float glu_limit = 0.f, glu_alpha = 0.f;
   const float* row_scale = nullptr;
+  const __nv_bfloat16* gate = nullptr;  // [M][gate_ld]: outputs times sigmoid(gate) (whole-K units of ungated products)
+  int64_t gate_ld = 0;
 };
 constexpr int kGatedSilu = 1, kGatedClamped = 2, kGatedPlain = 3;  // Params::gated
 
@@ -80,6 +82,9 @@ __device__ __forceinline__ float apply_act(float v, int act) {
     v *= v;
   }
   return v;
+}
+__device__ __forceinline__ float apply_gate(const Params& p, float v, int64_t m, int64_t column) {
+  return p.gate == nullptr ? v : v * __fdividef(1.f, 1.f + __expf(-__bfloat162float(p.gate[m * p.gate_ld + column])));
 }
 
 // Sum of the split-K partial tiles: y[m, n] = bf16(sum_s partial[s][m][n]) (+ bias), splits added in order
@@ -152,7 +157,7 @@ __device__ __forceinline__ void epilogue_barrier() { asm volatile("bar.sync 2, 1
 // stores (whole-K units), or stores the fp32 partial tile for splitk_reduce_kernel.
 template <int BT>
 __device__ __forceinline__ void epilogue(const Params& p, uint32_t tmem_base, uint8_t* stage_smem, int n_tile, int split,
-                                         int m0, int m_end, __nv_bfloat16* __restrict__ y) {
+                                         int m0, int m_end, __nv_bfloat16* __restrict__ y, int64_t gate_column = 0) {
   const int tid = threadIdx.x;
   const int warp = tid >> 5;
   const int lane = tid & 31;
@@ -242,6 +247,7 @@ __device__ __forceinline__ void epilogue(const Params& p, uint32_t tmem_base, ui
           for (int j = 0; j < 32; ++j) {
             float v = __uint_as_float(r[j]);
             if (p.bias != nullptr) v = bf16_round(v) + b;  // bias is added to the bf16-rounded product
+            if (p.gate != nullptr) v = apply_gate(p, v, min(m0 + h0 + c0 + j, m_end - 1), gate_column + n);
             tile[(c0 + j) * kTileN + warp * 32 + lane] = __float2bfloat16_rn(apply_act(v, p.act));
           }
         }
@@ -268,7 +274,7 @@ __device__ __forceinline__ void epilogue(const Params& p, uint32_t tmem_base, ui
               float v = __uint_as_float(r[j]);
               // bias is added to the bf16-rounded product, as `matmul(x, w.t()) + bias` does
               if (p.bias != nullptr) v = bf16_round(v) + b;
-              y[static_cast<int64_t>(m) * p.ldy + n] = __float2bfloat16_rn(apply_act(v, p.act));
+              y[static_cast<int64_t>(m) * p.ldy + n] = __float2bfloat16_rn(apply_gate(p, apply_act(v, p.act), m, gate_column + n));
             }
           }
         }
@@ -422,7 +428,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
   mbar_wait_bounded(accum_bar, 0, abort_flag, kStatusGemmTimeout);
   tcgen05_fence_after_sync();
 
-  epilogue<BT>(p, tmem_base, smem, n_tile, split, m0, p.M, p.y + batch * p.y_batch);
+  epilogue<BT>(p, tmem_base, smem, n_tile, split, m0, p.M, p.y + batch * p.y_batch, batch * p.y_batch);
 
   tcgen05_fence_before_sync();
   __syncthreads();
@@ -632,7 +638,8 @@ template <int BT>
 static int launch(const void* x, int64_t ldx, const void* w, const void* bias, void* y, int64_t ldy, int M, int N,
                   int K, void* workspace, size_t workspace_bytes, cudaStream_t stream, bool cache_maps = true,
                   float* partials_out = nullptr, size_t partials_bytes = 0, int* splits_out = nullptr,
-                  bool gated = false, int act = B200_ACT_NONE, int batch = 1, int x_batch = 0, int64_t y_batch = 0) {
+                  bool gated = false, int act = B200_ACT_NONE, int batch = 1, int x_batch = 0, int64_t y_batch = 0,
+                  const void* gate = nullptr, int64_t gate_ld = 0) {
   using C = Config<BT>;
   const uint64_t wd[2] = {static_cast<uint64_t>(K), static_cast<uint64_t>(N) * batch};
   const uint64_t ws[1] = {static_cast<uint64_t>(K) * 2};
@@ -656,7 +663,7 @@ static int launch(const void* x, int64_t ldx, const void* w, const void* bias, v
   const int n_tiles = (N + kTileN - 1) / kTileN;
   const int m_blocks = (M + BT - 1) / BT;
   const int num_kb = (K + kTileK - 1) / kTileK;
-  const int splits = batch > 1 ? 1 : choose_splits(n_tiles * m_blocks, num_kb);
+  const int splits = batch > 1 || gate != nullptr ? 1 : choose_splits(n_tiles * m_blocks, num_kb);
   Params p;
   p.bias = static_cast<const __nv_bfloat16*>(bias);
   p.y = static_cast<__nv_bfloat16*>(y);
@@ -674,6 +681,8 @@ static int launch(const void* x, int64_t ldx, const void* w, const void* bias, v
   p.m_blocks = m_blocks;
   p.x_batch = x_batch;
   p.y_batch = y_batch;
+  p.gate = static_cast<const __nv_bfloat16*>(gate);
+  p.gate_ld = gate_ld;
   if (static_cast<int64_t>(m_blocks) * batch > 65535) return B200_ERR_INVALID_ARGUMENT;
   if (gated && (splits != 1 || partials_out != nullptr)) return B200_ERR_INVALID_ARGUMENT;
   if (partials_out != nullptr) {
@@ -781,20 +790,22 @@ int b200_gemm_bf16(const void* x, int64_t ldx, const void* w, const void* bias, 
 }
 
 int b200_linear_bf16(const void* x, int64_t ldx, const void* w, void* y, int64_t ldy, int M, int N, int K, int act, int batch,
-                     int x_batch, int64_t y_batch, void* workspace, size_t workspace_bytes, b200_stream_t stream) {
+                     int x_batch, int64_t y_batch, void* workspace, size_t workspace_bytes, const void* gate, int64_t gate_ld,
+                     b200_stream_t stream) {
   using namespace b200;
   if (!x || !w || !y || M <= 0 || N <= 0 || K <= 0 || batch <= 0 || act < B200_ACT_NONE || act > B200_ACT_RELU2)
     return B200_ERR_INVALID_ARGUMENT;
   if (batch > 1 && (x_batch <= 0 || y_batch <= 0 || (batch - 1) * static_cast<int64_t>(x_batch) + K > ldx))
     return B200_ERR_INVALID_ARGUMENT;
   if (K % 8 != 0 || ldx % 8 != 0 || x_batch % 8 != 0 || ldx < K || ldy < N) return B200_ERR_ALIGNMENT;
+  if (gate && gate_ld < (batch - 1) * y_batch + N) return B200_ERR_INVALID_ARGUMENT;
   if (!aligned16(x) || !aligned16(w)) return B200_ERR_ALIGNMENT;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   switch (gemm::pick_bt(M)) {
-    case 32: return gemm::launch<32>(x, ldx, w, nullptr, y, ldy, M, N, K, workspace, workspace_bytes, s, true, nullptr, 0, nullptr, false, act, batch, x_batch, y_batch);
-    case 64: return gemm::launch<64>(x, ldx, w, nullptr, y, ldy, M, N, K, workspace, workspace_bytes, s, true, nullptr, 0, nullptr, false, act, batch, x_batch, y_batch);
-    case 128: return gemm::launch<128>(x, ldx, w, nullptr, y, ldy, M, N, K, workspace, workspace_bytes, s, true, nullptr, 0, nullptr, false, act, batch, x_batch, y_batch);
-    default: return gemm::launch<256>(x, ldx, w, nullptr, y, ldy, M, N, K, workspace, workspace_bytes, s, true, nullptr, 0, nullptr, false, act, batch, x_batch, y_batch);
+    case 32: return gemm::launch<32>(x, ldx, w, nullptr, y, ldy, M, N, K, workspace, workspace_bytes, s, true, nullptr, 0, nullptr, false, act, batch, x_batch, y_batch, gate, gate_ld);
+    case 64: return gemm::launch<64>(x, ldx, w, nullptr, y, ldy, M, N, K, workspace, workspace_bytes, s, true, nullptr, 0, nullptr, false, act, batch, x_batch, y_batch, gate, gate_ld);
+    case 128: return gemm::launch<128>(x, ldx, w, nullptr, y, ldy, M, N, K, workspace, workspace_bytes, s, true, nullptr, 0, nullptr, false, act, batch, x_batch, y_batch, gate, gate_ld);
+    default: return gemm::launch<256>(x, ldx, w, nullptr, y, ldy, M, N, K, workspace, workspace_bytes, s, true, nullptr, 0, nullptr, false, act, batch, x_batch, y_batch, gate, gate_ld);
   }
 }
 

@@ -17,7 +17,7 @@ __device__ __forceinline__ void store_as(__nv_bfloat16* p, float v) { *p = __flo
 template <typename T, typename TO>
 __global__ void __launch_bounds__(kThreads)
 linear_kernel(const T* __restrict__ x, int64_t ldx, const T* __restrict__ w, TO* __restrict__ y, int64_t ldy, int M, int N,
-              int K, int act, int x_batch, int64_t y_batch) {
+              int K, int act, int x_batch, int64_t y_batch, const T* __restrict__ gate, int64_t gate_ld) {
   __shared__ float xs[kK][kTile + 4];
   __shared__ float ws[kK][kTile + 4];
   pdl_launch_dependents();
@@ -27,6 +27,7 @@ linear_kernel(const T* __restrict__ x, int64_t ldx, const T* __restrict__ w, TO*
   x += static_cast<int64_t>(blockIdx.z) * x_batch;
   w += static_cast<int64_t>(blockIdx.z) * N * K;
   y += static_cast<int64_t>(blockIdx.z) * y_batch;
+  if (gate != nullptr) gate += static_cast<int64_t>(blockIdx.z) * y_batch;
   const int tr = (tid >> 4) * 4, tc = (tid & 15) * 4;
   float acc[4][4] = {};
   for (int k0 = 0; k0 < K; k0 += kK) {
@@ -65,6 +66,7 @@ linear_kernel(const T* __restrict__ x, int64_t ldx, const T* __restrict__ w, TO*
         v = fmaxf(v, 0.f);
         v *= v;
       }
+      if (gate != nullptr) v /= 1.f + expf(-to_f32(gate[m * gate_ld + n]));
       store_as(y + static_cast<int64_t>(m) * ldy + n, v);
     }
   }
@@ -76,26 +78,27 @@ linear_kernel(const T* __restrict__ x, int64_t ldx, const T* __restrict__ w, TO*
 extern "C" {
 
 int b200_linear_simt(const void* x, int64_t ldx, const void* w, void* y, int64_t ldy, int M, int N, int K, int act, int batch,
-                     int x_batch, int64_t y_batch, int dtype, int y_f32, b200_stream_t stream) {
+                     int x_batch, int64_t y_batch, int dtype, int y_f32, const void* gate, int64_t gate_ld, b200_stream_t stream) {
   using namespace b200;
   if (!x || !w || !y || M <= 0 || N <= 0 || K <= 0 || batch <= 0 || batch > 65535 || ldy < N || act < B200_ACT_NONE ||
       act > B200_ACT_RELU2)
     return B200_ERR_INVALID_ARGUMENT;
-  if ((batch - 1) * static_cast<int64_t>(x_batch) + K > ldx) return B200_ERR_INVALID_ARGUMENT;
+  if ((batch - 1) * static_cast<int64_t>(x_batch) + K > ldx || (gate && gate_ld < (batch - 1) * y_batch + N)) return B200_ERR_INVALID_ARGUMENT;
   const dim3 grid((N + simt::kTile - 1) / simt::kTile, (M + simt::kTile - 1) / simt::kTile, batch);
   if (grid.y > 65535) return B200_ERR_INVALID_ARGUMENT;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (dtype == B200_DTYPE_F32)
     return launch_pdl(simt::linear_kernel<float, float>, grid, dim3(simt::kThreads), 0, s, static_cast<const float*>(x), ldx,
-                      static_cast<const float*>(w), static_cast<float*>(y), ldy, M, N, K, act, x_batch, y_batch);
+                      static_cast<const float*>(w), static_cast<float*>(y), ldy, M, N, K, act, x_batch, y_batch, static_cast<const float*>(gate), gate_ld);
   if (dtype != B200_DTYPE_BF16) return B200_ERR_INVALID_ARGUMENT;
   const auto* xb = static_cast<const __nv_bfloat16*>(x);
   const auto* wb = static_cast<const __nv_bfloat16*>(w);
+  const auto* gb = static_cast<const __nv_bfloat16*>(gate);
   if (y_f32)
     return launch_pdl(simt::linear_kernel<__nv_bfloat16, float>, grid, dim3(simt::kThreads), 0, s, xb, ldx, wb,
-                      static_cast<float*>(y), ldy, M, N, K, act, x_batch, y_batch);
+                      static_cast<float*>(y), ldy, M, N, K, act, x_batch, y_batch, gb, gate_ld);
   return launch_pdl(simt::linear_kernel<__nv_bfloat16, __nv_bfloat16>, grid, dim3(simt::kThreads), 0, s, xb, ldx, wb,
-                    static_cast<__nv_bfloat16*>(y), ldy, M, N, K, act, x_batch, y_batch);
+                    static_cast<__nv_bfloat16*>(y), ldy, M, N, K, act, x_batch, y_batch, gb, gate_ld);
 }
 
 }  // extern "C"

@@ -43,6 +43,11 @@ __device__ __forceinline__ float gate_of(const b200_latent_args& a, int64_t t, i
   return sigmoid(simt::to_f32(static_cast<const T*>(a.proj)[t * a.proj_ld + a.gate_offset + head]));
 }
 
+// Weight of a head's sink in a softmax denominator whose terms are taken relative to 2^top.
+__device__ __forceinline__ float sink_weight(const b200_latent_args& a, int head, float top) {
+  return a.sinks == nullptr ? 0.f : exp2f(a.sinks[head] * kLog2e - top);
+}
+
 // ---------------------------------------------------------------------------------------------------------------
 // Append
 // ---------------------------------------------------------------------------------------------------------------
@@ -65,12 +70,13 @@ __device__ __forceinline__ void rotated_pair(const b200_latent_args& a, const T*
 template <typename T>
 __global__ void __launch_bounds__(kAppendThreads)
 latent_append_kernel(b200_latent_args a) {
-  __shared__ float red[kAppendThreads / 32];
+  __shared__ float red[2][kAppendThreads / 32];
   pdl_launch_dependents();
   pdl_wait();
   const int tid = threadIdx.x;
   const int64_t t = blockIdx.x;
   const T* row = static_cast<const T*>(a.proj) + t * a.proj_ld;
+  const T* q_row = a.q != nullptr ? static_cast<const T*>(a.q) + t * a.q_ld : row;
   int64_t pos = a.token_to_pos[t];
   pos = pos < 0 ? 0 : (pos >= a.max_positions ? a.max_positions - 1 : pos);
   const float* cs = a.rope_cos + pos * (a.rot_dims / 2);
@@ -80,10 +86,11 @@ latent_append_kernel(b200_latent_args a) {
   // queries
   T* qf = static_cast<T*>(a.q_full) + t * a.heads * a.q_stride;
   const int qd = a.dim + a.rot_dim;
-  for (int idx = tid; idx < a.heads * rot_pairs; idx += kAppendThreads) {
+  const int q_pairs = a.rot_dim > 0 || a.q_rot_at > 0 ? rot_pairs : 0;  // (expanded form without a rotated part: nothing to write)
+  for (int idx = tid; idx < a.heads * q_pairs; idx += kAppendThreads) {
     const int h = idx / rot_pairs, i = idx - h * rot_pairs;
     float u, v;
-    rotated_pair(a, row + h * qd + a.dim, cs, sn, i, u, v);
+    rotated_pair(a, q_row + h * qd + a.dim, cs, sn, i, u, v);
     T* dst = qf + h * a.q_stride + a.q_rot_at + 2 * i;
     simt::store_as(dst, u);
     simt::store_as(dst + 1, v);
@@ -91,22 +98,44 @@ latent_append_kernel(b200_latent_args a) {
   const int lat_pad = a.q_rot_at > 0 ? a.kv_pad - a.kv_rank : 0;
   for (int idx = tid; idx < a.heads * lat_pad; idx += kAppendThreads)
     simt::store_as(qf + (idx / lat_pad) * a.q_stride + a.kv_rank + idx % lat_pad, 0.f);
+  if (a.dkv_offset < 0 && a.q_latent_out == nullptr) return;
+
+  // sums of squares of the key / value latent and of the query latent
+  const T* lat = row + a.dkv_offset;
+  const T* q_lat = row + a.q_latent_offset;
+  float sq[2] = {0.f, 0.f};
+  if (a.dkv_offset >= 0)
+    for (int c = tid; c < a.kv_rank; c += kAppendThreads) {
+      const float v = simt::to_f32(lat[c]);
+      sq[0] += v * v;
+    }
+  if (a.q_latent_out != nullptr)
+    for (int c = tid; c < a.q_rank; c += kAppendThreads) {
+      const float v = simt::to_f32(q_lat[c]);
+      sq[1] += v * v;
+    }
+  float total[2] = {0.f, 0.f};
+#pragma unroll
+  for (int n = 0; n < 2; ++n) {
+    sq[n] = warp_sum(sq[n]);
+    if ((tid & 31) == 0) red[n][tid >> 5] = sq[n];
+  }
+  __syncthreads();
+#pragma unroll
+  for (int i = 0; i < kAppendThreads / 32; ++i) {
+    total[0] += red[0][i];
+    total[1] += red[1][i];
+  }
+  if (a.q_latent_out != nullptr) {
+    const float q_inv = 1.f / sqrtf(total[1] / a.q_rank + a.eps);
+    T* q_dst = static_cast<T*>(a.q_latent_out) + t * a.q_rank;
+    const T* q_g = static_cast<const T*>(a.q_norm_weight);
+    for (int c = tid; c < a.q_rank; c += kAppendThreads) simt::store_as(q_dst + c, simt::to_f32(q_lat[c]) * q_inv * simt::to_f32(q_g[c]));
+  }
   if (a.dkv_offset < 0) return;
 
   // this token's pool row
-  const T* lat = row + a.dkv_offset;
-  float sq = 0.f;
-  for (int c = tid; c < a.kv_rank; c += kAppendThreads) {
-    const float v = simt::to_f32(lat[c]);
-    sq += v * v;
-  }
-  sq = warp_sum(sq);
-  if ((tid & 31) == 0) red[tid >> 5] = sq;
-  __syncthreads();
-  float total = 0.f;
-#pragma unroll
-  for (int i = 0; i < kAppendThreads / 32; ++i) total += red[i];
-  const float inv = 1.f / sqrtf(total / a.kv_rank + a.eps);
+  const float inv = 1.f / sqrtf(total[0] / a.kv_rank + a.eps);
   const int64_t chunk = a.token_to_chunk_idx[t], local = a.token_to_local_pos[t];
   if (chunk < 0 || chunk >= a.num_chunks || local < 0 || local >= a.chunk_size) return;
   T* dst = static_cast<T*>(a.pool) + (chunk * a.chunk_size + local) * a.row_width;
@@ -377,8 +406,9 @@ latent_decode_kernel(b200_latent_args a, int stages) {
   for (int r = 0; r < SR; ++r) {
     const float l = warp_sum(l_run[r]);
     if (lane == 0) {
-      al[warp * SR + r] = 1.f / l;
-      lse[warp * SR + r] = m_run[r] + log2f(l);
+      const int head = warp * SR + r;
+      al[head] = 1.f / (a.num_splits == 1 && head < a.heads ? l + sink_weight(a, head, m_run[r]) : l);
+      lse[head] = m_run[r] + log2f(l);
     }
   }
   consumer_barrier();
@@ -796,7 +826,8 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap map, b200_latent_args a, 
         a.workspace[static_cast<int64_t>(a.num_tokens) * a.heads * a.num_splits * a.kv_rank + pair * a.num_splits + split] =
             l > 0.f ? m_s[tid] + log2f(l) : -INFINITY;
       } else {
-        al_s[tid] = inv * gate_of<__nv_bfloat16>(a, pair / a.heads, static_cast<int>(pair % a.heads));
+        const int head = static_cast<int>(pair % a.heads);
+        al_s[tid] = (l > 0.f ? 1.f / (l + sink_weight(a, head, m_s[tid])) : 0.f) * gate_of<__nv_bfloat16>(a, pair / a.heads, head);
       }
     }
     group_sync();
@@ -848,7 +879,8 @@ latent_combine_kernel(b200_latent_args a) {
   float m = -INFINITY, total = 0.f;
   for (int s = 0; s < used; ++s) m = fmaxf(m, lse[s]);
   for (int s = 0; s < used; ++s) total += exp2f(lse[s] - m);
-  const float g = gate_of<__nv_bfloat16>(a, t, static_cast<int>(pair % a.heads)) / total;
+  const int head = static_cast<int>(pair % a.heads);
+  const float g = gate_of<__nv_bfloat16>(a, t, head) / (total + sink_weight(a, head, m));
   const float* part = a.workspace + pair * a.num_splits * a.kv_rank;
   __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(a.out) + pair * a.kv_rank;
   for (int c = threadIdx.x; c < a.kv_rank; c += blockDim.x) {
@@ -941,13 +973,14 @@ latent_prompt_kernel(b200_latent_args a) {
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   {
-    const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(a.proj);
+    const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(a.q != nullptr ? a.q : a.proj);
+    const int64_t q_ld = a.q != nullptr ? a.q_ld : a.proj_ld;
     const __nv_bfloat16* qr = static_cast<const __nv_bfloat16*>(a.q_full);
     for (int x = tid; x < kPrQueries * (d8 + r8); x += kPrThreads) {
       const int r = x / (d8 + r8), c = x - r * (d8 + r8);
       const int64_t t = t_begin + q0 + min(r, n_q - 1);
       if (c < d8)
-        cp_async16(smem_u32(q_s + r * ks + c * 8), q + t * a.proj_ld + head * (a.dim + a.rot_dim) + c * 8, r < n_q && c * 8 < a.dim);
+        cp_async16(smem_u32(q_s + r * ks + c * 8), q + t * q_ld + head * (a.dim + a.rot_dim) + c * 8, r < n_q && c * 8 < a.dim);
       else
         cp_async16(smem_u32(q_s + r * ks + dp + (c - d8) * 8), qr + (t * a.heads + head) * a.q_stride + a.q_rot_at + (c - d8) * 8,
                    r < n_q && (c - d8) * 8 < rot_w);
@@ -1067,8 +1100,22 @@ latent_prompt_kernel(b200_latent_args a) {
     const int q = warp * 16 + gid + r * 8;
     if (q >= n_q) continue;
     const int64_t t = t_begin + q0 + q;
-    const float g = gate_of<__nv_bfloat16>(a, t, head) / l;
+    l += sink_weight(a, head, m_run[r]);
     __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(a.out) + (t * a.heads + head) * a.vdim;
+    if (a.value_gates) {  // one per channel (4-byte loads: even columns)
+      const float inv = 1.f / l;
+      const __nv_bfloat16* gates = static_cast<const __nv_bfloat16*>(a.proj) + t * a.proj_ld + a.gate_offset + head * a.vdim;
+#pragma unroll
+      for (int j = 0; j < MAXV / 8; ++j) {
+        const int col = j * 8 + tig * 2;
+        if (col >= a.vdim) continue;
+        const uint32_t g = *reinterpret_cast<const uint32_t*>(gates + col);
+        *reinterpret_cast<uint32_t*>(dst + col) = pack_bf16x2(__fdividef(o[j][2 * r] * inv, 1.f + __expf(-bf16_lo(g))),
+                                                              __fdividef(o[j][2 * r + 1] * inv, 1.f + __expf(-bf16_hi(g))));
+      }
+      continue;
+    }
+    const float g = gate_of<__nv_bfloat16>(a, t, head) / l;
 #pragma unroll
     for (int j = 0; j < MAXV / 8; ++j) {
       const int col = j * 8 + tig * 2;
@@ -1146,7 +1193,7 @@ latent_simt_kernel(b200_latent_args a) {
     m = m_new;
     __syncthreads();
   }
-  const float g = gate_of<T>(a, t, head) / l;
+  const float g = gate_of<T>(a, t, head) / (a.sinks != nullptr ? l + expf(a.sinks[head] - m) : l);
 #pragma unroll
   for (int j = 0; j < kSimtMaxCols; ++j) {
     const int c = j * kSimtThreads + tid;
@@ -1244,8 +1291,12 @@ int b200_latent_append(const b200_latent_args* a, b200_stream_t stream) {
   using namespace b200;
   if (!latent::valid_common(a) || !a->token_to_pos || a->max_positions <= 0 || (a->rot_dims > 0 && (!a->rope_cos || !a->rope_sin)))
     return B200_ERR_INVALID_ARGUMENT;
-  if (a->q_rot_at < 0 || a->q_stride < a->q_rot_at + a->row_width - a->kv_pad || (a->q_rot_at > 0 && a->q_rot_at < a->kv_pad))
+  const bool no_q = a->rot_dim == 0 && a->q_rot_at == 0;  // nothing of the queries is written
+  if (a->q_rot_at < 0 || (!no_q && a->q_stride < a->q_rot_at + a->row_width - a->kv_pad) || (a->q_rot_at > 0 && a->q_rot_at < a->kv_pad))
     return B200_ERR_INVALID_ARGUMENT;
+  if (a->q_latent_out && (!a->q_norm_weight || a->q_rank <= 0 || a->q_latent_offset < 0 || a->q_latent_offset + a->q_rank > a->proj_ld))
+    return B200_ERR_INVALID_ARGUMENT;
+  if (a->q && a->q_ld < static_cast<int64_t>(a->heads) * (a->dim + a->rot_dim)) return B200_ERR_INVALID_ARGUMENT;
   if (a->dkv_offset >= 0 && (!a->norm_weight || !a->token_to_chunk_idx || !a->token_to_local_pos)) return B200_ERR_INVALID_ARGUMENT;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (a->dtype == B200_DTYPE_F32)
@@ -1285,7 +1336,7 @@ int b200_latent_attention(const b200_latent_args* a, b200_stream_t stream) {
 
 int b200_latent_prompt_supported(int dim, int rot_dim, int vdim, int heads) {
   using namespace b200::latent;
-  return dim > 0 && rot_dim > 0 && vdim > 0 && heads > 0 && heads <= 65535 && dim % 8 == 0 && rot_dim % 8 == 0 && vdim % 8 == 0 &&
+  return dim > 0 && rot_dim >= 0 && vdim > 0 && heads > 0 && heads <= 65535 && dim % 8 == 0 && rot_dim % 8 == 0 && vdim % 8 == 0 &&
          vdim <= kPrMaxV && (dim + 15) / 16 + (rot_dim + 15) / 16 <= kPrSteps;
 }
 
@@ -1305,8 +1356,11 @@ int b200_latent_prompt_attention(const b200_latent_args* a, b200_stream_t stream
       !b200_latent_prompt_supported(a->dim, a->rot_dim, a->vdim, a->heads))
     return B200_ERR_INVALID_ARGUMENT;
   if (a->proj_ld % 8 != 0 || a->q_stride % 8 != 0 || a->q_rot_at % 8 != 0 || !aligned16(a->proj) || !aligned16(a->key_rows) ||
-      !aligned16(a->key_values) || a->q_stride < a->q_rot_at + a->row_width - a->kv_pad)
+      !aligned16(a->key_values) || (a->rot_dim > 0 && a->q_stride < a->q_rot_at + a->row_width - a->kv_pad))
     return B200_ERR_ALIGNMENT;
+  if (a->q && (!aligned16(a->q) || a->q_ld % 8 != 0 || a->q_ld < a->heads * (a->dim + a->rot_dim))) return B200_ERR_ALIGNMENT;
+  if (a->value_gates && (a->gate_offset < 0 || a->gate_offset % 2 != 0 || a->gate_offset + a->heads * a->vdim > a->proj_ld))
+    return B200_ERR_INVALID_ARGUMENT;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const int steps = (a->dim + 15) / 16 + (a->rot_dim + 15) / 16;
   return steps <= 8 && a->vdim <= 64 ? launch_prompt<8, 64>(*a, s) : launch_prompt<kPrSteps, kPrMaxV>(*a, s);

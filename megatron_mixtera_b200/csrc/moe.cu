@@ -4,7 +4,7 @@
 //   route_kernel   a warp per token: scores from the router's fp32 partial sums, the `top` best, a place behind the tokens that
 //                  already chose the same expert; the CTA that finishes last turns the counts into offsets and the tile list
 //   route_softmax_kernel  the same with softmax scores, a correction of the choice, groups of experts, identity experts and weights that
-//                  add up to one
+//                  add up to one; or (CHOSEN) biased logits as scores and the softmax over the chosen ones as weights
 //   gather_kernel  x_sorted[offset[expert] + rank] = x[token]
 //   simt_kernel    64 x 64 outputs per CTA in true fp32
 #include "common.cuh"
@@ -133,11 +133,13 @@ route_kernel(b200_moe_args a) {
   finish_routing(a);
 }
 
-// Softmax over experts and identity experts, choice by score + correction inside the best groups.
+// Softmax over experts and identity experts, choice by score + correction inside the best groups.  CHOSEN: scores are the logits plus a
+// bias, and the weights the softmax over the chosen ones.
 // Shared memory: [kWarps][columns + groups] scores and the groups' best choice scores.
-template <typename T>
+template <typename T, bool CHOSEN>
 __global__ void __launch_bounds__(kWarps * 32)
 route_softmax_kernel(b200_moe_args a) {
+  constexpr float kTaken = CHOSEN ? -INFINITY : -1.f;  // the score of what can no longer be chosen
   extern __shared__ float score_s[];
   __shared__ int chosen_s[kWarps][64];
   __shared__ float weight_s[kWarps][64];
@@ -155,17 +157,23 @@ route_softmax_kernel(b200_moe_args a) {
     for (int e = lane; e < C; e += 32) {
       float x = 0.f;
       for (int s = 0; s < a.router_splits; ++s) x += z[s * stride + e];
+      if (CHOSEN) x += simt::to_f32(correction[e]);
       score[e] = x;
       top = fmaxf(top, x);
     }
     top = warp_max(top);
-    for (int e = lane; e < C; e += 32) {
-      score[e] = expf(score[e] - top);
-      sum += score[e];
+    if (!CHOSEN) {
+      for (int e = lane; e < C; e += 32) {
+        score[e] = expf(score[e] - top);
+        sum += score[e];
+      }
+      sum = warp_sum(sum);
+      for (int e = lane; e < C; e += 32) score[e] /= sum;
     }
-    sum = warp_sum(sum);
-    for (int e = lane; e < C; e += 32) score[e] /= sum;
-    auto choice = [&](int e) { return score[e] < 0.f ? -INFINITY : score[e] + simt::to_f32(correction[e]); };  // (negative: marked)
+    auto choice = [&](int e) {
+      if (CHOSEN) return score[e];
+      return score[e] < 0.f ? -INFINITY : score[e] + simt::to_f32(correction[e]);  // (negative: marked)
+    };
     // The largest of f over [0, n), the smallest index among equals (n: nothing above minus infinity).
     auto best_of = [&](int n, auto f) {
       float best = -INFINITY;
@@ -204,19 +212,19 @@ route_softmax_kernel(b200_moe_args a) {
         __syncwarp();
       }
       for (int e = lane; e < C; e += 32)
-        if (group_best[e / size] != INFINITY) score[e] = -1.f;
+        if (group_best[e / size] != INFINITY) score[e] = kTaken;
       __syncwarp();
     }
     float total = 0.f;
     for (int k = 0; k < a.top; ++k) {
       int at = best_of(C, choice);
       if (at >= C) at = k;  // no number left (NaN scores): any expert, its output is NaN too
-      const float s = score[at];
+      const float s = CHOSEN ? expf(score[at] - top) : score[at];
       __syncwarp();
       if (lane == 0) {
         chosen_s[warp][k] = at;
         weight_s[warp][k] = s;
-        score[at] = -1.f;
+        score[at] = kTaken;
       }
       total += s;
       __syncwarp();
@@ -225,7 +233,7 @@ route_softmax_kernel(b200_moe_args a) {
       const int64_t pair = static_cast<int64_t>(t) * a.top + k;
       const int e = chosen_s[warp][k];
       reinterpret_cast<int2*>(a.pairs)[pair] = make_int2(e, e < E ? atomicAdd(&a.counts[e], 1) : 0);
-      a.pair_weight[pair] = weight_s[warp][k] / (total + 1e-20f) * a.weight_scale;
+      a.pair_weight[pair] = weight_s[warp][k] / (CHOSEN ? total : total + 1e-20f) * a.weight_scale;
     }
   }
   finish_routing(a);
@@ -259,9 +267,9 @@ gather_kernel(b200_moe_args a, int vectors) {
   for (; i < vectors; i += 32) dst[i] = src[i];
 }
 
-// CUDA-core grouped product.  GATED: 64 features of an up product (gate and up rows of one 128-row block), else 64 features of a down product.
-// blockIdx.y < shared_blocks: the shared expert's token blocks, then the tile list.
-template <typename T, bool GATED>
+// CUDA-core grouped product.  GATED: 64 features of an up product (gate and up rows of one 128-row block), else 64 features of a down product or
+// (UP) of an up product without gates.  blockIdx.y < shared_blocks: the shared expert's token blocks, then the tile list.
+template <typename T, bool GATED, bool UP>
 __global__ void __launch_bounds__(256)
 simt_kernel(b200_moe_args a, int shared_blocks) {
   constexpr int kK = 16, kTile = 64;
@@ -269,7 +277,7 @@ simt_kernel(b200_moe_args a, int shared_blocks) {
   pdl_launch_dependents();
   pdl_wait();
   const bool shared = static_cast<int>(blockIdx.y) < shared_blocks;
-  const int ff = shared ? a.shared_ff : a.ff, K = GATED ? a.width : ff, N = GATED ? ff : a.width;
+  const int ff = shared ? a.shared_ff : a.ff, K = UP ? a.width : ff, N = UP ? ff : a.width;
   const int n0 = blockIdx.x * kTile;
   if (n0 >= N) return;
   int m0 = blockIdx.y * kTile, rows = min(kTile, a.num_tokens - m0), expert = 0;
@@ -284,10 +292,10 @@ simt_kernel(b200_moe_args a, int shared_blocks) {
     m0 = e.y;
     rows = e.z;
   }
-  const T* x = static_cast<const T*>(GATED ? (shared ? a.x : a.x_sorted) : (shared ? a.shared_inter : a.inter));
-  const T* w = static_cast<const T*>(GATED ? (shared ? a.shared_up : a.up) : (shared ? a.shared_down : a.down)) +
-               static_cast<int64_t>(expert) * (GATED ? 2 * ff : a.width) * K + (GATED ? static_cast<int64_t>(blockIdx.x) * 128 * K : static_cast<int64_t>(n0) * K);
-  T* y = static_cast<T*>(GATED ? (shared ? a.shared_inter : a.inter) : (shared ? a.shared_y : a.y));
+  const T* x = static_cast<const T*>(UP ? (shared ? a.x : a.x_sorted) : (shared ? a.shared_inter : a.inter));
+  const T* w = static_cast<const T*>(UP ? (shared ? a.shared_up : a.up) : (shared ? a.shared_down : a.down)) +
+               static_cast<int64_t>(expert) * (GATED ? 2 * ff : N) * K + (GATED ? static_cast<int64_t>(blockIdx.x) * 128 * K : static_cast<int64_t>(n0) * K);
+  T* y = static_cast<T*>(UP ? (shared ? a.shared_inter : a.inter) : (shared ? a.shared_y : a.y));
   const int tid = threadIdx.x, tr = (tid >> 4) * 4, tc = (tid & 15) * 4;
   float acc[4][4] = {}, up[4][4] = {};
   for (int k0 = 0; k0 < K; k0 += kK) {
@@ -324,6 +332,8 @@ simt_kernel(b200_moe_args a, int shared_blocks) {
         v = v / (1.f + expf(-v)) * up[i][j];
       else if (GATED)
         v = gemm::clamped_glu(v * scale, up[i][j] * scale, shared ? a.shared_limit : a.limit, a.alpha);
+      else if (UP)
+        v = gemm::apply_act(v, B200_ACT_RELU2);
       simt::store_as(y + static_cast<int64_t>(m) * N + n0 + tc + j, v);
     }
   }
@@ -331,7 +341,7 @@ simt_kernel(b200_moe_args a, int shared_blocks) {
 
 static bool valid(const b200_moe_args* a) {
   return a && a->num_tokens > 0 && a->width > 0 && a->experts > 0 && a->experts <= kMaxExperts && a->top > 0 && a->top <= a->experts + (a->plain ? a->identity : 0) &&
-         a->top <= 64 && a->ff > 0 && a->ff % 64 == 0 && a->tile_tokens > 0 && a->max_tiles > 0 && a->pairs && a->offsets && a->tiles && a->num_tiles &&
+         a->top <= 64 && (!a->relu2 || a->plain) && a->ff > 0 && a->ff % 64 == 0 && a->tile_tokens > 0 && a->max_tiles > 0 && a->pairs && a->offsets && a->tiles && a->num_tiles &&
          static_cast<int64_t>(a->num_tokens) * a->top < (1 << 30) && (!a->shared_up || (a->shared_ff > 0 && a->shared_ff % 64 == 0)) &&
          (a->dtype == B200_DTYPE_BF16 || a->dtype == B200_DTYPE_F32);
 }
@@ -344,22 +354,25 @@ static int grouped(const b200_moe_args& a, bool up, cudaStream_t s) {
     const int widest = up ? (with_shared && a.shared_ff > a.ff ? a.shared_ff : a.ff) : a.width;
     if (shared_blocks + a.max_tiles > 65535) return B200_ERR_INVALID_ARGUMENT;
     const dim3 grid((widest + 63) / 64, shared_blocks + a.max_tiles);
-    if (a.dtype == B200_DTYPE_F32)
-      return up ? launch_pdl(simt_kernel<float, true>, grid, dim3(256), 0, s, a, shared_blocks)
-                : launch_pdl(simt_kernel<float, false>, grid, dim3(256), 0, s, a, shared_blocks);
-    return up ? launch_pdl(simt_kernel<__nv_bfloat16, true>, grid, dim3(256), 0, s, a, shared_blocks)
-              : launch_pdl(simt_kernel<__nv_bfloat16, false>, grid, dim3(256), 0, s, a, shared_blocks);
+    auto go = [&](auto zero) {
+      using T = decltype(zero);
+      if (!up) return launch_pdl(simt_kernel<T, false, false>, grid, dim3(256), 0, s, a, shared_blocks);
+      if (a.relu2) return launch_pdl(simt_kernel<T, false, true>, grid, dim3(256), 0, s, a, shared_blocks);
+      return launch_pdl(simt_kernel<T, true, true>, grid, dim3(256), 0, s, a, shared_blocks);
+    };
+    return a.dtype == B200_DTYPE_F32 ? go(0.f) : go(__nv_bfloat16{});
   }
   const int64_t pairs = static_cast<int64_t>(a.num_tokens) * a.top;
   gemm::GroupedProblem routed{up ? a.x_sorted : a.inter, up ? a.up : a.down, up ? a.width : a.ff, a.experts}, shared{};
   gemm::GroupedParams gp{};
   auto fill = [&](gemm::Params& p, int64_t M, int ff, void* y, float limit, const float* scale) {
     p.M = static_cast<int>(M);
-    p.N = up ? 2 * ff : a.width;
+    p.N = !up ? a.width : a.relu2 ? ff : 2 * ff;
     p.K = up ? a.width : ff;
     p.y = static_cast<__nv_bfloat16*>(y);
     p.ldy = up ? ff : a.width;
-    p.gated = !up ? 0 : a.plain ? gemm::kGatedPlain : gemm::kGatedClamped;
+    p.gated = !up || a.relu2 ? 0 : a.plain ? gemm::kGatedPlain : gemm::kGatedClamped;
+    p.act = up && a.relu2 ? B200_ACT_RELU2 : B200_ACT_NONE;
     p.glu_limit = limit;
     p.glu_alpha = a.alpha;
     p.row_scale = up && !a.plain ? scale : nullptr;
@@ -401,14 +414,15 @@ int b200_moe_route(const b200_moe_args* a, b200_stream_t stream) {
         columns % groups != 0 || a->keep_groups < 1 || a->keep_groups > groups || a->top > columns / groups * a->keep_groups)
       return B200_ERR_INVALID_ARGUMENT;
     const size_t bytes = static_cast<size_t>(moe::kWarps) * (columns + groups) * 4;
-    auto go = [&](auto zero) {
+    auto go = [&](auto zero, auto CHOSEN) {
       using T = decltype(zero);
       static std::atomic<uint64_t> done{0};
-      if (ensure_dynamic_smem(moe::route_softmax_kernel<T>, moe::kWarps * 2 * moe::kMaxExperts * 4, done) != B200_OK)
-        return static_cast<int>(B200_ERR_LAUNCH);
-      return launch_pdl(moe::route_softmax_kernel<T>, dim3(blocks), dim3(moe::kWarps * 32), bytes, reinterpret_cast<cudaStream_t>(stream), *a);
+      auto kernel = moe::route_softmax_kernel<T, CHOSEN.value>;
+      if (ensure_dynamic_smem(kernel, moe::kWarps * 2 * moe::kMaxExperts * 4, done) != B200_OK) return static_cast<int>(B200_ERR_LAUNCH);
+      return launch_pdl(kernel, dim3(blocks), dim3(moe::kWarps * 32), bytes, reinterpret_cast<cudaStream_t>(stream), *a);
     };
-    return a->dtype == B200_DTYPE_F32 ? go(0.f) : go(__nv_bfloat16{});
+    if (a->plain == 2) return a->dtype == B200_DTYPE_F32 ? go(0.f, std::true_type{}) : go(__nv_bfloat16{}, std::true_type{});
+    return a->dtype == B200_DTYPE_F32 ? go(0.f, std::false_type{}) : go(__nv_bfloat16{}, std::false_type{});
   }
   return launch_pdl(moe::route_kernel, dim3(blocks), dim3(moe::kWarps * 32), static_cast<size_t>(moe::kWarps) * a->experts * 4,
                     reinterpret_cast<cudaStream_t>(stream), *a);

@@ -29,12 +29,22 @@ __device__ __forceinline__ void store(T* p, const float (&v)[VEC]) {
     simt::store_as(p, v[0]);
 }
 
+// The value that a later load of a stored one gives.
+template <typename T>
+__device__ __forceinline__ float as_stored(float x) {
+  if constexpr (sizeof(T) == 4)
+    return x;
+  else
+    return bf16_round(x);
+}
+
 // SLOTS * VEC * kThreads >= width: the row lives in registers.
 template <typename T, int VEC, int SLOTS>
 __global__ void __launch_bounds__(kThreads)
 residual_norm_kernel(b200_residual_norm_args a) {
   __shared__ float red[kThreads / 32];
   __shared__ int64_t expert_row[kMaxTop];
+  __shared__ float expert_weight[kMaxTop];
   pdl_launch_dependents();
   const int tid = threadIdx.x, W = a.width;
   pdl_wait();
@@ -49,6 +59,7 @@ residual_norm_kernel(b200_residual_norm_args a) {
         if (at >= a.expert_row_count) at = -1;
       }
       expert_row[tid] = at;
+      expert_weight[tid] = ok && a.pair_weight != nullptr ? a.pair_weight[row * a.top + tid] : 1.f;
     }
     __syncthreads();
   }
@@ -90,7 +101,7 @@ residual_norm_kernel(b200_residual_norm_args a) {
         for (int j = 0; j < 4; ++j)
           if (k + j < a.top && expert_row[min(k + j, a.top - 1)] >= 0) {
 #pragma unroll
-            for (int e = 0; e < VEC; ++e) add[e] += rows[j][e];
+            for (int e = 0; e < VEC; ++e) add[e] = fmaf(expert_weight[k + j], rows[j][e], add[e]);
           }
       }
     }
@@ -126,6 +137,48 @@ residual_norm_kernel(b200_residual_norm_args a) {
 #pragma unroll
   for (int i = 0; i < kThreads / 32; ++i) total += red[i];
   const float inv = a.out_scale / sqrtf(total / W + a.eps);
+  if (a.taps > 0) {
+    // One token per row: the norm goes through the filters, whose earlier inputs are the row's state.
+    const T* gamma = static_cast<const T*>(a.gamma[0]);
+    const int back = a.taps - 1;
+    int in = ok ? a.state_in[row] : -1, out = ok ? a.state_out[row] : -1;
+    if (in >= a.state_slots) in = -1;
+    if (out >= a.state_slots) out = -1;
+#pragma unroll
+    for (int i = 0; i < SLOTS; ++i) {
+      const int c = (i * kThreads + tid) * VEC;
+      if (c >= W) continue;
+      float u[VEC], w[VEC], past[VEC], y[2][VEC];
+      load<T, VEC>(gamma + c, u);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) u[e] = as_stored<T>(v[i][e] * inv * (a.gain + u[e]));
+#pragma unroll
+      for (int n = 0; n < 2; ++n) {
+        if (a.filter[n] == nullptr) continue;
+        load<T, VEC>(static_cast<const T*>(a.filter[n]) + static_cast<int64_t>(back) * W + c, w);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) y[n][e] = fmaf(w[e], u[e], u[e]);
+      }
+      for (int j = 0; j < back; ++j) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) past[e] = 0.f;
+        if (in >= 0) load<T, VEC>(static_cast<const T*>(a.state) + (static_cast<int64_t>(in) * back + j) * W + c, past);
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+          if (a.filter[n] == nullptr) continue;
+          load<T, VEC>(static_cast<const T*>(a.filter[n]) + static_cast<int64_t>(j) * W + c, w);
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) y[n][e] = fmaf(w[e], past[e], y[n][e]);
+        }
+        if (out >= 0 && j > 0) store<T, VEC>(static_cast<T*>(a.state) + (static_cast<int64_t>(out) * back + j - 1) * W + c, past);
+      }
+      if (out >= 0 && back > 0) store<T, VEC>(static_cast<T*>(a.state) + (static_cast<int64_t>(out) * back + back - 1) * W + c, u);
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+        if (a.filter[n] != nullptr) store<T, VEC>(static_cast<T*>(a.y[n]) + static_cast<int64_t>(blockIdx.x) * W + c, y[n]);
+    }
+    return;
+  }
 #pragma unroll
   for (int n = 0; n < 2; ++n) {
     if (a.y[n] == nullptr) continue;
@@ -149,7 +202,7 @@ static int launch(const b200_residual_norm_args& a, cudaStream_t s) {
   bool aligned = a.width % 4 == 0;
   for (const void* p : {a.table, static_cast<const void*>(a.partials), a.branch, a.expert_rows, a.shared_rows,
                         static_cast<const void*>(a.hidden), a.gamma[0], a.gamma[1], static_cast<const void*>(a.y[0]),
-                        static_cast<const void*>(a.y[1])})
+                        static_cast<const void*>(a.y[1]), a.filter[0], a.filter[1], static_cast<const void*>(a.state)})
     aligned = aligned && aligned16(p);
   const dim3 grid(a.rows), block(kThreads);
   if (aligned) {
@@ -175,7 +228,11 @@ extern "C" int b200_residual_norm(const b200_residual_norm_args* a, b200_stream_
   if ((a->table && (!a->ids || a->table_rows <= 0)) || (a->partials && a->num_splits < 1) ||
       (a->expert_rows && (!a->pairs || !a->offsets || a->top < 1 || a->top > resnorm::kMaxTop || a->experts < 1)))
     return B200_ERR_INVALID_ARGUMENT;
-  if ((a->y[1] && !a->y[0]) || (a->y[0] && !a->gamma[0]) || (a->y[1] && !a->gamma[1])) return B200_ERR_INVALID_ARGUMENT;
+  if ((a->y[1] && !a->y[0]) || (a->y[0] && !a->gamma[0]) || (a->y[1] && !a->gamma[1] && a->taps == 0)) return B200_ERR_INVALID_ARGUMENT;
+  if (a->taps < 0 || a->taps > 8 ||
+      (a->taps > 0 && (a->row_index || !a->y[0] || !a->filter[0] || !a->filter[1] != !a->y[1] || !a->state_in || !a->state_out ||
+                       (a->taps > 1 && (!a->state || a->state_slots <= 0)))))
+    return B200_ERR_INVALID_ARGUMENT;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (a->dtype == B200_DTYPE_BF16) return resnorm::launch<__nv_bfloat16>(*a, s);
   if (a->dtype == B200_DTYPE_F32) return resnorm::launch<float>(*a, s);

@@ -64,6 +64,7 @@ __global__ void __launch_bounds__(kTokenThreads) vector_kernel(b200_rotate_appen
     const int64_t chunk = a.chunk_idx[t], pos = a.local_pos[t];
     if (chunk >= 0 && chunk < a.num_chunks && pos >= 0 && pos < a.chunk_size) slot = (chunk * a.chunk_size + pos) * a.pool_row_elems;
   }
+  const float mix = a.v_first_in != nullptr ? simt::to_f32(*static_cast<const T*>(a.mix)) : 0.f;
   float c[VEC], s[VEC];
   if (turns) {
     const int64_t angles = min(max(a.token_to_pos[t], int64_t{0}), static_cast<int64_t>(a.max_positions) - 1) * half;
@@ -127,6 +128,15 @@ __global__ void __launch_bounds__(kTokenThreads) vector_kernel(b200_rotate_appen
         for (int e = 0; e < VEC; ++e) x[e] *= inv;
       }
     }
+    if (ok && value && (a.v_first_in != nullptr || a.v_first_out != nullptr)) {
+      const int64_t first = t * a.v_vecs * a.vdim + at + i;
+      if (a.v_first_out != nullptr) conv::store<T, VEC>(static_cast<T*>(a.v_first_out) + first, x);
+      if (a.v_first_in != nullptr) {
+        conv::load<T, VEC>(static_cast<const T*>(a.v_first_in) + first, y);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) x[e] = fmaf(mix, y[e], (1.f - mix) * x[e]);
+      }
+    }
     if (!ok || (v >= keys_at && slot < 0)) continue;
     T* dst = v < keys_at ? static_cast<T*>(a.q_out) + t * a.q_vecs * a.dim : static_cast<T*>(value ? a.v_pool : a.k_pool) + slot;
     conv::store<T, VEC>(dst + at + i, x);
@@ -163,6 +173,17 @@ __global__ void __launch_bounds__(kThreads) element_kernel(b200_rotate_append_ar
   }
   float inv = 1.f;
   if (a.rms && u.kind < 2) inv = 1.f / sqrtf(warp_sum(sq) / a.dim + a.eps);
+  if (u.kind == 2 && (a.v_first_in != nullptr || a.v_first_out != nullptr)) {
+    const int64_t first = (u.t * a.v_vecs + u.index) * u.dim;
+    const float mix = a.v_first_in != nullptr ? simt::to_f32(*static_cast<const T*>(a.mix)) : 0.f;
+#pragma unroll
+    for (int e = 0; e < kElems; ++e) {
+      const int i = e * 32 + lane;
+      if (i >= u.dim) continue;
+      if (a.v_first_out != nullptr) simt::store_as(static_cast<T*>(a.v_first_out) + first + i, x[e]);
+      if (a.v_first_in != nullptr) x[e] = fmaf(mix, simt::to_f32(static_cast<const T*>(a.v_first_in)[first + i]), (1.f - mix) * x[e]);
+    }
+  }
   T* dst = target<T>(a, u);
   if (dst == nullptr) return;
 #pragma unroll
@@ -177,7 +198,7 @@ static int launch(const b200_rotate_append_args& a, cudaStream_t s) {
   bool vec = a.dim % 8 == 0 && (a.v_vecs == 0 || a.vdim % 8 == 0) && a.proj_ld % 8 == 0 && a.pool_row_elems % 8 == 0 && a.off_q % 8 == 0 &&
              a.off_k % 8 == 0 && a.off_v % 8 == 0 && a.rot_dims % (a.halves ? 16 : 8) == 0 && aligned16(a.rope_cos) && aligned16(a.rope_sin);
   for (const void* p : {a.proj, a.q_bias, a.k_bias, a.v_bias, static_cast<const void*>(a.q_out), static_cast<const void*>(a.k_pool),
-                        static_cast<const void*>(a.v_pool)})
+                        static_cast<const void*>(a.v_pool), a.v_first_in, static_cast<const void*>(a.v_first_out)})
     vec = vec && aligned16(p);
   const int widest = a.v_vecs > 0 && a.vdim > a.dim ? a.vdim : a.dim;
   if (!vec) return launch_pdl(element_kernel<T>, dim3(static_cast<unsigned>((units + kThreads / 32 - 1) / (kThreads / 32))), dim3(kThreads), 0, s, a);
@@ -200,6 +221,7 @@ extern "C" int b200_rotate_append(const b200_rotate_append_args* a, b200_stream_
   if (a->k_vecs + a->v_vecs > 0 && (!a->chunk_idx || !a->local_pos || a->chunk_size <= 0 || a->num_chunks <= 0 ||
                                     a->pool_row_elems < a->k_vecs * a->dim + a->v_vecs * a->vdim))
     return B200_ERR_INVALID_ARGUMENT;
+  if (a->v_first_in && !a->mix) return B200_ERR_INVALID_ARGUMENT;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (a->dtype == B200_DTYPE_F32) return rotapp::launch<float>(*a, s);
   if (a->dtype == B200_DTYPE_BF16) return rotapp::launch<__nv_bfloat16>(*a, s);

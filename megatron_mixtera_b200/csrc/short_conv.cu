@@ -4,6 +4,7 @@
 // last taps - 1 inputs, or the last row), read from one buffer of its slot and written to the other.
 //
 //   conv_silu_kernel    16 bytes of channels per thread, a run of tokens, the filter and the last inputs in registers
+//   conv_add_kernel     the same for inputs plus their filter, one or two filters of the same inputs
 //   conv_qkv_kernel     some lanes per (head, run of tokens): convolution, then the per-head RMS norm of queries and keys or the
 //                       value mixing, then the stores (queries, pool rows, first values)
 //   token_shift_kernel  16 bytes of a row per thread, a run of tokens, every mix from the two rows in registers
@@ -175,6 +176,63 @@ conv_silu_kernel(b200_conv_args a, int run) {
       if (t == r.end - 1) win.store_history(a, r, c);
 #pragma unroll
       for (int e = 0; e < VEC; ++e) y[e] = y[e] / (1.f + expf(-y[e]));
+      store<T, VEC>(static_cast<T*>(a.out) + static_cast<int64_t>(t) * a.channels + c, y);
+    }
+  }
+}
+
+template <typename T, int VEC, int TAPS, int OUTS>
+__global__ void __launch_bounds__(kThreads)
+conv_add_kernel(b200_conv_args a, int run) {
+  pdl_launch_dependents();
+  const int c = (blockIdx.x * kThreads + threadIdx.x) * VEC;
+  const int t0 = blockIdx.y * run, t1 = min(t0 + run, a.num_tokens);
+  Window<T, VEC, TAPS> win;
+  float w2[OUTS == 2 ? TAPS : 1][VEC];  // the second filter
+  if (c < a.channels) {
+    win.load_filter(a, c);
+    if constexpr (OUTS == 2) {
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) {
+        const int at = j - (TAPS - a.taps);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) w2[j][e] = 0.f;
+        if (at >= 0) load<T, VEC>(static_cast<const T*>(a.filter_2) + static_cast<int64_t>(at) * a.channels + c, w2[j]);
+      }
+    }
+  }
+  pdl_wait();
+  if (c >= a.channels) return;
+  constexpr int B = 4;  // tokens whose loads are in flight together
+  Row r{0, -1, -1, -1};
+  for (int tb = t0; tb < t1; tb += B) {
+    Raw<T, VEC> now[B];
+#pragma unroll
+    for (int q = 0; q < B; ++q) now[q] = *reinterpret_cast<const Raw<T, VEC>*>(static_cast<const T*>(a.proj) + min(tb + q, t1 - 1) * a.proj_ld + c);
+#pragma unroll
+    for (int q = 0; q < B; ++q) {
+      const int t = tb + q;
+      if (t >= t1) break;
+      if (t >= r.end) {
+        r = row_of(a, t);
+        win.load_history(a, r, t, c);
+      }
+      float x[VEC], y[VEC];
+      now[q].to(x);
+      if constexpr (OUTS == 2) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+          float s = x[e];
+#pragma unroll
+          for (int j = 0; j < TAPS - 1; ++j) s = fmaf(w2[j][e], win.u[j][e], s);
+          y[e] = fmaf(w2[TAPS - 1][e], x[e], s);
+        }
+        store<T, VEC>(static_cast<T*>(a.out_2) + static_cast<int64_t>(t) * a.channels + c, y);
+      }
+      win.step(x, y);
+      if (t == r.end - 1) win.store_history(a, r, c);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) y[e] += x[e];
       store<T, VEC>(static_cast<T*>(a.out) + static_cast<int64_t>(t) * a.channels + c, y);
     }
   }
@@ -381,6 +439,24 @@ static int silu(const b200_conv_args& a, cudaStream_t s) {
   return vec ? launch_silu<T, VEC, 8>(a, s) : launch_silu<T, 1, 8>(a, s);
 }
 
+template <typename T, int VEC, int TAPS, int OUTS>
+static int launch_add(const b200_conv_args& a, cudaStream_t s) {
+  const int blocks = (a.channels + kThreads * VEC - 1) / (kThreads * VEC);
+  const int run = run_length(a, static_cast<int64_t>(blocks) * 4);
+  if ((a.num_tokens + run - 1) / run > 65535) return B200_ERR_INVALID_ARGUMENT;
+  return launch_pdl(conv_add_kernel<T, VEC, TAPS, OUTS>, dim3(blocks, (a.num_tokens + run - 1) / run), dim3(kThreads), 0, s, a, run);
+}
+template <typename T, int OUTS>
+static int add(const b200_conv_args& a, cudaStream_t s) {
+  constexpr int VEC = 8 / sizeof(T);  // (two filters and the last inputs in registers)
+  bool vec = a.channels % VEC == 0 && a.proj_ld % VEC == 0;
+  for (const void* p : {a.proj, a.filter, a.filter_2, static_cast<const void*>(a.state), static_cast<const void*>(a.out),
+                        static_cast<const void*>(a.out_2)})
+    vec = vec && aligned16(p);
+  if (a.taps <= 4) return vec ? launch_add<T, VEC, 4, OUTS>(a, s) : launch_add<T, 1, 4, OUTS>(a, s);
+  return vec ? launch_add<T, VEC, 8, OUTS>(a, s) : launch_add<T, 1, 8, OUTS>(a, s);
+}
+
 template <typename T, int VEC, int EL, int LPH, int TAPS>
 static int launch_qkv(const b200_conv_args& a, int head0, int heads, cudaStream_t s) {
   const int run = run_length(a, static_cast<int64_t>(heads) * LPH / 32 + 1);
@@ -435,6 +511,15 @@ int b200_conv_silu(const b200_conv_args* a, b200_stream_t stream) {
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (a->dtype == B200_DTYPE_F32) return conv::silu<float>(*a, s);
   return a->dtype == B200_DTYPE_BF16 ? conv::silu<__nv_bfloat16>(*a, s) : B200_ERR_INVALID_ARGUMENT;
+}
+
+int b200_conv_add(const b200_conv_args* a, b200_stream_t stream) {
+  using namespace b200;
+  if (!a || !conv::valid(*a) || !a->filter_2 != !a->out_2) return B200_ERR_INVALID_ARGUMENT;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (a->dtype == B200_DTYPE_F32) return a->out_2 ? conv::add<float, 2>(*a, s) : conv::add<float, 1>(*a, s);
+  if (a->dtype == B200_DTYPE_BF16) return a->out_2 ? conv::add<__nv_bfloat16, 2>(*a, s) : conv::add<__nv_bfloat16, 1>(*a, s);
+  return B200_ERR_INVALID_ARGUMENT;
 }
 
 int b200_conv_qkv(const b200_conv_args* a, b200_stream_t stream) {

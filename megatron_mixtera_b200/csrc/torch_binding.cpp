@@ -294,7 +294,8 @@ void attention(const Tensor& args, const Tensor& anchor, int64_t which, const Op
 // struct (a CPU uint8 tensor of exactly its size, pointing at tensors the caller keeps alive).
 // ---------------------------------------------------------------------------------------------------------------
 void linear(const Tensor& x, int64_t ldx, const Tensor& w, Tensor y, int64_t ldy, int64_t M, int64_t N, int64_t K, int64_t act,
-            int64_t batch, int64_t x_batch, int64_t y_batch, const OptTensor& workspace, bool tensor_cores) {
+            int64_t batch, int64_t x_batch, int64_t y_batch, const OptTensor& workspace, bool tensor_cores, const OptTensor& gate,
+            int64_t gate_ld) {
   TORCH_CHECK(x.is_cuda() && w.is_cuda() && y.is_cuda(), "b200_decode.linear: CUDA tensors only (no CPU fallback exists)");
   const bool f32 = x.scalar_type() == F32;
   need(w, f32 ? F32 : BF16, "w");
@@ -307,6 +308,10 @@ void linear(const Tensor& x, int64_t ldx, const Tensor& w, Tensor y, int64_t ldy
   auto room = [](const Tensor& t) { return static_cast<int64_t>(t.storage().nbytes() / t.element_size()) - t.storage_offset(); };
   TORCH_CHECK((M - 1) * ldx + (batch - 1) * x_batch + K <= room(x), "b200_decode.linear: x is too small");
   TORCH_CHECK((M - 1) * ldy + (batch - 1) * y_batch + N <= room(y), "b200_decode.linear: y is too small");
+  if (gate.has_value()) {
+    TORCH_CHECK(gate->is_cuda() && gate->scalar_type() == x.scalar_type(), "b200_decode.linear: the gate has the type of x");
+    TORCH_CHECK((M - 1) * gate_ld + (batch - 1) * y_batch + N <= room(*gate), "b200_decode.linear: gate is too small");
+  }
   c10::cuda::CUDAGuard guard(x.device());
   auto s = stream_of(x);
   const int m = static_cast<int>(M), n = static_cast<int>(N), k = static_cast<int>(K);
@@ -314,11 +319,12 @@ void linear(const Tensor& x, int64_t ldx, const Tensor& w, Tensor y, int64_t ldy
     TORCH_CHECK(!f32 && !y_f32, "b200_decode.linear: the tensor-core path is bf16");
     ok(b200_linear_bf16(ptr(x), ldx, ptr(w), ptr(y), ldy, m, n, k, static_cast<int>(act), static_cast<int>(batch),
                         static_cast<int>(x_batch), y_batch, ptr(workspace),
-                        workspace.has_value() ? static_cast<size_t>(workspace->numel()) : 0, s),
+                        workspace.has_value() ? static_cast<size_t>(workspace->numel()) : 0, ptr(gate), gate_ld, s),
        "b200_linear_bf16");
   } else {
     ok(b200_linear_simt(ptr(x), ldx, ptr(w), ptr(y), ldy, m, n, k, static_cast<int>(act), static_cast<int>(batch),
-                        static_cast<int>(x_batch), y_batch, f32 ? B200_DTYPE_F32 : B200_DTYPE_BF16, y_f32 ? 1 : 0, s),
+                        static_cast<int>(x_batch), y_batch, f32 ? B200_DTYPE_F32 : B200_DTYPE_BF16, y_f32 ? 1 : 0,
+                        ptr(gate), gate_ld, s),
        "b200_linear_simt");
   }
 }
@@ -362,6 +368,8 @@ void hybrid(const Tensor& args, const Tensor& anchor, int64_t which) {
     case 22: ok(b200_rotate_append(struct_of<b200_rotate_append_args>(args, "b200_rotate_append_args"), s), "b200_rotate_append"); break;
     case 23: ok(b200_stream_norm(struct_of<b200_stream_norm_args>(args, "b200_stream_norm_args"), s), "b200_stream_norm"); break;
     case 24: ok(b200_swiglu(struct_of<b200_swiglu_args>(args, "b200_swiglu_args"), s), "b200_swiglu"); break;
+    case 25: ok(b200_conv_add(struct_of<b200_conv_args>(args, "b200_conv_args"), s), "b200_conv_add"); break;
+    case 26: ok(b200_gated_scan(struct_of<b200_gated_scan_args>(args, "b200_gated_scan_args"), s), "b200_gated_scan"); break;
     default: TORCH_CHECK(false, "b200_decode.hybrid: unknown kernel ", which);
   }
 }
@@ -500,7 +508,7 @@ TORCH_LIBRARY(b200_decode, m) {
         "Tensor(c!)? y_out, int M, int F, int K) -> ()");
   m.def("attention(Tensor args, Tensor(a!) anchor, int which, Tensor? units, int num_units) -> ()");
   m.def("linear(Tensor x, int ldx, Tensor w, Tensor(a!) y, int ldy, int M, int N, int K, int act, int batch, int x_batch, "
-        "int y_batch, Tensor? workspace, bool tensor_cores) -> ()");
+        "int y_batch, Tensor? workspace, bool tensor_cores, Tensor? gate, int gate_ld) -> ()");
   m.def("hybrid(Tensor args, Tensor(a!) anchor, int which) -> ()");
   m.def("argmax(Tensor logits, Tensor(a!) out) -> ()");
   m.def("argmax_shard(Tensor logits, Tensor(a!) keys, int index_offset) -> ()");

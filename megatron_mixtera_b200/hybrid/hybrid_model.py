@@ -56,7 +56,7 @@ class HybridDecoder(DynamicForward, torch.nn.Module):
         tokens it must hold (in whole chunks; one more chunk takes the padding tokens' writes)."""
         c = self.config
         widths = [layer.mixer.cached_row_width() for layer in c.layers]
-        states = [layer.mixer.request_state(c.hidden_size, c.params_dtype) for layer in c.layers]
+        states = [c.request_state(i) for i in range(c.num_layers)]
         if max_cached_tokens is not None:
             chunks = -(-max_cached_tokens // chunk_size_tokens) + 1
             nbytes = DynamicInferenceContext.latent_chunk_bytes(widths, chunk_size_tokens, c.params_dtype)

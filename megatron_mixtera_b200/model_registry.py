@@ -9,9 +9,10 @@ from typing import Callable, Dict, Tuple
 import torch
 
 from . import checkpoint
-from .transformer.hybrid_config import (DeltaRuleConfig, DistanceBias, ExpertConfig, GatedDeltaConfig, GroupedAttentionConfig, HybridConfig,
-                                        HybridLayerConfig, LatentAttentionConfig, MatrixMemoryConfig, MoeConfig, RotaryConfig,
-                                        ShortConvAttentionConfig, SideBySideConfig, SoftmaxRouting, WkvConfig, YarnScaling)
+from .transformer.hybrid_config import (ChosenSoftmaxRouting, DeltaRuleConfig, DistanceBias, ExpertConfig, GatedDeltaConfig, GatedScanConfig,
+                                        GroupedAttentionConfig, HybridConfig, HybridLayerConfig, LatentAttentionConfig, MatrixMemoryConfig,
+                                        MoeConfig, RotaryConfig, ShortConvAttentionConfig, SideBySideConfig, SoftmaxRouting, WkvConfig,
+                                        YarnScaling)
 from .transformer.transformer_config import TransformerConfig
 
 
@@ -146,6 +147,43 @@ def _build_lukarax(config: dict, shapes: Dict[str, tuple], dtype: torch.dtype, m
 
 
 # ---------------------------------------------------------------------------------------------------------------------
+# Maginex
+# ---------------------------------------------------------------------------------------------------------------------
+def maginex_config(config: dict, shapes: Dict[str, tuple], dtype: torch.dtype) -> HybridConfig:
+    """``config.json`` -> `HybridConfig`."""
+    layers = []
+    for i, layer in enumerate(config["layers"]):
+        m, mlp = layer["mixer"], layer.get("mlp")
+        if layer["type"] == "latent_attention":
+            mixer = LatentAttentionConfig(heads=m["heads"], dim=m["dim"], rot_dim=0, vdim=m["vdim"], kv_rank=m["kv_rank"], q_rank=m["q_rank"],
+                                          scale=float(m["scale"]), sink=True, gate="value")
+        elif layer["type"] == "mingru":
+            mixer = GatedScanConfig(width=m["width"])
+        elif layer["type"] == "attention":
+            mixer = _grouped(m, rot=_rotary(m["rot"], halves=True) if m.get("rot") else None, sink=True, head_gate=True,
+                             value_mix=bool(m.get("v_mix", False)))
+        else:
+            raise ValueError(f"layer {i}: unknown mixer {layer['type']!r}")
+        moe = None
+        if mlp is not None:
+            if mlp["kind"] != "moe":
+                raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+            shared = mlp.get("shared")
+            moe = MoeConfig(experts=mlp["router"]["experts"], top=mlp["router"]["top"], expert=ExpertConfig(ff=mlp["expert"]["ff"], gated=False),
+                            shared=ExpertConfig(ff=shared["ff"], gated=False) if shared else None, routing=ChosenSoftmaxRouting())
+        layers.append(HybridLayerConfig(mixer=mixer, moe=moe))
+    return HybridConfig(vocab_size=config["vocab"], hidden_size=config["width"], layers=tuple(layers), block="parallel",
+                        layernorm_epsilon=float(config["norm"]["eps"]), params_dtype=dtype, norm_offset=0.0, input_taps=config["canon"]["taps"],
+                        embedding_scale=float(config["embedding"]["scale"]))
+
+
+def _build_maginex(config: dict, shapes: Dict[str, tuple], dtype: torch.dtype, max_sequence_length: int):
+    from .hybrid.parallel_model import ParallelHybridModel
+
+    return ParallelHybridModel(maginex_config(config, shapes, dtype), max_sequence_length)
+
+
+# ---------------------------------------------------------------------------------------------------------------------
 # GPTModel: config.json holds TransformerConfig fields under "transformer" and the model's own beside it
 # ---------------------------------------------------------------------------------------------------------------------
 def _build_gpt(config: dict, shapes: Dict[str, tuple], dtype: torch.dtype, max_sequence_length: int):
@@ -159,7 +197,8 @@ def _build_gpt(config: dict, shapes: Dict[str, tuple], dtype: torch.dtype, max_s
 
 
 Builder = Callable[[dict, Dict[str, tuple], torch.dtype, int], torch.nn.Module]
-ARCHITECTURES: Dict[str, Builder] = {"Fabivik": _build_fabivik, "Lukarax": _build_lukarax, "Zinurax": _build_zinurax, "GPTModel": _build_gpt}
+ARCHITECTURES: Dict[str, Builder] = {"Fabivik": _build_fabivik, "Lukarax": _build_lukarax, "Maginex": _build_maginex, "Zinurax": _build_zinurax,
+                                     "GPTModel": _build_gpt}
 
 
 def load_model(folder: str, *, dtype: torch.dtype = torch.bfloat16, max_sequence_length: int) -> torch.nn.Module:

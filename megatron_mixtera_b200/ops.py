@@ -733,7 +733,8 @@ _OUT_NORM, _LATENT_APPEND, _LATENT_ATTENTION, _DELTA_DECODE, _DELTA_LORA, _DELTA
 # kernels that take an argument struct and nothing else (`struct_kernel`)
 _STRUCT_KERNELS = {name: 9 + i for i, name in enumerate((
     "residual_norm", "conv_silu", "conv_qkv", "token_shift", "recurrence_decode", "recurrence_scan", "recurrence_finish",
-    "recurrence_lora", "moe_route", "moe_gather", "moe_up", "moe_down", "recurrence_gates", "rotate_append", "stream_norm", "swiglu"))}
+    "recurrence_lora", "moe_route", "moe_gather", "moe_up", "moe_down", "recurrence_gates", "rotate_append", "stream_norm", "swiglu",
+    "conv_add", "gated_scan"))}
 
 
 def dtype_code(dtype) -> int:
@@ -743,11 +744,12 @@ def dtype_code(dtype) -> int:
 
 
 def linear(x, w, *, act: Optional[str] = None, out=None, batch: int = 1, x_batch: int = 0, y_batch: int = 0, K: Optional[int] = None,
-           out_dtype=None):
+           out_dtype=None, gate=None):
     """``act(x @ w.T)`` for x [rows, ...] (unit inner stride, possibly the first columns of a wider matrix) and w [N, K].
 
     ``batch`` > 1: one product per head: head b multiplies x columns [b * x_batch, b * x_batch + K) with w rows [b * N, ...)
-    into out columns b * y_batch (``out`` [rows, ...] given by the caller).  bf16 runs on the tensor cores where TMA can
+    into out columns b * y_batch (``out`` [rows, ...] given by the caller).  ``gate`` [rows, ...] (unit inner stride): every output
+    times sigmoid of the gate in its column.  bf16 runs on the tensor cores where TMA can
     address the rows (K and strides multiples of 8), everything else - fp32, odd sizes, fp32 output - on the CUDA cores."""
     _need(w, x.dtype, "w")
     if not x.is_cuda or x.stride(-1) != 1 or x.dim() != 2:
@@ -762,9 +764,12 @@ def linear(x, w, *, act: Optional[str] = None, out=None, batch: int = 1, x_batch
     tc = (x.dtype == BF16 and out.dtype == BF16 and K % 8 == 0 and ldx % 8 == 0 and x_batch % 8 == 0
           and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
     ws = None
-    if tc and batch == 1:
+    if gate is not None and (gate.dtype != x.dtype or gate.stride(-1) != 1 or gate.shape[0] != M):
+        raise B200Error("linear", -1, "the gate has a row per row of x, its type and unit inner stride")
+    if tc and batch == 1 and gate is None:
         ws = _gemm_workspace(x.device, _lib.load().b200_gemm_bf16_workspace_bytes(M, N, K), True)
-    _launch("linear", x, ldx, w, out, out.stride(0), M, N, K, _ACT[act], batch, x_batch, y_batch, ws, tc)
+    _launch("linear", x, ldx, w, out, out.stride(0), M, N, K, _ACT[act], batch, x_batch, y_batch, ws, tc, gate,
+            0 if gate is None else gate.stride(0))
     return out
 
 
@@ -913,8 +918,11 @@ class PendingRows:
 
 
 def residual_norm(hidden, pending: Optional[PendingRows], gammas, outs, *, eps: float, gain: float = 1.0, out_scale: float = 1.0,
-                  row_index=None) -> None:
-    """hidden += pending (the first rows of a stream: hidden = embeddings); outs[i] = rms norm of hidden times (gain + gammas[i])."""
+                  row_index=None, filters=None, state=None, state_slots=None) -> None:
+    """hidden += pending (the first rows of a stream: hidden = embeddings); outs[i] = rms norm of hidden times (gain + gammas[i]).
+
+    ``filters`` ([taps, width] each; steps of one token per row): outs[i] = the one norm plus its causal filter ``filters[i]``, whose earlier
+    inputs are ``state`` [slots, taps - 1, width] (None with one tap) at ``state_slots`` = (slots read, slots written)."""
     _need(hidden, F32, "hidden")
     a = _lib.ResidualNormArgs()
     a.hidden, a.source_rows, a.width = hidden.data_ptr(), hidden.shape[0], hidden.shape[1]
@@ -935,12 +943,21 @@ def residual_norm(hidden, pending: Optional[PendingRows], gammas, outs, *, eps: 
         e = pending.experts
         if e is not None:
             a.expert_rows, a.expert_row_count, a.pairs, a.offsets = e.rows.data_ptr(), e.rows.shape[0], e.pairs.data_ptr(), e.offsets.data_ptr()
-            a.top, a.experts = e.top, e.experts
+            a.top, a.experts, a.pair_weight = e.top, e.experts, _p(e.weights)
             if e.shared_rows is not None:
                 a.shared_rows, a.shared_gate = e.shared_rows.data_ptr(), _p(e.shared_gate)
-    for i, (g, y) in enumerate(zip(gammas, outs)):
+    for i, g in enumerate(gammas):
+        a.gamma[i] = g.data_ptr()
+    for i, y in enumerate(outs):
         _need(y, dtype, "out")
-        a.gamma[i], a.y[i] = g.data_ptr(), y.data_ptr()
+        a.y[i] = y.data_ptr()
+    if filters is not None:
+        for i, f in enumerate(filters):
+            _need(f, dtype, "filter")
+            a.filter[i] = f.data_ptr()
+        a.taps = filters[0].shape[0]
+        a.state, a.state_slots = (None, 0) if state is None else (state.data_ptr(), state.shape[0])
+        a.state_in, a.state_out = (s.data_ptr() for s in state_slots)
     struct_kernel("residual_norm", a, hidden)
 
 
@@ -987,7 +1004,7 @@ def stream_norm(hidden, pending: Optional[PendingStreams], *, blend=None, gamma=
         if e is not None:
             a.expert_rows, a.expert_row_count, a.pairs, a.offsets = e.rows.data_ptr(), e.rows.shape[0], e.pairs.data_ptr(), e.offsets.data_ptr()
             a.pair_weight, a.top, a.experts, a.identity = e.weights.data_ptr(), e.top, e.experts, e.identity
-            a.expert_input = e.input.data_ptr()
+            a.expert_input = _p(e.input)
     if blend is not None:
         _need(blend, F32, "blend")
         a.in_ = blend.data_ptr()

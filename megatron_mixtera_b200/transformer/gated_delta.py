@@ -7,7 +7,7 @@ import torch
 from .. import _lib, ops  # noqa: F401
 from ..tensor_parallel.layers import ColumnParallelLinear, RowParallelLinear, _device
 from .hybrid_config import GatedDeltaConfig, HybridConfig
-from .short_conv_attention import filter_of, short_conv_args
+from .short_conv import filter_of, short_conv_args
 from .wkv import DELTA, recurrence_args
 
 
@@ -46,7 +46,7 @@ class GatedDelta(torch.nn.Module):
                           (self.linear_proj.weight, "o")):
             dst.data.copy_(get(name))
 
-    def forward(self, x, ctx, step=None):
+    def forward(self, x, ctx, rope=None, step=None):
         """``x`` [T, H] -> the output linear's partial sums.  Decode steps run one fused kernel; other steps convolve all tokens
         and scan every request's."""
         m, T, dev = self.mixer, x.shape[0], x.device

@@ -29,8 +29,9 @@ class GroupedAttention(torch.nn.Module):
             self.inputs["k"] = m.kv_heads * m.maps * m.dim
             if not m.values_from_keys:
                 self.inputs["v"] = m.kv_heads * m.vdim
-        if m.gate:
-            self.inputs["g"] = m.heads * m.vdim
+        if m.gate or m.head_gate:
+            self.inputs["g"] = m.heads * (m.vdim if m.gate else 1)
+        self.first_values = config.mixes_values_first(layer_index)
         self.out_width = m.heads * m.vdim
 
         def param(shape, dtype):
@@ -41,6 +42,7 @@ class GroupedAttention(torch.nn.Module):
         self.sinks = param(m.heads, torch.float32) if m.sink else None
         self.bias_rows = m.distance_bias.rows_by_distance() if m.distance_bias is not None else None
         self.distance_bias = param((m.heads, len(self.bias_rows)), torch.float32) if self.bias_rows is not None else None
+        self.mix = param(1, dt) if m.value_mix and not self.first_values else None
         self.lambda_ = 0.0  # weight of the second map
 
     @property
@@ -61,14 +63,21 @@ class GroupedAttention(torch.nn.Module):
                 out["k.b"] = (self.inputs["k"],)
         if m.sink:
             out["sink"] = (m.heads,)
+        if self.mix is not None:
+            out["vmix"] = ()
         if m.distance_bias is not None:
             out["rel"] = (m.distance_bias.rows, m.heads)
         if m.diff is not None:
             out.update({k: (m.dim,) for k in ("lq1", "lk1", "lq2", "lk2")})
         return out
 
+    def ignored_tensors(self) -> set:
+        return {"vmix"} - set(self.checkpoint_tensors())
+
     def load(self, get) -> None:
         m = self.mixer
+        if self.mix is not None:
+            self.mix.data.copy_(get("vmix").reshape(1))
         for dst, name in ((self.q_bias, "q.b"), (self.k_bias, "k.b"), (self.sinks, "sink")):
             if dst is not None:
                 dst.data.copy_(get(name))
@@ -78,8 +87,9 @@ class GroupedAttention(torch.nn.Module):
             dots = [float((get("lq" + i).double() * get("lk" + i).double()).sum()) for i in "12"]
             self.lambda_ = math.exp(dots[0]) - math.exp(dots[1]) + m.diff
 
-    def forward(self, x, proj, column: int, out, out_column: int, scale: float, ctx, rope) -> None:
-        """``proj`` [T, ...]: this part's columns from ``column`` on; ``out`` [T, ...]: its output, times ``scale``, from ``out_column`` on."""
+    def forward(self, x, proj, column: int, out, out_column: int, scale: float, ctx, rope, step=None) -> None:
+        """``proj`` [T, ...]: this part's columns from ``column`` on; ``out`` [T, ...]: its output, times ``scale``, from ``out_column`` on.
+        ``step`` (shared by the layers of one forward) carries the first mixing layer's values on to the others."""
         m, T, es = self.mixer, proj.shape[0], proj.element_size()
         at, c = {}, column
         for name, n in self.inputs.items():
@@ -106,6 +116,11 @@ class GroupedAttention(torch.nn.Module):
             r.off_k, r.k_vecs, r.off_v, r.v_vecs = at["k"], m.kv_heads * m.maps, at.get("v", at["k"]), m.kv_heads
             r.k_bias = None if self.k_bias is None else self.k_bias.data_ptr()
             r.v_bias = r.k_bias if m.values_from_keys else None
+            if self.first_values:
+                step["first_values"] = torch.empty((T, m.kv_heads * m.vdim), dtype=proj.dtype, device=proj.device)
+                r.v_first_out = step["first_values"].data_ptr()
+            elif self.mix is not None:
+                r.v_first_in, r.mix = step["first_values"].data_ptr(), self.mix.data_ptr()
         if r.q_vecs or r.k_vecs:
             ops.struct_kernel("rotate_append", r, pool)
         decode, tc = ctx.is_decode_only(), self.tensor_cores
@@ -123,6 +138,8 @@ class GroupedAttention(torch.nn.Module):
         a.num_chunks, a.chunk_size, a.num_splits = pool.shape[0], pool.shape[1], 1
         a.softcap = m.softcap or 0.0
         a.sinks = None if self.sinks is None else self.sinks.data_ptr()
+        if m.head_gate:
+            a.gate, a.gate_ld = proj.data_ptr() + at["g"] * es, proj.stride(0)
         if self.distance_bias is not None:
             a.distance_bias, a.bias_len = self.distance_bias.data_ptr(), self.distance_bias.shape[1]
         if decode:

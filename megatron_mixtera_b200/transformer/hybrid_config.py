@@ -40,13 +40,20 @@ class LatentAttentionConfig:
     vdim: int
     kv_rank: int
     scale: float
-    rot: RotaryConfig
+    rot: Optional[RotaryConfig] = None
     window: Optional[int] = None   # keys seen, the token itself included; None: all earlier ones
     kv_from: Optional[int] = None  # 0-based layer whose cached rows this layer reads instead of making its own
+    q_rank: Optional[int] = None   # queries come from a normed latent of their own; None: straight from the layer's input
+    sink: bool = False             # one more term per head in the softmax denominator
+    gate: str = "head"             # sigmoid gates on the output: one per "head", or one per "value" channel of every head
 
     def __post_init__(self):
-        if self.rot.dims % 2 or not 0 <= self.rot.dims <= self.rot_dim:
+        if self.rot is not None and (self.rot.dims % 2 or not 0 <= self.rot.dims <= self.rot_dim):
             raise ValueError("rot.dims must be even and at most rot_dim")
+        if self.q_rank is not None and self.rot_dim:
+            raise ValueError("queries that come from a latent have no rotated part")
+        if self.gate not in ("head", "value"):
+            raise ValueError("gates belong to heads or to value channels")
         if self.window is not None and self.window < 1:
             raise ValueError("a window holds at least the token itself")
 
@@ -219,7 +226,9 @@ class GroupedAttentionConfig:
     sink: bool = False                   # one more term per head in the softmax denominator
     distance_bias: Optional[DistanceBias] = None
     diff: Optional[float] = None
-    gate: bool = False                   # heads times sigmoid of a projection (differential attention)
+    gate: bool = False                   # value channels times sigmoid of a projection (differential attention)
+    head_gate: bool = False              # heads times sigmoid of a projection, one number each (one map)
+    value_mix: bool = False              # values mixed with those of the first layer that mixes them
     kv_from: Optional[int] = None        # 0-based layer whose cached rows this layer reads instead of making its own
 
     def __post_init__(self):
@@ -233,8 +242,12 @@ class GroupedAttentionConfig:
             raise ValueError("rot.dims must be even and at most dim")
         if self.diff is None and self.gate or self.diff is not None and (self.sink or self.distance_bias is not None):
             raise ValueError("differential attention comes with a gate and without sinks or a distance bias")
+        if self.diff is not None and self.head_gate:
+            raise ValueError("differential attention gates value channels, not heads")
         if self.values_from_keys and (self.dim != self.vdim or self.diff is not None):
             raise ValueError("values that are keys have their size, and one map")
+        if self.value_mix and (self.values_from_keys or self.kv_from is not None):
+            raise ValueError("values are mixed where a layer projects its own")
 
     @property
     def maps(self) -> int:
@@ -279,6 +292,19 @@ class MatrixMemoryConfig:
 
 
 @dataclass(frozen=True)
+class GatedScanConfig:
+    """Gated recurrence, element by element, whose gates read the current token only (minGRU)."""
+
+    width: int
+
+    def cached_row_width(self) -> int:
+        return 0
+
+    def request_state(self, hidden_size: int, dtype: torch.dtype) -> Optional[dict]:
+        return {"state": ((self.width,), torch.float32)}
+
+
+@dataclass(frozen=True)
 class SideBySideConfig:
     """Mixers that read the same input and whose outputs are added up with constant factors."""
 
@@ -301,16 +327,22 @@ class SideBySideConfig:
 
 
 MixerConfig = Union[LatentAttentionConfig, DeltaRuleConfig, ShortConvAttentionConfig, WkvConfig, GatedDeltaConfig, GroupedAttentionConfig,
-                    MatrixMemoryConfig, SideBySideConfig]
+                    MatrixMemoryConfig, GatedScanConfig, SideBySideConfig]
 
 
 @dataclass(frozen=True)
 class ExpertConfig:
-    """One gated feed-forward: g' sigmoid(alpha g') (u' + 1), g' = min(g, limit), u' clamped to [-limit, limit]; without a limit silu(g) u."""
+    """One gated feed-forward: g' sigmoid(alpha g') (u' + 1), g' = min(g, limit), u' clamped to [-limit, limit]; without a limit silu(g) u.
+    ``gated`` False: max(u, 0)^2 of one projection."""
 
     ff: int
     limit: Optional[float] = None
     alpha: float = 1.702
+    gated: bool = True
+
+    def __post_init__(self):
+        if not self.gated and self.limit is not None:
+            raise ValueError("limits belong to gated feed-forwards")
 
 
 @dataclass(frozen=True)
@@ -326,19 +358,26 @@ class SoftmaxRouting:
 
 
 @dataclass(frozen=True)
+class ChosenSoftmaxRouting:
+    """Scores are logits plus a bias; the softmax over the chosen ones alone weighs the experts' outputs."""
+
+
+@dataclass(frozen=True)
 class MoeConfig:
     experts: int
     top: int  # experts per token; without ``routing`` their sigmoid scores weigh their inputs
     expert: ExpertConfig
-    shared: Optional[ExpertConfig] = None  # runs for every token, times a gate of its own
-    routing: Optional[SoftmaxRouting] = None
+    shared: Optional[ExpertConfig] = None  # runs for every token, times a gate of its own where the scores are sigmoids
+    routing: Union[SoftmaxRouting, ChosenSoftmaxRouting, None] = None
 
     def __post_init__(self):
         r = self.routing
         columns, reachable = self.experts, self.experts
-        if (r is None) != (self.expert.limit is not None) or (r is not None and self.shared is not None):
-            raise ValueError("softmax routing goes with plain gated experts and no shared one")
-        if r is not None:
+        if (r is None) != (self.expert.limit is not None) or (isinstance(r, SoftmaxRouting) and self.shared is not None):
+            raise ValueError("softmax routing goes with experts without limits, and without a shared one where groups are kept")
+        if self.shared is not None and (self.shared.gated != self.expert.gated or (self.shared.limit is None) != (self.expert.limit is None)):
+            raise ValueError("the shared expert has the form of the others")
+        if isinstance(r, SoftmaxRouting):
             columns = self.experts + r.identity
             if r.identity < 0 or not 1 <= r.keep_groups <= r.groups or columns % r.groups:
                 raise ValueError("experts and identity experts form equal groups, at least one of which is kept")
@@ -373,13 +412,15 @@ class HybridConfig:
     defer_logits_gather: bool = True
     # "output_norm": sublayers one after the other with norms on their outputs, embedding norm, tied head (`HybridModel`);
     # "parallel": mixer and feed-forward side by side on two norms of the same stream, scaled embedding, a head of its own
-    # (`ParallelHybridModel`)
+    # (`ParallelHybridModel`); with ``input_taps`` both read ONE norm, each through a short causal filter of its own
     # "streams": sublayers one after the other with layer norms on their inputs, ``streams`` residual streams that every sublayer blends
     # and mixes (0: one plain residual stream), scaled embedding, tied head (`StreamHybridModel`)
     block: str = "output_norm"
     streams: int = 0
     embedding_scale: float = 1.0
     logit_scale: float = 1.0
+    norm_offset: float = 1.0  # added to the norms' stored weights ("parallel")
+    input_taps: int = 0       # taps of the filters in front of the sublayers, 0: none ("parallel")
 
     def __post_init__(self):
         self.layers = tuple(self.layers)
@@ -388,9 +429,15 @@ class HybridConfig:
         if self.tensor_model_parallel_size != 1:
             raise NotImplementedError("hybrid decoders run on one GPU")
         if self.block == "parallel":
-            mixing = [x.mixer for x in self.layers if isinstance(x.mixer, ShortConvAttentionConfig) and x.mixer.value_mix]
+            mixing = [x.mixer for x in self.layers if getattr(x.mixer, "value_mix", False)]
             if len({(m.kv_heads, m.vdim) for m in mixing}) > 1:
                 raise ValueError("layers whose values are mixed must agree in their number and size")
+        if self.input_taps:
+            _check_taps(self.input_taps)
+            if self.block != "parallel":
+                raise ValueError("input filters belong to parallel blocks")
+        if self.block == "streams" and any(x.moe is not None and x.moe.shared is not None for x in self.layers):
+            raise ValueError("shared experts belong to parallel blocks")
         if self.streams > 16:
             raise ValueError("at most 16 residual streams")
         for i, layer in enumerate(self.layers):
@@ -413,6 +460,21 @@ class HybridConfig:
     @property
     def num_layers(self) -> int:
         return len(self.layers)
+
+    def mixes_values_first(self, index: int) -> bool:
+        """Whether layer ``index`` is the first whose values the others' are mixed with."""
+        mixing = [i for i, x in enumerate(self.layers) if getattr(x.mixer, "value_mix", False)]
+        return mixing[:1] == [index]
+
+    def request_state(self, index: int) -> Optional[dict]:
+        """What layer ``index`` keeps per request: its mixer's state and the inputs its filters look back at."""
+        state = self.layers[index].mixer.request_state(self.hidden_size, self.params_dtype)
+        if self.input_taps == 0:
+            return state
+        out = dict(state or {})  # (empty: nothing to keep, but the kernels ask for the slots)
+        if self.input_taps > 1:
+            out["input"] = ((self.input_taps - 1, self.hidden_size), self.params_dtype)
+        return out
 
     def for_layer(self, index: int) -> "HybridConfig":
         """The view of layer ``index`` that per-layer modules (MLP) read."""

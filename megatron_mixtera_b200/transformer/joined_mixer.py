@@ -5,11 +5,12 @@ from __future__ import annotations
 import torch
 
 from ..tensor_parallel.layers import ColumnParallelLinear, RowParallelLinear, _device
+from .gated_scan import GatedScan
 from .grouped_attention import GroupedAttention
-from .hybrid_config import GroupedAttentionConfig, HybridConfig, MatrixMemoryConfig, SideBySideConfig
+from .hybrid_config import GatedScanConfig, GroupedAttentionConfig, HybridConfig, MatrixMemoryConfig, SideBySideConfig
 from .matrix_memory import MatrixMemory
 
-PARTS = {GroupedAttentionConfig: GroupedAttention, MatrixMemoryConfig: MatrixMemory}
+PARTS = {GatedScanConfig: GatedScan, GroupedAttentionConfig: GroupedAttention, MatrixMemoryConfig: MatrixMemory}
 
 
 def _pad(n: int) -> int:
@@ -51,6 +52,9 @@ class JoinedMixer(torch.nn.Module):
             out["o.b"] = (H,)
         return out
 
+    def ignored_tensors(self) -> set:
+        return {pre + k for pre, p in zip(self.prefixes, self.parts) for k in getattr(p, "ignored_tensors", set)()}
+
     def load(self, get) -> None:
         w_in, w_out = self.linear_in.weight.data, self.linear_proj.weight.data
         w_in.zero_()
@@ -62,13 +66,15 @@ class JoinedMixer(torch.nn.Module):
         if self.output_bias is not None:
             self.output_bias.data.copy_(get("o.b"))
 
-    def forward(self, x, ctx, rope):
-        """``x`` [T, H] -> the output linear's partial sums.  ``rope``: per part, the rotation tables (or None)."""
-        proj, _ = self.linear_in(x)
+    def forward(self, x, ctx, rope, step=None):
+        """``x`` [T, H] -> the output linear's partial sums.  ``rope``: per part, the rotation tables (or None); ``step``: what the layers of
+        one forward share."""
+        takes_partials = len(self.parts) == 1 and ctx.is_decode_only() and getattr(self.parts[0], "takes_partials", False)
+        proj, _ = self.linear_in(x, defer_reduction=takes_partials)
         out = torch.empty((x.shape[0], self.linear_proj.weight.shape[1]), dtype=x.dtype, device=x.device)
         if self.padded_outputs or not ctx.is_decode_only() and (
                 ctx.using_cuda_graph_this_step() or ctx.padded_active_token_count != ctx.active_token_count):
             out.zero_()  # padding tokens belong to no row, padding columns to no part
         for p, c, o, s, tables in zip(self.parts, self.columns, self.out_columns, self.scales, rope):
-            p(x, proj, c, out, o, s, ctx, tables)
+            p(x, proj, c, out, o, s, ctx, tables, step)
         return self.linear_proj(out, defer_reduction=True)[0]

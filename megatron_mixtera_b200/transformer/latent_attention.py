@@ -40,14 +40,29 @@ class LatentAttention(torch.nn.Module):
         m, dt, dev = mixer, config.params_dtype, _device()
         self.cache_layer_number = (layer_index if m.kv_from is None else m.kv_from) + 1
         self.owns_rows = m.kv_from is None
-        # one linear for everything that reads the layer's input: [queries | latent, shared key | gates]
-        q_width = m.heads * (m.dim + m.rot_dim)
-        down = m.kv_rank + m.rot_dim if self.owns_rows else 0
-        self.dkv_offset = q_width if self.owns_rows else -1
-        self.gate_offset = q_width + down
-        self.in_width = q_width + down + m.heads
-        padded = -(-self.in_width // 8) * 8  # whole 16-byte vectors per row; the added rows are zero
+        # one linear for everything that reads the layer's input: [queries or their latent | latent, shared key | gates]
+        self.query_width = m.heads * (m.dim + m.rot_dim)
+        self.gate_width = m.heads * (m.vdim if m.gate == "value" else 1)
+        self.inputs = {"q": self.query_width} if m.q_rank is None else {"dq": m.q_rank}
+        if self.owns_rows:
+            self.inputs["dkv"] = m.kv_rank + m.rot_dim
+        self.inputs["g"] = self.gate_width
+        starts_at_vectors = m.gate == "value"  # (gates are read as vectors there)
+        self.offsets, at = {}, 0
+        for name, n in self.inputs.items():
+            at = -(-at // 8) * 8 if starts_at_vectors else at
+            self.offsets[name] = at
+            at += n
+        self.dkv_offset, self.gate_offset = self.offsets.get("dkv", -1), self.offsets["g"]
+        self.in_width = at
+        padded = -(-at // 8) * 8  # whole 16-byte vectors per row; the added rows are zero
         self.linear_in = ColumnParallelLinear(config.hidden_size, padded, config=config, bias=False)
+        self.query_up = self.query_norm = self.sinks = None
+        if m.q_rank is not None:
+            self.query_up = torch.nn.Parameter(torch.empty(self.query_width, m.q_rank, dtype=dt, device=dev), requires_grad=False)
+            self.query_norm = torch.nn.Parameter(torch.ones(m.q_rank, dtype=dt, device=dev), requires_grad=False)
+        if m.sink:
+            self.sinks = torch.nn.Parameter(torch.zeros(m.heads, dtype=torch.float32, device=dev), requires_grad=False)
         # absorbed: per head [latent][dim]; expanded: [keys of all heads | values of all heads] x latent
         self.key_up = torch.nn.Parameter(torch.empty(m.heads * m.kv_rank, m.dim, dtype=dt, device=dev), requires_grad=False)
         self.key_value_up = torch.nn.Parameter(torch.empty(m.heads * (m.dim + m.vdim), m.kv_rank, dtype=dt, device=dev),
@@ -61,18 +76,27 @@ class LatentAttention(torch.nn.Module):
     def checkpoint_tensors(self) -> dict:
         """Checkpoint name (below the layer's mixer) -> shape."""
         m, H = self.mixer, self.config.hidden_size
-        out = {"q": (m.heads * (m.dim + m.rot_dim), H), "uk": (m.heads * m.dim, m.kv_rank), "uv": (m.heads * m.vdim, m.kv_rank),
-               "g": (m.heads, H), "o": (H, m.heads * m.vdim)}
+        out = {name: (n, H) for name, n in self.inputs.items()}
+        out.update({"uk": (m.heads * m.dim, m.kv_rank), "uv": (m.heads * m.vdim, m.kv_rank), "o": (H, m.heads * m.vdim)})
+        if m.q_rank is not None:
+            out.update({"dq.norm": (m.q_rank,), "uq": (self.query_width, m.q_rank)})
+        if m.sink:
+            out["sink"] = (m.heads,)
         if self.owns_rows:
-            out.update({"dkv": (m.kv_rank + m.rot_dim, H), "dkv.norm": (m.kv_rank,)})
+            out["dkv.norm"] = (m.kv_rank,)
         return out
 
     def load(self, get) -> None:
         m = self.mixer
-        parts = [get("q")] + ([get("dkv")] if self.owns_rows else []) + [get("g")]
         w = self.linear_in.weight.data
         w.zero_()
-        w[: self.in_width].copy_(torch.cat([p.to(w.device) for p in parts]))
+        for name, n in self.inputs.items():
+            w[self.offsets[name]: self.offsets[name] + n].copy_(get(name))
+        if m.q_rank is not None:
+            self.query_up.data.copy_(get("uq"))
+            self.query_norm.data.copy_(get("dq.norm"))
+        if m.sink:
+            self.sinks.data.copy_(get("sink"))
         self.key_up.data.copy_(get("uk").view(m.heads, m.dim, m.kv_rank).transpose(1, 2).reshape(m.heads * m.kv_rank, m.dim))
         self.key_value_up.data.copy_(torch.cat([get("uk"), get("uv")]))
         if self.owns_rows:
@@ -85,26 +109,33 @@ class LatentAttention(torch.nn.Module):
 
     expand_prompts = True  # False: the absorbed form everywhere
 
+    def prefill_unit_tokens(self) -> int:
+        """Tokens per work unit of the absorbed prompt kernel (it cuts a unit into blocks of query rows itself)."""
+        return 16
+
     def _expansion(self, x, ctx):
         m = self.mixer
         if not (self.expand_prompts and x.dtype == torch.bfloat16 and ops.latent_prompt_supported(m.dim, m.rot_dim, m.vdim, m.heads)):
             return None
         return ctx.expanded_keys(m.window)
 
-    def forward(self, x, ctx, rope):
+    def forward(self, x, ctx, rope=None, step=None):
         """``x`` [T, H] -> the output linear's partial sums."""
         m, T, dev = self.mixer, x.shape[0], x.device
         proj, _ = self.linear_in(x)
         expanded = self._expansion(x, ctx)
         # queries: the absorbed form fills whole rows, the expanded one needs the rotated part alone
         q_stride, q_rot_at = (m.row_width, m.kv_pad) if expanded is None else (m.row_width - m.kv_pad, 0)
-        q_full = torch.empty((T, m.heads, q_stride), dtype=x.dtype, device=dev)
+        q_full = torch.empty((T, m.heads, max(q_stride, 8)), dtype=x.dtype, device=dev)
         pool = ctx.latent_cache(self.cache_layer_number)
         decode = ctx.is_decode_only()
         a = _lib.LatentArgs()
-        a.proj, a.proj_ld, a.dkv_offset, a.gate_offset = proj.data_ptr(), proj.stride(0), self.dkv_offset, self.gate_offset
+        a.proj, a.proj_ld, a.dkv_offset = proj.data_ptr(), proj.stride(0), self.dkv_offset
+        a.gate_offset = self.gate_offset if m.gate == "head" or expanded is not None else -1  # (absorbed: values are gated behind the kernel)
         a.norm_weight = None if self.latent_norm is None else self.latent_norm.data_ptr()
-        a.rope_cos, a.rope_sin, a.max_positions = rope[0].data_ptr(), rope[1].data_ptr(), rope[0].shape[0]
+        a.max_positions = 1
+        if rope is not None:
+            a.rope_cos, a.rope_sin, a.max_positions = rope[0].data_ptr(), rope[1].data_ptr(), rope[0].shape[0]
         a.token_to_pos = ctx.token_to_position_in_request.data_ptr()
         a.token_to_chunk_idx = ctx.token_to_chunk_idx.data_ptr()
         a.token_to_local_pos = ctx.token_to_local_position_within_kv_chunk.data_ptr()
@@ -112,16 +143,27 @@ class LatentAttention(torch.nn.Module):
         a.max_chunks_per_row = ctx.request_to_kv_chunk_ids_cudagraph_only.shape[1]
         a.pool, a.num_chunks, a.chunk_size = pool.data_ptr(), pool.shape[0], pool.shape[1]
         a.q_full, a.q_stride, a.q_rot_at = q_full.data_ptr(), q_stride, q_rot_at
-        a.num_tokens, a.heads, a.dim, a.rot_dim, a.rot_dims = T, m.heads, m.dim, m.rot_dim, m.rot.dims
+        a.num_tokens, a.heads, a.dim, a.rot_dim, a.rot_dims = T, m.heads, m.dim, m.rot_dim, 0 if m.rot is None else m.rot.dims
         a.kv_rank, a.kv_pad, a.row_width = m.kv_rank, m.kv_pad, m.row_width
         a.window, a.scale, a.eps = m.window or 0, m.scale, self.config.layernorm_epsilon
         a.dtype, a.num_splits = ops.dtype_code(x.dtype), 1
+        a.sinks = None if self.sinks is None else self.sinks.data_ptr()
         values = torch.empty((T, m.heads * m.vdim), dtype=x.dtype, device=dev)
+        queries = proj
+        if m.q_rank is not None:
+            q_latent = torch.empty((T, m.q_rank), dtype=x.dtype, device=dev)
+            a.q_latent_out, a.q_rank, a.q_latent_offset = q_latent.data_ptr(), m.q_rank, self.offsets["dq"]
+            a.q_norm_weight = self.query_norm.data_ptr()
+            queries = torch.empty((T, self.query_width), dtype=x.dtype, device=dev)
+            a.q, a.q_ld = queries.data_ptr(), queries.stride(0)
         if expanded is not None:
             table, num_keys = expanded
             key_rows = torch.empty((num_keys, m.row_width), dtype=x.dtype, device=dev)
             ops.latent_append(a, pool)
+            if m.q_rank is not None:
+                ops.linear(q_latent, self.query_up, out=queries)
             a.num_rows, a.num_keys, a.max_row_tokens, a.vdim = table.shape[1] - 1, num_keys, ctx.max_seqlen_q, m.vdim
+            a.value_gates = int(m.gate == "value")
             a.cu_tokens = ctx.cu_query_seq_lengths_cudagraph_only.data_ptr()
             a.cu_keys, a.key_start, a.key_rows = table[0].data_ptr(), table[1].data_ptr(), key_rows.data_ptr()
             ops.latent_gather(a, pool)
@@ -136,10 +178,17 @@ class LatentAttention(torch.nn.Module):
             if x.dtype == torch.bfloat16:
                 a.num_splits = choose_latent_splits(T, m.heads, m.window, ctx.max_sequence_length)
         else:
-            a.units, a.num_units, a.unit_tokens = ctx.prefill_units.data_ptr(), ctx.prefill_unit_count, ctx.prefill_q_block
+            a.unit_tokens = self.prefill_unit_tokens()
+            units, a.num_units = ctx.prefill_units_of(a.unit_tokens)
+            a.units = units.data_ptr()
+        if m.q_rank is not None:
+            ops.latent_append(a, pool)
+            ops.linear(q_latent, self.query_up, out=queries)
         # absorbed queries: per head W_uk^T q
-        ops.linear(proj, self.key_up, out=q_full.view(T, -1), batch=m.heads, x_batch=m.dim + m.rot_dim, y_batch=m.row_width, K=m.dim)
-        ops.latent_append(a, pool)
+        ops.linear(queries, self.key_up, out=q_full.view(T, -1), batch=m.heads, x_batch=m.dim + m.rot_dim, y_batch=m.row_width, K=m.dim)
+        if m.q_rank is None:
+            ops.latent_append(a, pool)
         ops.latent_attention(a, pool)
-        ops.linear(latent_out, self.value_up, out=values, batch=m.heads, x_batch=m.kv_rank, y_batch=m.vdim, K=m.kv_rank)
+        gates = proj[:, self.gate_offset:] if m.gate == "value" else None
+        ops.linear(latent_out, self.value_up, out=values, batch=m.heads, x_batch=m.kv_rank, y_batch=m.vdim, K=m.kv_rank, gate=gates)
         return self.linear_proj(values, defer_reduction=True)[0]

@@ -38,7 +38,7 @@ class MatrixMemory(torch.nn.Module):
         self.gate_bias.data.copy_(torch.cat([get("i.b"), get("f.b")]))
         self.norm_weight.data.copy_(get("norm"))
 
-    def forward(self, x, proj, column: int, out, out_column: int, scale: float, ctx, rope=None) -> None:
+    def forward(self, x, proj, column: int, out, out_column: int, scale: float, ctx, rope=None, step=None) -> None:
         """Decode steps run one fused kernel; other steps find every token's factors, scan and finish."""
         m, T, dev = self.mixer, proj.shape[0], proj.device
         state = ctx.recurrent_state(self.layer_number, "state")

@@ -1,5 +1,5 @@
 """Mixture of experts: every token runs its `top` best experts - on its input times their sigmoid scores, beside a gated shared expert, or
-(`SoftmaxRouting`) with their softmax scores as weights of the outputs.  Tokens are sorted by expert on the device; the products of all experts are
+(`SoftmaxRouting`, `ChosenSoftmaxRouting`) with softmax scores as weights of the outputs.  Tokens are sorted by expert on the device; the products of all experts are
 one grouped GEMM."""
 from __future__ import annotations
 
@@ -7,7 +7,7 @@ import torch
 
 from .. import _lib, ops
 from ..tensor_parallel.layers import _device
-from .hybrid_config import HybridConfig, MoeConfig
+from .hybrid_config import ChosenSoftmaxRouting, HybridConfig, MoeConfig, SoftmaxRouting
 
 
 def _padded(ff: int) -> int:
@@ -50,39 +50,53 @@ class MixtureOfExperts(torch.nn.Module):
 
         self.ff = _padded(moe.expert.ff)
         # router rows (identity experts' included), then the shared expert's gate
-        self.columns = moe.experts + (moe.routing.identity if moe.routing is not None else 0)
-        self.router = param(-(-(self.columns + (moe.shared is not None)) // 8) * 8, H)
+        self.columns = moe.experts + (moe.routing.identity if isinstance(moe.routing, SoftmaxRouting) else 0)
+        self.shared_gated = moe.shared is not None and moe.routing is None
+        self.router = param(-(-(self.columns + self.shared_gated) // 8) * 8, H)
+        # added to the scores that choose (a bias on the logits, part of the score, where the chosen ones' softmax weighs)
         self.correction = param(self.columns) if moe.routing is not None else None
-        self.up, self.down = param(moe.experts, 2 * self.ff, H), param(moe.experts, H, self.ff)
+        self.correction_name = "router.b" if isinstance(moe.routing, ChosenSoftmaxRouting) else "correction"
+        rows = 2 if moe.expert.gated else 1
+        self.names = ("gate", "up", "down") if moe.expert.gated else ("up", "down")
+        self.up, self.down = param(moe.experts, rows * self.ff, H), param(moe.experts, H, self.ff)
         self.shared_ff, self.shared_up, self.shared_down = 0, None, None
         if moe.shared is not None:
             self.shared_ff = _padded(moe.shared.ff)
-            self.shared_up, self.shared_down = param(2 * self.shared_ff, H), param(H, self.shared_ff)
+            self.shared_up, self.shared_down = param(rows * self.shared_ff, H), param(H, self.shared_ff)
 
     def checkpoint_tensors(self) -> dict:
         H, c = self.config.hidden_size, self.moe
         out = {"router": (self.columns, H)}
         if c.routing is not None:
-            out["correction"] = (self.columns,)
+            out[self.correction_name] = (self.columns,)
         parts = [(f"e{e}", c.expert.ff) for e in range(c.experts)]
         if c.shared is not None:
             parts.append(("shared", c.shared.ff))
-            out["shared.sg"] = (1, H)
+            if self.shared_gated:
+                out["shared.sg"] = (1, H)
         for name, ff in parts:
-            out.update({f"{name}.gate": (ff, H), f"{name}.up": (ff, H), f"{name}.down": (H, ff)})
+            out.update({f"{name}.{k}": (H, ff) if k == "down" else (ff, H) for k in self.names})
         return out
 
     def load(self, get) -> None:
         c, dev = self.moe, self.router.device
         self.router.data[: self.columns].copy_(get("router"))
         if self.correction is not None:
-            self.correction.data.copy_(get("correction"))
+            self.correction.data.copy_(get(self.correction_name))
+
+        def put_up(dst, name, ff):
+            if c.expert.gated:
+                dst.copy_(interleave_up(get(f"{name}.gate").to(dev), get(f"{name}.up").to(dev)))
+            else:
+                dst[:ff].copy_(get(f"{name}.up"))
+
         for e in range(c.experts):
-            self.up.data[e].copy_(interleave_up(get(f"e{e}.gate").to(dev), get(f"e{e}.up").to(dev)))
+            put_up(self.up.data[e], f"e{e}", c.expert.ff)
             self.down.data[e, :, : c.expert.ff].copy_(get(f"e{e}.down"))
         if c.shared is not None:
-            self.router.data[c.experts].copy_(get("shared.sg")[0])
-            self.shared_up.data.copy_(interleave_up(get("shared.gate").to(dev), get("shared.up").to(dev)))
+            if self.shared_gated:
+                self.router.data[c.experts].copy_(get("shared.sg")[0])
+            put_up(self.shared_up.data, "shared", c.shared.ff)
             self.shared_down.data[:, : c.shared.ff].copy_(get("shared.down"))
 
     @staticmethod
@@ -99,9 +113,14 @@ class MixtureOfExperts(torch.nn.Module):
         a = _lib.MoeArgs()
         a.num_tokens, a.width, a.experts, a.top, a.ff, a.shared_ff = T, H, c.experts, c.top, self.ff, self.shared_ff
         a.limit, a.alpha, a.simt, a.dtype = c.expert.limit or 0.0, c.expert.alpha, int(simt), ops.dtype_code(dt)
+        a.relu2 = int(not c.expert.gated)
+        identity = 0
+        if isinstance(c.routing, SoftmaxRouting):
+            r, identity = c.routing, c.routing.identity
+            a.plain, a.identity, a.groups, a.keep_groups, a.weight_scale = 1, identity, r.groups, r.keep_groups, r.scale
+        elif c.routing is not None:
+            a.plain, a.groups, a.keep_groups, a.weight_scale = 2, 1, 1, 1.0
         if c.routing is not None:
-            r = c.routing
-            a.plain, a.identity, a.groups, a.keep_groups, a.weight_scale = 1, r.identity, r.groups, r.keep_groups, r.scale
             a.correction = self.correction.data_ptr()
         a.tile_tokens = self.tile_tokens(pairs, c.experts, simt)
         a.max_tiles = pairs // a.tile_tokens + min(c.experts, pairs)
@@ -121,14 +140,14 @@ class MixtureOfExperts(torch.nn.Module):
         shared_rows = shared_inter = None
         if c.shared is not None:
             shared_inter, shared_rows = torch.empty((T, self.shared_ff), dtype=dt, device=dev), torch.empty((T, H), dtype=dt, device=dev)
-            a.shared_gate, a.shared_up, a.shared_down = shared_gate, self.shared_up.data_ptr(), self.shared_down.data_ptr()
-            a.shared_inter, a.shared_y, a.shared_limit = shared_inter.data_ptr(), shared_rows.data_ptr(), c.shared.limit
+            a.shared_gate = shared_gate if self.shared_gated else None
+            a.shared_up, a.shared_down = self.shared_up.data_ptr(), self.shared_down.data_ptr()
+            a.shared_inter, a.shared_y, a.shared_limit = shared_inter.data_ptr(), shared_rows.data_ptr(), c.shared.limit or 0.0
         logits = ops.linear_partials(x, self.router)  # fp32 sums of exact products: the router's 32-bit logits
         a.router, a.router_splits = ops.partials_of(logits)
         a.router_ld = self.router.shape[0]
         for kernel in ("moe_route", "moe_gather", "moe_up", "moe_down"):
             ops.struct_kernel(kernel, a, x)
-        if c.routing is not None:
-            return ExpertOutputs(rows, words, words[starts[4]:], c.top, c.experts, weights=words[starts[1]:], identity=c.routing.identity, input=x)
-        gates = words[starts[3]: starts[3] + T].view(torch.float32) if c.shared is not None else None
-        return ExpertOutputs(rows, words, words[starts[4]:], c.top, c.experts, shared_rows, gates)
+        gates = words[starts[3]: starts[3] + T].view(torch.float32) if self.shared_gated else None
+        weights = words[starts[1]:] if c.routing is not None else None
+        return ExpertOutputs(rows, words, words[starts[4]:], c.top, c.experts, shared_rows, gates, weights, identity, x if identity else None)

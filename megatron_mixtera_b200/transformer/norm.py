@@ -9,6 +9,7 @@ from __future__ import annotations
 import torch
 
 from .. import ops
+from .short_conv import short_conv_args
 
 
 class B200Norm(torch.nn.Module):
@@ -120,12 +121,12 @@ class StreamNorm(torch.nn.Module):
 
 class ParallelNorm(torch.nn.Module):
     """Everything a parallel block adds to the 32-bit residual stream and the RMS norms of the result, in one kernel.  ``outputs``
-    norms of the same row (weights stored as the distance from one) feed the branches that run side by side."""
+    norms of the same row (weights stored as the distance from ``config.norm_offset``) feed the branches that run side by side."""
 
     def __init__(self, config, hidden_size: int, eps: float, outputs: int = 2, out_scale: float = 1.0):
         super().__init__()
         dev = torch.device("cuda", torch.cuda.current_device()) if torch.cuda.is_available() else torch.device("cpu")
-        self.eps, self.out_scale = eps, out_scale
+        self.eps, self.out_scale, self.gain = eps, out_scale, config.norm_offset
         self.weight = torch.nn.Parameter(torch.zeros((outputs, hidden_size), dtype=config.params_dtype, device=dev), requires_grad=False)
 
     def forward(self, hidden, pending, row_index=None):
@@ -133,5 +134,38 @@ class ParallelNorm(torch.nn.Module):
         only those rows are computed and ``hidden`` stays as it is."""
         rows = hidden.shape[0] if row_index is None else row_index.numel()
         out = [torch.empty((rows, hidden.shape[1]), dtype=self.weight.dtype, device=hidden.device) for _ in range(self.weight.shape[0])]
-        ops.residual_norm(hidden, pending, list(self.weight), out, eps=self.eps, gain=1.0, out_scale=self.out_scale, row_index=row_index)
+        ops.residual_norm(hidden, pending, list(self.weight), out, eps=self.eps, gain=self.gain, out_scale=self.out_scale, row_index=row_index)
+        return out
+
+
+class FilteredNorm(torch.nn.Module):
+    """Everything a parallel block adds to the 32-bit residual stream, ONE RMS norm of the result, and in front of each branch a short causal
+    filter of the normed rows over time, added to them: branch i reads u + filter_i(u).  The last taps - 1 normed rows are a request's
+    state.  One kernel in decode steps; the filters are a kernel of their own in the others."""
+
+    def __init__(self, config, hidden_size: int, eps: float, outputs: int, layer_number: int):
+        super().__init__()
+        dev = torch.device("cuda", torch.cuda.current_device()) if torch.cuda.is_available() else torch.device("cpu")
+        self.eps, self.gain, self.layer_number = eps, config.norm_offset, layer_number
+
+        def param(*shape):
+            return torch.nn.Parameter(torch.zeros(shape, dtype=config.params_dtype, device=dev), requires_grad=False)
+
+        self.weight, self.filters = param(hidden_size), param(outputs, config.input_taps, hidden_size)
+
+    def forward(self, hidden, pending, ctx):
+        """Adds ``pending`` (a `PendingRows`) to ``hidden`` [T, H] in place; what the branches read."""
+        state = ctx.recurrent_state(self.layer_number, "input") if self.filters.shape[1] > 1 else None
+        out = [torch.empty(hidden.shape, dtype=self.weight.dtype, device=hidden.device) for _ in range(self.filters.shape[0])]
+        if ctx.is_decode_only():
+            ops.residual_norm(hidden, pending, [self.weight], out, eps=self.eps, gain=self.gain, filters=list(self.filters), state=state,
+                              state_slots=(ctx.state_read_slots, ctx.state_write_slots))
+            return out
+        normed = torch.empty(hidden.shape, dtype=self.weight.dtype, device=hidden.device)
+        ops.residual_norm(hidden, pending, [self.weight], [normed], eps=self.eps, gain=self.gain)
+        T, taps, width = hidden.shape[0], *self.filters.shape[1:]
+        a = short_conv_args(ctx, proj=normed, filter_=self.filters[0], state=state, channels=width, taps=taps, out=out[0])
+        if len(out) > 1:
+            a.filter_2, a.out_2 = self.filters[1].data_ptr(), out[1].data_ptr()
+        ops.struct_kernel("conv_add", a, normed)
         return out

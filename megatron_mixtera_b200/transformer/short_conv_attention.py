@@ -8,33 +8,7 @@ from .. import _lib, ops
 from ..tensor_parallel.layers import ColumnParallelLinear, RowParallelLinear, _device
 from .attention import choose_attention_splits
 from .hybrid_config import HybridConfig, ShortConvAttentionConfig
-
-
-def short_conv_args(ctx, *, proj, filter_, state, channels: int, taps: int, out) -> _lib.ConvArgs:
-    """What the short-convolution kernels need of a step: where every token's request starts and keeps its last inputs."""
-    a = _lib.ConvArgs()
-    a.proj, a.proj_ld, a.filter, a.channels, a.taps = proj.data_ptr(), proj.stride(0), filter_.data_ptr(), channels, taps
-    a.state, a.state_slots = (None, 0) if state is None else (state.data_ptr(), state.shape[0])
-    step_rows(a, ctx, proj.shape[0])
-    a.out, a.dtype = out.data_ptr(), ops.dtype_code(proj.dtype)
-    return a
-
-
-def step_rows(a, ctx, num_tokens: int) -> None:
-    """The step's rows in an argument struct: state slots, and (steps that are not one token per row) which tokens a row has."""
-    a.state_in, a.state_out, a.num_tokens = ctx.state_read_slots.data_ptr(), ctx.state_write_slots.data_ptr(), num_tokens
-    if ctx.is_decode_only():
-        a.num_rows = num_tokens
-    else:
-        a.num_rows = ctx.padded_active_request_count
-        a.cu_tokens = ctx.cu_query_seq_lengths_cudagraph_only.data_ptr()
-        if hasattr(a, "row_of_token"):
-            a.row_of_token = ctx.token_to_block_table_row.data_ptr()
-
-
-def filter_of(taps: torch.Tensor) -> torch.Tensor:
-    """[channels, taps] as a checkpoint holds it -> [taps, channels]."""
-    return taps.transpose(0, 1).contiguous()
+from .short_conv import filter_of, short_conv_args
 
 
 class ShortConvAttention(torch.nn.Module):
@@ -42,8 +16,7 @@ class ShortConvAttention(torch.nn.Module):
         super().__init__()
         self.config, self.mixer, self.layer_number = config, mixer, layer_index + 1
         m, dt, dev = mixer, config.params_dtype, _device()
-        self.first_values = m.value_mix and not any(
-            isinstance(x.mixer, ShortConvAttentionConfig) and x.mixer.value_mix for x in config.layers[:layer_index])
+        self.first_values = config.mixes_values_first(layer_index)
         # one linear for queries | keys | values
         self.linear_qkv = ColumnParallelLinear(config.hidden_size, -(-m.conv_channels // 8) * 8, config=config, bias=False)
 
@@ -87,7 +60,7 @@ class ShortConvAttention(torch.nn.Module):
             self.mix.data.copy_(get("vmix").reshape(1))
         self.linear_proj.weight.data.copy_(get("o"))
 
-    def forward(self, x, ctx, step: dict):
+    def forward(self, x, ctx, rope=None, step=None):
         """``x`` [T, H] -> the output linear's partial sums.  ``step`` (shared by the layers of one forward) carries the first
         mixing layer's values on to the others."""
         m, T, dev = self.mixer, x.shape[0], x.device

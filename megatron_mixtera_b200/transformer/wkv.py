@@ -7,7 +7,7 @@ import torch
 from .. import _lib, ops
 from ..tensor_parallel.layers import RowParallelLinear, _device
 from .hybrid_config import HybridConfig, WkvConfig
-from .short_conv_attention import step_rows
+from .short_conv import step_rows
 
 WKV, DELTA = 0, 1  # B200_RECURRENCE_*
 
@@ -53,7 +53,7 @@ class Wkv(torch.nn.Module):
             dst.data.copy_(get(name))
         self.bonus.data.copy_(get("u").reshape(-1))
 
-    def forward(self, x, ctx, step=None):
+    def forward(self, x, ctx, rope=None, step=None):
         """``x`` [T, H] -> the output linear's partial sums."""
         m, (T, H), n, dev = self.mixer, x.shape, self.width, x.device
         # every projection's input

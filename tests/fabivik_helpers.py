@@ -147,7 +147,7 @@ def run_mixer(model, ctx, index, hs, schedule):
             for j in range(index + 1):
                 mixer = model.layers[j].mixer
                 if j == index or getattr(mixer, "first_values", False):
-                    y = mixer(x, ctx, step)
+                    y = mixer(x, ctx, step=step)
             ops.residual_norm(out, ops.PendingRows(partials=y), [], [], eps=1.0)
         row = 0
         for i, n in part:

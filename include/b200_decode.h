@@ -437,6 +437,7 @@ typedef struct {
   int64_t gate_ld;
   float out_scale, softcap, lambda, diff_scale, eps;
   int32_t bias_len, keep_first, maps;
+  int32_t value_gates; /* != 0 (b200_paged_prefill_attention, maps < 2): the gates are num_q_heads * value_dim columns, one per value channel */
 } b200_attention_args;
 
 size_t b200_paged_attention_workspace_bytes(int num_tokens, int num_q_heads, int head_dim, int num_splits);
@@ -586,6 +587,7 @@ typedef struct b200_latent_args {
   int64_t q_ld;
   int32_t q_rank, q_latent_offset;
   int32_t value_gates; /* b200_latent_prompt_attention: the gates are heads * vdim columns, one per value channel */
+  const int32_t* key_end; /* [rows] or NULL: position behind a row's last key; what cu_keys counts beyond (rows padded to whole chunks) repeats it */
 } b200_latent_args;
 /* b200_latent_gather: key_rows[e] = the pool row of expanded key e.
  * b200_latent_prompt_attention: out[t][head][vdim] = sigmoid(gate) * sum_j softmax(scale * (q . k_j + q_rot . k_rot_j)) v_j, the same

@@ -167,6 +167,7 @@ class AttentionArgs(ctypes.Structure):
         ("bias_len", c_int32),
         ("keep_first", c_int32),
         ("maps", c_int32),
+        ("value_gates", c_int32),
     ]
 
 
@@ -192,7 +193,7 @@ class LatentArgs(ctypes.Structure):
         (n, c_void_p) for n in ("cu_tokens", "cu_keys", "key_start", "key_rows", "key_values")] + [
         (n, c_int32) for n in ("num_rows", "num_keys", "max_row_tokens", "vdim")] + [
         (n, c_void_p) for n in ("sinks", "q", "q_norm_weight", "q_latent_out")] + [
-        ("q_ld", c_int64)] + [(n, c_int32) for n in ("q_rank", "q_latent_offset", "value_gates")]
+        ("q_ld", c_int64)] + [(n, c_int32) for n in ("q_rank", "q_latent_offset", "value_gates")] + [("key_end", c_void_p)]
 
 
 class DeltaArgs(ctypes.Structure):

@@ -100,6 +100,7 @@ struct Params {
   float lambda, diff_scale, eps;
   const __nv_bfloat16* gate;  // [T][gate_ld]: the difference is multiplied with sigmoid(gate), or (diff 0) a head's output with its column's
   int64_t gate_ld;
+  int value_gates;  // 1: a gate per value channel, not per head (prompts)
 };
 
 // First key that a token whose newest visible key is kv_len - 1 sees, and the tile that holds it.
@@ -121,7 +122,7 @@ __device__ __forceinline__ int64_t query_offset(const Params& p, int h, int g) {
 }
 // Factor on a finished output (kExtra, one map).
 __device__ __forceinline__ float output_factor(const Params& p, int64_t t, int head) {
-  return p.gate == nullptr ? p.out_scale : p.out_scale / (1.f + expf(-__bfloat162float(p.gate[t * p.gate_ld + head])));
+  return p.gate == nullptr || p.value_gates ? p.out_scale : p.out_scale / (1.f + expf(-__bfloat162float(p.gate[t * p.gate_ld + head])));
 }
 __device__ __forceinline__ float capped(const Params& p, float qk) {
   return p.cap_out * (1.f - __fdividef(2.f, 1.f + exp2f(qk * p.cap_in * (2.f * kLog2e))));
@@ -917,6 +918,17 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_con
       continue;
     }
     __nv_bfloat16* o = p.out + tok_r[r] * p.out_ld + head * p.dv;
+    if (EXTRA && p.value_gates) {
+      const __nv_bfloat16* gates = p.gate + tok_r[r] * p.gate_ld + head * p.dv;
+      uint32_t g[DV / 8];
+#pragma unroll
+      for (int i2 = 0; i2 < DV / 8; ++i2) g[i2] = i2 * 8 < p.dv ? *reinterpret_cast<const uint32_t*>(gates + i2 * 8 + tig * 2) : 0u;
+#pragma unroll
+      for (int i2 = 0; i2 < DV / 8; ++i2) {
+        oacc[i2][2 * r] = __fdividef(oacc[i2][2 * r], 1.f + __expf(-bf16_lo(g[i2])));
+        oacc[i2][2 * r + 1] = __fdividef(oacc[i2][2 * r + 1], 1.f + __expf(-bf16_hi(g[i2])));
+      }
+    }
 #pragma unroll
     for (int i2 = 0; i2 < DV / 8; ++i2) {
       const int col = i2 * 8 + tig * 2;
@@ -1191,6 +1203,7 @@ static int fill_params(const b200_attention_args* a, Params& p) {
   p.cap_in = p.cap_out = 0.f;
   p.out_scale = 1.f;
   p.gate = nullptr;
+  p.value_gates = 0;
   if (a->separate == kExtra) {
     if (a->q_ld > 0) p.q_token = a->q_ld;
     if (a->out_ld > 0) p.out_ld = a->out_ld;
@@ -1202,7 +1215,9 @@ static int fill_params(const b200_attention_args* a, Params& p) {
     if (a->maps != 2) {
       p.gate = static_cast<const __nv_bfloat16*>(a->gate);
       p.gate_ld = a->gate_ld;
-      if (p.gate && p.gate_ld < p.nq) return B200_ERR_INVALID_ARGUMENT;
+      p.value_gates = a->gate != nullptr && a->value_gates != 0;
+      if (p.gate && p.gate_ld < p.nq * (p.value_gates ? p.dv : 1)) return B200_ERR_INVALID_ARGUMENT;
+      if (p.value_gates && (p.gate_ld % 2 != 0 || reinterpret_cast<uintptr_t>(p.gate) % 4 != 0)) return B200_ERR_ALIGNMENT;
     }
     if (a->softcap > 0.f) {
       p.cap_in = scale / a->softcap;
@@ -1379,7 +1394,7 @@ int b200_paged_attention(const b200_attention_args* a, b200_stream_t stream) {
   attn::Params p;
   int rc = attn::fill_params(a, p);
   if (rc != B200_OK) return rc;
-  if (!a->out && !a->out_q) return B200_ERR_INVALID_ARGUMENT;
+  if ((!a->out && !a->out_q) || p.value_gates) return B200_ERR_INVALID_ARGUMENT;
   if (a->fuse_rope_append && (!a->token_to_chunk_idx || !a->token_to_local_pos)) return B200_ERR_INVALID_ARGUMENT;
   if (a->qkv_partials && (a->num_q_heads / a->num_kv_heads + 2) * a->head_dim % 4 != 0) return B200_ERR_ALIGNMENT;
   rc = attn::set_maps(a, p, true);

@@ -100,6 +100,7 @@ extern "C" int b200_attention_simt(const b200_attention_args* a, int dtype, b200
   const bool extra = a->separate == attn::kExtra, diff = extra && a->maps == 2;
   if (a->maps == 2 && !extra) return B200_ERR_INVALID_ARGUMENT;
   if (extra && a->distance_bias && a->bias_len < 1) return B200_ERR_INVALID_ARGUMENT;
+  if (extra && !diff && a->value_gates) return B200_ERR_INVALID_ARGUMENT;
   if (extra && !diff && a->gate && a->gate_ld < a->num_q_heads) return B200_ERR_INVALID_ARGUMENT;
   if (diff && (!a->workspace || a->workspace_bytes < static_cast<size_t>(a->num_tokens) * 2 * a->num_q_heads * a->value_dim * sizeof(float)))
     return B200_ERR_WORKSPACE;

@@ -16,23 +16,43 @@ constexpr int kThreads = 256;
 constexpr int kLanes = 8;                        // threads next to one another along the channels
 constexpr int kSegments = kThreads / kLanes;     // and along the tokens
 
-// The 32-bit model keeps to the accurate functions; otherwise the fast ones (a few ulp) in front of bf16 outputs.
-template <bool EXACT>
-__device__ __forceinline__ float sigmoid(float x) {
-  return EXACT ? 1.f / (1.f + expf(-x)) : __fdividef(1.f, 1.f + __expf(-x));
+constexpr float kLog2e = 1.4426950408889634f;
+
+// 2^x and 1/x in one instruction each (a few ulp; infinities and zeros as they should be).
+__device__ __forceinline__ float exp2_fast(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
 }
-template <bool EXACT>
-__device__ __forceinline__ float silu(float x) {
-  return EXACT ? x / (1.f + expf(-x)) : __fdividef(x, 1.f + __expf(-x));
+__device__ __forceinline__ float reciprocal_fast(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
 }
-// S -> a S + b of one token.
+
+// The arithmetic of a token.  The 32-bit model keeps to the accurate functions; otherwise the fast ones, in front of bf16 outputs.
 template <bool EXACT>
-__device__ __forceinline__ void map_of(float xz, float u, float& a, float& b) {
-  const float x = fmaxf(xz, -80.f);  // (finite exponentials; z is below 1e-34 there)
-  const float t = EXACT ? expf(-x) : __expf(-x), z = EXACT ? 1.f / (1.f + t) : __fdividef(1.f, 1.f + t);
-  a = t * z;  // 1 - z, to full accuracy also where z is nearly one
-  b = z * (u >= 0.f ? u + 0.5f : sigmoid<EXACT>(u));
-}
+struct Maths {
+  // A bias as `map` wants it.
+  static __device__ __forceinline__ float update_bias(float b) { return EXACT ? b : -b * kLog2e; }
+  // S -> a S + b, from the update gate's logit without its bias and the input with it.
+  static __device__ __forceinline__ void map(float xz, float zb, float u, float& a, float& b) {
+    float z, low;
+    if (EXACT) {
+      z = 1.f / (1.f + expf(-(xz + zb)));
+      a = 1.f / (1.f + expf(xz + zb));
+      low = 1.f / (1.f + expf(-u));
+    } else {
+      z = reciprocal_fast(1.f + exp2_fast(fmaf(xz, -kLog2e, zb)));
+      a = 1.f - z;
+      low = reciprocal_fast(1.f + exp2_fast(u * -kLog2e));
+    }
+    b = z * (u >= 0.f ? u + 0.5f : low);
+  }
+  static __device__ __forceinline__ float gated(float s, float g) {
+    return EXACT ? s * (g / (1.f + expf(-g))) : s * g * reciprocal_fast(1.f + exp2_fast(g * -kLog2e));
+  }
+};
 
 template <typename T, int VEC>
 __global__ void __launch_bounds__(kThreads)
@@ -81,21 +101,25 @@ step_kernel(b200_gated_scan_args a) {
 #pragma unroll
   for (int e = 0; e < VEC; ++e) {
     float keep, add;
-    map_of<EXACT>(x[0][e] + zb[e], x[1][e] + ub[e], keep, add);
+    Maths<EXACT>::map(x[0][e], Maths<EXACT>::update_bias(zb[e]), x[1][e] + ub[e], keep, add);
     s[e] = fmaf(keep, s[e], add);
-    y[e] = s[e] * silu<EXACT>(x[2][e]);
+    y[e] = Maths<EXACT>::gated(s[e], x[2][e]);
   }
   if (out >= 0) conv::store<float, VEC>(a.state + static_cast<int64_t>(out) * a.width + c, s);
   conv::store<T, VEC>(static_cast<T*>(a.out) + row * a.out_ld + c, y);
 }
 
+// The update logit of a token that is not there: its map leaves the state alone.
+__device__ __forceinline__ void close_gate(float& x) { x = -INFINITY; }
+__device__ __forceinline__ void close_gate(__nv_bfloat16& x) { x = __ushort_as_bfloat16(0xff80); }
+
 template <typename T, int VEC, int TOK>
 __global__ void __launch_bounds__(kThreads, 2)
 scan_kernel(b200_gated_scan_args a) {
-  constexpr bool EXACT = sizeof(T) == 4;
+  using M = Maths<sizeof(T) == 4>;
   constexpr int kTile = kSegments * TOK, kWarps = kThreads / 32;
   using V = conv::Raw<T, VEC>;
-  __shared__ float whole[2][2][kWarps][kLanes][VEC];  // [buffer][a, b]: the composed maps of the warps
+  __shared__ float whole[2][kWarps][2][kLanes * VEC];  // [buffer][warp][a, b]: the composed maps of the warps
   pdl_launch_dependents();
   const int row = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int cl = threadIdx.x % kLanes, seg = threadIdx.x / kLanes;
@@ -108,6 +132,8 @@ scan_kernel(b200_gated_scan_args a) {
     conv::load<T, VEC>(static_cast<const T*>(a.z_bias) + c, zb);
     conv::load<T, VEC>(static_cast<const T*>(a.u_bias) + c, ub);
   }
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) zb[e] = M::update_bias(zb[e]);
   pdl_wait();
   const int first = max(a.cu_tokens[row], 0), end = min(a.cu_tokens[row + 1], a.num_tokens);
   if (first >= end) return;
@@ -122,9 +148,10 @@ scan_kernel(b200_gated_scan_args a) {
   if (live && in >= 0) conv::load<float, VEC>(a.state + static_cast<int64_t>(in) * a.width + c, s);
   V raw[TOK][3];
   auto fetch = [&](int t0) {
+    const int t = t0 + seg * TOK;
 #pragma unroll
     for (int k = 0; k < TOK; ++k) {
-      const T* p = src + static_cast<int64_t>(min(t0 + seg * TOK + k, end - 1)) * a.proj_ld;
+      const T* p = src + static_cast<int64_t>(min(t + k, end - 1)) * a.proj_ld;
       raw[k][0] = *reinterpret_cast<const V*>(p + a.off_z);
       raw[k][1] = *reinterpret_cast<const V*>(p + a.off_u);
       raw[k][2] = *reinterpret_cast<const V*>(p + a.off_g);
@@ -134,7 +161,8 @@ scan_kernel(b200_gated_scan_args a) {
   int buffer = 0;
   for (int t0 = first; t0 < end; t0 += kTile, buffer ^= 1) {
     const int mine = t0 + seg * TOK;
-    float keep[TOK][VEC], add[TOK][VEC], g[TOK][VEC], A[VEC], B[VEC];
+    float keep[TOK][VEC], add[TOK][VEC], A[VEC], B[VEC];
+    V gate[TOK];
 #pragma unroll
     for (int e = 0; e < VEC; ++e) {
       A[e] = 1.f;
@@ -142,18 +170,17 @@ scan_kernel(b200_gated_scan_args a) {
     }
 #pragma unroll
     for (int k = 0; k < TOK; ++k) {
+      if (mine + k >= end) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) close_gate(raw[k][0].e[e]);
+      }
       float xz[VEC], u[VEC];
       raw[k][0].to(xz);
       raw[k][1].to(u);
-      raw[k][2].to(g[k]);
-      const bool there = mine + k < end;
+      gate[k] = raw[k][2];
 #pragma unroll
       for (int e = 0; e < VEC; ++e) {
-        map_of<EXACT>(xz[e] + zb[e], u[e] + ub[e], keep[k][e], add[k][e]);
-        if (!there) {
-          keep[k][e] = 1.f;
-          add[k][e] = 0.f;
-        }
+        M::map(xz[e], zb[e], u[e] + ub[e], keep[k][e], add[k][e]);
         A[e] *= keep[k][e];
         B[e] = fmaf(keep[k][e], B[e], add[k][e]);
       }
@@ -172,11 +199,8 @@ scan_kernel(b200_gated_scan_args a) {
       }
     }
     if (lane >= 32 - kLanes) {
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) {
-        whole[buffer][0][warp][cl][e] = A[e];
-        whole[buffer][1][warp][cl][e] = B[e];
-      }
+      conv::store<float, VEC>(&whole[buffer][warp][0][cl * VEC], A);
+      conv::store<float, VEC>(&whole[buffer][warp][1][cl * VEC], B);
     }
     float xa[VEC], xb[VEC];
 #pragma unroll
@@ -192,21 +216,25 @@ scan_kernel(b200_gated_scan_args a) {
     float start[VEC];
 #pragma unroll
     for (int w = 0; w < kWarps; ++w) {
+      float wa[VEC], wb[VEC];
+      conv::load<float, VEC>(&whole[buffer][w][0][cl * VEC], wa);
+      conv::load<float, VEC>(&whole[buffer][w][1][cl * VEC], wb);
 #pragma unroll
       for (int e = 0; e < VEC; ++e) {
         if (w == warp) start[e] = s[e];
-        s[e] = fmaf(whole[buffer][0][w][cl][e], s[e], whole[buffer][1][w][cl][e]);
+        s[e] = fmaf(wa[e], s[e], wb[e]);
       }
     }
 #pragma unroll
     for (int e = 0; e < VEC; ++e) start[e] = fmaf(xa[e], start[e], xb[e]);
 #pragma unroll
     for (int k = 0; k < TOK; ++k) {
-      float y[VEC];
+      float y[VEC], g[VEC];
+      gate[k].to(g);
 #pragma unroll
       for (int e = 0; e < VEC; ++e) {
         start[e] = fmaf(keep[k][e], start[e], add[k][e]);
-        y[e] = start[e] * silu<EXACT>(g[k][e]);
+        y[e] = M::gated(start[e], g[e]);
       }
       if (live && mine + k < end) conv::store<T, VEC>(dst + static_cast<int64_t>(mine + k) * a.out_ld, y);
     }
@@ -228,10 +256,10 @@ static int launch(const b200_gated_scan_args& a, cudaStream_t s) {
   }
   if (a.num_rows > 65535) return B200_ERR_INVALID_ARGUMENT;
   if (a.num_rows == 0) return B200_OK;
-  const int per = kLanes * (vec ? VEC : 1);
+  constexpr int SVEC = 2;
+  const int per = kLanes * (vec ? SVEC : 1);
   const dim3 grid((a.width + per - 1) / per, a.num_rows);
-  if (vec) return launch_pdl(scan_kernel<T, VEC, 4>, grid, dim3(kThreads), 0, s, a);
-  return launch_pdl(scan_kernel<T, 1, 4>, grid, dim3(kThreads), 0, s, a);
+  return vec ? launch_pdl(scan_kernel<T, SVEC, 8>, grid, dim3(kThreads), 0, s, a) : launch_pdl(scan_kernel<T, 1, 8>, grid, dim3(kThreads), 0, s, a);
 }
 
 }  // namespace gscan

@@ -83,9 +83,6 @@ __device__ __forceinline__ float apply_act(float v, int act) {
   }
   return v;
 }
-__device__ __forceinline__ float apply_gate(const Params& p, float v, int64_t m, int64_t column) {
-  return p.gate == nullptr ? v : v * __fdividef(1.f, 1.f + __expf(-__bfloat162float(p.gate[m * p.gate_ld + column])));
-}
 
 // Sum of the split-K partial tiles: y[m, n] = bf16(sum_s partial[s][m][n]) (+ bias), splits added in order
 // (deterministic).  One thread per four consecutive features; all CTAs of the grid work in parallel, which
@@ -155,7 +152,7 @@ __device__ __forceinline__ void epilogue_barrier() { asm volatile("bar.sync 2, 1
 
 // Accumulator -> output.  TMEM lane = output feature, TMEM column = token.  Either rounds to bf16 and
 // stores (whole-K units), or stores the fp32 partial tile for splitk_reduce_kernel.
-template <int BT>
+template <int BT, bool GATE = false>
 __device__ __forceinline__ void epilogue(const Params& p, uint32_t tmem_base, uint8_t* stage_smem, int n_tile, int split,
                                          int m0, int m_end, __nv_bfloat16* __restrict__ y, int64_t gate_column = 0) {
   const int tid = threadIdx.x;
@@ -243,11 +240,17 @@ __device__ __forceinline__ void epilogue(const Params& p, uint32_t tmem_base, ui
           uint32_t r[32];
           tmem_ld_32x32b_x32(lane_addr + h0 + c0, r);
           tmem_ld_wait();
+          if constexpr (GATE) {  // (all loads in flight before the first store)
+            float gate[32];
+#pragma unroll
+            for (int j = 0; j < 32; ++j) gate[j] = __bfloat162float(p.gate[min(m0 + h0 + c0 + j, m_end - 1) * p.gate_ld + gate_column + n]);
+#pragma unroll
+            for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(__fdividef(__uint_as_float(r[j]), 1.f + __expf(-gate[j])));
+          }
 #pragma unroll
           for (int j = 0; j < 32; ++j) {
             float v = __uint_as_float(r[j]);
             if (p.bias != nullptr) v = bf16_round(v) + b;  // bias is added to the bf16-rounded product
-            if (p.gate != nullptr) v = apply_gate(p, v, min(m0 + h0 + c0 + j, m_end - 1), gate_column + n);
             tile[(c0 + j) * kTileN + warp * 32 + lane] = __float2bfloat16_rn(apply_act(v, p.act));
           }
         }
@@ -267,6 +270,13 @@ __device__ __forceinline__ void epilogue(const Params& p, uint32_t tmem_base, ui
         tmem_ld_32x32b_x32(lane_addr + c0, r);
         tmem_ld_wait();
         if (n_ok) {
+          if constexpr (GATE) {
+            float gate[32];
+#pragma unroll
+            for (int j = 0; j < 32; ++j) gate[j] = __bfloat162float(p.gate[min(m0 + c0 + j, m_end - 1) * p.gate_ld + gate_column + n]);
+#pragma unroll
+            for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(__fdividef(__uint_as_float(r[j]), 1.f + __expf(-gate[j])));
+          }
 #pragma unroll
           for (int j = 0; j < 32; ++j) {
             const int m = m0 + c0 + j;
@@ -274,7 +284,7 @@ __device__ __forceinline__ void epilogue(const Params& p, uint32_t tmem_base, ui
               float v = __uint_as_float(r[j]);
               // bias is added to the bf16-rounded product, as `matmul(x, w.t()) + bias` does
               if (p.bias != nullptr) v = bf16_round(v) + b;
-              y[static_cast<int64_t>(m) * p.ldy + n] = __float2bfloat16_rn(apply_gate(p, apply_act(v, p.act), m, gate_column + n));
+              y[static_cast<int64_t>(m) * p.ldy + n] = __float2bfloat16_rn(apply_act(v, p.act));
             }
           }
         }
@@ -325,7 +335,7 @@ __device__ __forceinline__ void epilogue(const Params& p, uint32_t tmem_base, ui
   }
 }
 
-template <int BT>
+template <int BT, bool GATE>
 __global__ void __launch_bounds__(kThreads, 1)
 gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x, Params p) {
   using C = Config<BT>;
@@ -428,7 +438,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
   mbar_wait_bounded(accum_bar, 0, abort_flag, kStatusGemmTimeout);
   tcgen05_fence_after_sync();
 
-  epilogue<BT>(p, tmem_base, smem, n_tile, split, m0, p.M, p.y + batch * p.y_batch, batch * p.y_batch);
+  epilogue<BT, GATE>(p, tmem_base, smem, n_tile, split, m0, p.M, p.y + batch * p.y_batch, batch * p.y_batch);
 
   tcgen05_fence_before_sync();
   __syncthreads();
@@ -694,10 +704,16 @@ static int launch(const void* x, int64_t ldx, const void* w, const void* bias, v
     if (workspace == nullptr || workspace_bytes < need || !aligned16(workspace)) return B200_ERR_WORKSPACE;
     p.partials = static_cast<float*>(workspace);
   }
-  static std::atomic<uint64_t> smem_attr_done{0};
-  if (ensure_dynamic_smem(gemm_bf16_kernel<BT>, C::kSmemBytes, smem_attr_done) != B200_OK) return B200_ERR_LAUNCH;
+  static std::atomic<uint64_t> smem_attr_done{0}, smem_attr_done_gate{0};
   dim3 grid(n_tiles, splits, m_blocks * batch);
-  const int rc = launch_pdl(gemm_bf16_kernel<BT>, grid, dim3(kThreads), C::kSmemBytes, stream, *mw, *mx, p);
+  int rc;
+  if (gate != nullptr) {
+    if (ensure_dynamic_smem(gemm_bf16_kernel<BT, true>, C::kSmemBytes, smem_attr_done_gate) != B200_OK) return B200_ERR_LAUNCH;
+    rc = launch_pdl(gemm_bf16_kernel<BT, true>, grid, dim3(kThreads), C::kSmemBytes, stream, *mw, *mx, p);
+  } else {
+    if (ensure_dynamic_smem(gemm_bf16_kernel<BT, false>, C::kSmemBytes, smem_attr_done) != B200_OK) return B200_ERR_LAUNCH;
+    rc = launch_pdl(gemm_bf16_kernel<BT, false>, grid, dim3(kThreads), C::kSmemBytes, stream, *mw, *mx, p);
+  }
   if (rc != B200_OK || splits == 1 || p.keep_partials) return rc;
   return launch_splitk_reduce(p, stream);
 }
@@ -798,7 +814,7 @@ int b200_linear_bf16(const void* x, int64_t ldx, const void* w, void* y, int64_t
   if (batch > 1 && (x_batch <= 0 || y_batch <= 0 || (batch - 1) * static_cast<int64_t>(x_batch) + K > ldx))
     return B200_ERR_INVALID_ARGUMENT;
   if (K % 8 != 0 || ldx % 8 != 0 || x_batch % 8 != 0 || ldx < K || ldy < N) return B200_ERR_ALIGNMENT;
-  if (gate && gate_ld < (batch - 1) * y_batch + N) return B200_ERR_INVALID_ARGUMENT;
+  if (gate && (gate_ld < (batch - 1) * y_batch + N || act != B200_ACT_NONE)) return B200_ERR_INVALID_ARGUMENT;
   if (!aligned16(x) || !aligned16(w)) return B200_ERR_ALIGNMENT;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   switch (gemm::pick_bt(M)) {

@@ -67,6 +67,72 @@ __device__ __forceinline__ void rotated_pair(const b200_latent_args& a, const T*
   }
 }
 
+// Rows without a rotated part or padding: the two norms, 16 bytes a thread.
+constexpr int kNormThreads = 128;
+constexpr int kNormPieces = 4;
+template <typename T>
+__global__ void __launch_bounds__(kNormThreads)
+latent_norm_kernel(b200_latent_args a) {
+  constexpr int VEC = 16 / sizeof(T);
+  __shared__ float red[2][kNormThreads / 32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int tid = threadIdx.x;
+  const int64_t t = blockIdx.x;
+  const T* row = static_cast<const T*>(a.proj) + t * a.proj_ld;
+  const int own = a.dkv_offset >= 0 ? a.kv_rank / VEC : 0, all = own + (a.q_latent_out != nullptr ? a.q_rank / VEC : 0);
+  const int64_t chunk = own > 0 ? a.token_to_chunk_idx[t] : 0, local = own > 0 ? a.token_to_local_pos[t] : 0;
+  float v[kNormPieces][VEC], sq[2] = {0.f, 0.f};
+#pragma unroll
+  for (int i = 0; i < kNormPieces; ++i) {
+    const int p = i * kNormThreads + tid;
+    if (p >= all) continue;
+    const bool latent = p < own;
+    conv::load<T, VEC>(row + (latent ? a.dkv_offset + p * VEC : a.q_latent_offset + (p - own) * VEC), v[i]);
+    float s = 0.f;
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) s = fmaf(v[i][e], v[i][e], s);
+    sq[latent ? 0 : 1] += s;
+  }
+#pragma unroll
+  for (int n = 0; n < 2; ++n) {
+    sq[n] = warp_sum(sq[n]);
+    if ((tid & 31) == 0) red[n][tid >> 5] = sq[n];
+  }
+  __syncthreads();
+  float inv[2];
+#pragma unroll
+  for (int n = 0; n < 2; ++n) {
+    float total = 0.f;
+#pragma unroll
+    for (int i = 0; i < kNormThreads / 32; ++i) total += red[n][i];
+    inv[n] = 1.f / sqrtf(total / (n == 0 ? a.kv_rank : a.q_rank) + a.eps);
+  }
+  const bool there = chunk >= 0 && chunk < a.num_chunks && local >= 0 && local < a.chunk_size;
+  T* dst = static_cast<T*>(a.pool) + (chunk * a.chunk_size + local) * a.row_width;
+  T* q_dst = static_cast<T*>(a.q_latent_out) + t * a.q_rank;
+#pragma unroll
+  for (int i = 0; i < kNormPieces; ++i) {
+    const int p = i * kNormThreads + tid;
+    if (p >= all || (p < own && !there)) continue;
+    const bool latent = p < own;
+    const int c = (latent ? p : p - own) * VEC;
+    float g[VEC];
+    conv::load<T, VEC>(static_cast<const T*>(latent ? a.norm_weight : a.q_norm_weight) + c, g);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) v[i][e] *= inv[latent ? 0 : 1] * g[e];
+    conv::store<T, VEC>((latent ? dst : q_dst) + c, v[i]);
+  }
+}
+template <typename T>
+static bool norm_fits(const b200_latent_args& a) {
+  constexpr int VEC = 16 / sizeof(T);
+  const int own = a.dkv_offset >= 0 ? a.kv_rank : 0, q = a.q_latent_out ? a.q_rank : 0;
+  return a.rot_dim == 0 && (a.q_rot_at == 0 || a.row_width == a.kv_rank) && (own == 0 || a.row_width == a.kv_rank) && a.q != nullptr && own + q > 0 &&
+         own % VEC == 0 && q % VEC == 0 && (own + q) / VEC <= kNormPieces * kNormThreads && a.proj_ld % VEC == 0 && a.q_latent_offset % VEC == 0 &&
+         (own == 0 || a.dkv_offset % VEC == 0) && aligned16(a.proj) && aligned16(a.norm_weight) && aligned16(a.q_norm_weight) && aligned16(a.q_latent_out);
+}
+
 template <typename T>
 __global__ void __launch_bounds__(kAppendThreads)
 latent_append_kernel(b200_latent_args a) {
@@ -471,14 +537,13 @@ __device__ __forceinline__ int piece_offset(int r, int c8) {
 //   S^T [64 keys x N]           = tile (K-major, rows = keys)      x Q (K-major, rows = query rows)
 //   O^T [128 channels x 2N] (+)= tile (MN-major, the same bytes)  x P (K-major, rows = query rows: N of the weights' bf16 values,
 //                                                                      N of what that rounding left over; added at the end)
-// Warps 0-3: softmax - a thread owns a key (a 64-row accumulator sits in lanes 0-15 of each warp's part of tensor memory): it
-// reads its N scores and writes its 2N weight terms to shared memory as the B operand.  Weights are taken relative to a
+// Softmax: groups of four warps, 16 query rows a group - a thread owns a key (a 64-row accumulator sits in lanes 0-15 of each warp's
+// part of tensor memory): it reads its 16 scores and writes its 32 weight terms to shared memory as the B operand.  Weights are taken relative to a
 // reference per query row that trails the running maximum by at most kGrow (in log2): only when a score exceeds that are
-// maxima exchanged and O rescaled, which after the first tiles hardly ever happens.  Warp 4: TMA, warp 5: MMA issue.
+// maxima exchanged and O rescaled, which after the first tiles hardly ever happens.  Two more warps: TMA and MMA issue.
 // The scores of the next tile are computed before the values of the current one, so that its softmax runs beside them.
 // ---------------------------------------------------------------------------------------------------------------
 constexpr int kUmKeys = 64;
-constexpr int kUmThreads = 192;
 constexpr int kUmMaxStages = 4;
 constexpr int kSubBytes = kUmKeys * 128;
 constexpr float kGrow = 8.f;
@@ -491,6 +556,9 @@ __device__ __forceinline__ float exp2_approx(float x) {  // 2^x to fp32 accuracy
 
 template <int N>
 struct UmmaShape {
+  static constexpr int kGroups = N / 16;          // groups of four softmax warps, 16 query rows each
+  static constexpr int kSoftmax = 128 * kGroups;  // their threads
+  static constexpr int kThreads = kSoftmax + 64;
   static __host__ __device__ int subs(int row_width, int kv_pad) {
     const int s = (row_width + 63) / 64, o = (kv_pad + 127) / 128 * 2;
     return s > o ? s : o;
@@ -504,9 +572,10 @@ struct UmmaShape {
 };
 
 template <int N>
-__global__ void __launch_bounds__(kUmThreads, 1)
+__global__ void __launch_bounds__(UmmaShape<N>::kThreads, 1)
 latent_umma_kernel(const __grid_constant__ CUtensorMap map, b200_latent_args a, int stages, int tmem_cols) {
   using U = UmmaShape<N>;
+  constexpr int kTmaWarp = 4 * U::kGroups, kMmaWarp = kTmaWarp + 1;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -535,7 +604,7 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap map, b200_latent_args a, 
     }
     for (int s = 0; s < 2; ++s) {
       mbar_init(&s_full[s], 1);
-      mbar_init(&p_ready[s], 128);
+      mbar_init(&p_ready[s], U::kSoftmax);
       mbar_init(&pv_done[s], 1);
       mbar_init(&patched[s], 128);
     }
@@ -599,19 +668,19 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap map, b200_latent_args a, 
   };
   // Decode: only the newest token's row is written by this step (by the append kernel before this one); the others are there.
   int loaded = 0;
-  if (warp == 4 && lane == 0 && a.units == nullptr)
+  if (warp == kTmaWarp && lane == 0 && a.units == nullptr)
     for (; loaded < min(stages, n_tiles) && base + (loaded + 1) * kUmKeys <= last_pos; ++loaded) load(loaded);
   pdl_wait();
   // Q as a K-major operand, rows past q_rows and columns past row_width zero
   if (n_tiles > 0) {
     const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(a.q_full) + (static_cast<int64_t>(tok0) * a.heads + sub * N) * a.row_width;
-    for (int i = tid; i < subs_loaded * 8 * N; i += kUmThreads) {
+    for (int i = tid; i < subs_loaded * 8 * N; i += U::kThreads) {
       const int r = i / (subs_loaded * 8), c8 = i - r * (subs_loaded * 8);
       uint4 v = make_uint4(0, 0, 0, 0);
       if (r < q_rows && c8 * 8 < a.row_width) v = *reinterpret_cast<const uint4*>(q + static_cast<int64_t>(r) * a.row_width + c8 * 8);
       *reinterpret_cast<uint4*>(q_s + piece_offset<N>(r, c8)) = v;
     }
-    for (int n = tid; n < N; n += kUmThreads) {
+    for (int n = tid; n < N; n += U::kThreads) {
       const int pos = first_pos + (sub * N + n) / a.heads - (sub * N) / a.heads;
       hi_s[n] = n < q_rows ? min(pos, end - 1) : -1;
       lo_s[n] = max(window_start(pos, a.window), start);
@@ -621,12 +690,12 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap map, b200_latent_args a, 
   fence_proxy_async_smem();
   __syncthreads();
 
-  if (n_tiles > 0 && warp == 4) {
+  if (n_tiles > 0 && warp == kTmaWarp) {
     // ------------------------------- TMA -------------------------------
     if (lane == 0)
       for (; loaded < n_tiles; ++loaded) load(loaded);
     __syncwarp();
-  } else if (n_tiles > 0 && warp == 5) {
+  } else if (n_tiles > 0 && warp == kMmaWarp) {
     if (lane == 0) {
       // ------------------------------- MMA -------------------------------
       constexpr uint32_t idesc_s = umma_idesc_bf16(kUmKeys, N);
@@ -679,30 +748,32 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap map, b200_latent_args a, 
     __syncwarp();
   } else if (n_tiles > 0) {
     // ------------------------------- softmax -------------------------------
-    const uint32_t lanes = static_cast<uint32_t>(warp * 32) << 16;
+    const int quad = warp & 3, n_base = (warp >> 2) * 16;  // part of tensor memory; first of this warp's query rows
+    const uint32_t lanes = static_cast<uint32_t>(quad * 32) << 16;
     const float scale_log2 = a.scale * kLog2e;
     const bool owner = lane < 16;                  // this thread owns key `mine` of every tile
-    const int mine = warp * 16 + (lane & 15);
+    const int mine = quad * 16 + (lane & 15);
     // tiles whose keys every query row sees need no masks
     const int all_lo = max(window_start(last_pos, a.window), start), all_hi = min(first_pos, end - 1);
-    float l_part[N], m[N];  // sums of this thread's weights, references
+    float l_part[16], m[16];  // sums of this thread's weights, references
 #pragma unroll
-    for (int n = 0; n < N; ++n) {
+    for (int n = 0; n < 16; ++n) {
       l_part[n] = 0.f;
       m[n] = -INFINITY;
     }
-    auto group_sync = [] { asm volatile("bar.sync 1, 128;" ::: "memory"); };
+    auto group_sync = [] { asm volatile("bar.sync 1, %0;" ::"n"(U::kSoftmax) : "memory"); };
     auto group_any = [](bool p) {
       int r;
       asm volatile(
-          "{\n.reg .pred p, q;\nsetp.ne.s32 p, %1, 0;\nbarrier.red.or.pred q, 2, 128, p;\nselp.s32 %0, 1, 0, q;\n}\n"
+          "{\n.reg .pred p, q;\nsetp.ne.s32 p, %1, 0;\nbarrier.red.or.pred q, 2, %2, p;\nselp.s32 %0, 1, 0, q;\n}\n"
           : "=r"(r)
-          : "r"(static_cast<int>(p))
+          : "r"(static_cast<int>(p)), "n"(U::kSoftmax)
           : "memory");
       return r != 0;
     };
     int patches = 0, f_stage = 0, f_phase = 0;
-    auto patch = [&](int i) {  // tiles in order: clear the rows of a boundary tile that are not keys of the range
+    auto patch = [&](int i) {  // (the first group) tiles in order: clear the rows of a boundary tile that are not keys of the range
+      if (n_base > 0) return;
       const int k0 = base + i * kUmKeys;
       if (k0 < start || k0 + kUmKeys > end) {
         const int lo = max(start - k0, 0), hi = min(end - k0, kUmKeys), r = tid >> 1;
@@ -722,7 +793,7 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap map, b200_latent_args a, 
       }
     };
     // where this key's weights go: 2 bytes in row n of a buffer, its 16-byte pieces swizzled
-    const uint32_t p_addr = smem_u32(p_s) + (mine & 7) * 2;
+    const uint32_t p_addr = smem_u32(p_s) + n_base * 128 + (mine & 7) * 2;
     const int piece = mine >> 3;
     patch(0);
     for (int i = 0; i < n_tiles; ++i) {
@@ -730,33 +801,28 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap map, b200_latent_args a, 
       mbar_wait_bounded(&s_full[i & 1], (i >> 1) & 1, abort_flag, kStatusAttnTimeout);
       tcgen05_fence_after_sync();
       const int key0 = base + i * kUmKeys, key = key0 + mine;
-      uint32_t raw[N];
-#pragma unroll
-      for (int n0 = 0; n0 < N; n0 += 16)
-        tmem_ld_32x32b_x16(tmem + (i & 1) * N + n0 + lanes, *reinterpret_cast<uint32_t(*)[16]>(raw + n0));
+      uint32_t raw[16];
+      tmem_ld_32x32b_x16(tmem + (i & 1) * N + n_base + lanes, raw);
       tmem_ld_wait();
-      float x[N];
+      float x[16];
 #pragma unroll
-      for (int n = 0; n < N; ++n) x[n] = owner ? __uint_as_float(raw[n]) * scale_log2 : -INFINITY;
+      for (int n = 0; n < 16; ++n) x[n] = owner ? __uint_as_float(raw[n]) * scale_log2 : -INFINITY;
       if (key0 < all_lo || key0 + kUmKeys - 1 > all_hi) {
 #pragma unroll
-        for (int n = 0; n < N; ++n) x[n] = key >= lo_s[n] && key <= hi_s[n] ? x[n] : -INFINITY;
+        for (int n = 0; n < 16; ++n) x[n] = key >= lo_s[n_base + n] && key <= hi_s[n_base + n] ? x[n] : -INFINITY;
       }
       float over[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};  // how far a score exceeds its row's reference
 #pragma unroll
-      for (int n = 0; n < N; ++n) over[n & 3] = fmaxf(over[n & 3], x[n] - m[n]);  // (-inf less -inf: NaN, which fmaxf drops)
+      for (int n = 0; n < 16; ++n) over[n & 3] = fmaxf(over[n & 3], x[n] - m[n]);  // (-inf less -inf: NaN, which fmaxf drops)
       if (group_any(fmaxf(fmaxf(over[0], over[1]), fmaxf(over[2], over[3])) > kGrow)) {
         // New references: the column maxima cross the warp by redux and the warps through shared memory.
+        float best = -INFINITY;
 #pragma unroll
-        for (int n0 = 0; n0 < N; n0 += 32) {
-          float best = -INFINITY;
-#pragma unroll
-          for (int n = 0; n < (N < 32 ? N : 32); ++n) {
-            const float c = warp_redux_max(x[n0 + n]);
-            if (lane == n) best = c;
-          }
-          if (N >= 32 || lane < N) red[warp * N + n0 + lane] = best;
+        for (int n = 0; n < 16; ++n) {
+          const float c = warp_redux_max(x[n]);
+          if (lane == n) best = c;
         }
+        if (lane < 16) red[quad * N + n_base + lane] = best;
         group_sync();
         if (tid < N) {
           const float m_old = m_s[tid];
@@ -769,20 +835,20 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap map, b200_latent_args a, 
           mbar_wait_bounded(&pv_done[(i - 1) & 1], ((i - 1) >> 1) & 1, abort_flag, kStatusAttnTimeout);  // O is at rest
           tcgen05_fence_after_sync();
 #pragma unroll 1
-          for (int c = 0; c < m_tiles * 2 * N; c += 16) {
+          for (int c = n_base; c < m_tiles * 2 * N; c += N) {
             uint32_t r[16];
             tmem_ld_32x32b_x16(tmem_o + c + lanes, r);
             tmem_ld_wait();
 #pragma unroll
-            for (int n = 0; n < 16; ++n) r[n] = __float_as_uint(__uint_as_float(r[n]) * al_s[(c & (N - 1)) + n]);
+            for (int n = 0; n < 16; ++n) r[n] = __float_as_uint(__uint_as_float(r[n]) * al_s[n_base + n]);
             tmem_st_32x32b_x16(tmem_o + c + lanes, r);
           }
           tmem_st_wait();
         }
 #pragma unroll
-        for (int n = 0; n < N; ++n) {
-          l_part[n] *= al_s[n];
-          m[n] = m_s[n];
+        for (int n = 0; n < 16; ++n) {
+          l_part[n] *= al_s[n_base + n];
+          m[n] = m_s[n_base + n];
         }
       }
       // this key's weights: two bf16 terms each, into rows n and N + n
@@ -790,7 +856,7 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap map, b200_latent_args a, 
       if (owner) {
         const uint32_t dst = p_addr + (i & 1) * U::kPBytes;
 #pragma unroll
-        for (int n = 0; n < N; ++n) {
+        for (int n = 0; n < 16; ++n) {
           const float p = exp2_approx(fmaxf(x[n] - m[n], -1000.f));  // (a row without a key so far: NaN -> 0)
           l_part[n] += p;
           const __nv_bfloat16 hi = __float2bfloat16_rn(p), lo = __float2bfloat16_rn(p - __bfloat162float(hi));
@@ -805,16 +871,13 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap map, b200_latent_args a, 
       if (stages == 1 && i + 1 < n_tiles) patch(i + 1);
     }
     // ---- row sums, output factors, output ----
+    float best = 0.f;
 #pragma unroll
-    for (int n0 = 0; n0 < N; n0 += 32) {
-      float best = 0.f;
-#pragma unroll
-      for (int n = 0; n < (N < 32 ? N : 32); ++n) {
-        const float l = warp_sum(l_part[n0 + n]);
-        if (lane == n) best = l;
-      }
-      if (N >= 32 || lane < N) red[warp * N + n0 + lane] = best;
+    for (int n = 0; n < 16; ++n) {
+      const float l = warp_sum(l_part[n]);
+      if (lane == n) best = l;
     }
+    if (lane < 16) red[quad * N + n_base + lane] = best;
     group_sync();
     const int64_t pair0 = static_cast<int64_t>(tok0) * a.heads + sub * N;  // token * heads + head of row 0
     if (tid < q_rows) {
@@ -835,25 +898,22 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap map, b200_latent_args a, 
     tcgen05_fence_after_sync();
 #pragma unroll 1
     for (int j = 0; j < m_tiles; ++j) {
-      const int ch = j * 128 + tid;
-#pragma unroll 1
-      for (int n0 = 0; n0 < N; n0 += 16) {
-        if (n0 >= q_rows) break;
-        uint32_t r[16], q[16];
-        tmem_ld_32x32b_x16(tmem_o + j * 2 * N + n0 + lanes, r);
-        tmem_ld_32x32b_x16(tmem_o + j * 2 * N + N + n0 + lanes, q);
-        tmem_ld_wait();
-        if (ch < a.kv_rank) {
+      const int ch = j * 128 + quad * 32 + lane;
+      if (n_base >= q_rows) break;
+      uint32_t r[16], q[16];
+      tmem_ld_32x32b_x16(tmem_o + j * 2 * N + n_base + lanes, r);
+      tmem_ld_32x32b_x16(tmem_o + j * 2 * N + N + n_base + lanes, q);
+      tmem_ld_wait();
+      if (ch < a.kv_rank) {
 #pragma unroll
-          for (int n = 0; n < 16; ++n) {
-            if (n0 + n >= q_rows) break;
-            const float o = (__uint_as_float(r[n]) + __uint_as_float(q[n])) * al_s[n0 + n];
-            const int64_t pair = pair0 + n0 + n;
-            if (a.num_splits > 1)
-              a.workspace[(pair * a.num_splits + split) * a.kv_rank + ch] = o;
-            else
-              static_cast<__nv_bfloat16*>(a.out)[pair * a.kv_rank + ch] = __float2bfloat16_rn(o);
-          }
+        for (int n = 0; n < 16; ++n) {
+          if (n_base + n >= q_rows) break;
+          const float o = (__uint_as_float(r[n]) + __uint_as_float(q[n])) * al_s[n_base + n];
+          const int64_t pair = pair0 + n_base + n;
+          if (a.num_splits > 1)
+            a.workspace[(pair * a.num_splits + split) * a.kv_rank + ch] = o;
+          else
+            static_cast<__nv_bfloat16*>(a.out)[pair * a.kv_rank + ch] = __float2bfloat16_rn(o);
         }
       }
     }
@@ -905,7 +965,9 @@ latent_gather_kernel(b200_latent_args a) {
     const int mid = (lo + hi + 1) >> 1;
     if (a.cu_keys[mid] <= e) lo = mid; else hi = mid - 1;
   }
-  const int key = a.key_start[lo] + e - a.cu_keys[lo];
+  int key = a.key_start[lo] + e - a.cu_keys[lo];
+  if (a.key_end != nullptr) key = min(key, a.key_end[lo] - 1);
+  if (key < 0) return;
   const int32_t* bt = a.block_table + static_cast<int64_t>(lo) * a.max_chunks_per_row;
   const uint4* src = reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(a.pool) + pool_row(a, bt, key) * a.row_width);
   uint4* dst = reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(a.key_rows) + static_cast<int64_t>(e) * a.row_width);
@@ -1242,7 +1304,7 @@ static int launch_umma(const b200_latent_args& a, cudaStream_t s) {
   if (ensure_dynamic_smem(latent_umma_kernel<N>, kMaxSmem, done) != B200_OK) return B200_ERR_LAUNCH;
   const int q_tokens = a.units ? a.unit_tokens : 1;
   const dim3 grid(a.units ? a.num_units : a.num_tokens, (q_tokens * a.heads + N - 1) / N, a.num_splits);
-  const int rc = launch_pdl(latent_umma_kernel<N>, grid, dim3(kUmThreads), UmmaShape<N>::bytes(a.row_width, a.kv_pad, stages), s, *map,
+  const int rc = launch_pdl(latent_umma_kernel<N>, grid, dim3(UmmaShape<N>::kThreads), UmmaShape<N>::bytes(a.row_width, a.kv_pad, stages), s, *map,
                             a, stages, cols);
   if (rc != B200_OK || a.num_splits == 1) return rc;
   return launch_pdl(latent_combine_kernel, dim3(a.num_tokens * a.heads), dim3(128), 0, s, a);
@@ -1299,6 +1361,10 @@ int b200_latent_append(const b200_latent_args* a, b200_stream_t stream) {
   if (a->q && a->q_ld < static_cast<int64_t>(a->heads) * (a->dim + a->rot_dim)) return B200_ERR_INVALID_ARGUMENT;
   if (a->dkv_offset >= 0 && (!a->norm_weight || !a->token_to_chunk_idx || !a->token_to_local_pos)) return B200_ERR_INVALID_ARGUMENT;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (a->dtype == B200_DTYPE_F32 && latent::norm_fits<float>(*a))
+    return launch_pdl(latent::latent_norm_kernel<float>, dim3(a->num_tokens), dim3(latent::kNormThreads), 0, s, *a);
+  if (a->dtype == B200_DTYPE_BF16 && latent::norm_fits<__nv_bfloat16>(*a))
+    return launch_pdl(latent::latent_norm_kernel<__nv_bfloat16>, dim3(a->num_tokens), dim3(latent::kNormThreads), 0, s, *a);
   if (a->dtype == B200_DTYPE_F32)
     return launch_pdl(latent::latent_append_kernel<float>, dim3(a->num_tokens), dim3(latent::kAppendThreads), 0, s, *a);
   return launch_pdl(latent::latent_append_kernel<__nv_bfloat16>, dim3(a->num_tokens), dim3(latent::kAppendThreads), 0, s, *a);

@@ -6,7 +6,6 @@
 namespace b200 {
 namespace resnorm {
 
-constexpr int kThreads = 256;
 constexpr int kMaxTop = 64;
 
 template <typename T, int VEC>
@@ -39,7 +38,7 @@ __device__ __forceinline__ float as_stored(float x) {
 }
 
 // SLOTS * VEC * kThreads >= width: the row lives in registers.
-template <typename T, int VEC, int SLOTS>
+template <typename T, int VEC, int SLOTS, int kThreads>
 __global__ void __launch_bounds__(kThreads)
 residual_norm_kernel(b200_residual_norm_args a) {
   __shared__ float red[kThreads / 32];
@@ -47,6 +46,13 @@ residual_norm_kernel(b200_residual_norm_args a) {
   __shared__ float expert_weight[kMaxTop];
   pdl_launch_dependents();
   const int tid = threadIdx.x, W = a.width;
+  if (a.taps > 0) {  // the filters' weights, on their way while the kernel before ends
+    const int pieces = (a.taps * W * static_cast<int>(sizeof(T)) + 127) / 128;
+    for (int n = 0; n < 2; ++n)
+      if (a.filter[n] != nullptr)
+        for (int i = blockIdx.x * kThreads + tid; i < pieces; i += gridDim.x * kThreads)
+          asm volatile("prefetch.global.L2 [%0];" ::"l"(static_cast<const char*>(a.filter[n]) + i * 128));
+  }
   pdl_wait();
   const int64_t row = a.row_index ? a.row_index[blockIdx.x] : blockIdx.x;
   const bool ok = row >= 0 && row < a.source_rows;
@@ -204,17 +210,22 @@ static int launch(const b200_residual_norm_args& a, cudaStream_t s) {
                         static_cast<const void*>(a.hidden), a.gamma[0], a.gamma[1], static_cast<const void*>(a.y[0]),
                         static_cast<const void*>(a.y[1]), a.filter[0], a.filter[1], static_cast<const void*>(a.state)})
     aligned = aligned && aligned16(p);
-  const dim3 grid(a.rows), block(kThreads);
+  const dim3 grid(a.rows), block(256);
+  if (aligned && a.rows <= 2 * sm_count()) {  // few rows: more threads for each
+    if (a.width > 2048 && a.width <= 4096) return launch_pdl(residual_norm_kernel<T, 4, 1, 1024>, grid, dim3(1024), 0, s, a);
+    if (a.width > 4096 && a.width <= 8192) return launch_pdl(residual_norm_kernel<T, 4, 2, 1024>, grid, dim3(1024), 0, s, a);
+    if (a.width > 1024 && a.width <= 2048) return launch_pdl(residual_norm_kernel<T, 4, 1, 512>, grid, dim3(512), 0, s, a);
+  }
   if (aligned) {
-    if (a.width <= 1024) return launch_pdl(residual_norm_kernel<T, 4, 1>, grid, block, 0, s, a);
-    if (a.width <= 2048) return launch_pdl(residual_norm_kernel<T, 4, 2>, grid, block, 0, s, a);
-    if (a.width <= 4096) return launch_pdl(residual_norm_kernel<T, 4, 4>, grid, block, 0, s, a);
-    if (a.width <= 8192) return launch_pdl(residual_norm_kernel<T, 4, 8>, grid, block, 0, s, a);
-    if (a.width <= 16384) return launch_pdl(residual_norm_kernel<T, 4, 16>, grid, block, 0, s, a);
+    if (a.width <= 1024) return launch_pdl(residual_norm_kernel<T, 4, 1, 256>, grid, block, 0, s, a);
+    if (a.width <= 2048) return launch_pdl(residual_norm_kernel<T, 4, 2, 256>, grid, block, 0, s, a);
+    if (a.width <= 4096) return launch_pdl(residual_norm_kernel<T, 4, 4, 256>, grid, block, 0, s, a);
+    if (a.width <= 8192) return launch_pdl(residual_norm_kernel<T, 4, 8, 256>, grid, block, 0, s, a);
+    if (a.width <= 16384) return launch_pdl(residual_norm_kernel<T, 4, 16, 256>, grid, block, 0, s, a);
     return B200_ERR_INVALID_ARGUMENT;
   }
-  if (a.width <= 1024) return launch_pdl(residual_norm_kernel<T, 1, 4>, grid, block, 0, s, a);
-  if (a.width <= 16384) return launch_pdl(residual_norm_kernel<T, 1, 64>, grid, block, 0, s, a);
+  if (a.width <= 1024) return launch_pdl(residual_norm_kernel<T, 1, 4, 256>, grid, block, 0, s, a);
+  if (a.width <= 16384) return launch_pdl(residual_norm_kernel<T, 1, 64, 256>, grid, block, 0, s, a);
   return B200_ERR_INVALID_ARGUMENT;
 }
 

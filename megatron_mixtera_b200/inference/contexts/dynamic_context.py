@@ -515,13 +515,18 @@ class DynamicInferenceContext(BaseInferenceContext):
 
     token_rows = latent_cache
 
-    def expanded_keys(self, window: Optional[int]):
+    def expanded_keys(self, window: Optional[int], whole_chunks: int = 0):
         """For attention that spells out the keys of a prompt step: which keys the step's queries see under ``window``.
         Returns (device int32 ``[2, rows + 1]`` = cumulative key counts, position of a row's first key; total) or None where
-        that does not pay - decode steps, CUDA-graph steps, or more than twice as many keys as query tokens."""
+        that does not pay - decode steps, CUDA-graph steps, or more than twice as many keys as query tokens.
+
+        ``whole_chunks`` > 0 (without a window): every row's keys fill whole chunks of that many; a third row of the table holds the position
+        behind a row's last key, and a block table ``[rows, chunks]`` over the expanded keys comes as third result."""
         if self.is_decode_only() or self.using_cuda_graph_this_step():
             return None
-        if window not in self._expanded:
+        assert window is None or not whole_chunks
+        which = (window, whole_chunks)
+        if which not in self._expanded:
             p, t = self.paused_request_count, self.total_request_count
             ql = self.request_query_lengths.numpy()[p:t].astype(np.int64)
             off = self.request_kv_length_offsets.numpy()[p:t].astype(np.int64)
@@ -529,15 +534,28 @@ class DynamicInferenceContext(BaseInferenceContext):
             counts = off + ql - first
             total = int(counts.sum())
             if total > 2 * int(ql.sum()):
-                self._expanded[window] = None
+                self._expanded[which] = None
             else:
-                table = torch.zeros((2, ql.size + 1), dtype=torch.int32, pin_memory=self.device.type == "cuda")
-                table[0, 1:] = torch.from_numpy(np.cumsum(counts))
-                table[1, :-1] = torch.from_numpy(first)
+                rows, chunks = ql.size, 0
+                if whole_chunks:
+                    filled = -(-counts // whole_chunks)
+                    chunks, total = int(filled.max()), int(filled.sum()) * whole_chunks
+                table = torch.zeros(3 * (rows + 1) + rows * chunks, dtype=torch.int32, pin_memory=self.device.type == "cuda")
+                head = table[: 3 * (rows + 1)].view(3, rows + 1)
+                head[0, 1:] = torch.from_numpy(np.cumsum(filled * whole_chunks if whole_chunks else counts))
+                head[1, :-1] = torch.from_numpy(first)
+                head[2, :-1] = torch.from_numpy(first + counts)
+                if whole_chunks:
+                    starts = np.cumsum(filled) - filled
+                    table[3 * (rows + 1):].view(rows, chunks)[:] = torch.from_numpy(starts[:, None] + np.minimum(np.arange(chunks)[None], filled[:, None] - 1))
                 self.h2d_bytes += table.numel() * 4
-                self._expanded[window] = (table.to(self.device, non_blocking=True), total, table)  # (the staging copy lives as long)
-        entry = self._expanded[window]
-        return None if entry is None else entry[:2]
+                device = table.to(self.device, non_blocking=True)
+                entry = (device[: 3 * (rows + 1)].view(3, rows + 1), total, device[3 * (rows + 1):].view(rows, chunks) if whole_chunks else None)
+                self._expanded[which] = (entry, table)  # (the staging copy lives as long)
+        entry = self._expanded[which]
+        if entry is None:
+            return None
+        return entry[0] if whole_chunks else entry[0][:2]
 
     def key_value_cache(self, layer_number: int) -> Tuple[Tensor, Tensor, Tensor]:
         """(K pool, V pool, block table) of 1-based ``layer_number`` (reference :547-564)."""

@@ -12,6 +12,7 @@ import torch
 from .. import _lib, ops
 from ..tensor_parallel.layers import ColumnParallelLinear, RowParallelLinear, _device
 from .attention import _sm_count
+from .grouped_attention import EXTRA
 from .hybrid_config import HybridConfig, LatentAttentionConfig
 
 
@@ -109,15 +110,42 @@ class LatentAttention(torch.nn.Module):
 
     expand_prompts = True  # False: the absorbed form everywhere
 
-    def prefill_unit_tokens(self) -> int:
-        """Tokens per work unit of the absorbed prompt kernel (it cuts a unit into blocks of query rows itself)."""
-        return 16
+    UNIT_TOKENS = 16   # per work unit of the absorbed prompt kernel (it cuts a unit into blocks of query rows itself)
+    BLOCK_TOKENS = 64  # queries, and keys of a chunk, of the prompt kernel of grouped attention
+
+    @property
+    def prompts_as_grouped(self) -> bool:
+        """Whether expanded keys and values are an ordinary pool to the prompt kernel of grouped attention: nothing rotated beside them."""
+        m = self.mixer
+        return (self.config.params_dtype == torch.bfloat16 and m.rot_dim == 0 and m.window is None and m.dim % 8 == 0 and m.vdim % 8 == 0
+                and max(m.dim, m.vdim) <= 128 and m.q_rank is not None)
+
+    def prefill_unit_tokens(self) -> set:
+        """Tokens per work unit of the prompt kernels."""
+        return {self.UNIT_TOKENS} | ({self.BLOCK_TOKENS} if self.prompts_as_grouped else set())
 
     def _expansion(self, x, ctx):
         m = self.mixer
         if not (self.expand_prompts and x.dtype == torch.bfloat16 and ops.latent_prompt_supported(m.dim, m.rot_dim, m.vdim, m.heads)):
             return None
-        return ctx.expanded_keys(m.window)
+        return ctx.expanded_keys(m.window, self.BLOCK_TOKENS if self.prompts_as_grouped else 0)
+
+    def _attend_grouped(self, queries, key_values, block_table, proj, out, ctx) -> None:
+        """Attention of a prompt step over its expanded rows [keys of all heads | values of all heads] in whole chunks."""
+        m = self.mixer
+        a = _lib.AttentionArgs()
+        a.separate, a.softmax_scale, a.out_scale = EXTRA, m.scale, 1.0
+        a.qkv, a.q_ld, a.out, a.out_ld = queries.data_ptr(), queries.stride(0), out.data_ptr(), out.stride(0)
+        a.k_cache, a.v_cache = key_values.data_ptr(), key_values.data_ptr() + m.heads * m.dim * key_values.element_size()
+        a.pool_row_elems, a.num_chunks, a.chunk_size = key_values.stride(0), key_values.shape[0] // self.BLOCK_TOKENS, self.BLOCK_TOKENS
+        a.block_table, a.max_chunks_per_row = block_table.data_ptr(), block_table.shape[1]
+        a.num_tokens, a.num_q_heads, a.num_kv_heads, a.head_dim, a.value_dim = queries.shape[0], m.heads, m.heads, m.dim, m.vdim
+        a.num_splits, a.kv_seq_lengths, a.row_of_token = 1, ctx.token_kv_lengths.data_ptr(), ctx.token_to_block_table_row.data_ptr()
+        a.sinks = None if self.sinks is None else self.sinks.data_ptr()
+        a.gate, a.gate_ld = proj.data_ptr() + self.gate_offset * proj.element_size(), proj.stride(0)
+        a.value_gates, a._anchor = int(m.gate == "value"), key_values
+        units, count = ctx.prefill_units_of(self.BLOCK_TOKENS)
+        ops.separate_attention(a, queries.dtype, units=units, num_units=count, tensor_cores=True)
 
     def forward(self, x, ctx, rope=None, step=None):
         """``x`` [T, H] -> the output linear's partial sums."""
@@ -157,7 +185,7 @@ class LatentAttention(torch.nn.Module):
             queries = torch.empty((T, self.query_width), dtype=x.dtype, device=dev)
             a.q, a.q_ld = queries.data_ptr(), queries.stride(0)
         if expanded is not None:
-            table, num_keys = expanded
+            table, num_keys = expanded[:2]
             key_rows = torch.empty((num_keys, m.row_width), dtype=x.dtype, device=dev)
             ops.latent_append(a, pool)
             if m.q_rank is not None:
@@ -166,8 +194,12 @@ class LatentAttention(torch.nn.Module):
             a.value_gates = int(m.gate == "value")
             a.cu_tokens = ctx.cu_query_seq_lengths_cudagraph_only.data_ptr()
             a.cu_keys, a.key_start, a.key_rows = table[0].data_ptr(), table[1].data_ptr(), key_rows.data_ptr()
+            a.key_end = table[2].data_ptr()
             ops.latent_gather(a, pool)
             key_values = ops.linear(key_rows, self.key_value_up, K=m.kv_rank)
+            if self.prompts_as_grouped:
+                self._attend_grouped(queries, key_values, expanded[2], proj, values, ctx)
+                return self.linear_proj(values, defer_reduction=True)[0]
             a.key_values, a.out = key_values.data_ptr(), values.data_ptr()
             ops.latent_prompt_attention(a, pool)
             return self.linear_proj(values, defer_reduction=True)[0]
@@ -178,7 +210,7 @@ class LatentAttention(torch.nn.Module):
             if x.dtype == torch.bfloat16:
                 a.num_splits = choose_latent_splits(T, m.heads, m.window, ctx.max_sequence_length)
         else:
-            a.unit_tokens = self.prefill_unit_tokens()
+            a.unit_tokens = self.UNIT_TOKENS
             units, a.num_units = ctx.prefill_units_of(a.unit_tokens)
             a.units = units.data_ptr()
         if m.q_rank is not None:

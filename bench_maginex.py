@@ -53,7 +53,9 @@ def label(name, args):
     from megatron_mixtera_b200 import _lib, ops
 
     if name == "attention":
-        return "window_decode" if args[2] == 1 else "window_prompt", None
+        a = _lib.AttentionArgs.from_buffer_copy(args[0].numpy().tobytes())
+        if a.separate == 2:
+            return ("latent_prompt" if a.value_gates else "window_decode" if args[2] == 1 else "window_prompt"), None
     if name == "hybrid":
         kernel = (Z.HYBRID + tuple(ops._STRUCT_KERNELS))[args[2]]
         if kernel == "residual_norm":
@@ -77,7 +79,7 @@ def costs(s, T, visible_pairs, keys, design, decode, requests):
         out["window_" + k] = (2.0 * keys * G * 2 * a + 4.0 * T * H * a, 4.0 * visible_pairs * H * a, 0)
     out["latent_append"] = (4.0 * T * (s["q_rank"] + rank), 0, 0)
     out["latent_attention"] = (2.0 * (keys * r + T * H * (r + rank)), 2.0 * visible_pairs * H * (r + rank), 0)
-    out["latent_prompt_attention"] = (2.0 * (keys * H * 2 * d + T * H * 3 * d), 4.0 * visible_pairs * H * d, 0)
+    out["latent_prompt"] = (2.0 * (keys * H * 2 * d + T * H * 3 * d), 4.0 * visible_pairs * H * d, 0)
     out["latent_gather"] = (4.0 * keys * r, 0, 0)
     out["gated_scan"] = (T * n * ((12.0 if decode else 6.0) + 2) + 8.0 * requests * n, 0, 0)
     used, f, g = min(s["experts"], pairs), s["ff"], s["shared"]

@@ -595,6 +595,8 @@ typedef struct b200_latent_args {
  *   it where the expansion serves many queries.  bf16; dim, vdim, rot_dim multiples of 8, dim and rot_dim rounded up to 16 at
  *   most 192 together, vdim at most 128 (b200_latent_prompt_supported). */
 size_t b200_latent_attention_workspace_bytes(int num_tokens, int heads, int kv_rank, int num_splits);
+/* CTAs per row and key split of a bf16 decode step. */
+int b200_latent_decode_blocks(int heads, int kv_rank, int row_width, int chunk_size);
 int b200_latent_append(const b200_latent_args* args, b200_stream_t stream);
 int b200_latent_attention(const b200_latent_args* args, b200_stream_t stream);
 int b200_latent_prompt_supported(int dim, int rot_dim, int vdim, int heads);

@@ -79,6 +79,7 @@ EXPORTED_SYMBOLS = (
     "b200_linear_simt",
     "b200_out_norm",
     "b200_latent_attention_workspace_bytes",
+    "b200_latent_decode_blocks",
     "b200_latent_append",
     "b200_latent_attention",
     "b200_latent_prompt_supported",
@@ -448,6 +449,7 @@ def load() -> ctypes.CDLL:
     lib.b200_out_norm.argtypes = [POINTER(OutNormArgs), c_void_p]
     lib.b200_latent_attention_workspace_bytes.restype = c_size_t
     lib.b200_latent_attention_workspace_bytes.argtypes = [c_int, c_int, c_int, c_int]
+    lib.b200_latent_decode_blocks.argtypes = [c_int, c_int, c_int, c_int]
     lib.b200_latent_prompt_supported.argtypes = [c_int, c_int, c_int, c_int]
     for name in ("b200_latent_append", "b200_latent_attention", "b200_latent_gather", "b200_latent_prompt_attention"):
         getattr(lib, name).argtypes = [POINTER(LatentArgs), c_void_p]

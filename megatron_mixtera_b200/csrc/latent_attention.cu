@@ -604,7 +604,7 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap map, b200_latent_args a, 
     }
     for (int s = 0; s < 2; ++s) {
       mbar_init(&s_full[s], 1);
-      mbar_init(&p_ready[s], U::kSoftmax);
+      mbar_init(&p_ready[s], U::kSoftmax / 32);
       mbar_init(&pv_done[s], 1);
       mbar_init(&patched[s], 128);
     }
@@ -867,7 +867,8 @@ latent_umma_kernel(const __grid_constant__ CUtensorMap map, b200_latent_args a, 
       }
       fence_proxy_async_smem();
       tcgen05_fence_before_sync();
-      mbar_arrive(&p_ready[i & 1]);
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&p_ready[i & 1]);
       if (stages == 1 && i + 1 < n_tiles) patch(i + 1);
     }
     // ---- row sums, output factors, output ----
@@ -1347,6 +1348,21 @@ extern "C" {
 size_t b200_latent_attention_workspace_bytes(int num_tokens, int heads, int kv_rank, int num_splits) {
   if (num_tokens <= 0 || heads <= 0 || kv_rank <= 0 || num_splits <= 1) return 0;
   return static_cast<size_t>(num_tokens) * heads * num_splits * (static_cast<size_t>(kv_rank) + 1) * sizeof(float);
+}
+
+int b200_latent_decode_blocks(int heads, int kv_rank, int row_width, int chunk_size) {
+  using namespace b200::latent;
+  if (heads <= 0 || kv_rank <= 0 || row_width <= 0 || chunk_size <= 0) return 0;
+  b200_latent_args a{};
+  a.heads = heads;
+  a.kv_rank = kv_rank;
+  a.kv_pad = (kv_rank + 15) / 16 * 16;
+  a.row_width = row_width;
+  a.chunk_size = chunk_size;
+  if (decode_fits<256>(a) || decode_fits<512>(a)) return 1;
+  if (heads > 32 && umma_stages<64>(a) > 1) return (heads + 63) / 64;
+  if (heads > 16 && umma_stages<32>(a) > 1) return (heads + 31) / 32;
+  return (heads + 15) / 16;
 }
 
 int b200_latent_append(const b200_latent_args* a, b200_stream_t stream) {

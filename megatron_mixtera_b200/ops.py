@@ -847,6 +847,11 @@ def latent_prompt_supported(dim: int, rot_dim: int, vdim: int, heads: int) -> bo
     return bool(_lib.load().b200_latent_prompt_supported(dim, rot_dim, vdim, heads))
 
 
+def latent_decode_blocks(heads: int, kv_rank: int, row_width: int, chunk_size: int) -> int:
+    """CTAs per row and key split of a decode step."""
+    return _lib.load().b200_latent_decode_blocks(heads, kv_rank, row_width, chunk_size)
+
+
 def latent_gather(args, anchor) -> None:
     _launch("hybrid", _blob(args), anchor, _LATENT_GATHER)
 

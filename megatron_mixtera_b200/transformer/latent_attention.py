@@ -16,11 +16,11 @@ from .grouped_attention import EXTRA
 from .hybrid_config import HybridConfig, LatentAttentionConfig
 
 
-def choose_latent_splits(num_rows: int, heads: int, window, max_sequence_length: int) -> int:
-    """Key splits of a decode row: a function of capture-time constants.  The fewest splits that fill the CTAs the GPU holds
-    at once to 85 % (else the best there is), none below 256 keys at the longest visible range."""
+def choose_latent_splits(num_rows: int, heads: int, window, max_sequence_length: int, blocks_per_row: int) -> int:
+    """Key splits of a decode row, each of them ``blocks_per_row`` CTAs: a function of capture-time constants.  The fewest splits that
+    fill the CTAs the GPU holds at once to 85 % (else the best there is), none below 256 keys at the longest visible range."""
     slots = _sm_count() * (2 if heads <= 16 else 1)
-    blocks = max(1, num_rows * (1 if heads <= 32 else -(-heads // 32)))
+    blocks = max(1, num_rows * blocks_per_row)
     keys = max_sequence_length if window is None else min(window, max_sequence_length)
     best, best_fill = 1, 0.0
     for splits in range(1, max(1, min(keys // 256, 64)) + 1):
@@ -208,7 +208,8 @@ class LatentAttention(torch.nn.Module):
         if decode:
             a.kv_seq_lengths = ctx.kv_seq_lengths_cudagraph_only.data_ptr()
             if x.dtype == torch.bfloat16:
-                a.num_splits = choose_latent_splits(T, m.heads, m.window, ctx.max_sequence_length)
+                a.num_splits = choose_latent_splits(T, m.heads, m.window, ctx.max_sequence_length,
+                                                    ops.latent_decode_blocks(m.heads, m.kv_rank, m.row_width, pool.shape[1]))
         else:
             a.unit_tokens = self.UNIT_TOKENS
             units, a.num_units = ctx.prefill_units_of(a.unit_tokens)

@@ -36,7 +36,7 @@ def test_ops_module_calls_the_torch_ops(b200_ops):
     src = inspect.getsource(ops)
     direct = set(re.findall(r"\.(b200_[a-z0-9_]+)\(", src))
     allowed_suffixes = ("_bytes", "_supported")
-    allowed = {"b200_device_status", "b200_set_wait_limit_ns", "b200_copy_rows_h2d", "b200_fp8_value_position"}
+    allowed = {"b200_device_status", "b200_set_wait_limit_ns", "b200_copy_rows_h2d", "b200_fp8_value_position", "b200_latent_decode_blocks"}
     assert all(name in allowed or name.endswith(allowed_suffixes) for name in direct), direct
 
 
